@@ -1,0 +1,352 @@
+// fp32 residual stream of models whose layers read one scalar-gain RMS norm through short causal
+// depthwise convolutions: embedding + learned position, residual add + norm + convolutions, exact
+// gelu. The convolution of a row needs the normalised rows ahead of it; a CTA recomputes the few
+// rows ahead of its block from the residual instead of reading another CTA's output, so one pass
+// over the rows is enough and the residual goes to a second buffer.
+#include "common.cuh"
+
+using namespace msgl;
+
+namespace {
+
+template <typename T>
+__global__ void __launch_bounds__(256) embed_positions_kernel(const int32_t* __restrict__ ids, const T* __restrict__ w,
+                                                              const T* __restrict__ pos,
+                                                              const int32_t* __restrict__ positions,
+                                                              float* __restrict__ out, int width, int start, int len,
+                                                              int n_pos) {
+  pdl_enter();
+  const int t = blockIdx.x;
+  const int id = ids[t] - start;
+  const bool in = id >= 0 && id < len;
+  int p = pos != nullptr ? positions[t] : 0;
+  const bool has_pos = pos != nullptr && !MSGL_OOB(p, n_pos) && p >= 0 && p < n_pos;
+  for (int c = threadIdx.x; c < width; c += 256) {
+    float v = in ? to_float(w[(size_t)id * width + c]) : 0.f;
+    if (has_pos) v += to_float(pos[(size_t)p * width + c]);
+    out[(size_t)t * width + c] = v;
+  }
+}
+
+struct NormConvArgs {
+  const float* x;         // [rows, width] residual
+  float* x_out;           // residual + delta (may equal x when there is no delta)
+  const float* delta;     // [planes][rows][ldd], summed in ascending order
+  int planes;
+  long long plane_stride, ldd;
+  const float* gain;
+  float eps;
+  const float* w1;        // [width, taps] or null
+  const float* w2;
+  void* y1;               // [rows, cols]
+  void* y2;
+  float* state;           // [slots, width, taps - 1]
+  const int32_t* cu_q;
+  const int32_t* slots;
+  const int32_t* has_state;
+  int rows, width, cols, taps, block_rows;
+};
+
+// V consecutive channels per thread, NC such groups; MT >= taps: the filter is right-aligned in MT taps.
+template <typename T, int V, int NC, int MT>
+__global__ void __launch_bounds__(1024) norm_conv_kernel(const NormConvArgs a) {
+  pdl_enter();
+  __shared__ float red[2][32];
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, n_warps = blockDim.x >> 5;
+  const bool conv = a.w1 != nullptr;
+  const int b = blockIdx.y;
+  const int lo = conv ? a.cu_q[b] : 0;
+  const int n = (conv ? a.cu_q[b + 1] : a.rows) - lo;
+  const int r0 = blockIdx.x * a.block_rows;
+  if (r0 >= n) return;
+  const int r1 = min(r0 + a.block_rows, n);
+  const int hist_n = a.taps - 1;
+  const float gain = a.gain[0];
+
+  float hist[NC][V][MT > 1 ? MT - 1 : 1];
+  float f1[NC][V][MT], f2[NC][V][MT];
+  int ch[NC];
+#pragma unroll
+  for (int g = 0; g < NC; ++g) {
+    ch[g] = (g * blockDim.x + tid) * V;
+#pragma unroll
+    for (int v = 0; v < V; ++v) {
+#pragma unroll
+      for (int j = 0; j < MT - 1; ++j) hist[g][v][j] = 0.f;
+#pragma unroll
+      for (int j = 0; j < MT; ++j) {
+        const int src = j - (MT - a.taps);
+        const bool ok = conv && src >= 0 && ch[g] + v < a.width;
+        f1[g][v][j] = ok ? a.w1[(size_t)(ch[g] + v) * a.taps + src] : 0.f;
+        f2[g][v][j] = ok && a.w2 != nullptr ? a.w2[(size_t)(ch[g] + v) * a.taps + src] : 0.f;
+      }
+    }
+  }
+  float* st = nullptr;
+  if (conv && hist_n > 0 && r0 == 0) {
+    st = a.state + (size_t)a.slots[b] * a.width * hist_n;
+    if (a.has_state[b] != 0) {
+#pragma unroll
+      for (int g = 0; g < NC; ++g)
+#pragma unroll
+        for (int v = 0; v < V; ++v)
+#pragma unroll
+          for (int j = 0; j < MT - 1; ++j) {
+            const int src = j - (MT - 1 - hist_n);
+            if (src >= 0 && ch[g] + v < a.width) hist[g][v][j] = st[(size_t)(ch[g] + v) * hist_n + src];
+          }
+    }
+  }
+
+  auto load_row = [&](int r, float (&x)[NC][V]) {
+    const size_t row = (size_t)(lo + r);
+#pragma unroll
+    for (int g = 0; g < NC; ++g) {
+#pragma unroll
+      for (int v = 0; v < V; ++v) x[g][v] = 0.f;
+      if (ch[g] < a.width) {
+        if constexpr (V == 4) {
+          const float4 q = *reinterpret_cast<const float4*>(a.x + row * a.width + ch[g]);
+          x[g][0] = q.x; x[g][1] = q.y; x[g][2] = q.z; x[g][3] = q.w;
+          for (int p = 0; p < a.planes; ++p) {
+            const float4 d = *reinterpret_cast<const float4*>(a.delta + p * a.plane_stride + row * a.ldd + ch[g]);
+            x[g][0] += d.x; x[g][1] += d.y; x[g][2] += d.z; x[g][3] += d.w;
+          }
+        } else {
+#pragma unroll
+          for (int v = 0; v < V; ++v) {
+            x[g][v] = a.x[row * a.width + ch[g] + v];
+            for (int p = 0; p < a.planes; ++p) x[g][v] += a.delta[p * a.plane_stride + row * a.ldd + ch[g] + v];
+          }
+        }
+      }
+    }
+  };
+  int flip = 0;
+  auto rms_scale = [&](const float (&x)[NC][V]) {   // gain / rms of the row; one barrier (alternating scratch)
+    float s = 0.f;
+#pragma unroll
+    for (int g = 0; g < NC; ++g)
+#pragma unroll
+      for (int v = 0; v < V; ++v) s = fmaf(x[g][v], x[g][v], s);
+    s = warp_sum(s);
+    if (lane == 0) red[flip][warp] = s;
+    __syncthreads();
+    s = lane < n_warps ? red[flip][lane] : 0.f;
+    s = warp_sum(s);
+    flip ^= 1;
+    return gain / sqrtf(s / (float)a.width + a.eps);
+  };
+  auto push = [&](const float (&h)[NC][V]) {
+#pragma unroll
+    for (int g = 0; g < NC; ++g)
+#pragma unroll
+      for (int v = 0; v < V; ++v) {
+#pragma unroll
+        for (int j = 0; j + 1 < MT - 1; ++j) hist[g][v][j] = hist[g][v][j + 1];
+        if (MT > 1) hist[g][v][MT - 2 > 0 ? MT - 2 : 0] = h[g][v];
+      }
+  };
+  T* y1 = reinterpret_cast<T*>(a.y1);
+  T* y2 = reinterpret_cast<T*>(a.y2);
+
+  float x[NC][V], nx[NC][V];
+  const int first = conv ? max(r0 - hist_n, 0) : r0;
+  load_row(first, x);
+  for (int r = first; r < r1; ++r) {
+    if (r + 1 < r1) load_row(r + 1, nx);
+    const float sc = rms_scale(x);
+    const size_t row = (size_t)(lo + r);
+    if (r >= r0) {
+#pragma unroll
+      for (int g = 0; g < NC; ++g) {
+        if (ch[g] < a.width) {
+          if (a.x_out != a.x) {
+            if constexpr (V == 4)
+              *reinterpret_cast<float4*>(a.x_out + row * a.width + ch[g]) =
+                  make_float4(x[g][0], x[g][1], x[g][2], x[g][3]);
+            else
+#pragma unroll
+              for (int v = 0; v < V; ++v) a.x_out[row * a.width + ch[g] + v] = x[g][v];
+          }
+        }
+        if (ch[g] < a.cols) {
+          float o1[V], o2[V];
+#pragma unroll
+          for (int v = 0; v < V; ++v) {
+            const float h = x[g][v] * sc;
+            o1[v] = fmaf(f1[g][v][MT - 1], h, h);
+            o2[v] = fmaf(f2[g][v][MT - 1], h, h);
+#pragma unroll
+            for (int j = 0; j < MT - 1; ++j) {
+              o1[v] = fmaf(f1[g][v][j], hist[g][v][j], o1[v]);
+              o2[v] = fmaf(f2[g][v][j], hist[g][v][j], o2[v]);
+            }
+          }
+          const size_t off = row * a.cols + ch[g];
+          if constexpr (V == 4 && sizeof(T) == 2) {
+            uint2 q;
+            *reinterpret_cast<typename Pack2<T>::type*>(&q.x) = Pack2<T>::make(o1[0], o1[1]);
+            *reinterpret_cast<typename Pack2<T>::type*>(&q.y) = Pack2<T>::make(o1[2], o1[3]);
+            *reinterpret_cast<uint2*>(y1 + off) = q;
+            if (y2 != nullptr) {
+              *reinterpret_cast<typename Pack2<T>::type*>(&q.x) = Pack2<T>::make(o2[0], o2[1]);
+              *reinterpret_cast<typename Pack2<T>::type*>(&q.y) = Pack2<T>::make(o2[2], o2[3]);
+              *reinterpret_cast<uint2*>(y2 + off) = q;
+            }
+          } else {
+#pragma unroll
+            for (int v = 0; v < V; ++v) {
+              y1[off + v] = from_float<T>(o1[v]);
+              if (y2 != nullptr) y2[off + v] = from_float<T>(o2[v]);
+            }
+          }
+        }
+      }
+    }
+#pragma unroll
+    for (int g = 0; g < NC; ++g)
+#pragma unroll
+      for (int v = 0; v < V; ++v) x[g][v] *= sc;
+    push(x);
+#pragma unroll
+    for (int g = 0; g < NC; ++g)
+#pragma unroll
+      for (int v = 0; v < V; ++v) x[g][v] = nx[g][v];
+  }
+  if (st == nullptr) return;
+  // The CTA that read the request's tail also writes the new one (recomputing the last rows when they
+  // are another CTA's), so no CTA reads a tail that another one is replacing.
+  if (r1 < n) {
+    for (int r = n - hist_n; r < n; ++r) {
+      load_row(r, x);
+      const float sc = rms_scale(x);
+#pragma unroll
+      for (int g = 0; g < NC; ++g)
+#pragma unroll
+        for (int v = 0; v < V; ++v) x[g][v] *= sc;
+      push(x);
+    }
+  }
+#pragma unroll
+  for (int g = 0; g < NC; ++g)
+#pragma unroll
+    for (int v = 0; v < V; ++v)
+#pragma unroll
+      for (int j = 0; j < MT - 1; ++j) {
+        const int dst = j - (MT - 1 - hist_n);
+        if (dst >= 0 && ch[g] + v < a.width) st[(size_t)(ch[g] + v) * hist_n + dst] = hist[g][v][j];
+      }
+}
+
+template <typename T, int V, int NC>
+void launch_norm_conv(const NormConvArgs& a, dim3 grid, int threads, cudaStream_t s) {
+  if (a.taps <= 1)
+    msgl_launch(norm_conv_kernel<T, V, NC, 1>, grid, dim3(threads), 0, s, a);
+  else if (a.taps <= 4)
+    msgl_launch(norm_conv_kernel<T, V, NC, 4>, grid, dim3(threads), 0, s, a);
+  else if (a.taps <= 8)
+    msgl_launch(norm_conv_kernel<T, V, NC, 8>, grid, dim3(threads), 0, s, a);
+  else
+    msgl_launch(norm_conv_kernel<T, V, NC, 32>, grid, dim3(threads), 0, s, a);
+}
+
+template <typename T>
+int norm_conv_typed(NormConvArgs a, int B, int max_q, cudaStream_t s) {
+  const bool conv = a.w1 != nullptr;
+  // enough rows per CTA to make the recomputed rows cheap (and at least taps - 1 of them)
+  a.block_rows = conv ? (a.taps > 8 ? 32 : 16) : 1;
+  const int n = conv ? max_q : a.rows;
+  dim3 grid((n + a.block_rows - 1) / a.block_rows, conv ? B : 1);
+  const bool vec = a.width % 4 == 0 && a.cols % 4 == 0 && a.ldd % 4 == 0 && (uintptr_t)a.delta % 16 == 0;
+  const int per = vec ? 4 : 1;
+  const int groups = (a.cols + per - 1) / per;
+  const int threads = groups >= 1024 ? 1024 : (groups + 31) / 32 * 32;
+  const int nc = (groups + threads - 1) / threads;
+  if (vec) {
+    if (nc == 1) launch_norm_conv<T, 4, 1>(a, grid, threads, s);
+    else if (nc == 2) launch_norm_conv<T, 4, 2>(a, grid, threads, s);
+    else return MSGL_BAD_ARG;
+  } else {
+    if (nc <= 1) launch_norm_conv<T, 1, 1>(a, grid, threads, s);
+    else if (nc <= 4) launch_norm_conv<T, 1, 4>(a, grid, threads, s);
+    else return MSGL_BAD_ARG;
+  }
+  MSGL_CHECK_LAUNCH("norm_conv");
+  return MSGL_OK;
+}
+
+// Exact gelu of [rows, n] with row strides; n a multiple of 4.
+template <typename T>
+__global__ void __launch_bounds__(256) gelu_erf_kernel(const T* __restrict__ x, long long ldx, T* __restrict__ out,
+                                                       long long ldo, int n, long long total) {
+  pdl_enter();
+  constexpr int V = 16 / sizeof(T);
+  const long long i = (long long)blockIdx.x * 256 + threadIdx.x;
+  if (i >= total) return;
+  const int per = n / V;
+  const long long r = i / per;
+  const int c = (int)(i - r * per) * V;
+  float v[V];
+  if constexpr (sizeof(T) == 2) {
+    load8(x + r * ldx + c, v);
+  } else {
+    const float4 q = *reinterpret_cast<const float4*>(x + r * ldx + c);
+    v[0] = q.x; v[1] = q.y; v[2] = q.z; v[3] = q.w;
+  }
+#pragma unroll
+  for (int e = 0; e < V; ++e) v[e] = 0.5f * v[e] * (1.f + erff(v[e] * 0.70710678118654752f));
+  if constexpr (sizeof(T) == 2)
+    store8(out + r * ldo + c, v);
+  else
+    *reinterpret_cast<float4*>(out + r * ldo + c) = make_float4(v[0], v[1], v[2], v[3]);
+}
+
+}  // namespace
+
+MSGL_API int msgl_embed_positions(const void* ids, const void* w, const void* pos, const void* positions, void* out,
+                                  int rows, int width, int start, int len, int n_pos, int dtype, cudaStream_t stream) {
+  if (rows <= 0) return rows == 0 ? MSGL_OK : MSGL_BAD_ARG;
+#define EMB(T)                                                                                                      \
+  msgl_launch(embed_positions_kernel<T>, dim3(rows), dim3(256), 0, stream, (const int32_t*)ids, (const T*)w,        \
+              (const T*)pos, (const int32_t*)positions, (float*)out, width, start, len, n_pos)
+  if (dtype == MSGL_BF16) EMB(__nv_bfloat16);
+  else if (dtype == MSGL_F32) EMB(float);
+  else return MSGL_BAD_ARG;
+#undef EMB
+  MSGL_CHECK_LAUNCH("embed_positions");
+  return MSGL_OK;
+}
+
+MSGL_API int msgl_norm_conv(const void* x, void* x_out, const void* delta, int planes, long long plane_stride,
+                            long long ldd, const void* gain, float eps, const void* w1, const void* w2, void* y1,
+                            void* y2, void* state, const void* cu_q, const void* slots, const void* has_state, int rows,
+                            int width, int cols, int taps, int B, int max_q, int dtype, cudaStream_t stream) {
+  if (rows <= 0) return rows == 0 ? MSGL_OK : MSGL_BAD_ARG;
+  if (taps < 1 || taps > 32 || cols < width || (planes > 0 && x == x_out)) return MSGL_BAD_ARG;
+  if (w1 != nullptr && (B <= 0 || max_q <= 0)) return MSGL_BAD_ARG;
+  NormConvArgs a{(const float*)x, (float*)x_out, (const float*)delta, planes, plane_stride, ldd, (const float*)gain, eps,
+                 (const float*)w1, (const float*)w2, y1, y2, (float*)state, (const int32_t*)cu_q,
+                 (const int32_t*)slots, (const int32_t*)has_state, rows, width, cols, taps, 0};
+  if (dtype == MSGL_BF16) return norm_conv_typed<__nv_bfloat16>(a, B, max_q, stream);
+  if (dtype == MSGL_F32) return norm_conv_typed<float>(a, B, max_q, stream);
+  return MSGL_BAD_ARG;
+}
+
+MSGL_API int msgl_gelu_erf(const void* x, long long ldx, void* out, long long ldo, int rows, int n, int dtype,
+                           cudaStream_t stream) {
+  if (rows <= 0 || n <= 0) return rows == 0 || n == 0 ? MSGL_OK : MSGL_BAD_ARG;
+  const int v = dtype == MSGL_BF16 ? 8 : 4;
+  if (n % v || ldx % v || ldo % v || (uintptr_t)x % 16 || (uintptr_t)out % 16) return MSGL_BAD_ARG;
+  const long long total = (long long)rows * (n / v);
+  dim3 grid((unsigned)((total + 255) / 256));
+  if (dtype == MSGL_BF16)
+    msgl_launch(gelu_erf_kernel<__nv_bfloat16>, grid, dim3(256), 0, stream, (const __nv_bfloat16*)x, ldx,
+                (__nv_bfloat16*)out, ldo, n, total);
+  else if (dtype == MSGL_F32)
+    msgl_launch(gelu_erf_kernel<float>, grid, dim3(256), 0, stream, (const float*)x, ldx, (float*)out, ldo, n, total);
+  else
+    return MSGL_BAD_ARG;
+  MSGL_CHECK_LAUNCH("gelu_erf");
+  return MSGL_OK;
+}

@@ -81,8 +81,10 @@ def _resolve_dtype(cfg: EngineConfig, model_cfg: ModelConfig, device: str) -> to
              "bf16": torch.bfloat16, "bfloat16": torch.bfloat16,
              "fp32": torch.float32, "float32": torch.float32, "float": torch.float32}
     dt = table[name]
-    if device == "cuda" and dt == torch.float32:
-        dt = torch.bfloat16
+    if device == "cuda" and dt == torch.float32 and not model_cfg.latent_layers:
+        dt = torch.bfloat16            # the other families' kernels are 16-bit
+    if device == "cuda" and dt == torch.float16 and model_cfg.latent_layers:
+        raise ValueError("models with a latent pool run in bfloat16 or float32 on a GPU")
     return dt
 
 
@@ -278,6 +280,8 @@ class Engine:
         # latent-attention models can keep the compressed latent per token instead of per-head K/V
         # (MSGL_MLA_LATENT): absorbed attention through tensor ops, eager steps, no draft verification
         self.mla_latent = bool(ENV.MLA_LATENT.value and mc.is_mla)
+        if mc.latent_layers and (self.kv_fp8 or self.kv_calibrating):
+            raise ValueError("the latent pool has no fp8 form")
         if self.mla_latent:
             if self.kv_fp8 or self.kv_calibrating:
                 raise ValueError("the latent pool (MSGL_MLA_LATENT) is 16-bit only")
@@ -293,6 +297,11 @@ class Engine:
                                            int(mc.qk_rope_head_dim), self.dtype, self.device)
             logger.info_rank0("latent K/V pool: %d values per token and layer (per-head K/V would take %d)",
                               self.kv_cache.width, 2 * self.kv_heads_local * mc.head_dim)
+        elif mc.latent_layers:
+            from ..kvcache.mla_pool import MLALatentCache
+
+            self.kv_cache = MLALatentCache(self.kv_layers, self.num_pages, self.page_size, max(mc.latent_widths), 0,
+                                           self.dtype, self.device, widths=mc.latent_widths)
         else:
             self.kv_cache = MHAKVCache(
                 self.kv_layers, self.num_pages, self.page_size, self.kv_heads_local, mc.head_dim,
@@ -341,9 +350,10 @@ class Engine:
             from ..kvcache.gdn_state import GDNStateCache
 
             conv_dim, st_heads, st_rows, st_cols = mc.recurrent_geometry
-            conv_dim, st_heads = conv_dim // config.tp_size, st_heads // config.tp_size   # this rank's heads
+            if not mc.input_conv_taps:             # (an input convolution runs on whole rows, on every rank)
+                conv_dim, st_heads = conv_dim // config.tp_size, st_heads // config.tp_size   # this rank's heads
             self.gdn_state = GDNStateCache(mc.num_linear_layers, self.num_slots, conv_dim, mc.linear_conv_kernel_dim,
-                                           st_heads, st_rows, st_cols, self.dtype, self.device)
+                                           st_heads, st_rows, st_cols, self._conv_state_dtype, self.device)
             self.ledger.add("recurrent state", self.gdn_state.conv.numel() * self.gdn_state.conv.element_size()
                             + self.gdn_state.ssm.numel() * 4)
         self.ctx.gdn_state = self.gdn_state
@@ -352,7 +362,7 @@ class Engine:
         self.ctx.attn_backend = create_attention_backend(
             config.attention_backend, self.q_heads_local, self.kv_heads_local, mc.head_dim, self.device,
             max_batch=config.max_running_req, max_seq_len=self.max_seq_len,
-            single_split=config.spec_algorithm != "none",
+            single_split=config.spec_algorithm != "none", latent=bool(mc.latent_layers),
         )
         self.ctx.comm = comm_mod.get_comm()
         self._spec_exact = config.spec_algorithm != "none" and dev_kind == "cuda"
@@ -472,7 +482,8 @@ class Engine:
 
                     symm = SymmetricCollectives(self.tp_group, self.cpu_group, self.device, cfg.tp_rank, cfg.tp_size)
                     comm.register(symm)
-                    if not ENV.DISABLE_ROW_SHARD.value and not self.model_config.is_moe:
+                    if (not ENV.DISABLE_ROW_SHARD.value and not self.model_config.is_moe
+                            and not self.model_config.latent_layers):
                         # prefill chunks: GEMM -> reduce-scatter -> add + norm -> all-gather -> GEMM
                         symm.enable_row_shard(int(getattr(cfg, "max_extend_tokens", 8192)),
                                               self.model_config.hidden_size)
@@ -519,6 +530,11 @@ class Engine:
         logger.info_rank0("host expert tier: %d of %d experts resident per layer (plan %s, %.2f GiB pinned)",
                           plan.layers[0].device_slots, mc.num_experts, plan.digest, plan.host_bytes / (1 << 30))
 
+    @property
+    def _conv_state_dtype(self) -> torch.dtype:
+        # the tail of an input convolution holds normalised rows of an fp32 residual stream
+        return torch.float32 if self.model_config.input_conv_taps else self.dtype
+
     def _free_memory(self) -> int:
         if self.device.type == "cuda":
             torch.cuda.synchronize(self.device)
@@ -543,6 +559,8 @@ class Engine:
 
             per_page = MLALatentCache.token_bytes(self.kv_layers, int(mc.kv_lora_rank), int(mc.qk_rope_head_dim),
                                                   itemsize) * self.page_size
+        if mc.latent_layers:
+            per_page = sum(mc.latent_widths) * itemsize * self.page_size
         if cfg.spec_algorithm in ("eagle3", "mtp"):
             # the draft head keeps one 16-bit, unsharded layer of K/V on the same page table
             per_page += MHAKVCache.token_bytes(1, mc.num_kv_heads, mc.head_dim, 2) * self.page_size
@@ -561,9 +579,11 @@ class Engine:
             from ..kvcache.gdn_state import GDNStateCache
 
             conv_dim, st_heads, st_rows, st_cols = mc.recurrent_geometry
-            conv_dim, st_heads = conv_dim // cfg.tp_size, st_heads // cfg.tp_size
+            if not mc.input_conv_taps:
+                conv_dim, st_heads = conv_dim // cfg.tp_size, st_heads // cfg.tp_size
             budget -= (cfg.max_running_req + 1) * GDNStateCache.slot_bytes(
-                mc.num_linear_layers, conv_dim, mc.linear_conv_kernel_dim, st_heads, st_rows, st_cols, 2)
+                mc.num_linear_layers, conv_dim, mc.linear_conv_kernel_dim, st_heads, st_rows, st_cols,
+                4 if mc.input_conv_taps else 2)
         pages = budget // per_page
         if self.cpu_group is not None:
             t = torch.tensor([pages], dtype=torch.int64)
@@ -577,6 +597,8 @@ class Engine:
         cfg, mc = self.config, self.model_config
         limit = cfg.max_seq_len_override or mc.max_position_embeddings
         limit = min(limit, mc.rotary_config.max_position, self.num_pages * self.page_size)
+        if mc.latent_layers:
+            return int(limit)                  # learned positions: every one of them can be used
         return int(limit // self.page_size * self.page_size) or self.page_size
 
     # ------------------------------------------------------------------ step
@@ -791,7 +813,7 @@ class Engine:
 
     def _row_shard_rows(self, tokens: int) -> bool:
         """Whether a step of ``tokens`` rows takes the row-sharded tensor-parallel path."""
-        if self.config.tp_size == 1 or self.model_config.is_moe:
+        if self.config.tp_size == 1 or self.model_config.is_moe or self.model_config.latent_layers:
             return False
         for impl in comm_mod.get_comm().impls:
             rs = getattr(impl, "row_shard", None)

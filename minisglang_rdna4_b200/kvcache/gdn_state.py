@@ -17,6 +17,7 @@ import torch
 class GDNStateCache:
     def __init__(self, num_layers: int, num_slots: int, conv_dim: int, conv_kernel: int, num_v_heads: int,
                  head_k_dim: int, head_v_dim: int, dtype: torch.dtype, device) -> None:
+        # no state matrix (num_v_heads 0): the state is the convolution tail alone
         self.num_layers, self.num_slots = num_layers, num_slots
         self.conv = torch.zeros((num_layers, num_slots, conv_dim, conv_kernel - 1), dtype=dtype, device=device)
         self.ssm = torch.zeros((num_layers, num_slots, num_v_heads, head_k_dim, head_v_dim), dtype=torch.float32,

@@ -43,10 +43,12 @@ class VocabParallelEmbedding(BaseOP):
 
 class ParallelLMHead(BaseOP):
     def __init__(self, vocab: int, hidden: int, dtype, device,
-                 tied: Optional[VocabParallelEmbedding] = None) -> None:
+                 tied: Optional[VocabParallelEmbedding] = None, align: int = 1) -> None:
+        """``align``: a rank's rows are padded to a multiple of it (the GEMM kernel takes 8 output columns at a
+        time), for vocabularies of any size."""
         tp = get_tp_info()
         self._vocab = vocab
-        self._per_rank = cdiv(vocab, tp.size)
+        self._per_rank = cdiv(cdiv(vocab, tp.size), align) * align
         self._start = tp.rank * self._per_rank
         self._len = max(0, min(self._per_rank, vocab - self._start))
         self._tp = tp

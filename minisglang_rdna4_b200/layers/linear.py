@@ -144,3 +144,21 @@ class RowParallelLinear(_LinearBase):
                 K.set_next_gemm_planes(False)
         y = self._method.apply(self, x, bias)
         return comm.all_reduce(y) if reduce else y
+
+    def forward_partial32(self, x: torch.Tensor):
+        """fp32 result for an fp32 residual stream (16- or 32-bit dense weights): the finished sum over ranks, or on one
+        GPU in a small step possibly the unreduced K ranges (``SplitPartial``) for the next add + norm to sum."""
+        from .. import ops
+
+        comm = get_comm()
+        if x.is_cuda and comm.size == 1 and x.dtype != torch.float32 and x.shape[0] <= 256:
+            from ..ops import cuda as K
+
+            if K.SPLIT_K_DECODE:
+                K.set_next_gemm_planes(True)
+                try:
+                    return ops.gemm(x, self.weight, None, torch.float32)
+                finally:
+                    K.set_next_gemm_planes(False)
+        y = ops.gemm(x, self.weight, None, torch.float32)
+        return comm.all_reduce(y) if comm.size > 1 else y

@@ -63,6 +63,11 @@ def _register_defaults() -> None:
     if "NemotronHForCausalLM" not in MODEL_REGISTRY:
         MODEL_REGISTRY.register("NemotronHForCausalLM")(NemotronHForCausalLM)
 
+    from .mitilix import MitilixForCausalLM
+
+    if "MitilixForCausalLM" not in MODEL_REGISTRY:
+        MODEL_REGISTRY.register("MitilixForCausalLM")(MitilixForCausalLM)
+
 
 def create_model(cfg: ModelConfig, dtype: torch.dtype, device):
     """Instantiate the model for ``cfg`` with uninitialised (or meta) parameters."""

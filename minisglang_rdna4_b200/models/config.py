@@ -34,6 +34,40 @@ class RotaryConfig:
         )
 
 
+def _round_up(n: int, m: int) -> int:
+    return (n + m - 1) // m * m
+
+
+@dataclass(frozen=True)
+class LatentLayer:
+    """One layer whose attention keeps a shared latent per token (no rotary part): ``heads`` query heads of ``dim``
+    channels, values of ``vdim``, a latent of ``kv_rank``; ``window`` 0 = every earlier position is visible;
+    ``kv_from``: the layer whose latent is read instead of an own one; ``ff`` 0 = no feed-forward. The ``*_pad``
+    widths are what the kernels see: zero channels that change no dot product."""
+
+    heads: int
+    dim: int
+    vdim: int
+    kv_rank: int
+    scale: float
+    window: int = 0
+    kv_from: Optional[int] = None
+    ff: int = 0
+
+    @property
+    def dim_pad(self) -> int:
+        return _round_up(self.dim, 16)
+
+    @property
+    def vdim_pad(self) -> int:
+        return _round_up(self.vdim, 16)
+
+    @property
+    def rank_pad(self) -> int:
+        r = _round_up(self.kv_rank, 64)
+        return r if r <= 256 else _round_up(r, 256)
+
+
 @dataclass(frozen=True)
 class ModelConfig:
     num_layers: int
@@ -91,6 +125,10 @@ class ModelConfig:
     mlp_hidden_act: str = "silu"          # "relu2": non-gated squared-ReLU MLPs and experts
     attn_output_gate: bool = False        # q_proj also emits a per-head sigmoid gate of the attention output
     norm_plus_one: bool = False           # RMSNorm weights are stored as (w - 1)
+    # layers that keep an attention latent per token, each with its own sizes; a short causal convolution ahead of
+    # every sublayer (taps, 0 = none) whose last inputs are per-request state
+    latent_layers: Optional[Tuple[LatentLayer, ...]] = None
+    input_conv_taps: int = 0
     # misc
     sliding_window: Optional[int] = None
     layer_types: Optional[Tuple[str, ...]] = None
@@ -143,18 +181,33 @@ class ModelConfig:
         return self.kv_lora_rank is not None
 
     @property
+    def latent_widths(self) -> Tuple[int, ...]:
+        """Pool row width of every layer that keeps a latent of its own, in layer order."""
+        return tuple(s.rank_pad for s in self.latent_layers or () if s.kv_from is None)
+
+    def latent_row(self, layer: int) -> int:
+        """Index in the latent pool of the layer whose latent ``layer`` reads."""
+        specs = self.latent_layers
+        owner = layer if specs[layer].kv_from is None else specs[layer].kv_from
+        return sum(1 for s in specs[:owner] if s.kv_from is None)
+
+    @property
     def is_recurrent(self) -> bool:
-        """Some layers keep a recurrent state per request instead of K/V pages."""
-        return bool(self.layer_types) and any(t in ("linear_attention", "mamba") for t in self.layer_types)
+        """Some layers keep a recurrent state (or a convolution tail) per request besides or instead of K/V pages."""
+        return self.input_conv_taps > 0 or bool(self.layer_types) and any(t in ("linear_attention", "mamba") for t in self.layer_types)
 
     @property
     def num_linear_layers(self) -> int:
-        """Layers with a recurrent state (gated delta net or Mamba-2)."""
+        """Layers with a recurrent state (gated delta net, Mamba-2, input convolutions)."""
+        if self.input_conv_taps:
+            return self.num_layers
         return sum(1 for t in (self.layer_types or ()) if t in ("linear_attention", "mamba"))
 
     @property
     def num_kv_layers(self) -> int:
         """Layers that keep K/V pages."""
+        if self.latent_layers:
+            return len(self.latent_widths)
         if self.model_type == "nemotron_h":
             return sum(1 for t in (self.layer_types or ()) if t == "attention")
         return self.num_layers - self.num_linear_layers - self.num_kv_shared_layers
@@ -194,7 +247,9 @@ class ModelConfig:
     @property
     def recurrent_geometry(self) -> Tuple[int, int, int, int]:
         """``(conv channels, heads, rows, cols)`` of one recurrent layer's state: a convolution window
-        over ``conv channels`` inputs and a ``[heads, rows, cols]`` fp32 state matrix per request."""
+        over ``conv channels`` inputs and a ``[heads, rows, cols]`` fp32 state matrix per request (``heads`` 0: the window alone)."""
+        if self.input_conv_taps:
+            return self.hidden_size, 0, 0, 0
         if self.mamba_num_heads:
             inter = self.mamba_num_heads * self.mamba_head_dim
             return (inter + 2 * self.mamba_n_groups * self.ssm_state_size, self.mamba_num_heads, self.mamba_head_dim,
@@ -247,6 +302,8 @@ class ModelConfig:
                 cfg = json.load(fh)
         if not isinstance(cfg, dict):
             cfg = cfg.to_dict()
+        if cfg.get("architecture") == "Mitilix":
+            return _mitilix_config(cfg)
         vision = None
         if "text_config" in cfg and isinstance(cfg["text_config"], dict):
             if str(cfg.get("model_type", "")).startswith("gemma3") and cfg.get("vision_config"):
@@ -471,6 +528,42 @@ class ModelConfig:
             draft_vocab_size=g("draft_vocab_size"),
             eagle_aux_layers=tuple(g("eagle_aux_hidden_state_layer_ids") or ()) or None,
         )
+
+
+def _mitilix_config(cfg: Dict[str, Any]) -> ModelConfig:
+    """``layers`` lists every layer's mixer and feed-forward with sizes of their own."""
+    specs = []
+    for i, layer in enumerate(cfg["layers"]):
+        kind, mix, mlp = layer["type"], layer["mixer"], layer.get("mlp")
+        if kind != "latent_attention":
+            raise ValueError(f"layer {i}: unknown mixer type {kind!r}")
+        if mlp is not None and mlp["kind"] != "dense":
+            raise ValueError(f"layer {i}: unknown feed-forward kind {mlp['kind']!r}")
+        donor = mix.get("kv_from")
+        if donor is not None:
+            donor = int(donor)
+            if not 0 <= donor < i or specs[donor].kv_from is not None or specs[donor].kv_rank != int(mix["kv_rank"]):
+                raise ValueError(f"layer {i}: kv_from {donor} names no earlier layer with a latent of this size")
+        window = int((mix.get("mask") or {}).get("size") or 0)
+        specs.append(LatentLayer(heads=int(mix["heads"]), dim=int(mix["dim"]), vdim=int(mix["vdim"]),
+                                 kv_rank=int(mix["kv_rank"]), scale=float(mix["scale"]), window=window, kv_from=donor,
+                                 ff=int(mlp["ff"]) if mlp is not None else 0))
+    width, max_pos = int(cfg["width"]), int(cfg["max_positions"])
+    first = specs[0]
+    eos = cfg.get("eos_token_id")
+    eos_ids = tuple(eos) if isinstance(eos, (list, tuple)) else (() if eos is None else (int(eos),))
+    return ModelConfig(
+        num_layers=len(specs), num_qo_heads=first.heads, num_kv_heads=1, head_dim=first.rank_pad, hidden_size=width,
+        vocab_size=int(cfg["vocab"]),
+        # the widest activations of a step: queries in the latent space and the feed-forward
+        intermediate_size=max(max(s.ff, s.heads * s.rank_pad) for s in specs),
+        rms_norm_eps=float(cfg["norm"]["eps"]),
+        rotary_config=RotaryConfig(head_dim=first.rank_pad, rotary_dim=0, max_position=max_pos, base=10000.0),
+        hidden_act="gelu", model_type="mitilix", architectures=("MitilixForCausalLM",),
+        latent_layers=tuple(specs), input_conv_taps=int(cfg["canon"]["taps"]),
+        linear_conv_kernel_dim=int(cfg["canon"]["taps"]), max_position_embeddings=max_pos, eos_token_ids=eos_ids,
+        bos_token_id=cfg.get("bos_token_id"),
+    )
 
 
 def _default_arch(model_type: str) -> List[str]:

@@ -79,6 +79,8 @@ class _Collector:
 
 
 def load_weights(model, path: str, cfg: ModelConfig, device, tensors: Optional[Iterator] = None) -> None:
+    if hasattr(model, "checkpoint_map"):
+        return _load_mapped(model, tensors if tensors is not None else iter_safetensors(path), device)
     tp = get_tp_info()
     ep = get_ep_info() if ep_enabled() else None
     modules: Dict[str, object] = {}
@@ -451,6 +453,30 @@ def load_weights(model, path: str, cfg: ModelConfig, device, tensors: Optional[I
     for n, t, owner, attr in model.named_parameters():
         if n not in loaded and n.endswith("bias"):
             setattr(owner, attr, torch.zeros_like(t))  # all-zero biases are dropped by exporters
+
+
+def _load_mapped(model, stream: Iterator, device) -> None:
+    """Models that name their checkpoint tensors themselves (``checkpoint_map``): every parameter starts at zero (what
+    no tensor covers is padding) and each tensor is written into its place."""
+    wanted = model.checkpoint_map()
+    for _, t, owner, attr in list(model.named_parameters()):
+        setattr(owner, attr, torch.zeros(t.shape, dtype=t.dtype, device=device))
+    seen = set()
+    for name, tensor in stream:
+        places = wanted.get(name)
+        if places is None:
+            logger.debug_rank0("skipping unexpected tensor %s", name)
+            continue
+        for owner, attr, fill in places:
+            param = getattr(owner, attr)
+            try:
+                fill(param, tensor.to(device=device, dtype=param.dtype))
+            except RuntimeError as exc:
+                raise ValueError(f"{name}: checkpoint shape {tuple(tensor.shape)} does not fit: {exc}") from None
+        seen.add(name)
+    missing = sorted(set(wanted) - seen)
+    if missing:
+        raise KeyError(f"checkpoint is missing parameters: {missing[:8]} (+{max(len(missing) - 8, 0)} more)")
 
 
 def _optional(name: str) -> bool:

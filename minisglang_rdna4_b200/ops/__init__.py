@@ -207,6 +207,49 @@ def rms_norm_gated(x, z, w, eps: float):
     return ref.rms_norm_gated(x, z.reshape(x.shape), w, eps)
 
 
+# ---------------------------------------------------------------------------- fp32 residual, latent attention
+def embed_positions(ids, weight, pos, positions, vocab_start: int = 0, vocab_len: Optional[int] = None):
+    if weight.is_cuda:
+        return _cuda().embed_positions(ids, weight, pos, positions, vocab_start, vocab_len)
+    return ref.embed_positions(ids, weight, pos, positions, vocab_start, vocab_len)
+
+
+def add_scalar_norm_conv(x, delta, gain, eps: float, w1, w2, state, cu_q, slots, has_state, max_q: int, out_dtype,
+                         out_cols: int):
+    """Residual add, scalar-gain RMS norm and one or two short causal convolutions in one pass:
+    ``(new residual, y1, y2)``. ``delta`` may be the unreduced K ranges of a GEMM (``SplitPartial``)."""
+    if x.is_cuda:
+        return _cuda().add_scalar_norm_conv(x, delta, gain, eps, w1, w2, state, cu_q, slots, has_state, max_q,
+                                            out_dtype, out_cols)
+    return ref.add_scalar_norm_conv(x, delta, gain, eps, w1, w2, state, cu_q, slots, has_state, out_dtype, out_cols)
+
+
+def gelu_erf(x, out):
+    """Exact gelu of ``x [T, N]`` into ``out [T, N]`` (any row stride)."""
+    if x.is_cuda:
+        return _cuda().gelu_erf(x, out)
+    return ref.gelu_erf(x, out)
+
+
+def latent_norm_store(c, weight, rank: int, eps: float, rows, out_loc):
+    if c.is_cuda:
+        return _cuda().latent_norm_store(c, weight, rank, eps, rows, out_loc)
+    return ref.latent_norm_store(c, weight, rank, eps, rows, out_loc)
+
+
+def head_gemm(x, w, out=None):
+    if x.is_cuda:
+        return _cuda().head_gemm(x, w, out)
+    return ref.head_gemm(x, w, out)
+
+
+def latent_attention(q, rows, block_table, cu_q, seq_lens, scale: float, window: int, max_q: int, max_kv: int,
+                     splits: int = 1):
+    if q.is_cuda:
+        return _cuda().latent_attention(q, rows, block_table, cu_q, seq_lens, scale, window, max_q, max_kv, splits)
+    return ref.latent_attention(q, rows, block_table, cu_q, seq_lens, scale, window)
+
+
 # ---------------------------------------------------------------------------- sampling
 def argmax(logits):
     if logits.is_cuda:

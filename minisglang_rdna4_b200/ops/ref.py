@@ -605,3 +605,99 @@ def rms_norm_gated(x: torch.Tensor, z: torch.Tensor, w: torch.Tensor, eps: float
     y = xf * torch.rsqrt(xf.pow(2).mean(-1, keepdim=True) + eps)
     y = (w.float() * y.to(x.dtype).float()) * F.silu(z.float())
     return y.to(x.dtype)
+
+
+# ------------------------------------------------------------------------------------------
+# fp32 residual stream with a scalar-gain norm and short input convolutions; windowed latent attention
+# ------------------------------------------------------------------------------------------
+def embed_positions(ids: torch.Tensor, weight: torch.Tensor, pos: Optional[torch.Tensor], positions: torch.Tensor,
+                    vocab_start: int = 0, vocab_len: Optional[int] = None) -> torch.Tensor:
+    """Token embedding (zero outside this rank's vocabulary range) plus a learned position vector, fp32 ``[T, W]``."""
+    x = embedding(ids, weight, vocab_start, vocab_len).float()
+    return x if pos is None else x + pos[positions.long()].float()
+
+
+def add_scalar_norm_conv(x: torch.Tensor, delta: Optional[torch.Tensor], gain: torch.Tensor, eps: float,
+                         w1: Optional[torch.Tensor], w2: Optional[torch.Tensor], state: Optional[torch.Tensor],
+                         cu_q: Optional[torch.Tensor], slots: Optional[torch.Tensor],
+                         has_state: Optional[torch.Tensor], out_dtype: torch.dtype, out_cols: int):
+    """``x += delta``; ``h = x / rms(x) * gain`` (one number); ``y_k = h + conv_k(h)`` for the one or two depthwise
+    causal filters ``w_k [W, taps]``. Returns ``(x, y_1, y_2)``; with no filter ``y_1 = h``.
+
+    The convolutions read the same ``h``, so one tail ``state [slots, W, taps - 1]`` (fp32) serves both; it is
+    advanced in place. Outputs have ``out_cols >= W`` columns, zero past W."""
+    xn = x if delta is None else x + delta[:, :x.shape[1]].float()
+    h = xn * torch.rsqrt(xn.pow(2).mean(-1, keepdim=True) + eps) * gain.float().reshape(())
+
+    def cast(y):
+        return F.pad(y, (0, out_cols - y.shape[1])).to(out_dtype)
+
+    if w1 is None and w2 is None:
+        return xn, cast(h), None
+    taps = (w1 if w1 is not None else w2).shape[1]
+    ys = [h.clone() if w is not None else None for w in (w1, w2)]
+    for b in range(cu_q.numel() - 1):
+        lo, hi = int(cu_q[b]), int(cu_q[b + 1])
+        if hi <= lo:
+            continue
+        slot = int(slots[b])
+        hist = state[slot].t() if int(has_state[b]) else h.new_zeros((taps - 1, h.shape[1]))
+        seq = torch.cat([hist, h[lo:hi]])
+        for w, y in zip((w1, w2), ys):
+            if w is not None:
+                for j in range(taps):
+                    y[lo:hi] += seq[j:j + hi - lo] * w[:, j].float()
+        if taps > 1:
+            state[slot] = seq[seq.shape[0] - (taps - 1):].t()
+    return xn, *(None if y is None else cast(y) for y in ys)
+
+
+def gelu_erf(x: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
+    out.copy_(F.gelu(x.float()))
+    return out
+
+
+def latent_norm_store(c: torch.Tensor, weight: torch.Tensor, rank: int, eps: float, rows: torch.Tensor,
+                      out_loc: torch.Tensor) -> None:
+    """RMS norm over the first ``rank`` of ``c [T, width]`` with a plain weight, written to the token slots
+    ``out_loc`` of one layer of the latent pool ``rows [pages, page_size, width]`` (zero past ``rank``)."""
+    cf = c[:, :rank].float()
+    y = cf * torch.rsqrt(cf.pow(2).mean(-1, keepdim=True) + eps) * weight[:rank].float()
+    flat = rows.view(-1, rows.shape[-1])
+    flat.index_copy_(0, out_loc.long(), F.pad(y, (0, flat.shape[1] - rank)).to(flat.dtype))
+
+
+def head_gemm(x: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """Per-head projection: ``x [T, H, K]``, ``w [H, N, K]`` -> ``[T, H, N]``."""
+    y = torch.einsum("thk,hnk->thn", x.float(), w.float())
+    if out is None:
+        return y.to(x.dtype)
+    out.copy_(y)
+    return out
+
+
+def latent_attention(q: torch.Tensor, rows: torch.Tensor, block_table: torch.Tensor, cu_q: torch.Tensor,
+                     seq_lens: torch.Tensor, scale: float, window: int) -> torch.Tensor:
+    """Causal attention of ``q [T, H, R]`` over one shared latent per position that is key and value at once
+    (``rows [pages, page_size, R]``); ``window > 0``: the last ``window`` positions, the query's own included."""
+    t, h, r = q.shape
+    ps = rows.shape[1]
+    out = torch.zeros((t, h, r), dtype=torch.float32, device=q.device)
+    cu, lens = cu_q.tolist(), seq_lens.tolist()
+    for b, kv_len in enumerate(lens):
+        qs, qe = cu[b], cu[b + 1]
+        n = qe - qs
+        if n <= 0 or kv_len <= 0:
+            continue
+        lo = max(0, kv_len - n - window + 1) if window > 0 else 0
+        idx = torch.arange(lo, kv_len)
+        flat = rows.reshape(-1, r)
+        c = flat[block_table[b].long()[idx // ps] * ps + idx % ps].float()
+        s = torch.einsum("qhr,kr->hqk", q[qs:qe].float(), c) * scale
+        gap = torch.arange(kv_len - n, kv_len)[:, None] - idx[None, :]
+        hidden = gap < 0
+        if window > 0:
+            hidden |= gap >= window
+        s = s.masked_fill(hidden[None], float("-inf"))
+        out[qs:qe] = torch.einsum("hqk,kr->qhr", torch.softmax(s, -1), c)
+    return out.to(q.dtype)
