@@ -18,7 +18,7 @@ import os
 import shutil
 import subprocess
 import sys
-from typing import List
+from typing import List, Optional
 
 HERE = os.path.dirname(os.path.abspath(__file__))
 CSRC = os.path.join(HERE, "csrc")
@@ -56,21 +56,37 @@ def _headers() -> List[str]:
 
 
 def _compile(cmd: List[str], out: str, log: str) -> str:
+    # into a temporary file first: an interrupted build leaves no half-written object behind
+    tmp = f"{out}.{os.getpid()}.tmp"
+    cmd = [tmp if a == out else a for a in cmd]
     proc = subprocess.run(cmd, capture_output=True, text=True)
     with open(log, "w") as fh:
         fh.write(" ".join(cmd) + "\n" + proc.stdout + proc.stderr)
     if proc.returncode != 0:
         raise RuntimeError(f"build failed: {' '.join(cmd)}\n{proc.stdout}\n{proc.stderr}")
+    os.replace(tmp, out)
     return out
 
 
-def build_cuda(verbose: bool = True, checked: bool = False) -> str:
+# Sources of a library that holds one model family's kernels only (``build_cuda(part=...)``): a first start
+# on a fresh checkout compiles what that family needs.
+PARTS = {
+    "latent": ["elementwise", "gemm_tcgen05", "gemm_f32", "norm_conv", "latent_attention", "sampling"],
+}
+
+
+def part_lib(part: str) -> str:
+    return os.path.join(OPS, f"libmsgl_cuda_{part}.so")
+
+
+def build_cuda(verbose: bool = True, checked: bool = False, part: Optional[str] = None) -> str:
     os.makedirs(OBJ, exist_ok=True)
     nvcc = _nvcc()
     flags = NVCC_FLAGS + (["-DMSGL_CHECK_BOUNDS=1"] if checked else [])
-    out_lib = CHECKED_LIB if checked else CUDA_LIB
+    out_lib = part_lib(part) if part else CHECKED_LIB if checked else CUDA_LIB
     variant = ".chk" if checked else ""
-    sources = sorted(os.path.join(CSRC, f) for f in os.listdir(CSRC) if f.endswith(".cu"))
+    sources = sorted(os.path.join(CSRC, f) for f in os.listdir(CSRC) if f.endswith(".cu")
+                     and (part is None or f[:-3] in PARTS[part]))
     headers = _headers()
     jobs, objs = [], []
     for src in sources:
@@ -91,6 +107,8 @@ def build_cuda(verbose: bool = True, checked: bool = False) -> str:
                  os.path.join(OBJ, f"link{variant}.log"))
         with open(stamp_file, "w") as fh:
             fh.write(stamp)
+    if part:
+        return out_lib
     # drop stale objects
     keep = {os.path.basename(o) for o in objs}
     for f in os.listdir(OBJ):

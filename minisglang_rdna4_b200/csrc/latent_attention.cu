@@ -1,0 +1,562 @@
+// Latent attention: every query head attends to one latent row per position that is key and value
+// at once ([pages, page_size, R] of one layer of the latent pool), causal, with a sliding window.
+//
+//   latent_norm_store_kernel   RMS norm of this step's latents, into their pool slots
+//   head_gemm_kernel           per-head projections into and out of the latent space
+//   latent_attention_kernel    bf16: 16 / 32 / 64 (position, head) rows per CTA against 64-token tiles
+//                              that are fetched once (cp.async, two stages, through the block table)
+//                              and serve QK^T and PV; warp-level tensor products, fp32 scores,
+//                              softmax and accumulation; optional split of the key range
+//   latent_combine_kernel      merges the ranges of a split
+//   latent_attention_simt_kernel   fp32 pools (and latents wider than the tensor kernel holds)
+//
+// Tiles are absolute (0, 64, ...), so what a row adds up does not depend on how its prompt was cut.
+#include "common.cuh"
+#include "ptx.cuh"
+
+using namespace msgl;
+using namespace msgl::ptx;
+
+namespace {
+
+constexpr float kLog2eL = 1.4426950408889634f;
+
+__device__ __forceinline__ float ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
+// ------------------------------------------------------------------------------------------ store
+template <typename T>
+__global__ void __launch_bounds__(128) latent_norm_store_kernel(const T* __restrict__ c, long long ldc,
+                                                                const float* __restrict__ weight, T* __restrict__ pool,
+                                                                const int32_t* __restrict__ out_loc, int rows, int rank,
+                                                                int width, float eps, long long num_slots) {
+  pdl_enter();
+  const int t = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (t >= rows) return;
+  const T* src = c + (size_t)t * ldc;
+  float s = 0.f;
+  for (int i = lane; i < rank; i += 32) {
+    const float v = to_float(src[i]);
+    s = fmaf(v, v, s);
+  }
+  s = warp_sum(s);
+  const float sc = 1.f / sqrtf(s / (float)rank + eps);
+  const long long slot = out_loc[t];
+  if (MSGL_OOB(slot, num_slots) || slot < 0 || slot >= num_slots) return;
+  T* dst = pool + slot * width;
+  for (int i = lane; i < width; i += 32) dst[i] = from_float<T>(i < rank ? to_float(src[i]) * sc * weight[i] : 0.f);
+}
+
+// ------------------------------------------------------------------------------------------ attention args
+struct LatArgs {
+  const void* q;          // [T, H, R]
+  const void* pool;       // [pages + 1, page_size, R]
+  void* out;              // [T, H, R]
+  const int32_t* block_table;
+  int bt_stride;
+  const int32_t* cu_q;
+  const int32_t* seq_lens;
+  float* ws_o;            // [splits, T * H, R]
+  float* ws_lse;          // [splits, T * H]
+  int H, page_size, num_pages, window, splits, total_rows;   // num_pages includes the scratch page
+  float scale;
+};
+
+__device__ __forceinline__ long long token_slot(const LatArgs& a, const int32_t* bt, int tok) {
+  int col = tok / a.page_size;
+  col = col < a.bt_stride ? col : a.bt_stride - 1;
+  int page = bt[col];
+  (void)MSGL_OOB(page, a.num_pages);
+  page = page < 0 ? 0 : (page >= a.num_pages ? a.num_pages - 1 : page);
+  return (long long)page * a.page_size + tok % a.page_size;
+}
+
+// One warp per (query row, head); lane i holds the latent channels i, i + 32, ...
+template <typename T, int NR>
+__global__ void __launch_bounds__(128) latent_attention_simt_kernel(const LatArgs a, int R) {
+  pdl_enter();
+  const int lane = threadIdx.x & 31;
+  const int b = blockIdx.y;
+  const int q0 = a.cu_q[b], q_len = a.cu_q[b + 1] - q0;
+  const int row = blockIdx.x * 4 + (threadIdx.x >> 5);
+  if (row >= q_len * a.H) return;
+  const int kv_len = a.seq_lens[b];
+  const int pos = kv_len - q_len + row / a.H;
+  const int lo = a.window > 0 ? max(0, pos - a.window + 1) : 0;
+  const size_t off = ((size_t)q0 * a.H + row) * R;
+  const T* q = reinterpret_cast<const T*>(a.q) + off;
+  const T* pool = reinterpret_cast<const T*>(a.pool);
+  const int32_t* bt = a.block_table + (size_t)b * a.bt_stride;
+  float qr[NR], o[NR];
+#pragma unroll
+  for (int i = 0; i < NR; ++i) {
+    const int c = lane + 32 * i;
+    qr[i] = c < R ? to_float(q[c]) * a.scale : 0.f;
+    o[i] = 0.f;
+  }
+  float m = -INFINITY, l = 0.f;
+  for (int tok = lo; tok <= pos; ++tok) {
+    const T* k = pool + token_slot(a, bt, tok) * R;
+    float kr[NR], s = 0.f;
+#pragma unroll
+    for (int i = 0; i < NR; ++i) {
+      const int c = lane + 32 * i;
+      kr[i] = c < R ? to_float(k[c]) : 0.f;
+      s = fmaf(qr[i], kr[i], s);
+    }
+    s = warp_sum(s);
+    const float mn = fmaxf(m, s);
+    const float al = expf(m - mn), p = expf(s - mn);
+    m = mn;
+    l = fmaf(l, al, p);
+#pragma unroll
+    for (int i = 0; i < NR; ++i) o[i] = fmaf(o[i], al, p * kr[i]);
+  }
+  T* out = reinterpret_cast<T*>(a.out) + off;
+  const float inv = l > 0.f ? 1.f / l : 0.f;
+#pragma unroll
+  for (int i = 0; i < NR; ++i) {
+    const int c = lane + 32 * i;
+    if (c < R) out[c] = from_float<T>(o[i] * inv);
+  }
+}
+
+// ------------------------------------------------------------------------------------------ tensor-core pieces
+__device__ __forceinline__ void ldm_x4(uint32_t addr, uint32_t (&r)[4]) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+__device__ __forceinline__ void ldm_x4_trans(uint32_t addr, uint32_t (&r)[4]) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+__device__ __forceinline__ void mma_bf16(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+               : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+               : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+// 16 bytes global -> shared; bytes past ``valid`` (0 or 16) are zero-filled without being read
+__device__ __forceinline__ void cp16(uint32_t dst, const void* src, bool valid) {
+  const int n = valid ? 16 : 0;
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(n) : "memory");
+}
+__device__ __forceinline__ void cp_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N> __device__ __forceinline__ void cp_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
+__device__ __forceinline__ uint32_t pack_bf(float a, float b) {
+  __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
+  return *reinterpret_cast<uint32_t*>(&h);
+}
+// byte offset of 16-byte chunk c of row r in a tile of `chunks` chunks per row (chunks a multiple of 8)
+__device__ __forceinline__ uint32_t swz(int r, int c, int chunks) {
+  return (uint32_t)(r * chunks + (c ^ (r & 7))) * 16u;
+}
+
+// ------------------------------------------------------------------------------------------ per-head GEMM
+// out[t, h, n] = sum_k x[t, h, k] w[h, n, k]. 64 rows x 64 columns per CTA, K in panels of 64, two stages;
+// four warps, each 16 rows x 64 columns.
+struct HeadGemmArgs {
+  const __nv_bfloat16* x;
+  long long ldx, hx;      // element strides of t and h
+  const __nv_bfloat16* w; // [H, N, K]
+  __nv_bfloat16* out;
+  long long ldo, ho;
+  int T, N, K, static_weights;
+};
+
+__global__ void __launch_bounds__(128) head_gemm_kernel(const HeadGemmArgs a) {
+  __shared__ __align__(128) uint8_t smem[2][2][64 * 128];
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int n0 = blockIdx.x * 64, h = blockIdx.y, t0 = blockIdx.z * 64;
+  const int panels = (a.K + 63) / 64;
+  const __nv_bfloat16* xh = a.x + (long long)h * a.hx;
+  const __nv_bfloat16* wh = a.w + (long long)h * a.N * a.K;
+  auto load = [&](int p, int s, bool weights) {
+    const uint32_t dst = smem_u32(smem[s][weights]);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int id = tid + i * 128, r = id >> 3, c = id & 7, k = p * 64 + c * 8;
+      if (weights) {
+        const bool ok = n0 + r < a.N && k < a.K;
+        cp16(dst + swz(r, c, 8), ok ? wh + (long long)(n0 + r) * a.K + k : wh, ok);
+      } else {
+        const bool ok = t0 + r < a.T && k < a.K;
+        cp16(dst + swz(r, c, 8), ok ? xh + (long long)(t0 + r) * a.ldx + k : xh, ok);
+      }
+    }
+  };
+  if (a.static_weights) load(0, 0, true);   // weights no earlier kernel writes: fetched ahead of the dependency
+  pdl_enter();
+  if (!a.static_weights) load(0, 0, true);
+  load(0, 0, false);
+  cp_commit();
+  float acc[8][4] = {};
+  for (int p = 0; p < panels; ++p) {
+    if (p + 1 < panels) {
+      load(p + 1, (p + 1) & 1, true);
+      load(p + 1, (p + 1) & 1, false);
+    }
+    cp_commit();
+    cp_wait<1>();
+    __syncthreads();
+    const uint32_t as = smem_u32(smem[p & 1][0]), bs = smem_u32(smem[p & 1][1]);
+    uint32_t af[4][4];
+#pragma unroll
+    for (int kk = 0; kk < 4; ++kk) ldm_x4(as + swz(warp * 16 + (lane & 15), kk * 2 + (lane >> 4), 8), af[kk]);
+#pragma unroll
+    for (int nb = 0; nb < 8; ++nb) {
+#pragma unroll
+      for (int half = 0; half < 2; ++half) {
+        uint32_t bf[4];
+        ldm_x4(bs + swz(nb * 8 + (lane & 7), half * 4 + (lane >> 3), 8), bf);
+        mma_bf16(acc[nb], af[half * 2], bf[0], bf[1]);
+        mma_bf16(acc[nb], af[half * 2 + 1], bf[2], bf[3]);
+      }
+    }
+    __syncthreads();
+  }
+  const int r = t0 + warp * 16 + (lane >> 2), col = n0 + (lane & 3) * 2;
+  __nv_bfloat16* o = a.out + (long long)h * a.ho;
+#pragma unroll
+  for (int nb = 0; nb < 8; ++nb) {
+    const int n = col + nb * 8;
+    if (n >= a.N) break;
+    if (r < a.T) *reinterpret_cast<uint32_t*>(o + (long long)r * a.ldo + n) = pack_bf(acc[nb][0], acc[nb][1]);
+    if (r + 8 < a.T) *reinterpret_cast<uint32_t*>(o + (long long)(r + 8) * a.ldo + n) = pack_bf(acc[nb][2], acc[nb][3]);
+  }
+}
+
+// ------------------------------------------------------------------------------------------ attention
+// NP: latent panels of 64 channels (R = 64 NP). WM row groups of 16 x WN = 8 / WM column groups: a warp
+// computes 16 rows x (64 / WN) keys of S and 16 rows x (R / WN) channels of O.
+template <int NP, int WM>
+__global__ void __launch_bounds__(256) latent_attention_kernel(const LatArgs a) {
+  pdl_enter();
+  constexpr int R = NP * 64, WN = 8 / WM, MT = 16 * WM, TK = 64;
+  constexpr int CH = R / 8;                      // 16-byte chunks per row
+  constexpr int NS = TK / WN / 8;                // key blocks of 8 per warp
+  constexpr int NO = R / WN / 8;                 // channel blocks of 8 per warp
+  constexpr int Q_BYTES = MT * R * 2, C_BYTES = TK * R * 2;
+  extern __shared__ __align__(128) uint8_t smem[];
+  uint8_t* base = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem) + 127) & ~uintptr_t(127));
+  const uint32_t q_s = smem_u32(base), c_s = q_s + Q_BYTES, p_s = c_s + 2 * C_BYTES;
+  float* red = reinterpret_cast<float*>(base + Q_BYTES + 2 * C_BYTES + MT * 128);   // [WN][MT]
+
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int wm = warp / WN, wn = warp % WN;
+  const int b = blockIdx.y, split = blockIdx.z;
+  const int q0 = a.cu_q[b], q_len = a.cu_q[b + 1] - q0;
+  const int n_rows = q_len * a.H;
+  const int row0 = (int)(gridDim.x - 1 - blockIdx.x) * MT;      // late (long) tiles first
+  if (row0 >= n_rows) return;
+  const int row1 = min(row0 + MT, n_rows);
+  const int kv_len = a.seq_lens[b];
+  const int pos_first = kv_len - q_len + row0 / a.H, pos_last = kv_len - q_len + (row1 - 1) / a.H;
+  const int kv_lo = a.window > 0 ? max(0, pos_first - a.window + 1) : 0;
+  const int tile_lo = kv_lo / TK, tiles_all = pos_last / TK + 1 - tile_lo;
+  const int per = (tiles_all + a.splits - 1) / a.splits;
+  const int t_begin = tile_lo + split * per;
+  const int n_tiles = max(0, min(tile_lo + tiles_all, t_begin + per) - t_begin);
+  const __nv_bfloat16* pool = reinterpret_cast<const __nv_bfloat16*>(a.pool);
+  const int32_t* bt = a.block_table + (size_t)b * a.bt_stride;
+
+  auto load_tile = [&](int t) {
+    const uint32_t dst = c_s + (t & 1) * C_BYTES;
+    const int tok0 = (t_begin + t) * TK;
+    for (int id = tid; id < TK * CH; id += 256) {
+      const int r = id / CH, c = id % CH, tok = tok0 + r;
+      const bool ok = tok < kv_len;
+      const __nv_bfloat16* src = ok ? pool + token_slot(a, bt, tok) * R + c * 8 : pool;
+      cp16(dst + swz(r, c, CH), src, ok);
+    }
+  };
+  {
+    const __nv_bfloat16* q = reinterpret_cast<const __nv_bfloat16*>(a.q) + ((size_t)q0 * a.H + row0) * R;
+    for (int id = tid; id < MT * CH; id += 256) {
+      const int r = id / CH, c = id % CH;
+      const bool ok = row0 + r < row1;
+      cp16(q_s + swz(r, c, CH), ok ? q + (size_t)r * R + c * 8 : q, ok);
+    }
+  }
+  if (n_tiles > 0) load_tile(0);
+  cp_commit();
+
+  // this thread's two rows of the 16-row group
+  const int ra = wm * 16 + (lane >> 2), rb = ra + 8;
+  const int pa = kv_len - q_len + min(row0 + ra, row1 - 1) / a.H, pb = kv_len - q_len + min(row0 + rb, row1 - 1) / a.H;
+  const int lo_a = a.window > 0 ? pa - a.window + 1 : 0, lo_b = a.window > 0 ? pb - a.window + 1 : 0;
+  const float sc = a.scale * kLog2eL;
+  float o[NO][4];
+#pragma unroll
+  for (int i = 0; i < NO; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
+  float m_a = -INFINITY, m_b = -INFINITY, l_a = 0.f, l_b = 0.f;
+
+  for (int t = 0; t < n_tiles; ++t) {
+    cp_wait<0>();
+    __syncthreads();                              // tile t has landed; everyone is done with tile t - 1
+    if (t + 1 < n_tiles) load_tile(t + 1);
+    cp_commit();
+    const uint32_t cb = c_s + (t & 1) * C_BYTES;
+    float s[NS][4];
+#pragma unroll
+    for (int i = 0; i < NS; ++i) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.f;
+#pragma unroll 4
+    for (int kk = 0; kk < R / 32; ++kk) {
+      uint32_t a0[4], a1[4];
+      ldm_x4(q_s + swz(wm * 16 + (lane & 15), kk * 4 + (lane >> 4), CH), a0);
+      ldm_x4(q_s + swz(wm * 16 + (lane & 15), kk * 4 + 2 + (lane >> 4), CH), a1);
+#pragma unroll
+      for (int nb = 0; nb < NS; ++nb) {
+        uint32_t bf[4];
+        ldm_x4(cb + swz(wn * (TK / WN) + nb * 8 + (lane & 7), kk * 4 + (lane >> 3), CH), bf);
+        mma_bf16(s[nb], a0, bf[0], bf[1]);
+        mma_bf16(s[nb], a1, bf[2], bf[3]);
+      }
+    }
+    const int tok0 = (t_begin + t) * TK + wn * (TK / WN) + (lane & 3) * 2;
+    float mx_a = -INFINITY, mx_b = -INFINITY;
+#pragma unroll
+    for (int nb = 0; nb < NS; ++nb)
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const int tok = tok0 + nb * 8 + e;
+        const float va = tok <= pa && tok >= lo_a ? s[nb][e] * sc : -INFINITY;
+        const float vb = tok <= pb && tok >= lo_b ? s[nb][2 + e] * sc : -INFINITY;
+        s[nb][e] = va;
+        s[nb][2 + e] = vb;
+        mx_a = fmaxf(mx_a, va);
+        mx_b = fmaxf(mx_b, vb);
+      }
+    mx_a = fmaxf(mx_a, __shfl_xor_sync(0xffffffffu, mx_a, 1));
+    mx_a = fmaxf(mx_a, __shfl_xor_sync(0xffffffffu, mx_a, 2));
+    mx_b = fmaxf(mx_b, __shfl_xor_sync(0xffffffffu, mx_b, 1));
+    mx_b = fmaxf(mx_b, __shfl_xor_sync(0xffffffffu, mx_b, 2));
+    if ((lane & 3) == 0) {
+      red[wn * MT + ra] = mx_a;
+      red[wn * MT + rb] = mx_b;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int w = 0; w < WN; ++w) {
+      mx_a = fmaxf(mx_a, red[w * MT + ra]);
+      mx_b = fmaxf(mx_b, red[w * MT + rb]);
+    }
+    const float mn_a = fmaxf(m_a, mx_a), mn_b = fmaxf(m_b, mx_b);
+    const float ms_a = mn_a == -INFINITY ? 0.f : mn_a, ms_b = mn_b == -INFINITY ? 0.f : mn_b;
+    const float al_a = ex2(m_a - ms_a), al_b = ex2(m_b - ms_b);
+    m_a = mn_a;
+    m_b = mn_b;
+    float sum_a = 0.f, sum_b = 0.f;
+#pragma unroll
+    for (int nb = 0; nb < NS; ++nb) {
+      const float p0 = ex2(s[nb][0] - ms_a), p1 = ex2(s[nb][1] - ms_a);
+      const float p2 = ex2(s[nb][2] - ms_b), p3 = ex2(s[nb][3] - ms_b);
+      sum_a += p0 + p1;
+      sum_b += p2 + p3;
+      const int chunk = wn * NS + nb, in = (lane & 3) * 4;
+      *reinterpret_cast<uint32_t*>(base + (p_s - q_s) + swz(ra, chunk, 8) + in) = pack_bf(p0, p1);
+      *reinterpret_cast<uint32_t*>(base + (p_s - q_s) + swz(rb, chunk, 8) + in) = pack_bf(p2, p3);
+    }
+    l_a = fmaf(l_a, al_a, sum_a);
+    l_b = fmaf(l_b, al_b, sum_b);
+    if (__any_sync(0xffffffffu, al_a != 1.f || al_b != 1.f)) {
+#pragma unroll
+      for (int i = 0; i < NO; ++i) {
+        o[i][0] *= al_a; o[i][1] *= al_a;
+        o[i][2] *= al_b; o[i][3] *= al_b;
+      }
+    }
+    __syncthreads();
+    uint32_t pf[4][4];
+#pragma unroll
+    for (int kk = 0; kk < 4; ++kk) ldm_x4(p_s + swz(wm * 16 + (lane & 15), kk * 2 + (lane >> 4), 8), pf[kk]);
+#pragma unroll
+    for (int nb = 0; nb < NO; ++nb) {
+      const int chunk = wn * NO + nb;
+#pragma unroll
+      for (int half = 0; half < 2; ++half) {
+        uint32_t bf[4];
+        ldm_x4_trans(cb + swz(half * 32 + lane, chunk, CH), bf);
+        mma_bf16(o[nb], pf[half * 2], bf[0], bf[1]);
+        mma_bf16(o[nb], pf[half * 2 + 1], bf[2], bf[3]);
+      }
+    }
+  }
+  cp_wait<0>();
+
+  // row sums: quads, then the column groups (every warp kept the sum of its own keys)
+  l_a += __shfl_xor_sync(0xffffffffu, l_a, 1);
+  l_a += __shfl_xor_sync(0xffffffffu, l_a, 2);
+  l_b += __shfl_xor_sync(0xffffffffu, l_b, 1);
+  l_b += __shfl_xor_sync(0xffffffffu, l_b, 2);
+  __syncthreads();
+  if ((lane & 3) == 0) {
+    red[wn * MT + ra] = l_a;
+    red[wn * MT + rb] = l_b;
+  }
+  __syncthreads();
+  l_a = l_b = 0.f;
+#pragma unroll
+  for (int w = 0; w < WN; ++w) {
+    l_a += red[w * MT + ra];
+    l_b += red[w * MT + rb];
+  }
+  const float inv_a = l_a > 0.f ? 1.f / l_a : 0.f, inv_b = l_b > 0.f ? 1.f / l_b : 0.f;
+  const size_t row_base = (size_t)q0 * a.H + row0;
+  const bool ok_a = row0 + ra < row1, ok_b = row0 + rb < row1;
+  const int col = wn * (R / WN) + (lane & 3) * 2;
+  if (a.splits == 1) {
+    __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(a.out) + row_base * R;
+#pragma unroll
+    for (int nb = 0; nb < NO; ++nb) {
+      if (ok_a) *reinterpret_cast<uint32_t*>(out + (size_t)ra * R + col + nb * 8) = pack_bf(o[nb][0] * inv_a, o[nb][1] * inv_a);
+      if (ok_b) *reinterpret_cast<uint32_t*>(out + (size_t)rb * R + col + nb * 8) = pack_bf(o[nb][2] * inv_b, o[nb][3] * inv_b);
+    }
+    return;
+  }
+  float* wo = a.ws_o + ((size_t)split * a.total_rows + row_base) * R;
+#pragma unroll
+  for (int nb = 0; nb < NO; ++nb) {
+    if (ok_a) *reinterpret_cast<float2*>(wo + (size_t)ra * R + col + nb * 8) = make_float2(o[nb][0] * inv_a, o[nb][1] * inv_a);
+    if (ok_b) *reinterpret_cast<float2*>(wo + (size_t)rb * R + col + nb * 8) = make_float2(o[nb][2] * inv_b, o[nb][3] * inv_b);
+  }
+  if (wn == 0 && (lane & 3) == 0) {
+    float* lse = a.ws_lse + (size_t)split * a.total_rows + row_base;
+    if (ok_a) lse[ra] = l_a > 0.f ? m_a + log2f(l_a) : -INFINITY;
+    if (ok_b) lse[rb] = l_b > 0.f ? m_b + log2f(l_b) : -INFINITY;
+  }
+}
+
+// One warp per (row, head); R a multiple of 64.
+__global__ void __launch_bounds__(128) latent_combine_kernel(const float* __restrict__ ws_o,
+                                                             const float* __restrict__ ws_lse,
+                                                             __nv_bfloat16* __restrict__ out, int rows, int R,
+                                                             int splits) {
+  pdl_enter();
+  const int row = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (row >= rows) return;
+  float m = -INFINITY;
+  for (int s = 0; s < splits; ++s) m = fmaxf(m, ws_lse[(size_t)s * rows + row]);
+  float total = 0.f;
+  for (int s = 0; s < splits; ++s) total += m == -INFINITY ? 0.f : ex2(ws_lse[(size_t)s * rows + row] - m);
+  const float inv = total > 0.f ? 1.f / total : 0.f;
+  for (int c = lane * 2; c < R; c += 64) {
+    float x = 0.f, y = 0.f;
+    for (int s = 0; s < splits; ++s) {
+      const float w = m == -INFINITY ? 0.f : ex2(ws_lse[(size_t)s * rows + row] - m) * inv;
+      const float2 v = *reinterpret_cast<const float2*>(ws_o + ((size_t)s * rows + row) * R + c);
+      x = fmaf(w, v.x, x);
+      y = fmaf(w, v.y, y);
+    }
+    *reinterpret_cast<uint32_t*>(out + (size_t)row * R + c) = pack_bf(x, y);
+  }
+}
+
+template <int NP, int WM>
+int launch_latent(const LatArgs& a, int B, int max_q, cudaStream_t s) {
+  constexpr int R = NP * 64, MT = 16 * WM, WN = 8 / WM;
+  constexpr int bytes = MT * R * 2 + 2 * 64 * R * 2 + MT * 128 + WN * MT * 4 + 128;
+  static bool set = false;
+  if (!set) {
+    const cudaError_t e = cudaFuncSetAttribute(latent_attention_kernel<NP, WM>,
+                                               cudaFuncAttributeMaxDynamicSharedMemorySize, bytes);
+    if (e != cudaSuccess) {
+      msgl_set_error("latent_attention smem", e);
+      return MSGL_CUDA_ERROR;
+    }
+    set = true;
+  }
+  dim3 grid((max_q * a.H + MT - 1) / MT, B, a.splits);
+  msgl_launch(latent_attention_kernel<NP, WM>, grid, dim3(256), bytes, s, a);
+  MSGL_CHECK_LAUNCH("latent_attention");
+  return MSGL_OK;
+}
+
+template <int NP>
+int launch_latent_rows(const LatArgs& a, int B, int max_q, cudaStream_t s) {
+  const long long rows = (long long)max_q * a.H;
+  if (rows <= 16) return launch_latent<NP, 1>(a, B, max_q, s);
+  if (rows <= 32) return launch_latent<NP, 2>(a, B, max_q, s);
+  return launch_latent<NP, 4>(a, B, max_q, s);
+}
+
+template <typename T>
+int launch_simt(const LatArgs& a, int R, int B, int max_q, cudaStream_t s) {
+  dim3 grid((max_q * a.H + 3) / 4, B);
+  if (R <= 64) msgl_launch(latent_attention_simt_kernel<T, 2>, grid, dim3(128), 0, s, a, R);
+  else if (R <= 128) msgl_launch(latent_attention_simt_kernel<T, 4>, grid, dim3(128), 0, s, a, R);
+  else if (R <= 256) msgl_launch(latent_attention_simt_kernel<T, 8>, grid, dim3(128), 0, s, a, R);
+  else if (R <= 512) msgl_launch(latent_attention_simt_kernel<T, 16>, grid, dim3(128), 0, s, a, R);
+  else if (R <= 1024) msgl_launch(latent_attention_simt_kernel<T, 32>, grid, dim3(128), 0, s, a, R);
+  else return MSGL_BAD_ARG;
+  MSGL_CHECK_LAUNCH("latent_attention_simt");
+  return MSGL_OK;
+}
+
+}  // namespace
+
+MSGL_API int msgl_latent_norm_store(const void* c, long long ldc, const void* weight, void* pool, const void* out_loc,
+                                    int rows, int rank, int width, float eps, long long num_slots, int dtype,
+                                    cudaStream_t stream) {
+  if (rows <= 0) return rows == 0 ? MSGL_OK : MSGL_BAD_ARG;
+  if (rank <= 0 || rank > width) return MSGL_BAD_ARG;
+  dim3 grid((rows + 3) / 4);
+#define STORE(T)                                                                                                    \
+  msgl_launch(latent_norm_store_kernel<T>, grid, dim3(128), 0, stream, (const T*)c, ldc, (const float*)weight,      \
+              (T*)pool, (const int32_t*)out_loc, rows, rank, width, eps, num_slots)
+  if (dtype == MSGL_BF16) STORE(__nv_bfloat16);
+  else if (dtype == MSGL_F32) STORE(float);
+  else return MSGL_BAD_ARG;
+#undef STORE
+  MSGL_CHECK_LAUNCH("latent_norm_store");
+  return MSGL_OK;
+}
+
+MSGL_API int msgl_head_gemm(const void* x, long long ldx, long long hx, const void* w, void* out, long long ldo,
+                            long long ho, int T, int H, int N, int K, int static_weights, cudaStream_t stream) {
+  if (T <= 0) return T == 0 ? MSGL_OK : MSGL_BAD_ARG;
+  if (H <= 0 || H > 65535 || N % 8 || K % 8 || ldx % 8 || hx % 8 || ldo % 2 || ho % 2 || (uintptr_t)x % 16 ||
+      (uintptr_t)w % 16 || (uintptr_t)out % 4 || T > 65535 * 64)
+    return MSGL_BAD_ARG;
+  HeadGemmArgs a{(const __nv_bfloat16*)x, ldx, hx, (const __nv_bfloat16*)w, (__nv_bfloat16*)out, ldo, ho, T, N, K, static_weights};
+  dim3 grid((N + 63) / 64, H, (T + 63) / 64);
+  msgl_launch(head_gemm_kernel, grid, dim3(128), 0, stream, a);
+  MSGL_CHECK_LAUNCH("head_gemm");
+  return MSGL_OK;
+}
+
+MSGL_API int msgl_latent_attention(const void* q, const void* pool, void* out, const void* block_table, int bt_stride,
+                                   const void* cu_q, const void* seq_lens, void* ws_o, void* ws_lse, int B, int total_q,
+                                   int max_q, int H, int R, int page_size, int num_pages, int window, int splits,
+                                   float scale, int dtype, cudaStream_t stream) {
+  if (B <= 0 || total_q <= 0) return B == 0 || total_q == 0 ? MSGL_OK : MSGL_BAD_ARG;
+  if (max_q <= 0 || H <= 0 || R % 64 || page_size <= 0 || num_pages <= 0 || B > 65535 || splits < 1 || bt_stride < 1 ||
+      (uintptr_t)q % 16 || (uintptr_t)pool % 16 || (uintptr_t)out % 16)
+    return MSGL_BAD_ARG;
+  LatArgs a{q, pool, out, (const int32_t*)block_table, bt_stride, (const int32_t*)cu_q, (const int32_t*)seq_lens,
+            (float*)ws_o, (float*)ws_lse, H, page_size, num_pages, window, splits, total_q * H, scale};
+  if (dtype == MSGL_F32) return launch_simt<float>(a, R, B, max_q, stream);
+  if (dtype != MSGL_BF16) return MSGL_BAD_ARG;
+  if (R > 512) {
+    a.splits = 1;
+    if (splits > 1) return MSGL_BAD_ARG;
+    return launch_simt<__nv_bfloat16>(a, R, B, max_q, stream);
+  }
+  if (splits > 1 && (ws_o == nullptr || ws_lse == nullptr)) return MSGL_BAD_ARG;
+  int rc;
+  switch (R / 64) {
+    case 1: rc = launch_latent_rows<1>(a, B, max_q, stream); break;
+    case 2: rc = launch_latent_rows<2>(a, B, max_q, stream); break;
+    case 3: rc = launch_latent_rows<3>(a, B, max_q, stream); break;
+    case 4: rc = launch_latent_rows<4>(a, B, max_q, stream); break;
+    case 8: rc = launch_latent_rows<8>(a, B, max_q, stream); break;
+    default: return MSGL_BAD_ARG;
+  }
+  if (rc != MSGL_OK || splits == 1) return rc;
+  msgl_launch(latent_combine_kernel, dim3((total_q * H + 3) / 4), dim3(128), 0, stream, (const float*)ws_o,
+              (const float*)ws_lse, (__nv_bfloat16*)out, total_q * H, R, splits);
+  MSGL_CHECK_LAUNCH("latent_combine");
+  return MSGL_OK;
+}

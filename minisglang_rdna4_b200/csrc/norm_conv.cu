@@ -261,14 +261,14 @@ int norm_conv_typed(NormConvArgs a, int B, int max_q, cudaStream_t s) {
   const bool vec = a.width % 4 == 0 && a.cols % 4 == 0 && a.ldd % 4 == 0 && (uintptr_t)a.delta % 16 == 0;
   const int per = vec ? 4 : 1;
   const int groups = (a.cols + per - 1) / per;
-  const int threads = groups >= 1024 ? 1024 : (groups + 31) / 32 * 32;
-  const int nc = (groups + threads - 1) / threads;
+  const int nc = (groups + 1023) / 1024;
+  const int threads = ((groups + nc - 1) / nc + 31) / 32 * 32;
   if (vec) {
     if (nc == 1) launch_norm_conv<T, 4, 1>(a, grid, threads, s);
     else if (nc == 2) launch_norm_conv<T, 4, 2>(a, grid, threads, s);
     else return MSGL_BAD_ARG;
   } else {
-    if (nc <= 1) launch_norm_conv<T, 1, 1>(a, grid, threads, s);
+    if (nc == 1) launch_norm_conv<T, 1, 1>(a, grid, threads, s);
     else if (nc <= 4) launch_norm_conv<T, 1, 4>(a, grid, threads, s);
     else return MSGL_BAD_ARG;
   }

@@ -16,10 +16,21 @@ LIB_PATH = os.path.join(_HERE, "libmsgl_cuda.so")
 CHECKED_LIB_PATH = os.path.join(_HERE, "libmsgl_cuda_checked.so")
 
 
+# a library with one model family's kernels (build.PARTS), used where the full one was not built
+_part: Optional[str] = None
+
+
+def use_part(path: str) -> None:
+    global _part
+    _part = path
+
+
 def _wanted_lib() -> str:
     flag = (os.environ.get("MSGL_CHECK_BOUNDS") or os.environ.get("MINISGL_CHECK_BOUNDS") or "").strip().lower()
     if flag in ("1", "true", "yes", "on") and os.path.exists(CHECKED_LIB_PATH):
         return CHECKED_LIB_PATH
+    if _part is not None and not os.path.exists(LIB_PATH):
+        return _part
     return LIB_PATH
 
 c_p = ctypes.c_void_p

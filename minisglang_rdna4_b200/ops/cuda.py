@@ -570,6 +570,10 @@ def gemm(x, w, bias=None, out_dtype=None, bn=0, max_ctas=0):
     if x2.stride(1) != 1:
         x2 = x2.contiguous()
     kind = KIND_BF16 if x2.dtype == torch.bfloat16 else KIND_F16
+    if x2.dtype == torch.float32 and w.dtype == torch.float32:
+        if bias is not None:
+            raise NotImplementedError("gemm: no bias in the fp32 form")
+        return gemm_f32(x2, w).view(*shape[:-1], w.shape[0])
     if w.dtype != x2.dtype:
         raise TypeError(f"gemm: activation {x2.dtype} vs weight {w.dtype}")
     n, k = w.shape
@@ -729,6 +733,8 @@ def gemm_static_weights(on) -> int:
     (written long before the kernels in flight): the decode GEMMs then fetch their first weight
     tiles while the kernel ahead of them is still running (1), and also request the rest of their
     first work item's weight stream into L2 (2). Returns the previous setting."""
+    global STATIC_WEIGHTS
+    STATIC_WEIGHTS = bool(on)
     return int(lib().msgl_gemm_static_weights(int(on)))
 
 
@@ -892,4 +898,139 @@ def rms_norm_gated(x, z, w, eps):
     check(lib().msgl_rms_norm_gated(_p(x), _p(z), z.stride(0), heads, _p(w), _p(out), t * heads, d, eps, _dt(x),
                                     _stream()), "rms_norm_gated")
     _count("rms_norm_gated", "rms_norm_gated_kernel")
+    return out
+
+
+# ------------------------------------------------------------------------------------------ fp32 GEMM
+def _bind_latent():
+    from ._lib import bind, c_f, c_i, c_ll, c_p
+
+    if hasattr(_bind_latent, "_done"):
+        return
+    bind("msgl_gemm_f32", c_i, [c_p, c_ll, c_ll, c_p, c_ll, c_ll, c_p, c_ll, c_ll, c_i, c_i, c_i, c_i, c_p])
+    bind("msgl_embed_positions", c_i, [c_p] * 5 + [c_i] * 6 + [c_p])
+    bind("msgl_norm_conv", c_i, [c_p, c_p, c_p, c_i, c_ll, c_ll, c_p, c_f] + [c_p] * 8 + [c_i] * 7 + [c_p])
+    bind("msgl_gelu_erf", c_i, [c_p, c_ll, c_p, c_ll, c_i, c_i, c_i, c_p])
+    bind("msgl_latent_norm_store", c_i, [c_p, c_ll, c_p, c_p, c_p, c_i, c_i, c_i, c_f, c_ll, c_i, c_p])
+    bind("msgl_head_gemm", c_i, [c_p, c_ll, c_ll, c_p, c_p, c_ll, c_ll, c_i, c_i, c_i, c_i, c_i, c_p])
+    bind("msgl_latent_attention", c_i, [c_p, c_p, c_p, c_p, c_i] + [c_p] * 4 + [c_i] * 9 + [c_f, c_i, c_p])
+    _bind_latent._done = True
+
+
+def gemm_f32(x, w):
+    """``x [M, K] @ w [N, K]^T`` in fp32 on the FMA pipe (no tensor-core mode)."""
+    _bind_latent()
+    assert x.dim() == 2 and x.stride(1) == 1 and w.is_contiguous() and w.shape[1] == x.shape[1]
+    out = torch.empty((x.shape[0], w.shape[0]), dtype=torch.float32, device=x.device)
+    check(lib().msgl_gemm_f32(_p(x), x.stride(0), 0, _p(w), w.stride(0), 0, _p(out), out.stride(0), 0, x.shape[0],
+                              w.shape[0], w.shape[1], 1, _stream()), "gemm_f32")
+    _count("gemm_f32", "gemm_f32_kernel")
+    return out
+
+
+# ------------------------------------------------------------------------------------------ fp32 residual, input convolutions
+def embed_positions(ids, weight, pos, positions, vocab_start=0, vocab_len=None):
+    _bind_latent()
+    ids = ids.to(torch.int32) if ids.dtype != torch.int32 else ids
+    n = weight.shape[0] if vocab_len is None else vocab_len
+    out = torch.empty((ids.numel(), weight.shape[1]), dtype=torch.float32, device=weight.device)
+    check(lib().msgl_embed_positions(_p(ids), _p(weight), _p(pos), _p(positions), _p(out), ids.numel(), weight.shape[1],
+                                     vocab_start, n, 0 if pos is None else pos.shape[0], _dt(weight), _stream()),
+          "embed_positions")
+    _count("embed_positions", "embed_positions_kernel")
+    return out
+
+
+def add_scalar_norm_conv(x, delta, gain, eps, w1, w2, state, cu_q, slots, has_state, max_q, out_dtype, out_cols):
+    _bind_latent()
+    assert x.is_contiguous() and x.dtype == torch.float32
+    rows, width = x.shape
+    planes, plane_stride, ldd = 0, 0, 0
+    if isinstance(delta, SplitPartial):
+        delta = delta.planes
+        planes, plane_stride, ldd = delta.shape[0], delta.stride(0), delta.stride(1)
+    elif delta is not None:
+        planes, plane_stride, ldd = 1, 0, delta.stride(0)
+    if delta is not None:
+        assert delta.dtype == torch.float32 and delta.stride(-1) == 1 and delta.shape[-2] == rows
+    x_out = torch.empty_like(x) if delta is not None else x
+    y1 = torch.empty((rows, out_cols), dtype=out_dtype, device=x.device)
+    y2 = torch.empty_like(y1) if w2 is not None else None
+    taps, b = 1, 1
+    if w1 is not None:
+        taps, b = w1.shape[1], cu_q.numel() - 1
+        assert w1.is_contiguous() and w1.dtype == torch.float32 and state.is_contiguous()
+        assert state.dtype == torch.float32 and state.shape[1:] == (width, taps - 1)
+    check(lib().msgl_norm_conv(_p(x), _p(x_out), _p(delta), planes, plane_stride, ldd, _p(gain), eps, _p(w1), _p(w2),
+                               _p(y1), _p(y2), _p(state), _p(cu_q), _p(slots), _p(has_state), rows, width, out_cols,
+                               taps, b, int(max_q), _DT[out_dtype], _stream()), "norm_conv")
+    _count("add_scalar_norm_conv", "norm_conv_kernel")
+    return x_out, y1, y2
+
+
+def gelu_erf(x, out):
+    _bind_latent()
+    assert x.stride(1) == 1 and out.stride(1) == 1 and x.shape == out.shape and x.dtype == out.dtype
+    check(lib().msgl_gelu_erf(_p(x), x.stride(0), _p(out), out.stride(0), x.shape[0], x.shape[1], _dt(x), _stream()),
+          "gelu_erf")
+    _count("gelu_erf", "gelu_erf_kernel")
+    return out
+
+
+# ------------------------------------------------------------------------------------------ latent attention
+STATIC_WEIGHTS = False
+
+
+def latent_norm_store(c, weight, rank, eps, rows, out_loc):
+    _bind_latent()
+    assert c.stride(1) == 1 and rows.is_contiguous() and rows.dtype == c.dtype and weight.dtype == torch.float32
+    check(lib().msgl_latent_norm_store(_p(c), c.stride(0), _p(weight), _p(rows), _p(out_loc), c.shape[0], rank,
+                                       rows.shape[2], eps, rows.shape[0] * rows.shape[1], _dt(c), _stream()),
+          "latent_norm_store")
+    _count("latent_norm_store", "latent_norm_store_kernel")
+
+
+def head_gemm(x, w, out=None):
+    """``x [T, H, K]`` (any row and head stride), ``w [H, N, K]`` -> ``[T, H, N]``."""
+    _bind_latent()
+    t, h, k = x.shape
+    n = w.shape[1]
+    assert x.stride(2) == 1 and w.is_contiguous() and w.shape == (h, n, k) and w.dtype == x.dtype
+    if out is None:
+        out = torch.empty((t, h, n), dtype=x.dtype, device=x.device)
+    assert out.stride(2) == 1 and out.shape == (t, h, n) and out.dtype == x.dtype
+    if x.dtype == torch.float32:
+        check(lib().msgl_gemm_f32(_p(x), x.stride(0), x.stride(1), _p(w), k, n * k, _p(out), out.stride(0),
+                                  out.stride(1), t, n, k, h, _stream()), "head_gemm")
+        _count("head_gemm", "gemm_f32_kernel")
+        return out
+    check(lib().msgl_head_gemm(_p(x), x.stride(0), x.stride(1), _p(w), _p(out), out.stride(0), out.stride(1), t, h, n, k,
+                               int(STATIC_WEIGHTS), _stream()), "head_gemm")
+    _count("head_gemm", "head_gemm_kernel")
+    return out
+
+
+def latent_splits(batch: int, heads: int, up_to: int) -> int:
+    """Key ranges per query tile of a decode step: enough CTAs for the SMs, at least two 64-token tiles each."""
+    tiles = -(-up_to // 64) + 1
+    ctas = batch * -(-heads // 64)
+    return int(max(1, min(296 // max(ctas, 1), tiles // 2, 16)))
+
+
+def latent_attention(q, rows, block_table, cu_q, seq_lens, scale, window, max_q, max_kv, splits=1):
+    _bind_latent()
+    t, h, r = q.shape
+    assert q.is_contiguous() and rows.is_contiguous() and rows.shape[2] == r and rows.dtype == q.dtype
+    out = torch.empty_like(q)
+    if q.dtype == torch.float32 or r > 512:
+        splits = 1
+    ws_o = ws_l = None
+    if splits > 1:
+        ws_o = torch.empty((splits, t * h, r), dtype=torch.float32, device=q.device)
+        ws_l = torch.empty((splits, t * h), dtype=torch.float32, device=q.device)
+    check(lib().msgl_latent_attention(
+        _p(q), _p(rows), _p(out), _p(block_table), block_table.stride(0), _p(cu_q), _p(seq_lens), _p(ws_o), _p(ws_l),
+        seq_lens.numel(), t, int(max_q), h, r, rows.shape[1], rows.shape[0], int(window), splits, float(scale), _dt(q),
+        _stream()), "latent_attention")
+    _count("latent_attention", "latent_attention_kernel", 2 if splits > 1 else 1)
     return out

@@ -1,0 +1,169 @@
+"""Kernels of the Mitilix design against plain fp32 restatements of the same step."""
+import pytest
+import torch
+
+from minisglang_rdna4_b200 import ops
+from minisglang_rdna4_b200.ops import ref
+
+pytestmark = pytest.mark.gpu
+DEV = "cuda"
+
+
+def _gen(seed=0):
+    return torch.Generator().manual_seed(seed)
+
+
+def _batch(lens, starts, ps, pages, gen):
+    """cu_q, seq_lens, block table over a shuffled page pool, token slots."""
+    cu = torch.tensor([0] + list(torch.tensor(lens).cumsum(0)), dtype=torch.int32)
+    seq = torch.tensor([s + n for s, n in zip(starts, lens)], dtype=torch.int32)
+    width = int((seq.max() + ps - 1) // ps)
+    perm = torch.randperm(pages, generator=gen).to(torch.int32)
+    bt = torch.zeros((len(lens), width), dtype=torch.int32)
+    at = 0
+    for i, s in enumerate(seq.tolist()):
+        n = -(-s // ps)
+        bt[i, :n] = perm[at:at + n]
+        at += n
+    assert at <= pages
+    return cu, seq, bt
+
+
+@pytest.mark.parametrize("width,taps,cols", [(256, 4, 256), (200, 3, 208), (1000, 2, 1008), (97, 5, 112), (64, 1, 64),
+                                             (4096, 4, 4096), (5120, 4, 5120), (96, 12, 96)])
+@pytest.mark.parametrize("dtype", [torch.bfloat16, torch.float32])
+def test_norm_conv(width, taps, cols, dtype):
+    g = _gen(width + taps)
+    lens, has = [1, 2, 40, 1, 16, 17, 3], [1, 1, 0, 0, 1, 1, 0]
+    t = sum(lens)
+    cu = torch.tensor([0] + list(torch.tensor(lens).cumsum(0)), dtype=torch.int32)
+    slots = torch.tensor([3, 0, 7, 5, 1, 2, 6], dtype=torch.int32)
+    has = torch.tensor(has, dtype=torch.int32)
+    x, d = torch.randn(t, width, generator=g), torch.randn(t, cols, generator=g)
+    w1, w2 = (torch.randn(width, taps, generator=g) * 0.5 for _ in range(2))
+    gain = torch.tensor([1.3])
+    state = torch.randn(9, width, taps - 1, generator=g)
+    for delta, two in ((d, True), (None, True), (d, False)):
+        st_ref, st = state.clone(), state.clone().to(DEV)
+        want = ref.add_scalar_norm_conv(x, delta, gain, 1e-5, w1, w2 if two else None, st_ref, cu, slots, has, dtype, cols)
+        got = ops.add_scalar_norm_conv(
+            x.to(DEV), None if delta is None else delta.to(DEV), gain.to(DEV), 1e-5, w1.to(DEV),
+            w2.to(DEV) if two else None, st, cu.to(DEV), slots.to(DEV), has.to(DEV), max(lens), dtype, cols)
+        tol = dict(rtol=1e-5, atol=2e-5) if dtype == torch.float32 else dict(rtol=1e-2, atol=1e-2)
+        torch.testing.assert_close(got[0].cpu(), want[0], rtol=1e-6, atol=1e-6)
+        torch.testing.assert_close(got[1].float().cpu(), want[1].float(), **tol)
+        assert (got[2] is None) == (not two)
+        if two:
+            torch.testing.assert_close(got[2].float().cpu(), want[2].float(), **tol)
+        torch.testing.assert_close(st.cpu(), st_ref, rtol=1e-5, atol=1e-5)
+    # the norm alone, and split-K planes as the added term
+    from minisglang_rdna4_b200.ops.cuda import SplitPartial
+
+    planes = torch.randn(3, t, cols, generator=g)
+    want = ref.add_scalar_norm_conv(x, planes.sum(0), gain, 1e-5, None, None, None, None, None, None, dtype, cols)
+    got = ops.add_scalar_norm_conv(x.to(DEV), SplitPartial(planes.to(DEV), torch.float32), gain.to(DEV), 1e-5, None,
+                                   None, None, None, None, None, 0, dtype, cols)
+    torch.testing.assert_close(got[0].cpu(), want[0], rtol=1e-5, atol=1e-5)
+    torch.testing.assert_close(got[1].float().cpu(), want[1].float(), rtol=1e-2, atol=1e-2)
+
+
+@pytest.mark.parametrize("m,n,k", [(1, 8, 16), (65, 70, 33), (200, 130, 257)])
+def test_gemm_f32(m, n, k):
+    g = _gen(m)
+    a, b = torch.randn(m, k, generator=g), torch.randn(n, k, generator=g)
+    got = ops.gemm(a.to(DEV), b.to(DEV)).cpu()
+    torch.testing.assert_close(got, (a.double() @ b.double().T).float(), rtol=1e-5, atol=2e-5)
+
+
+@pytest.mark.parametrize("t,h,n,k", [(1, 3, 64, 48), (70, 5, 80, 64), (130, 2, 512, 128), (9, 4, 128, 512), (64, 1, 16, 16)])
+@pytest.mark.parametrize("dtype", [torch.bfloat16, torch.float32])
+def test_head_gemm(t, h, n, k, dtype):
+    g = _gen(t)
+    wide = torch.randn(t, h * k + 32, generator=g).to(dtype)
+    w = torch.randn(h, n, k, generator=g).to(dtype)
+    x = wide[:, :h * k].unflatten(1, (h, k))
+    want = torch.einsum("thk,hnk->thn", x.double(), w.double())
+    out = torch.zeros(t, h * n + 16, dtype=dtype, device=DEV)
+    ops.head_gemm(wide.to(DEV)[:, :h * k].unflatten(1, (h, k)), w.to(DEV), out[:, :h * n].unflatten(1, (h, n)))
+    tol = 2e-5 if dtype == torch.float32 else 1e-2
+    torch.testing.assert_close(out[:, :h * n].unflatten(1, (h, n)).double().cpu(), want, rtol=tol, atol=tol * k ** 0.5)
+    assert float(out[:, h * n:].abs().max()) == 0.0
+
+
+def test_gelu_and_embedding():
+    g = _gen(4)
+    x = torch.randn(33, 48, generator=g) * 3
+    for dtype, tol in ((torch.float32, 1e-6), (torch.bfloat16, 1e-2)):
+        out = torch.zeros(33, 64, dtype=dtype, device=DEV)
+        ops.gelu_erf(x.to(DEV, dtype), out[:, 16:])
+        want = torch.nn.functional.gelu(x.to(dtype).double())
+        torch.testing.assert_close(out[:, 16:].double().cpu(), want, rtol=tol, atol=tol)
+        emb, pos = torch.randn(50, 40, generator=g).to(dtype), torch.randn(70, 40, generator=g).to(dtype)
+        ids, p = torch.randint(0, 50, (21,), generator=g), torch.randint(0, 70, (21,), generator=g)
+        got = ops.embed_positions(ids.int().to(DEV), emb.to(DEV), pos.to(DEV), p.int().to(DEV))
+        torch.testing.assert_close(got.cpu(), emb[ids].float() + pos[p].float())
+
+
+@pytest.mark.parametrize("rank,width", [(64, 64), (40, 64), (300, 512)])
+def test_latent_norm_store(rank, width):
+    g = _gen(rank)
+    for dtype, tol in ((torch.float32, 1e-5), (torch.bfloat16, 1e-2)):
+        c, w = torch.randn(13, width + 24, generator=g).to(dtype), torch.rand(width, generator=g)
+        loc = torch.randperm(5 * 16, generator=g)[:13].int()
+        pool = torch.zeros(5, 16, width, dtype=dtype)
+        dev = pool.to(DEV)
+        ref.latent_norm_store(c[:, 24:], w, rank, 1e-5, pool, loc)
+        ops.latent_norm_store(c.to(DEV)[:, 24:], w.to(DEV), rank, 1e-5, dev, loc.to(DEV))
+        torch.testing.assert_close(dev.cpu(), pool, rtol=tol, atol=tol)
+
+
+@pytest.mark.parametrize("r", [64, 128, 192, 256, 512, 1024])
+@pytest.mark.parametrize("h,window,ps", [(6, 72, 16), (3, 64, 16), (17, 1, 32), (64, 200, 64), (5, 0, 8)])
+def test_latent_attention(r, h, window, ps):
+    g = _gen(r + h)
+    lens, starts = [1, 70, 2, 1, 33], [300, 0, 129, 63, 90]
+    cu, seq, bt = _batch(lens, starts, ps, 96 if ps == 16 else 200, g)
+    pool = torch.randn(201, ps, r, generator=g)
+    q = torch.randn(sum(lens), h, r, generator=g)
+    # one key far outside its neighbours' scores: a window that is one token off shows
+    for dtype, tol in ((torch.bfloat16, 2e-2), (torch.float32, 1e-4)):
+        qd, pd = q.to(dtype), pool.to(dtype)
+        scale = 2.0 / r ** 0.5
+        want = ref.latent_attention(qd.float(), pd.float(), bt, cu, seq, scale, window)
+        got = ops.latent_attention(qd.to(DEV), pd.to(DEV), bt.to(DEV), cu.to(DEV), seq.to(DEV), scale, window, max(lens),
+                                   int(seq.max()))
+        torch.testing.assert_close(got.float().cpu(), want, rtol=tol, atol=tol)
+
+
+@pytest.mark.parametrize("r,h,window,splits", [(64, 6, 72, 2), (128, 4, 500, 4), (512, 32, 333, 7), (512, 40, 0, 16)])
+def test_latent_attention_decode_splits(r, h, window, splits):
+    g = _gen(splits)
+    starts = [0, 63, 64, 65, 640, 999]
+    cu, seq, bt = _batch([1] * 6, starts, 16, 300, g)
+    pool = torch.randn(301, 16, r, generator=g).bfloat16()
+    q = torch.randn(6, h, r, generator=g).bfloat16()
+    want = ref.latent_attention(q.float(), pool.float(), bt, cu, seq, 0.1, window)
+    got = ops.latent_attention(q.to(DEV), pool.to(DEV), bt.to(DEV), cu.to(DEV), seq.to(DEV), 0.1, window, 1, 1000, splits)
+    torch.testing.assert_close(got.float().cpu(), want, rtol=2e-2, atol=2e-2)
+
+
+@pytest.mark.parametrize("r", [64, 512])
+def test_latent_attention_window_edge(r):
+    """The key at the window's far edge is made to dominate; one token further back must not be seen."""
+    window, kv = 50, 400
+    pool = torch.zeros(26, 16, r)
+    flat = pool.view(-1, r)
+    bt = torch.randperm(25, generator=_gen(1)).int()[None]
+    slot = lambda p: int(bt[0, p // 16]) * 16 + p % 16        # noqa: E731
+    for p in range(kv):
+        flat[slot(p), 1] = 1.0
+    for loud, seen in ((kv - window, True), (kv - window - 1, False)):
+        flat2 = flat.clone()
+        flat2[slot(loud), 0] = 8.0
+        q = torch.zeros(1, 2, r)
+        q[:, :, 0] = 8.0
+        args = [t.to(DEV) for t in (bt, torch.tensor([0, 1], dtype=torch.int32), torch.tensor([kv], dtype=torch.int32))]
+        for splits in (1, 3):
+            got = ops.latent_attention(q.bfloat16().to(DEV), flat2.view_as(pool).bfloat16().to(DEV), *args, 1.0, window, 1,
+                                       kv, splits).float().cpu()
+            assert (float(got[0, 0, 0]) > 7.0) == seen
