@@ -84,6 +84,11 @@ def parse_args():
     ap.add_argument("--no-matched", action="store_true",
                     help="skip the extra bf16-weights / bf16-KV run of this repository that is reported beside "
                          "the quantised number for a like-for-like ratio against the bf16 reference arm")
+    ap.add_argument("--design", default=None, choices=["mitilix"],
+                    help="instead of the workload: prefill / decode throughput and kernel rooflines of this design "
+                         "beside the closest family at equal size (minisglang_rdna4_b200/benchmark/design.py)")
+    ap.add_argument("--size", default="all", choices=["small", "large", "all"], help="with --design")
+    ap.add_argument("--design-part", default="all", choices=["throughput", "kernels", "all"], help="with --design")
     args = ap.parse_args()
     preset = dict(shared_prefix=0, spec="none", spec_draft=4, spec_tree_width=1)
     preset.update(PRESETS[args.config])
@@ -244,6 +249,12 @@ def main() -> None:
     args = parse_args()
     if args.impl == "reference":
         run_reference(args)
+        return
+
+    if args.design:
+        from minisglang_rdna4_b200.benchmark import design
+
+        design.run(args.size, args.design_part, ClockSampler(0))
         return
 
     matched = None
