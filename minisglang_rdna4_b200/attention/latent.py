@@ -1,6 +1,10 @@
 """Attention backend of models that cache latents instead of per-head keys and values
 (``layers/latent_attention.py``). Prefill, portions of prompts, decode and draft verification in one batch: every row
-reads the paged latent pool after the step's latents were stored."""
+reads the paged latent pool after the step's latents were stored.
+
+Two forms of the same sum. Absorbed: queries go into the latent space and attend to the latents themselves; any mix of
+rows. Expanded (16-bit prefill steps on a GPU, ``ops.cuda.LatentPrefillPlan``): per-head keys and values of the latents
+in sight are computed first, which takes fewer operations when a step has many rows, and runs on tcgen05."""
 from __future__ import annotations
 
 from typing import Optional
@@ -13,8 +17,10 @@ from .base import AttnMetadata, BaseAttnBackend
 
 
 class LatentAttentionBackend(BaseAttnBackend):
-    def __init__(self, device, max_seq_len: int, single_split: bool = False) -> None:
+    def __init__(self, layers, device, max_seq_len: int, single_split: bool = False) -> None:
         self.device = torch.device(device)
+        windows = [s.window for s in layers]
+        self.reach = max(windows) if min(windows) > 0 else 0
         self.max_seq_len = max_seq_len
         self.single_split = single_split
 
@@ -23,26 +29,52 @@ class LatentAttentionBackend(BaseAttnBackend):
                          host_seq_lens=None, mask_window: int = 0, mask_swa=None) -> None:
         if mask is not None or not causal:
             raise NotImplementedError("latent attention is causal and takes no mask")
+        plan = None
+        if host_cu_q is not None and batch.is_prefill and not batch.spec_verify and self.device.type == "cuda":
+            from ..env import ENV
+            from ..ops.cuda import LatentPrefillPlan
+
+            if not ENV.DISABLE_TC_PREFILL.value and LatentPrefillPlan.pays(host_cu_q, host_seq_lens, self.reach):
+                plan = LatentPrefillPlan(host_cu_q, host_seq_lens, self.reach, self.device)
         batch.attn_metadata = AttnMetadata(cu_q=cu_q, seq_lens=seq_lens, block_table=block_table, max_q=max_q,
-                                           max_kv=max_kv, decode=max_q == 1)
+                                           max_kv=max_kv, decode=max_q == 1, prefill_plan=plan)
 
     def forward(self, q, layer: int, batch: Batch, *, scale: float, window: int = 0, swa: bool = False):
         raise NotImplementedError("models with a latent pool call latent_forward")
 
-    def latent_forward(self, q, up_k, up_v, row: int, batch: Batch, *, scale: float, window: int, out) -> None:
-        """``q [T, H, dim]``, ``up_k [H, rank, dim]``, ``up_v [H, vdim, rank]`` -> ``out [T, H, vdim]``."""
+    def latent_forward(self, q, up_k, up_v, row: int, batch: Batch, *, scale: float, window: int, out,
+                       expand_k=None) -> None:
+        """``q [T, H, dim]``, ``up_k [H, rank, dim]``, ``up_v [H, vdim, rank]`` -> ``out [T, H, vdim]``. ``expand_k``:
+        ``up_k`` as ``[H * dim, rank]``, where the expanded form may be used."""
         md = batch.attn_metadata
+        if md.prefill_plan is not None and expand_k is not None:
+            from ..ops import cuda as K
+
+            if K.latent_prefill_ok(q.shape[2], up_v.shape[1], scale):
+                K.latent_prefill(q, expand_k, up_v, get_global_ctx().kv_cache.rows(row), row, md.block_table,
+                                 md.prefill_plan, scale, window, out)
+                return
         q_lat = ops.head_gemm(q, up_k)
-        o_lat = ops.latent_attention(q_lat, get_global_ctx().kv_cache.rows(row), md.block_table, md.cu_q, md.seq_lens,
-                                     scale, window, md.max_q, md.max_kv, self._splits(q, md, window))
+        rows = get_global_ctx().kv_cache.rows(row)
+        splits = self._splits(q_lat, md, window)
+        if splits > 1:                        # the value projection merges the key ranges
+            from ..ops import cuda as K
+
+            parts = K.latent_attention(q_lat, rows, md.block_table, md.cu_q, md.seq_lens, scale, window, md.max_q,
+                                       md.max_kv, splits, merge=False)
+            K.head_gemm_combine(parts, up_v, out)
+            return
+        o_lat = ops.latent_attention(q_lat, rows, md.block_table, md.cu_q, md.seq_lens, scale, window, md.max_q,
+                                     md.max_kv)
         ops.head_gemm(o_lat, up_v, out)
 
     def _splits(self, q, md: AttnMetadata, window: int) -> int:
         """Key ranges per query tile of a decode step. Depends on the batch size and on what the window or the pool
         can hold, never on the lengths in the batch: a captured graph and an eager step reduce in the same order."""
-        if not md.decode or self.single_split or not q.is_cuda:
+        if (not md.decode or self.single_split or not q.is_cuda or q.dtype != torch.bfloat16
+                or q.shape[2] > 512):
             return 1
         from ..ops.cuda import latent_splits
 
         reach = min(window, self.max_seq_len) if window > 0 else self.max_seq_len
-        return latent_splits(md.seq_lens.numel(), q.shape[1], up_to=reach)
+        return latent_splits(md.seq_lens.numel(), q.shape[1], q.shape[2], up_to=reach)

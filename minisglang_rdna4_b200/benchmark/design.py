@@ -159,8 +159,8 @@ def kernels(s: Dict) -> List[Dict]:
             seen, distinct = min(win, ctx_len), b * min(win, ctx_len)
         # ---- Mitilix
         x, y = rnd(t, w, dtype=torch.float32), rnd(t, w, dtype=torch.float32)
-        c1, c2 = rnd(w, 4, dtype=torch.float32), rnd(w, 4, dtype=torch.float32)
-        gain, state = torch.ones(1, device=dev), torch.zeros(b, w, 3, device=dev)
+        c1, c2 = rnd(4, w, dtype=torch.float32), rnd(4, w, dtype=torch.float32)
+        gain, state = torch.ones(1, device=dev), torch.zeros(b, 3, w, device=dev)
         has = torch.ones(b, dtype=torch.int32, device=dev)
         us = _time(lambda: ops.add_scalar_norm_conv(x, y, gain, 1e-5, c1, c2, state, cu, slots, has, n, bf, w))
         add("mitilix", "norm_conv", phase, us, t * w * (4 + 4 + 4 + 2 + 2) + 2 * b * w * 12, 0)
@@ -170,29 +170,49 @@ def kernels(s: Dict) -> List[Dict]:
         ctx = Context(page_size=ps)
         ctx.kv_cache = pool
         set_global_ctx(ctx)
-        be = LatentAttentionBackend(dev, MAX_POS)
+        be = LatentAttentionBackend(mitilix_config(s).latent_layers, dev, MAX_POS)
         batch = Batch(reqs=[], phase="prefill" if n > 1 else "decode")
         be.prepare_metadata(batch, bt, cu, seq, n, ctx_len, host_cu_q=cu.cpu().numpy(), host_seq_lens=seq.cpu().numpy())
         q, uk, uv = rnd(t, h, d), rnd(h, r, d), rnd(h, d, r)
         out = torch.empty(t, h, d, dtype=bf, device=dev)
+        uk_rows = uk.transpose(1, 2).reshape(h * d, r).contiguous()
+        ones = torch.ones(r, device=dev)
         lat = rnd(t, r)
-        us = _time(lambda: ops.latent_norm_store(lat, torch.ones(r, device=dev), r, 1e-5, pool.rows(0), loc))
+        us = _time(lambda: ops.latent_norm_store(lat, ones, r, 1e-5, pool.rows(0), loc))
         add("mitilix", "latent_norm_store", phase, us, t * r * 4, 0)
         # all of q -> latent space -> attention -> values: fewest operations of the absorbed and expanded forms
-        us = _time(lambda: be.latent_forward(q, uk, uv, 0, batch, scale=d ** -0.5, window=win, out=out))
+        def forward():
+            if batch.attn_metadata.prefill_plan is not None:
+                batch.attn_metadata.prefill_plan.dense = None
+            be.latent_forward(q, uk, uv, 0, batch, scale=d ** -0.5, window=win, out=out, expand_k=uk_rows)
+
+        us = _time(forward)
         expand = 2 * distinct * r * h * 2 * d + 2 * t * h * seen * 2 * d
         absorb = 2 * 2 * t * h * r * d + 2 * t * h * seen * 2 * r
         add("mitilix", "latent attention (projections in and out included)", phase, us,
             t * h * d * 2 * 2 + distinct * r * 2 + 2 * h * r * d * 2, min(expand, absorb))
         if n == 1:
             q_lat = rnd(t, h, r)
-            sp = be._splits(q, batch.attn_metadata, win)
-            us = _time(lambda: ops.latent_attention(q_lat, pool.rows(0), bt, cu, seq, d ** -0.5, win, n, ctx_len, sp))
+            sp = be._splits(q_lat, batch.attn_metadata, win)
+            us = _time(lambda: K.latent_attention(q_lat, pool.rows(0), bt, cu, seq, d ** -0.5, win, n, ctx_len, sp, merge=sp == 1))
             add("mitilix", "latent_attention", phase, us, t * h * r * 4 + distinct * r * 2, 2 * t * h * seen * 2 * r)
             us = _time(lambda: ops.head_gemm(q, uk))
             add("mitilix", "head_gemm (keys)", phase, us, t * h * (d + r) * 2 + h * r * d * 2, 2 * t * h * r * d)
             us = _time(lambda: ops.head_gemm(q_lat, uv, out))
             add("mitilix", "head_gemm (values)", phase, us, t * h * (d + r) * 2 + h * r * d * 2, 2 * t * h * r * d)
+        else:
+            plan = batch.attn_metadata.prefill_plan
+            dense = plan.dense[1]
+            k_all, vt = K.gemm(dense, uk_rows), torch.empty(h * d, plan.t_pad, dtype=bf, device=dev).normal_()
+            from ..ops._lib import lib
+
+            base = plan.tables.data_ptr()
+            us = _time(lambda: lib().msgl_attn_prefill_pos(
+                q.data_ptr(), q.stride(0), q.stride(1), k_all.data_ptr(), vt.data_ptr(), plan.t_pad, out.data_ptr(),
+                out.stride(0), out.stride(1), base, plan.n_items, t, h, d, d, win, d ** -0.5, 0,
+                torch.cuda.current_stream().cuda_stream))
+            add("mitilix", "expanded attention (window, tcgen05)", phase, us, t * h * d * 2 * 4, 2 * t * h * seen * 2 * d)
+            del k_all, vt
         u, cat = rnd(t, ff), torch.empty(t, h * d + ff, dtype=bf, device=dev)
         us = _time(lambda: ops.gelu_erf(u, cat[:, h * d:]))
         add("mitilix", "gelu_erf", phase, us, t * ff * 4, 0)

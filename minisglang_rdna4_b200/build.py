@@ -71,7 +71,7 @@ def _compile(cmd: List[str], out: str, log: str) -> str:
 # Sources of a library that holds one model family's kernels only (``build_cuda(part=...)``): a first start
 # on a fresh checkout compiles what that family needs.
 PARTS = {
-    "latent": ["elementwise", "gemm_tcgen05", "gemm_f32", "norm_conv", "latent_attention", "sampling"],
+    "latent": ["elementwise", "gemm_tcgen05", "gemm_f32", "norm_conv", "latent_attention", "attention_tc", "sampling"],
 }
 
 

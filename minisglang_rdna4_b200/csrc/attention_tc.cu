@@ -48,7 +48,9 @@ struct TcItem {        // one per (request, block of 128 query positions); eight
   int q_pos0;          // absolute position of the first row
   int kv_off;          // first scratch row of the request (multiple of 128)
   int n_blocks;        // KV blocks of 128 the tile can see
-  int req, pad0, pad1;
+  int req;
+  int kv_pos0;         // absolute position of the first of those blocks (a multiple of 128; 0 without a window)
+  int pad1;
 };
 
 struct TcArgs {
@@ -61,6 +63,10 @@ struct TcArgs {
   const float* v_scale;
   float scale;
   int* status;
+  // position-pair form: one head, 256 consecutive query positions per CTA
+  int window;          // > 0: a row sees the last ``window`` positions, its own included
+  long long ldo, ho;   // element strides of a row and a head of out
+  int v_chunks;        // 16-byte chunks of a value head
 };
 
 __device__ int g_attn_tc_status = 0;
@@ -167,7 +173,9 @@ kv_gather_kernel(const void* __restrict__ k_pool, const void* __restrict__ v_poo
 // ------------------------------------------------------------------------------------------
 // 2. The attention kernel. grid = items x head pairs (heaviest items first), 320 threads.
 // ------------------------------------------------------------------------------------------
-template <typename T>
+// POS: the two tiles of a CTA are consecutive blocks of 128 positions of one head (every head has keys and
+// values of its own, so K / V tiles can only be shared along the positions) instead of two heads.
+template <typename T, bool POS>
 __global__ void __launch_bounds__(kTcThreads, 1)
 attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_constant__ CUtensorMap tma_k,
                        const __grid_constant__ CUtensorMap tma_v, const TcArgs args) {
@@ -180,8 +188,8 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
 
   const int item_idx = blockIdx.x / args.pairs, pair = blockIdx.x - item_idx * args.pairs;
   const TcItem it = args.items[item_idx];
-  const int head0 = pair * 2;
-  const int hk = head0 / (args.Hq / args.Hk);
+  const int head0 = POS ? pair : pair * 2;
+  const int hk = POS ? pair : head0 / (args.Hq / args.Hk);
   const int nb = it.n_blocks;
 
   const uint32_t q_s = s_base + TcSmem::off_q, p_s = s_base + TcSmem::off_p, kv_s = s_base + TcSmem::off_kv;
@@ -231,14 +239,20 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
       mbar_expect_tx(q_full(), 4 * kPanel);
       for (int t = 0; t < 2; ++t)
         for (int p = 0; p < 2; ++p)
-          tma_load_3d(q_s + (t * 2 + p) * kPanel, &tma_q, q_full(), 64 * p, head0 + t, it.q_row0);
+          tma_load_3d(q_s + (t * 2 + p) * kPanel, &tma_q, q_full(), 64 * p, head0 + (POS ? 0 : t),
+                      it.q_row0 + (POS ? t * kTile : 0));
       const int k_row0 = (int)((long long)hk * args.t_cap) + it.kv_off;
       for (int i = 0; i < 2 * nb && !*abort_flag; ++i) {
         const int slot = i % 3, n = i / 3, j = i >> 1;
         if (!mbar_wait(kv_empty(slot), (uint32_t)((n & 1) ^ 1), abort_flag, args.status, 201)) break;
         mbar_expect_tx(kv_full(slot), 2 * kPanel);
         const uint32_t dst = kv_s + slot * 2 * kPanel;
-        if ((i & 1) == 0) {
+        if constexpr (POS) {
+          for (int p = 0; p < 2; ++p) {
+            if ((i & 1) == 0) tma_load_3d(dst + p * kPanel, &tma_k, kv_full(slot), 64 * p, hk, it.kv_off + j * kTile);
+            else tma_load_3d(dst + p * kPanel, &tma_v, kv_full(slot), it.kv_off + j * kTile + 64 * p, 0, hk);
+          }
+        } else if ((i & 1) == 0) {
           tma_load_2d(dst, &tma_k, kv_full(slot), 0, k_row0 + j * kTile);
           tma_load_2d(dst + kPanel, &tma_k, kv_full(slot), 64, k_row0 + j * kTile);
         } else {
@@ -306,8 +320,9 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
     const int t = (warp - 4) >> 2;               // head of the pair
     const int quarter = warp & 3;                // tensor-memory lanes this warp may read
     const int row = quarter * 32 + lane;
-    const int head = head0 + t;
-    const int q_pos = it.q_pos0 + row;
+    const int head = head0 + (POS ? 0 : t);
+    const int tile_pos0 = it.q_pos0 + (POS ? t * kTile : 0);
+    const int q_pos = tile_pos0 + row;
     const uint32_t lane_base = tmem_base + ((uint32_t)(quarter * 32) << 16);
     const uint32_t s_addr = lane_base + t * 128, o_addr = lane_base + 256 + t * 128;
     const uint32_t p_row = p_s + t * 2 * kPanel + row * 128;
@@ -323,8 +338,11 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
     uint32_t s[4][32];
     bool ok = true;
     for (int j = 0; j < nb; ++j) {
-      const int kv0 = j * kTile;
-      const bool masked = kv0 + kTile - 1 > it.q_pos0;   // the block reaches past some row's position
+      const int kv0 = (POS ? it.kv_pos0 : 0) + j * kTile;
+      // the block reaches past some row's position, or starts below some row's window
+      const bool masked = kv0 + kTile - 1 > tile_pos0 ||
+                          (POS && args.window > 0 && kv0 <= tile_pos0 + kTile - 1 - args.window);
+      const int lo = POS && args.window > 0 ? q_pos - args.window : -1;
       if (!mbar_wait(s_full(t), (uint32_t)(j & 1), abort_flag, args.status, 209)) { ok = false; break; }
       tc_fence_after();
 #pragma unroll
@@ -337,7 +355,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
       for (int c = 0; c < 4; ++c) {
 #pragma unroll
         for (int i = 0; i < 32; ++i) {
-          if (masked && kv0 + c * 32 + i > q_pos) s[c][i] = 0xFF800000u;   // -inf
+          if (masked && (kv0 + c * 32 + i > q_pos || (POS && kv0 + c * 32 + i <= lo))) s[c][i] = 0xFF800000u;   // -inf
           mx = fmaxf(mx, __uint_as_float(s[c][i]));
         }
       }
@@ -396,13 +414,17 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
     if (ok && nb > 0 && mbar_wait(o_full(t), (uint32_t)((nb - 1) & 1), abort_flag, args.status, 211)) {
       tc_fence_after();
       const float inv = (l > 0.f ? 1.f / l : 0.f) * (args.v_scale != nullptr ? args.v_scale[hk] : 1.f);
-      T* dst = reinterpret_cast<T*>(args.out) + ((long long)(it.q_row0 + row) * args.Hq + head) * kD;
+      const int out_row = row + (POS ? t * kTile : 0);
+      T* dst = reinterpret_cast<T*>(args.out) +
+               (POS ? (long long)(it.q_row0 + out_row) * args.ldo + head * args.ho
+                    : ((long long)(it.q_row0 + row) * args.Hq + head) * kD);
 #pragma unroll
       for (int c = 0; c < 4; ++c) tmem_ld_32x32b_x32(o_addr + c * 32, s[c]);
       tmem_ld_wait();
-      if (row < it.q_rows) {
+      if (out_row < it.q_rows) {
 #pragma unroll
         for (int c = 0; c < 16; ++c) {
+          if (POS && c >= args.v_chunks) break;
           const uint32_t* o = &s[c >> 2][(c & 3) * 8];
           uint4 v;
           v.x = pack2_tc<T>(__uint_as_float(o[0]) * inv, __uint_as_float(o[1]) * inv);
@@ -435,22 +457,96 @@ bool encode_map(CUtensorMap* map, const void* base, int rank, const cuuint64_t* 
   return true;
 }
 
-template <typename T>
+template <typename T, bool POS>
 int launch_tc(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const TcArgs& a,
               cudaStream_t stream) {
   static bool configured = false;
   if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(attn_prefill_tc_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+    cudaError_t e = cudaFuncSetAttribute(attn_prefill_tc_kernel<T, POS>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                          TcSmem::bytes);
     if (e != cudaSuccess) { msgl_set_error("prefill attention smem attribute", e); return MSGL_CUDA_ERROR; }
     configured = true;
   }
-  msgl_launch(attn_prefill_tc_kernel<T>, dim3(a.n_items * a.pairs), dim3(kTcThreads), TcSmem::bytes, stream, mq, mk, mv, a);
+  msgl_launch(attn_prefill_tc_kernel<T, POS>, dim3(a.n_items * a.pairs), dim3(kTcThreads), TcSmem::bytes, stream, mq, mk, mv, a);
   MSGL_CHECK_LAUNCH("attn_prefill_tc");
   return MSGL_OK;
 }
 
+// Rows of a latent pool ([pages, page_size, R]) a step can see -> dense [t_pad, R]; rows past a request's length are
+// zero. req_info: per request (scratch offset, KV length, absolute position of the first scratch row). One warp per row.
+__global__ void __launch_bounds__(256)
+latent_gather_kernel(const uint4* __restrict__ pool, uint4* __restrict__ out, const int* __restrict__ blk_req,
+                     const int* __restrict__ req_info, const int* __restrict__ block_table, int bt_stride,
+                     int page_size, int num_pages, int chunks, int t_pad) {
+  pdl_enter();
+  const int row = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (row >= t_pad) return;
+  const int req = blk_req[row >> 7];
+  const int tok = row - req_info[3 * req] + req_info[3 * req + 2];
+  const bool in = tok >= 0 && tok < req_info[3 * req + 1];
+  long long src = 0;
+  if (in) {
+    int page = block_table[(long long)req * bt_stride + min(tok / page_size, bt_stride - 1)];
+    (void)MSGL_OOB(page, num_pages);
+    page = page < 0 ? 0 : (page >= num_pages ? num_pages - 1 : page);
+    src = ((long long)page * page_size + tok % page_size) * chunks;
+  }
+  for (int c = lane; c < chunks; c += 32)
+    out[(long long)row * chunks + c] = in ? pool[src + c] : make_uint4(0, 0, 0, 0);
+}
+
 }  // namespace
+
+MSGL_API int msgl_latent_gather(const void* pool, void* out, const void* blk_req, const void* req_info,
+                                const void* block_table, int bt_stride, int page_size, int num_pages, int R, int t_pad,
+                                cudaStream_t stream) {
+  if (t_pad <= 0 || t_pad % 128 || R % 8 || (uintptr_t)pool % 16 || (uintptr_t)out % 16 || page_size <= 0 || bt_stride < 1)
+    return MSGL_BAD_ARG;
+  msgl_launch(latent_gather_kernel, dim3(t_pad / 8), dim3(256), 0, stream, (const uint4*)pool, (uint4*)out,
+              (const int*)blk_req, (const int*)req_info, (const int*)block_table, bt_stride, page_size, num_pages, R / 8,
+              t_pad);
+  MSGL_CHECK_LAUNCH("latent_gather");
+  return MSGL_OK;
+}
+
+// Windowed causal prefill over keys and values of a step in dense scratch, every head with its own: q [total_q, h]
+// heads of dk channels (element strides ldq, hq_stride), k [t_pad, h * dk] row-major, vt [h * dv, t_pad]; out rows of
+// h heads of dv channels (strides ldo, ho). dk and dv up to 128, multiples of 8 (channels up to 128 read as zero).
+MSGL_API int msgl_attn_prefill_pos(const void* q, long long ldq, long long hq_stride, const void* k, const void* vt,
+                                   int t_pad, void* out, long long ldo, long long ho, const void* items, int n_items,
+                                   int total_q, int h, int dk, int dv, int window, float scale, int dtype,
+                                   cudaStream_t stream) {
+  if (n_items == 0 || total_q == 0) return MSGL_OK;
+  if (h <= 0 || t_pad % 128 || dk % 8 || dv % 8 || dk > kD || dv > kD || ldq % 8 || hq_stride % 8 || ldo % 8 || ho % 8 ||
+      (uintptr_t)q % 16 || (uintptr_t)out % 16 || scale <= 0.f || dtype != MSGL_BF16) {
+    msgl_set_error_text("prefill attention: needs bf16 heads of up to 128 channels and a positive scale");
+    return MSGL_BAD_ARG;
+  }
+  CUtensorMap mq, mk, mv;
+  cuuint32_t box[3] = {64, 1, 128};
+  {
+    cuuint64_t dims[3] = {(cuuint64_t)dk, (cuuint64_t)h, (cuuint64_t)total_q};
+    cuuint64_t strides[2] = {(cuuint64_t)hq_stride * 2, (cuuint64_t)ldq * 2};
+    if (!encode_map(&mq, q, 3, dims, strides, box, "q")) return MSGL_CUDA_ERROR;
+  }
+  {
+    cuuint64_t dims[3] = {(cuuint64_t)dk, (cuuint64_t)h, (cuuint64_t)t_pad};
+    cuuint64_t strides[2] = {(cuuint64_t)dk * 2, (cuuint64_t)h * dk * 2};
+    if (!encode_map(&mk, k, 3, dims, strides, box, "k")) return MSGL_CUDA_ERROR;
+  }
+  {
+    cuuint64_t dims[3] = {(cuuint64_t)t_pad, (cuuint64_t)dv, (cuuint64_t)h};
+    cuuint64_t strides[2] = {(cuuint64_t)t_pad * 2, (cuuint64_t)dv * t_pad * 2};
+    cuuint32_t vbox[3] = {64, 128, 1};
+    if (!encode_map(&mv, vt, 3, dims, strides, vbox, "v")) return MSGL_CUDA_ERROR;
+  }
+  TcArgs a = {};
+  int* status = nullptr;
+  cudaGetSymbolAddress((void**)&status, g_attn_tc_status);
+  a.items = (const TcItem*)items; a.n_items = n_items; a.pairs = h; a.Hq = h; a.Hk = h; a.t_cap = t_pad;
+  a.out = out; a.scale = scale; a.status = status; a.window = window; a.ldo = ldo; a.ho = ho; a.v_chunks = dv / 8;
+  return launch_tc<__nv_bfloat16, true>(mq, mk, mv, a, stream);
+}
 
 // Causal prefill / extend attention for one layer. `kc` / `vt` are scratch buffers of
 // hk * t_cap * 128 16-bit elements each; `items` (n_items x 8 int32), `blk_req` (t_pad / 128
@@ -499,12 +595,12 @@ MSGL_API int msgl_attn_prefill_tc(const void* q, long long q_row_stride, void* o
   else { if (kv_fp8) GATHER(__half, true); else GATHER(__half, false); }
 #undef GATHER
   MSGL_CHECK_LAUNCH("kv_gather");
-  TcArgs a;
+  TcArgs a = {};
   a.items = (const TcItem*)items; a.n_items = n_items; a.pairs = hq / 2; a.Hq = hq; a.Hk = hk; a.t_cap = t_cap;
   a.out = out; a.k_scale = (const float*)k_scale; a.v_scale = (const float*)v_scale; a.scale = scale;
   a.status = status;
-  if (dtype == MSGL_BF16) return launch_tc<__nv_bfloat16>(mq, mk, mv, a, stream);
-  return launch_tc<__half>(mq, mk, mv, a, stream);
+  if (dtype == MSGL_BF16) return launch_tc<__nv_bfloat16, false>(mq, mk, mv, a, stream);
+  return launch_tc<__half, false>(mq, mk, mv, a, stream);
 }
 
 MSGL_API int msgl_attn_tc_status(int reset) {

@@ -2,9 +2,9 @@
 // at once ([pages, page_size, R] of one layer of the latent pool), causal, with a sliding window.
 //
 //   latent_norm_store_kernel   RMS norm of this step's latents, into their pool slots
-//   head_gemm_kernel           per-head projections into and out of the latent space
+//   head_gemm_kernel           per-head projections into and out of the latent space (merging a split's ranges)
 //   latent_attention_kernel    bf16: 16 / 32 / 64 (position, head) rows per CTA against 64-token tiles
-//                              that are fetched once (cp.async, two stages, through the block table)
+//                              that are fetched once (cp.async, two or three stages, through the block table)
 //                              and serve QK^T and PV; warp-level tensor products, fp32 scores,
 //                              softmax and accumulation; optional split of the key range
 //   latent_combine_kernel      merges the ranges of a split
@@ -61,17 +61,19 @@ struct LatArgs {
   const int32_t* seq_lens;
   float* ws_o;            // [splits, T * H, R]
   float* ws_lse;          // [splits, T * H]
-  int H, page_size, num_pages, window, splits, total_rows;   // num_pages includes the scratch page
+  int H, page_size, page_shift, num_pages, window, splits, total_rows;   // num_pages includes the scratch page
   float scale;
 };
 
 __device__ __forceinline__ long long token_slot(const LatArgs& a, const int32_t* bt, int tok) {
-  int col = tok / a.page_size;
+  // page_shift >= 0: the page size is a power of two
+  int col = a.page_shift >= 0 ? tok >> a.page_shift : tok / a.page_size;
+  const int in = tok - col * a.page_size;
   col = col < a.bt_stride ? col : a.bt_stride - 1;
   int page = bt[col];
   (void)MSGL_OOB(page, a.num_pages);
   page = page < 0 ? 0 : (page >= a.num_pages ? a.num_pages - 1 : page);
-  return (long long)page * a.page_size + tok % a.page_size;
+  return (long long)page * a.page_size + in;
 }
 
 // One warp per (query row, head); lane i holds the latent channels i, i + 32, ...
@@ -164,10 +166,18 @@ struct HeadGemmArgs {
   __nv_bfloat16* out;
   long long ldo, ho;
   int T, N, K, static_weights;
+  // COMBINE: the rows are the ranges of a split attention, merged while they are read
+  const float* ws_o;      // [splits, T * H, K]
+  const float* ws_lse;    // [splits, T * H]
+  int splits, H;
 };
 
+constexpr int kMaxSplits = 16;
+
+template <bool COMBINE>
 __global__ void __launch_bounds__(128) head_gemm_kernel(const HeadGemmArgs a) {
   __shared__ __align__(128) uint8_t smem[2][2][64 * 128];
+  __shared__ float part[COMBINE ? kMaxSplits : 1][64];
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int n0 = blockIdx.x * 64, h = blockIdx.y, t0 = blockIdx.z * 64;
   const int panels = (a.K + 63) / 64;
@@ -181,6 +191,22 @@ __global__ void __launch_bounds__(128) head_gemm_kernel(const HeadGemmArgs a) {
       if (weights) {
         const bool ok = n0 + r < a.N && k < a.K;
         cp16(dst + swz(r, c, 8), ok ? wh + (long long)(n0 + r) * a.K + k : wh, ok);
+      } else if constexpr (COMBINE) {
+        float v[8] = {};
+        if (t0 + r < a.T && k < a.K) {
+          const long long rows = (long long)a.T * a.H;
+          const float* src = a.ws_o + ((long long)(t0 + r) * a.H + h) * a.K + k;
+#pragma unroll 4
+          for (int sp = 0; sp < a.splits; ++sp) {
+            const float f = part[sp][r];
+            const float4 x = *reinterpret_cast<const float4*>(src + sp * rows * a.K);
+            const float4 y = *reinterpret_cast<const float4*>(src + sp * rows * a.K + 4);
+            v[0] = fmaf(f, x.x, v[0]); v[1] = fmaf(f, x.y, v[1]); v[2] = fmaf(f, x.z, v[2]); v[3] = fmaf(f, x.w, v[3]);
+            v[4] = fmaf(f, y.x, v[4]); v[5] = fmaf(f, y.y, v[5]); v[6] = fmaf(f, y.z, v[6]); v[7] = fmaf(f, y.w, v[7]);
+          }
+        }
+        *reinterpret_cast<uint4*>(smem[s][0] + swz(r, c, 8)) =
+            make_uint4(pack_bf(v[0], v[1]), pack_bf(v[2], v[3]), pack_bf(v[4], v[5]), pack_bf(v[6], v[7]));
       } else {
         const bool ok = t0 + r < a.T && k < a.K;
         cp16(dst + swz(r, c, 8), ok ? xh + (long long)(t0 + r) * a.ldx + k : xh, ok);
@@ -190,6 +216,22 @@ __global__ void __launch_bounds__(128) head_gemm_kernel(const HeadGemmArgs a) {
   if (a.static_weights) load(0, 0, true);   // weights no earlier kernel writes: fetched ahead of the dependency
   pdl_enter();
   if (!a.static_weights) load(0, 0, true);
+  if constexpr (COMBINE) {
+    if (tid < 64 && t0 + tid < a.T) {
+      const long long rows = (long long)a.T * a.H;
+      const float* lse = a.ws_lse + (long long)(t0 + tid) * a.H + h;
+      float m = -INFINITY, total = 0.f;
+      for (int sp = 0; sp < a.splits; ++sp) m = fmaxf(m, lse[sp * rows]);
+      for (int sp = 0; sp < a.splits; ++sp) {
+        const float f = m == -INFINITY ? 0.f : ex2(lse[sp * rows] - m);
+        part[sp][tid] = f;
+        total += f;
+      }
+      const float inv = total > 0.f ? 1.f / total : 0.f;
+      for (int sp = 0; sp < a.splits; ++sp) part[sp][tid] *= inv;
+    }
+    __syncthreads();
+  }
   load(0, 0, false);
   cp_commit();
   float acc[8][4] = {};
@@ -229,6 +271,8 @@ __global__ void __launch_bounds__(128) head_gemm_kernel(const HeadGemmArgs a) {
 }
 
 // ------------------------------------------------------------------------------------------ attention
+template <int NP> struct LatentStages { static constexpr int value = NP <= 4 ? 3 : 2; };
+
 // NP: latent panels of 64 channels (R = 64 NP). WM row groups of 16 x WN = 8 / WM column groups: a warp
 // computes 16 rows x (64 / WN) keys of S and 16 rows x (R / WN) channels of O.
 template <int NP, int WM>
@@ -238,11 +282,11 @@ __global__ void __launch_bounds__(256) latent_attention_kernel(const LatArgs a) 
   constexpr int CH = R / 8;                      // 16-byte chunks per row
   constexpr int NS = TK / WN / 8;                // key blocks of 8 per warp
   constexpr int NO = R / WN / 8;                 // channel blocks of 8 per warp
-  constexpr int Q_BYTES = MT * R * 2, C_BYTES = TK * R * 2;
+  constexpr int Q_BYTES = MT * R * 2, C_BYTES = TK * R * 2, ST = LatentStages<NP>::value;
   extern __shared__ __align__(128) uint8_t smem[];
   uint8_t* base = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem) + 127) & ~uintptr_t(127));
-  const uint32_t q_s = smem_u32(base), c_s = q_s + Q_BYTES, p_s = c_s + 2 * C_BYTES;
-  float* red = reinterpret_cast<float*>(base + Q_BYTES + 2 * C_BYTES + MT * 128);   // [WN][MT]
+  const uint32_t q_s = smem_u32(base), c_s = q_s + Q_BYTES, p_s = c_s + ST * C_BYTES;
+  float* red = reinterpret_cast<float*>(base + Q_BYTES + ST * C_BYTES + MT * 128);   // [WN][MT]
 
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int wm = warp / WN, wn = warp % WN;
@@ -263,7 +307,7 @@ __global__ void __launch_bounds__(256) latent_attention_kernel(const LatArgs a) 
   const int32_t* bt = a.block_table + (size_t)b * a.bt_stride;
 
   auto load_tile = [&](int t) {
-    const uint32_t dst = c_s + (t & 1) * C_BYTES;
+    const uint32_t dst = c_s + (t % ST) * C_BYTES;
     const int tok0 = (t_begin + t) * TK;
     for (int id = tid; id < TK * CH; id += 256) {
       const int r = id / CH, c = id % CH, tok = tok0 + r;
@@ -280,8 +324,11 @@ __global__ void __launch_bounds__(256) latent_attention_kernel(const LatArgs a) 
       cp16(q_s + swz(r, c, CH), ok ? q + (size_t)r * R + c * 8 : q, ok);
     }
   }
-  if (n_tiles > 0) load_tile(0);
-  cp_commit();
+#pragma unroll
+  for (int t = 0; t < ST - 1; ++t) {             // (the queries belong to the first group)
+    if (t < n_tiles) load_tile(t);
+    cp_commit();
+  }
 
   // this thread's two rows of the 16-row group
   const int ra = wm * 16 + (lane >> 2), rb = ra + 8;
@@ -294,11 +341,11 @@ __global__ void __launch_bounds__(256) latent_attention_kernel(const LatArgs a) 
   float m_a = -INFINITY, m_b = -INFINITY, l_a = 0.f, l_b = 0.f;
 
   for (int t = 0; t < n_tiles; ++t) {
-    cp_wait<0>();
+    cp_wait<ST - 2>();
     __syncthreads();                              // tile t has landed; everyone is done with tile t - 1
-    if (t + 1 < n_tiles) load_tile(t + 1);
+    if (t + ST - 1 < n_tiles) load_tile(t + ST - 1);
     cp_commit();
-    const uint32_t cb = c_s + (t & 1) * C_BYTES;
+    const uint32_t cb = c_s + (t % ST) * C_BYTES;
     float s[NS][4];
 #pragma unroll
     for (int i = 0; i < NS; ++i) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.f;
@@ -457,7 +504,7 @@ __global__ void __launch_bounds__(128) latent_combine_kernel(const float* __rest
 template <int NP, int WM>
 int launch_latent(const LatArgs& a, int B, int max_q, cudaStream_t s) {
   constexpr int R = NP * 64, MT = 16 * WM, WN = 8 / WM;
-  constexpr int bytes = MT * R * 2 + 2 * 64 * R * 2 + MT * 128 + WN * MT * 4 + 128;
+  constexpr int bytes = MT * R * 2 + LatentStages<NP>::value * 64 * R * 2 + MT * 128 + WN * MT * 4 + 128;
   static bool set = false;
   if (!set) {
     const cudaError_t e = cudaFuncSetAttribute(latent_attention_kernel<NP, WM>,
@@ -515,14 +562,21 @@ MSGL_API int msgl_latent_norm_store(const void* c, long long ldc, const void* we
 }
 
 MSGL_API int msgl_head_gemm(const void* x, long long ldx, long long hx, const void* w, void* out, long long ldo,
-                            long long ho, int T, int H, int N, int K, int static_weights, cudaStream_t stream) {
+                            long long ho, int T, int H, int N, int K, int static_weights, const void* ws_o, const void* ws_lse,
+                            int splits, cudaStream_t stream) {
   if (T <= 0) return T == 0 ? MSGL_OK : MSGL_BAD_ARG;
   if (H <= 0 || H > 65535 || N % 8 || K % 8 || ldx % 8 || hx % 8 || ldo % 2 || ho % 2 || (uintptr_t)x % 16 ||
       (uintptr_t)w % 16 || (uintptr_t)out % 4 || T > 65535 * 64)
     return MSGL_BAD_ARG;
-  HeadGemmArgs a{(const __nv_bfloat16*)x, ldx, hx, (const __nv_bfloat16*)w, (__nv_bfloat16*)out, ldo, ho, T, N, K, static_weights};
+  HeadGemmArgs a{(const __nv_bfloat16*)x, ldx, hx, (const __nv_bfloat16*)w, (__nv_bfloat16*)out, ldo, ho, T, N, K,
+                 static_weights, (const float*)ws_o, (const float*)ws_lse, splits, H};
   dim3 grid((N + 63) / 64, H, (T + 63) / 64);
-  msgl_launch(head_gemm_kernel, grid, dim3(128), 0, stream, a);
+  if (splits > 1) {
+    if (splits > kMaxSplits || ws_o == nullptr || ws_lse == nullptr || (uintptr_t)ws_o % 16) return MSGL_BAD_ARG;
+    msgl_launch(head_gemm_kernel<true>, grid, dim3(128), 0, stream, a);
+  } else {
+    msgl_launch(head_gemm_kernel<false>, grid, dim3(128), 0, stream, a);
+  }
   MSGL_CHECK_LAUNCH("head_gemm");
   return MSGL_OK;
 }
@@ -533,10 +587,13 @@ MSGL_API int msgl_latent_attention(const void* q, const void* pool, void* out, c
                                    float scale, int dtype, cudaStream_t stream) {
   if (B <= 0 || total_q <= 0) return B == 0 || total_q == 0 ? MSGL_OK : MSGL_BAD_ARG;
   if (max_q <= 0 || H <= 0 || R % 64 || page_size <= 0 || num_pages <= 0 || B > 65535 || splits < 1 || bt_stride < 1 ||
-      (uintptr_t)q % 16 || (uintptr_t)pool % 16 || (uintptr_t)out % 16)
+      (uintptr_t)q % 16 || (uintptr_t)pool % 16 || (uintptr_t)out % 16 || (out == nullptr && splits == 1))
     return MSGL_BAD_ARG;
+  int shift = -1;
+  for (int i = 0; i < 31; ++i)
+    if ((1 << i) == page_size) shift = i;
   LatArgs a{q, pool, out, (const int32_t*)block_table, bt_stride, (const int32_t*)cu_q, (const int32_t*)seq_lens,
-            (float*)ws_o, (float*)ws_lse, H, page_size, num_pages, window, splits, total_q * H, scale};
+            (float*)ws_o, (float*)ws_lse, H, page_size, shift, num_pages, window, splits, total_q * H, scale};
   if (dtype == MSGL_F32) return launch_simt<float>(a, R, B, max_q, stream);
   if (dtype != MSGL_BF16) return MSGL_BAD_ARG;
   if (R > 512) {
@@ -554,7 +611,8 @@ MSGL_API int msgl_latent_attention(const void* q, const void* pool, void* out, c
     case 8: rc = launch_latent_rows<8>(a, B, max_q, stream); break;
     default: return MSGL_BAD_ARG;
   }
-  if (rc != MSGL_OK || splits == 1) return rc;
+  // without a destination the ranges stay apart: the projection out of the latent space merges them
+  if (rc != MSGL_OK || splits == 1 || out == nullptr) return rc;
   msgl_launch(latent_combine_kernel, dim3((total_q * H + 3) / 4), dim3(128), 0, stream, (const float*)ws_o,
               (const float*)ws_lse, (__nv_bfloat16*)out, total_q * H, R, splits);
   MSGL_CHECK_LAUNCH("latent_combine");

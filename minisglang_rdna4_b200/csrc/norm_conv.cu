@@ -36,11 +36,11 @@ struct NormConvArgs {
   long long plane_stride, ldd;
   const float* gain;
   float eps;
-  const float* w1;        // [width, taps] or null
+  const float* w1;        // [taps, width] or null
   const float* w2;
   void* y1;               // [rows, cols]
   void* y2;
-  float* state;           // [slots, width, taps - 1]
+  float* state;           // [slots, taps - 1, width]
   const int32_t* cu_q;
   const int32_t* slots;
   const int32_t* has_state;
@@ -77,8 +77,8 @@ __global__ void __launch_bounds__(1024) norm_conv_kernel(const NormConvArgs a) {
       for (int j = 0; j < MT; ++j) {
         const int src = j - (MT - a.taps);
         const bool ok = conv && src >= 0 && ch[g] + v < a.width;
-        f1[g][v][j] = ok ? a.w1[(size_t)(ch[g] + v) * a.taps + src] : 0.f;
-        f2[g][v][j] = ok && a.w2 != nullptr ? a.w2[(size_t)(ch[g] + v) * a.taps + src] : 0.f;
+        f1[g][v][j] = ok ? a.w1[(size_t)src * a.width + ch[g] + v] : 0.f;
+        f2[g][v][j] = ok && a.w2 != nullptr ? a.w2[(size_t)src * a.width + ch[g] + v] : 0.f;
       }
     }
   }
@@ -93,7 +93,7 @@ __global__ void __launch_bounds__(1024) norm_conv_kernel(const NormConvArgs a) {
 #pragma unroll
           for (int j = 0; j < MT - 1; ++j) {
             const int src = j - (MT - 1 - hist_n);
-            if (src >= 0 && ch[g] + v < a.width) hist[g][v][j] = st[(size_t)(ch[g] + v) * hist_n + src];
+            if (src >= 0 && ch[g] + v < a.width) hist[g][v][j] = st[(size_t)src * a.width + ch[g] + v];
           }
     }
   }
@@ -235,8 +235,133 @@ __global__ void __launch_bounds__(1024) norm_conv_kernel(const NormConvArgs a) {
 #pragma unroll
       for (int j = 0; j < MT - 1; ++j) {
         const int dst = j - (MT - 1 - hist_n);
-        if (dst >= 0 && ch[g] + v < a.width) st[(size_t)(ch[g] + v) * hist_n + dst] = hist[g][v][j];
+        if (dst >= 0 && ch[g] + v < a.width) st[(size_t)dst * a.width + ch[g] + v] = hist[g][v][j];
       }
+}
+
+// Prefill form: kRows rows per CTA. First every warp takes rows of its own (residual add, sum of squares), then every
+// thread walks down the rows of its four channels, which needs no barrier per row. width and cols multiples of 4.
+constexpr int kRows = 16;
+
+template <typename T, int MT>
+__global__ void __launch_bounds__(256, MT <= 4 ? 3 : 2) norm_conv_rows_kernel(const NormConvArgs a) {
+  pdl_enter();
+  __shared__ float s_scale[kRows + 2 * MT];
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int b = blockIdx.y;
+  const int lo = a.cu_q[b], n = a.cu_q[b + 1] - lo;
+  const int r0 = blockIdx.x * kRows;
+  if (r0 >= n) return;
+  const int r1 = min(r0 + kRows, n), hist_n = a.taps - 1;
+  const int first = max(r0 - hist_n, 0);
+  // the CTA that reads a request's tail also writes the new one, from rows that may be another CTA's
+  const int tail = r0 == 0 && r1 < n ? n - hist_n : n;
+  const int n_main = r1 - first, n_all = n_main + (n - tail);
+  const float gain = a.gain[0];
+  auto residual = [&](int r, int c) {
+    const size_t row = (size_t)(lo + r);
+    float4 x = *reinterpret_cast<const float4*>(a.x + row * a.width + c);
+    for (int p = 0; p < a.planes; ++p) {
+      const float4 d = *reinterpret_cast<const float4*>(a.delta + p * a.plane_stride + row * a.ldd + c);
+      x.x += d.x; x.y += d.y; x.z += d.z; x.w += d.w;
+    }
+    return x;
+  };
+  for (int i = warp; i < n_all; i += 8) {
+    const int r = i < n_main ? first + i : tail + i - n_main;
+    const bool own = i < n_main && r >= r0 && a.x_out != a.x;
+    float s = 0.f;
+#pragma unroll 4
+    for (int c = lane * 4; c < a.width; c += 128) {
+      const float4 x = residual(r, c);
+      s = fmaf(x.x, x.x, s);
+      s = fmaf(x.y, x.y, s);
+      s = fmaf(x.z, x.z, s);
+      s = fmaf(x.w, x.w, s);
+      if (own) *reinterpret_cast<float4*>(a.x_out + (size_t)(lo + r) * a.width + c) = x;
+    }
+    s = warp_sum(s);
+    if (lane == 0) s_scale[i] = gain / sqrtf(s / (float)a.width + a.eps);
+  }
+  __syncthreads();
+  float* st = r0 == 0 && hist_n > 0 ? a.state + (size_t)a.slots[b] * a.width * hist_n : nullptr;
+  const bool keep = st != nullptr && a.has_state[b] != 0;
+  T* y1 = reinterpret_cast<T*>(a.y1);
+  T* y2 = reinterpret_cast<T*>(a.y2);
+  for (int c = tid * 4; c < a.cols; c += 1024) {
+    const bool in = c < a.width;
+    float f1[MT][4], f2[MT][4], hist[MT][4];
+#pragma unroll
+    for (int j = 0; j < MT; ++j) {
+      const int src = j - (MT - a.taps);
+      float4 q1 = make_float4(0.f, 0.f, 0.f, 0.f), q2 = q1, q3 = q1;
+      if (in && src >= 0) {
+        q1 = *reinterpret_cast<const float4*>(a.w1 + (size_t)src * a.width + c);
+        if (a.w2 != nullptr) q2 = *reinterpret_cast<const float4*>(a.w2 + (size_t)src * a.width + c);
+        if (keep && src < hist_n) q3 = *reinterpret_cast<const float4*>(st + (size_t)src * a.width + c);
+      }
+      f1[j][0] = q1.x; f1[j][1] = q1.y; f1[j][2] = q1.z; f1[j][3] = q1.w;
+      f2[j][0] = q2.x; f2[j][1] = q2.y; f2[j][2] = q2.z; f2[j][3] = q2.w;
+      hist[j][0] = q3.x; hist[j][1] = q3.y; hist[j][2] = q3.z; hist[j][3] = q3.w;
+    }
+    // hist[MT - taps .. MT - 2]: the rows ahead; hist[MT - 1]: the row itself
+#pragma unroll 2
+    for (int i = 0; i < n_main; ++i) {
+      const int r = first + i;
+      float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (in) x = r >= r0 ? *reinterpret_cast<const float4*>(a.x_out + (size_t)(lo + r) * a.width + c) : residual(r, c);
+      const float sc = s_scale[i];
+      hist[MT - 1][0] = x.x * sc; hist[MT - 1][1] = x.y * sc; hist[MT - 1][2] = x.z * sc; hist[MT - 1][3] = x.w * sc;
+      if (r >= r0) {
+        float o1[4], o2[4];
+#pragma unroll
+        for (int v = 0; v < 4; ++v) {
+          o1[v] = o2[v] = hist[MT - 1][v];
+#pragma unroll
+          for (int j = 0; j < MT; ++j) {
+            o1[v] = fmaf(f1[j][v], hist[j][v], o1[v]);
+            o2[v] = fmaf(f2[j][v], hist[j][v], o2[v]);
+          }
+        }
+        const size_t off = (size_t)(lo + r) * a.cols + c;
+        if constexpr (sizeof(T) == 2) {
+          uint2 q;
+          *reinterpret_cast<typename Pack2<T>::type*>(&q.x) = Pack2<T>::make(o1[0], o1[1]);
+          *reinterpret_cast<typename Pack2<T>::type*>(&q.y) = Pack2<T>::make(o1[2], o1[3]);
+          *reinterpret_cast<uint2*>(y1 + off) = q;
+          if (y2 != nullptr) {
+            *reinterpret_cast<typename Pack2<T>::type*>(&q.x) = Pack2<T>::make(o2[0], o2[1]);
+            *reinterpret_cast<typename Pack2<T>::type*>(&q.y) = Pack2<T>::make(o2[2], o2[3]);
+            *reinterpret_cast<uint2*>(y2 + off) = q;
+          }
+        } else {
+          *reinterpret_cast<float4*>(y1 + off) = make_float4(o1[0], o1[1], o1[2], o1[3]);
+          if (y2 != nullptr) *reinterpret_cast<float4*>(y2 + off) = make_float4(o2[0], o2[1], o2[2], o2[3]);
+        }
+      }
+#pragma unroll
+      for (int j = 0; j + 1 < MT; ++j)
+#pragma unroll
+        for (int v = 0; v < 4; ++v) hist[j][v] = hist[j + 1][v];
+    }
+    if (st == nullptr || !in) continue;
+    for (int i = n_main; i < n_all; ++i) {
+      const float4 x = residual(tail + i - n_main, c);
+      const float sc = s_scale[i];
+      hist[MT - 1][0] = x.x * sc; hist[MT - 1][1] = x.y * sc; hist[MT - 1][2] = x.z * sc; hist[MT - 1][3] = x.w * sc;
+#pragma unroll
+      for (int j = 0; j + 1 < MT; ++j)
+#pragma unroll
+        for (int v = 0; v < 4; ++v) hist[j][v] = hist[j + 1][v];
+    }
+#pragma unroll
+    for (int j = 0; j + 1 < MT; ++j) {
+      const int dst = j - (MT - a.taps);
+      if (dst >= 0)
+        *reinterpret_cast<float4*>(st + (size_t)dst * a.width + c) =
+            make_float4(hist[j][0], hist[j][1], hist[j][2], hist[j][3]);
+    }
+  }
 }
 
 template <typename T, int V, int NC>
@@ -261,6 +386,16 @@ int norm_conv_typed(NormConvArgs a, int B, int max_q, cudaStream_t s) {
   const bool vec = a.width % 4 == 0 && a.cols % 4 == 0 && a.ldd % 4 == 0 && (uintptr_t)a.delta % 16 == 0;
   const int per = vec ? 4 : 1;
   const int groups = (a.cols + per - 1) / per;
+  if (vec && conv && max_q > 4 && a.taps <= 8) {
+    a.block_rows = kRows;
+    const dim3 rows_grid((n + kRows - 1) / kRows, B);
+    if (a.taps <= 4)
+      msgl_launch(norm_conv_rows_kernel<T, 4>, rows_grid, dim3(256), 0, s, a);
+    else
+      msgl_launch(norm_conv_rows_kernel<T, 8>, rows_grid, dim3(256), 0, s, a);
+    MSGL_CHECK_LAUNCH("norm_conv_rows");
+    return MSGL_OK;
+  }
   const int nc = (groups + 1023) / 1024;
   const int threads = ((groups + nc - 1) / nc + 31) / 32 * 32;
   if (vec) {
@@ -276,17 +411,15 @@ int norm_conv_typed(NormConvArgs a, int B, int max_q, cudaStream_t s) {
   return MSGL_OK;
 }
 
-// Exact gelu of [rows, n] with row strides; n a multiple of 4.
+// Exact gelu of [rows, n] with row strides; n a multiple of the vector width.
 template <typename T>
 __global__ void __launch_bounds__(256) gelu_erf_kernel(const T* __restrict__ x, long long ldx, T* __restrict__ out,
-                                                       long long ldo, int n, long long total) {
+                                                       long long ldo, int n) {
   pdl_enter();
   constexpr int V = 16 / sizeof(T);
-  const long long i = (long long)blockIdx.x * 256 + threadIdx.x;
-  if (i >= total) return;
-  const int per = n / V;
-  const long long r = i / per;
-  const int c = (int)(i - r * per) * V;
+  const int c = (blockIdx.y * 256 + threadIdx.x) * V;
+  if (c >= n) return;
+  const long long r = blockIdx.x;
   float v[V];
   if constexpr (sizeof(T) == 2) {
     load8(x + r * ldx + c, v);
@@ -338,13 +471,12 @@ MSGL_API int msgl_gelu_erf(const void* x, long long ldx, void* out, long long ld
   if (rows <= 0 || n <= 0) return rows == 0 || n == 0 ? MSGL_OK : MSGL_BAD_ARG;
   const int v = dtype == MSGL_BF16 ? 8 : 4;
   if (n % v || ldx % v || ldo % v || (uintptr_t)x % 16 || (uintptr_t)out % 16) return MSGL_BAD_ARG;
-  const long long total = (long long)rows * (n / v);
-  dim3 grid((unsigned)((total + 255) / 256));
+  dim3 grid(rows, (n / v + 255) / 256);
   if (dtype == MSGL_BF16)
     msgl_launch(gelu_erf_kernel<__nv_bfloat16>, grid, dim3(256), 0, stream, (const __nv_bfloat16*)x, ldx,
-                (__nv_bfloat16*)out, ldo, n, total);
+                (__nv_bfloat16*)out, ldo, n);
   else if (dtype == MSGL_F32)
-    msgl_launch(gelu_erf_kernel<float>, grid, dim3(256), 0, stream, (const float*)x, ldx, (float*)out, ldo, n, total);
+    msgl_launch(gelu_erf_kernel<float>, grid, dim3(256), 0, stream, (const float*)x, ldx, (float*)out, ldo, n);
   else
     return MSGL_BAD_ARG;
   MSGL_CHECK_LAUNCH("gelu_erf");

@@ -362,7 +362,7 @@ class Engine:
         self.ctx.attn_backend = create_attention_backend(
             config.attention_backend, self.q_heads_local, self.kv_heads_local, mc.head_dim, self.device,
             max_batch=config.max_running_req, max_seq_len=self.max_seq_len,
-            single_split=config.spec_algorithm != "none", latent=bool(mc.latent_layers),
+            single_split=config.spec_algorithm != "none", latent=mc.latent_layers,
         )
         self.ctx.comm = comm_mod.get_comm()
         self._spec_exact = config.spec_algorithm != "none" and dev_kind == "cuda"

@@ -1,7 +1,7 @@
 """Latent attention without positions: a layer caches one latent per token (its own, or it reads another layer's),
 and its per-head keys and values are linear in that latent.
 
-The serving form is absorbed: queries move into the latent space through the key half (``q W_uk``), every head attends
+The decoding form is absorbed: queries move into the latent space through the key half (``q W_uk``), every head attends
 to the same latent rows, and the attended latents come back through the value half (``W_uv``). Each layer has sizes,
 scale, window and heads of its own."""
 from __future__ import annotations
@@ -31,6 +31,7 @@ class LatentAttentionLayer(BaseOP):
             self.latent_norm = torch.empty((self._rank,), dtype=torch.float32, device=device)
         self.up_k = torch.empty((self._h, self._rank, self._dim), dtype=dtype, device=device)
         self.up_v = torch.empty((self._h, self._vdim, self._rank), dtype=dtype, device=device)
+        self._expand_k = None        # up_k as [heads * dim, rank]: the expanded prefill form (16-bit, GPU)
 
     @property
     def out_width(self) -> int:
@@ -47,7 +48,12 @@ class LatentAttentionLayer(BaseOP):
                                   ctx.kv_cache.rows(self._row), batch.out_loc)
         q = qc[:, :nq].unflatten(1, (self._h, self._dim))
         ctx.attn_backend.latent_forward(q, self.up_k, self.up_v, self._row, batch, scale=self._spec.scale,
-                                        window=self._spec.window, out=out.unflatten(1, (self._h, self._vdim)))
+                                        window=self._spec.window, out=out.unflatten(1, (self._h, self._vdim)),
+                                        expand_k=self._expand_k)
+
+    def _post_load_self(self) -> None:
+        if self.up_k.is_cuda and self.up_k.dtype == torch.bfloat16:
+            self._expand_k = self.up_k.transpose(1, 2).reshape(self._h * self._dim, self._rank).contiguous()
 
     def init_dummy(self, gen: torch.Generator, std: float = 0.02) -> None:
         for name in ("up_k", "up_v"):

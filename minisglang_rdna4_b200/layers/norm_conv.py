@@ -24,9 +24,9 @@ class ScalarNormConv(BaseOP):
         self._taps, self._state_id, self._eps = taps, state_id, eps
         self._dtype, self._cols = dtype, out_cols
         if filters > 0:
-            self.conv1 = torch.empty((width, taps), dtype=torch.float32, device=device)
+            self.conv1 = torch.empty((taps, width), dtype=torch.float32, device=device)
         if filters > 1:
-            self.conv2 = torch.empty((width, taps), dtype=torch.float32, device=device)
+            self.conv2 = torch.empty((taps, width), dtype=torch.float32, device=device)
         self._filters = filters
 
     def forward(self, x: torch.Tensor, delta) -> Tuple[torch.Tensor, torch.Tensor, Optional[torch.Tensor]]:
@@ -43,7 +43,9 @@ class ScalarNormConv(BaseOP):
         return out
 
     def _apply(self, x, delta, cu_q, slots, has_state, max_q: int):
+        # the cache keeps [slots, width * (taps - 1)] values per layer; here they are taps - 1 rows
         state = get_global_ctx().gdn_state.conv_state(self._state_id)
+        state = state.view(state.shape[0], self._taps - 1, self.conv1.shape[1])
         return ops.add_scalar_norm_conv(x, delta, self.gain, self._eps, self.conv1, getattr(self, "conv2", None),
                                         state, cu_q, slots, has_state, max_q, self._dtype, self._cols)
 

@@ -107,6 +107,9 @@ class MitilixForCausalLM(BaseOP):
         def corner(p, t):
             p[:t.shape[0], :t.shape[1]].copy_(t)
 
+        def taps_first(p, t):
+            p.copy_(t.t())
+
         def vocab(start):
             def fill(p, t):
                 rows = t[start:start + p.shape[0]]
@@ -152,7 +155,7 @@ class MitilixForCausalLM(BaseOP):
 
             name = f"l{i}."
             out[name + "norm1"] = [(layer.norm, "gain", whole)]
-            out[name + "canon1"] = [(layer.norm, "conv1", corner)]
+            out[name + "canon1"] = [(layer.norm, "conv1", taps_first)]
             out[name + "mix.q"] = [(a.q_proj, "weight", q)]
             out[name + "mix.uk"] = [(a, "up_k", uk)]
             out[name + "mix.uv"] = [(a, "up_v", uv)]
@@ -161,7 +164,7 @@ class MitilixForCausalLM(BaseOP):
                 out[name + "mix.dkv"] = [(a.q_proj, "weight", dkv)]
                 out[name + "mix.dkv.norm"] = [(a, "latent_norm", whole)]
             if s.ff:
-                out[name + "canon2"] = [(layer.norm, "conv2", corner)]
+                out[name + "canon2"] = [(layer.norm, "conv2", taps_first)]
                 out[name + "mlp.up"] = [(layer.up_proj, "weight", up)]
                 out[name + "mlp.down"] = [(layer.out_proj, "weight", down)]
         return out

@@ -912,7 +912,10 @@ def _bind_latent():
     bind("msgl_norm_conv", c_i, [c_p, c_p, c_p, c_i, c_ll, c_ll, c_p, c_f] + [c_p] * 8 + [c_i] * 7 + [c_p])
     bind("msgl_gelu_erf", c_i, [c_p, c_ll, c_p, c_ll, c_i, c_i, c_i, c_p])
     bind("msgl_latent_norm_store", c_i, [c_p, c_ll, c_p, c_p, c_p, c_i, c_i, c_i, c_f, c_ll, c_i, c_p])
-    bind("msgl_head_gemm", c_i, [c_p, c_ll, c_ll, c_p, c_p, c_ll, c_ll, c_i, c_i, c_i, c_i, c_i, c_p])
+    bind("msgl_head_gemm", c_i, [c_p, c_ll, c_ll, c_p, c_p, c_ll, c_ll, c_i, c_i, c_i, c_i, c_i, c_p, c_p, c_i, c_p])
+    bind("msgl_latent_gather", c_i, [c_p] * 5 + [c_i] * 5 + [c_p])
+    bind("msgl_attn_prefill_pos", c_i, [c_p, c_ll, c_ll, c_p, c_p, c_i, c_p, c_ll, c_ll, c_p, c_i, c_i, c_i, c_i, c_i, c_i,
+                                        c_f, c_i, c_p])
     bind("msgl_latent_attention", c_i, [c_p, c_p, c_p, c_p, c_i] + [c_p] * 4 + [c_i] * 9 + [c_f, c_i, c_p])
     _bind_latent._done = True
 
@@ -958,9 +961,9 @@ def add_scalar_norm_conv(x, delta, gain, eps, w1, w2, state, cu_q, slots, has_st
     y2 = torch.empty_like(y1) if w2 is not None else None
     taps, b = 1, 1
     if w1 is not None:
-        taps, b = w1.shape[1], cu_q.numel() - 1
+        taps, b = w1.shape[0], cu_q.numel() - 1
         assert w1.is_contiguous() and w1.dtype == torch.float32 and state.is_contiguous()
-        assert state.dtype == torch.float32 and state.shape[1:] == (width, taps - 1)
+        assert state.dtype == torch.float32 and state.shape[1:] == (taps - 1, width)
     check(lib().msgl_norm_conv(_p(x), _p(x_out), _p(delta), planes, plane_stride, ldd, _p(gain), eps, _p(w1), _p(w2),
                                _p(y1), _p(y2), _p(state), _p(cu_q), _p(slots), _p(has_state), rows, width, out_cols,
                                taps, b, int(max_q), _DT[out_dtype], _stream()), "norm_conv")
@@ -1005,25 +1008,50 @@ def head_gemm(x, w, out=None):
         _count("head_gemm", "gemm_f32_kernel")
         return out
     check(lib().msgl_head_gemm(_p(x), x.stride(0), x.stride(1), _p(w), _p(out), out.stride(0), out.stride(1), t, h, n, k,
-                               int(STATIC_WEIGHTS), _stream()), "head_gemm")
+                               int(STATIC_WEIGHTS), None, None, 1, _stream()), "head_gemm")
     _count("head_gemm", "head_gemm_kernel")
     return out
 
 
-def latent_splits(batch: int, heads: int, up_to: int) -> int:
-    """Key ranges per query tile of a decode step: enough CTAs for the SMs, at least two 64-token tiles each."""
+class LatentSplit:
+    """Attention of a decode step whose key ranges were not merged: ``ws_o [splits, T * H, R]`` (each range's own
+    normalised sum) and its log2 weights ``ws_lse [splits, T * H]``; ``head_gemm_combine`` merges them."""
+
+    __slots__ = ("ws_o", "ws_lse", "shape")
+
+    def __init__(self, ws_o, ws_lse, shape) -> None:
+        self.ws_o, self.ws_lse, self.shape = ws_o, ws_lse, shape
+
+
+def head_gemm_combine(x: LatentSplit, w, out):
+    """The value projection of a split attention: merges the key ranges while it reads them."""
+    _bind_latent()
+    t, h, k = x.shape
+    n = w.shape[1]
+    assert w.is_contiguous() and w.shape == (h, n, k) and out.stride(2) == 1 and out.shape == (t, h, n)
+    check(lib().msgl_head_gemm(None, 0, 0, _p(w), _p(out), out.stride(0), out.stride(1), t, h, n, k, int(STATIC_WEIGHTS),
+                               _p(x.ws_o), _p(x.ws_lse), x.ws_o.shape[0], _stream()), "head_gemm")
+    _count("head_gemm", "head_gemm_kernel")
+    return out
+
+
+def latent_splits(batch: int, heads: int, rank: int, up_to: int) -> int:
+    """Key ranges per query tile of a decode step: one wave of CTAs on the 148 SMs (a wide latent's tiles fill an SM),
+    at least two 64-token tiles each."""
     tiles = -(-up_to // 64) + 1
     ctas = batch * -(-heads // 64)
-    return int(max(1, min(296 // max(ctas, 1), tiles // 2, 16)))
+    wave = 148 if rank > 256 else 296
+    return int(max(1, min(wave // max(ctas, 1), tiles // 2, 16)))
 
 
-def latent_attention(q, rows, block_table, cu_q, seq_lens, scale, window, max_q, max_kv, splits=1):
+def latent_attention(q, rows, block_table, cu_q, seq_lens, scale, window, max_q, max_kv, splits=1, merge=True):
+    """``merge=False``: a split result stays a ``LatentSplit``."""
     _bind_latent()
     t, h, r = q.shape
     assert q.is_contiguous() and rows.is_contiguous() and rows.shape[2] == r and rows.dtype == q.dtype
-    out = torch.empty_like(q)
     if q.dtype == torch.float32 or r > 512:
         splits = 1
+    out = torch.empty_like(q) if merge or splits == 1 else None
     ws_o = ws_l = None
     if splits > 1:
         ws_o = torch.empty((splits, t * h, r), dtype=torch.float32, device=q.device)
@@ -1032,5 +1060,93 @@ def latent_attention(q, rows, block_table, cu_q, seq_lens, scale, window, max_q,
         _p(q), _p(rows), _p(out), _p(block_table), block_table.stride(0), _p(cu_q), _p(seq_lens), _p(ws_o), _p(ws_l),
         seq_lens.numel(), t, int(max_q), h, r, rows.shape[1], rows.shape[0], int(window), splits, float(scale), _dt(q),
         _stream()), "latent_attention")
-    _count("latent_attention", "latent_attention_kernel", 2 if splits > 1 else 1)
+    _count("latent_attention", "latent_attention_kernel", 2 if splits > 1 and merge else 1)
+    return out if out is not None else LatentSplit(ws_o, ws_l, (t, h, r))
+
+
+class LatentPrefillPlan:
+    """Per-step tables of the expanded prefill: the latents a step can see (each request from the block of 128 that
+    holds the far edge of its first row's window) in one dense scratch, and one item per (request, block of 256 query
+    positions), longest first. ``reach``: the widest window of the model's layers (0: everything is visible)."""
+
+    __slots__ = ("tables", "n_items", "t_pad", "off_blk", "off_req", "dense")
+
+    def __init__(self, cu_q: np.ndarray, seq_lens: np.ndarray, reach: int, device) -> None:
+        cu_q, kv = np.asarray(cu_q, dtype=np.int64), np.asarray(seq_lens, dtype=np.int64)
+        b = int(kv.size)
+        q_len = cu_q[1:b + 1] - cu_q[:b]
+        lo = self._first(kv - q_len, reach)
+        pad = (kv - lo + 127) // 128 * 128
+        off = np.concatenate([[0], np.cumsum(pad)[:-1]])
+        self.t_pad = int(pad.sum())
+        n_tiles = (q_len + 255) // 256
+        req = np.repeat(np.arange(b), n_tiles)
+        qb = np.arange(int(n_tiles.sum())) - np.repeat(np.cumsum(n_tiles) - n_tiles, n_tiles)
+        rows = np.minimum(256, q_len[req] - qb * 256)
+        pos0 = kv[req] - q_len[req] + qb * 256
+        kv0 = self._first(pos0, reach)
+        items = np.zeros((req.size, 8), dtype=np.int32)
+        items[:, 0] = cu_q[req] + qb * 256
+        items[:, 1] = rows
+        items[:, 2] = pos0
+        items[:, 3] = off[req] + kv0 - lo[req]
+        items[:, 4] = (pos0 + rows - 1) // 128 - kv0 // 128 + 1
+        items[:, 5] = req
+        items[:, 6] = kv0
+        items = items[np.argsort(-items[:, 4], kind="stable")]
+        blk_req = np.repeat(np.arange(b), pad // 128).astype(np.int32)
+        req_info = np.stack([off, kv, lo], axis=1).astype(np.int32).reshape(-1)
+        self.n_items = int(items.shape[0])
+        self.off_blk = items.size
+        self.off_req = self.off_blk + blk_req.size
+        self.tables = _upload_tables(np.concatenate([items.reshape(-1), blk_req, req_info]), device)
+        self.dense: Optional[Tuple[int, torch.Tensor]] = None      # (pool row, its latents) of the last layer
+
+    @staticmethod
+    def _first(pos: np.ndarray, reach: int) -> np.ndarray:
+        return np.maximum(pos - reach + 1, 0) // 128 * 128 if reach > 0 else np.zeros_like(pos)
+
+    @staticmethod
+    def pays(cu_q: np.ndarray, seq_lens: np.ndarray, reach: int) -> bool:
+        """Expanding costs a matrix product over every latent the step can see: worth it when those rows are not many
+        more than the step's own, and the step is not a handful of rows."""
+        kv = np.asarray(seq_lens, dtype=np.int64)
+        q_len = np.diff(np.asarray(cu_q, dtype=np.int64)[:kv.size + 1])
+        total = int(q_len.sum())
+        lo = LatentPrefillPlan._first(kv - q_len, reach)
+        return total >= 64 and int(((kv - lo + 127) // 128 * 128).sum()) <= 4 * total
+
+
+def latent_prefill_ok(dim: int, vdim: int, scale: float) -> bool:
+    return dim <= 128 and vdim <= 128 and dim % 8 == 0 and vdim % 8 == 0 and scale > 0
+
+
+def latent_prefill(q, expand_k, up_v, rows, row_id, block_table, plan: LatentPrefillPlan, scale, window, out):
+    """Prefill with per-head keys and values expanded from the latents: ``q [T, H, dim]``, ``expand_k [H * dim, R]``,
+    ``up_v [H, vdim, R]``, one layer of the latent pool ``rows`` -> ``out [T, H, vdim]``. The values come out of their
+    matrix product transposed (``[H * vdim, tokens]``), the layout the tensor core reads them in."""
+    _bind_latent()
+    t, h, dim = q.shape
+    vdim, r = up_v.shape[1], up_v.shape[2]
+    assert q.dtype == torch.bfloat16 and rows.is_contiguous() and rows.shape[2] == r
+    base = plan.tables.data_ptr()
+    if plan.dense is None or plan.dense[0] != row_id:
+        dense = torch.empty((plan.t_pad, r), dtype=q.dtype, device=q.device)
+        check(lib().msgl_latent_gather(_p(rows), _p(dense), base + 4 * plan.off_blk, base + 4 * plan.off_req,
+                                       _p(block_table), block_table.stride(0), rows.shape[1], rows.shape[0], r,
+                                       plan.t_pad, _stream()), "latent_gather")
+        _count("latent_gather", "latent_gather_kernel")
+        plan.dense = (row_id, dense)
+    dense = plan.dense[1]
+    k = _gemm(KIND_BF16, dense, expand_k, h * dim, r, q.dtype)
+    # the latents are the second operand here: no fetch of it ahead of the kernel that gathers them
+    static = gemm_static_weights(0)
+    try:
+        vt = _gemm(KIND_BF16, up_v.view(h * vdim, r), dense, plan.t_pad, r, q.dtype)
+    finally:
+        gemm_static_weights(static)
+    check(lib().msgl_attn_prefill_pos(_p(q), q.stride(0), q.stride(1), _p(k), _p(vt), plan.t_pad, _p(out), out.stride(0),
+                                      out.stride(1), base, plan.n_items, t, h, dim, vdim, int(window), float(scale),
+                                      _dt(q), _stream()), "attn_prefill_pos")
+    _count("latent_prefill", "attn_prefill_tc_kernel")
     return out

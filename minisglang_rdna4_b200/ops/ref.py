@@ -622,9 +622,9 @@ def add_scalar_norm_conv(x: torch.Tensor, delta: Optional[torch.Tensor], gain: t
                          cu_q: Optional[torch.Tensor], slots: Optional[torch.Tensor],
                          has_state: Optional[torch.Tensor], out_dtype: torch.dtype, out_cols: int):
     """``x += delta``; ``h = x / rms(x) * gain`` (one number); ``y_k = h + conv_k(h)`` for the one or two depthwise
-    causal filters ``w_k [W, taps]``. Returns ``(x, y_1, y_2)``; with no filter ``y_1 = h``.
+    causal filters ``w_k [taps, W]``. Returns ``(x, y_1, y_2)``; with no filter ``y_1 = h``.
 
-    The convolutions read the same ``h``, so one tail ``state [slots, W, taps - 1]`` (fp32) serves both; it is
+    The convolutions read the same ``h``, so one tail ``state [slots, taps - 1, W]`` (fp32) serves both; it is
     advanced in place. Outputs have ``out_cols >= W`` columns, zero past W."""
     xn = x if delta is None else x + delta[:, :x.shape[1]].float()
     h = xn * torch.rsqrt(xn.pow(2).mean(-1, keepdim=True) + eps) * gain.float().reshape(())
@@ -634,21 +634,21 @@ def add_scalar_norm_conv(x: torch.Tensor, delta: Optional[torch.Tensor], gain: t
 
     if w1 is None and w2 is None:
         return xn, cast(h), None
-    taps = (w1 if w1 is not None else w2).shape[1]
+    taps = (w1 if w1 is not None else w2).shape[0]
     ys = [h.clone() if w is not None else None for w in (w1, w2)]
     for b in range(cu_q.numel() - 1):
         lo, hi = int(cu_q[b]), int(cu_q[b + 1])
         if hi <= lo:
             continue
         slot = int(slots[b])
-        hist = state[slot].t() if int(has_state[b]) else h.new_zeros((taps - 1, h.shape[1]))
+        hist = state[slot] if int(has_state[b]) else h.new_zeros((taps - 1, h.shape[1]))
         seq = torch.cat([hist, h[lo:hi]])
         for w, y in zip((w1, w2), ys):
             if w is not None:
                 for j in range(taps):
-                    y[lo:hi] += seq[j:j + hi - lo] * w[:, j].float()
+                    y[lo:hi] += seq[j:j + hi - lo] * w[j].float()
         if taps > 1:
-            state[slot] = seq[seq.shape[0] - (taps - 1):].t()
+            state[slot] = seq[seq.shape[0] - (taps - 1):]
     return xn, *(None if y is None else cast(y) for y in ys)
 
 

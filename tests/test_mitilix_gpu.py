@@ -40,9 +40,9 @@ def test_norm_conv(width, taps, cols, dtype):
     slots = torch.tensor([3, 0, 7, 5, 1, 2, 6], dtype=torch.int32)
     has = torch.tensor(has, dtype=torch.int32)
     x, d = torch.randn(t, width, generator=g), torch.randn(t, cols, generator=g)
-    w1, w2 = (torch.randn(width, taps, generator=g) * 0.5 for _ in range(2))
+    w1, w2 = (torch.randn(taps, width, generator=g) * 0.5 for _ in range(2))
     gain = torch.tensor([1.3])
-    state = torch.randn(9, width, taps - 1, generator=g)
+    state = torch.randn(9, taps - 1, width, generator=g)
     for delta, two in ((d, True), (None, True), (d, False)):
         st_ref, st = state.clone(), state.clone().to(DEV)
         want = ref.add_scalar_norm_conv(x, delta, gain, 1e-5, w1, w2 if two else None, st_ref, cu, slots, has, dtype, cols)
@@ -145,6 +145,53 @@ def test_latent_attention_decode_splits(r, h, window, splits):
     want = ref.latent_attention(q.float(), pool.float(), bt, cu, seq, 0.1, window)
     got = ops.latent_attention(q.to(DEV), pool.to(DEV), bt.to(DEV), cu.to(DEV), seq.to(DEV), 0.1, window, 1, 1000, splits)
     torch.testing.assert_close(got.float().cpu(), want, rtol=2e-2, atol=2e-2)
+
+
+@pytest.mark.parametrize("t,h,n,k,splits", [(1, 4, 128, 64, 2), (70, 3, 80, 512, 5)])
+def test_head_gemm_merges_splits(t, h, n, k, splits):
+    from minisglang_rdna4_b200.ops import cuda as K
+
+    g = _gen(splits)
+    ws, lse = torch.randn(splits, t * h, k, generator=g), torch.randn(splits, t * h, generator=g) * 3
+    lse[1, ::2] = float("-inf")
+    w = torch.randn(h, n, k, generator=g).bfloat16()
+    f = torch.softmax(lse * 0.6931471805599453, 0)
+    want = torch.einsum("thk,hnk->thn", (ws * f[..., None]).sum(0).view(t, h, k), w.float())
+    out = torch.empty(t, h, n, dtype=torch.bfloat16, device=DEV)
+    wd = w.to(DEV)
+    torch.cuda.synchronize()
+    K.head_gemm_combine(K.LatentSplit(ws.to(DEV), lse.to(DEV), (t, h, k)), wd, out)
+    torch.testing.assert_close(out.float().cpu(), want, rtol=2e-2, atol=2e-2 * k ** 0.5)
+
+
+@pytest.mark.parametrize("h,dim,vdim,r,window,reach", [(6, 64, 80, 64, 72, 72), (3, 128, 128, 192, 300, 300),
+                                                       (2, 16, 96, 512, 128, 500), (5, 112, 48, 128, 0, 0),
+                                                       (1, 96, 16, 64, 1, 129)])
+def test_latent_prefill_expanded(h, dim, vdim, r, window, reach):
+    from minisglang_rdna4_b200.ops import cuda as K
+
+    g = _gen(h + r)
+    lens, starts = [257, 70, 300, 1, 640], [0, 200, 129, 63, 511]
+    cu, seq, bt = _batch(lens, starts, 16, 200, g)
+    pool = (torch.randn(201, 16, r, generator=g) * 0.5).bfloat16()
+    t = sum(lens)
+    q = torch.randn(t, h * dim + 32, generator=g).bfloat16()[:, :h * dim].unflatten(1, (h, dim))
+    uk = (torch.randn(h, r, dim, generator=g) * r ** -0.5).bfloat16()
+    uv = (torch.randn(h, vdim, r, generator=g) * r ** -0.5).bfloat16()
+    scale = 2.0 * dim ** -0.5
+    o = ref.latent_attention(torch.einsum("thd,hrd->thr", q.float(), uk.float()), pool.float(), bt, cu, seq, scale, window)
+    want = torch.einsum("thr,hvr->thv", o, uv.float())
+    plan = K.LatentPrefillPlan(cu.numpy(), seq.numpy(), reach, DEV)
+    out = torch.zeros(t, h * vdim + 64, dtype=torch.bfloat16, device=DEV)
+    qd = torch.zeros(t, h * dim + 32, dtype=torch.bfloat16, device=DEV)
+    qd[:, :h * dim] = q.reshape(t, -1).to(DEV)
+    ukd = uk.transpose(1, 2).reshape(h * dim, r).contiguous().to(DEV)
+    args = (qd[:, :h * dim].unflatten(1, (h, dim)), ukd, uv.to(DEV), pool.to(DEV), 0, bt.to(DEV))
+    torch.cuda.synchronize()
+    K.latent_prefill(*args, plan, scale, window, out[:, :h * vdim].unflatten(1, (h, vdim)))
+    got = out.float().cpu()
+    torch.testing.assert_close(got[:, :h * vdim].unflatten(1, (h, vdim)), want, rtol=3e-2, atol=3e-2)
+    assert float(got[:, h * vdim:].abs().max()) == 0.0
 
 
 @pytest.mark.parametrize("r", [64, 512])
