@@ -43,21 +43,27 @@ class LatentAttentionBackend(BaseAttnBackend):
         raise NotImplementedError("models with a latent pool call latent_forward")
 
     def latent_forward(self, q, up_k, up_v, row: int, batch: Batch, *, scale: float, window: int, out,
-                       expand_k=None) -> None:
+                       expand_k=None, store=None) -> None:
         """``q [T, H, dim]``, ``up_k [H, rank, dim]``, ``up_v [H, vdim, rank]`` -> ``out [T, H, vdim]``. ``expand_k``:
-        ``up_k`` as ``[H * dim, rank]``, where the expanded form may be used."""
+        ``up_k`` as ``[H * dim, rank]``, where the expanded form may be used. ``store`` (a layer with latents of its own):
+        ``(raw latents [T, rank], norm weight, rank, eps)`` to norm and store ahead of the attention."""
         md = batch.attn_metadata
+        rows = get_global_ctx().kv_cache.rows(row)
+        if store is not None:
+            store = (*store, rows, batch.out_loc)
+            if not (md.decode and q.is_cuda and q.dtype == torch.bfloat16):
+                ops.latent_norm_store(*store)
+                store = None
         if md.prefill_plan is not None and expand_k is not None:
             from ..ops import cuda as K
 
             if K.latent_prefill_ok(q.shape[2], up_v.shape[1], scale):
-                K.latent_prefill(q, expand_k, up_v, get_global_ctx().kv_cache.rows(row), row, md.block_table,
+                K.latent_prefill(q, expand_k, up_v, rows, row, md.block_table,
                                  md.prefill_plan, scale, window, out)
                 return
-        q_lat = ops.head_gemm(q, up_k)
-        rows = get_global_ctx().kv_cache.rows(row)
+        q_lat = ops.head_gemm(q, up_k, store=store)
         splits = self._splits(q_lat, md, window)
-        if splits > 1:                        # the value projection merges the key ranges
+        if 1 < splits and q.shape[0] <= 32:   # few rows: the value projection merges the key ranges itself
             from ..ops import cuda as K
 
             parts = K.latent_attention(q_lat, rows, md.block_table, md.cu_q, md.seq_lens, scale, window, md.max_q,
@@ -65,7 +71,7 @@ class LatentAttentionBackend(BaseAttnBackend):
             K.head_gemm_combine(parts, up_v, out)
             return
         o_lat = ops.latent_attention(q_lat, rows, md.block_table, md.cu_q, md.seq_lens, scale, window, md.max_q,
-                                     md.max_kv)
+                                     md.max_kv, splits)
         ops.head_gemm(o_lat, up_v, out)
 
     def _splits(self, q, md: AttnMetadata, window: int) -> int:

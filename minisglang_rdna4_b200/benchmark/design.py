@@ -8,6 +8,7 @@ from __future__ import annotations
 
 import gc
 import json
+import multiprocessing as mp
 import os
 import statistics
 from typing import Callable, Dict, List, Tuple
@@ -194,7 +195,7 @@ def kernels(s: Dict) -> List[Dict]:
         if n == 1:
             q_lat = rnd(t, h, r)
             sp = be._splits(q_lat, batch.attn_metadata, win)
-            us = _time(lambda: K.latent_attention(q_lat, pool.rows(0), bt, cu, seq, d ** -0.5, win, n, ctx_len, sp, merge=sp == 1))
+            us = _time(lambda: K.latent_attention(q_lat, pool.rows(0), bt, cu, seq, d ** -0.5, win, n, ctx_len, sp, merge=t > 32))
             add("mitilix", "latent_attention", phase, us, t * h * r * 4 + distinct * r * 2, 2 * t * h * seen * 2 * r)
             us = _time(lambda: ops.head_gemm(q, uk))
             add("mitilix", "head_gemm (keys)", phase, us, t * h * (d + r) * 2 + h * r * d * 2, 2 * t * h * r * d)
@@ -266,8 +267,10 @@ def run(size: str, what: str, clocks) -> None:
         lines = []
         if what in ("all", "throughput"):
             for model, make in (("mitilix", mitilix_config), ("mistral", mistral_config)):
-                lines.append({"design": model, "size": name, "shape": s, "prompt": 2048, "dtype": "bf16",
-                              "data": "synthetic", **throughput(make(s))})
+                # a process per model: the device memory of one is gone when the next sizes its pool
+                with mp.get_context("spawn").Pool(1) as pool:
+                    lines.append({"design": model, "size": name, "shape": s, "prompt": 2048, "dtype": "bf16",
+                                  "data": "synthetic", **pool.apply(throughput, (make(s),))})
         if what in ("all", "kernels"):
             lines += [{"size": name, **r} for r in kernels(s)]
         seen = clocks.stop()

@@ -1,7 +1,8 @@
 // Latent attention: every query head attends to one latent row per position that is key and value
 // at once ([pages, page_size, R] of one layer of the latent pool), causal, with a sliding window.
 //
-//   latent_norm_store_kernel   RMS norm of this step's latents, into their pool slots
+//   latent_norm_store_kernel   RMS norm of this step's latents, into their pool slots (in a decode step extra CTAs
+//                              of the query projection do it)
 //   head_gemm_kernel           per-head projections into and out of the latent space (merging a split's ranges)
 //   latent_attention_kernel    bf16: 16 / 32 / 64 (position, head) rows per CTA against 64-token tiles
 //                              that are fetched once (cp.async, two or three stages, through the block table)
@@ -28,26 +29,40 @@ __device__ __forceinline__ float ex2(float x) {
 }
 
 // ------------------------------------------------------------------------------------------ store
-template <typename T>
-__global__ void __launch_bounds__(128) latent_norm_store_kernel(const T* __restrict__ c, long long ldc,
-                                                                const float* __restrict__ weight, T* __restrict__ pool,
-                                                                const int32_t* __restrict__ out_loc, int rows, int rank,
-                                                                int width, float eps, long long num_slots) {
-  pdl_enter();
-  const int t = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-  if (t >= rows) return;
-  const T* src = c + (size_t)t * ldc;
+template <typename T> struct StoreArgs {
+  const T* c;             // [rows, width] with row stride ldc
+  long long ldc;
+  const float* weight;
+  T* pool;
+  const int32_t* out_loc;
+  int rows, rank, width;
+  float eps;
+  long long num_slots;
+};
+
+// one warp per row
+template <typename T> __device__ __forceinline__ void store_latent(const StoreArgs<T>& a, int t, int lane) {
+  const T* src = a.c + (size_t)t * a.ldc;
   float s = 0.f;
-  for (int i = lane; i < rank; i += 32) {
+#pragma unroll 4
+  for (int i = lane; i < a.rank; i += 32) {
     const float v = to_float(src[i]);
     s = fmaf(v, v, s);
   }
   s = warp_sum(s);
-  const float sc = 1.f / sqrtf(s / (float)rank + eps);
-  const long long slot = out_loc[t];
-  if (MSGL_OOB(slot, num_slots) || slot < 0 || slot >= num_slots) return;
-  T* dst = pool + slot * width;
-  for (int i = lane; i < width; i += 32) dst[i] = from_float<T>(i < rank ? to_float(src[i]) * sc * weight[i] : 0.f);
+  const float sc = 1.f / sqrtf(s / (float)a.rank + a.eps);
+  const long long slot = a.out_loc[t];
+  if (MSGL_OOB(slot, a.num_slots) || slot < 0 || slot >= a.num_slots) return;
+  T* dst = a.pool + slot * a.width;
+#pragma unroll 4
+  for (int i = lane; i < a.width; i += 32)
+    dst[i] = from_float<T>(i < a.rank ? to_float(src[i]) * sc * a.weight[i] : 0.f);
+}
+
+template <typename T> __global__ void __launch_bounds__(128) latent_norm_store_kernel(const StoreArgs<T> a) {
+  pdl_enter();
+  const int t = blockIdx.x * 4 + (threadIdx.x >> 5);
+  if (t < a.rows) store_latent(a, t, threadIdx.x & 31);
 }
 
 // ------------------------------------------------------------------------------------------ attention args
@@ -170,6 +185,7 @@ struct HeadGemmArgs {
   const float* ws_o;      // [splits, T * H, K]
   const float* ws_lse;    // [splits, T * H]
   int splits, H;
+  StoreArgs<__nv_bfloat16> store;   // store.c != null: the CTAs at blockIdx.y == H store the step's latents
 };
 
 constexpr int kMaxSplits = 16;
@@ -180,6 +196,12 @@ __global__ void __launch_bounds__(128) head_gemm_kernel(const HeadGemmArgs a) {
   __shared__ float part[COMBINE ? kMaxSplits : 1][64];
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int n0 = blockIdx.x * 64, h = blockIdx.y, t0 = blockIdx.z * 64;
+  if (h == a.H) {
+    pdl_enter();
+    for (int r = blockIdx.x * 4 + warp; r < 64; r += gridDim.x * 4)
+      if (t0 + r < a.T) store_latent(a.store, t0 + r, lane);
+    return;
+  }
   const int panels = (a.K + 63) / 64;
   const __nv_bfloat16* xh = a.x + (long long)h * a.hx;
   const __nv_bfloat16* wh = a.w + (long long)h * a.N * a.K;
@@ -551,8 +573,9 @@ MSGL_API int msgl_latent_norm_store(const void* c, long long ldc, const void* we
   if (rank <= 0 || rank > width) return MSGL_BAD_ARG;
   dim3 grid((rows + 3) / 4);
 #define STORE(T)                                                                                                    \
-  msgl_launch(latent_norm_store_kernel<T>, grid, dim3(128), 0, stream, (const T*)c, ldc, (const float*)weight,      \
-              (T*)pool, (const int32_t*)out_loc, rows, rank, width, eps, num_slots)
+  msgl_launch(latent_norm_store_kernel<T>, grid, dim3(128), 0, stream,                                              \
+              StoreArgs<T>{(const T*)c, ldc, (const float*)weight, (T*)pool, (const int32_t*)out_loc, rows, rank,   \
+                           width, eps, num_slots})
   if (dtype == MSGL_BF16) STORE(__nv_bfloat16);
   else if (dtype == MSGL_F32) STORE(float);
   else return MSGL_BAD_ARG;
@@ -563,14 +586,19 @@ MSGL_API int msgl_latent_norm_store(const void* c, long long ldc, const void* we
 
 MSGL_API int msgl_head_gemm(const void* x, long long ldx, long long hx, const void* w, void* out, long long ldo,
                             long long ho, int T, int H, int N, int K, int static_weights, const void* ws_o, const void* ws_lse,
-                            int splits, cudaStream_t stream) {
+                            int splits, const void* c, long long ldc, const void* norm, void* pool,
+                            const void* out_loc, int rank, int width, float eps, long long num_slots,
+                            cudaStream_t stream) {
   if (T <= 0) return T == 0 ? MSGL_OK : MSGL_BAD_ARG;
   if (H <= 0 || H > 65535 || N % 8 || K % 8 || ldx % 8 || hx % 8 || ldo % 2 || ho % 2 || (uintptr_t)x % 16 ||
       (uintptr_t)w % 16 || (uintptr_t)out % 4 || T > 65535 * 64)
     return MSGL_BAD_ARG;
   HeadGemmArgs a{(const __nv_bfloat16*)x, ldx, hx, (const __nv_bfloat16*)w, (__nv_bfloat16*)out, ldo, ho, T, N, K,
-                 static_weights, (const float*)ws_o, (const float*)ws_lse, splits, H};
-  dim3 grid((N + 63) / 64, H, (T + 63) / 64);
+                 static_weights, (const float*)ws_o, (const float*)ws_lse, splits, H,
+                 StoreArgs<__nv_bfloat16>{(const __nv_bfloat16*)c, ldc, (const float*)norm, (__nv_bfloat16*)pool,
+                                          (const int32_t*)out_loc, T, rank, width, eps, num_slots}};
+  if (c != nullptr && (rank <= 0 || rank > width || H >= 65535)) return MSGL_BAD_ARG;
+  dim3 grid((N + 63) / 64, H + (c != nullptr), (T + 63) / 64);
   if (splits > 1) {
     if (splits > kMaxSplits || ws_o == nullptr || ws_lse == nullptr || (uintptr_t)ws_o % 16) return MSGL_BAD_ARG;
     msgl_launch(head_gemm_kernel<true>, grid, dim3(128), 0, stream, a);

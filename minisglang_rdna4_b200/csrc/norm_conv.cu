@@ -1,8 +1,9 @@
 // fp32 residual stream of models whose layers read one scalar-gain RMS norm through short causal
 // depthwise convolutions: embedding + learned position, residual add + norm + convolutions, exact
-// gelu. The convolution of a row needs the normalised rows ahead of it; a CTA recomputes the few
-// rows ahead of its block from the residual instead of reading another CTA's output, so one pass
-// over the rows is enough and the residual goes to a second buffer.
+// gelu. The convolution of a row needs the normalised rows ahead of it. Steps of few rows per request
+// take one kernel, in which a CTA recomputes the rows ahead of its block from the residual instead of
+// reading another CTA's output; steps of many rows take a pass for the residual and the row norms and
+// a pass for the convolutions. The new residual goes to a second buffer.
 #include "common.cuh"
 
 using namespace msgl;
@@ -239,128 +240,116 @@ __global__ void __launch_bounds__(1024) norm_conv_kernel(const NormConvArgs a) {
       }
 }
 
-// Prefill form: kRows rows per CTA. First every warp takes rows of its own (residual add, sum of squares), then every
-// thread walks down the rows of its four channels, which needs no barrier per row. width and cols multiples of 4.
+// Prefill form, two streaming passes. First a warp per row: residual add and gain / rms (one float per row). Then a
+// thread per four channels walks down kRows rows; the rows ahead of its block are read back from the new residual, so
+// no CTA waits for another. width and cols multiples of 4.
 constexpr int kRows = 16;
 
-template <typename T, int MT>
-__global__ void __launch_bounds__(256, MT <= 4 ? 3 : 2) norm_conv_rows_kernel(const NormConvArgs a) {
+__global__ void __launch_bounds__(256) residual_rms_kernel(const NormConvArgs a, float* __restrict__ scale) {
   pdl_enter();
-  __shared__ float s_scale[kRows + 2 * MT];
-  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-  const int b = blockIdx.y;
-  const int lo = a.cu_q[b], n = a.cu_q[b + 1] - lo;
-  const int r0 = blockIdx.x * kRows;
-  if (r0 >= n) return;
-  const int r1 = min(r0 + kRows, n), hist_n = a.taps - 1;
-  const int first = max(r0 - hist_n, 0);
-  // the CTA that reads a request's tail also writes the new one, from rows that may be another CTA's
-  const int tail = r0 == 0 && r1 < n ? n - hist_n : n;
-  const int n_main = r1 - first, n_all = n_main + (n - tail);
-  const float gain = a.gain[0];
-  auto residual = [&](int r, int c) {
-    const size_t row = (size_t)(lo + r);
-    float4 x = *reinterpret_cast<const float4*>(a.x + row * a.width + c);
-    for (int p = 0; p < a.planes; ++p) {
-      const float4 d = *reinterpret_cast<const float4*>(a.delta + p * a.plane_stride + row * a.ldd + c);
-      x.x += d.x; x.y += d.y; x.z += d.z; x.w += d.w;
-    }
-    return x;
-  };
-  for (int i = warp; i < n_all; i += 8) {
-    const int r = i < n_main ? first + i : tail + i - n_main;
-    const bool own = i < n_main && r >= r0 && a.x_out != a.x;
-    float s = 0.f;
+  const int row = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (row >= a.rows) return;
+  const float* src = a.x + (size_t)row * a.width;
+  const float* add = a.delta + (size_t)row * a.ldd;
+  float* dst = a.x_out + (size_t)row * a.width;
+  float s = 0.f;
 #pragma unroll 4
-    for (int c = lane * 4; c < a.width; c += 128) {
-      const float4 x = residual(r, c);
-      s = fmaf(x.x, x.x, s);
-      s = fmaf(x.y, x.y, s);
-      s = fmaf(x.z, x.z, s);
-      s = fmaf(x.w, x.w, s);
-      if (own) *reinterpret_cast<float4*>(a.x_out + (size_t)(lo + r) * a.width + c) = x;
+  for (int c = lane * 4; c < a.width; c += 128) {
+    float4 x = *reinterpret_cast<const float4*>(src + c);
+    if (a.planes > 0) {
+      for (int p = 0; p < a.planes; ++p) {
+        const float4 d = *reinterpret_cast<const float4*>(add + p * a.plane_stride + c);
+        x.x += d.x; x.y += d.y; x.z += d.z; x.w += d.w;
+      }
+      *reinterpret_cast<float4*>(dst + c) = x;
     }
-    s = warp_sum(s);
-    if (lane == 0) s_scale[i] = gain / sqrtf(s / (float)a.width + a.eps);
+    s = fmaf(x.x, x.x, s);
+    s = fmaf(x.y, x.y, s);
+    s = fmaf(x.z, x.z, s);
+    s = fmaf(x.w, x.w, s);
   }
-  __syncthreads();
+  s = warp_sum(s);
+  if (lane == 0) scale[row] = a.gain[0] / sqrtf(s / (float)a.width + a.eps);
+}
+
+// x_out holds the residual; grid (cols / 1024, row blocks, requests).
+template <typename T, int MT>
+__global__ void __launch_bounds__(256) conv_rows_kernel(const NormConvArgs a, const float* __restrict__ scale) {
+  pdl_enter();
+  const int b = blockIdx.z;
+  const int lo = a.cu_q[b], n = a.cu_q[b + 1] - lo;
+  const int r0 = blockIdx.y * kRows, c = (blockIdx.x * 256 + threadIdx.x) * 4;
+  if (r0 >= n || c >= a.cols) return;
+  const int r1 = min(r0 + kRows, n), hist_n = a.taps - 1;
+  const bool in = c < a.width;
   float* st = r0 == 0 && hist_n > 0 ? a.state + (size_t)a.slots[b] * a.width * hist_n : nullptr;
   const bool keep = st != nullptr && a.has_state[b] != 0;
-  T* y1 = reinterpret_cast<T*>(a.y1);
-  T* y2 = reinterpret_cast<T*>(a.y2);
-  for (int c = tid * 4; c < a.cols; c += 1024) {
-    const bool in = c < a.width;
-    float f1[MT][4], f2[MT][4], hist[MT][4];
+  T* y1 = reinterpret_cast<T*>(a.y1) + c;
+  T* y2 = a.y2 != nullptr ? reinterpret_cast<T*>(a.y2) + c : nullptr;
+  auto row_h = [&](int r, float (&h)[4]) {
+    const float4 x = in ? *reinterpret_cast<const float4*>(a.x_out + (size_t)(lo + r) * a.width + c)
+                        : make_float4(0.f, 0.f, 0.f, 0.f);
+    const float sc = scale[lo + r];
+    h[0] = x.x * sc; h[1] = x.y * sc; h[2] = x.z * sc; h[3] = x.w * sc;
+  };
+  // hist[MT - taps .. MT - 2]: the rows ahead; hist[MT - 1]: the row itself
+  float f1[MT][4], f2[MT][4], hist[MT][4];
 #pragma unroll
-    for (int j = 0; j < MT; ++j) {
-      const int src = j - (MT - a.taps);
-      float4 q1 = make_float4(0.f, 0.f, 0.f, 0.f), q2 = q1, q3 = q1;
-      if (in && src >= 0) {
-        q1 = *reinterpret_cast<const float4*>(a.w1 + (size_t)src * a.width + c);
-        if (a.w2 != nullptr) q2 = *reinterpret_cast<const float4*>(a.w2 + (size_t)src * a.width + c);
-        if (keep && src < hist_n) q3 = *reinterpret_cast<const float4*>(st + (size_t)src * a.width + c);
+  for (int j = 0; j < MT; ++j) {
+    const int src = j - (MT - a.taps);
+    float4 q1 = make_float4(0.f, 0.f, 0.f, 0.f), q2 = q1, q3 = q1;
+    if (in && src >= 0) {
+      q1 = *reinterpret_cast<const float4*>(a.w1 + (size_t)src * a.width + c);
+      if (y2 != nullptr) q2 = *reinterpret_cast<const float4*>(a.w2 + (size_t)src * a.width + c);
+      if (keep && src < hist_n) q3 = *reinterpret_cast<const float4*>(st + (size_t)src * a.width + c);
+    }
+    f1[j][0] = q1.x; f1[j][1] = q1.y; f1[j][2] = q1.z; f1[j][3] = q1.w;
+    f2[j][0] = q2.x; f2[j][1] = q2.y; f2[j][2] = q2.z; f2[j][3] = q2.w;
+    hist[j][0] = q3.x; hist[j][1] = q3.y; hist[j][2] = q3.z; hist[j][3] = q3.w;
+    if (r0 > 0 && src >= 0 && src < hist_n) row_h(r0 - hist_n + src, hist[j]);
+  }
+#pragma unroll 4
+  for (int r = r0; r < r1; ++r) {
+    row_h(r, hist[MT - 1]);
+    float o1[4], o2[4];
+#pragma unroll
+    for (int v = 0; v < 4; ++v) {
+      o1[v] = o2[v] = hist[MT - 1][v];
+#pragma unroll
+      for (int j = 0; j < MT; ++j) {
+        o1[v] = fmaf(f1[j][v], hist[j][v], o1[v]);
+        o2[v] = fmaf(f2[j][v], hist[j][v], o2[v]);
       }
-      f1[j][0] = q1.x; f1[j][1] = q1.y; f1[j][2] = q1.z; f1[j][3] = q1.w;
-      f2[j][0] = q2.x; f2[j][1] = q2.y; f2[j][2] = q2.z; f2[j][3] = q2.w;
-      hist[j][0] = q3.x; hist[j][1] = q3.y; hist[j][2] = q3.z; hist[j][3] = q3.w;
     }
-    // hist[MT - taps .. MT - 2]: the rows ahead; hist[MT - 1]: the row itself
-#pragma unroll 2
-    for (int i = 0; i < n_main; ++i) {
-      const int r = first + i;
-      float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
-      if (in) x = r >= r0 ? *reinterpret_cast<const float4*>(a.x_out + (size_t)(lo + r) * a.width + c) : residual(r, c);
-      const float sc = s_scale[i];
-      hist[MT - 1][0] = x.x * sc; hist[MT - 1][1] = x.y * sc; hist[MT - 1][2] = x.z * sc; hist[MT - 1][3] = x.w * sc;
-      if (r >= r0) {
-        float o1[4], o2[4];
-#pragma unroll
-        for (int v = 0; v < 4; ++v) {
-          o1[v] = o2[v] = hist[MT - 1][v];
-#pragma unroll
-          for (int j = 0; j < MT; ++j) {
-            o1[v] = fmaf(f1[j][v], hist[j][v], o1[v]);
-            o2[v] = fmaf(f2[j][v], hist[j][v], o2[v]);
-          }
-        }
-        const size_t off = (size_t)(lo + r) * a.cols + c;
-        if constexpr (sizeof(T) == 2) {
-          uint2 q;
-          *reinterpret_cast<typename Pack2<T>::type*>(&q.x) = Pack2<T>::make(o1[0], o1[1]);
-          *reinterpret_cast<typename Pack2<T>::type*>(&q.y) = Pack2<T>::make(o1[2], o1[3]);
-          *reinterpret_cast<uint2*>(y1 + off) = q;
-          if (y2 != nullptr) {
-            *reinterpret_cast<typename Pack2<T>::type*>(&q.x) = Pack2<T>::make(o2[0], o2[1]);
-            *reinterpret_cast<typename Pack2<T>::type*>(&q.y) = Pack2<T>::make(o2[2], o2[3]);
-            *reinterpret_cast<uint2*>(y2 + off) = q;
-          }
-        } else {
-          *reinterpret_cast<float4*>(y1 + off) = make_float4(o1[0], o1[1], o1[2], o1[3]);
-          if (y2 != nullptr) *reinterpret_cast<float4*>(y2 + off) = make_float4(o2[0], o2[1], o2[2], o2[3]);
-        }
+    const size_t off = (size_t)(lo + r) * a.cols;
+    if constexpr (sizeof(T) == 2) {
+      uint2 q;
+      *reinterpret_cast<typename Pack2<T>::type*>(&q.x) = Pack2<T>::make(o1[0], o1[1]);
+      *reinterpret_cast<typename Pack2<T>::type*>(&q.y) = Pack2<T>::make(o1[2], o1[3]);
+      *reinterpret_cast<uint2*>(y1 + off) = q;
+      if (y2 != nullptr) {
+        *reinterpret_cast<typename Pack2<T>::type*>(&q.x) = Pack2<T>::make(o2[0], o2[1]);
+        *reinterpret_cast<typename Pack2<T>::type*>(&q.y) = Pack2<T>::make(o2[2], o2[3]);
+        *reinterpret_cast<uint2*>(y2 + off) = q;
       }
-#pragma unroll
-      for (int j = 0; j + 1 < MT; ++j)
-#pragma unroll
-        for (int v = 0; v < 4; ++v) hist[j][v] = hist[j + 1][v];
-    }
-    if (st == nullptr || !in) continue;
-    for (int i = n_main; i < n_all; ++i) {
-      const float4 x = residual(tail + i - n_main, c);
-      const float sc = s_scale[i];
-      hist[MT - 1][0] = x.x * sc; hist[MT - 1][1] = x.y * sc; hist[MT - 1][2] = x.z * sc; hist[MT - 1][3] = x.w * sc;
-#pragma unroll
-      for (int j = 0; j + 1 < MT; ++j)
-#pragma unroll
-        for (int v = 0; v < 4; ++v) hist[j][v] = hist[j + 1][v];
+    } else {
+      *reinterpret_cast<float4*>(y1 + off) = make_float4(o1[0], o1[1], o1[2], o1[3]);
+      if (y2 != nullptr) *reinterpret_cast<float4*>(y2 + off) = make_float4(o2[0], o2[1], o2[2], o2[3]);
     }
 #pragma unroll
-    for (int j = 0; j + 1 < MT; ++j) {
-      const int dst = j - (MT - a.taps);
-      if (dst >= 0)
-        *reinterpret_cast<float4*>(st + (size_t)dst * a.width + c) =
-            make_float4(hist[j][0], hist[j][1], hist[j][2], hist[j][3]);
-    }
+    for (int j = 0; j + 1 < MT; ++j)
+#pragma unroll
+      for (int v = 0; v < 4; ++v) hist[j][v] = hist[j + 1][v];
+  }
+  if (st == nullptr || !in) return;
+  // the thread that read this part of the tail also writes the new one, whichever block the last rows are in
+#pragma unroll
+  for (int j = 0; j + 1 < MT; ++j) {
+    const int dst = j - (MT - a.taps);
+    if (dst < 0) continue;
+    if (r1 < n) row_h(n - hist_n + dst, hist[j]);
+    *reinterpret_cast<float4*>(st + (size_t)dst * a.width + c) =
+        make_float4(hist[j][0], hist[j][1], hist[j][2], hist[j][3]);
   }
 }
 
@@ -377,7 +366,7 @@ void launch_norm_conv(const NormConvArgs& a, dim3 grid, int threads, cudaStream_
 }
 
 template <typename T>
-int norm_conv_typed(NormConvArgs a, int B, int max_q, cudaStream_t s) {
+int norm_conv_typed(NormConvArgs a, float* scale, int B, int max_q, cudaStream_t s) {
   const bool conv = a.w1 != nullptr;
   // enough rows per CTA to make the recomputed rows cheap (and at least taps - 1 of them)
   a.block_rows = conv ? (a.taps > 8 ? 32 : 16) : 1;
@@ -386,13 +375,13 @@ int norm_conv_typed(NormConvArgs a, int B, int max_q, cudaStream_t s) {
   const bool vec = a.width % 4 == 0 && a.cols % 4 == 0 && a.ldd % 4 == 0 && (uintptr_t)a.delta % 16 == 0;
   const int per = vec ? 4 : 1;
   const int groups = (a.cols + per - 1) / per;
-  if (vec && conv && max_q > 4 && a.taps <= 8) {
-    a.block_rows = kRows;
-    const dim3 rows_grid((n + kRows - 1) / kRows, B);
+  if (vec && conv && scale != nullptr && a.taps <= 8 && n <= 65535 * kRows) {
+    msgl_launch(residual_rms_kernel, dim3((a.rows + 7) / 8), dim3(256), 0, s, a, scale);
+    const dim3 conv_grid((a.cols + 1023) / 1024, (n + kRows - 1) / kRows, B);
     if (a.taps <= 4)
-      msgl_launch(norm_conv_rows_kernel<T, 4>, rows_grid, dim3(256), 0, s, a);
+      msgl_launch(conv_rows_kernel<T, 4>, conv_grid, dim3(256), 0, s, a, scale);
     else
-      msgl_launch(norm_conv_rows_kernel<T, 8>, rows_grid, dim3(256), 0, s, a);
+      msgl_launch(conv_rows_kernel<T, 8>, conv_grid, dim3(256), 0, s, a, scale);
     MSGL_CHECK_LAUNCH("norm_conv_rows");
     return MSGL_OK;
   }
@@ -409,6 +398,18 @@ int norm_conv_typed(NormConvArgs a, int B, int max_q, cudaStream_t s) {
   }
   MSGL_CHECK_LAUNCH("norm_conv");
   return MSGL_OK;
+}
+
+// erf by formula 7.1.26 of Abramowitz and Stegun, Handbook of Mathematical Functions (absolute error at
+// most 1.5e-7): far below what a 16-bit result keeps. The fp32 form calls erff.
+__device__ __forceinline__ float erf_as(float x) {
+  const float ax = fabsf(x);
+  const float t = __fdividef(1.f, fmaf(0.3275911f, ax, 1.f));
+  float p = fmaf(1.061405429f, t, -1.453152027f);
+  p = fmaf(p, t, 1.421413741f);
+  p = fmaf(p, t, -0.284496736f);
+  p = fmaf(p, t, 0.254829592f);
+  return copysignf(1.f - p * t * __expf(-ax * ax), x);
 }
 
 // Exact gelu of [rows, n] with row strides; n a multiple of the vector width.
@@ -428,7 +429,10 @@ __global__ void __launch_bounds__(256) gelu_erf_kernel(const T* __restrict__ x, 
     v[0] = q.x; v[1] = q.y; v[2] = q.z; v[3] = q.w;
   }
 #pragma unroll
-  for (int e = 0; e < V; ++e) v[e] = 0.5f * v[e] * (1.f + erff(v[e] * 0.70710678118654752f));
+  for (int e = 0; e < V; ++e) {
+    const float z = v[e] * 0.70710678118654752f;
+    v[e] = 0.5f * v[e] * (1.f + (sizeof(T) == 2 ? erf_as(z) : erff(z)));
+  }
   if constexpr (sizeof(T) == 2)
     store8(out + r * ldo + c, v);
   else
@@ -453,16 +457,16 @@ MSGL_API int msgl_embed_positions(const void* ids, const void* w, const void* po
 
 MSGL_API int msgl_norm_conv(const void* x, void* x_out, const void* delta, int planes, long long plane_stride,
                             long long ldd, const void* gain, float eps, const void* w1, const void* w2, void* y1,
-                            void* y2, void* state, const void* cu_q, const void* slots, const void* has_state, int rows,
-                            int width, int cols, int taps, int B, int max_q, int dtype, cudaStream_t stream) {
+                            void* y2, void* state, const void* cu_q, const void* slots, const void* has_state, void* scale,
+                            int rows, int width, int cols, int taps, int B, int max_q, int dtype, cudaStream_t stream) {
   if (rows <= 0) return rows == 0 ? MSGL_OK : MSGL_BAD_ARG;
   if (taps < 1 || taps > 32 || cols < width || (planes > 0 && x == x_out)) return MSGL_BAD_ARG;
   if (w1 != nullptr && (B <= 0 || max_q <= 0)) return MSGL_BAD_ARG;
   NormConvArgs a{(const float*)x, (float*)x_out, (const float*)delta, planes, plane_stride, ldd, (const float*)gain, eps,
                  (const float*)w1, (const float*)w2, y1, y2, (float*)state, (const int32_t*)cu_q,
                  (const int32_t*)slots, (const int32_t*)has_state, rows, width, cols, taps, 0};
-  if (dtype == MSGL_BF16) return norm_conv_typed<__nv_bfloat16>(a, B, max_q, stream);
-  if (dtype == MSGL_F32) return norm_conv_typed<float>(a, B, max_q, stream);
+  if (dtype == MSGL_BF16) return norm_conv_typed<__nv_bfloat16>(a, (float*)scale, B, max_q, stream);
+  if (dtype == MSGL_F32) return norm_conv_typed<float>(a, (float*)scale, B, max_q, stream);
   return MSGL_BAD_ARG;
 }
 

@@ -8,7 +8,6 @@ from __future__ import annotations
 
 import torch
 
-from .. import ops
 from ..core import get_global_ctx
 from ..parallel.info import get_tp_info
 from ..utils import div_even
@@ -43,13 +42,11 @@ class LatentAttentionLayer(BaseOP):
         batch = ctx.batch
         t, nq = x.shape[0], self._h * self._dim
         qc = self.q_proj.forward(x)
-        if self._own:
-            ops.latent_norm_store(qc[:, nq:], self.latent_norm, self._spec.kv_rank, self._eps,
-                                  ctx.kv_cache.rows(self._row), batch.out_loc)
+        store = (qc[:, nq:], self.latent_norm, self._spec.kv_rank, self._eps) if self._own else None
         q = qc[:, :nq].unflatten(1, (self._h, self._dim))
         ctx.attn_backend.latent_forward(q, self.up_k, self.up_v, self._row, batch, scale=self._spec.scale,
                                         window=self._spec.window, out=out.unflatten(1, (self._h, self._vdim)),
-                                        expand_k=self._expand_k)
+                                        expand_k=self._expand_k, store=store)
 
     def _post_load_self(self) -> None:
         if self.up_k.is_cuda and self.up_k.dtype == torch.bfloat16:

@@ -237,9 +237,10 @@ def latent_norm_store(c, weight, rank: int, eps: float, rows, out_loc):
     return ref.latent_norm_store(c, weight, rank, eps, rows, out_loc)
 
 
-def head_gemm(x, w, out=None):
+def head_gemm(x, w, out=None, store=None):
     if x.is_cuda:
-        return _cuda().head_gemm(x, w, out)
+        return _cuda().head_gemm(x, w, out, store)
+    assert store is None
     return ref.head_gemm(x, w, out)
 
 

@@ -909,10 +909,11 @@ def _bind_latent():
         return
     bind("msgl_gemm_f32", c_i, [c_p, c_ll, c_ll, c_p, c_ll, c_ll, c_p, c_ll, c_ll, c_i, c_i, c_i, c_i, c_p])
     bind("msgl_embed_positions", c_i, [c_p] * 5 + [c_i] * 6 + [c_p])
-    bind("msgl_norm_conv", c_i, [c_p, c_p, c_p, c_i, c_ll, c_ll, c_p, c_f] + [c_p] * 8 + [c_i] * 7 + [c_p])
+    bind("msgl_norm_conv", c_i, [c_p, c_p, c_p, c_i, c_ll, c_ll, c_p, c_f] + [c_p] * 9 + [c_i] * 7 + [c_p])
     bind("msgl_gelu_erf", c_i, [c_p, c_ll, c_p, c_ll, c_i, c_i, c_i, c_p])
     bind("msgl_latent_norm_store", c_i, [c_p, c_ll, c_p, c_p, c_p, c_i, c_i, c_i, c_f, c_ll, c_i, c_p])
-    bind("msgl_head_gemm", c_i, [c_p, c_ll, c_ll, c_p, c_p, c_ll, c_ll, c_i, c_i, c_i, c_i, c_i, c_p, c_p, c_i, c_p])
+    bind("msgl_head_gemm", c_i, [c_p, c_ll, c_ll, c_p, c_p, c_ll, c_ll, c_i, c_i, c_i, c_i, c_i, c_p, c_p, c_i,
+                                 c_p, c_ll, c_p, c_p, c_p, c_i, c_i, c_f, c_ll, c_p])
     bind("msgl_latent_gather", c_i, [c_p] * 5 + [c_i] * 5 + [c_p])
     bind("msgl_attn_prefill_pos", c_i, [c_p, c_ll, c_ll, c_p, c_p, c_i, c_p, c_ll, c_ll, c_p, c_i, c_i, c_i, c_i, c_i, c_i,
                                         c_f, c_i, c_p])
@@ -964,10 +965,12 @@ def add_scalar_norm_conv(x, delta, gain, eps, w1, w2, state, cu_q, slots, has_st
         taps, b = w1.shape[0], cu_q.numel() - 1
         assert w1.is_contiguous() and w1.dtype == torch.float32 and state.is_contiguous()
         assert state.dtype == torch.float32 and state.shape[1:] == (taps - 1, width)
+    # many rows per request: two streaming passes with the row norms in between
+    scale = torch.empty(rows, dtype=torch.float32, device=x.device) if w1 is not None and max_q > 4 else None
     check(lib().msgl_norm_conv(_p(x), _p(x_out), _p(delta), planes, plane_stride, ldd, _p(gain), eps, _p(w1), _p(w2),
-                               _p(y1), _p(y2), _p(state), _p(cu_q), _p(slots), _p(has_state), rows, width, out_cols,
-                               taps, b, int(max_q), _DT[out_dtype], _stream()), "norm_conv")
-    _count("add_scalar_norm_conv", "norm_conv_kernel")
+                               _p(y1), _p(y2), _p(state), _p(cu_q), _p(slots), _p(has_state), _p(scale), rows, width,
+                               out_cols, taps, b, int(max_q), _DT[out_dtype], _stream()), "norm_conv")
+    _count("add_scalar_norm_conv", "norm_conv_kernel", 1 if scale is None else 2)
     return x_out, y1, y2
 
 
@@ -993,8 +996,12 @@ def latent_norm_store(c, weight, rank, eps, rows, out_loc):
     _count("latent_norm_store", "latent_norm_store_kernel")
 
 
-def head_gemm(x, w, out=None):
-    """``x [T, H, K]`` (any row and head stride), ``w [H, N, K]`` -> ``[T, H, N]``."""
+_NO_STORE = (None, 0, None, None, None, 0, 0, 0.0, 0)
+
+
+def head_gemm(x, w, out=None, store=None):
+    """``x [T, H, K]`` (any row and head stride), ``w [H, N, K]`` -> ``[T, H, N]``. ``store``: the arguments of
+    ``latent_norm_store`` to run in the same launch (16-bit)."""
     _bind_latent()
     t, h, k = x.shape
     n = w.shape[1]
@@ -1003,12 +1010,19 @@ def head_gemm(x, w, out=None):
         out = torch.empty((t, h, n), dtype=x.dtype, device=x.device)
     assert out.stride(2) == 1 and out.shape == (t, h, n) and out.dtype == x.dtype
     if x.dtype == torch.float32:
+        assert store is None
         check(lib().msgl_gemm_f32(_p(x), x.stride(0), x.stride(1), _p(w), k, n * k, _p(out), out.stride(0),
                                   out.stride(1), t, n, k, h, _stream()), "head_gemm")
         _count("head_gemm", "gemm_f32_kernel")
         return out
+    stored = _NO_STORE
+    if store is not None:
+        c, norm, rank, eps, rows, out_loc = store
+        assert c.stride(1) == 1 and c.shape[0] == t and c.dtype == x.dtype == rows.dtype and norm.dtype == torch.float32
+        stored = (_p(c), c.stride(0), _p(norm), _p(rows), _p(out_loc), rank, rows.shape[2], eps,
+                  rows.shape[0] * rows.shape[1])
     check(lib().msgl_head_gemm(_p(x), x.stride(0), x.stride(1), _p(w), _p(out), out.stride(0), out.stride(1), t, h, n, k,
-                               int(STATIC_WEIGHTS), None, None, 1, _stream()), "head_gemm")
+                               int(STATIC_WEIGHTS), None, None, 1, *stored, _stream()), "head_gemm")
     _count("head_gemm", "head_gemm_kernel")
     return out
 
@@ -1030,7 +1044,7 @@ def head_gemm_combine(x: LatentSplit, w, out):
     n = w.shape[1]
     assert w.is_contiguous() and w.shape == (h, n, k) and out.stride(2) == 1 and out.shape == (t, h, n)
     check(lib().msgl_head_gemm(None, 0, 0, _p(w), _p(out), out.stride(0), out.stride(1), t, h, n, k, int(STATIC_WEIGHTS),
-                               _p(x.ws_o), _p(x.ws_lse), x.ws_o.shape[0], _stream()), "head_gemm")
+                               _p(x.ws_o), _p(x.ws_lse), x.ws_o.shape[0], *_NO_STORE, _stream()), "head_gemm")
     _count("head_gemm", "head_gemm_kernel")
     return out
 

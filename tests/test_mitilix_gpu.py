@@ -96,6 +96,8 @@ def test_gelu_and_embedding():
     for dtype, tol in ((torch.float32, 1e-6), (torch.bfloat16, 1e-2)):
         out = torch.zeros(33, 64, dtype=dtype, device=DEV)
         ops.gelu_erf(x.to(DEV, dtype), out[:, 16:])
+        x[0] = torch.linspace(-6, 6, 48)
+        ops.gelu_erf(x.to(DEV, dtype), out[:, 16:])
         want = torch.nn.functional.gelu(x.to(dtype).double())
         torch.testing.assert_close(out[:, 16:].double().cpu(), want, rtol=tol, atol=tol)
         emb, pos = torch.randn(50, 40, generator=g).to(dtype), torch.randn(70, 40, generator=g).to(dtype)
@@ -115,6 +117,13 @@ def test_latent_norm_store(rank, width):
         ref.latent_norm_store(c[:, 24:], w, rank, 1e-5, pool, loc)
         ops.latent_norm_store(c.to(DEV)[:, 24:], w.to(DEV), rank, 1e-5, dev, loc.to(DEV))
         torch.testing.assert_close(dev.cpu(), pool, rtol=tol, atol=tol)
+        if dtype == torch.bfloat16:        # in the launch of the query projection
+            dev2 = torch.zeros_like(dev)
+            q, uk = torch.randn(13, 2, 32, generator=g).to(DEV, dtype), torch.randn(2, width, 32, generator=g).to(DEV, dtype)
+            torch.cuda.synchronize()
+            y = ops.head_gemm(q, uk, store=(c.to(DEV)[:, 24:], w.to(DEV), rank, 1e-5, dev2, loc.to(DEV)))
+            torch.testing.assert_close(dev2, dev, rtol=0, atol=0)
+            torch.testing.assert_close(y, ops.head_gemm(q, uk), rtol=0, atol=0)
 
 
 @pytest.mark.parametrize("r", [64, 128, 192, 256, 512, 1024])
