@@ -185,7 +185,7 @@ struct HeadGemmArgs {
   const float* ws_o;      // [splits, T * H, K]
   const float* ws_lse;    // [splits, T * H]
   int splits, H;
-  StoreArgs<__nv_bfloat16> store;   // store.c != null: the CTAs at blockIdx.y == H store the step's latents
+  StoreArgs<__nv_bfloat16> store;   // store.c != null: the CTAs at blockIdx.y >= H store the step's latents
 };
 
 constexpr int kMaxSplits = 16;
@@ -196,10 +196,10 @@ __global__ void __launch_bounds__(128) head_gemm_kernel(const HeadGemmArgs a) {
   __shared__ float part[COMBINE ? kMaxSplits : 1][64];
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int n0 = blockIdx.x * 64, h = blockIdx.y, t0 = blockIdx.z * 64;
-  if (h == a.H) {
+  if (h >= a.H) {                          // a warp per row of this block of 64
     pdl_enter();
-    for (int r = blockIdx.x * 4 + warp; r < 64; r += gridDim.x * 4)
-      if (t0 + r < a.T) store_latent(a.store, t0 + r, lane);
+    const int r = ((h - a.H) * gridDim.x + blockIdx.x) * 4 + warp;
+    if (r < 64 && t0 + r < a.T) store_latent(a.store, t0 + r, lane);
     return;
   }
   const int panels = (a.K + 63) / 64;
@@ -295,12 +295,12 @@ __global__ void __launch_bounds__(128) head_gemm_kernel(const HeadGemmArgs a) {
 // ------------------------------------------------------------------------------------------ attention
 template <int NP> struct LatentStages { static constexpr int value = NP <= 4 ? 3 : 2; };
 
-// NP: latent panels of 64 channels (R = 64 NP). WM row groups of 16 x WN = 8 / WM column groups: a warp
-// computes 16 rows x (64 / WN) keys of S and 16 rows x (R / WN) channels of O.
-template <int NP, int WM>
-__global__ void __launch_bounds__(256) latent_attention_kernel(const LatArgs a) {
+// NP: latent panels of 64 channels (R = 64 NP). WM row groups of 16 x WN column groups: a warp computes
+// 16 rows x (64 / WN) keys of S and 16 rows x (R / WN) channels of O.
+template <int NP, int WM, int WN>
+__global__ void __launch_bounds__(32 * WM * WN) latent_attention_kernel(const LatArgs a) {
   pdl_enter();
-  constexpr int R = NP * 64, WN = 8 / WM, MT = 16 * WM, TK = 64;
+  constexpr int R = NP * 64, MT = 16 * WM, TK = 64, NT = 32 * WM * WN;
   constexpr int CH = R / 8;                      // 16-byte chunks per row
   constexpr int NS = TK / WN / 8;                // key blocks of 8 per warp
   constexpr int NO = R / WN / 8;                 // channel blocks of 8 per warp
@@ -328,19 +328,32 @@ __global__ void __launch_bounds__(256) latent_attention_kernel(const LatArgs a) 
   const __nv_bfloat16* pool = reinterpret_cast<const __nv_bfloat16*>(a.pool);
   const int32_t* bt = a.block_table + (size_t)b * a.bt_stride;
 
-  auto load_tile = [&](int t) {
-    const uint32_t dst = c_s + (t % ST) * C_BYTES;
-    const int tok0 = (t_begin + t) * TK;
-    for (int id = tid; id < TK * CH; id += 256) {
-      const int r = id / CH, c = id % CH, tok = tok0 + r;
-      const bool ok = tok < kv_len;
-      const __nv_bfloat16* src = ok ? pool + token_slot(a, bt, tok) * R + c * 8 : pool;
-      cp16(dst + swz(r, c, CH), src, ok);
+  // Pool slots of the tile that is fetched next: lane i knows those of its rows i and i + 32 (-1 past the end), looked
+  // up one tile ahead so that the block table's latency is not in front of the copies.
+  int next_slot[2];
+  auto look_up = [&](int t) {
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      const int tok = (t_begin + t) * TK + i * 32 + lane;
+      next_slot[i] = t < n_tiles && tok < kv_len ? (int)token_slot(a, bt, tok) : -1;
     }
   };
+  auto load_tile = [&](int t) {
+    const uint32_t dst = c_s + (t % ST) * C_BYTES;
+    const int slot[2] = {next_slot[0], next_slot[1]};
+    look_up(t + 1);
+#pragma unroll
+    for (int i = 0; i < TK * CH / NT; ++i) {
+      const int id = tid + i * NT, r = id / CH, c = id % CH;
+      const int s0 = __shfl_sync(0xffffffffu, slot[0], r & 31), s1 = __shfl_sync(0xffffffffu, slot[1], r & 31);
+      const int sl = r < 32 ? s0 : s1;
+      cp16(dst + swz(r, c, CH), pool + (long long)(sl < 0 ? 0 : sl) * R + c * 8, sl >= 0);
+    }
+  };
+  look_up(0);
   {
     const __nv_bfloat16* q = reinterpret_cast<const __nv_bfloat16*>(a.q) + ((size_t)q0 * a.H + row0) * R;
-    for (int id = tid; id < MT * CH; id += 256) {
+    for (int id = tid; id < MT * CH; id += NT) {
       const int r = id / CH, c = id % CH;
       const bool ok = row0 + r < row1;
       cp16(q_s + swz(r, c, CH), ok ? q + (size_t)r * R + c * 8 : q, ok);
@@ -357,6 +370,8 @@ __global__ void __launch_bounds__(256) latent_attention_kernel(const LatArgs a) 
   const int pa = kv_len - q_len + min(row0 + ra, row1 - 1) / a.H, pb = kv_len - q_len + min(row0 + rb, row1 - 1) / a.H;
   const int lo_a = a.window > 0 ? pa - a.window + 1 : 0, lo_b = a.window > 0 ? pb - a.window + 1 : 0;
   const float sc = a.scale * kLog2eL;
+  constexpr bool QREG = WM == 1 && R <= 256;     // few rows: the queries fit in registers
+  uint32_t qf[QREG ? R / 16 : 1][4];
   float o[NO][4];
 #pragma unroll
   for (int i = 0; i < NO; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
@@ -368,20 +383,37 @@ __global__ void __launch_bounds__(256) latent_attention_kernel(const LatArgs a) 
     if (t + ST - 1 < n_tiles) load_tile(t + ST - 1);
     cp_commit();
     const uint32_t cb = c_s + (t % ST) * C_BYTES;
-    float s[NS][4];
+    float s[NS][4], s2[NS][4];                    // two accumulators: half as long a chain of dependent products
 #pragma unroll
-    for (int i = 0; i < NS; ++i) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.f;
-#pragma unroll 4
+    for (int i = 0; i < NS; ++i) {
+      s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.f;
+      s2[i][0] = s2[i][1] = s2[i][2] = s2[i][3] = 0.f;
+    }
+    if constexpr (QREG) {
+      if (t == 0) {
+#pragma unroll
+        for (int kk = 0; kk < R / 16; ++kk) ldm_x4(q_s + swz(wm * 16 + (lane & 15), kk * 2 + (lane >> 4), CH), qf[kk]);
+      }
+    }
+#pragma unroll (QREG ? R / 32 : 4)
     for (int kk = 0; kk < R / 32; ++kk) {
       uint32_t a0[4], a1[4];
-      ldm_x4(q_s + swz(wm * 16 + (lane & 15), kk * 4 + (lane >> 4), CH), a0);
-      ldm_x4(q_s + swz(wm * 16 + (lane & 15), kk * 4 + 2 + (lane >> 4), CH), a1);
+      if constexpr (QREG) {
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          a0[i] = qf[2 * kk][i];
+          a1[i] = qf[2 * kk + 1][i];
+        }
+      } else {
+        ldm_x4(q_s + swz(wm * 16 + (lane & 15), kk * 4 + (lane >> 4), CH), a0);
+        ldm_x4(q_s + swz(wm * 16 + (lane & 15), kk * 4 + 2 + (lane >> 4), CH), a1);
+      }
 #pragma unroll
       for (int nb = 0; nb < NS; ++nb) {
         uint32_t bf[4];
         ldm_x4(cb + swz(wn * (TK / WN) + nb * 8 + (lane & 7), kk * 4 + (lane >> 3), CH), bf);
         mma_bf16(s[nb], a0, bf[0], bf[1]);
-        mma_bf16(s[nb], a1, bf[2], bf[3]);
+        mma_bf16(s2[nb], a1, bf[2], bf[3]);
       }
     }
     const int tok0 = (t_begin + t) * TK + wn * (TK / WN) + (lane & 3) * 2;
@@ -391,8 +423,8 @@ __global__ void __launch_bounds__(256) latent_attention_kernel(const LatArgs a) 
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
         const int tok = tok0 + nb * 8 + e;
-        const float va = tok <= pa && tok >= lo_a ? s[nb][e] * sc : -INFINITY;
-        const float vb = tok <= pb && tok >= lo_b ? s[nb][2 + e] * sc : -INFINITY;
+        const float va = tok <= pa && tok >= lo_a ? (s[nb][e] + s2[nb][e]) * sc : -INFINITY;
+        const float vb = tok <= pb && tok >= lo_b ? (s[nb][2 + e] + s2[nb][2 + e]) * sc : -INFINITY;
         s[nb][e] = va;
         s[nb][2 + e] = vb;
         mx_a = fmaxf(mx_a, va);
@@ -498,7 +530,7 @@ __global__ void __launch_bounds__(256) latent_attention_kernel(const LatArgs a) 
   }
 }
 
-// One warp per (row, head); R a multiple of 64.
+// One warp per (row, head); R a multiple of 64, up to 512 (four float4 per lane).
 __global__ void __launch_bounds__(128) latent_combine_kernel(const float* __restrict__ ws_o,
                                                              const float* __restrict__ ws_lse,
                                                              __nv_bfloat16* __restrict__ out, int rows, int R,
@@ -506,30 +538,49 @@ __global__ void __launch_bounds__(128) latent_combine_kernel(const float* __rest
   pdl_enter();
   const int row = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
   if (row >= rows) return;
-  float m = -INFINITY;
-  for (int s = 0; s < splits; ++s) m = fmaxf(m, ws_lse[(size_t)s * rows + row]);
-  float total = 0.f;
-  for (int s = 0; s < splits; ++s) total += m == -INFINITY ? 0.f : ex2(ws_lse[(size_t)s * rows + row] - m);
-  const float inv = total > 0.f ? 1.f / total : 0.f;
-  for (int c = lane * 2; c < R; c += 64) {
-    float x = 0.f, y = 0.f;
-    for (int s = 0; s < splits; ++s) {
-      const float w = m == -INFINITY ? 0.f : ex2(ws_lse[(size_t)s * rows + row] - m) * inv;
-      const float2 v = *reinterpret_cast<const float2*>(ws_o + ((size_t)s * rows + row) * R + c);
-      x = fmaf(w, v.x, x);
-      y = fmaf(w, v.y, y);
+  const float lse = lane < splits ? ws_lse[(size_t)lane * rows + row] : -INFINITY;    // splits <= 16
+  float acc[4][4] = {};
+  float4 v[4];
+  auto fetch = [&](int s) {
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int c = lane * 4 + i * 128;
+      v[i] = c < R ? *reinterpret_cast<const float4*>(ws_o + ((size_t)s * rows + row) * R + c)
+                   : make_float4(0.f, 0.f, 0.f, 0.f);
     }
-    *reinterpret_cast<uint32_t*>(out + (size_t)row * R + c) = pack_bf(x, y);
+  };
+  const float m = warp_max(lse);
+  float w = m == -INFINITY ? 0.f : ex2(lse - m);
+  const float total = warp_sum(w);
+  w = total > 0.f ? w / total : 0.f;
+#pragma unroll 4
+  for (int s = 0; s < splits; ++s) {
+    fetch(s);
+    const float f = __shfl_sync(0xffffffffu, w, s);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      acc[i][0] = fmaf(f, v[i].x, acc[i][0]);
+      acc[i][1] = fmaf(f, v[i].y, acc[i][1]);
+      acc[i][2] = fmaf(f, v[i].z, acc[i][2]);
+      acc[i][3] = fmaf(f, v[i].w, acc[i][3]);
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const int c = lane * 4 + i * 128;
+    if (c < R)
+      *reinterpret_cast<uint2*>(out + (size_t)row * R + c) =
+          make_uint2(pack_bf(acc[i][0], acc[i][1]), pack_bf(acc[i][2], acc[i][3]));
   }
 }
 
-template <int NP, int WM>
+template <int NP, int WM, int WN>
 int launch_latent(const LatArgs& a, int B, int max_q, cudaStream_t s) {
-  constexpr int R = NP * 64, MT = 16 * WM, WN = 8 / WM;
+  constexpr int R = NP * 64, MT = 16 * WM;
   constexpr int bytes = MT * R * 2 + LatentStages<NP>::value * 64 * R * 2 + MT * 128 + WN * MT * 4 + 128;
   static bool set = false;
   if (!set) {
-    const cudaError_t e = cudaFuncSetAttribute(latent_attention_kernel<NP, WM>,
+    const cudaError_t e = cudaFuncSetAttribute(latent_attention_kernel<NP, WM, WN>,
                                                cudaFuncAttributeMaxDynamicSharedMemorySize, bytes);
     if (e != cudaSuccess) {
       msgl_set_error("latent_attention smem", e);
@@ -538,7 +589,7 @@ int launch_latent(const LatArgs& a, int B, int max_q, cudaStream_t s) {
     set = true;
   }
   dim3 grid((max_q * a.H + MT - 1) / MT, B, a.splits);
-  msgl_launch(latent_attention_kernel<NP, WM>, grid, dim3(256), bytes, s, a);
+  msgl_launch(latent_attention_kernel<NP, WM, WN>, grid, dim3(32 * WM * WN), bytes, s, a);
   MSGL_CHECK_LAUNCH("latent_attention");
   return MSGL_OK;
 }
@@ -546,9 +597,11 @@ int launch_latent(const LatArgs& a, int B, int max_q, cudaStream_t s) {
 template <int NP>
 int launch_latent_rows(const LatArgs& a, int B, int max_q, cudaStream_t s) {
   const long long rows = (long long)max_q * a.H;
-  if (rows <= 16) return launch_latent<NP, 1>(a, B, max_q, s);
-  if (rows <= 32) return launch_latent<NP, 2>(a, B, max_q, s);
-  return launch_latent<NP, 4>(a, B, max_q, s);
+  // a wide latent leaves room for one CTA per SM: sixteen warps of it
+  constexpr int W = NP > 4 ? 16 : 8;
+  if (rows <= 16) return launch_latent<NP, 1, 8>(a, B, max_q, s);
+  if (rows <= 32) return launch_latent<NP, 2, W / 2>(a, B, max_q, s);
+  return launch_latent<NP, 4, W / 4>(a, B, max_q, s);
 }
 
 template <typename T>
@@ -597,8 +650,9 @@ MSGL_API int msgl_head_gemm(const void* x, long long ldx, long long hx, const vo
                  static_weights, (const float*)ws_o, (const float*)ws_lse, splits, H,
                  StoreArgs<__nv_bfloat16>{(const __nv_bfloat16*)c, ldc, (const float*)norm, (__nv_bfloat16*)pool,
                                           (const int32_t*)out_loc, T, rank, width, eps, num_slots}};
-  if (c != nullptr && (rank <= 0 || rank > width || H >= 65535)) return MSGL_BAD_ARG;
-  dim3 grid((N + 63) / 64, H + (c != nullptr), (T + 63) / 64);
+  if (c != nullptr && (rank <= 0 || rank > width || H > 65000)) return MSGL_BAD_ARG;
+  const int nx = (N + 63) / 64;
+  dim3 grid(nx, H + (c != nullptr ? (16 + nx - 1) / nx : 0), (T + 63) / 64);
   if (splits > 1) {
     if (splits > kMaxSplits || ws_o == nullptr || ws_lse == nullptr || (uintptr_t)ws_o % 16) return MSGL_BAD_ARG;
     msgl_launch(head_gemm_kernel<true>, grid, dim3(128), 0, stream, a);
@@ -615,7 +669,7 @@ MSGL_API int msgl_latent_attention(const void* q, const void* pool, void* out, c
                                    float scale, int dtype, cudaStream_t stream) {
   if (B <= 0 || total_q <= 0) return B == 0 || total_q == 0 ? MSGL_OK : MSGL_BAD_ARG;
   if (max_q <= 0 || H <= 0 || R % 64 || page_size <= 0 || num_pages <= 0 || B > 65535 || splits < 1 || bt_stride < 1 ||
-      (uintptr_t)q % 16 || (uintptr_t)pool % 16 || (uintptr_t)out % 16 || (out == nullptr && splits == 1))
+      splits > kMaxSplits || (uintptr_t)q % 16 || (uintptr_t)pool % 16 || (uintptr_t)out % 16 || (out == nullptr && splits == 1))
     return MSGL_BAD_ARG;
   int shift = -1;
   for (int i = 0; i < 31; ++i)

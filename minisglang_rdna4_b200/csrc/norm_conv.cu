@@ -48,6 +48,20 @@ struct NormConvArgs {
   int rows, width, cols, taps, block_rows;
 };
 
+// V consecutive floats, zeros unless ``ok``
+template <int V> __device__ __forceinline__ void load_vec(const float* p, size_t off, bool ok, float (&q)[V]) {
+#pragma unroll
+  for (int v = 0; v < V; ++v) q[v] = 0.f;
+  if (!ok) return;
+  if constexpr (V == 4) {
+    const float4 x = *reinterpret_cast<const float4*>(p + off);
+    q[0] = x.x; q[1] = x.y; q[2] = x.z; q[3] = x.w;
+  } else {
+#pragma unroll
+    for (int v = 0; v < V; ++v) q[v] = p[off + v];
+  }
+}
+
 // V consecutive channels per thread, NC such groups; MT >= taps: the filter is right-aligned in MT taps.
 template <typename T, int V, int NC, int MT>
 __global__ void __launch_bounds__(1024) norm_conv_kernel(const NormConvArgs a) {
@@ -71,33 +85,31 @@ __global__ void __launch_bounds__(1024) norm_conv_kernel(const NormConvArgs a) {
   for (int g = 0; g < NC; ++g) {
     ch[g] = (g * blockDim.x + tid) * V;
 #pragma unroll
-    for (int v = 0; v < V; ++v) {
+    for (int j = 0; j < MT; ++j) {
+      const int src = j - (MT - a.taps);
+      float q1[V], q2[V];
+      load_vec<V>(a.w1, (size_t)src * a.width + ch[g], conv && src >= 0 && ch[g] < a.width, q1);
+      load_vec<V>(a.w2, (size_t)src * a.width + ch[g], a.w2 != nullptr && src >= 0 && ch[g] < a.width, q2);
 #pragma unroll
-      for (int j = 0; j < MT - 1; ++j) hist[g][v][j] = 0.f;
-#pragma unroll
-      for (int j = 0; j < MT; ++j) {
-        const int src = j - (MT - a.taps);
-        const bool ok = conv && src >= 0 && ch[g] + v < a.width;
-        f1[g][v][j] = ok ? a.w1[(size_t)src * a.width + ch[g] + v] : 0.f;
-        f2[g][v][j] = ok && a.w2 != nullptr ? a.w2[(size_t)src * a.width + ch[g] + v] : 0.f;
-      }
+      for (int v = 0; v < V; ++v) { f1[g][v][j] = q1[v]; f2[g][v][j] = q2[v]; }
     }
   }
   float* st = nullptr;
+  bool keep = false;
   if (conv && hist_n > 0 && r0 == 0) {
     st = a.state + (size_t)a.slots[b] * a.width * hist_n;
-    if (a.has_state[b] != 0) {
-#pragma unroll
-      for (int g = 0; g < NC; ++g)
-#pragma unroll
-        for (int v = 0; v < V; ++v)
-#pragma unroll
-          for (int j = 0; j < MT - 1; ++j) {
-            const int src = j - (MT - 1 - hist_n);
-            if (src >= 0 && ch[g] + v < a.width) hist[g][v][j] = st[(size_t)src * a.width + ch[g] + v];
-          }
-    }
+    keep = a.has_state[b] != 0;
   }
+#pragma unroll
+  for (int g = 0; g < NC; ++g)
+#pragma unroll
+    for (int j = 0; j < MT - 1; ++j) {
+      const int src = j - (MT - 1 - hist_n);
+      float q[V];
+      load_vec<V>(st, (size_t)src * a.width + ch[g], keep && src >= 0 && ch[g] < a.width, q);
+#pragma unroll
+      for (int v = 0; v < V; ++v) hist[g][v][j] = q[v];
+    }
 
   auto load_row = [&](int r, float (&x)[NC][V]) {
     const size_t row = (size_t)(lo + r);
@@ -232,12 +244,16 @@ __global__ void __launch_bounds__(1024) norm_conv_kernel(const NormConvArgs a) {
 #pragma unroll
   for (int g = 0; g < NC; ++g)
 #pragma unroll
-    for (int v = 0; v < V; ++v)
+    for (int j = 0; j < MT - 1; ++j) {
+      const int dst = j - (MT - 1 - hist_n);
+      if (dst < 0 || ch[g] >= a.width) continue;
+      float* p = st + (size_t)dst * a.width + ch[g];
+      if constexpr (V == 4)
+        *reinterpret_cast<float4*>(p) = make_float4(hist[g][0][j], hist[g][1][j], hist[g][2][j], hist[g][3][j]);
+      else
 #pragma unroll
-      for (int j = 0; j < MT - 1; ++j) {
-        const int dst = j - (MT - 1 - hist_n);
-        if (dst >= 0 && ch[g] + v < a.width) st[(size_t)dst * a.width + ch[g] + v] = hist[g][v][j];
-      }
+        for (int v = 0; v < V; ++v) p[v] = hist[g][v][j];
+    }
 }
 
 // Prefill form, two streaming passes. First a warp per row: residual add and gain / rms (one float per row). Then a
