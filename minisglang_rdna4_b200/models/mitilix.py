@@ -94,12 +94,12 @@ class MitilixForCausalLM(BaseOP):
         return self.model.norm.forward(x, delta)[1]
 
     # ---- checkpoint names ----
-    def checkpoint_map(self) -> Dict[str, List[Tuple]]:
-        """Checkpoint tensor -> ``[(owner, attribute, fill)]``; ``fill(param, tensor)`` writes this rank's share of the
-        tensor into its place in the (zero-initialised) parameter."""
+    def checkpoint_map(self) -> Dict[str, Tuple]:
+        """Checkpoint tensor -> ``(shape, owner, attribute, fill)``; ``fill(param, tensor)`` writes this rank's share of
+        the tensor into its place in the (zero-initialised) parameter."""
         cfg, tp = self._cfg, get_tp_info()
         w = cfg.hidden_size
-        out: Dict[str, List[Tuple]] = {}
+        out: Dict[str, Tuple] = {}
 
         def whole(p, t):
             p.view(-1)[:t.numel()].copy_(t.reshape(-1))
@@ -121,10 +121,11 @@ class MitilixForCausalLM(BaseOP):
             return t.narrow(dim, tp.rank * n, n)
 
         body = self.model
-        out["embed"] = [(body.embed_tokens, "weight", vocab(body.embed_tokens._start))]
-        out["pos"] = [(body, "positions", corner)]
-        out["final.norm"] = [(body.norm, "gain", whole)]
-        out["head"] = [(self.lm_head, "weight", vocab(self.lm_head._start))]
+        v, taps = cfg.vocab_size, cfg.input_conv_taps
+        out["embed"] = ((v, w), body.embed_tokens, "weight", vocab(body.embed_tokens._start))
+        out["pos"] = ((cfg.max_position_embeddings, w), body, "positions", corner)
+        out["final.norm"] = ((), body.norm, "gain", whole)
+        out["head"] = ((v, w), self.lm_head, "weight", vocab(self.lm_head._start))
         for i, layer in enumerate(body.layers):
             s: LatentLayer = cfg.latent_layers[i]
             a, h = layer.attn, layer.attn._h
@@ -154,19 +155,19 @@ class MitilixForCausalLM(BaseOP):
                 p[:w, n:n + part.shape[1]].copy_(part)
 
             name = f"l{i}."
-            out[name + "norm1"] = [(layer.norm, "gain", whole)]
-            out[name + "canon1"] = [(layer.norm, "conv1", taps_first)]
-            out[name + "mix.q"] = [(a.q_proj, "weight", q)]
-            out[name + "mix.uk"] = [(a, "up_k", uk)]
-            out[name + "mix.uv"] = [(a, "up_v", uv)]
-            out[name + "mix.o"] = [(layer.out_proj, "weight", o)]
+            out[name + "norm1"] = ((), layer.norm, "gain", whole)
+            out[name + "canon1"] = ((w, taps), layer.norm, "conv1", taps_first)
+            out[name + "mix.q"] = ((s.heads * s.dim, w), a.q_proj, "weight", q)
+            out[name + "mix.uk"] = ((s.heads * s.dim, s.kv_rank), a, "up_k", uk)
+            out[name + "mix.uv"] = ((s.heads * s.vdim, s.kv_rank), a, "up_v", uv)
+            out[name + "mix.o"] = ((w, s.heads * s.vdim), layer.out_proj, "weight", o)
             if s.kv_from is None:
-                out[name + "mix.dkv"] = [(a.q_proj, "weight", dkv)]
-                out[name + "mix.dkv.norm"] = [(a, "latent_norm", whole)]
+                out[name + "mix.dkv"] = ((s.kv_rank, w), a.q_proj, "weight", dkv)
+                out[name + "mix.dkv.norm"] = ((s.kv_rank,), a, "latent_norm", whole)
             if s.ff:
-                out[name + "canon2"] = [(layer.norm, "conv2", taps_first)]
-                out[name + "mlp.up"] = [(layer.up_proj, "weight", up)]
-                out[name + "mlp.down"] = [(layer.out_proj, "weight", down)]
+                out[name + "canon2"] = ((w, taps), layer.norm, "conv2", taps_first)
+                out[name + "mlp.up"] = ((s.ff, w), layer.up_proj, "weight", up)
+                out[name + "mlp.down"] = ((w, s.ff), layer.out_proj, "weight", down)
         return out
 
     def init_dummy(self, seed: int, std: float = 0.02, gen_device: str = "cpu") -> None:

@@ -463,16 +463,15 @@ def _load_mapped(model, stream: Iterator, device) -> None:
         setattr(owner, attr, torch.zeros(t.shape, dtype=t.dtype, device=device))
     seen = set()
     for name, tensor in stream:
-        places = wanted.get(name)
-        if places is None:
+        place = wanted.get(name)
+        if place is None:
             logger.debug_rank0("skipping unexpected tensor %s", name)
             continue
-        for owner, attr, fill in places:
-            param = getattr(owner, attr)
-            try:
-                fill(param, tensor.to(device=device, dtype=param.dtype))
-            except RuntimeError as exc:
-                raise ValueError(f"{name}: checkpoint shape {tuple(tensor.shape)} does not fit: {exc}") from None
+        shape, owner, attr, fill = place
+        if tuple(tensor.shape) != shape and not (shape == () and tensor.numel() == 1):
+            raise ValueError(f"{name}: checkpoint shape {tuple(tensor.shape)} != model {shape}")
+        param = getattr(owner, attr)
+        fill(param, tensor.to(device=device, dtype=param.dtype))
         seen.add(name)
     missing = sorted(set(wanted) - seen)
     if missing:
