@@ -223,3 +223,73 @@ def test_latent_attention_window_edge(r):
             got = ops.latent_attention(q.bfloat16().to(DEV), flat2.view_as(pool).bfloat16().to(DEV), *args, 1.0, window, 1,
                                        kv, splits).float().cpu()
             assert (float(got[0, 0, 0]) > 7.0) == seen
+
+
+# ---------------------------------------------------------------------------------- the engine on the GPU
+import mitilix_util as U  # noqa: E402
+import plain_mitilix as plain  # noqa: E402
+from minisglang_rdna4_b200 import LLM, SamplingParams  # noqa: E402
+from minisglang_rdna4_b200.replay import make_replayer  # noqa: E402
+
+# latents of one and two panels, heads that fill neither 16, 32 nor 64 rows, a window past a tile and one below it
+BIG = U.config([U.layer(5, 32, 48, 128, 100, 96), U.layer(9, 64, 128, 64, 40, 130),
+                U.layer(20, 16, 32, 128, 150, 64, kv_from=0)], width=96, vocab=131, taps=4, max_positions=400)
+CASES = {"mixed": (U.MIXED, U.SEQS), "plain": (U.PLAIN, U.SEQS),
+         "big": (BIG, {"a": 330, "b": 140, "c": 201, "d": 70})}
+
+
+@pytest.fixture(scope="module", params=list(CASES))
+def model(request, tmp_path_factory):
+    cfg, lengths = CASES[request.param]
+    w = U.weights(cfg, 1, sharp=1.5)
+    path = U.save(tmp_path_factory.mktemp(request.param), cfg, w)
+    seqs = {n: U.tokens(cfg, k, i) for i, (n, k) in enumerate(lengths.items())}
+    return cfg, w, path, seqs, U.reference(cfg, w, seqs)
+
+
+@pytest.mark.parametrize("dtype,limit", [("float32", 2e-4), ("bfloat16", 0.06)])
+def test_engine_portions_batches_and_reuse(model, dtype, limit):
+    cfg, w, path, seqs, want = model
+    rep = make_replayer(path, dtype, 896, "cuda")
+    for sizes in ([1000], [100, 1, 2, 63], [2, 65]):
+        for name in seqs:
+            U.play(rep, seqs, [[(name, n)] for n in U.cuts(len(seqs[name]), sizes)], want, limit)
+    # decoding alone (captured graphs) after most of the prompt
+    U.play(rep, seqs, [[("c", len(seqs["c"]) - 24)]] + [[("c", 1)]] * 24, want, limit)
+    # everyone together, then mixed portions and single tokens with slots and pages taken again
+    U.play(rep, seqs, [[(n, len(s)) for n, s in seqs.items()]], want, limit)
+    at = {n: 0 for n in seqs}
+    plan, k = [], 0
+    while any(at[n] < len(seqs[n]) for n in seqs):
+        step = []
+        for j, n in enumerate(seqs):
+            left = len(seqs[n]) - at[n]
+            if left and (k + j) % 5:
+                size = min(left, (1, 37, 2, 64, 1)[(k + 2 * j) % 5])
+                step.append((n, size))
+                at[n] += size
+        k += 1
+        if step:
+            plan.append(step)
+    U.play(rep, seqs, plan, want, limit)
+    assert rep.engine.graph_runner is None or rep.engine.graph_runner.replays > 0
+    rep.engine.shutdown()
+
+
+def test_engine_generates_the_greedy_tokens(model):
+    cfg, w, path, seqs, _ = model
+    llm = LLM(path, device="cuda", dtype="fp32", page_size=16, max_running_req=4, num_page_override=128,
+              max_extend_tokens=48)
+    prompts = [seqs["a"][:59], seqs["b"], seqs["c"][:1], seqs["d"][:64]]
+    outs = llm.generate(prompts, SamplingParams(max_tokens=6, ignore_eos=True))
+    for p, o in zip(prompts, outs):
+        seq = list(p)
+        for _ in range(6):
+            seq.append(int(plain.logits(cfg, w, seq)[-1].argmax()))
+        assert o.token_ids == seq[len(p):]
+    # a prefix the cache holds, with the state kept at its boundary
+    again = seqs["d"][:64] + seqs["b"][:5]
+    o = llm.generate([again], SamplingParams(max_tokens=3, ignore_eos=True))[0]
+    assert o.cached_tokens > 0
+    assert o.token_ids[0] == int(plain.logits(cfg, w, again)[-1].argmax())
+    llm.shutdown()
