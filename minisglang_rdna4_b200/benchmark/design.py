@@ -70,9 +70,10 @@ def throughput(cfg: ModelConfig, batches=(1, 16, 64, 256), prompt: int = 2048, o
     res: Dict = {"decode": {}, "prefill": {}}
     launches = K.LAUNCHES
     for b in (max(batches), *batches):              # the first pass warms up
-        steps.clear()
-        prompts = [torch.randint(0, cfg.vocab_size, (prompt,), generator=g).tolist() for _ in range(b)]
-        llm.generate(prompts, SamplingParams(max_tokens=out, ignore_eos=True))
+        for _ in range(2):                          # ... and so does the first of two at every batch size
+            steps.clear()
+            prompts = [torch.randint(0, cfg.vocab_size, (prompt,), generator=g).tolist() for _ in range(b)]
+            llm.generate(prompts, SamplingParams(max_tokens=out, ignore_eos=True))
         torch.cuda.synchronize()
         dec = [s.elapsed_time(e) for s, e, ph, n in steps if ph == "decode" and n == b][4:]
         pre = [(s.elapsed_time(e), n) for s, e, ph, n in steps if ph == "prefill"]

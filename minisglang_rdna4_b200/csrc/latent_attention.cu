@@ -40,23 +40,46 @@ template <typename T> struct StoreArgs {
   long long num_slots;
 };
 
-// one warp per row
+// One warp per row, eight channels per lane and step (width a multiple of 64, up to 1024).
 template <typename T> __device__ __forceinline__ void store_latent(const StoreArgs<T>& a, int t, int lane) {
   const T* src = a.c + (size_t)t * a.ldc;
+  const long long slot = a.out_loc[t];
+  float v[4][8];
   float s = 0.f;
-#pragma unroll 4
-  for (int i = lane; i < a.rank; i += 32) {
-    const float v = to_float(src[i]);
-    s = fmaf(v, v, s);
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const int c = (lane + 32 * i) * 8;
+    if (c < a.width) {
+      if constexpr (sizeof(T) == 2) {
+        load8(src + c, v[i]);
+      } else {
+#pragma unroll
+        for (int e = 0; e < 8; ++e) v[i][e] = src[c + e];
+      }
+    }
+#pragma unroll
+    for (int e = 0; e < 8; ++e) {
+      if (c + e >= a.rank) v[i][e] = 0.f;
+      s = fmaf(v[i][e], v[i][e], s);
+    }
   }
   s = warp_sum(s);
   const float sc = 1.f / sqrtf(s / (float)a.rank + a.eps);
-  const long long slot = a.out_loc[t];
   if (MSGL_OOB(slot, a.num_slots) || slot < 0 || slot >= a.num_slots) return;
   T* dst = a.pool + slot * a.width;
-#pragma unroll 4
-  for (int i = lane; i < a.width; i += 32)
-    dst[i] = from_float<T>(i < a.rank ? to_float(src[i]) * sc * a.weight[i] : 0.f);
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const int c = (lane + 32 * i) * 8;
+    if (c >= a.width) break;
+#pragma unroll
+    for (int e = 0; e < 8; ++e) v[i][e] *= c + e < a.rank ? sc * a.weight[c + e] : 0.f;
+    if constexpr (sizeof(T) == 2) {
+      store8(dst + c, v[i]);
+    } else {
+#pragma unroll
+      for (int e = 0; e < 8; ++e) dst[c + e] = v[i][e];
+    }
+  }
 }
 
 template <typename T> __global__ void __launch_bounds__(128) latent_norm_store_kernel(const StoreArgs<T> a) {
@@ -295,20 +318,24 @@ __global__ void __launch_bounds__(128) head_gemm_kernel(const HeadGemmArgs a) {
 // ------------------------------------------------------------------------------------------ attention
 template <int NP> struct LatentStages { static constexpr int value = NP <= 4 ? 3 : 2; };
 
-// NP: latent panels of 64 channels (R = 64 NP). WM row groups of 16 x WN column groups: a warp computes
-// 16 rows x (64 / WN) keys of S and 16 rows x (R / WN) channels of O.
-template <int NP, int WM, int WN>
+// NP: latent panels of 64 channels (R = 64 NP). WM row groups of 16 x WN column groups: a warp owns 16 rows x
+// (64 / WN) keys of S and 16 rows x (R / WN) channels of O. KS = 2: the two warps of a pair of column groups
+// compute their keys' scores together, half of the channels each (so that the queries are read from shared memory
+// half as often, or fit in registers), and exchange the halves.
+template <int NP, int WM, int WN, int KS>
 __global__ void __launch_bounds__(32 * WM * WN) latent_attention_kernel(const LatArgs a) {
   pdl_enter();
   constexpr int R = NP * 64, MT = 16 * WM, TK = 64, NT = 32 * WM * WN;
   constexpr int CH = R / 8;                      // 16-byte chunks per row
   constexpr int NS = TK / WN / 8;                // key blocks of 8 per warp
+  constexpr int NX = NS * KS;                    // ... whose scores it computes over R / KS channels
   constexpr int NO = R / WN / 8;                 // channel blocks of 8 per warp
   constexpr int Q_BYTES = MT * R * 2, C_BYTES = TK * R * 2, ST = LatentStages<NP>::value;
   extern __shared__ __align__(128) uint8_t smem[];
   uint8_t* base = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem) + 127) & ~uintptr_t(127));
   const uint32_t q_s = smem_u32(base), c_s = q_s + Q_BYTES, p_s = c_s + ST * C_BYTES;
   float* red = reinterpret_cast<float*>(base + Q_BYTES + ST * C_BYTES + MT * 128);   // [WN][MT]
+  float4* swap = reinterpret_cast<float4*>(red + WN * MT);                            // [warps][NS][32], KS = 2
 
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int wm = warp / WN, wn = warp % WN;
@@ -370,8 +397,10 @@ __global__ void __launch_bounds__(32 * WM * WN) latent_attention_kernel(const La
   const int pa = kv_len - q_len + min(row0 + ra, row1 - 1) / a.H, pb = kv_len - q_len + min(row0 + rb, row1 - 1) / a.H;
   const int lo_a = a.window > 0 ? pa - a.window + 1 : 0, lo_b = a.window > 0 ? pb - a.window + 1 : 0;
   const float sc = a.scale * kLog2eL;
-  constexpr bool QREG = WM == 1 && R <= 256;     // few rows: the queries fit in registers
-  uint32_t qf[QREG ? R / 16 : 1][4];
+  constexpr int KK = R / 32 / KS;                // steps of 32 channels
+  constexpr bool QREG = WM <= KS && KK <= 8;     // few rows: the queries fit in registers
+  const int kk0 = KS == 2 ? (wn & 1) * KK : 0, key0 = (KS == 2 ? wn & ~1 : wn) * NS * 8;
+  uint32_t qf[QREG ? 2 * KK : 1][4];
   float o[NO][4];
 #pragma unroll
   for (int i = 0; i < NO; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
@@ -383,20 +412,21 @@ __global__ void __launch_bounds__(32 * WM * WN) latent_attention_kernel(const La
     if (t + ST - 1 < n_tiles) load_tile(t + ST - 1);
     cp_commit();
     const uint32_t cb = c_s + (t % ST) * C_BYTES;
-    float s[NS][4], s2[NS][4];                    // two accumulators: half as long a chain of dependent products
+    float x[NX][4], x2[NX][4];                    // two accumulators: half as long a chain of dependent products
 #pragma unroll
-    for (int i = 0; i < NS; ++i) {
-      s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.f;
-      s2[i][0] = s2[i][1] = s2[i][2] = s2[i][3] = 0.f;
+    for (int i = 0; i < NX; ++i) {
+      x[i][0] = x[i][1] = x[i][2] = x[i][3] = 0.f;
+      x2[i][0] = x2[i][1] = x2[i][2] = x2[i][3] = 0.f;
     }
     if constexpr (QREG) {
       if (t == 0) {
 #pragma unroll
-        for (int kk = 0; kk < R / 16; ++kk) ldm_x4(q_s + swz(wm * 16 + (lane & 15), kk * 2 + (lane >> 4), CH), qf[kk]);
+        for (int kk = 0; kk < 2 * KK; ++kk)
+          ldm_x4(q_s + swz(wm * 16 + (lane & 15), (kk0 * 2 + kk) * 2 + (lane >> 4), CH), qf[kk]);
       }
     }
-#pragma unroll (QREG ? R / 32 : 4)
-    for (int kk = 0; kk < R / 32; ++kk) {
+#pragma unroll (QREG ? KK : 4)
+    for (int kk = 0; kk < KK; ++kk) {
       uint32_t a0[4], a1[4];
       if constexpr (QREG) {
 #pragma unroll
@@ -405,16 +435,41 @@ __global__ void __launch_bounds__(32 * WM * WN) latent_attention_kernel(const La
           a1[i] = qf[2 * kk + 1][i];
         }
       } else {
-        ldm_x4(q_s + swz(wm * 16 + (lane & 15), kk * 4 + (lane >> 4), CH), a0);
-        ldm_x4(q_s + swz(wm * 16 + (lane & 15), kk * 4 + 2 + (lane >> 4), CH), a1);
+        ldm_x4(q_s + swz(wm * 16 + (lane & 15), (kk0 + kk) * 4 + (lane >> 4), CH), a0);
+        ldm_x4(q_s + swz(wm * 16 + (lane & 15), (kk0 + kk) * 4 + 2 + (lane >> 4), CH), a1);
       }
 #pragma unroll
-      for (int nb = 0; nb < NS; ++nb) {
+      for (int nb = 0; nb < NX; ++nb) {
         uint32_t bf[4];
-        ldm_x4(cb + swz(wn * (TK / WN) + nb * 8 + (lane & 7), kk * 4 + (lane >> 3), CH), bf);
-        mma_bf16(s[nb], a0, bf[0], bf[1]);
-        mma_bf16(s2[nb], a1, bf[2], bf[3]);
+        ldm_x4(cb + swz(key0 + nb * 8 + (lane & 7), (kk0 + kk) * 4 + (lane >> 3), CH), bf);
+        mma_bf16(x[nb], a0, bf[0], bf[1]);
+        mma_bf16(KS == 1 ? x2[nb] : x[nb], a1, bf[2], bf[3]);
       }
+    }
+    float s[NS][4];
+    if constexpr (KS == 2) {
+      // the partner's key blocks out, this warp's other half of the channels in
+      const bool hi = wn & 1;
+#pragma unroll
+      for (int nb = 0; nb < NS; ++nb) {
+        float out_[4];                            // (selected by value: the accumulators stay in registers)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) out_[e] = hi ? x[nb][e] : x[NS + nb][e];
+        swap[((warp ^ 1) * NS + nb) * 32 + lane] = make_float4(out_[0], out_[1], out_[2], out_[3]);
+      }
+      asm volatile("bar.sync %0, 64;" ::"r"(1 + (warp >> 1)) : "memory");
+#pragma unroll
+      for (int nb = 0; nb < NS; ++nb) {
+        const float4 v = swap[(warp * NS + nb) * 32 + lane];
+        const float in[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+        for (int e = 0; e < 4; ++e) s[nb][e] = (hi ? x[NS + nb][e] : x[nb][e]) + in[e];
+      }
+    } else {
+#pragma unroll
+      for (int nb = 0; nb < NS; ++nb)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) s[nb][e] = x[nb][e] + x2[nb][e];
     }
     const int tok0 = (t_begin + t) * TK + wn * (TK / WN) + (lane & 3) * 2;
     float mx_a = -INFINITY, mx_b = -INFINITY;
@@ -423,8 +478,8 @@ __global__ void __launch_bounds__(32 * WM * WN) latent_attention_kernel(const La
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
         const int tok = tok0 + nb * 8 + e;
-        const float va = tok <= pa && tok >= lo_a ? (s[nb][e] + s2[nb][e]) * sc : -INFINITY;
-        const float vb = tok <= pb && tok >= lo_b ? (s[nb][2 + e] + s2[nb][2 + e]) * sc : -INFINITY;
+        const float va = tok <= pa && tok >= lo_a ? s[nb][e] * sc : -INFINITY;
+        const float vb = tok <= pb && tok >= lo_b ? s[nb][2 + e] * sc : -INFINITY;
         s[nb][e] = va;
         s[nb][2 + e] = vb;
         mx_a = fmaxf(mx_a, va);
@@ -574,13 +629,14 @@ __global__ void __launch_bounds__(128) latent_combine_kernel(const float* __rest
   }
 }
 
-template <int NP, int WM, int WN>
+template <int NP, int WM, int WN, int KS>
 int launch_latent(const LatArgs& a, int B, int max_q, cudaStream_t s) {
   constexpr int R = NP * 64, MT = 16 * WM;
-  constexpr int bytes = MT * R * 2 + LatentStages<NP>::value * 64 * R * 2 + MT * 128 + WN * MT * 4 + 128;
+  constexpr int bytes = MT * R * 2 + LatentStages<NP>::value * 64 * R * 2 + MT * 128 + WN * MT * 4 + 128 +
+                        (KS == 2 ? WM * WN * (8 / WN) * 512 : 0);
   static bool set = false;
   if (!set) {
-    const cudaError_t e = cudaFuncSetAttribute(latent_attention_kernel<NP, WM, WN>,
+    const cudaError_t e = cudaFuncSetAttribute(latent_attention_kernel<NP, WM, WN, KS>,
                                                cudaFuncAttributeMaxDynamicSharedMemorySize, bytes);
     if (e != cudaSuccess) {
       msgl_set_error("latent_attention smem", e);
@@ -589,7 +645,7 @@ int launch_latent(const LatArgs& a, int B, int max_q, cudaStream_t s) {
     set = true;
   }
   dim3 grid((max_q * a.H + MT - 1) / MT, B, a.splits);
-  msgl_launch(latent_attention_kernel<NP, WM, WN>, grid, dim3(32 * WM * WN), bytes, s, a);
+  msgl_launch(latent_attention_kernel<NP, WM, WN, KS>, grid, dim3(32 * WM * WN), bytes, s, a);
   MSGL_CHECK_LAUNCH("latent_attention");
   return MSGL_OK;
 }
@@ -597,11 +653,15 @@ int launch_latent(const LatArgs& a, int B, int max_q, cudaStream_t s) {
 template <int NP>
 int launch_latent_rows(const LatArgs& a, int B, int max_q, cudaStream_t s) {
   const long long rows = (long long)max_q * a.H;
-  // a wide latent leaves room for one CTA per SM: sixteen warps of it
-  constexpr int W = NP > 4 ? 16 : 8;
-  if (rows <= 16) return launch_latent<NP, 1, 8>(a, B, max_q, s);
-  if (rows <= 32) return launch_latent<NP, 2, W / 2>(a, B, max_q, s);
-  return launch_latent<NP, 4, W / 4>(a, B, max_q, s);
+  if constexpr (NP > 4) {                  // a wide latent leaves room for one CTA per SM: sixteen warps of it
+    if (rows <= 16) return launch_latent<NP, 1, 8, 2>(a, B, max_q, s);
+    if (rows <= 32) return launch_latent<NP, 2, 8, 2>(a, B, max_q, s);
+    return launch_latent<NP, 4, 4, 1>(a, B, max_q, s);
+  } else {
+    if (rows <= 16) return launch_latent<NP, 1, 8, 1>(a, B, max_q, s);
+    if (rows <= 32) return launch_latent<NP, 2, 4, 1>(a, B, max_q, s);
+    return launch_latent<NP, 4, 2, 1>(a, B, max_q, s);
+  }
 }
 
 template <typename T>
@@ -623,7 +683,8 @@ MSGL_API int msgl_latent_norm_store(const void* c, long long ldc, const void* we
                                     int rows, int rank, int width, float eps, long long num_slots, int dtype,
                                     cudaStream_t stream) {
   if (rows <= 0) return rows == 0 ? MSGL_OK : MSGL_BAD_ARG;
-  if (rank <= 0 || rank > width) return MSGL_BAD_ARG;
+  if (rank <= 0 || rank > width || width % 64 || width > 1024 || ldc % 8 || (uintptr_t)c % 16 || (uintptr_t)pool % 16)
+    return MSGL_BAD_ARG;
   dim3 grid((rows + 3) / 4);
 #define STORE(T)                                                                                                    \
   msgl_launch(latent_norm_store_kernel<T>, grid, dim3(128), 0, stream,                                              \
@@ -650,7 +711,9 @@ MSGL_API int msgl_head_gemm(const void* x, long long ldx, long long hx, const vo
                  static_weights, (const float*)ws_o, (const float*)ws_lse, splits, H,
                  StoreArgs<__nv_bfloat16>{(const __nv_bfloat16*)c, ldc, (const float*)norm, (__nv_bfloat16*)pool,
                                           (const int32_t*)out_loc, T, rank, width, eps, num_slots}};
-  if (c != nullptr && (rank <= 0 || rank > width || H > 65000)) return MSGL_BAD_ARG;
+  if (c != nullptr && (rank <= 0 || rank > width || width % 64 || width > 1024 || ldc % 8 || (uintptr_t)c % 16 ||
+                       (uintptr_t)pool % 16 || H > 65000))
+    return MSGL_BAD_ARG;
   const int nx = (N + 63) / 64;
   dim3 grid(nx, H + (c != nullptr ? (16 + nx - 1) / nx : 0), (T + 63) / 64);
   if (splits > 1) {
