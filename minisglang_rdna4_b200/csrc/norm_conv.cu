@@ -406,6 +406,7 @@ int norm_conv_typed(NormConvArgs a, float* scale, int B, int max_q, cudaStream_t
   if (vec) {
     if (nc == 1) launch_norm_conv<T, 4, 1>(a, grid, threads, s);
     else if (nc == 2) launch_norm_conv<T, 4, 2>(a, grid, threads, s);
+    else if (nc <= 4) launch_norm_conv<T, 4, 4>(a, grid, threads, s);
     else return MSGL_BAD_ARG;
   } else {
     if (nc == 1) launch_norm_conv<T, 1, 1>(a, grid, threads, s);

@@ -14,7 +14,7 @@ def build_parser() -> argparse.ArgumentParser:
     p = argparse.ArgumentParser(prog="python -m minisglang_rdna4_b200", description="B200-native LLM server")
     p.add_argument("--model-path", "--model", dest="model_path", required=True)
     p.add_argument("--served-model-name", default=None)
-    p.add_argument("--dtype", default="auto", choices=["auto", "fp16", "bf16", "fp32"])
+    p.add_argument("--dtype", default="auto", choices=["auto", "fp16", "bf16", "fp32", "float16", "bfloat16", "float32"])
     p.add_argument("--tensor-parallel-size", "--tp-size", "--tp", dest="tp_size", type=int, default=1)
     p.add_argument("--data-parallel-size", "--dp-size", "--dp", dest="dp_size", type=int, default=1)
     p.add_argument("--enable-ep", action="store_true")

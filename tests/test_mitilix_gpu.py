@@ -30,7 +30,7 @@ def _batch(lens, starts, ps, pages, gen):
 
 
 @pytest.mark.parametrize("width,taps,cols", [(256, 4, 256), (200, 3, 208), (1000, 2, 1008), (97, 5, 112), (64, 1, 64),
-                                             (4096, 4, 4096), (5120, 4, 5120), (96, 12, 96)])
+                                             (4096, 4, 4096), (5120, 4, 5120), (96, 12, 96), (8208, 3, 8208)])
 @pytest.mark.parametrize("dtype", [torch.bfloat16, torch.float32])
 def test_norm_conv(width, taps, cols, dtype):
     g = _gen(width + taps)
@@ -273,6 +273,22 @@ def test_engine_portions_batches_and_reuse(model, dtype, limit):
             plan.append(step)
     U.play(rep, seqs, plan, want, limit)
     assert rep.engine.graph_runner is None or rep.engine.graph_runner.replays > 0
+    rep.engine.shutdown()
+
+
+@pytest.mark.parametrize("dtype,limit", [("float32", 2e-4), ("bfloat16", 0.06)])
+@pytest.mark.parametrize("cfg", [
+    U.config([U.layer(heads=1, dim=1, vdim=1, rank=1, window=1, ff=1)], width=5, vocab=7, taps=1, max_positions=90),
+    U.config([U.layer(heads=7, dim=130, vdim=150, rank=300, window=50, ff=33)], width=40, vocab=64, taps=9),
+    U.config([U.layer(heads=40, rank=520, ff=0), U.layer(heads=2, window=70, ff=40)], taps=32, width=98, vocab=100),
+    U.config([U.layer(heads=33, dim=64, vdim=64, rank=200, window=65), U.layer(rank=200, kv_from=0, ff=8)], width=64, taps=2),
+], ids=["ones", "wide", "taps32", "rank200"])
+def test_engine_other_sizes(cfg, dtype, limit, tmp_path):
+    w = U.weights(cfg, 2, sharp=1.0)
+    seqs = {"a": U.tokens(cfg, 90, 1), "b": U.tokens(cfg, 3, 2)}
+    rep = make_replayer(U.save(tmp_path, cfg, w), dtype, 256, "cuda")
+    steps = [[("a", 70)], [("a", 1), ("b", 2)], [("a", 1), ("b", 1)], [("a", 2)], [("a", 1)], [("a", 1)], [("a", 14)]]
+    U.play(rep, seqs, steps, U.reference(cfg, w, seqs), limit)
     rep.engine.shutdown()
 
 
