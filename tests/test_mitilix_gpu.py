@@ -278,7 +278,8 @@ def test_engine_portions_batches_and_reuse(model, dtype, limit):
 
 @pytest.mark.parametrize("dtype,limit", [("float32", 2e-4), ("bfloat16", 0.06)])
 @pytest.mark.parametrize("cfg", [
-    U.config([U.layer(heads=1, dim=1, vdim=1, rank=1, window=1, ff=1)], width=5, vocab=7, taps=1, max_positions=90),
+    # (a latent of one channel is a sign after its norm: nothing to compare in 16 bits)
+    U.config([U.layer(heads=1, dim=1, vdim=1, rank=4, window=1, ff=1)], width=5, vocab=7, taps=1, max_positions=90),
     U.config([U.layer(heads=7, dim=130, vdim=150, rank=300, window=50, ff=33)], width=40, vocab=64, taps=9),
     U.config([U.layer(heads=40, rank=520, ff=0), U.layer(heads=2, window=70, ff=40)], taps=32, width=98, vocab=100),
     U.config([U.layer(heads=33, dim=64, vdim=64, rank=200, window=65), U.layer(rank=200, kv_from=0, ff=8)], width=64, taps=2),
