@@ -22,7 +22,7 @@ class LatentAttentionBackend(BaseAttnBackend):
         windows = [s.window for s in layers]
         self.reach = max(windows) if min(windows) > 0 else 0
         self.max_seq_len = max_seq_len
-        self.single_split = single_split
+        self.single_split = single_split       # speculative verification must reproduce decode rows bit for bit
 
     def prepare_metadata(self, batch: Batch, block_table, cu_q, seq_lens, max_q: int, max_kv: int,
                          causal: bool = True, mask: Optional[torch.Tensor] = None, host_cu_q=None,
@@ -71,7 +71,7 @@ class LatentAttentionBackend(BaseAttnBackend):
             K.head_gemm_combine(parts, up_v, out)
             return
         o_lat = ops.latent_attention(q_lat, rows, md.block_table, md.cu_q, md.seq_lens, scale, window, md.max_q,
-                                     md.max_kv, splits)
+                                     md.max_kv, splits, one_form=self.single_split)
         ops.head_gemm(o_lat, up_v, out)
 
     def _splits(self, q, md: AttnMetadata, window: int) -> int:

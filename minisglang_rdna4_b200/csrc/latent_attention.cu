@@ -651,8 +651,8 @@ int launch_latent(const LatArgs& a, int B, int max_q, cudaStream_t s) {
 }
 
 template <int NP>
-int launch_latent_rows(const LatArgs& a, int B, int max_q, cudaStream_t s) {
-  const long long rows = (long long)max_q * a.H;
+int launch_latent_rows(const LatArgs& a, int B, int max_q, bool one_form, cudaStream_t s) {
+  const long long rows = one_form ? 64 : (long long)max_q * a.H;
   if constexpr (NP > 4) {                  // a wide latent leaves room for one CTA per SM: sixteen warps of it
     if (rows <= 16) return launch_latent<NP, 1, 8, 2>(a, B, max_q, s);
     if (rows <= 32) return launch_latent<NP, 2, 8, 2>(a, B, max_q, s);
@@ -726,10 +726,12 @@ MSGL_API int msgl_head_gemm(const void* x, long long ldx, long long hx, const vo
   return MSGL_OK;
 }
 
+// one_form: the 64-row form whatever the step's size, for callers whose rows must come out bit for bit the same in
+// steps of different sizes.
 MSGL_API int msgl_latent_attention(const void* q, const void* pool, void* out, const void* block_table, int bt_stride,
                                    const void* cu_q, const void* seq_lens, void* ws_o, void* ws_lse, int B, int total_q,
                                    int max_q, int H, int R, int page_size, int num_pages, int window, int splits,
-                                   float scale, int dtype, cudaStream_t stream) {
+                                   float scale, int one_form, int dtype, cudaStream_t stream) {
   if (B <= 0 || total_q <= 0) return B == 0 || total_q == 0 ? MSGL_OK : MSGL_BAD_ARG;
   if (max_q <= 0 || H <= 0 || R % 64 || page_size <= 0 || num_pages <= 0 || B > 65535 || splits < 1 || bt_stride < 1 ||
       splits > kMaxSplits || (uintptr_t)q % 16 || (uintptr_t)pool % 16 || (uintptr_t)out % 16 || (out == nullptr && splits == 1))
@@ -749,11 +751,11 @@ MSGL_API int msgl_latent_attention(const void* q, const void* pool, void* out, c
   if (splits > 1 && (ws_o == nullptr || ws_lse == nullptr)) return MSGL_BAD_ARG;
   int rc;
   switch (R / 64) {
-    case 1: rc = launch_latent_rows<1>(a, B, max_q, stream); break;
-    case 2: rc = launch_latent_rows<2>(a, B, max_q, stream); break;
-    case 3: rc = launch_latent_rows<3>(a, B, max_q, stream); break;
-    case 4: rc = launch_latent_rows<4>(a, B, max_q, stream); break;
-    case 8: rc = launch_latent_rows<8>(a, B, max_q, stream); break;
+    case 1: rc = launch_latent_rows<1>(a, B, max_q, one_form != 0, stream); break;
+    case 2: rc = launch_latent_rows<2>(a, B, max_q, one_form != 0, stream); break;
+    case 3: rc = launch_latent_rows<3>(a, B, max_q, one_form != 0, stream); break;
+    case 4: rc = launch_latent_rows<4>(a, B, max_q, one_form != 0, stream); break;
+    case 8: rc = launch_latent_rows<8>(a, B, max_q, one_form != 0, stream); break;
     default: return MSGL_BAD_ARG;
   }
   // without a destination the ranges stay apart: the projection out of the latent space merges them

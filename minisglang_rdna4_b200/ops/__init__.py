@@ -245,9 +245,10 @@ def head_gemm(x, w, out=None, store=None):
 
 
 def latent_attention(q, rows, block_table, cu_q, seq_lens, scale: float, window: int, max_q: int, max_kv: int,
-                     splits: int = 1):
+                     splits: int = 1, one_form: bool = False):
     if q.is_cuda:
-        return _cuda().latent_attention(q, rows, block_table, cu_q, seq_lens, scale, window, max_q, max_kv, splits)
+        return _cuda().latent_attention(q, rows, block_table, cu_q, seq_lens, scale, window, max_q, max_kv, splits,
+                                        one_form=one_form)
     return ref.latent_attention(q, rows, block_table, cu_q, seq_lens, scale, window)
 
 

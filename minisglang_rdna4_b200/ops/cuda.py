@@ -917,7 +917,7 @@ def _bind_latent():
     bind("msgl_latent_gather", c_i, [c_p] * 5 + [c_i] * 5 + [c_p])
     bind("msgl_attn_prefill_pos", c_i, [c_p, c_ll, c_ll, c_p, c_p, c_i, c_p, c_ll, c_ll, c_p, c_i, c_i, c_i, c_i, c_i, c_i,
                                         c_f, c_i, c_p])
-    bind("msgl_latent_attention", c_i, [c_p, c_p, c_p, c_p, c_i] + [c_p] * 4 + [c_i] * 9 + [c_f, c_i, c_p])
+    bind("msgl_latent_attention", c_i, [c_p, c_p, c_p, c_p, c_i] + [c_p] * 4 + [c_i] * 9 + [c_f, c_i, c_i, c_p])
     _bind_latent._done = True
 
 
@@ -966,7 +966,7 @@ def add_scalar_norm_conv(x, delta, gain, eps, w1, w2, state, cu_q, slots, has_st
         assert w1.is_contiguous() and w1.dtype == torch.float32 and state.is_contiguous()
         assert state.dtype == torch.float32 and state.shape[1:] == (taps - 1, width)
     # many rows per request: two streaming passes with the row norms in between
-    scale = torch.empty(rows, dtype=torch.float32, device=x.device) if w1 is not None and max_q > 4 else None
+    scale = torch.empty(rows, dtype=torch.float32, device=x.device) if w1 is not None and max_q > 16 else None
     check(lib().msgl_norm_conv(_p(x), _p(x_out), _p(delta), planes, plane_stride, ldd, _p(gain), eps, _p(w1), _p(w2),
                                _p(y1), _p(y2), _p(state), _p(cu_q), _p(slots), _p(has_state), _p(scale), rows, width,
                                out_cols, taps, b, int(max_q), _DT[out_dtype], _stream()), "norm_conv")
@@ -1058,8 +1058,10 @@ def latent_splits(batch: int, heads: int, rank: int, up_to: int) -> int:
     return int(max(1, min(wave // max(ctas, 1), tiles // 2, 16)))
 
 
-def latent_attention(q, rows, block_table, cu_q, seq_lens, scale, window, max_q, max_kv, splits=1, merge=True):
-    """``merge=False``: a split result stays a ``LatentSplit``."""
+def latent_attention(q, rows, block_table, cu_q, seq_lens, scale, window, max_q, max_kv, splits=1, merge=True,
+                     one_form=False):
+    """``merge=False``: a split result stays a ``LatentSplit``. ``one_form``: the same kernel variant whatever the number
+    of rows per request (verification rows must reproduce decode rows bit for bit)."""
     _bind_latent()
     t, h, r = q.shape
     assert q.is_contiguous() and rows.is_contiguous() and rows.shape[2] == r and rows.dtype == q.dtype
@@ -1072,8 +1074,8 @@ def latent_attention(q, rows, block_table, cu_q, seq_lens, scale, window, max_q,
         ws_l = torch.empty((splits, t * h), dtype=torch.float32, device=q.device)
     check(lib().msgl_latent_attention(
         _p(q), _p(rows), _p(out), _p(block_table), block_table.stride(0), _p(cu_q), _p(seq_lens), _p(ws_o), _p(ws_l),
-        seq_lens.numel(), t, int(max_q), h, r, rows.shape[1], rows.shape[0], int(window), splits, float(scale), _dt(q),
-        _stream()), "latent_attention")
+        seq_lens.numel(), t, int(max_q), h, r, rows.shape[1], rows.shape[0], int(window), splits, float(scale),
+        int(one_form), _dt(q), _stream()), "latent_attention")
     _count("latent_attention", "latent_attention_kernel", 2 if splits > 1 and merge else 1)
     return out if out is not None else LatentSplit(ws_o, ws_l, (t, h, r))
 

@@ -310,3 +310,20 @@ def test_engine_generates_the_greedy_tokens(model):
     assert o.cached_tokens > 0
     assert o.token_ids[0] == int(plain.logits(cfg, w, again)[-1].argmax())
     llm.shutdown()
+
+
+def test_draft_verification_keeps_the_greedy_tokens(model):
+    cfg, w, path, seqs, _ = model
+    prompts = [(seqs["b"][:20] * 4), seqs["c"][:12] * 6, seqs["d"]]
+    sp = SamplingParams(max_tokens=24, ignore_eos=True)
+    outs = []
+    for spec in ({}, dict(spec_algorithm="ngram", spec_num_draft=4)):
+        # without drafts, but on the code path that verification rows share
+        llm = LLM(path, device="cuda", dtype="bf16", page_size=16, max_running_req=4, num_page_override=128,
+                  spec_algorithm=spec.get("spec_algorithm", "ngram"), spec_num_draft=spec.get("spec_num_draft", 0) or 1)
+        if not spec:
+            llm.proposer = None
+        outs.append([o.token_ids for o in llm.generate(prompts, sp)])
+        assert not spec or llm.stats["spec_steps"] > 0
+        llm.shutdown()
+    assert outs[0] == outs[1]
