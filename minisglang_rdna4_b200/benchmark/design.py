@@ -121,7 +121,6 @@ def kernels(s: Dict) -> List[Dict]:
     """Every kernel of a Mitilix layer and the like one of the Mistral layer: prefill (8192 rows: four prompts of
     2048) and decode (64 requests at 2048 tokens)."""
     from .. import ops
-    from ..attention import create_attention_backend  # noqa: F401  (the backend's own split rules are used below)
     from ..attention.latent import LatentAttentionBackend
     from ..core import Batch, Context, set_global_ctx
     from ..kvcache import MHAKVCache
@@ -239,7 +238,7 @@ def kernels(s: Dict) -> List[Dict]:
         cs = get_rope_cache(RotaryConfig(d, d, MAX_POS, 1e4), torch.device(dev))
         qkv = rnd(t, (h + 2 * hk) * d)
         us = _time(lambda: ops.qk_norm_rope_store(qkv, None, None, pos, cs, h, hk, d, d, 1e-5, kv.k_cache(0), kv.v_cache(0), loc))
-        add("mistral", "rope + store", phase, us, t * (2 * h + 4 * hk) * d * 2 - t * h * d * 0, 0)
+        add("mistral", "rope + store", phase, us, t * (2 * h + 4 * hk) * d * 2, 0)
         q3 = rnd(t, h, d)
         spl = K.choose_splits(b, hk, MAX_POS, n == 1)
         us = _time(lambda: ops.paged_attention(q3, kv.k_cache(0), kv.v_cache(0), bt, cu, seq, d ** -0.5, window=win, max_q=n,
