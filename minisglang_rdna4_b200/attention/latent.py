@@ -19,8 +19,8 @@ from .base import AttnMetadata, BaseAttnBackend
 class LatentAttentionBackend(BaseAttnBackend):
     def __init__(self, layers, device, max_seq_len: int, single_split: bool = False) -> None:
         self.device = torch.device(device)
-        windows = [s.window for s in layers]
-        self.reach = max(windows) if min(windows) > 0 else 0
+        windows = [s.window for s in layers if s is not None]
+        self.reach = max(windows) if windows and min(windows) > 0 else 0
         self.max_seq_len = max_seq_len
         self.single_split = single_split       # speculative verification must reproduce decode rows bit for bit
 
@@ -43,12 +43,19 @@ class LatentAttentionBackend(BaseAttnBackend):
         raise NotImplementedError("models with a latent pool call latent_forward")
 
     def latent_forward(self, q, up_k, up_v, row: int, batch: Batch, *, scale: float, window: int, out,
-                       expand_k=None, store=None) -> None:
+                       expand_k=None, store=None, rope=None, sink=None, gate=None) -> None:
         """``q [T, H, dim]``, ``up_k [H, rank, dim]``, ``up_v [H, vdim, rank]`` -> ``out [T, H, vdim]``. ``expand_k``:
         ``up_k`` as ``[H * dim, rank]``, where the expanded form may be used. ``store`` (a layer with latents of its own):
-        ``(raw latents [T, rank], norm weight, rank, eps)`` to norm and store ahead of the attention."""
+        ``(raw latents [T, rank], norm weight, rank, eps)`` to norm and store ahead of the attention. ``rope``: ``(first
+        rotary channel of a query head, rotated channels, cos / sin table, width of the shared key part)``. ``sink [H]``,
+        ``gate [T, H]``: logits in the softmax denominator and of the sigmoid on the output."""
         md = batch.attn_metadata
         rows = get_global_ctx().kv_cache.rows(row)
+        if rope is not None:
+            dim, dims, table, rot_dim = rope
+            ops.latent_rope(q, dim, dims, table, batch.positions,
+                            None if store is None else (*store, rows, batch.out_loc, rot_dim))
+            store = None
         if store is not None:
             store = (*store, rows, batch.out_loc)
             if not (md.decode and q.is_cuda and q.dtype == torch.bfloat16):
@@ -59,7 +66,7 @@ class LatentAttentionBackend(BaseAttnBackend):
 
             if K.latent_prefill_ok(q.shape[2], up_v.shape[1], scale):
                 K.latent_prefill(q, expand_k, up_v, rows, row, md.block_table,
-                                 md.prefill_plan, scale, window, out)
+                                 md.prefill_plan, scale, window, out, sink=sink, gate=gate)
                 return
         q_lat = ops.head_gemm(q, up_k, store=store)
         splits = self._splits(q_lat, md, window)
@@ -67,18 +74,18 @@ class LatentAttentionBackend(BaseAttnBackend):
             from ..ops import cuda as K
 
             parts = K.latent_attention(q_lat, rows, md.block_table, md.cu_q, md.seq_lens, scale, window, md.max_q,
-                                       md.max_kv, splits, merge=False)
-            K.head_gemm_combine(parts, up_v, out)
+                                       md.max_kv, splits, merge=False, sink=sink)
+            K.head_gemm_combine(parts, up_v, out, gate=gate)
             return
         o_lat = ops.latent_attention(q_lat, rows, md.block_table, md.cu_q, md.seq_lens, scale, window, md.max_q,
-                                     md.max_kv, splits, one_form=self.single_split)
-        ops.head_gemm(o_lat, up_v, out)
+                                     md.max_kv, splits, one_form=self.single_split, sink=sink)
+        ops.head_gemm(o_lat, up_v, out, gate=gate)
 
     def _splits(self, q, md: AttnMetadata, window: int) -> int:
         """Key ranges per query tile of a decode step. Depends on the batch size and on what the window or the pool
         can hold, never on the lengths in the batch: a captured graph and an eager step reduce in the same order."""
         if (not md.decode or self.single_split or not q.is_cuda or q.dtype != torch.bfloat16
-                or q.shape[2] > 512):
+                or q.shape[2] > 576):
             return 1
         from ..ops.cuda import latent_splits
 

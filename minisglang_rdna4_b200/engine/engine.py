@@ -300,8 +300,9 @@ class Engine:
         elif mc.latent_layers:
             from ..kvcache.mla_pool import MLALatentCache
 
-            self.kv_cache = MLALatentCache(self.kv_layers, self.num_pages, self.page_size, max(mc.latent_widths), 0,
-                                           self.dtype, self.device, widths=mc.latent_widths)
+            self.kv_cache = MLALatentCache(self.kv_layers, self.num_pages, self.page_size,
+                                           max(mc.latent_widths, default=64), 0, self.dtype, self.device,
+                                           widths=mc.latent_widths)
         else:
             self.kv_cache = MHAKVCache(
                 self.kv_layers, self.num_pages, self.page_size, self.kv_heads_local, mc.head_dim,
@@ -349,11 +350,10 @@ class Engine:
         if mc.is_recurrent:
             from ..kvcache.gdn_state import GDNStateCache
 
-            conv_dim, st_heads, st_rows, st_cols = mc.recurrent_geometry
-            if not mc.input_conv_taps:             # (an input convolution runs on whole rows, on every rank)
-                conv_dim, st_heads = conv_dim // config.tp_size, st_heads // config.tp_size   # this rank's heads
+            conv_dim, st_heads, st_rows, st_cols = self._state_shape()
             self.gdn_state = GDNStateCache(mc.num_linear_layers, self.num_slots, conv_dim, mc.linear_conv_kernel_dim,
-                                           st_heads, st_rows, st_cols, self._conv_state_dtype, self.device)
+                                           st_heads, st_rows, st_cols, self._conv_state_dtype, self.device,
+                                           geometries=mc.state_geometries(config.tp_size))
             self.ledger.add("recurrent state", self.gdn_state.conv.numel() * self.gdn_state.conv.element_size()
                             + self.gdn_state.ssm.numel() * 4)
         self.ctx.gdn_state = self.gdn_state
@@ -535,6 +535,16 @@ class Engine:
         # the tail of an input convolution holds normalised rows of an fp32 residual stream
         return torch.float32 if self.model_config.input_conv_taps else self.dtype
 
+    def _state_shape(self):
+        """``ModelConfig.recurrent_geometry`` with this rank's heads."""
+        mc, tp = self.model_config, self.config.tp_size
+        conv_dim, heads, rows, cols = mc.recurrent_geometry
+        if mc.input_conv_taps:                     # an input convolution runs on whole rows, on every rank
+            return conv_dim, heads, rows, cols
+        if mc.linear_layers:
+            return conv_dim, heads, rows, cols // tp
+        return conv_dim // tp, heads // tp, rows, cols
+
     def _free_memory(self) -> int:
         if self.device.type == "cuda":
             torch.cuda.synchronize(self.device)
@@ -560,7 +570,7 @@ class Engine:
             per_page = MLALatentCache.token_bytes(self.kv_layers, int(mc.kv_lora_rank), int(mc.qk_rope_head_dim),
                                                   itemsize) * self.page_size
         if mc.latent_layers:
-            per_page = sum(mc.latent_widths) * itemsize * self.page_size
+            per_page = (sum(mc.latent_widths) or 64) * itemsize * self.page_size
         if cfg.spec_algorithm in ("eagle3", "mtp"):
             # the draft head keeps one 16-bit, unsharded layer of K/V on the same page table
             per_page += MHAKVCache.token_bytes(1, mc.num_kv_heads, mc.head_dim, 2) * self.page_size
@@ -578,12 +588,10 @@ class Engine:
         if mc.is_recurrent:
             from ..kvcache.gdn_state import GDNStateCache
 
-            conv_dim, st_heads, st_rows, st_cols = mc.recurrent_geometry
-            if not mc.input_conv_taps:
-                conv_dim, st_heads = conv_dim // cfg.tp_size, st_heads // cfg.tp_size
+            conv_dim, st_heads, st_rows, st_cols = self._state_shape()
             budget -= (cfg.max_running_req + 1) * GDNStateCache.slot_bytes(
-                mc.num_linear_layers, conv_dim, mc.linear_conv_kernel_dim, st_heads, st_rows, st_cols,
-                4 if mc.input_conv_taps else 2)
+                1 if mc.linear_layers else mc.num_linear_layers, conv_dim, mc.linear_conv_kernel_dim, st_heads, st_rows,
+                st_cols, 4 if mc.input_conv_taps else 2)
         pages = budget // per_page
         if self.cpu_group is not None:
             t = torch.tensor([pages], dtype=torch.int64)

@@ -1,4 +1,4 @@
-"""Per-request recurrent state of the gated-delta-net layers.
+"""Per-request recurrent state of the linear-attention layers (gated delta net, Mamba-2, decaying states).
 
 Every linear-attention layer keeps, per request slot (the request's row of the page table), the
 last ``kernel - 1`` inputs of its causal convolution and one ``[Dk, Dv]`` fp32 state matrix per
@@ -9,19 +9,28 @@ python/minisgl/scheduler/recurrent_slots.py:48-94).
 """
 from __future__ import annotations
 
-from typing import Dict, Optional, Tuple
+from typing import Dict, Optional, Sequence, Tuple
 
 import torch
 
 
 class GDNStateCache:
     def __init__(self, num_layers: int, num_slots: int, conv_dim: int, conv_kernel: int, num_v_heads: int,
-                 head_k_dim: int, head_v_dim: int, dtype: torch.dtype, device) -> None:
-        # no state matrix (num_v_heads 0): the state is the convolution tail alone
+                 head_k_dim: int, head_v_dim: int, dtype: torch.dtype, device,
+                 geometries: Optional[Sequence[Tuple[int, int, int]]] = None) -> None:
+        # no state matrix (num_v_heads 0): the state is the convolution tail alone. ``geometries``: (heads, rows, cols)
+        # of every layer where they differ: a request's state matrices are then one run of floats, layer after layer
+        self._geometries = tuple(geometries) if geometries is not None else None
+        if self._geometries is not None:
+            self.num_layers, self.num_slots = num_layers, num_slots
+            sizes = [h * r * c for h, r, c in self._geometries]
+            self._offsets = [sum(sizes[:i]) for i in range(len(sizes))]
+            self.ssm = torch.zeros((1, num_slots, 1, 1, sum(sizes)), dtype=torch.float32, device=device)
+        else:
+            self.ssm = torch.zeros((num_layers, num_slots, num_v_heads, head_k_dim, head_v_dim), dtype=torch.float32,
+                                   device=device)
         self.num_layers, self.num_slots = num_layers, num_slots
         self.conv = torch.zeros((num_layers, num_slots, conv_dim, conv_kernel - 1), dtype=dtype, device=device)
-        self.ssm = torch.zeros((num_layers, num_slots, num_v_heads, head_k_dim, head_v_dim), dtype=torch.float32,
-                               device=device)
         self._snapshots: Dict[object, Tuple[torch.Tensor, torch.Tensor]] = {}
         self._arena = None                      # pinned frames for snapshots kept on the host
         self.stream = None                      # the stream the snapshot / restore copies are issued on
@@ -49,6 +58,11 @@ class GDNStateCache:
         return self.conv[layer]
 
     def ssm_state(self, layer: int) -> torch.Tensor:
+        """``[slots, heads, rows, cols]`` of one layer (the slot stride may be longer than that)."""
+        if self._geometries is not None:
+            h, r, c = self._geometries[layer]
+            at = self._offsets[layer]
+            return self.ssm[0, :, 0, 0, at:at + h * r * c].unflatten(1, (h, r, c))
         return self.ssm[layer]
 
     # ---- speculative verify: keep the state of a batch's slots and put (some of) them back ----

@@ -35,9 +35,9 @@ class MLALatentCache(BaseKVCachePool):
         else:
             assert len(widths) == num_layers
             tokens = (num_pages + 1) * page_size
-            self.width = max(widths)
+            self.width = max(widths, default=self.width)
             self._buf = torch.zeros(tokens * sum(widths), dtype=dtype, device=device)
-            parts = self._buf.split([tokens * w for w in widths])
+            parts = self._buf.split([tokens * w for w in widths]) if widths else ()
             self._rows = [p.view(num_pages + 1, page_size, w) for p, w in zip(parts, widths)]
 
     @property

@@ -68,6 +68,11 @@ def _register_defaults() -> None:
     if "MitilixForCausalLM" not in MODEL_REGISTRY:
         MODEL_REGISTRY.register("MitilixForCausalLM")(MitilixForCausalLM)
 
+    from .rafodra import RafodraForCausalLM
+
+    if "RafodraForCausalLM" not in MODEL_REGISTRY:
+        MODEL_REGISTRY.register("RafodraForCausalLM")(RafodraForCausalLM)
+
 
 def create_model(cfg: ModelConfig, dtype: torch.dtype, device):
     """Instantiate the model for ``cfg`` with uninitialised (or meta) parameters."""

@@ -40,10 +40,13 @@ def _round_up(n: int, m: int) -> int:
 
 @dataclass(frozen=True)
 class LatentLayer:
-    """One layer whose attention keeps a shared latent per token (no rotary part): ``heads`` query heads of ``dim``
-    channels, values of ``vdim``, a latent of ``kv_rank``; ``window`` 0 = every earlier position is visible;
-    ``kv_from``: the layer whose latent is read instead of an own one; ``ff`` 0 = no feed-forward. The ``*_pad``
-    widths are what the kernels see: zero channels that change no dot product."""
+    """One layer whose attention keeps a shared latent per token: ``heads`` query heads of ``dim`` channels, values of
+    ``vdim``, a latent of ``kv_rank``; ``window`` 0 = every earlier position is visible; ``kv_from``: the layer whose
+    latent is read instead of an own one; ``ff`` 0 = no feed-forward (of this kind). ``rot_dim`` further query channels
+    per head score against one rotary key that all heads share and that is cached behind the latent: its first
+    ``rotary.rotary_dim`` channels are rotated. ``sink``: a learned logit per head in the softmax denominator;
+    ``gate``: a sigmoid gate per head on the output. The ``*_pad`` widths are what the kernels see: zero channels that
+    change no dot product."""
 
     heads: int
     dim: int
@@ -53,6 +56,44 @@ class LatentLayer:
     window: int = 0
     kv_from: Optional[int] = None
     ff: int = 0
+    rot_dim: int = 0
+    rotary: Optional[RotaryConfig] = None
+    sink: bool = False
+    gate: bool = False
+
+    @property
+    def dim_pad(self) -> int:
+        return _round_up(self.dim + self.rot_dim, 16)
+
+    @property
+    def vdim_pad(self) -> int:
+        return _round_up(self.vdim, 16)
+
+    @property
+    def rank_pad(self) -> int:
+        """Pool row: the latent, the shared rotary key, zeros."""
+        r = _round_up(self.kv_rank + self.rot_dim, 64)
+        return r if r <= 256 or r == 576 else _round_up(r, 256)
+
+
+@dataclass(frozen=True)
+class LinearAttnLayer:
+    """One linear-attention layer without a delta rule: per head a ``[dim, vdim]`` state that decays and takes up
+    ``k v^T`` of every token. The decay is one number per head (``decay``) or comes from the input, one per key channel:
+    ``sigmoid(z) ** (1 / tau)`` with ``z`` a projection of rank ``gate_rank`` plus a bias (``decay`` None). ``act``: silu on
+    the projected q, k and v. The output is RMS-normed over all heads together (``joint_norm``) or per head with one
+    shared weight, and gated by ``gate_act`` of a projection."""
+
+    heads: int
+    dim: int
+    vdim: int
+    decay: Optional[Tuple[float, ...]] = None
+    gate_rank: int = 0
+    tau: float = 1.0
+    act: bool = False
+    q_scale: float = 1.0
+    joint_norm: bool = False
+    gate_act: str = "silu"
 
     @property
     def dim_pad(self) -> int:
@@ -62,10 +103,33 @@ class LatentLayer:
     def vdim_pad(self) -> int:
         return _round_up(self.vdim, 16)
 
-    @property
-    def rank_pad(self) -> int:
-        r = _round_up(self.kv_rank, 64)
-        return r if r <= 256 else _round_up(r, 256)
+
+@dataclass(frozen=True)
+class ExpertSpec:
+    """A mixture of ``experts`` feed-forwards of width ``ff`` of which each token uses ``top``, chosen among the best
+    ``keep`` of ``groups`` groups; ``shared_ff`` > 0: a further one for every token behind a sigmoid gate. Expert
+    activation: gate and up halves clamped at ``limit``, ``g * sigmoid(alpha g) * (u + 1)``."""
+
+    experts: int
+    top: int
+    ff: int
+    limit: float
+    groups: int = 1
+    keep: int = 1
+    scale: float = 1.0
+    shared_ff: int = 0
+    shared_limit: float = 0.0
+    alpha: float = 1.702
+
+
+@dataclass(frozen=True)
+class LayerSpec:
+    """A sequential layer of a model whose layers are listed one by one: a mixer, and a feed-forward that is dense and
+    gated (``ff`` > 0), a mixture of experts (``moe``) or absent."""
+
+    mixer: Any                              # LatentLayer | LinearAttnLayer
+    ff: int = 0
+    moe: Optional[ExpertSpec] = None
 
 
 @dataclass(frozen=True)
@@ -127,8 +191,11 @@ class ModelConfig:
     norm_plus_one: bool = False           # RMSNorm weights are stored as (w - 1)
     # layers that keep an attention latent per token, each with its own sizes; a short causal convolution ahead of
     # every sublayer (taps, 0 = none) whose last inputs are per-request state
-    latent_layers: Optional[Tuple[LatentLayer, ...]] = None
+    latent_layers: Optional[Tuple[Optional[LatentLayer], ...]] = None    # None at a layer that keeps no latent
     input_conv_taps: int = 0
+    # models whose layers are described one by one (mixer and feed-forward of different kinds and sizes)
+    layer_specs: Optional[Tuple[LayerSpec, ...]] = None
+    embedding_multiplier: float = 1.0
     # misc
     sliding_window: Optional[int] = None
     layer_types: Optional[Tuple[str, ...]] = None
@@ -183,24 +250,42 @@ class ModelConfig:
     @property
     def latent_widths(self) -> Tuple[int, ...]:
         """Pool row width of every layer that keeps a latent of its own, in layer order."""
-        return tuple(s.rank_pad for s in self.latent_layers or () if s.kv_from is None)
+        return tuple(s.rank_pad for s in self.latent_layers or () if s is not None and s.kv_from is None)
 
     def latent_row(self, layer: int) -> int:
         """Index in the latent pool of the layer whose latent ``layer`` reads."""
         specs = self.latent_layers
         owner = layer if specs[layer].kv_from is None else specs[layer].kv_from
-        return sum(1 for s in specs[:owner] if s.kv_from is None)
+        return sum(1 for s in specs[:owner] if s is not None and s.kv_from is None)
 
     @property
     def is_recurrent(self) -> bool:
         """Some layers keep a recurrent state (or a convolution tail) per request besides or instead of K/V pages."""
-        return self.input_conv_taps > 0 or bool(self.layer_types) and any(t in ("linear_attention", "mamba") for t in self.layer_types)
+        return (self.input_conv_taps > 0 or bool(self.linear_layers)
+                or bool(self.layer_types) and any(t in ("linear_attention", "mamba") for t in self.layer_types))
+
+    @property
+    def linear_layers(self) -> Tuple[Tuple[int, LinearAttnLayer], ...]:
+        """``(layer, spec)`` of the linear-attention layers of a model with ``layer_specs``."""
+        return tuple((i, s.mixer) for i, s in enumerate(self.layer_specs or ()) if isinstance(s.mixer, LinearAttnLayer))
+
+    def state_row(self, layer: int) -> int:
+        """Index of a linear-attention layer in the state cache."""
+        return sum(1 for i, _ in self.linear_layers if i < layer)
+
+    def state_geometries(self, tp: int = 1) -> Optional[Tuple[Tuple[int, int, int], ...]]:
+        """``(heads, rows, cols)`` of every state layer where layers may differ; ``None``: ``recurrent_geometry``."""
+        if not self.linear_layers:
+            return None
+        return tuple((m.heads // tp, m.dim_pad, m.vdim_pad) for _, m in self.linear_layers)
 
     @property
     def num_linear_layers(self) -> int:
         """Layers with a recurrent state (gated delta net, Mamba-2, input convolutions)."""
         if self.input_conv_taps:
             return self.num_layers
+        if self.layer_specs:
+            return len(self.linear_layers)
         return sum(1 for t in (self.layer_types or ()) if t in ("linear_attention", "mamba"))
 
     @property
@@ -250,6 +335,8 @@ class ModelConfig:
         over ``conv channels`` inputs and a ``[heads, rows, cols]`` fp32 state matrix per request (``heads`` 0: the window alone)."""
         if self.input_conv_taps:
             return self.hidden_size, 0, 0, 0
+        if self.linear_layers:                 # no convolution; the state matrices of all layers as one row
+            return 0, 1, 1, sum(m.heads * m.dim_pad * m.vdim_pad for _, m in self.linear_layers)
         if self.mamba_num_heads:
             inter = self.mamba_num_heads * self.mamba_head_dim
             return (inter + 2 * self.mamba_n_groups * self.ssm_state_size, self.mamba_num_heads, self.mamba_head_dim,
@@ -294,16 +381,19 @@ class ModelConfig:
     @staticmethod
     def from_hf(cfg: Any) -> "ModelConfig":
         """Build from a dict, a ``transformers`` config object or a path to ``config.json``."""
+        folder = None
         if isinstance(cfg, (str, os.PathLike)):
             path = os.fspath(cfg)
             if os.path.isdir(path):
-                path = os.path.join(path, "config.json")
+                folder, path = path, os.path.join(path, "config.json")
             with open(path) as fh:
                 cfg = json.load(fh)
         if not isinstance(cfg, dict):
             cfg = cfg.to_dict()
         if cfg.get("architecture") == "Mitilix":
             return _mitilix_config(cfg)
+        if cfg.get("architecture") == "Rafodra":
+            return _rafodra_config(cfg, folder)
         vision = None
         if "text_config" in cfg and isinstance(cfg["text_config"], dict):
             if str(cfg.get("model_type", "")).startswith("gemma3") and cfg.get("vision_config"):
@@ -564,6 +654,103 @@ def _mitilix_config(cfg: Dict[str, Any]) -> ModelConfig:
         linear_conv_kernel_dim=int(cfg["canon"]["taps"]), max_position_embeddings=max_pos, eos_token_ids=eos_ids,
         bos_token_id=cfg.get("bos_token_id"),
     )
+
+
+def _tensor_rows(folder: Optional[str]) -> Dict[str, int]:
+    """First dimension of every tensor of the checkpoint in ``folder`` (sizes its config.json does not give)."""
+    import glob
+    import struct
+
+    rows: Dict[str, int] = {}
+    for path in sorted(glob.glob(os.path.join(folder, "*.safetensors"))) if folder else ():
+        with open(path, "rb") as fh:
+            header = json.loads(fh.read(struct.unpack("<Q", fh.read(8))[0]))
+        rows.update({k: int(v["shape"][0]) for k, v in header.items() if k != "__metadata__" and v["shape"]})
+    return rows
+
+
+def _latent_mixer(i: int, mix: Dict[str, Any], specs: List[LayerSpec], max_pos: int) -> LatentLayer:
+    rot_dim, rot = int(mix.get("rot_dim") or 0), mix.get("rot") or {}
+    dims = int(rot.get("dims", rot_dim)) if rot_dim else 0
+    if rot_dim and not 0 < dims <= rot_dim or dims % 2:
+        raise ValueError(f"layer {i}: {dims} rotated of {rot_dim} rotary channels")
+    rotary = RotaryConfig(rot_dim, dims, max_pos, float(rot["base"]), interleaved=True) if dims else None
+    spec = LatentLayer(heads=int(mix["heads"]), dim=int(mix["dim"]), vdim=int(mix["vdim"]), kv_rank=int(mix["kv_rank"]),
+                       scale=float(mix["scale"]), kv_from=None if mix.get("kv_from") is None else int(mix["kv_from"]),
+                       rot_dim=rot_dim, rotary=rotary, sink=True, gate=True)
+    if spec.kv_from is not None:
+        donor = specs[spec.kv_from].mixer if 0 <= spec.kv_from < i else None
+        if not (isinstance(donor, LatentLayer) and donor.kv_from is None
+                and (donor.kv_rank, donor.rot_dim, donor.rotary) == (spec.kv_rank, rot_dim, rotary)):
+            raise ValueError(f"layer {i}: kv_from {spec.kv_from} names no earlier layer with a latent of this size")
+    return spec
+
+
+def _rafodra_config(cfg: Dict[str, Any], folder: Optional[str]) -> ModelConfig:
+    """``layers`` lists every layer's mixer and feed-forward with sizes of their own. The rank of a channel-decay gate is
+    only in the checkpoint's tensor shapes (``gate_rank`` of the mixer where there is no checkpoint)."""
+    rows = _tensor_rows(folder)
+    max_pos = int(cfg.get("max_positions") or 131072)      # the design sets no limit: one for tables and buffers
+    specs: List[LayerSpec] = []
+    for i, layer in enumerate(cfg["layers"]):
+        kind, mix, mlp = layer["type"], layer["mixer"], layer.get("mlp")
+        if kind == "latent_attention":
+            mixer: Any = _latent_mixer(i, mix, specs, max_pos)
+        elif kind in ("lightning", "gla"):
+            sizes = dict(heads=int(mix["heads"]), dim=int(mix["dim"]), vdim=int(mix["vdim"]))
+            if kind == "lightning":
+                decay = tuple(float(d) for d in mix["decay"])
+                if len(decay) != sizes["heads"]:
+                    raise ValueError(f"layer {i}: {len(decay)} decays for {sizes['heads']} heads")
+                mixer = LinearAttnLayer(**sizes, decay=decay, act=True, joint_norm=True, gate_act="sigmoid")
+            else:
+                rank = int(mix.get("gate_rank") or rows.get(f"l{i}.mix.a1") or 0)
+                if rank <= 0:
+                    raise ValueError(f"layer {i}: the rank of its decay gate is neither in the checkpoint nor given")
+                mixer = LinearAttnLayer(**sizes, gate_rank=rank, tau=float(mix["tau"]), q_scale=sizes["dim"] ** -0.5)
+        else:
+            raise ValueError(f"layer {i}: unknown mixer type {kind!r}")
+        ff, moe = 0, None
+        if mlp is not None and mlp["kind"] == "dense":
+            ff = int(mlp["ff"])
+        elif mlp is not None and mlp["kind"] == "moe":
+            router, groups, shared = mlp["router"], mlp["router"].get("groups") or {}, mlp.get("shared")
+            moe = ExpertSpec(
+                experts=int(router["experts"]), top=int(router["top"]), ff=int(mlp["expert"]["ff"]),
+                limit=float(mlp["expert"]["limit"]), groups=int(groups.get("count", 1)), keep=int(groups.get("keep", 1)),
+                scale=float(router.get("scale", 1.0)), shared_ff=int(shared["ff"]) if shared else 0,
+                shared_limit=float(shared["limit"]) if shared else 0.0)
+            if moe.experts % moe.groups or not 0 < moe.top <= moe.experts // moe.groups * moe.keep:
+                raise ValueError(f"layer {i}: {moe.top} of {moe.experts} experts in {moe.groups} groups, {moe.keep} kept")
+        elif mlp is not None:
+            raise ValueError(f"layer {i}: unknown feed-forward kind {mlp['kind']!r}")
+        specs.append(LayerSpec(mixer, ff, moe))
+    eos = cfg.get("eos_token_id")
+    eos_ids = tuple(eos) if isinstance(eos, (list, tuple)) else (() if eos is None else (int(eos),))
+    return layered_config(specs, width=int(cfg["width"]), vocab=int(cfg["vocab"]), eps=float(cfg["norm"]["eps"]),
+                          embedding_multiplier=float(cfg["embedding"]["scale"]), max_positions=max_pos,
+                          eos_token_ids=eos_ids, bos_token_id=cfg.get("bos_token_id"))
+
+
+def layered_config(specs, width: int, vocab: int, eps: float, embedding_multiplier: float = 1.0,
+                   max_positions: int = 131072, eos_token_ids: Tuple[int, ...] = (), bos_token_id=None) -> ModelConfig:
+    """A Rafodra configuration from its layers."""
+    latent = tuple(s.mixer if isinstance(s.mixer, LatentLayer) else None for s in specs)
+    first = next((m for m in latent if m is not None), None)
+    row = first.rank_pad if first is not None else 64
+
+    def widest(s: LayerSpec) -> int:        # activations of one token
+        m = s.mixer
+        mix = m.heads * m.rank_pad if isinstance(m, LatentLayer) else m.heads * (2 * m.dim + 2 * m.vdim)
+        return max(mix, s.ff, s.moe.top * s.moe.ff + s.moe.shared_ff if s.moe else 0)
+
+    return ModelConfig(
+        num_layers=len(specs), num_qo_heads=first.heads if first is not None else specs[0].mixer.heads, num_kv_heads=1,
+        head_dim=row, hidden_size=width, vocab_size=vocab, intermediate_size=max(widest(s) for s in specs),
+        rms_norm_eps=eps, rotary_config=RotaryConfig(row, 0, max_positions, base=10000.0), model_type="rafodra",
+        architectures=("RafodraForCausalLM",), latent_layers=latent, layer_specs=tuple(specs), linear_conv_kernel_dim=1,
+        embedding_multiplier=embedding_multiplier, max_position_embeddings=max_positions, eos_token_ids=eos_token_ids,
+        bos_token_id=bos_token_id)
 
 
 def _default_arch(model_type: str) -> List[str]:

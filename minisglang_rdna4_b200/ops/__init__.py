@@ -208,10 +208,11 @@ def rms_norm_gated(x, z, w, eps: float):
 
 
 # ---------------------------------------------------------------------------- fp32 residual, latent attention
-def embed_positions(ids, weight, pos, positions, vocab_start: int = 0, vocab_len: Optional[int] = None):
+def embed_positions(ids, weight, pos, positions, vocab_start: int = 0, vocab_len: Optional[int] = None,
+                    scale: float = 1.0):
     if weight.is_cuda:
-        return _cuda().embed_positions(ids, weight, pos, positions, vocab_start, vocab_len)
-    return ref.embed_positions(ids, weight, pos, positions, vocab_start, vocab_len)
+        return _cuda().embed_positions(ids, weight, pos, positions, vocab_start, vocab_len, scale)
+    return ref.embed_positions(ids, weight, pos, positions, vocab_start, vocab_len, scale)
 
 
 def add_scalar_norm_conv(x, delta, gain, eps: float, w1, w2, state, cu_q, slots, has_state, max_q: int, out_dtype,
@@ -237,19 +238,57 @@ def latent_norm_store(c, weight, rank: int, eps: float, rows, out_loc):
     return ref.latent_norm_store(c, weight, rank, eps, rows, out_loc)
 
 
-def head_gemm(x, w, out=None, store=None):
+def latent_rope(q, dim: int, dims: int, cos_sin, positions, store=None):
+    """Rotates the rotary channels of the query heads in place and, with ``store``, norms, rotates and stores the step's
+    latents in the same launch."""
+    if q.is_cuda:
+        return _cuda().latent_rope(q, dim, dims, cos_sin, positions, store)
+    return ref.latent_rope(q, dim, dims, cos_sin, positions, store)
+
+
+def head_gemm(x, w, out=None, store=None, gate=None):
     if x.is_cuda:
-        return _cuda().head_gemm(x, w, out, store)
+        return _cuda().head_gemm(x, w, out, store, gate)
     assert store is None
-    return ref.head_gemm(x, w, out)
+    return ref.head_gemm(x, w, out, gate)
 
 
 def latent_attention(q, rows, block_table, cu_q, seq_lens, scale: float, window: int, max_q: int, max_kv: int,
-                     splits: int = 1, one_form: bool = False):
+                     splits: int = 1, one_form: bool = False, sink=None):
     if q.is_cuda:
         return _cuda().latent_attention(q, rows, block_table, cu_q, seq_lens, scale, window, max_q, max_kv, splits,
-                                        one_form=one_form)
-    return ref.latent_attention(q, rows, block_table, cu_q, seq_lens, scale, window)
+                                        one_form=one_form, sink=sink)
+    return ref.latent_attention(q, rows, block_table, cu_q, seq_lens, scale, window, sink)
+
+
+# ---------------------------------------------------------------------------- weighted norm, decaying linear attention
+def add_norm(x, delta, weight, eps: float, center: bool, out_dtype, out_cols: int):
+    """Residual add and norm (layer norm without a bias, or RMS) in one pass: ``(new residual, y)``. ``delta`` may be
+    the unreduced K ranges of a GEMM (``SplitPartial``)."""
+    if x.is_cuda:
+        return _cuda().add_norm(x, delta, weight, eps, center, out_dtype, out_cols)
+    return ref.add_norm(x, delta, weight, eps, center, out_dtype, out_cols)
+
+
+def linear_attention(q, k, v, state, cu_q, slots, has_state, decay=None, gate=None, tau: float = 1.0,
+                     q_scale: float = 1.0, act: bool = False, chunked: bool = False):
+    """``chunked``: the step may take the tensor-core form (prompts); otherwise every row takes the recurrent one."""
+    if q.is_cuda:
+        return _cuda().linear_attention(q, k, v, state, cu_q, slots, has_state, decay, gate, tau, q_scale, act, chunked)
+    return ref.linear_attention(q, k, v, state, cu_q, slots, has_state, decay, gate, tau, q_scale, act)
+
+
+def norm_gate(o, g, weight, eps: float, vdim: int, joint: bool, act: str, out_cols: int, total=None,
+              total_heads: int = 0):
+    if o.is_cuda:
+        return _cuda().norm_gate(o, g, weight, eps, vdim, joint, act, out_cols, total, total_heads)
+    return ref.norm_gate(o, g, weight, eps, vdim, joint, act, out_cols, total, total_heads)
+
+
+def clamped_glu(x, limit: float, alpha: float):
+    if x.is_cuda:
+        return _cuda().act_and_mul(x, "clamped", alpha, limit)
+    return ref.clamped_glu(x, limit, alpha)
 
 
 # ---------------------------------------------------------------------------- sampling
@@ -271,6 +310,16 @@ def moe_route(router_logits, top_k: int, renormalize: bool, scoring: str = "soft
     if router_logits.is_cuda:
         return _cuda().moe_route(router_logits, top_k, renormalize, scoring, bias, scale)
     return ref.moe_route(router_logits, top_k, renormalize, scoring, bias, scale)
+
+
+def experts_partial32(x, w13, w2, topk_w, topk_ids, limit: float, alpha: float, shared=None, shared_gate=None,
+                      counts=None):
+    """fp32 sum of the routed clamped experts and a gated shared one, for an fp32 residual stream."""
+    if x.is_cuda:
+        from . import moe_kernels
+
+        return moe_kernels.experts_partial32(x, w13, w2, topk_w, topk_ids, limit, alpha, shared, shared_gate, counts)
+    return ref.experts_partial32(x, w13, w2, topk_w, topk_ids, limit, alpha, shared, shared_gate)
 
 
 def moe_forward(x, w13, w2, topk_w, topk_ids, expert_offset: int = 0):

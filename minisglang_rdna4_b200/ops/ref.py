@@ -611,9 +611,10 @@ def rms_norm_gated(x: torch.Tensor, z: torch.Tensor, w: torch.Tensor, eps: float
 # fp32 residual stream with a scalar-gain norm and short input convolutions; windowed latent attention
 # ------------------------------------------------------------------------------------------
 def embed_positions(ids: torch.Tensor, weight: torch.Tensor, pos: Optional[torch.Tensor], positions: torch.Tensor,
-                    vocab_start: int = 0, vocab_len: Optional[int] = None) -> torch.Tensor:
-    """Token embedding (zero outside this rank's vocabulary range) plus a learned position vector, fp32 ``[T, W]``."""
-    x = embedding(ids, weight, vocab_start, vocab_len).float()
+                    vocab_start: int = 0, vocab_len: Optional[int] = None, scale: float = 1.0) -> torch.Tensor:
+    """Token embedding (zero outside this rank's vocabulary range) times ``scale`` plus a learned position vector,
+    fp32 ``[T, W]``."""
+    x = embedding(ids, weight, vocab_start, vocab_len).float() * scale
     return x if pos is None else x + pos[positions.long()].float()
 
 
@@ -667,9 +668,35 @@ def latent_norm_store(c: torch.Tensor, weight: torch.Tensor, rank: int, eps: flo
     flat.index_copy_(0, out_loc.long(), F.pad(y, (0, flat.shape[1] - rank)).to(flat.dtype))
 
 
-def head_gemm(x: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """Per-head projection: ``x [T, H, K]``, ``w [H, N, K]`` -> ``[T, H, N]``."""
+def rotate_pairs_(x: torch.Tensor, dims: int, cos_sin: torch.Tensor, positions: torch.Tensor) -> None:
+    """Turns neighbouring pairs of the first ``dims`` channels of ``x [T, ..., n]`` in place (``cos_sin [P, dims]``)."""
+    t = cos_sin[positions.long()].view(x.shape[0], *[1] * (x.dim() - 2), dims)
+    c, s = t[..., :dims // 2], t[..., dims // 2:]
+    u, v = x[..., 0:dims:2].float(), x[..., 1:dims:2].float()
+    x[..., 0:dims:2], x[..., 1:dims:2] = (u * c - v * s).to(x.dtype), (v * c + u * s).to(x.dtype)
+
+
+def latent_rope(q: torch.Tensor, dim: int, dims: int, cos_sin: torch.Tensor, positions: torch.Tensor,
+                store=None) -> None:
+    """Rotates channels ``dim .. dim + dims`` of every query head ``q [T, H, D]`` in place. ``store``: the arguments of
+    ``latent_norm_store``: the latents are normed and stored with the shared key part behind them, which is rotated
+    too (``dims`` channels; the rest of the row as it is)."""
+    rotate_pairs_(q[..., dim:], dims, cos_sin, positions)
+    if store is not None:
+        c, weight, rank, eps, rows, out_loc, rot_dim = store
+        latent_norm_store(c, weight, rank, eps, rows, out_loc)
+        k = c[:, rank:rank + rot_dim].float().clone()
+        rotate_pairs_(k, dims, cos_sin, positions)
+        flat = rows.view(-1, rows.shape[-1])
+        flat[out_loc.long(), rank:rank + rot_dim] = k.to(flat.dtype)
+
+
+def head_gemm(x: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = None,
+              gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """Per-head projection: ``x [T, H, K]``, ``w [H, N, K]`` -> ``[T, H, N]``, times ``sigmoid(gate [T, H])``."""
     y = torch.einsum("thk,hnk->thn", x.float(), w.float())
+    if gate is not None:
+        y = y * torch.sigmoid(gate.float())[..., None]
     if out is None:
         return y.to(x.dtype)
     out.copy_(y)
@@ -677,9 +704,11 @@ def head_gemm(x: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = No
 
 
 def latent_attention(q: torch.Tensor, rows: torch.Tensor, block_table: torch.Tensor, cu_q: torch.Tensor,
-                     seq_lens: torch.Tensor, scale: float, window: int) -> torch.Tensor:
+                     seq_lens: torch.Tensor, scale: float, window: int,
+                     sink: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Causal attention of ``q [T, H, R]`` over one shared latent per position that is key and value at once
-    (``rows [pages, page_size, R]``); ``window > 0``: the last ``window`` positions, the query's own included."""
+    (``rows [pages, page_size, R]``); ``window > 0``: the last ``window`` positions, the query's own included;
+    ``sink [H]``: a logit per head that only the denominator counts."""
     t, h, r = q.shape
     ps = rows.shape[1]
     out = torch.zeros((t, h, r), dtype=torch.float32, device=q.device)
@@ -699,5 +728,86 @@ def latent_attention(q: torch.Tensor, rows: torch.Tensor, block_table: torch.Ten
         if window > 0:
             hidden |= gap >= window
         s = s.masked_fill(hidden[None], float("-inf"))
-        out[qs:qe] = torch.einsum("hqk,kr->qhr", torch.softmax(s, -1), c)
+        if sink is not None:
+            s = torch.cat([s, sink.float()[:, None, None].expand(h, n, 1)], -1)
+        p = torch.softmax(s, -1)[..., :idx.numel()]
+        out[qs:qe] = torch.einsum("hqk,kr->qhr", p, c)
     return out.to(q.dtype)
+
+
+# ------------------------------------------------------------------------------------------
+# fp32 residual stream with a weighted norm; decaying linear attention; clamped experts
+# ------------------------------------------------------------------------------------------
+def add_norm(x: torch.Tensor, delta: Optional[torch.Tensor], weight: torch.Tensor, eps: float, center: bool,
+             out_dtype: torch.dtype, out_cols: int) -> Tuple[torch.Tensor, torch.Tensor]:
+    """``x += delta`` (fp32); layer norm without a bias (``center``) or RMS norm. Returns ``(x, y [T, out_cols])``."""
+    xn = x if delta is None else x + delta[:, :x.shape[1]].float()
+    d = xn - xn.mean(-1, keepdim=True) if center else xn
+    y = d * torch.rsqrt(d.pow(2).mean(-1, keepdim=True) + eps) * weight[:x.shape[1]].float()
+    return xn, F.pad(y, (0, out_cols - y.shape[1])).to(out_dtype)
+
+
+def linear_attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, state: torch.Tensor, cu_q: torch.Tensor,
+                     slots: torch.Tensor, has_state: torch.Tensor, decay: Optional[torch.Tensor] = None, gate=None,
+                     tau: float = 1.0, q_scale: float = 1.0, act: bool = False) -> torch.Tensor:
+    """Per head ``S <- diag(alpha_t) S + k_t v_t^T``, ``o_t = S^T q_t`` over packed sequences; ``q``, ``k [T, H, dk]``,
+    ``v [T, H, dv]``, ``state [slots, H, dk, dv]`` fp32, updated in place. ``alpha``: ``decay [H]``, or per key channel
+    ``sigmoid(low W^T + bias) ** (1 / tau)`` from ``gate = (low [T, r], W [H * dk, r], bias [H * dk])``."""
+    t, h, dk = q.shape
+    qf, kf, vf = (F.silu(x.float()) if act else x.float() for x in (q, k, v))
+    qf = qf * q_scale
+    if gate is not None:
+        low, w, bias = gate
+        z = low.float() @ w.float().t() + bias.float()
+        alpha = torch.exp(F.logsigmoid(z) / tau).view(t, h, dk)
+    else:
+        alpha = decay.float().view(1, h, 1).expand(t, h, dk)
+    out = torch.zeros(t, h, v.shape[2], dtype=torch.float32, device=q.device)
+    for b in range(cu_q.numel() - 1):
+        slot = int(slots[b])
+        s = state[slot].clone() if int(has_state[b]) else torch.zeros_like(state[slot])
+        for i in range(int(cu_q[b]), int(cu_q[b + 1])):
+            s = s * alpha[i][..., None] + kf[i][..., None] * vf[i][:, None, :]
+            out[i] = torch.einsum("hkv,hk->hv", s, qf[i])
+        state[slot] = s
+    return out.to(q.dtype)
+
+
+def norm_gate(o: torch.Tensor, g: torch.Tensor, weight: torch.Tensor, eps: float, vdim: int, joint: bool, act: str,
+              out_cols: int, total: Optional[torch.Tensor] = None, total_heads: int = 0) -> torch.Tensor:
+    """``o [T, H, dv_pad]`` (zero past ``vdim``): RMS norm per head (one weight for all heads) or over all heads together
+    (``joint``), times ``sigmoid`` or ``silu`` of ``g [T, H * dv_pad]`` -> ``[T, out_cols]``. ``total [T]``: the sum of
+    squares over ``total_heads`` heads, where other ranks hold some of them."""
+    t, h, dv = o.shape
+    x = o.float()
+    if joint:
+        ss = x.pow(2).sum((1, 2)) if total is None else total
+        x = x * torch.rsqrt(ss / ((total_heads or h) * vdim) + eps)[:, None, None]
+        x = x * weight.float().view(1, h, dv)
+    else:
+        x = x * torch.rsqrt(x.pow(2).sum(-1, keepdim=True) / vdim + eps) * weight.float().view(1, 1, dv)
+    gf = g.float().reshape(t, h, dv)
+    y = x * (torch.sigmoid(gf) if act == "sigmoid" else F.silu(gf))
+    return F.pad(y.reshape(t, h * dv), (0, out_cols - h * dv)).to(o.dtype)
+
+
+def clamped_glu(x: torch.Tensor, limit: float, alpha: float) -> torch.Tensor:
+    """``g sigmoid(alpha g) (u + 1)`` of the halves ``[gate, up]`` clamped at ``limit`` (the gate from above only)."""
+    g, u = x.float().chunk(2, -1)
+    g, u = g.clamp(max=limit), u.clamp(-limit, limit)
+    return (g * torch.sigmoid(alpha * g) * (u + 1.0)).to(x.dtype)
+
+
+def experts_partial32(x: torch.Tensor, w13: torch.Tensor, w2: torch.Tensor, topk_w: torch.Tensor,
+                      topk_ids: torch.Tensor, limit: float, alpha: float, shared: Optional[torch.Tensor] = None,
+                      shared_gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """fp32 ``sum_k w_k * expert_k(x) + sigmoid(shared_gate) * shared`` with clamped experts."""
+    out = torch.zeros(x.shape[0], w2.shape[1], dtype=torch.float32, device=x.device)
+    if shared is not None:
+        out[:, :shared.shape[1]] += shared.float() * torch.sigmoid(shared_gate.float())[:, None]
+    for e in range(w13.shape[0]):
+        rows, slot = (topk_ids == e).nonzero(as_tuple=True)
+        if rows.numel():
+            y = clamped_glu((x[rows].float() @ w13[e].float().t()).to(x.dtype), limit, alpha)
+            out.index_add_(0, rows, (y.float() @ w2[e].float().t()).to(x.dtype).float() * topk_w[rows, slot][:, None])
+    return out
