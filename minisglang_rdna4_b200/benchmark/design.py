@@ -210,7 +210,7 @@ def kernels(s: Dict) -> List[Dict]:
             base = plan.tables.data_ptr()
             us = _time(lambda: lib().msgl_attn_prefill_pos(
                 q.data_ptr(), q.stride(0), q.stride(1), k_all.data_ptr(), vt.data_ptr(), plan.t_pad, out.data_ptr(),
-                out.stride(0), out.stride(1), base, plan.n_items, t, h, d, d, win, d ** -0.5, 0,
+                out.stride(0), out.stride(1), base, plan.n_items, t, h, d, d, win, d ** -0.5, None, None, 0, 0,
                 torch.cuda.current_stream().cuda_stream))
             add("mitilix", "expanded attention (window, tcgen05)", phase, us, t * h * d * 2 * 4, 2 * t * h * seen * 2 * d)
             del k_all, vt

@@ -72,6 +72,8 @@ def _compile(cmd: List[str], out: str, log: str) -> str:
 # on a fresh checkout compiles what that family needs.
 PARTS = {
     "latent": ["elementwise", "gemm_tcgen05", "gemm_f32", "norm_conv", "latent_attention", "attention_tc", "sampling"],
+    "layered": ["elementwise", "gemm_tcgen05", "gemm_f32", "norm_conv", "residual_norm", "latent_attention",
+                "attention_tc", "linear_attention", "moe", "sampling"],
 }
 
 

@@ -67,6 +67,9 @@ struct TcArgs {
   int window;          // > 0: a row sees the last ``window`` positions, its own included
   long long ldo, ho;   // element strides of a row and a head of out
   int v_chunks;        // 16-byte chunks of a value head
+  const float* sink;   // [Hq] logits that only the softmax denominator counts, or null
+  const void* gate;    // [rows, ...] logits of a sigmoid gate per row and head (row stride ldg), or null
+  long long ldg;
 };
 
 __device__ int g_attn_tc_status = 0;
@@ -413,8 +416,17 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
     }
     if (ok && nb > 0 && mbar_wait(o_full(t), (uint32_t)((nb - 1) & 1), abort_flag, args.status, 211)) {
       tc_fence_after();
-      const float inv = (l > 0.f ? 1.f / l : 0.f) * (args.v_scale != nullptr ? args.v_scale[hk] : 1.f);
       const int out_row = row + (POS ? t * kTile : 0);
+      float num = args.v_scale != nullptr ? args.v_scale[hk] : 1.f;
+      if (POS && args.sink != nullptr) {
+        // m is in units of raw scores; the sink is not scaled
+        const float sk = args.sink[head] * kLog2eTc, ms = (m == -INFINITY ? 0.f : m) * sl2, mn = fmaxf(ms, sk);
+        num *= ex2f(ms - mn);
+        l = fmaf(l, ex2f(ms - mn), ex2f(sk - mn));
+      }
+      if (POS && args.gate != nullptr && out_row < it.q_rows)
+        num *= 1.f / (1.f + __expf(-to_float(reinterpret_cast<const T*>(args.gate)[(it.q_row0 + out_row) * args.ldg + head])));
+      const float inv = l > 0.f ? num / l : 0.f;
       T* dst = reinterpret_cast<T*>(args.out) +
                (POS ? (long long)(it.q_row0 + out_row) * args.ldo + head * args.ho
                     : ((long long)(it.q_row0 + row) * args.Hq + head) * kD);
@@ -514,8 +526,8 @@ MSGL_API int msgl_latent_gather(const void* pool, void* out, const void* blk_req
 // h heads of dv channels (strides ldo, ho). dk and dv up to 128, multiples of 8 (channels up to 128 read as zero).
 MSGL_API int msgl_attn_prefill_pos(const void* q, long long ldq, long long hq_stride, const void* k, const void* vt,
                                    int t_pad, void* out, long long ldo, long long ho, const void* items, int n_items,
-                                   int total_q, int h, int dk, int dv, int window, float scale, int dtype,
-                                   cudaStream_t stream) {
+                                   int total_q, int h, int dk, int dv, int window, float scale, const void* sink,
+                                   const void* gate, long long ldg, int dtype, cudaStream_t stream) {
   if (n_items == 0 || total_q == 0) return MSGL_OK;
   if (h <= 0 || t_pad % 128 || dk % 8 || dv % 8 || dk > kD || dv > kD || ldq % 8 || hq_stride % 8 || ldo % 8 || ho % 8 ||
       (uintptr_t)q % 16 || (uintptr_t)out % 16 || scale <= 0.f || dtype != MSGL_BF16) {
@@ -545,6 +557,7 @@ MSGL_API int msgl_attn_prefill_pos(const void* q, long long ldq, long long hq_st
   cudaGetSymbolAddress((void**)&status, g_attn_tc_status);
   a.items = (const TcItem*)items; a.n_items = n_items; a.pairs = h; a.Hq = h; a.Hk = h; a.t_cap = t_pad;
   a.out = out; a.scale = scale; a.status = status; a.window = window; a.ldo = ldo; a.ho = ho; a.v_chunks = dv / 8;
+  a.sink = (const float*)sink; a.gate = gate; a.ldg = ldg;
   return launch_tc<__nv_bfloat16, true>(mq, mk, mv, a, stream);
 }
 

@@ -63,6 +63,16 @@ template <typename T> __device__ __forceinline__ void store8(T* p, const float (
   *reinterpret_cast<Vec8<T>*>(p) = v;
 }
 
+__device__ __forceinline__ void load8(const float* p, float (&out)[8]) {
+  const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
+  out[0] = a.x; out[1] = a.y; out[2] = a.z; out[3] = a.w;
+  out[4] = b.x; out[5] = b.y; out[6] = b.z; out[7] = b.w;
+}
+__device__ __forceinline__ void store8(float* p, const float (&in)[8]) {
+  *reinterpret_cast<float4*>(p) = make_float4(in[0], in[1], in[2], in[3]);
+  *reinterpret_cast<float4*>(p + 4) = make_float4(in[4], in[5], in[6], in[7]);
+}
+
 // e4m3 pair from two floats, saturating to +-448
 __device__ __forceinline__ uint16_t float2_to_e4m3x2(float a, float b) {
   return (uint16_t)__nv_cvt_float2_to_fp8x2(make_float2(a, b), __NV_SATFINITE, __NV_E4M3);

@@ -232,7 +232,7 @@ MSGL_API int msgl_rms_norm(const void* x, void* residual, const void* w, void* o
 // ------------------------------------------------------------------------------------------
 // gated activation: out[m, i] = act(x[m, i]) * x[m, I + i]
 // ------------------------------------------------------------------------------------------
-enum ActKind : int { ACT_SILU = 0, ACT_GELU = 1, ACT_GELU_TANH = 2 };
+enum ActKind : int { ACT_SILU = 0, ACT_GELU = 1, ACT_GELU_TANH = 2, ACT_CLAMPED = 3 };
 __device__ __forceinline__ float act_fn(float g, int kind) {
   if (kind == ACT_SILU) {
     // x * sigmoid(x) = h + h * tanh(h) with h = x / 2: one special-function op instead of two
@@ -247,9 +247,17 @@ __device__ __forceinline__ float act_fn(float g, int kind) {
   return 0.5f * g * (1.f + tanhf(k0 * (g + k1 * g * g * g)));
 }
 
+// g sigmoid(alpha g) (u + 1), g clamped at limit from above, u on both sides
+template <typename T> __device__ __forceinline__ float clamped_glu(float g, float u, float alpha, float limit) {
+  g = fminf(g, limit);
+  u = fminf(fmaxf(u, -limit), limit);
+  const float z = -alpha * g;
+  return g / (1.f + (sizeof(T) == 4 ? expf(z) : __expf(z))) * (u + 1.f);
+}
+
 template <typename T>
 __global__ void act_mul_kernel(const T* __restrict__ x, T* __restrict__ out, int inter, size_t total_vecs,
-                               int kind) {
+                               int kind, float alpha, float limit) {
   pdl_enter();
   size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
   if (idx >= total_vecs) return;
@@ -261,7 +269,11 @@ __global__ void act_mul_kernel(const T* __restrict__ x, T* __restrict__ out, int
   load8(g, a);
   load8(g + inter, b);
 #pragma unroll
-  for (int k = 0; k < 8; ++k) y[k] = act_fn(a[k], kind) * b[k];
+  for (int k = 0; k < 8; ++k) {
+    if (kind == ACT_CLAMPED) y[k] = clamped_glu<T>(a[k], b[k], alpha, limit);
+    else if (sizeof(T) == 4 && kind == ACT_SILU) y[k] = a[k] / (1.f + expf(-a[k])) * b[k];
+    else y[k] = act_fn(a[k], kind) * b[k];
+  }
   store8(out + row * inter + col, y);
 }
 
@@ -340,8 +352,10 @@ static int launch_act_quant(const void* x, void* out_q, void* out_scale, int row
   return MSGL_OK;
 }
 
+// alpha, limit: constants of kind 3 (clamped), which has no quantised form
 MSGL_API int msgl_act_and_mul(const void* x, void* out, void* out_q, void* out_scale, int rows, int inter,
-                              int kind, int dtype, cudaStream_t stream) {
+                              int kind, float alpha, float limit, int dtype, cudaStream_t stream) {
+  if (kind == ACT_CLAMPED && out_q != nullptr) return MSGL_BAD_ARG;
   if (inter % 8) return MSGL_BAD_ARG;
   if (rows == 0) return MSGL_OK;
   if (out_q == nullptr) {
@@ -350,9 +364,13 @@ MSGL_API int msgl_act_and_mul(const void* x, void* out, void* out_q, void* out_s
     unsigned blocks = (unsigned)((vecs + threads - 1) / threads);
     if (dtype == MSGL_BF16)
       msgl_launch(act_mul_kernel<__nv_bfloat16>, dim3(blocks), dim3(threads), 0, stream, (const __nv_bfloat16*)x, (__nv_bfloat16*)out,
-                                                                    inter, vecs, kind);
+                                                                    inter, vecs, kind, alpha, limit);
     else if (dtype == MSGL_F16)
-      msgl_launch(act_mul_kernel<__half>, dim3(blocks), dim3(threads), 0, stream, (const __half*)x, (__half*)out, inter, vecs, kind);
+      msgl_launch(act_mul_kernel<__half>, dim3(blocks), dim3(threads), 0, stream, (const __half*)x, (__half*)out, inter, vecs, kind,
+                  alpha, limit);
+    else if (dtype == MSGL_F32)
+      msgl_launch(act_mul_kernel<float>, dim3(blocks), dim3(threads), 0, stream, (const float*)x, (float*)out, inter, vecs, kind,
+                  alpha, limit);
     else
       return MSGL_BAD_ARG;
   } else {

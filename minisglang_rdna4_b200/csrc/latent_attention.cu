@@ -1,6 +1,10 @@
 // Latent attention: every query head attends to one latent row per position that is key and value
-// at once ([pages, page_size, R] of one layer of the latent pool), causal, with a sliding window.
+// at once ([pages, page_size, R] of one layer of the latent pool), causal, with a sliding window. A row may end in
+// a rotary key that all heads share (the values' projection has zeros there); a head may have a sink, a logit that
+// only the softmax denominator counts.
 //
+//   latent_rope_kernel         rotary channels of the query heads, in place, and in the same launch norm, rotation and
+//                              store of this step's latents
 //   latent_norm_store_kernel   RMS norm of this step's latents, into their pool slots (in a decode step extra CTAs
 //                              of the query projection do it)
 //   head_gemm_kernel           per-head projections into and out of the latent space (merging a split's ranges)
@@ -38,7 +42,23 @@ template <typename T> struct StoreArgs {
   int rows, rank, width;
   float eps;
   long long num_slots;
+  // a shared key behind the latent: rot_dim channels, the first rot_dims of which are rotated (0: none)
+  int rot_dim, rot_dims;
+  const float* cos_sin;   // [table_rows, rot_dims]: cosines, then sines
+  const int32_t* positions;
+  int table_rows;
 };
+
+__device__ __forceinline__ void rotate(float& u, float& v, float c, float s) {
+  const float a = u * c - v * s;
+  v = v * c + u * s;
+  u = a;
+}
+__device__ __forceinline__ int table_row(const int32_t* positions, int t, int rows) {
+  int p = positions[t];
+  (void)MSGL_OOB(p, rows);
+  return p < 0 ? 0 : (p >= rows ? rows - 1 : p);
+}
 
 // One warp per row, eight channels per lane and step (width a multiple of 64, up to 1024).
 template <typename T> __device__ __forceinline__ void store_latent(const StoreArgs<T>& a, int t, int lane) {
@@ -80,12 +100,42 @@ template <typename T> __device__ __forceinline__ void store_latent(const StoreAr
       for (int e = 0; e < 8; ++e) dst[c + e] = v[i][e];
     }
   }
+  if (a.rot_dim > 0) {
+    __syncwarp();                          // over the zeros just written
+    const float* cs = a.rot_dims > 0 ? a.cos_sin + (size_t)table_row(a.positions, t, a.table_rows) * a.rot_dims : nullptr;
+    const int half = a.rot_dims / 2;
+    for (int i = lane; 2 * i < a.rot_dim; i += 32) {
+      float x = to_float(src[a.rank + 2 * i]), y = 2 * i + 1 < a.rot_dim ? to_float(src[a.rank + 2 * i + 1]) : 0.f;
+      if (i < half) rotate(x, y, cs[i], cs[half + i]);
+      dst[a.rank + 2 * i] = from_float<T>(x);
+      if (2 * i + 1 < a.rot_dim) dst[a.rank + 2 * i + 1] = from_float<T>(y);
+    }
+  }
 }
 
 template <typename T> __global__ void __launch_bounds__(128) latent_norm_store_kernel(const StoreArgs<T> a) {
   pdl_enter();
   const int t = blockIdx.x * 4 + (threadIdx.x >> 5);
   if (t < a.rows) store_latent(a, t, threadIdx.x & 31);
+}
+
+// CTA per row: the warps rotate the query heads' pairs; warp 0 stores the row's latent first (store.c != null).
+template <typename T>
+__global__ void __launch_bounds__(128) latent_rope_kernel(T* __restrict__ q, long long ldq, long long hq, int H, int first,
+                                                          int dims, const StoreArgs<T> a) {
+  pdl_enter();
+  const int t = blockIdx.x;
+  if (a.c != nullptr && threadIdx.x < 32) store_latent(a, t, threadIdx.x);
+  const float* cs = a.cos_sin + (size_t)table_row(a.positions, t, a.table_rows) * dims;
+  const int half = dims / 2;
+  for (int id = threadIdx.x; id < H * half; id += 128) {
+    const int h = id / half, i = id - h * half;
+    T* p = q + t * ldq + h * hq + first + 2 * i;
+    float x = to_float(p[0]), y = to_float(p[1]);
+    rotate(x, y, cs[i], cs[half + i]);
+    p[0] = from_float<T>(x);
+    p[1] = from_float<T>(y);
+  }
 }
 
 // ------------------------------------------------------------------------------------------ attention args
@@ -101,6 +151,7 @@ struct LatArgs {
   float* ws_lse;          // [splits, T * H]
   int H, page_size, page_shift, num_pages, window, splits, total_rows;   // num_pages includes the scratch page
   float scale;
+  const float* sink;      // [H] or null
 };
 
 __device__ __forceinline__ long long token_slot(const LatArgs& a, const int32_t* bt, int tok) {
@@ -137,7 +188,7 @@ __global__ void __launch_bounds__(128) latent_attention_simt_kernel(const LatArg
     qr[i] = c < R ? to_float(q[c]) * a.scale : 0.f;
     o[i] = 0.f;
   }
-  float m = -INFINITY, l = 0.f;
+  float m = a.sink != nullptr ? a.sink[row % a.H] : -INFINITY, l = a.sink != nullptr ? 1.f : 0.f;
   for (int tok = lo; tok <= pos; ++tok) {
     const T* k = pool + token_slot(a, bt, tok) * R;
     float kr[NR], s = 0.f;
@@ -208,6 +259,8 @@ struct HeadGemmArgs {
   const float* ws_o;      // [splits, T * H, K]
   const float* ws_lse;    // [splits, T * H]
   int splits, H;
+  const __nv_bfloat16* gate;        // [T, ...] logits of the heads' output gates with row stride ldg, or null
+  long long ldg;
   StoreArgs<__nv_bfloat16> store;   // store.c != null: the CTAs at blockIdx.y >= H store the step's latents
 };
 
@@ -306,6 +359,15 @@ __global__ void __launch_bounds__(128) head_gemm_kernel(const HeadGemmArgs a) {
   }
   const int r = t0 + warp * 16 + (lane >> 2), col = n0 + (lane & 3) * 2;
   __nv_bfloat16* o = a.out + (long long)h * a.ho;
+  if (a.gate != nullptr) {
+    const float g0 = r < a.T ? 1.f / (1.f + __expf(-to_float(a.gate[(long long)r * a.ldg + h]))) : 0.f;
+    const float g1 = r + 8 < a.T ? 1.f / (1.f + __expf(-to_float(a.gate[(long long)(r + 8) * a.ldg + h]))) : 0.f;
+#pragma unroll
+    for (int nb = 0; nb < 8; ++nb) {
+      acc[nb][0] *= g0; acc[nb][1] *= g0;
+      acc[nb][2] *= g1; acc[nb][3] *= g1;
+    }
+  }
 #pragma unroll
   for (int nb = 0; nb < 8; ++nb) {
     const int n = col + nb * 8;
@@ -559,7 +621,18 @@ __global__ void __launch_bounds__(32 * WM * WN) latent_attention_kernel(const La
     l_a += red[w * MT + ra];
     l_b += red[w * MT + rb];
   }
-  const float inv_a = l_a > 0.f ? 1.f / l_a : 0.f, inv_b = l_b > 0.f ? 1.f / l_b : 0.f;
+  float num_a = 1.f, num_b = 1.f;
+  if (a.sink != nullptr && split == 0) {         // counted once, by the first key range
+    auto add_sink = [&](int r, float& m, float& l, float& num) {
+      const float sk = a.sink[min(row0 + r, row1 - 1) % a.H] * kLog2eL, mn = fmaxf(m, sk);
+      num = ex2(m - mn);                         // m = -inf: no key in this range
+      l = fmaf(l, num, ex2(sk - mn));
+      m = mn;
+    };
+    add_sink(ra, m_a, l_a, num_a);
+    add_sink(rb, m_b, l_b, num_b);
+  }
+  const float inv_a = l_a > 0.f ? num_a / l_a : 0.f, inv_b = l_b > 0.f ? num_b / l_b : 0.f;
   const size_t row_base = (size_t)q0 * a.H + row0;
   const bool ok_a = row0 + ra < row1, ok_b = row0 + rb < row1;
   const int col = wn * (R / WN) + (lane & 3) * 2;
@@ -585,7 +658,7 @@ __global__ void __launch_bounds__(32 * WM * WN) latent_attention_kernel(const La
   }
 }
 
-// One warp per (row, head); R a multiple of 64, up to 512 (four float4 per lane).
+// One warp per (row, head); R a multiple of 64, up to 640 (five float4 per lane).
 __global__ void __launch_bounds__(128) latent_combine_kernel(const float* __restrict__ ws_o,
                                                              const float* __restrict__ ws_lse,
                                                              __nv_bfloat16* __restrict__ out, int rows, int R,
@@ -594,11 +667,11 @@ __global__ void __launch_bounds__(128) latent_combine_kernel(const float* __rest
   const int row = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
   if (row >= rows) return;
   const float lse = lane < splits ? ws_lse[(size_t)lane * rows + row] : -INFINITY;    // splits <= 16
-  float acc[4][4] = {};
-  float4 v[4];
+  float acc[5][4] = {};
+  float4 v[5];
   auto fetch = [&](int s) {
 #pragma unroll
-    for (int i = 0; i < 4; ++i) {
+    for (int i = 0; i < 5; ++i) {
       const int c = lane * 4 + i * 128;
       v[i] = c < R ? *reinterpret_cast<const float4*>(ws_o + ((size_t)s * rows + row) * R + c)
                    : make_float4(0.f, 0.f, 0.f, 0.f);
@@ -613,7 +686,7 @@ __global__ void __launch_bounds__(128) latent_combine_kernel(const float* __rest
     fetch(s);
     const float f = __shfl_sync(0xffffffffu, w, s);
 #pragma unroll
-    for (int i = 0; i < 4; ++i) {
+    for (int i = 0; i < 5; ++i) {
       acc[i][0] = fmaf(f, v[i].x, acc[i][0]);
       acc[i][1] = fmaf(f, v[i].y, acc[i][1]);
       acc[i][2] = fmaf(f, v[i].z, acc[i][2]);
@@ -621,7 +694,7 @@ __global__ void __launch_bounds__(128) latent_combine_kernel(const float* __rest
     }
   }
 #pragma unroll
-  for (int i = 0; i < 4; ++i) {
+  for (int i = 0; i < 5; ++i) {
     const int c = lane * 4 + i * 128;
     if (c < R)
       *reinterpret_cast<uint2*>(out + (size_t)row * R + c) =
@@ -653,7 +726,10 @@ int launch_latent(const LatArgs& a, int B, int max_q, cudaStream_t s) {
 template <int NP>
 int launch_latent_rows(const LatArgs& a, int B, int max_q, bool one_form, cudaStream_t s) {
   const long long rows = one_form ? 64 : (long long)max_q * a.H;
-  if constexpr (NP > 4) {                  // a wide latent leaves room for one CTA per SM: sixteen warps of it
+  if constexpr (NP > 8) {                  // 64 rows of queries would not fit beside two tiles
+    if (rows <= 16) return launch_latent<NP, 1, 8, 2>(a, B, max_q, s);
+    return launch_latent<NP, 2, 8, 2>(a, B, max_q, s);
+  } else if constexpr (NP > 4) {                  // a wide latent leaves room for one CTA per SM: sixteen warps of it
     if (rows <= 16) return launch_latent<NP, 1, 8, 2>(a, B, max_q, s);
     if (rows <= 32) return launch_latent<NP, 2, 8, 2>(a, B, max_q, s);
     return launch_latent<NP, 4, 4, 1>(a, B, max_q, s);
@@ -689,7 +765,7 @@ MSGL_API int msgl_latent_norm_store(const void* c, long long ldc, const void* we
 #define STORE(T)                                                                                                    \
   msgl_launch(latent_norm_store_kernel<T>, grid, dim3(128), 0, stream,                                              \
               StoreArgs<T>{(const T*)c, ldc, (const float*)weight, (T*)pool, (const int32_t*)out_loc, rows, rank,   \
-                           width, eps, num_slots})
+                           width, eps, num_slots, 0, 0, nullptr, nullptr, 0})
   if (dtype == MSGL_BF16) STORE(__nv_bfloat16);
   else if (dtype == MSGL_F32) STORE(float);
   else return MSGL_BAD_ARG;
@@ -698,9 +774,34 @@ MSGL_API int msgl_latent_norm_store(const void* c, long long ldc, const void* we
   return MSGL_OK;
 }
 
+// q [rows, H, ...] (element strides ldq, hq): channels first .. first + dims of every head are rotated in place by
+// cos_sin [table_rows, dims] at positions [rows]. c != null: the rows' latents (and rot_dim channels of shared key behind
+// them) are normed, rotated and stored as in msgl_latent_norm_store.
+MSGL_API int msgl_latent_rope(void* q, long long ldq, long long hq, int H, int first, int dims, const void* cos_sin,
+                              const void* positions, int table_rows, const void* c, long long ldc, const void* weight,
+                              void* pool, const void* out_loc, int rows, int rank, int width, int rot_dim, float eps,
+                              long long num_slots, int dtype, cudaStream_t stream) {
+  if (rows <= 0) return rows == 0 ? MSGL_OK : MSGL_BAD_ARG;
+  if (H <= 0 || dims <= 0 || dims % 2 || first < 0 || table_rows <= 0) return MSGL_BAD_ARG;
+  if (c != nullptr && (rank <= 0 || rot_dim < dims || rank + rot_dim > width || width % 64 || width > 1024 || ldc % 8 ||
+                       (uintptr_t)c % 16 || (uintptr_t)pool % 16))
+    return MSGL_BAD_ARG;
+#define ROPE(T)                                                                                                     \
+  msgl_launch(latent_rope_kernel<T>, dim3(rows), dim3(128), 0, stream, (T*)q, ldq, hq, H, first, dims,              \
+              StoreArgs<T>{(const T*)c, ldc, (const float*)weight, (T*)pool, (const int32_t*)out_loc, rows, rank,   \
+                           width, eps, num_slots, rot_dim, dims, (const float*)cos_sin, (const int32_t*)positions,  \
+                           table_rows})
+  if (dtype == MSGL_BF16) ROPE(__nv_bfloat16);
+  else if (dtype == MSGL_F32) ROPE(float);
+  else return MSGL_BAD_ARG;
+#undef ROPE
+  MSGL_CHECK_LAUNCH("latent_rope");
+  return MSGL_OK;
+}
+
 MSGL_API int msgl_head_gemm(const void* x, long long ldx, long long hx, const void* w, void* out, long long ldo,
                             long long ho, int T, int H, int N, int K, int static_weights, const void* ws_o, const void* ws_lse,
-                            int splits, const void* c, long long ldc, const void* norm, void* pool,
+                            int splits, const void* gate, long long ldg, const void* c, long long ldc, const void* norm, void* pool,
                             const void* out_loc, int rank, int width, float eps, long long num_slots,
                             cudaStream_t stream) {
   if (T <= 0) return T == 0 ? MSGL_OK : MSGL_BAD_ARG;
@@ -708,9 +809,10 @@ MSGL_API int msgl_head_gemm(const void* x, long long ldx, long long hx, const vo
       (uintptr_t)w % 16 || (uintptr_t)out % 4 || T > 65535 * 64)
     return MSGL_BAD_ARG;
   HeadGemmArgs a{(const __nv_bfloat16*)x, ldx, hx, (const __nv_bfloat16*)w, (__nv_bfloat16*)out, ldo, ho, T, N, K,
-                 static_weights, (const float*)ws_o, (const float*)ws_lse, splits, H,
+                 static_weights, (const float*)ws_o, (const float*)ws_lse, splits, H, (const __nv_bfloat16*)gate, ldg,
                  StoreArgs<__nv_bfloat16>{(const __nv_bfloat16*)c, ldc, (const float*)norm, (__nv_bfloat16*)pool,
-                                          (const int32_t*)out_loc, T, rank, width, eps, num_slots}};
+                                          (const int32_t*)out_loc, T, rank, width, eps, num_slots, 0, 0, nullptr, nullptr,
+                                          0}};
   if (c != nullptr && (rank <= 0 || rank > width || width % 64 || width > 1024 || ldc % 8 || (uintptr_t)c % 16 ||
                        (uintptr_t)pool % 16 || H > 65000))
     return MSGL_BAD_ARG;
@@ -731,7 +833,7 @@ MSGL_API int msgl_head_gemm(const void* x, long long ldx, long long hx, const vo
 MSGL_API int msgl_latent_attention(const void* q, const void* pool, void* out, const void* block_table, int bt_stride,
                                    const void* cu_q, const void* seq_lens, void* ws_o, void* ws_lse, int B, int total_q,
                                    int max_q, int H, int R, int page_size, int num_pages, int window, int splits,
-                                   float scale, int one_form, int dtype, cudaStream_t stream) {
+                                   float scale, const void* sink, int one_form, int dtype, cudaStream_t stream) {
   if (B <= 0 || total_q <= 0) return B == 0 || total_q == 0 ? MSGL_OK : MSGL_BAD_ARG;
   if (max_q <= 0 || H <= 0 || R % 64 || page_size <= 0 || num_pages <= 0 || B > 65535 || splits < 1 || bt_stride < 1 ||
       splits > kMaxSplits || (uintptr_t)q % 16 || (uintptr_t)pool % 16 || (uintptr_t)out % 16 || (out == nullptr && splits == 1))
@@ -740,10 +842,11 @@ MSGL_API int msgl_latent_attention(const void* q, const void* pool, void* out, c
   for (int i = 0; i < 31; ++i)
     if ((1 << i) == page_size) shift = i;
   LatArgs a{q, pool, out, (const int32_t*)block_table, bt_stride, (const int32_t*)cu_q, (const int32_t*)seq_lens,
-            (float*)ws_o, (float*)ws_lse, H, page_size, shift, num_pages, window, splits, total_q * H, scale};
+            (float*)ws_o, (float*)ws_lse, H, page_size, shift, num_pages, window, splits, total_q * H, scale,
+            (const float*)sink};
   if (dtype == MSGL_F32) return launch_simt<float>(a, R, B, max_q, stream);
   if (dtype != MSGL_BF16) return MSGL_BAD_ARG;
-  if (R > 512) {
+  if (R > 512 && R != 576) {
     a.splits = 1;
     if (splits > 1) return MSGL_BAD_ARG;
     return launch_simt<__nv_bfloat16>(a, R, B, max_q, stream);
@@ -756,6 +859,7 @@ MSGL_API int msgl_latent_attention(const void* q, const void* pool, void* out, c
     case 3: rc = launch_latent_rows<3>(a, B, max_q, one_form != 0, stream); break;
     case 4: rc = launch_latent_rows<4>(a, B, max_q, one_form != 0, stream); break;
     case 8: rc = launch_latent_rows<8>(a, B, max_q, one_form != 0, stream); break;
+    case 9: rc = launch_latent_rows<9>(a, B, max_q, one_form != 0, stream); break;
     default: return MSGL_BAD_ARG;
   }
   // without a destination the ranges stay apart: the projection out of the latent space merges them

@@ -10,6 +10,8 @@
 //   moe_permute    : gather token rows into expert-sorted order
 //   moe_combine    : out[t] = sum_k w[t,k] * y[row_of(t,k)] in a fixed k order
 //                    (mmq_fp8_moe_gather_reduce, python/minisgl/quant/kernels.py:877)
+//   moe_combine32  : the same sum in fp32 for an fp32 residual stream, with a shared expert's
+//                    output behind a sigmoid gate per token
 //
 // Shapes are static for CUDA graphs: the sorted buffers are sized for the worst case
 // T*k + E*127 rows and tiles past the live count carry expert id -1, which the GEMM skips.
@@ -27,7 +29,7 @@ template <typename T>
 __global__ void moe_route_kernel(const T* __restrict__ logits, const float* __restrict__ bias,
                                  float* __restrict__ topk_w, int32_t* __restrict__ topk_ids,
                                  int32_t* __restrict__ counts, int tokens, int E, int k, int renorm, int sigmoid,
-                                 float scale, int e_start, int e_local) {
+                                 float scale, int e_start, int e_local, long long ld, int groups, int keep) {
   pdl_enter();
   const int t = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
   if (t >= tokens) return;
@@ -38,7 +40,7 @@ __global__ void moe_route_kernel(const T* __restrict__ logits, const float* __re
 #pragma unroll
   for (int i = 0; i < PER; ++i) {
     const int e = lane + 32 * i;
-    v[i] = e < E ? to_float(logits[(size_t)t * E + e]) : -INFINITY;
+    v[i] = e < E ? to_float(logits[t * ld + e]) : -INFINITY;
     mx = fmaxf(mx, v[i]);
   }
   if (sigmoid) {
@@ -63,6 +65,37 @@ __global__ void moe_route_kernel(const T* __restrict__ logits, const float* __re
   for (int i = 0; i < PER; ++i) {
     const int e = lane + 32 * i;
     c[i] = (bias != nullptr && e < E) ? v[i] + bias[e] : v[i];
+  }
+  if (groups > 1) {
+    // only experts of the best `keep` groups stay eligible; a group's score is its best member's
+    const int size = E / groups;
+    float g0 = -INFINITY, g1 = -INFINITY;      // lane l holds the groups l and l + 32
+    for (int g = 0; g < groups; ++g) {
+      float best = -INFINITY;
+#pragma unroll
+      for (int i = 0; i < PER; ++i)
+        if ((lane + 32 * i) / size == g) best = fmaxf(best, c[i]);
+      best = warp_max(best);
+      if (lane == (g & 31)) (g < 32 ? g0 : g1) = best;
+    }
+    unsigned long long open = 0;
+    for (int kk = 0; kk < keep; ++kk) {
+      float best = g0 >= g1 ? g0 : g1;
+      int bi = g0 >= g1 ? lane : lane + 32;
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) {
+        const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+        const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
+        if (ob > best || (ob == best && oi < bi)) { best = ob; bi = oi; }
+      }
+      open |= 1ull << bi;
+      if ((bi & 31) == lane) (bi < 32 ? g0 : g1) = -INFINITY;
+    }
+#pragma unroll
+    for (int i = 0; i < PER; ++i) {
+      const int e = lane + 32 * i;
+      if (e < E && !(open >> (e / size) & 1)) c[i] = -INFINITY;
+    }
   }
   float wsel[kMaxTopK];
   int isel[kMaxTopK];
@@ -194,12 +227,68 @@ __global__ void moe_combine_kernel(const T* __restrict__ y, const float* __restr
   }
 }
 
+// out [tokens, cols] fp32; shared [tokens, shared_cols] (columns past that: no shared part), shared_gate: one logit
+// per token, ldg elements apart
+template <typename T>
+__global__ void __launch_bounds__(256) moe_combine32_kernel(const T* __restrict__ y, const float* __restrict__ topk_w,
+                                                            const int32_t* __restrict__ pair_row,
+                                                            const T* __restrict__ shared, int shared_cols,
+                                                            const float* __restrict__ shared_gate, long long ldg,
+                                                            float* __restrict__ out, int cols, int k) {
+  pdl_enter();
+  const int t = blockIdx.x;
+  const float sg = shared != nullptr ? 1.f / (1.f + expf(-shared_gate[t * ldg])) : 0.f;
+  for (int i = threadIdx.x * 8; i < cols; i += blockDim.x * 8) {
+    float acc[8], v[8];
+#pragma unroll
+    for (int e = 0; e < 8; ++e) acc[e] = 0.f;
+    if (shared != nullptr && i < shared_cols) {
+      load8(shared + (size_t)t * shared_cols + i, v);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) acc[e] = sg * v[e];
+    }
+    for (int kk = 0; kk < k; ++kk) {
+      const int row = pair_row[(size_t)t * k + kk];
+      if (row < 0) continue;
+      const float w = topk_w[(size_t)t * k + kk];
+      load8(y + (size_t)row * cols + i, v);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) acc[e] = fmaf(w, v[e], acc[e]);
+    }
+    store8(out + (size_t)t * cols + i, acc);
+  }
+}
+
 }  // namespace
 
+MSGL_API int msgl_moe_combine32(const void* y, const void* topk_w, const void* pair_row, const void* shared,
+                                int shared_cols, const void* shared_gate, long long ldg, void* out, int tokens, int cols,
+                                int k, int dtype, cudaStream_t stream) {
+  if (tokens == 0) return MSGL_OK;
+  if (tokens < 0 || cols % 8 || shared_cols % 8 || (shared != nullptr && shared_gate == nullptr)) return MSGL_BAD_ARG;
+  const int threads = cols / 8 < 256 ? ((cols / 8 + 31) / 32) * 32 : 256;
+#define COMBINE32(T)                                                                                                 \
+  msgl_launch(moe_combine32_kernel<T>, dim3(tokens), dim3(threads), 0, stream, (const T*)y, (const float*)topk_w,    \
+              (const int32_t*)pair_row, (const T*)shared, shared_cols, (const float*)shared_gate, ldg, (float*)out,  \
+              cols, k)
+  if (dtype == MSGL_BF16) COMBINE32(__nv_bfloat16);
+  else if (dtype == MSGL_F32) COMBINE32(float);
+  else return MSGL_BAD_ARG;
+#undef COMBINE32
+  MSGL_CHECK_LAUNCH("moe_combine32");
+  return MSGL_OK;
+}
+
+// logits [tokens, E] with row stride ld. groups > 1: experts are chosen among the best `keep` of that many groups of
+// neighbours, a group scoring as its best member (up to 64 groups)
 MSGL_API int msgl_moe_route(const void* logits, const void* bias, void* topk_w, void* topk_ids, void* counts,
                             int tokens, int E, int k, int renorm, int sigmoid, float scale, int e_start, int e_local,
-                            int dtype, cudaStream_t stream) {
-  if (E > kMaxExperts || k > kMaxTopK || k > E) return MSGL_BAD_ARG;
+                            long long ld, int groups, int keep, int dtype, cudaStream_t stream) {
+  if (E > kMaxExperts || k > kMaxTopK || k > E) {
+    msgl_set_error_text("moe_route: up to 512 experts, 16 per token");
+    return MSGL_BAD_ARG;
+  }
+  if (groups > 1 && (groups > 64 || E % groups || keep <= 0 || keep > groups || k > E / groups * keep)) return MSGL_BAD_ARG;
   // counts (optional): tokens per local expert, for the alignment step; zeroed here
   if (counts != nullptr) cudaMemsetAsync(counts, 0, sizeof(int32_t) * e_local, stream);
   if (tokens == 0) return MSGL_OK;
@@ -208,7 +297,7 @@ MSGL_API int msgl_moe_route(const void* logits, const void* bias, void* topk_w, 
 #define ROUTE(T)                                                                                                   \
   msgl_launch(moe_route_kernel<T>, dim3(blocks), dim3(warps * 32), 0, stream, (const T*)logits, (const float*)bias, \
               (float*)topk_w, (int32_t*)topk_ids, (int32_t*)counts, tokens, E, k, renorm, sigmoid, scale, e_start,   \
-              e_local)
+              e_local, ld, groups, keep)
   if (dtype == MSGL_F32) ROUTE(float);
   else if (dtype == MSGL_BF16) ROUTE(__nv_bfloat16);
   else if (dtype == MSGL_F16) ROUTE(__half);

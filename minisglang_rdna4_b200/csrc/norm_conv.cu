@@ -15,7 +15,7 @@ __global__ void __launch_bounds__(256) embed_positions_kernel(const int32_t* __r
                                                               const T* __restrict__ pos,
                                                               const int32_t* __restrict__ positions,
                                                               float* __restrict__ out, int width, int start, int len,
-                                                              int n_pos) {
+                                                              int n_pos, float scale) {
   pdl_enter();
   const int t = blockIdx.x;
   const int id = ids[t] - start;
@@ -23,7 +23,7 @@ __global__ void __launch_bounds__(256) embed_positions_kernel(const int32_t* __r
   int p = pos != nullptr ? positions[t] : 0;
   const bool has_pos = pos != nullptr && !MSGL_OOB(p, n_pos) && p >= 0 && p < n_pos;
   for (int c = threadIdx.x; c < width; c += 256) {
-    float v = in ? to_float(w[(size_t)id * width + c]) : 0.f;
+    float v = in ? to_float(w[(size_t)id * width + c]) * scale : 0.f;
     if (has_pos) v += to_float(pos[(size_t)p * width + c]);
     out[(size_t)t * width + c] = v;
   }
@@ -459,11 +459,12 @@ __global__ void __launch_bounds__(256) gelu_erf_kernel(const T* __restrict__ x, 
 }  // namespace
 
 MSGL_API int msgl_embed_positions(const void* ids, const void* w, const void* pos, const void* positions, void* out,
-                                  int rows, int width, int start, int len, int n_pos, int dtype, cudaStream_t stream) {
+                                  int rows, int width, int start, int len, int n_pos, float scale, int dtype,
+                                  cudaStream_t stream) {
   if (rows <= 0) return rows == 0 ? MSGL_OK : MSGL_BAD_ARG;
 #define EMB(T)                                                                                                      \
   msgl_launch(embed_positions_kernel<T>, dim3(rows), dim3(256), 0, stream, (const int32_t*)ids, (const T*)w,        \
-              (const T*)pos, (const int32_t*)positions, (float*)out, width, start, len, n_pos)
+              (const T*)pos, (const int32_t*)positions, (float*)out, width, start, len, n_pos, scale)
   if (dtype == MSGL_BF16) EMB(__nv_bfloat16);
   else if (dtype == MSGL_F32) EMB(float);
   else return MSGL_BAD_ARG;

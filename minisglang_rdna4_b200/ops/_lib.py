@@ -42,7 +42,7 @@ _SIGNATURES = {
     "msgl_last_error": (ctypes.c_char_p, []),
     "msgl_embedding": (c_i, [c_p, c_p, c_p, c_i, c_i, c_i, c_i, c_p]),
     "msgl_rms_norm": (c_i, [c_p, c_p, c_p, c_p, c_p, c_p, c_i, c_i, c_f, c_i, c_i, c_p]),
-    "msgl_act_and_mul": (c_i, [c_p, c_p, c_p, c_p, c_i, c_i, c_i, c_i, c_p]),
+    "msgl_act_and_mul": (c_i, [c_p, c_p, c_p, c_p, c_i, c_i, c_i, c_f, c_f, c_i, c_p]),
     "msgl_quant_fp8": (c_i, [c_p, c_p, c_p, c_i, c_i, c_i, c_i, c_p]),
     "msgl_qk_norm_rope_store": (c_i, [c_p] * 11 + [c_i, c_i, c_i, c_i, c_i, c_i, c_f, c_i, c_i, c_i, c_i, c_i, c_p]),
     "msgl_store_kv": (c_i, [c_p] * 7 + [c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_p]),

@@ -176,15 +176,16 @@ def per_group_quant_fp8(x, group):
     return q, s
 
 
-_ACT = {"silu": 0, "gelu": 1, "gelu_tanh": 2}
+_ACT = {"silu": 0, "gelu": 1, "gelu_tanh": 2, "clamped": 3}
 
 
-def act_and_mul(x, kind="silu"):
+def act_and_mul(x, kind="silu", alpha=0.0, limit=0.0):
+    """``act(gate) * up`` of rows ``[gate, up]``; ``clamped``: ``g sigmoid(alpha g) (u + 1)`` within ``limit``."""
     assert x.is_contiguous() and x.dim() == 2
     rows, two_i = x.shape
     out = torch.empty((rows, two_i // 2), dtype=x.dtype, device=x.device)
-    check(lib().msgl_act_and_mul(_p(x), _p(out), None, None, rows, two_i // 2, _ACT[kind], _dt(x), _stream()),
-          "act_and_mul")
+    check(lib().msgl_act_and_mul(_p(x), _p(out), None, None, rows, two_i // 2, _ACT[kind], alpha, limit, _dt(x),
+                                 _stream()), "act_and_mul")
     _count("act_and_mul", "act_mul_kernel")
     return out
 
@@ -194,7 +195,7 @@ def silu_and_mul_quant(x):
     rows, two_i = x.shape
     q = torch.empty((rows, two_i // 2), dtype=torch.float8_e4m3fn, device=x.device)
     s = torch.empty((rows,), dtype=torch.float32, device=x.device)
-    check(lib().msgl_act_and_mul(_p(x), None, _p(q), _p(s), rows, two_i // 2, 0, _dt(x), _stream()),
+    check(lib().msgl_act_and_mul(_p(x), None, _p(q), _p(s), rows, two_i // 2, 0, 0.0, 0.0, _dt(x), _stream()),
           "silu_and_mul_quant")
     _count("silu_and_mul_quant", "act_mul_quant_kernel")
     return q, s
@@ -907,17 +908,19 @@ def _bind_latent():
 
     if hasattr(_bind_latent, "_done"):
         return
-    bind("msgl_gemm_f32", c_i, [c_p, c_ll, c_ll, c_p, c_ll, c_ll, c_p, c_ll, c_ll, c_i, c_i, c_i, c_i, c_p])
-    bind("msgl_embed_positions", c_i, [c_p] * 5 + [c_i] * 6 + [c_p])
+    bind("msgl_gemm_f32", c_i, [c_p, c_ll, c_ll, c_p, c_ll, c_ll, c_p, c_ll, c_ll, c_i, c_i, c_i, c_i, c_p, c_ll, c_p])
+    bind("msgl_embed_positions", c_i, [c_p] * 5 + [c_i] * 5 + [c_f, c_i, c_p])
+    bind("msgl_latent_rope", c_i, [c_p, c_ll, c_ll, c_i, c_i, c_i, c_p, c_p, c_i, c_p, c_ll, c_p, c_p, c_p] + [c_i] * 4
+         + [c_f, c_ll, c_i, c_p])
     bind("msgl_norm_conv", c_i, [c_p, c_p, c_p, c_i, c_ll, c_ll, c_p, c_f] + [c_p] * 9 + [c_i] * 7 + [c_p])
     bind("msgl_gelu_erf", c_i, [c_p, c_ll, c_p, c_ll, c_i, c_i, c_i, c_p])
     bind("msgl_latent_norm_store", c_i, [c_p, c_ll, c_p, c_p, c_p, c_i, c_i, c_i, c_f, c_ll, c_i, c_p])
     bind("msgl_head_gemm", c_i, [c_p, c_ll, c_ll, c_p, c_p, c_ll, c_ll, c_i, c_i, c_i, c_i, c_i, c_p, c_p, c_i,
-                                 c_p, c_ll, c_p, c_p, c_p, c_i, c_i, c_f, c_ll, c_p])
+                                 c_p, c_ll, c_p, c_ll, c_p, c_p, c_p, c_i, c_i, c_f, c_ll, c_p])
     bind("msgl_latent_gather", c_i, [c_p] * 5 + [c_i] * 5 + [c_p])
     bind("msgl_attn_prefill_pos", c_i, [c_p, c_ll, c_ll, c_p, c_p, c_i, c_p, c_ll, c_ll, c_p, c_i, c_i, c_i, c_i, c_i, c_i,
-                                        c_f, c_i, c_p])
-    bind("msgl_latent_attention", c_i, [c_p, c_p, c_p, c_p, c_i] + [c_p] * 4 + [c_i] * 9 + [c_f, c_i, c_i, c_p])
+                                        c_f, c_p, c_p, c_ll, c_i, c_p])
+    bind("msgl_latent_attention", c_i, [c_p, c_p, c_p, c_p, c_i] + [c_p] * 4 + [c_i] * 9 + [c_f, c_p, c_i, c_i, c_p])
     _bind_latent._done = True
 
 
@@ -927,19 +930,19 @@ def gemm_f32(x, w):
     assert x.dim() == 2 and x.stride(1) == 1 and w.is_contiguous() and w.shape[1] == x.shape[1]
     out = torch.empty((x.shape[0], w.shape[0]), dtype=torch.float32, device=x.device)
     check(lib().msgl_gemm_f32(_p(x), x.stride(0), 0, _p(w), w.stride(0), 0, _p(out), out.stride(0), 0, x.shape[0],
-                              w.shape[0], w.shape[1], 1, _stream()), "gemm_f32")
+                              w.shape[0], w.shape[1], 1, None, 0, _stream()), "gemm_f32")
     _count("gemm_f32", "gemm_f32_kernel")
     return out
 
 
 # ------------------------------------------------------------------------------------------ fp32 residual, input convolutions
-def embed_positions(ids, weight, pos, positions, vocab_start=0, vocab_len=None):
+def embed_positions(ids, weight, pos, positions, vocab_start=0, vocab_len=None, scale=1.0):
     _bind_latent()
     ids = ids.to(torch.int32) if ids.dtype != torch.int32 else ids
     n = weight.shape[0] if vocab_len is None else vocab_len
     out = torch.empty((ids.numel(), weight.shape[1]), dtype=torch.float32, device=weight.device)
     check(lib().msgl_embed_positions(_p(ids), _p(weight), _p(pos), _p(positions), _p(out), ids.numel(), weight.shape[1],
-                                     vocab_start, n, 0 if pos is None else pos.shape[0], _dt(weight), _stream()),
+                                     vocab_start, n, 0 if pos is None else pos.shape[0], scale, _dt(weight), _stream()),
           "embed_positions")
     _count("embed_positions", "embed_positions_kernel")
     return out
@@ -983,6 +986,77 @@ def gelu_erf(x, out):
     return out
 
 
+# ------------------------------------------------------------------------------------------ weighted norm, linear attention
+def _bind_linear():
+    from ._lib import bind, c_f, c_i, c_ll, c_p
+
+    if hasattr(_bind_linear, "_done"):
+        return
+    bind("msgl_add_norm", c_i, [c_p, c_p, c_p, c_i, c_ll, c_ll, c_p, c_p, c_i, c_i, c_i, c_f, c_i, c_i, c_p])
+    bind("msgl_linear_attention", c_i, [c_p, c_p, c_p, c_ll, c_p, c_ll] + [c_p] * 8 + [c_i] * 7 + [c_f, c_f, c_i, c_i, c_p])
+    bind("msgl_norm_gate", c_i, [c_p, c_p, c_ll, c_p, c_p, c_p, c_ll, c_i, c_i, c_f, c_f, c_i, c_i, c_p])
+    _bind_linear._done = True
+
+
+def add_norm(x, delta, weight, eps, center, out_dtype, out_cols):
+    _bind_linear()
+    assert x.is_contiguous() and x.dtype == torch.float32 and weight.dtype == torch.float32
+    rows, width = x.shape
+    planes, plane_stride, ldd = 0, 0, 0
+    if isinstance(delta, SplitPartial):
+        delta = delta.planes
+        planes, plane_stride, ldd = delta.shape[0], delta.stride(0), delta.stride(1)
+    elif delta is not None:
+        planes, ldd = 1, delta.stride(0)
+    if delta is not None:
+        assert delta.dtype == torch.float32 and delta.stride(-1) == 1 and delta.shape[-2] == rows and delta.shape[-1] >= width
+    x_out = torch.empty_like(x) if delta is not None else x
+    y = torch.empty((rows, out_cols), dtype=out_dtype, device=x.device)
+    check(lib().msgl_add_norm(_p(x), _p(x_out), _p(delta), planes, plane_stride, ldd, _p(weight), _p(y), rows, width,
+                              out_cols, eps, int(center), _DT[out_dtype], _stream()), "add_norm")
+    _count("add_norm", "add_norm_kernel")
+    return x_out, y
+
+
+def linear_attention(q, k, v, state, cu_q, slots, has_state, decay=None, gate=None, tau=1.0, q_scale=1.0, act=False,
+                     chunked=False):
+    """See ``ref.linear_attention``; ``q``, ``k``, ``v`` and the low-rank input are views of the same projected rows, head
+    widths multiples of 16. ``chunked``: the tensor-core form where it covers the sizes (16-bit prompts)."""
+    _bind_linear()
+    t, h, dk = q.shape
+    dv = v.shape[2]
+    ld = q.stride(0)
+    low, up, bias = gate if gate is not None else (None, None, None)
+    for x, n in ((q, dk), (k, dk), (v, dv)):
+        assert x.stride(2) == 1 and (h == 1 or x.stride(1) == n) and (t == 1 or x.stride(0) == ld) and x.dtype == q.dtype
+    assert state.dtype == torch.float32 and state.shape[1:] == (h, dk, dv) and (state.shape[0] == 1 or state[0].is_contiguous())
+    if gate is not None:
+        assert (t == 1 or low.stride(0) == ld) and low.stride(-1) == 1 and up.is_contiguous() and up.dtype == low.dtype == q.dtype
+        assert bias.dtype == torch.float32 and up.shape == (h * dk, low.shape[1])
+    out = torch.empty((t, h, dv), dtype=q.dtype, device=q.device)
+    check(lib().msgl_linear_attention(
+        _p(q), _p(k), _p(v), ld, _p(state), state.stride(0), _p(cu_q), _p(slots), _p(has_state), _p(out), _p(decay), _p(low),
+        _p(up), _p(bias), cu_q.numel() - 1, h, dk, dv, 0 if low is None else low.shape[1], int(act), state.shape[0], 1.0 / tau,
+        q_scale, int(chunked), _dt(q), _stream()), "linear_attention")
+    _count("linear_attention" + ("_chunked" if chunked else ""),
+           "linear_attn_chunk_kernel" if chunked and q.dtype == torch.bfloat16 else "linear_attn_recurrent_kernel")
+    return out
+
+
+def norm_gate(o, g, weight, eps, vdim, joint, act, out_cols, total=None, total_heads=0):
+    _bind_linear()
+    t, h, dv = o.shape
+    assert o.is_contiguous() and g.stride(1) == 1 and g.dtype == o.dtype and weight.dtype == torch.float32
+    assert out_cols == h * dv and act in ("sigmoid", "silu")
+    per_row, group = (1, h * dv) if joint else (h, dv)
+    width = (total_heads if joint and total is not None else h if joint else 1) * vdim
+    out = torch.empty((t, out_cols), dtype=o.dtype, device=o.device)
+    check(lib().msgl_norm_gate(_p(o), _p(g), g.stride(0), _p(weight), _p(total), _p(out), t, per_row, group, float(width), eps,
+                               int(act == "silu"), _dt(o), _stream()), "norm_gate")
+    _count("norm_gate", "norm_gate_kernel")
+    return out
+
+
 # ------------------------------------------------------------------------------------------ latent attention
 STATIC_WEIGHTS = False
 
@@ -999,9 +1073,32 @@ def latent_norm_store(c, weight, rank, eps, rows, out_loc):
 _NO_STORE = (None, 0, None, None, None, 0, 0, 0.0, 0)
 
 
-def head_gemm(x, w, out=None, store=None):
+def _gate(gate):
+    if gate is None:
+        return None, 0
+    assert gate.shape[1] == 1 or gate.stride(1) == 1
+    return _p(gate), gate.stride(0)
+
+
+def latent_rope(q, dim, dims, cos_sin, positions, store=None):
+    """Rotates channels ``dim .. dim + dims`` of the heads ``q [T, H, D]`` (a view) in place. ``store``: ``(raw latents
+    [T, width], norm weight, rank, eps, pool rows, out_loc, width of the shared key part)``."""
+    _bind_latent()
+    assert q.stride(2) == 1 and cos_sin.dtype == torch.float32 and cos_sin.is_contiguous() and cos_sin.shape[1] == dims
+    stored = (None, 0, None, None, None, q.shape[0], 0, 0, 0, 0.0, 0)
+    if store is not None:
+        c, weight, rank, eps, rows, out_loc, rot_dim = store
+        assert c.stride(1) == 1 and rows.is_contiguous() and rows.dtype == c.dtype == q.dtype and weight.dtype == torch.float32
+        stored = (_p(c), c.stride(0), _p(weight), _p(rows), _p(out_loc), q.shape[0], rank, rows.shape[2], rot_dim, eps,
+                  rows.shape[0] * rows.shape[1])
+    check(lib().msgl_latent_rope(_p(q), q.stride(0), q.stride(1), q.shape[1], dim, dims, _p(cos_sin), _p(positions),
+                                 cos_sin.shape[0], *stored, _dt(q), _stream()), "latent_rope")
+    _count("latent_rope", "latent_rope_kernel")
+
+
+def head_gemm(x, w, out=None, store=None, gate=None):
     """``x [T, H, K]`` (any row and head stride), ``w [H, N, K]`` -> ``[T, H, N]``. ``store``: the arguments of
-    ``latent_norm_store`` to run in the same launch (16-bit)."""
+    ``latent_norm_store`` to run in the same launch (16-bit). ``gate [T, H]``: logits of a sigmoid on the result."""
     _bind_latent()
     t, h, k = x.shape
     n = w.shape[1]
@@ -1012,7 +1109,7 @@ def head_gemm(x, w, out=None, store=None):
     if x.dtype == torch.float32:
         assert store is None
         check(lib().msgl_gemm_f32(_p(x), x.stride(0), x.stride(1), _p(w), k, n * k, _p(out), out.stride(0),
-                                  out.stride(1), t, n, k, h, _stream()), "head_gemm")
+                                  out.stride(1), t, n, k, h, *_gate(gate), _stream()), "head_gemm")
         _count("head_gemm", "gemm_f32_kernel")
         return out
     stored = _NO_STORE
@@ -1022,7 +1119,7 @@ def head_gemm(x, w, out=None, store=None):
         stored = (_p(c), c.stride(0), _p(norm), _p(rows), _p(out_loc), rank, rows.shape[2], eps,
                   rows.shape[0] * rows.shape[1])
     check(lib().msgl_head_gemm(_p(x), x.stride(0), x.stride(1), _p(w), _p(out), out.stride(0), out.stride(1), t, h, n, k,
-                               int(STATIC_WEIGHTS), None, None, 1, *stored, _stream()), "head_gemm")
+                               int(STATIC_WEIGHTS), None, None, 1, *_gate(gate), *stored, _stream()), "head_gemm")
     _count("head_gemm", "head_gemm_kernel")
     return out
 
@@ -1037,14 +1134,14 @@ class LatentSplit:
         self.ws_o, self.ws_lse, self.shape = ws_o, ws_lse, shape
 
 
-def head_gemm_combine(x: LatentSplit, w, out):
+def head_gemm_combine(x: LatentSplit, w, out, gate=None):
     """The value projection of a split attention: merges the key ranges while it reads them."""
     _bind_latent()
     t, h, k = x.shape
     n = w.shape[1]
     assert w.is_contiguous() and w.shape == (h, n, k) and out.stride(2) == 1 and out.shape == (t, h, n)
     check(lib().msgl_head_gemm(None, 0, 0, _p(w), _p(out), out.stride(0), out.stride(1), t, h, n, k, int(STATIC_WEIGHTS),
-                               _p(x.ws_o), _p(x.ws_lse), x.ws_o.shape[0], *_NO_STORE, _stream()), "head_gemm")
+                               _p(x.ws_o), _p(x.ws_lse), x.ws_o.shape[0], *_gate(gate), *_NO_STORE, _stream()), "head_gemm")
     _count("head_gemm", "head_gemm_kernel")
     return out
 
@@ -1059,13 +1156,13 @@ def latent_splits(batch: int, heads: int, rank: int, up_to: int) -> int:
 
 
 def latent_attention(q, rows, block_table, cu_q, seq_lens, scale, window, max_q, max_kv, splits=1, merge=True,
-                     one_form=False):
-    """``merge=False``: a split result stays a ``LatentSplit``. ``one_form``: the same kernel variant whatever the number
+                     one_form=False, sink=None):
+    """``sink [H]`` fp32: logits only the denominator counts. ``merge=False``: a split result stays a ``LatentSplit``. ``one_form``: the same kernel variant whatever the number
     of rows per request (verification rows must reproduce decode rows bit for bit)."""
     _bind_latent()
     t, h, r = q.shape
     assert q.is_contiguous() and rows.is_contiguous() and rows.shape[2] == r and rows.dtype == q.dtype
-    if q.dtype == torch.float32 or r > 512:
+    if q.dtype == torch.float32 or r > 576:
         splits = 1
     out = torch.empty_like(q) if merge or splits == 1 else None
     ws_o = ws_l = None
@@ -1075,7 +1172,7 @@ def latent_attention(q, rows, block_table, cu_q, seq_lens, scale, window, max_q,
     check(lib().msgl_latent_attention(
         _p(q), _p(rows), _p(out), _p(block_table), block_table.stride(0), _p(cu_q), _p(seq_lens), _p(ws_o), _p(ws_l),
         seq_lens.numel(), t, int(max_q), h, r, rows.shape[1], rows.shape[0], int(window), splits, float(scale),
-        int(one_form), _dt(q), _stream()), "latent_attention")
+        _p(sink), int(one_form), _dt(q), _stream()), "latent_attention")
     _count("latent_attention", "latent_attention_kernel", 2 if splits > 1 and merge else 1)
     return out if out is not None else LatentSplit(ws_o, ws_l, (t, h, r))
 
@@ -1137,7 +1234,8 @@ def latent_prefill_ok(dim: int, vdim: int, scale: float) -> bool:
     return dim <= 128 and vdim <= 128 and dim % 8 == 0 and vdim % 8 == 0 and scale > 0
 
 
-def latent_prefill(q, expand_k, up_v, rows, row_id, block_table, plan: LatentPrefillPlan, scale, window, out):
+def latent_prefill(q, expand_k, up_v, rows, row_id, block_table, plan: LatentPrefillPlan, scale, window, out, sink=None,
+                   gate=None):
     """Prefill with per-head keys and values expanded from the latents: ``q [T, H, dim]``, ``expand_k [H * dim, R]``,
     ``up_v [H, vdim, R]``, one layer of the latent pool ``rows`` -> ``out [T, H, vdim]``. The values come out of their
     matrix product transposed (``[H * vdim, tokens]``), the layout the tensor core reads them in."""
@@ -1163,6 +1261,6 @@ def latent_prefill(q, expand_k, up_v, rows, row_id, block_table, plan: LatentPre
         gemm_static_weights(static)
     check(lib().msgl_attn_prefill_pos(_p(q), q.stride(0), q.stride(1), _p(k), _p(vt), plan.t_pad, _p(out), out.stride(0),
                                       out.stride(1), base, plan.n_items, t, h, dim, vdim, int(window), float(scale),
-                                      _dt(q), _stream()), "attn_prefill_pos")
+                                      _p(sink), *_gate(gate), _dt(q), _stream()), "attn_prefill_pos")
     _count("latent_prefill", "attn_prefill_tc_kernel")
     return out

@@ -10,7 +10,9 @@ from . import _lib
 from . import cuda as K
 from ._lib import c_f, c_i, c_ll, c_p, check, lib
 
-_lib.bind("msgl_moe_route", c_i, [c_p, c_p, c_p, c_p, c_p, c_i, c_i, c_i, c_i, c_i, c_f, c_i, c_i, c_i, c_p])
+_lib.bind("msgl_moe_route", c_i, [c_p] * 5 + [c_i] * 5 + [c_f, c_i, c_i, c_ll, c_i, c_i, c_i, c_p])
+_lib.bind("msgl_moe_combine32", c_i, [c_p, c_p, c_p, c_p, c_i, c_p, c_ll, c_p, c_i, c_i, c_i, c_i, c_p])
+_lib.bind("msgl_gemm_f32_grouped", c_i, [c_p, c_p, c_p, c_i, c_i, c_i, c_p, c_p])
 _lib.bind("msgl_moe_align", c_i, [c_p, c_p, c_p, c_p, c_p, c_p, c_p, c_p, c_i, c_i, c_i, c_i, c_i, c_i, c_p])
 _lib.bind("msgl_moe_permute", c_i, [c_p, c_p, c_p, c_i, c_i, c_i, c_i, c_p])
 _lib.bind("msgl_moe_combine", c_i, [c_p, c_p, c_p, c_p, c_i, c_i, c_i, c_i, c_p])
@@ -21,12 +23,12 @@ _DT = {torch.bfloat16: 0, torch.float16: 1, torch.float32: 2}
 
 
 def moe_route(router_logits, top_k, renormalize, scoring="softmax", scale=1.0, counts=None, e_start=0, e_local=None,
-              bias=None):
-    """Softmax / sigmoid scores, top-k by score (+ selection ``bias`` when given), optional
+              bias=None, groups=1, keep=1):
+    """``groups > 1``: group-limited choice, a group scoring as its best member. Softmax / sigmoid scores, top-k by score (+ selection ``bias`` when given), optional
     renormalisation, in one launch. ``counts [e_local]`` (int32), when given, receives the number
     of tokens routed to every local expert, which is what the alignment step needs."""
     t, e = router_logits.shape
-    assert router_logits.is_contiguous()
+    assert router_logits.stride(1) == 1
     w = torch.empty((t, top_k), dtype=torch.float32, device=router_logits.device)
     ids = torch.empty((t, top_k), dtype=torch.int32, device=router_logits.device)
     if bias is not None:
@@ -35,7 +37,7 @@ def moe_route(router_logits, top_k, renormalize, scoring="softmax", scale=1.0, c
                                ids.data_ptr(), None if counts is None else counts.data_ptr(), t, e, top_k,
                                int(renormalize),
                                int(scoring != "softmax"), float(scale), e_start, e if e_local is None else e_local,
-                               _DT[router_logits.dtype], K._stream()), "moe_route")
+                               router_logits.stride(0), groups, keep, _DT[router_logits.dtype], K._stream()), "moe_route")
     K._count("moe_route", "moe_route_kernel")
     return w, ids
 
@@ -106,6 +108,39 @@ def moe_forward(x, w13, w2, topk_w, topk_ids, expert_offset=0, counts=None):
     check(lib().msgl_moe_combine(y.data_ptr(), topk_w.data_ptr(), pair_row.data_ptr(), out.data_ptr(), t, h, k,
                                  _DT[x.dtype], K._stream()), "moe_combine")
     K._count("moe_combine", "moe_combine_kernel")
+    return out
+
+
+def gemm_f32_grouped(a, b, tile_expert):
+    """The true-fp32 form of ``gemm_grouped``."""
+    e, n, k = b.shape
+    out = torch.empty((a.shape[0], n), dtype=torch.float32, device=a.device)
+    assert a.is_contiguous() and b.is_contiguous() and a.shape[1] == k
+    check(lib().msgl_gemm_f32_grouped(a.data_ptr(), b.data_ptr(), out.data_ptr(), a.shape[0], n, k, tile_expert.data_ptr(),
+                                      K._stream()), "gemm_f32_grouped")
+    K._count("moe_gemm_f32_grouped", "gemm_f32_kernel")
+    return out
+
+
+def experts_partial32(x, w13, w2, topk_w, topk_ids, limit, alpha, shared=None, shared_gate=None, counts=None):
+    """Clamped experts for an fp32 residual stream: ``w13 [E, 2I, K]``, ``w2 [E, N, I]`` -> fp32 ``[T, N]``; ``shared``
+    rows are added behind the sigmoid of ``shared_gate [T]`` (fp32 logits)."""
+    t, k = topk_ids.shape
+    sorted_pair, pair_row, tile_expert, _meta = moe_align(topk_ids, 0, w13.shape[0], counts)
+    f32 = x.dtype == torch.float32
+    # rows of fp32 are permuted as twice as many 16-bit values
+    xs = _permute(x.view(torch.bfloat16), sorted_pair, k).view(torch.float32) if f32 else _permute(x, sorted_pair, k)
+    mm = gemm_f32_grouped if f32 else gemm_grouped
+    y = mm(K.act_and_mul(mm(xs, w13, tile_expert), "clamped", alpha, limit), w2, tile_expert)
+    n = w2.shape[1]
+    out = torch.empty((t, n), dtype=torch.float32, device=x.device)
+    if shared is not None:
+        assert shared.is_contiguous() and shared.dtype == x.dtype and shared.shape[1] <= n
+    check(lib().msgl_moe_combine32(y.data_ptr(), topk_w.data_ptr(), pair_row.data_ptr(), K._p(shared),
+                                   0 if shared is None else shared.shape[1], K._p(shared_gate),
+                                   0 if shared_gate is None else shared_gate.stride(0), out.data_ptr(), t, n, k, _DT[x.dtype],
+                                   K._stream()), "moe_combine32")
+    K._count("moe_combine32", "moe_combine32_kernel")
     return out
 
 

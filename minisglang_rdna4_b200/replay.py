@@ -133,7 +133,7 @@ def main(argv: Optional[Sequence[str]] = None) -> int:
 
         if not os.path.exists(_lib.LIB_PATH):
             if mc.latent_layers:
-                _lib.use_part(build.build_cuda(part="latent"))
+                _lib.use_part(build.build_cuda(part="layered" if mc.layer_specs else "latent"))
             else:
                 build.build_cuda()
     torch.backends.cuda.matmul.allow_tf32 = False
