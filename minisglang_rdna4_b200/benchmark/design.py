@@ -1,7 +1,8 @@
-"""Prefill and decode throughput of the Mitilix design beside the closest family at equal size (a Mistral-shaped
-decoder: grouped-query sliding-window attention, gated MLP), and the time of every kernel of both against its roofline.
+"""Prefill and decode throughput of a design beside the closest family at equal size, and the time of every kernel of
+both against its roofline: Mitilix beside a Mistral-shaped decoder (grouped-query sliding-window attention, gated MLP);
+Rafodra beside the Qwen3-Next hybrid (``design_rafodra.py``).
 
-``python bench.py --design mitilix [--size small|large]`` prints one JSON line per (size, model) and one per kernel.
+``python bench.py --design mitilix|rafodra [--size small|large]`` prints one JSON line per (size, model) and one per kernel.
 Random weights, synthetic token ids, one GPU. Throughput comes from CUDA events around every engine step of
 ``LLM.generate``; a kernel is timed with CUDA events over many launches of which each flushes L2 first."""
 from __future__ import annotations
@@ -259,20 +260,26 @@ def kernels(s: Dict) -> List[Dict]:
     return rows
 
 
-def run(size: str, what: str, clocks) -> None:
-    names = list(SIZES) if size == "all" else [size]
+def run(design: str, size: str, what: str, clocks) -> None:
+    if design == "rafodra":
+        from . import design_rafodra as d
+
+        sizes, pair, kernel_rows = d.SIZES, (("rafodra", d.rafodra_config), ("qwen3_next", d.qwen_config)), d.kernels
+    else:
+        sizes, pair, kernel_rows = SIZES, (("mitilix", mitilix_config), ("mistral", mistral_config)), kernels
+    names = list(sizes) if size == "all" else [size]
     for name in names:
-        s = SIZES[name]
+        s = sizes[name]
         clocks.start()
         lines = []
         if what in ("all", "throughput"):
-            for model, make in (("mitilix", mitilix_config), ("mistral", mistral_config)):
+            for model, make in pair:
                 # a process per model: the device memory of one is gone when the next sizes its pool
                 with mp.get_context("spawn").Pool(1) as pool:
                     lines.append({"design": model, "size": name, "shape": s, "prompt": 2048, "dtype": "bf16",
                                   "data": "synthetic", **pool.apply(throughput, (make(s),))})
         if what in ("all", "kernels"):
-            lines += [{"size": name, **r} for r in kernels(s)]
+            lines += [{"size": name, **r} for r in kernel_rows(s)]
         seen = clocks.stop()
         for ln in lines:
             print(json.dumps({**ln, "clocks": {k: seen[k] for k in ("sm_mhz", "sm_max_mhz", "reasons")}}), flush=True)

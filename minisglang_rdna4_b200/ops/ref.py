@@ -782,7 +782,7 @@ def norm_gate(o: torch.Tensor, g: torch.Tensor, weight: torch.Tensor, eps: float
     x = o.float()
     if joint:
         ss = x.pow(2).sum((1, 2)) if total is None else total
-        x = x * torch.rsqrt(ss / ((total_heads or h) * vdim) + eps)[:, None, None]
+        x = x * torch.rsqrt(ss / ((h if total is None else total_heads) * vdim) + eps)[:, None, None]
         x = x * weight.float().view(1, h, dv)
     else:
         x = x * torch.rsqrt(x.pow(2).sum(-1, keepdim=True) / vdim + eps) * weight.float().view(1, 1, dv)

@@ -84,10 +84,11 @@ def reference(cfg, w, seqs):
     return {n: plain.logits(cfg, w, s) for n, s in seqs.items()}
 
 
-def play(rep, seqs, schedule, want, limit):
+def play(rep, seqs, schedule, want, limit, cap=None):
     """``schedule``: steps of (request, count); a request ends with its last token, ``name#k`` replays ``name`` under
-    another id. Every row's logits are compared."""
-    at = {}
+    another id. Every row's logits are compared. With a ``cap`` (routed experts in 16 bits, where a close choice may fall
+    the other way) one row in twenty may be over the limit, none over the cap."""
+    at, errs = {}, []
     for step in schedule:
         entries, end, rows = [], [], []
         for name, n in step:
@@ -99,7 +100,10 @@ def play(rep, seqs, schedule, want, limit):
                 end.append(name)
         got = rep.step(entries, end)
         err = spread(got, torch.cat(rows))
-        assert float(err.max()) <= limit, (step, float(err.max()), int(err.argmax()))
+        assert float(err.max()) <= (cap or limit), (step, float(err.max()), int(err.argmax()))
+        errs.append(err)
+    over = torch.cat(errs) > limit
+    assert float(over.float().mean()) <= 0.05 or int(over.sum()) <= 1, (int(over.sum()), over.numel())
     held = sum(-(-r.device_len // rep.page_size) for r in rep._live.values())
     assert rep.cache.free_pages == rep.cache.num_pages - held
 
