@@ -128,9 +128,19 @@ __global__ void __launch_bounds__(128) latent_rope_kernel(T* __restrict__ q, lon
   if (a.c != nullptr && threadIdx.x < 32) store_latent(a, t, threadIdx.x);
   const float* cs = a.cos_sin + (size_t)table_row(a.positions, t, a.table_rows) * dims;
   const int half = dims / 2;
+  const bool whole = ((first | hq | ldq) & 1) == 0;      // a pair is one aligned word
   for (int id = threadIdx.x; id < H * half; id += 128) {
     const int h = id / half, i = id - h * half;
     T* p = q + t * ldq + h * hq + first + 2 * i;
+    if constexpr (sizeof(T) == 2) {
+      if (whole) {
+        auto* w = reinterpret_cast<typename Pack2<T>::type*>(p);
+        float2 f = to_float2(*w);
+        rotate(f.x, f.y, cs[i], cs[half + i]);
+        *w = Pack2<T>::make(f.x, f.y);
+        continue;
+      }
+    }
     float x = to_float(p[0]), y = to_float(p[1]);
     rotate(x, y, cs[i], cs[half + i]);
     p[0] = from_float<T>(x);

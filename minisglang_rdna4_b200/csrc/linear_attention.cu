@@ -29,7 +29,7 @@ __device__ __forceinline__ float lg2a(float x) {
   asm("lg2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
 }
-__device__ __forceinline__ float silu(float x) { return x / (1.f + __expf(-x)); }
+__device__ __forceinline__ float silu(float x) { return __fdividef(x, 1.f + __expf(-x)); }
 template <typename T> __device__ __forceinline__ float silu_as(float x) {
   if constexpr (sizeof(T) == 4) return x / (1.f + expf(-x));
   return silu(x);
@@ -203,6 +203,7 @@ __device__ __forceinline__ void cp16z(uint32_t dst, const void* src, bool valid)
 constexpr int kC = 16;        // tokens per chunk
 constexpr int kCols = 64;     // value columns per CTA: four warps of 16
 constexpr int kStages = 2;
+constexpr int kRaw = 3;       // chunks of raw rows in flight
 constexpr float kMaxLog2 = 80.f;
 
 template <int DK> struct ChunkSmem {
@@ -215,12 +216,17 @@ template <int DK> struct ChunkSmem {
   static constexpr int off_score = off_dec + DK * 4;      // [NP][2][32] float4
   static constexpr int off_meta = off_score + NP * 1024;
   static constexpr int stage = off_meta + 16;
+  // raw rows as they come: per producer warp and chunk 16 x 32 of q and of k, and 16 x 64 values per chunk
+  static constexpr int off_raw = kStages * stage;
+  static constexpr int raw_warp = 2 * kC * 64;
+  static constexpr int raw = NP * raw_warp + kC * kCols * 2;
+  static constexpr int off_gate = off_raw + kRaw * raw;
   static constexpr int gate_bytes(int rank) {
     const int r = (rank + 15) / 16 * 16;
-    // W transposed [r][DK] fp32, and per producer warp two raw blocks [16][r] and one [r][16] in fp32
-    return rank > 0 ? r * DK * 4 + NP * (2 * kC * r * 2 + r * kC * 4) : 0;
+    // W transposed [r][DK] fp32, and per producer warp raw blocks [16][r] and one [r][16] in fp32
+    return rank > 0 ? r * DK * 4 + NP * (kRaw * kC * r * 2 + r * kC * 4) : 0;
   }
-  static constexpr int bytes(int rank) { return kStages * stage + gate_bytes(rank); }
+  static constexpr int bytes(int rank) { return off_gate + gate_bytes(rank); }
 };
 
 // Warps 0-3: a slice of 16 value columns each, S^T slice in the accumulators of v^T k, which is also the layout in which
@@ -355,79 +361,86 @@ __global__ void __launch_bounds__(128 + DK, DK <= 128 ? 2 : 1) linear_attn_chunk
   using bf = __nv_bfloat16;
   const int pw = warp - 4, ch = pw * 32 + lane;
   const bool live = ch < a.dk;
-  const bf* q = reinterpret_cast<const bf*>(a.q) + (size_t)lo * a.ld + (size_t)h * a.dk + (live ? ch : 0);
-  const bf* k = reinterpret_cast<const bf*>(a.k) + (size_t)lo * a.ld + (size_t)h * a.dk + (live ? ch : 0);
-  const int r16 = (a.rank + 15) / 16 * 16;
-  float* up = reinterpret_cast<float*>(smem + kStages * L::stage);          // [r16][DK]
-  uint8_t* mine = reinterpret_cast<uint8_t*>(up + r16 * DK) + pw * (2 * kC * r16 * 2 + r16 * kC * 4);
-  float* lowf = reinterpret_cast<float*>(mine + 2 * kC * r16 * 2);          // [r16][16]
-  const bool channel = a.decay == nullptr;
-  float bias = 0.f, fixed = 0.f;
+  const bf* q = reinterpret_cast<const bf*>(a.q) + (size_t)lo * a.ld + (size_t)h * a.dk;
+  const bf* k = reinterpret_cast<const bf*>(a.k) + (size_t)lo * a.ld + (size_t)h * a.dk;
+  const bf* v = reinterpret_cast<const bf*>(a.v) + (size_t)lo * a.ld + (size_t)h * a.dv + blockIdx.x * kCols;
   const bf* low = reinterpret_cast<const bf*>(a.low) + (size_t)lo * a.ld;
-  auto fetch_low = [&](int start, int buf) {      // a block of 16 tokens, rows past the end as zeros
-    const int per = r16 / 8;
-    for (int id = lane; id < kC * per; id += 32) {
-      const int t = id / per, c = id - t * per;
-      const bool ok = start + t < len;
-      cp16z(smem_u32(mine) + (buf * kC * r16 + t * r16 + c * 8) * 2, low + (ok ? (long long)(start + t) * a.ld + c * 8 : 0), ok);
+  const int vcols = min(kCols, a.dv - (int)blockIdx.x * kCols);
+  const int r16 = (a.rank + 15) / 16 * 16;
+  float* up = reinterpret_cast<float*>(smem + L::off_gate);                 // [r16][DK]
+  uint8_t* mine = reinterpret_cast<uint8_t*>(up + r16 * DK) + pw * (kRaw * kC * r16 * 2 + r16 * kC * 4);
+  float* lowf = reinterpret_cast<float*>(mine + kRaw * kC * r16 * 2);       // [r16][16]
+  const bool channel = a.decay == nullptr;
+  constexpr int NV = L::NP >= 4 ? 1 : 4 / L::NP;       // 16-byte pieces of the value block per thread
+  // Raw rows of a chunk: this warp's channels of q and k, this thread's pieces of v (which only it reads), this warp's
+  // copy of the low-rank rows. Rows past the end are zeros.
+  auto fetch = [&](int start) {
+    if (start < len) {
+      const int buf = (start / kC) % kRaw;
+      const uint32_t dst = base + L::off_raw + buf * L::raw;
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const int id = lane + (i & 1) * 32, t = id >> 2, c = pw * 32 + (id & 3) * 8;
+        const bool ok = start + t < len && c < a.dk;
+        cp16z(dst + pw * L::raw_warp + (i >> 1) * kC * 64 + id * 16,
+              (i >> 1 ? k : q) + (ok ? (long long)(start + t) * a.ld + c : 0), ok);
+      }
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+        const int id = ch + i * DK, t = id >> 3, c = (id & 7) * 8;
+        if (id >= 128) break;
+        const bool ok = start + t < len && c < vcols;
+        cp16z(dst + L::NP * L::raw_warp + id * 16, v + (ok ? (long long)(start + t) * a.ld + c : 0), ok);
+      }
+      const int per = r16 / 8;
+      for (int id = lane; id < kC * per; id += 32) {
+        const int t = id / per, c = id - t * per;
+        const bool ok = start + t < len;
+        cp16z(smem_u32(mine) + (buf * kC * r16 + t * r16 + c * 8) * 2, low + (ok ? (long long)(start + t) * a.ld + c * 8 : 0), ok);
+      }
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
+#pragma unroll
+  for (int i = 0; i < kRaw - 1; ++i) fetch(i * kC);
+  float bias = 0.f, fixed = 0.f;
   if (channel) {
-    fetch_low(0, 0);
     const bf* w = reinterpret_cast<const bf*>(a.up) + (size_t)(h * a.dk + (live ? ch : 0)) * a.rank;
     for (int r = 0; r < r16; ++r) up[r * DK + ch] = live && r < a.rank ? to_float(w[r]) : 0.f;
     bias = live ? a.bias[h * a.dk + ch] : 0.f;
   } else {
     fixed = fmaxf(log2f(a.decay[h]), -1e4f);
   }
-  bf qn[kC], kn[kC];
-  uint4 vn[4];
-  // the value block [16][64]: eight columns per thread and step
-  const bf* v = reinterpret_cast<const bf*>(a.v) + (size_t)lo * a.ld + (size_t)h * a.dv + blockIdx.x * kCols;
-  const int vcols = min(kCols, a.dv - (int)blockIdx.x * kCols);
-  auto fetch = [&](int start) {
-#pragma unroll
-    for (int t = 0; t < kC; ++t) {
-      const bool ok = live && start + t < len;
-      qn[t] = ok ? q[(long long)(start + t) * a.ld] : __float2bfloat16(0.f);
-      kn[t] = ok ? k[(long long)(start + t) * a.ld] : __float2bfloat16(0.f);
-    }
-#pragma unroll
-    for (int i = 0; i < (L::NP >= 4 ? 1 : 4 / L::NP); ++i) {
-      const int id = ch + i * DK, t = id >> 3, c = (id & 7) * 8;
-      vn[i] = id < 128 && start + t < len && c < vcols
-                  ? *reinterpret_cast<const uint4*>(v + (long long)(start + t) * a.ld + c)
-                  : make_uint4(0, 0, 0, 0);
-    }
-  };
-  fetch(0);
   int stage = 0;
   for (int start = 0; start < len; start += kC) {
     const int n = min(kC, len - start);
     float qf[kC], kf[kC], cum[kC];
+    const int raw_buf = (start / kC) % kRaw;
+    const uint8_t* raw = smem + L::off_raw + raw_buf * L::raw;
+    asm volatile("cp.async.wait_group %0;" ::"n"(kRaw - 2) : "memory");
+    __syncwarp();                          // this chunk's rows are there, and everyone is done with the one before
+    fetch(start + (kRaw - 1) * kC);
+    {
+      const bf* qr = reinterpret_cast<const bf*>(raw + pw * L::raw_warp) + lane;
 #pragma unroll
-    for (int t = 0; t < kC; ++t) {
-      qf[t] = to_float(qn[t]);
-      kf[t] = to_float(kn[t]);
-      if (a.act) {
-        qf[t] = silu(qf[t]);
-        kf[t] = silu(kf[t]);
+      for (int t = 0; t < kC; ++t) {
+        qf[t] = to_float(qr[t * 32]);
+        kf[t] = to_float(qr[(kC + t) * 32]);
       }
-      qf[t] *= a.q_scale;
-    }
-    uint4 vc[4];
+      if (a.act) {                         // (outside the loop over tokens: no branch between independent chains)
 #pragma unroll
-    for (int i = 0; i < 4; ++i) vc[i] = vn[i];
-    if (start + kC < len) fetch(start + kC);
+        for (int t = 0; t < kC; ++t) {
+          qf[t] = silu(qf[t]);
+          kf[t] = silu(kf[t]);
+        }
+      }
+#pragma unroll
+      for (int t = 0; t < kC; ++t) qf[t] *= a.q_scale;
+    }
     if (channel) {
-      const int buf = (start / kC) & 1;
-      asm volatile("cp.async.wait_group 0;" ::: "memory");
+      const bf* lr = reinterpret_cast<const bf*>(mine) + raw_buf * kC * r16;
+      for (int id = lane; id < kC * r16; id += 32) lowf[id] = to_float(lr[(id % kC) * r16 + id / kC]);
       __syncwarp();
-      const bf* raw = reinterpret_cast<const bf*>(mine) + buf * kC * r16;
-      for (int id = lane; id < kC * r16; id += 32) lowf[id] = to_float(raw[(id % kC) * r16 + id / kC]);
-      __syncwarp();
-      if (start + kC < len) fetch_low(start + kC, buf ^ 1);
 #pragma unroll
       for (int t = 0; t < kC; ++t) cum[t] = bias;
       for (int r = 0; r < a.rank; ++r) {
@@ -444,8 +457,8 @@ __global__ void __launch_bounds__(128 + DK, DK <= 128 ? 2 : 1) linear_attn_chunk
 #pragma unroll
       for (int t = 0; t < kC; ++t) {
         // log2 sigmoid(z) = -log2(1 + 2^(-z log2 e))
-        const float y = -cum[t] * kLog2e;
-        cum[t] = (y > 64.f ? y : lg2a(1.f + ex2a(y))) * -a.inv_tau;
+        const float y = -cum[t] * kLog2e, soft = lg2a(1.f + ex2a(fminf(y, 64.f)));
+        cum[t] = (y > 64.f ? y : soft) * -a.inv_tau;
       }
       __syncwarp();
     } else {
@@ -464,35 +477,38 @@ __global__ void __launch_bounds__(128 + DK, DK <= 128 ? 2 : 1) linear_attn_chunk
       uint8_t* sp = smem + st * L::stage;
       bf* qh = reinterpret_cast<bf*>(sp) + ch;
       float step = total;
-#pragma unroll
-      for (int t = 0; t < kC; ++t) {
-        float x = qf[t] * ex2a(cum[t] - total), y = kf[t] * ex2a(total - cum[t]);
-        if (slow) {
-          const bool here = t == part;
-          x = here ? qf[t] : 0.f;
-          y = here ? kf[t] : 0.f;
-          if (here) step = cum[t] - (t > 0 ? cum[t - 1] : 0.f);
-        }
+      auto put = [&](int t, float x, float y) {
         const bf xh = __float2bfloat16(x), yh = __float2bfloat16(y);
         qh[t * L::LD] = xh;
         qh[(kC + t) * L::LD] = __float2bfloat16(x - to_float(xh));
         qh[(2 * kC + t) * L::LD] = yh;
         qh[(3 * kC + t) * L::LD] = __float2bfloat16(y - to_float(yh));
+      };
+      if (!slow) {
+#pragma unroll
+        for (int t = 0; t < kC; ++t) put(t, qf[t] * ex2a(cum[t] - total), kf[t] * ex2a(total - cum[t]));
+      } else {
+#pragma unroll
+        for (int t = 0; t < kC; ++t) {
+          if (t == part) step = cum[t] - (t > 0 ? cum[t - 1] : 0.f);
+          put(t, t == part ? qf[t] : 0.f, t == part ? kf[t] : 0.f);
+        }
       }
       reinterpret_cast<float*>(sp + L::off_dec)[ch] = ex2a(step);
 #pragma unroll
-      for (int i = 0; i < (L::NP >= 4 ? 1 : 4 / L::NP); ++i) {
+      for (int i = 0; i < NV; ++i) {
         const int id = ch + i * DK, t = id >> 3, c = (id & 7) * 8;
         if (id < 128) {
+          const bf* src = reinterpret_cast<const bf*>(raw + L::NP * L::raw_warp) + id * 8;
           bf* dst = reinterpret_cast<bf*>(sp + L::off_v) + t * L::LDV + c;
           if (a.act) {
             float x[8];
-            load8(reinterpret_cast<const bf*>(&vc[i]), x);
+            load8(src, x);
 #pragma unroll
             for (int e = 0; e < 8; ++e) x[e] = silu(x[e]);
             store8(dst, x);
           } else {
-            *reinterpret_cast<uint4*>(dst) = vc[i];
+            *reinterpret_cast<uint4*>(dst) = *reinterpret_cast<const uint4*>(src);
           }
         }
       }
