@@ -202,14 +202,16 @@ __device__ __forceinline__ void cp16z(uint32_t dst, const void* src, bool valid)
 
 constexpr int kC = 16;        // tokens per chunk
 constexpr int kCols = 64;     // value columns per CTA: four warps of 16
-constexpr int kStages = 2;
-constexpr int kRaw = 3;       // chunks of raw rows in flight
 constexpr float kMaxLog2 = 80.f;
 
+// G groups of producer warps take the chunks in turn; NS stage buffers and RAW blocks of raw rows per group.
 template <int DK> struct ChunkSmem {
+  static constexpr int G = DK <= 128 ? 3 : 1;
+  static constexpr int NS = G > 1 ? 1 : 2;
+  static constexpr int RAW = G > 1 ? 2 : 3;
   static constexpr int LD = DK + 8;                       // row stride in elements: rows on different banks
   static constexpr int LDV = kCols + 8;
-  static constexpr int NP = DK / 32;                      // producer warps
+  static constexpr int NP = DK / 32;                      // producer warps per group
   // at 0: q hi, q lo, k hi, k lo, [16][LD] each
   static constexpr int off_v = 4 * kC * LD * 2;
   static constexpr int off_dec = off_v + kC * LDV * 2;
@@ -217,29 +219,33 @@ template <int DK> struct ChunkSmem {
   static constexpr int off_meta = off_score + NP * 1024;
   static constexpr int stage = off_meta + 16;
   // raw rows as they come: per producer warp and chunk 16 x 32 of q and of k, and 16 x 64 values per chunk
-  static constexpr int off_raw = kStages * stage;
+  static constexpr int off_raw = G * NS * stage;
   static constexpr int raw_warp = 2 * kC * 64;
   static constexpr int raw = NP * raw_warp + kC * kCols * 2;
-  static constexpr int off_gate = off_raw + kRaw * raw;
+  static constexpr int off_gate = off_raw + G * RAW * raw;
   static constexpr int gate_bytes(int rank) {
     const int r = (rank + 15) / 16 * 16;
     // W transposed [r][DK] fp32, and per producer warp raw blocks [16][r] and one [r][16] in fp32
-    return rank > 0 ? r * DK * 4 + NP * (kRaw * kC * r * 2 + r * kC * 4) : 0;
+    return rank > 0 ? r * DK * 4 + G * NP * (RAW * kC * r * 2 + r * kC * 4) : 0;
   }
   static constexpr int bytes(int rank) { return off_gate + gate_bytes(rank); }
 };
 
 // Warps 0-3: a slice of 16 value columns each, S^T slice in the accumulators of v^T k, which is also the layout in which
-// the tensor core takes S as the right operand of q S. Warps 4..: 32 key channels each; they turn 16 tokens into
+// the tensor core takes S as the right operand of q S. The other warps: 32 key channels each; they turn 16 tokens into
 // q 2^(b_i - b_end) and k 2^(b_end - b_j) (b: running sum of log2 alpha in the chunk), so that the state only has to be
-// multiplied by 2^b_end once, and the scores q k^T between the chunk's tokens over their channels. A chunk whose decay
-// leaves the range of that is handed over token by token. Stages go through named barriers.
+// multiplied by 2^b_end once, and the scores q k^T between the chunk's tokens over their channels. None of that depends
+// on the chunks before, so groups of such warps work on different chunks at once. A chunk whose decay leaves the range
+// of the factors is handed over token by token. Stages go through named barriers.
 template <int DK>
-__global__ void __launch_bounds__(128 + DK, DK <= 128 ? 2 : 1) linear_attn_chunk_kernel(const LinArgs a) {
+__global__ void __launch_bounds__(128 + ChunkSmem<DK>::G * DK, DK <= 64 ? 2 : 1) linear_attn_chunk_kernel(const LinArgs a) {
   pdl_enter();
   using L = ChunkSmem<DK>;
   extern __shared__ __align__(128) uint8_t smem[];
-  constexpr int NT = 128 + DK, VOTE = 1 + 2 * kStages;
+  constexpr int G = L::G, NS = L::NS, RAW = L::RAW, NT = 128 + DK;
+  // barriers: a stage is full, a stage is empty, a group's vote, all producers
+  constexpr int FULL = 1, EMPTY = FULL + G * NS, VOTE = EMPTY + G * NS, PRODUCERS = VOTE + G;
+  static_assert((G == 1 || NS == 1) && PRODUCERS < 16, "stages in order, sixteen barriers");
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int h = blockIdx.y, b = blockIdx.z;
   const int lo = a.cu_q[b], len = a.cu_q[b + 1] - lo;
@@ -265,12 +271,13 @@ __global__ void __launch_bounds__(128 + DK, DK <= 128 ? 2 : 1) linear_attn_chunk
       }
     __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(a.out) + ((size_t)lo * a.H + h) * a.dv + n0 + t2;
     const long long ldo = (long long)a.H * a.dv;
-    for (int i = 0;; ++i) {
-      const int st = i % kStages;
-      bar_sync(1 + st, NT);
+    const int chunks = (len + kC - 1) / kC;
+    for (int chunk = 0, i = 0; chunk < chunks; ++i) {
+      const int st = G > 1 ? chunk % G : i % NS;
+      bar_sync(FULL + st, NT);
       const uint32_t sb = base + st * L::stage;
       const uint8_t* sp = smem + st * L::stage;
-      const int4 meta = *reinterpret_cast<const int4*>(sp + L::off_meta);      // chunk start, rows [y, z), last
+      const int4 meta = *reinterpret_cast<const int4*>(sp + L::off_meta);      // chunk start, rows [y, z), end of the chunk
       if (active) {
         float o[2][4] = {};
 #pragma unroll
@@ -342,8 +349,8 @@ __global__ void __launch_bounds__(128 + DK, DK <= 128 ? 2 : 1) linear_attn_chunk
         }
       }
       __syncwarp();
-      bar_arrive(1 + kStages + st, NT);
-      if (meta.w) break;
+      bar_arrive(EMPTY + st, NT);
+      chunk += meta.w;
     }
     if (active) {
 #pragma unroll
@@ -359,7 +366,7 @@ __global__ void __launch_bounds__(128 + DK, DK <= 128 ? 2 : 1) linear_attn_chunk
 
   // ---------------------------------------------------------------- key channels
   using bf = __nv_bfloat16;
-  const int pw = warp - 4, ch = pw * 32 + lane;
+  const int grp = (warp - 4) / L::NP, pw = (warp - 4) % L::NP, ch = pw * 32 + lane;
   const bool live = ch < a.dk;
   const bf* q = reinterpret_cast<const bf*>(a.q) + (size_t)lo * a.ld + (size_t)h * a.dk;
   const bf* k = reinterpret_cast<const bf*>(a.k) + (size_t)lo * a.ld + (size_t)h * a.dk;
@@ -368,16 +375,16 @@ __global__ void __launch_bounds__(128 + DK, DK <= 128 ? 2 : 1) linear_attn_chunk
   const int vcols = min(kCols, a.dv - (int)blockIdx.x * kCols);
   const int r16 = (a.rank + 15) / 16 * 16;
   float* up = reinterpret_cast<float*>(smem + L::off_gate);                 // [r16][DK]
-  uint8_t* mine = reinterpret_cast<uint8_t*>(up + r16 * DK) + pw * (kRaw * kC * r16 * 2 + r16 * kC * 4);
-  float* lowf = reinterpret_cast<float*>(mine + kRaw * kC * r16 * 2);       // [r16][16]
+  uint8_t* mine = reinterpret_cast<uint8_t*>(up + r16 * DK) +
+                  (grp * L::NP + pw) * (RAW * kC * r16 * 2 + r16 * kC * 4);
+  float* lowf = reinterpret_cast<float*>(mine + RAW * kC * r16 * 2);        // [r16][16]
   const bool channel = a.decay == nullptr;
   constexpr int NV = L::NP >= 4 ? 1 : 4 / L::NP;       // 16-byte pieces of the value block per thread
   // Raw rows of a chunk: this warp's channels of q and k, this thread's pieces of v (which only it reads), this warp's
   // copy of the low-rank rows. Rows past the end are zeros.
-  auto fetch = [&](int start) {
+  auto fetch = [&](int start, int buf) {
     if (start < len) {
-      const int buf = (start / kC) % kRaw;
-      const uint32_t dst = base + L::off_raw + buf * L::raw;
+      const uint32_t dst = base + L::off_raw + (grp * RAW + buf) * L::raw;
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
         const int id = lane + (i & 1) * 32, t = id >> 2, c = pw * 32 + (id & 3) * 8;
@@ -402,24 +409,25 @@ __global__ void __launch_bounds__(128 + DK, DK <= 128 ? 2 : 1) linear_attn_chunk
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
 #pragma unroll
-  for (int i = 0; i < kRaw - 1; ++i) fetch(i * kC);
+  for (int i = 0; i < RAW - 1; ++i) fetch((grp + i * G) * kC, i);
   float bias = 0.f, fixed = 0.f;
   if (channel) {
     const bf* w = reinterpret_cast<const bf*>(a.up) + (size_t)(h * a.dk + (live ? ch : 0)) * a.rank;
-    for (int r = 0; r < r16; ++r) up[r * DK + ch] = live && r < a.rank ? to_float(w[r]) : 0.f;
+    for (int r = grp; r < r16; r += G) up[r * DK + ch] = live && r < a.rank ? to_float(w[r]) : 0.f;
     bias = live ? a.bias[h * a.dk + ch] : 0.f;
+    bar_sync(PRODUCERS, G * DK);
   } else {
     fixed = fmaxf(log2f(a.decay[h]), -1e4f);
   }
-  int stage = 0;
-  for (int start = 0; start < len; start += kC) {
+  int stage = 0, round = 0;
+  for (int start = grp * kC; start < len; start += G * kC, ++round) {
     const int n = min(kC, len - start);
     float qf[kC], kf[kC], cum[kC];
-    const int raw_buf = (start / kC) % kRaw;
-    const uint8_t* raw = smem + L::off_raw + raw_buf * L::raw;
-    asm volatile("cp.async.wait_group %0;" ::"n"(kRaw - 2) : "memory");
+    const int raw_buf = round % RAW;
+    const uint8_t* raw = smem + L::off_raw + (grp * RAW + raw_buf) * L::raw;
+    asm volatile("cp.async.wait_group %0;" ::"n"(RAW - 2) : "memory");
     __syncwarp();                          // this chunk's rows are there, and everyone is done with the one before
-    fetch(start + (kRaw - 1) * kC);
+    fetch(start + (RAW - 1) * G * kC, (round + RAW - 1) % RAW);
     {
       const bf* qr = reinterpret_cast<const bf*>(raw + pw * L::raw_warp) + lane;
 #pragma unroll
@@ -443,7 +451,8 @@ __global__ void __launch_bounds__(128 + DK, DK <= 128 ? 2 : 1) linear_attn_chunk
       __syncwarp();
 #pragma unroll
       for (int t = 0; t < kC; ++t) cum[t] = bias;
-      for (int r = 0; r < a.rank; ++r) {
+#pragma unroll 4
+      for (int r = 0; r < r16; ++r) {
         const float w = up[r * DK + ch];
 #pragma unroll
         for (int t = 0; t < kC; t += 4) {
@@ -469,10 +478,10 @@ __global__ void __launch_bounds__(128 + DK, DK <= 128 ? 2 : 1) linear_attn_chunk
     for (int t = 0; t < kC; ++t) cum[t] = (t > 0 ? cum[t - 1] : 0.f) + (live && t < n ? cum[t] : 0.f);
     const float total = cum[kC - 1];
     const bool far = -total > kMaxLog2;
-    const bool slow = bar_any(VOTE, DK, far);
+    const bool slow = bar_any(VOTE + grp, DK, far);
     for (int part = 0; part < (slow ? n : 1); ++part, ++stage) {
-      const int st = stage % kStages;
-      if (stage >= kStages) bar_sync(1 + kStages + st, NT);
+      const int st = grp * NS + stage % NS;
+      if (stage >= NS) bar_sync(EMPTY + st, NT);
       const uint32_t sb = base + st * L::stage;
       uint8_t* sp = smem + st * L::stage;
       bf* qh = reinterpret_cast<bf*>(sp) + ch;
@@ -536,13 +545,13 @@ __global__ void __launch_bounds__(128 + DK, DK <= 128 ? 2 : 1) linear_attn_chunk
             make_float4(sc[nb][0], sc[nb][1], sc[nb][2], sc[nb][3]);
       if (ch == 0)
         *reinterpret_cast<int4*>(sp + L::off_meta) =
-            make_int4(start, slow ? part : 0, slow ? part + 1 : n, start + kC >= len && (!slow || part == n - 1));
+            make_int4(start, slow ? part : 0, slow ? part + 1 : n, !slow || part == n - 1);
       __syncwarp();
-      bar_arrive(1 + st, NT);
+      bar_arrive(FULL + st, NT);
     }
   }
   // every arrival at an "empty" barrier is matched before the warps leave
-  for (int i = max(stage - kStages, 0); i < stage; ++i) bar_sync(1 + kStages + i % kStages, NT);
+  for (int i = max(stage - NS, 0); i < stage; ++i) bar_sync(EMPTY + grp * NS + i % NS, NT);
 }
 
 template <int DK> int launch_chunk(const LinArgs& a, int B, cudaStream_t s) {
@@ -557,7 +566,8 @@ template <int DK> int launch_chunk(const LinArgs& a, int B, cudaStream_t s) {
     }
     set = bytes;
   }
-  msgl_launch(linear_attn_chunk_kernel<DK>, dim3((a.dv + kCols - 1) / kCols, a.H, B), dim3(128 + DK), bytes, s, a);
+  msgl_launch(linear_attn_chunk_kernel<DK>, dim3((a.dv + kCols - 1) / kCols, a.H, B), dim3(128 + ChunkSmem<DK>::G * DK), bytes,
+              s, a);
   MSGL_CHECK_LAUNCH("linear_attn_chunk");
   return MSGL_OK;
 }
