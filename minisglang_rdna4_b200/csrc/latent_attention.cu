@@ -119,33 +119,44 @@ template <typename T> __global__ void __launch_bounds__(128) latent_norm_store_k
   if (t < a.rows) store_latent(a, t, threadIdx.x & 31);
 }
 
-// CTA per row: the warps rotate the query heads' pairs; warp 0 stores the row's latent first (store.c != null).
+// `per_row` warps (1 or 4) per row rotate the query heads' pairs; the last of them stores the row's latent after that
+// (store.c != null). vec: four pairs are one aligned 16-byte piece (the fp32 form takes them as two).
 template <typename T>
 __global__ void __launch_bounds__(128) latent_rope_kernel(T* __restrict__ q, long long ldq, long long hq, int H, int first,
-                                                          int dims, const StoreArgs<T> a) {
+                                                          int dims, int per_row, int vec, const StoreArgs<T> a) {
   pdl_enter();
-  const int t = blockIdx.x;
-  if (a.c != nullptr && threadIdx.x < 32) store_latent(a, t, threadIdx.x);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int t = blockIdx.x * (4 / per_row) + warp / per_row, part = warp % per_row;
+  if (t >= a.rows) return;
   const float* cs = a.cos_sin + (size_t)table_row(a.positions, t, a.table_rows) * dims;
   const int half = dims / 2;
-  const bool whole = ((first | hq | ldq) & 1) == 0;      // a pair is one aligned word
-  for (int id = threadIdx.x; id < H * half; id += 128) {
-    const int h = id / half, i = id - h * half;
-    T* p = q + t * ldq + h * hq + first + 2 * i;
-    if constexpr (sizeof(T) == 2) {
-      if (whole) {
-        auto* w = reinterpret_cast<typename Pack2<T>::type*>(p);
-        float2 f = to_float2(*w);
-        rotate(f.x, f.y, cs[i], cs[half + i]);
-        *w = Pack2<T>::make(f.x, f.y);
-        continue;
-      }
+  T* row = q + t * ldq + first;
+  if (vec) {
+    const int pieces = dims / 8;
+#pragma unroll 2
+    for (int id = part * 32 + lane; id < H * pieces; id += per_row * 32) {
+      const int h = id / pieces, i = (id - h * pieces) * 4;
+      T* p = row + h * hq + 2 * i;
+      float x[8];
+      load8(p, x);
+      const float4 c = *reinterpret_cast<const float4*>(cs + i), n = *reinterpret_cast<const float4*>(cs + half + i);
+      rotate(x[0], x[1], c.x, n.x);
+      rotate(x[2], x[3], c.y, n.y);
+      rotate(x[4], x[5], c.z, n.z);
+      rotate(x[6], x[7], c.w, n.w);
+      store8(p, x);
     }
-    float x = to_float(p[0]), y = to_float(p[1]);
-    rotate(x, y, cs[i], cs[half + i]);
-    p[0] = from_float<T>(x);
-    p[1] = from_float<T>(y);
+  } else {
+    for (int id = part * 32 + lane; id < H * half; id += per_row * 32) {
+      const int h = id / half, i = id - h * half;
+      T* p = row + h * hq + 2 * i;
+      float x = to_float(p[0]), y = to_float(p[1]);
+      rotate(x, y, cs[i], cs[half + i]);
+      p[0] = from_float<T>(x);
+      p[1] = from_float<T>(y);
+    }
   }
+  if (a.c != nullptr && part == per_row - 1) store_latent(a, t, lane);
 }
 
 // ------------------------------------------------------------------------------------------ attention args
@@ -796,8 +807,13 @@ MSGL_API int msgl_latent_rope(void* q, long long ldq, long long hq, int H, int f
   if (c != nullptr && (rank <= 0 || rot_dim < dims || rank + rot_dim > width || width % 64 || width > 1024 || ldc % 8 ||
                        (uintptr_t)c % 16 || (uintptr_t)pool % 16))
     return MSGL_BAD_ARG;
+  // many rows: a warp each, the loads in flight come from the grid
+  const int per_row = rows <= 1024 ? 4 : 1;
+  const int vec = first % 8 == 0 && dims % 8 == 0 && ldq % 8 == 0 && hq % 8 == 0 && (uintptr_t)q % 16 == 0 &&
+                  (uintptr_t)cos_sin % 16 == 0;
 #define ROPE(T)                                                                                                     \
-  msgl_launch(latent_rope_kernel<T>, dim3(rows), dim3(128), 0, stream, (T*)q, ldq, hq, H, first, dims,              \
+  msgl_launch(latent_rope_kernel<T>, dim3((rows * per_row + 3) / 4), dim3(128), 0, stream, (T*)q, ldq, hq, H, first, \
+              dims, per_row, vec,                                                                                   \
               StoreArgs<T>{(const T*)c, ldc, (const float*)weight, (T*)pool, (const int32_t*)out_loc, rows, rank,   \
                            width, eps, num_slots, rot_dim, dims, (const float*)cos_sin, (const int32_t*)positions,  \
                            table_rows})

@@ -43,18 +43,19 @@ def test_add_norm(width, cols, rows, center):
             torch.testing.assert_close(got[1].float().cpu(), want[1].float(), rtol=tol, atol=tol)
 
 
-@pytest.mark.parametrize("dims,rot,rank,dim,heads", [(16, 16, 64, 32, 6), (12, 14, 50, 9, 3), (64, 64, 512, 96, 32), (2, 2, 33, 1, 1)])
-def test_latent_rope_and_store(dims, rot, rank, dim, heads):
+@pytest.mark.parametrize("dims,rot,rank,dim,heads", [(16, 16, 64, 32, 6), (12, 14, 50, 9, 3), (16, 24, 40, 8, 5), (64, 64, 512, 96, 32), (2, 2, 33, 1, 1)])
+@pytest.mark.parametrize("t", [37, 1100])
+def test_latent_rope_and_store(dims, rot, rank, dim, heads, t):
     g = _gen(rank)
-    t, width, dp = 37, -(-(rank + rot) // 64) * 64, -(-(dim + rot) // 16) * 16
+    width, dp = -(-(rank + rot) // 64) * 64, -(-(dim + rot) // 16) * 16
     proj, w = torch.randn(t, heads * dp + width + 16, generator=g), torch.rand(width, generator=g)
     pos = torch.randint(0, 3000, (t,), generator=g).int()
     table = get_rope_cache(RotaryConfig(rot, dims, 3000, 1e4, interleaved=True), "cpu")
-    loc = torch.randperm(5 * 16, generator=g)[:t].int()
+    loc = torch.randperm(70 * 16, generator=g)[:t].int()
     for dtype, tol in ((torch.float32, 1e-5), (BF, 1e-2)):
         for own in (True, False):
             a, b = proj.to(dtype), proj.to(DEV, dtype)
-            pools = [torch.full((5, 16, width), 3.0, dtype=dtype, device=d) for d in ("cpu", DEV)]
+            pools = [torch.full((70, 16, width), 3.0, dtype=dtype, device=d) for d in ("cpu", DEV)]
             for x, pool in zip((a, b), pools):
                 q = x[:, :heads * dp].unflatten(1, (heads, dp))
                 store = (x[:, heads * dp:heads * dp + width], w.to(x.device), rank, 1e-5, pool, loc.to(x.device), rot)
