@@ -43,7 +43,7 @@ def test_add_norm(width, cols, rows, center):
             torch.testing.assert_close(got[1].float().cpu(), want[1].float(), rtol=tol, atol=tol)
 
 
-@pytest.mark.parametrize("dims,rot,rank,dim,heads", [(16, 16, 64, 32, 6), (12, 14, 50, 9, 3), (16, 24, 40, 8, 5), (64, 64, 512, 96, 32), (2, 2, 33, 1, 1)])
+@pytest.mark.parametrize("dims,rot,rank,dim,heads", [(24, 24, 72, 40, 5), (12, 14, 50, 9, 3), (16, 24, 40, 8, 5), (64, 64, 512, 96, 32), (2, 2, 33, 1, 1)])
 @pytest.mark.parametrize("t", [37, 1100])
 def test_latent_rope_and_store(dims, rot, rank, dim, heads, t):
     g = _gen(rank)
@@ -194,7 +194,7 @@ def _linear_run(case, h, dk, dv, rank, dev, chunked, tau=8.0, dtype=None, **kw):
 LENS = [1, 16, 17, 40, 2, 70, 15, 1, 33]
 
 
-@pytest.mark.parametrize("h,dk,dv,rank", [(3, 16, 16, 0), (2, 32, 48, 0), (2, 48, 64, 16), (4, 64, 80, 5), (2, 128, 128, 16),
+@pytest.mark.parametrize("h,dk,dv,rank", [(3, 16, 16, 0), (2, 32, 48, 0), (2, 80, 64, 24), (4, 64, 80, 5), (2, 128, 128, 16),
                                           (1, 112, 144, 40), (2, 256, 96, 8), (1, 256, 256, 0)])
 @pytest.mark.parametrize("act", [True, False])
 def test_linear_attention_forms(h, dk, dv, rank, act):
@@ -247,7 +247,7 @@ def test_wide_key_heads_take_the_recurrent_form():
     torch.testing.assert_close(got, want, rtol=1e-2, atol=2e-2)
 
 
-@pytest.mark.parametrize("h,dv,vdim,joint", [(4, 32, 32, True), (3, 16, 10, True), (6, 64, 64, False), (2, 48, 33, False), (16, 128, 128, True)])
+@pytest.mark.parametrize("h,dv,vdim,joint", [(5, 48, 48, True), (3, 16, 10, True), (5, 80, 80, False), (2, 48, 33, False), (16, 128, 128, True)])
 @pytest.mark.parametrize("act", ["sigmoid", "silu"])
 def test_norm_gate(h, dv, vdim, joint, act):
     g = _gen(h)
@@ -264,7 +264,7 @@ def test_norm_gate(h, dv, vdim, joint, act):
 
 
 # ---------------------------------------------------------------------------------- experts
-@pytest.mark.parametrize("e,groups,keep,top", [(8, 4, 3, 4), (6, 3, 1, 2), (64, 8, 2, 6), (128, 64, 5, 8), (5, 1, 1, 3), (512, 16, 16, 16)])
+@pytest.mark.parametrize("e,groups,keep,top", [(12, 4, 2, 5), (6, 3, 1, 2), (64, 8, 2, 6), (128, 64, 5, 8), (5, 1, 1, 3), (512, 16, 16, 16)])
 def test_group_limited_routing(e, groups, keep, top):
     from minisglang_rdna4_b200.ops import moe_kernels as M
 
