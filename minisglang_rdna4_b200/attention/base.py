@@ -24,6 +24,7 @@ class AttnMetadata:
     mask_swa: Optional[torch.Tensor] = None   # the mask sliding-window layers take instead (a mask replaces the window rule)
     workspace: Optional[torch.Tensor] = None
     prefill_plan: Optional[object] = None  # ops.cuda.PrefillPlan of a prefill-phase step on a GPU
+    layer_plans: Optional[object] = None   # the same for layers with reaches of their own, made when one asks for it
 
 
 class BaseAttnBackend(ABC):

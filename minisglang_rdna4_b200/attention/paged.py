@@ -15,10 +15,34 @@ from ..core import Batch, get_global_ctx
 from .base import AttnMetadata, BaseAttnBackend
 
 
+class LayerPlans:
+    """Tables of the tensor-core prefill kernel for the layers of one step, one set per reach (window and chunk) and
+    tile form."""
+
+    def __init__(self, cu_q, seq_lens, device) -> None:
+        self._lens, self._device, self._plans = (cu_q, seq_lens), device, {}
+
+    def of(self, window: int, chunk: int, group: int):
+        """``None``: too few rows for the keys in reach (``ops.cuda.tc_prefill_pays``)."""
+        from ..env import ENV
+        from ..ops import cuda as K
+
+        key = (window, chunk, group % 2)
+        if key not in self._plans:
+            plan = None
+            if not ENV.DISABLE_TC_PREFILL.value and K.tc_prefill_pays(
+                    int(self._lens[0][len(self._lens[1])]), K.PrefillPlan.rows_in_reach(*self._lens, window, chunk)):
+                plan = K.PrefillPlan(*self._lens, self._device, window, chunk, tile=256 if group % 2 else 128)
+            self._plans[key] = plan
+        return self._plans[key]
+
+
 class PagedAttentionBackend(BaseAttnBackend):
     def __init__(self, num_q_heads: int, num_kv_heads: int, head_dim: int, device,
-                 max_batch: int = 0, max_seq_len: int = 0, single_split: bool = False) -> None:
+                 max_batch: int = 0, max_seq_len: int = 0, single_split: bool = False, heads=None) -> None:
+        """``heads``: ``(query heads, row width)`` per layer where layers differ."""
         self.hq, self.hk, self.d = num_q_heads, num_kv_heads, head_dim
+        self.layered = bool(heads)
         self.device = device
         # The number of KV splits of a decode step depends only on the batch size and the
         # longest sequence the pool can hold, never on the lengths in the batch: a captured
@@ -30,7 +54,8 @@ class PagedAttentionBackend(BaseAttnBackend):
         if torch.device(device).type == "cuda":
             from ..ops import cuda as K
 
-            self._workspace = K.attention_workspace(max(max_batch, 1), num_q_heads, head_dim, device)
+            hq, d = max(heads, key=lambda s: s[0] * (s[1] + 1)) if heads else (num_q_heads, head_dim)
+            self._workspace = K.attention_workspace(max(max_batch, 1), hq, d, device)
             K.force_general_decode_attention(single_split)
 
     def prepare_metadata(self, batch: Batch, block_table, cu_q, seq_lens, max_q: int, max_kv: int,
@@ -42,8 +67,13 @@ class PagedAttentionBackend(BaseAttnBackend):
         step whatever its size, so that a row's result does not depend on how its prompt was chunked;
         a short extend over a long cached prefix reads the pool in place with the general kernel).
         Decode and verification steps stay on the general kernel."""
-        plan = None
-        if (host_cu_q is not None and batch.is_prefill and not batch.spec_verify and mask is None and causal
+        plan = layer_plans = None
+        if self.layered:
+            if mask is not None or not causal:
+                raise NotImplementedError("layers with windows and chunks of their own take no attention mask")
+            if host_cu_q is not None and batch.is_prefill and not batch.spec_verify and self._workspace is not None:
+                layer_plans = LayerPlans(host_cu_q, host_seq_lens, self.device)
+        elif (host_cu_q is not None and batch.is_prefill and not batch.spec_verify and mask is None and causal
                 and self._workspace is not None and self.d == 128 and (self.hq // self.hk) % 2 == 0):
             from ..env import ENV
             from ..ops import cuda as K
@@ -57,8 +87,31 @@ class PagedAttentionBackend(BaseAttnBackend):
             cu_q=cu_q, seq_lens=seq_lens, block_table=block_table, max_q=max_q, max_kv=max_kv,
             decode=(max_q == 1 and plan is None), causal=causal, mask=mask, mask_window=mask_window, mask_swa=mask_swa,
             workspace=self._workspace,
-            prefill_plan=plan,
+            prefill_plan=plan, layer_plans=layer_plans,
         )
+
+    def forward_heads(self, q, layer: int, batch: Batch, *, scale: float, window: int = 0, chunk: int = 0,
+                      softcap: float = 0.0, gate=None):
+        """One layer of a model whose layers differ: ``q [T, H, width]`` against row ``layer`` of the pool, with the layer's
+        reach and soft cap; ``gate [T, H * width]``: logits of a sigmoid on the output channels."""
+        md = batch.attn_metadata
+        pool = get_global_ctx().kv_cache
+        k_cache, v_cache = pool.k_cache(layer), pool.v_cache(layer)
+        extra = dict(window=window, chunk=chunk, softcap=softcap, gate=gate)
+        splits = 1
+        if q.is_cuda:
+            from ..ops import cuda as K
+
+            if md.layer_plans is not None and K.prefill_heads_tc_ok(q, k_cache, scale):
+                plan = md.layer_plans.of(window, chunk, q.shape[1] // k_cache.shape[1])
+                if plan is not None:
+                    return K.prefill_attention_tc(q, k_cache, v_cache, md.block_table, plan, scale, **extra)
+            if md.decode and not self.single_split:
+                reach = min([r for r in (window, chunk, self.max_seq_len or md.max_kv) if r > 0])
+                splits = K.choose_splits(md.seq_lens.numel(), k_cache.shape[1], reach, True)
+        return ops.paged_attention(q, k_cache, v_cache, md.block_table, md.cu_q, md.seq_lens, scale, causal=True,
+                                   max_q=md.max_q, max_kv=md.max_kv, decode=md.decode, workspace=md.workspace,
+                                   splits=splits, **extra)
 
     def forward(self, q, layer: int, batch: Batch, *, scale: float, window: int = 0, swa: bool = False):
         md = batch.attn_metadata

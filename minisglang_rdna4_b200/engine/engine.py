@@ -23,7 +23,7 @@ from ..attention import create_attention_backend
 from ..config import EngineConfig
 from ..core import Batch, Context, set_global_ctx
 from ..env import ENV
-from ..kvcache import MHAKVCache
+from ..kvcache import LayeredKVCache, MHAKVCache
 from ..models import create_model
 from ..models.config import NAMED_CONFIGS, ModelConfig
 from ..parallel import comm as comm_mod
@@ -81,10 +81,10 @@ def _resolve_dtype(cfg: EngineConfig, model_cfg: ModelConfig, device: str) -> to
              "bf16": torch.bfloat16, "bfloat16": torch.bfloat16,
              "fp32": torch.float32, "float32": torch.float32, "float": torch.float32}
     dt = table[name]
-    if device == "cuda" and dt == torch.float32 and not model_cfg.latent_layers:
+    if device == "cuda" and dt == torch.float32 and not model_cfg.has_fp32_kernels:
         dt = torch.bfloat16            # the other families' kernels are 16-bit
-    if device == "cuda" and dt == torch.float16 and model_cfg.latent_layers:
-        raise ValueError("models with a latent pool run in bfloat16 or float32 on a GPU")
+    if device == "cuda" and dt == torch.float16 and model_cfg.has_fp32_kernels:
+        raise ValueError(f"{model_cfg.model_type} runs in bfloat16 or float32 on a GPU")
     return dt
 
 
@@ -280,8 +280,9 @@ class Engine:
         # latent-attention models can keep the compressed latent per token instead of per-head K/V
         # (MSGL_MLA_LATENT): absorbed attention through tensor ops, eager steps, no draft verification
         self.mla_latent = bool(ENV.MLA_LATENT.value and mc.is_mla)
-        if mc.latent_layers and (self.kv_fp8 or self.kv_calibrating):
-            raise ValueError("the latent pool has no fp8 form")
+        if mc.has_fp32_kernels and (self.kv_fp8 or self.kv_calibrating):
+            raise ValueError(f"the K/V pool of {mc.model_type} has no fp8 form")
+        self._head_geometry = mc.head_geometry(tp_) if mc.head_layers else None
         if self.mla_latent:
             if self.kv_fp8 or self.kv_calibrating:
                 raise ValueError("the latent pool (MSGL_MLA_LATENT) is 16-bit only")
@@ -303,6 +304,8 @@ class Engine:
             self.kv_cache = MLALatentCache(self.kv_layers, self.num_pages, self.page_size,
                                            max(mc.latent_widths, default=64), 0, self.dtype, self.device,
                                            widths=mc.latent_widths)
+        elif self._head_geometry:
+            self.kv_cache = LayeredKVCache(self.num_pages, self.page_size, self._head_geometry, self.dtype, self.device)
         else:
             self.kv_cache = MHAKVCache(
                 self.kv_layers, self.num_pages, self.page_size, self.kv_heads_local, mc.head_dim,
@@ -322,7 +325,8 @@ class Engine:
         if self.kv_calibrating:
             self.kv_cache.start_calibration()
             logger.info_rank0("fp8 KV calibration run: 16-bit pool, eager steps")
-        self.ledger.add("kv pool", self.kv_cache._buf.numel() * self.kv_cache._buf.element_size())
+        self.ledger.add("kv pool", self.kv_cache.nbytes if self._head_geometry
+                        else self.kv_cache._buf.numel() * self.kv_cache._buf.element_size())
         if self._swa_layers:
             from ..kvcache.swa_pages import SwaPages
 
@@ -363,6 +367,7 @@ class Engine:
             config.attention_backend, self.q_heads_local, self.kv_heads_local, mc.head_dim, self.device,
             max_batch=config.max_running_req, max_seq_len=self.max_seq_len,
             single_split=config.spec_algorithm != "none", latent=mc.latent_layers,
+            heads=[(div_even(m.heads, config.tp_size), m.row_pad) for m in mc.head_layers],
         )
         self.ctx.comm = comm_mod.get_comm()
         self._spec_exact = config.spec_algorithm != "none" and dev_kind == "cuda"
@@ -483,7 +488,7 @@ class Engine:
                     symm = SymmetricCollectives(self.tp_group, self.cpu_group, self.device, cfg.tp_rank, cfg.tp_size)
                     comm.register(symm)
                     if (not ENV.DISABLE_ROW_SHARD.value and not self.model_config.is_moe
-                            and not self.model_config.latent_layers):
+                            and not self.model_config.has_fp32_kernels):
                         # prefill chunks: GEMM -> reduce-scatter -> add + norm -> all-gather -> GEMM
                         symm.enable_row_shard(int(getattr(cfg, "max_extend_tokens", 8192)),
                                               self.model_config.hidden_size)
@@ -571,6 +576,8 @@ class Engine:
                                                   itemsize) * self.page_size
         if mc.latent_layers:
             per_page = (sum(mc.latent_widths) or 64) * itemsize * self.page_size
+        if self._head_geometry:
+            per_page = LayeredKVCache.token_bytes(self._head_geometry, itemsize) * self.page_size
         if cfg.spec_algorithm in ("eagle3", "mtp"):
             # the draft head keeps one 16-bit, unsharded layer of K/V on the same page table
             per_page += MHAKVCache.token_bytes(1, mc.num_kv_heads, mc.head_dim, 2) * self.page_size
@@ -605,8 +612,8 @@ class Engine:
         cfg, mc = self.config, self.model_config
         limit = cfg.max_seq_len_override or mc.max_position_embeddings
         limit = min(limit, mc.rotary_config.max_position, self.num_pages * self.page_size)
-        if mc.latent_layers:
-            return int(limit)                  # learned positions: every one of them can be used
+        if mc.has_fp32_kernels:
+            return int(limit)                  # every position of the table can be used
         return int(limit // self.page_size * self.page_size) or self.page_size
 
     # ------------------------------------------------------------------ step
@@ -821,7 +828,7 @@ class Engine:
 
     def _row_shard_rows(self, tokens: int) -> bool:
         """Whether a step of ``tokens`` rows takes the row-sharded tensor-parallel path."""
-        if self.config.tp_size == 1 or self.model_config.is_moe or self.model_config.latent_layers:
+        if self.config.tp_size == 1 or self.model_config.is_moe or self.model_config.has_fp32_kernels:
             return False
         for impl in comm_mod.get_comm().impls:
             rs = getattr(impl, "row_shard", None)

@@ -4,7 +4,7 @@ from __future__ import annotations
 from .base import BaseCacheHandle, BaseKVCachePool, BasePrefixCache, SizeInfo
 from .naive_cache import NaivePrefixCache
 from .radix_cache import RadixPrefixCache, SnapshotRadixCache
-from .mha_pool import MHAKVCache
+from .mha_pool import LayeredKVCache, MHAKVCache
 
 
 def create_prefix_cache(kind: str, page_size: int) -> BasePrefixCache:
@@ -26,6 +26,7 @@ __all__ = [
     "NaivePrefixCache",
     "RadixPrefixCache",
     "SnapshotRadixCache",
+    "LayeredKVCache",
     "MHAKVCache",
     "create_prefix_cache",
 ]

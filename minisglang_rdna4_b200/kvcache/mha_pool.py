@@ -152,3 +152,48 @@ class MHAKVCache(BaseKVCachePool):
             scale = (self.k_scale if which == 0 else self.v_scale)[layer]
             return rows.to(torch.float32) * scale[None, :, None]
         return rows
+
+
+class LayeredKVCache(BaseKVCachePool):
+    """Pool of a model whose layers differ in heads and row width: every layer has dense planes of its own, in the page
+    layout of ``MHAKVCache`` (``[2, 1, pages + 1, heads, page_size, width]``). ``geometry``: ``(kv heads, width)`` per
+    layer; 16 or 32 bits."""
+
+    fp8 = False
+
+    def __init__(self, num_pages: int, page_size: int, geometry, dtype: torch.dtype, device) -> None:
+        self.num_layers, self.num_pages, self.page_size = len(geometry), num_pages, page_size
+        self.geometry = [(int(h), int(d)) for h, d in geometry]
+        self._planes = [torch.zeros((2, 1, num_pages + 1, h, page_size, d), dtype=dtype, device=device)
+                        for h, d in self.geometry]
+
+    @staticmethod
+    def token_bytes(geometry, itemsize: int) -> int:
+        return 2 * sum(h * d for h, d in geometry) * itemsize
+
+    @property
+    def nbytes(self) -> int:
+        return sum(p.numel() * p.element_size() for p in self._planes)
+
+    @property
+    def dummy_page(self) -> int:
+        return self.num_pages
+
+    @property
+    def device(self) -> torch.device:
+        return self._planes[0].device
+
+    @property
+    def dtype(self) -> torch.dtype:
+        return self._planes[0].dtype
+
+    def k_cache(self, layer: int) -> torch.Tensor:
+        return self._planes[layer][0, 0]
+
+    def v_cache(self, layer: int) -> torch.Tensor:
+        return self._planes[layer][1, 0]
+
+    def store_kv(self, k: torch.Tensor, v: torch.Tensor, out_loc: torch.Tensor, layer: int) -> None:
+        from ..ops import store_kv
+
+        store_kv(k, v, self.k_cache(layer), self.v_cache(layer), out_loc)

@@ -240,11 +240,10 @@ class MoELayer(BaseOP):
         self.gate.init_dummy(gen, std)
 
 
-class ClampedExperts(BaseOP):
-    """Feed-forward of a model with an fp32 residual stream: routed experts with the clamped activation
-    (``models.config.ExpertSpec``) and, behind a sigmoid gate per token, a shared one. The router (and the shared expert's
-    gate, one more column of it) gives fp32 logits; the weighted sum is fp32 (``forward_partial32``). Under tensor
-    parallelism every rank has a part of every expert's width."""
+class ResidualExperts(BaseOP):
+    """Feed-forward of a model with an fp32 residual stream: routed experts and a shared one (``models.config.ExpertSpec``).
+    The router (and the shared expert's gate, where it has one: one more column of it) gives fp32 logits; the sum is fp32
+    (``forward_partial32``). Under tensor parallelism every rank has a part of every expert's width."""
 
     def __init__(self, spec, width: int, width_pad: int, dtype, device) -> None:
         tp = get_tp_info().size
@@ -256,8 +255,9 @@ class ClampedExperts(BaseOP):
         self._ff = pad(div_even(spec.ff, tp), 16)
         self._out = pad(width, 32)
         self._shared_ff = pad(div_even(spec.shared_ff, tp), 16) if spec.shared_ff else 0
+        self._gated = bool(self._shared_ff and spec.shared_gated)
         # rows: the experts, then the shared expert's gate
-        self.router = torch.empty((pad(spec.experts + (1 if self._shared_ff else 0), 8), width_pad), dtype=dtype, device=device)
+        self.router = torch.empty((pad(spec.experts + int(self._gated), 8), width_pad), dtype=dtype, device=device)
         self.w13 = torch.empty((spec.experts, 2 * self._ff, width_pad), dtype=dtype, device=device)
         self.w2 = torch.empty((spec.experts, self._out, self._ff), dtype=dtype, device=device)
         if self._shared_ff:
@@ -269,23 +269,26 @@ class ClampedExperts(BaseOP):
         logits = ops.gemm(x, self.router, None, torch.float32)
         shared = gate = None
         if self._shared_ff:
-            shared = self.shared_down.forward(ops.clamped_glu(self.shared_up.forward(x), s.shared_limit, s.alpha))
-            gate = logits[:, s.experts]
+            up = self.shared_up.forward(x)
+            shared = self.shared_down.forward(ops.silu_and_mul(up) if s.act == "silu"
+                                              else ops.clamped_glu(up, s.shared_limit, s.alpha))
+            gate = logits[:, s.experts] if self._gated else None
         counts = None
         if x.is_cuda:
             from ..ops import moe_kernels
 
             counts = torch.empty(s.experts, dtype=torch.int32, device=x.device)
-            topk_w, topk_ids = moe_kernels.moe_route(logits[:, :s.experts], s.top, False, "softmax", s.scale, counts,
+            topk_w, topk_ids = moe_kernels.moe_route(logits[:, :s.experts], s.top, False, s.scoring, s.scale, counts,
                                                      groups=s.groups, keep=s.keep)
         elif s.groups > 1:
             from ..ops import ref
 
-            topk_w, topk_ids = ref.moe_route_grouped(logits[:, :s.experts], s.top, False, "softmax", None, s.scale, s.groups,
+            topk_w, topk_ids = ref.moe_route_grouped(logits[:, :s.experts], s.top, False, s.scoring, None, s.scale, s.groups,
                                                      s.keep)
         else:
-            topk_w, topk_ids = ops.moe_route(logits[:, :s.experts], s.top, False, "softmax", None, s.scale)
-        y = ops.experts_partial32(x, self.w13, self.w2, topk_w, topk_ids, s.limit, s.alpha, shared, gate, counts)
+            topk_w, topk_ids = ops.moe_route(logits[:, :s.experts], s.top, False, s.scoring, None, s.scale)
+        y = ops.experts_partial32(x, self.w13, self.w2, topk_w, topk_ids, s.limit, s.alpha, shared, gate, counts, s.act,
+                                  s.on_input)
         return get_comm().all_reduce(y) if get_tp_info().size > 1 else y
 
     def init_dummy(self, gen: torch.Generator, std: float = 0.02) -> None:

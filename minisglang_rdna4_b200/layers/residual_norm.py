@@ -1,6 +1,8 @@
 """Norm of a layer with an fp32 residual stream: residual add and layer norm (no bias) or RMS norm in one pass."""
 from __future__ import annotations
 
+from typing import Optional
+
 import torch
 
 from .. import ops
@@ -8,15 +10,18 @@ from .base import BaseOP
 
 
 class ResidualNorm(BaseOP):
-    """``center``: subtract the mean (layer norm). Outputs have ``out_cols`` columns (zero past the width)."""
+    """``center``: subtract the mean (layer norm). Outputs have ``out_cols`` columns (zero past the width). The norm of a
+    sublayer's output (``post`` of the next one's ``forward``) is one of these that is never called itself."""
 
     def __init__(self, width: int, eps: float, center: bool, dtype, device, out_cols: int) -> None:
         self.weight = torch.empty((width,), dtype=torch.float32, device=device)
         self._eps, self._center, self._dtype, self._cols = eps, center, dtype, out_cols
 
-    def forward(self, x: torch.Tensor, delta):
-        """``(x + delta, norm)``; ``delta`` None: nothing to add."""
-        return ops.add_norm(x, delta, self.weight, self._eps, self._center, self._dtype, self._cols)
+    def forward(self, x: torch.Tensor, delta, post: Optional["ResidualNorm"] = None, mult: float = 1.0):
+        """``(x + delta, norm)``; ``delta`` None: nothing to add. ``post``: ``mult`` times that RMS norm of ``delta`` is
+        what is added."""
+        return ops.add_norm(x, delta, self.weight, self._eps, self._center, self._dtype, self._cols,
+                            None if post is None else post.weight, mult)
 
     def init_dummy(self, gen: torch.Generator, std: float = 0.02) -> None:
         self.weight = torch.ones_like(self.weight)

@@ -74,6 +74,12 @@ def _register_defaults() -> None:
         MODEL_REGISTRY.register("RafodraForCausalLM")(RafodraForCausalLM)
 
 
+    from .zobelorn import ZobelornForCausalLM
+
+    if "ZobelornForCausalLM" not in MODEL_REGISTRY:
+        MODEL_REGISTRY.register("ZobelornForCausalLM")(ZobelornForCausalLM)
+
+
 def create_model(cfg: ModelConfig, dtype: torch.dtype, device):
     """Instantiate the model for ``cfg`` with uninitialised (or meta) parameters."""
     _register_defaults()

@@ -105,21 +105,57 @@ class LinearAttnLayer:
 
 
 @dataclass(frozen=True)
+class HeadLayer:
+    """One layer of grouped-query attention with sizes of its own: ``heads`` query heads over ``kv_heads`` key / value
+    heads, keys of ``dim`` and values of ``vdim`` channels. A row sees the last ``window`` positions (its own included)
+    or, with ``chunk``, the positions of its own block of ``chunk`` that are not ahead of it; 0 = no such limit.
+    ``softcap`` c > 0: scores go through ``c tanh(s / c)``. ``joint_norm``: weighted RMS norms over all query heads and
+    over all key heads together, ahead of the rotation. ``unit_norm``: every query and key head divided by its root mean
+    square after the rotation. ``gate``: a sigmoid gate per output channel. ``kv_from``: the layer whose keys and
+    values are read instead of own ones."""
+
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    rotary: Optional[RotaryConfig] = None
+    window: int = 0
+    chunk: int = 0
+    softcap: float = 0.0
+    joint_norm: bool = False
+    unit_norm: bool = False
+    gate: bool = False
+    kv_from: Optional[int] = None
+
+    @property
+    def row_pad(self) -> int:
+        """Width of a head in the pool and in the kernels (keys, values and queries alike), zeros past its channels."""
+        n = max(self.dim, self.vdim)
+        return next((p for p in (64, 128, 256) if n <= p), _round_up(n, 256))
+
+
+@dataclass(frozen=True)
 class ExpertSpec:
-    """A mixture of ``experts`` feed-forwards of width ``ff`` of which each token uses ``top``, chosen among the best
-    ``keep`` of ``groups`` groups; ``shared_ff`` > 0: a further one for every token behind a sigmoid gate. Expert
-    activation: gate and up halves clamped at ``limit``, ``g * sigmoid(alpha g) * (u + 1)``."""
+    """A mixture of ``experts`` feed-forwards of width ``ff`` of which each token uses ``top``, chosen by ``scoring`` among
+    the best ``keep`` of ``groups`` groups; ``shared_ff`` > 0: a further one for every token, behind a sigmoid gate with
+    ``shared_gated``. Activation: silu-gated, or with ``act`` "clamped" gate and up halves clamped at ``limit``,
+    ``g * sigmoid(alpha g) * (u + 1)``. ``on_input``: a chosen expert's weight multiplies what goes into it."""
 
     experts: int
     top: int
     ff: int
-    limit: float
+    limit: float = 0.0
     groups: int = 1
     keep: int = 1
     scale: float = 1.0
     shared_ff: int = 0
     shared_limit: float = 0.0
     alpha: float = 1.702
+    act: str = "clamped"
+    scoring: str = "softmax"
+    on_input: bool = False
+    shared_gated: bool = True
 
 
 @dataclass(frozen=True)
@@ -127,7 +163,7 @@ class LayerSpec:
     """A sequential layer of a model whose layers are listed one by one: a mixer, and a feed-forward that is dense and
     gated (``ff`` > 0), a mixture of experts (``moe``) or absent."""
 
-    mixer: Any                              # LatentLayer | LinearAttnLayer
+    mixer: Any                              # LatentLayer | LinearAttnLayer | HeadLayer
     ff: int = 0
     moe: Optional[ExpertSpec] = None
 
@@ -196,6 +232,7 @@ class ModelConfig:
     # models whose layers are described one by one (mixer and feed-forward of different kinds and sizes)
     layer_specs: Optional[Tuple[LayerSpec, ...]] = None
     embedding_multiplier: float = 1.0
+    residual_multiplier: float = 1.0        # of a sublayer's output where it joins the residual stream
     # misc
     sliding_window: Optional[int] = None
     layer_types: Optional[Tuple[str, ...]] = None
@@ -259,6 +296,27 @@ class ModelConfig:
         return sum(1 for s in specs[:owner] if s is not None and s.kv_from is None)
 
     @property
+    def head_layers(self) -> Tuple[HeadLayer, ...]:
+        """The layers of a model whose attention layers each have a geometry of their own."""
+        mixers = tuple(s.mixer for s in self.layer_specs or ())
+        return mixers if mixers and all(isinstance(m, HeadLayer) for m in mixers) else ()
+
+    def head_geometry(self, tp: int = 1) -> Tuple[Tuple[int, int], ...]:
+        """``(kv heads of a rank, row width)`` of every layer with keys and values of its own, in layer order."""
+        return tuple((max(m.kv_heads // tp, 1), m.row_pad) for m in self.head_layers if m.kv_from is None)
+
+    def head_row(self, layer: int) -> int:
+        """Index in the pool of the layer whose keys and values ``layer`` reads."""
+        mixers = self.head_layers
+        owner = layer if mixers[layer].kv_from is None else mixers[layer].kv_from
+        return sum(1 for m in mixers[:owner] if m.kv_from is None)
+
+    @property
+    def has_fp32_kernels(self) -> bool:
+        """Every kernel the model runs on a GPU has an fp32 form."""
+        return bool(self.latent_layers or self.head_layers)
+
+    @property
     def is_recurrent(self) -> bool:
         """Some layers keep a recurrent state (or a convolution tail) per request besides or instead of K/V pages."""
         return (self.input_conv_taps > 0 or bool(self.linear_layers)
@@ -293,6 +351,8 @@ class ModelConfig:
         """Layers that keep K/V pages."""
         if self.latent_layers:
             return len(self.latent_widths)
+        if self.head_layers:
+            return len(self.head_geometry())
         if self.model_type == "nemotron_h":
             return sum(1 for t in (self.layer_types or ()) if t == "attention")
         return self.num_layers - self.num_linear_layers - self.num_kv_shared_layers
@@ -394,6 +454,8 @@ class ModelConfig:
             return _mitilix_config(cfg)
         if cfg.get("architecture") == "Rafodra":
             return _rafodra_config(cfg, folder)
+        if cfg.get("architecture") == "Zobelorn":
+            return _zobelorn_config(cfg)
         vision = None
         if "text_config" in cfg and isinstance(cfg["text_config"], dict):
             if str(cfg.get("model_type", "")).startswith("gemma3") and cfg.get("vision_config"):
@@ -750,6 +812,86 @@ def layered_config(specs, width: int, vocab: int, eps: float, embedding_multipli
         rms_norm_eps=eps, rotary_config=RotaryConfig(row, 0, max_positions, base=10000.0), model_type="rafodra",
         architectures=("RafodraForCausalLM",), latent_layers=latent, layer_specs=tuple(specs), linear_conv_kernel_dim=1,
         embedding_multiplier=embedding_multiplier, max_position_embeddings=max_positions, eos_token_ids=eos_token_ids,
+        bos_token_id=bos_token_id)
+
+
+def _head_mixer(i: int, kind: str, mix: Dict[str, Any], specs: List[LayerSpec], max_pos: int) -> HeadLayer:
+    rot, size = mix.get("rot") or {}, int((mix.get("mask") or {}).get("size") or 0)
+    dim, dims = int(mix["dim"]), int(rot.get("dims", 0))
+    if dims % 2 or not 0 <= dims <= dim:
+        raise ValueError(f"layer {i}: {dims} rotated of {dim} channels")
+    windowed, scaling = kind == "attention", rot.get("scaling")
+    if scaling and windowed:
+        scaling = {"rope_type": "linear", "factor": float(scaling["factor"])}
+    elif scaling:
+        scaling = {"rope_type": "llama3", "factor": float(scaling["factor"]), "low_freq_factor": float(scaling["low"]),
+                   "high_freq_factor": float(scaling["high"]),
+                   "original_max_position_embeddings": float(scaling["original"])}
+    rotary = RotaryConfig(dim, dims, max_pos, float(rot["base"]), scaling or None, interleaved=not windowed) if dims else None
+    spec = HeadLayer(
+        heads=int(mix["heads"]), kv_heads=int(mix["kv_heads"]), dim=dim, vdim=int(mix["vdim"]), scale=float(mix["scale"]),
+        rotary=rotary, window=size if windowed else 0, chunk=0 if windowed else size,
+        softcap=float(mix.get("softcap") or 0.0) if windowed else 0.0, joint_norm=windowed, unit_norm=not windowed,
+        gate=windowed, kv_from=None if mix.get("kv_from") is None else int(mix["kv_from"]))
+    if spec.heads % spec.kv_heads:
+        raise ValueError(f"layer {i}: {spec.heads} query heads over {spec.kv_heads} key / value heads")
+    if spec.kv_from is not None:
+        donor = specs[spec.kv_from].mixer if 0 <= spec.kv_from < i else None
+        if donor is None or donor.kv_from is not None or any(
+                getattr(donor, f) != getattr(spec, f)
+                for f in ("kv_heads", "dim", "vdim", "rotary", "joint_norm", "unit_norm")):
+            raise ValueError(f"layer {i}: kv_from {spec.kv_from} names no earlier layer with keys and values of this kind")
+    return spec
+
+
+def _zobelorn_config(cfg: Dict[str, Any]) -> ModelConfig:
+    """``layers`` lists every layer's mixer ("attention": sliding window; "attention_2": chunks) and feed-forward with
+    sizes of their own."""
+    max_pos = int(cfg.get("max_positions") or 131072)      # the design sets no limit: one for tables and buffers
+    specs: List[LayerSpec] = []
+    for i, layer in enumerate(cfg["layers"]):
+        kind, mix, mlp = layer["type"], layer["mixer"], layer.get("mlp")
+        if kind not in ("attention", "attention_2"):
+            raise ValueError(f"layer {i}: unknown mixer type {kind!r}")
+        mixer = _head_mixer(i, kind, mix, specs, max_pos)
+        ff, moe = 0, None
+        if mlp is not None and mlp["kind"] == "dense":
+            ff = int(mlp["ff"])
+        elif mlp is not None and mlp["kind"] == "moe":
+            router, shared = mlp["router"], mlp.get("shared")
+            moe = ExpertSpec(experts=int(router["experts"]), top=int(router["top"]), ff=int(mlp["expert"]["ff"]),
+                             shared_ff=int(shared["ff"]) if shared else 0, act="silu", scoring="sigmoid", on_input=True,
+                             shared_gated=False)
+            if not 0 < moe.top <= moe.experts:
+                raise ValueError(f"layer {i}: {moe.top} of {moe.experts} experts")
+        elif mlp is not None:
+            raise ValueError(f"layer {i}: unknown feed-forward kind {mlp['kind']!r}")
+        specs.append(LayerSpec(mixer, ff, moe))
+    eos = cfg.get("eos_token_id")
+    eos_ids = tuple(eos) if isinstance(eos, (list, tuple)) else (() if eos is None else (int(eos),))
+    return heads_config(specs, width=int(cfg["width"]), vocab=int(cfg["vocab"]), eps=float(cfg["norm"]["eps"]),
+                        embedding_multiplier=float(cfg["embedding"]["scale"]),
+                        residual_multiplier=float(cfg["residual_mult"]), max_positions=max_pos, eos_token_ids=eos_ids,
+                        bos_token_id=cfg.get("bos_token_id"))
+
+
+def heads_config(specs, width: int, vocab: int, eps: float, embedding_multiplier: float = 1.0,
+                 residual_multiplier: float = 1.0, max_positions: int = 131072, eos_token_ids: Tuple[int, ...] = (),
+                 bos_token_id=None) -> ModelConfig:
+    """A Zobelorn configuration from its layers."""
+    first: HeadLayer = specs[0].mixer
+
+    def widest(s: LayerSpec) -> int:        # activations of one token
+        m: HeadLayer = s.mixer
+        mix = (2 * m.heads + 2 * m.kv_heads) * m.row_pad
+        return max(mix, s.ff, s.moe.top * s.moe.ff + s.moe.shared_ff if s.moe else 0)
+
+    return ModelConfig(
+        num_layers=len(specs), num_qo_heads=first.heads, num_kv_heads=first.kv_heads, head_dim=first.row_pad,
+        hidden_size=width, vocab_size=vocab, intermediate_size=max(widest(s) for s in specs), rms_norm_eps=eps,
+        rotary_config=RotaryConfig(first.row_pad, 0, max_positions, base=10000.0), model_type="zobelorn",
+        architectures=("ZobelornForCausalLM",), layer_specs=tuple(specs), embedding_multiplier=embedding_multiplier,
+        residual_multiplier=residual_multiplier, max_position_embeddings=max_positions, eos_token_ids=eos_token_ids,
         bos_token_id=bos_token_id)
 
 

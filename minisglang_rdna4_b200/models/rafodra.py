@@ -18,31 +18,18 @@ import torch
 from .. import ops
 from ..core import get_global_ctx
 from ..layers import BaseOP, ParallelLMHead, ReplicatedLinear, RowParallelLinear, VocabParallelEmbedding
+from ..layers.gated_mlp import DenseGatedMLP
 from ..layers.latent_attention import LatentAttentionLayer
 from ..layers.linear_attention import LinearAttentionLayer
-from ..layers.moe import ClampedExperts
+from ..layers.moe import ResidualExperts
 from ..layers.residual_norm import ResidualNorm
 from ..parallel.comm import get_comm
 from ..parallel.info import get_tp_info
-from ..utils import div_even
 from .config import LatentLayer, ModelConfig
 
 
 def _pad16(n: int) -> int:
     return (n + 15) // 16 * 16
-
-
-class DenseGatedMLP(BaseOP):
-    """silu-gated feed-forward with an fp32 result."""
-
-    def __init__(self, ff: int, width_pad: int, dtype, device) -> None:
-        tp = get_tp_info().size
-        self._ff = _pad16(div_even(ff, tp))
-        self.gate_up = ReplicatedLinear(width_pad, 2 * self._ff, dtype, device)
-        self.down = RowParallelLinear(self._ff * tp, width_pad, dtype, device)
-
-    def forward_partial32(self, x: torch.Tensor):
-        return self.down.forward_partial32(ops.silu_and_mul(self.gate_up.forward(x)))
 
 
 class RafodraLayer(BaseOP):
@@ -59,7 +46,7 @@ class RafodraLayer(BaseOP):
         self._has_mlp = bool(spec.ff or spec.moe)
         if self._has_mlp:
             self.norm2 = ResidualNorm(w, cfg.rms_norm_eps, True, dtype, device, wp)
-            self.mlp = (ClampedExperts(spec.moe, w, wp, dtype, device) if spec.moe is not None
+            self.mlp = (ResidualExperts(spec.moe, w, wp, dtype, device) if spec.moe is not None
                         else DenseGatedMLP(spec.ff, wp, dtype, device))
 
     def forward(self, x: torch.Tensor, delta):

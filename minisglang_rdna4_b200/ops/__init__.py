@@ -102,6 +102,19 @@ def qk_norm_rope_store(qkv, q_w, k_w, positions, cos_sin, num_q_heads: int, num_
     return q.reshape(-1, num_q_heads, head_dim)
 
 
+def heads_rope_store(x, heads: int, kv_heads: int, width: int, dim: int, positions, cos_sin, interleaved: bool,
+                     eps: float, q_w=None, k_w=None, totals=None, unit: bool = False, store=None):
+    """Norms and rotation of projected query and key heads, and the store of keys and values, in one pass.
+
+    ``x [T, ld]``: ``heads`` queries and, with ``store = (k_cache, v_cache, out_loc)``, ``kv_heads`` keys and as many
+    values, each ``width`` columns of which ``dim`` count (values may use more). ``q_w`` / ``k_w`` (fp32, as wide as the
+    columns): RMS norm over all heads together first; ``totals = (sums [T, 2], q count, k count)`` where other ranks hold
+    some of them. Then the rotation (``cos_sin`` None: none), then, with ``unit``, every head divided by its root mean
+    square. Returns the queries ``[T, heads, width]``."""
+    fn = _cuda().heads_rope_store if x.is_cuda else ref.heads_rope_store
+    return fn(x, heads, kv_heads, width, dim, positions, cos_sin, interleaved, eps, q_w, k_w, totals, unit, store)
+
+
 def q_norm_rope(q, q_w, positions, cos_sin, num_q_heads: int, head_dim: int, rotary_dim: int, eps: float,
                 interleaved: bool = False):
     """Per-head RMSNorm + rotary embedding of the queries alone ``[T, Hq * D]`` → ``[T, Hq, D]``: the form a
@@ -121,14 +134,16 @@ def store_kv(k, v, k_cache, v_cache, out_loc, k_scale=None, v_scale=None):
 
 def paged_attention(q, k_cache, v_cache, block_table, cu_q, seq_lens, scale: float, *, causal: bool = True,
                     window: int = 0, mask=None, k_scale=None, v_scale=None, max_q: int = 0,
-                    max_kv: int = 0, decode: bool = False, workspace=None, splits=None, mask_window: int = 0):
+                    max_kv: int = 0, decode: bool = False, workspace=None, splits=None, mask_window: int = 0,
+                    chunk: int = 0, softcap: float = 0.0, gate=None):
     if q.is_cuda:
         return _cuda().paged_attention(q, k_cache, v_cache, block_table, cu_q, seq_lens, scale,
                                        causal=causal, window=window, mask=mask, k_scale=k_scale,
                                        v_scale=v_scale, max_q=max_q, max_kv=max_kv, decode=decode,
-                                       workspace=workspace, splits=splits, mask_window=mask_window)
+                                       workspace=workspace, splits=splits, mask_window=mask_window, chunk=chunk,
+                                       softcap=softcap, gate=gate)
     return ref.paged_attention(q, k_cache, v_cache, block_table, cu_q, seq_lens, scale, causal, window,
-                               mask, k_scale, v_scale, mask_window)
+                               mask, k_scale, v_scale, mask_window, chunk, softcap, gate)
 
 
 # ---------------------------------------------------------------------------- GEMMs
@@ -262,12 +277,13 @@ def latent_attention(q, rows, block_table, cu_q, seq_lens, scale: float, window:
 
 
 # ---------------------------------------------------------------------------- weighted norm, decaying linear attention
-def add_norm(x, delta, weight, eps: float, center: bool, out_dtype, out_cols: int):
+def add_norm(x, delta, weight, eps: float, center: bool, out_dtype, out_cols: int, post=None, mult: float = 1.0):
     """Residual add and norm (layer norm without a bias, or RMS) in one pass: ``(new residual, y)``. ``delta`` may be
-    the unreduced K ranges of a GEMM (``SplitPartial``)."""
+    the unreduced K ranges of a GEMM (``SplitPartial``). ``post``: weight of an RMS norm that ``delta`` takes before it
+    is multiplied by ``mult`` and added."""
     if x.is_cuda:
-        return _cuda().add_norm(x, delta, weight, eps, center, out_dtype, out_cols)
-    return ref.add_norm(x, delta, weight, eps, center, out_dtype, out_cols)
+        return _cuda().add_norm(x, delta, weight, eps, center, out_dtype, out_cols, post, mult)
+    return ref.add_norm(x, delta, weight, eps, center, out_dtype, out_cols, post, mult)
 
 
 def linear_attention(q, k, v, state, cu_q, slots, has_state, decay=None, gate=None, tau: float = 1.0,
@@ -313,13 +329,15 @@ def moe_route(router_logits, top_k: int, renormalize: bool, scoring: str = "soft
 
 
 def experts_partial32(x, w13, w2, topk_w, topk_ids, limit: float, alpha: float, shared=None, shared_gate=None,
-                      counts=None):
-    """fp32 sum of the routed clamped experts and a gated shared one, for an fp32 residual stream."""
+                      counts=None, act: str = "clamped", on_input: bool = False):
+    """fp32 sum of the routed experts and a shared one (behind the sigmoid of ``shared_gate`` where given), for an fp32
+    residual stream. ``on_input``: the weights multiply the experts' inputs."""
     if x.is_cuda:
         from . import moe_kernels
 
-        return moe_kernels.experts_partial32(x, w13, w2, topk_w, topk_ids, limit, alpha, shared, shared_gate, counts)
-    return ref.experts_partial32(x, w13, w2, topk_w, topk_ids, limit, alpha, shared, shared_gate)
+        return moe_kernels.experts_partial32(x, w13, w2, topk_w, topk_ids, limit, alpha, shared, shared_gate, counts, act,
+                                             on_input)
+    return ref.experts_partial32(x, w13, w2, topk_w, topk_ids, limit, alpha, shared, shared_gate, act, on_input)
 
 
 def moe_forward(x, w13, w2, topk_w, topk_ids, expert_offset: int = 0):

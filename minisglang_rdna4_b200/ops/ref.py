@@ -207,7 +207,8 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
                     block_table: torch.Tensor, cu_q: torch.Tensor, seq_lens: torch.Tensor,
                     scale: float, causal: bool = True, window: int = 0,
                     mask: Optional[torch.Tensor] = None, k_scale: Optional[torch.Tensor] = None,
-                    v_scale: Optional[torch.Tensor] = None, mask_window: int = 0) -> torch.Tensor:
+                    v_scale: Optional[torch.Tensor] = None, mask_window: int = 0, chunk: int = 0, softcap: float = 0.0,
+                    gate: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Attention of packed queries over paged KV.
 
     ``q`` ``[T, Hq, D]``; request ``b`` owns rows ``cu_q[b]:cu_q[b+1]`` which are the LAST
@@ -218,6 +219,8 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
     With ``mask_window`` > 0 the mask is ``[T, mask_window]`` and covers only the last
     ``mask_window`` KV positions of each request; earlier positions are visible to every row
     (of a sliding-window layer: to the rows that have them inside their window).
+    ``chunk`` > 0: a row sees its own block of ``chunk`` positions only. ``softcap`` c > 0: ``c tanh(score / c)``.
+    ``gate [T, Hq * D]``: the output is multiplied by its sigmoid.
     """
     t, hq, d = q.shape
     hk, ps = k_cache.shape[1], k_cache.shape[2]
@@ -240,6 +243,8 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
         qq = q[qs:qe].float().permute(1, 0, 2).reshape(hk, group * q_len, d)  # head h -> kv h//group
         qq = q[qs:qe].float().view(q_len, hk, group, d).permute(1, 2, 0, 3)    # [hk, g, q, d]
         s = torch.einsum("hgqd,hkd->hgqk", qq, kk) * scale
+        if softcap > 0:
+            s = softcap * torch.tanh(s / softcap)
         q_pos = torch.arange(kv_len - q_len, kv_len, device=q.device)[:, None]
         k_pos = torch.arange(kv_len, device=q.device)[None, :]
         if mask is not None and mask_window:
@@ -257,11 +262,41 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
                 s = s.masked_fill((k_pos > q_pos)[None, None], float("-inf"))
             if window and window > 0:
                 s = s.masked_fill((k_pos <= q_pos - window)[None, None], float("-inf"))
+            if chunk > 0:
+                s = s.masked_fill((k_pos < q_pos - q_pos % chunk)[None, None], float("-inf"))
         p = torch.softmax(s, dim=-1)
         p = torch.nan_to_num(p, nan=0.0)
         o = torch.einsum("hgqk,hkd->hgqd", p, vv)  # [hk, g, q, d]
         out[qs:qe] = o.permute(2, 0, 1, 3).reshape(q_len, hq, d)
+    if gate is not None:
+        out = out * torch.sigmoid(gate.float()).view(t, hq, d)
     return out.to(q.dtype)
+
+
+def heads_rope_store(x: torch.Tensor, heads: int, kv_heads: int, width: int, dim: int, positions: torch.Tensor,
+                     cos_sin: Optional[torch.Tensor], interleaved: bool, eps: float, q_w: Optional[torch.Tensor] = None,
+                     k_w: Optional[torch.Tensor] = None, totals=None, unit: bool = False, store=None) -> torch.Tensor:
+    t = x.shape[0]
+
+    def turn(y, n, w, col):
+        y = y.float()
+        if w is not None:
+            ss, count = (y.pow(2).sum(-1), n * dim) if totals is None else (totals[0][:, col], totals[1 + col])
+            y = y * torch.rsqrt(ss / count + eps)[:, None] * w.float()
+        y = y.reshape(t, n, width)
+        if cos_sin is not None:
+            rot = cos_sin.shape[1]
+            cs = cos_sin[positions.long()].float()
+            y = torch.cat([_rotate(y[..., :rot], cs[:, :rot // 2], cs[:, rot // 2:], interleaved), y[..., rot:]], -1)
+        if unit:
+            y = y * torch.rsqrt(y.pow(2).sum(-1, keepdim=True) / dim + eps)
+        return y.to(x.dtype)
+
+    nq, nk = heads * width, kv_heads * width
+    if store is not None:
+        k_cache, v_cache, out_loc = store
+        store_kv(turn(x[:, nq:nq + nk], kv_heads, k_w, 1), x[:, nq + nk:nq + 2 * nk], k_cache, v_cache, out_loc)
+    return turn(x[:, :nq], heads, q_w, 0)
 
 
 def mla_attention(q_lat: torch.Tensor, q_rot: torch.Tensor, rows: torch.Tensor, block_table: torch.Tensor,
@@ -739,9 +774,15 @@ def latent_attention(q: torch.Tensor, rows: torch.Tensor, block_table: torch.Ten
 # fp32 residual stream with a weighted norm; decaying linear attention; clamped experts
 # ------------------------------------------------------------------------------------------
 def add_norm(x: torch.Tensor, delta: Optional[torch.Tensor], weight: torch.Tensor, eps: float, center: bool,
-             out_dtype: torch.dtype, out_cols: int) -> Tuple[torch.Tensor, torch.Tensor]:
-    """``x += delta`` (fp32); layer norm without a bias (``center``) or RMS norm. Returns ``(x, y [T, out_cols])``."""
-    xn = x if delta is None else x + delta[:, :x.shape[1]].float()
+             out_dtype: torch.dtype, out_cols: int, post: Optional[torch.Tensor] = None,
+             mult: float = 1.0) -> Tuple[torch.Tensor, torch.Tensor]:
+    """``x += delta`` (fp32; with ``post`` ``mult`` times the RMS norm of ``delta`` with that weight); layer norm without
+    a bias (``center``) or RMS norm. Returns ``(x, y [T, out_cols])``."""
+    if delta is not None:
+        delta = delta[:, :x.shape[1]].float()
+    if post is not None:
+        delta = delta * torch.rsqrt(delta.pow(2).mean(-1, keepdim=True) + eps) * post.float() * mult
+    xn = x if delta is None else x + delta
     d = xn - xn.mean(-1, keepdim=True) if center else xn
     y = d * torch.rsqrt(d.pow(2).mean(-1, keepdim=True) + eps) * weight[:x.shape[1]].float()
     return xn, F.pad(y, (0, out_cols - y.shape[1])).to(out_dtype)
@@ -800,14 +841,22 @@ def clamped_glu(x: torch.Tensor, limit: float, alpha: float) -> torch.Tensor:
 
 def experts_partial32(x: torch.Tensor, w13: torch.Tensor, w2: torch.Tensor, topk_w: torch.Tensor,
                       topk_ids: torch.Tensor, limit: float, alpha: float, shared: Optional[torch.Tensor] = None,
-                      shared_gate: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """fp32 ``sum_k w_k * expert_k(x) + sigmoid(shared_gate) * shared`` with clamped experts."""
+                      shared_gate: Optional[torch.Tensor] = None, act: str = "clamped",
+                      on_input: bool = False) -> torch.Tensor:
+    """fp32 ``sum_k w_k * expert_k(x) + sigmoid(shared_gate) * shared`` (no gate: the shared rows as they are), or
+    ``sum_k expert_k(w_k * x) + ...`` with ``on_input``; clamped or silu-gated experts."""
     out = torch.zeros(x.shape[0], w2.shape[1], dtype=torch.float32, device=x.device)
     if shared is not None:
-        out[:, :shared.shape[1]] += shared.float() * torch.sigmoid(shared_gate.float())[:, None]
+        g = 1.0 if shared_gate is None else torch.sigmoid(shared_gate.float())[:, None]
+        out[:, :shared.shape[1]] += shared.float() * g
     for e in range(w13.shape[0]):
         rows, slot = (topk_ids == e).nonzero(as_tuple=True)
         if rows.numel():
-            y = clamped_glu((x[rows].float() @ w13[e].float().t()).to(x.dtype), limit, alpha)
-            out.index_add_(0, rows, (y.float() @ w2[e].float().t()).to(x.dtype).float() * topk_w[rows, slot][:, None])
+            weight, xe = topk_w[rows, slot][:, None], x[rows].float()
+            if on_input:
+                xe = (xe * weight).to(x.dtype).float()
+            h = (xe @ w13[e].float().t()).to(x.dtype)
+            y = silu_and_mul(h) if act == "silu" else clamped_glu(h, limit, alpha)
+            y = (y.float() @ w2[e].float().t()).to(x.dtype).float()
+            out.index_add_(0, rows, y if on_input else y * weight)
     return out

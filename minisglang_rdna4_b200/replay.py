@@ -124,7 +124,7 @@ def main(argv: Optional[Sequence[str]] = None) -> int:
     from .models.config import ModelConfig
 
     mc = ModelConfig.from_hf(args.model)
-    if args.dtype == "float32" and args.device == "cuda" and not mc.latent_layers:
+    if args.dtype == "float32" and args.device == "cuda" and not mc.has_fp32_kernels:
         print(f"trace_run: {mc.model_type} has no 32-bit kernels", file=sys.stderr)
         return 3
     if args.device == "cuda":
@@ -132,8 +132,9 @@ def main(argv: Optional[Sequence[str]] = None) -> int:
         from .ops import _lib
 
         if not os.path.exists(_lib.LIB_PATH):
-            if mc.latent_layers:
-                _lib.use_part(build.build_cuda(part="layered" if mc.layer_specs else "latent"))
+            if mc.has_fp32_kernels:
+                part = "heads" if mc.head_layers else "layered" if mc.layer_specs else "latent"
+                _lib.use_part(build.build_cuda(part=part))
             else:
                 build.build_cuda()
     torch.backends.cuda.matmul.allow_tf32 = False
