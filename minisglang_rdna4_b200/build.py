@@ -74,6 +74,8 @@ PARTS = {
     "latent": ["elementwise", "gemm_tcgen05", "gemm_f32", "norm_conv", "latent_attention", "attention_tc", "sampling"],
     "layered": ["elementwise", "gemm_tcgen05", "gemm_f32", "norm_conv", "residual_norm", "latent_attention",
                 "attention_tc", "linear_attention", "moe", "sampling"],
+    "heads": ["elementwise", "gemm_tcgen05", "gemm_f32", "norm_conv", "residual_norm", "rope_kv", "attention",
+              "attention_f32", "attention_tc", "moe", "sampling"],
 }
 
 

@@ -49,9 +49,21 @@ struct AttnArgs {
   int causal, window, splits, total_q;
   float scale;
   int* status;
+  int chunk;         // > 0: a row sees its own block of this many positions only
+  float softcap;     // c > 0: scores go through c tanh(s / c)
+  const void* gate;  // [rows, Hq * D] logits of a sigmoid on the output (row stride ldg), or null
+  long long ldg;
 };
 
 __device__ int g_attn_status = 0;
+
+// first position that a row at pos can see
+__device__ __forceinline__ int first_visible(const AttnArgs& a, int pos) {
+  int lo = 0;
+  if (a.window > 0) lo = max(lo, pos - a.window + 1);
+  if (a.chunk > 0) lo = max(lo, pos - pos % a.chunk);
+  return lo;
+}
 
 __device__ __forceinline__ void ldmatrix_x4(uint32_t addr, uint32_t (&r)[4]) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
@@ -81,6 +93,15 @@ __device__ __forceinline__ float fast_exp2(float x) {
   float y;
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
+}
+// cap_out tanh(x) with cap_in s = 2 x log2(e): tanh(x) = 1 - 2 / (1 + e^(2x))
+__device__ __forceinline__ float cap_score(float s, float cap_in, float cap_out) {
+  return fmaf(-2.f * cap_out, __fdividef(1.f, 1.f + fast_exp2(s * cap_in)), cap_out);
+}
+// sigmoid of two neighbouring gate logits times (a, b)
+template <typename T> __device__ __forceinline__ void gate2(const T* g, float& a, float& b) {
+  a *= __fdividef(1.f, 1.f + fast_exp2(-kLog2e * to_float(g[0])));
+  b *= __fdividef(1.f, 1.f + fast_exp2(-kLog2e * to_float(g[1])));
 }
 __device__ __forceinline__ uint32_t pack_f16x2(float a, float b) {
   __half2 h = __floats2half2_rn(a, b);
@@ -138,7 +159,7 @@ paged_attention_kernel(const __grid_constant__ CUtensorMap kv_map, const AttnArg
   const bool use_mask = args.mask != nullptr;
   int kv_hi = (args.causal && !use_mask) ? min(kv_len, kv_len - q_len + q_end) : kv_len;
   int kv_lo = 0;
-  if (args.window > 0 && !use_mask) kv_lo = max(0, (kv_len - q_len + q_start) - args.window + 1);
+  if (!use_mask) kv_lo = first_visible(args, kv_len - q_len + q_start);
   const int tile_lo = kv_lo / TK;
   const int n_tiles_all = kv_hi > kv_lo ? (kv_hi + TK - 1) / TK - tile_lo : 0;
   const int per_split = (n_tiles_all + args.splits - 1) / args.splits;
@@ -235,13 +256,16 @@ paged_attention_kernel(const __grid_constant__ CUtensorMap kv_map, const AttnArg
 
   const float k_sc = args.k_scale != nullptr ? args.k_scale[h] : 1.f;
   const float v_sc = args.v_scale != nullptr ? args.v_scale[h] : 1.f;
-  const float sm_scale = args.scale * k_sc * kLog2e;
+  const bool capped = args.softcap > 0.f;
+  const float sm_scale = capped ? 1.f : args.scale * k_sc * kLog2e;
+  const float cap_in = capped ? 2.f * kLog2e * args.scale * k_sc / args.softcap : 0.f, cap_out = args.softcap * kLog2e;
   // per-row visible KV interval [lo, hi)
   const int pos_a = kv_len - q_len + qi_a, pos_b = kv_len - q_len + qi_b;
   int hi_a = kv_len, hi_b = kv_len, lo_a = 0, lo_b = 0;
   if (!use_mask) {
     if (args.causal) { hi_a = min(kv_len, pos_a + 1); hi_b = min(kv_len, pos_b + 1); }
-    if (args.window > 0) { lo_a = max(0, pos_a - args.window + 1); lo_b = max(0, pos_b - args.window + 1); }
+    lo_a = first_visible(args, pos_a);
+    lo_b = first_visible(args, pos_b);
   }
   if (!ok_a) hi_a = 0;
   if (!ok_b) hi_b = 0;
@@ -294,6 +318,12 @@ paged_attention_kernel(const __grid_constant__ CUtensorMap kv_map, const AttnArg
       }
     }
 
+    if (capped) {
+#pragma unroll
+      for (int nb = 0; nb < TK / 8; ++nb)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) s[nb][e] = cap_score(s[nb][e], cap_in, cap_out);
+    }
     // ---- scale, mask, online softmax (base-2)
     float mx_a = -INFINITY, mx_b = -INFINITY;
 #pragma unroll
@@ -450,6 +480,15 @@ paged_attention_kernel(const __grid_constant__ CUtensorMap kv_map, const AttnArg
   if (args.splits == 1) {
     T* oa = reinterpret_cast<T*>(args.out) + qoff_a;
     T* ob = reinterpret_cast<T*>(args.out) + qoff_b;
+    if (!KV8 && args.gate != nullptr) {
+      const T* ga = reinterpret_cast<const T*>(args.gate) + (q_begin + (ok_a ? qi_a : q_start)) * args.ldg + head_a * D + 2 * j;
+      const T* gb = reinterpret_cast<const T*>(args.gate) + (q_begin + (ok_b ? qi_b : q_start)) * args.ldg + head_b * D + 2 * j;
+#pragma unroll
+      for (int i = 0; i < NDB; ++i) {
+        gate2(ga + i * 8, o[i][0], o[i][1]);
+        gate2(gb + i * 8, o[i][2], o[i][3]);
+      }
+    }
     if (KV8) {
 #pragma unroll
       for (int c = 0; c < D / 16; ++c) {
@@ -499,7 +538,8 @@ paged_attention_kernel(const __grid_constant__ CUtensorMap kv_map, const AttnArg
 template <typename T, int D>
 __global__ void attn_combine_kernel(const float* __restrict__ ws_o, const float* __restrict__ ws_lse,
                                     T* __restrict__ out, int rows_heads, int splits,
-                                    const int32_t* __restrict__ cu_q, int B, int hq) {
+                                    const int32_t* __restrict__ cu_q, int B, int hq, const T* __restrict__ gate,
+                                    long long ldg) {
   pdl_enter();
   const int idx = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
   if (idx >= rows_heads) return;
@@ -531,6 +571,11 @@ __global__ void attn_combine_kernel(const float* __restrict__ ws_o, const float*
   }
   const float inv = wsum > 0.f ? 1.f / wsum : 0.f;
   T* dst = out + (size_t)idx * D + lane * PER;
+  if (gate != nullptr) {
+    const T* g = gate + (idx / hq) * ldg + (idx % hq) * D + lane * PER;
+#pragma unroll
+    for (int i = 0; i < PER; i += 2) gate2(g + i, acc[i], acc[i + 1]);
+  }
 #pragma unroll
   for (int i = 0; i < PER; ++i) dst[i] = from_float<T>(acc[i] * inv);
 }
@@ -583,7 +628,7 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap kv_map, const AttnArgs a
   const int q_row = args.cu_q[b];
   const int kv_len = args.seq_lens[b];
   const int kv_hi = kv_len;
-  const int kv_lo = args.window > 0 ? max(0, kv_len - args.window) : 0;
+  const int kv_lo = first_visible(args, kv_len - 1);
   const int tile_lo = kv_lo / TK;
   const int n_tiles_all = kv_hi > kv_lo ? (kv_hi + TK - 1) / TK - tile_lo : 0;
   const int per_split = (n_tiles_all + args.splits - 1) / args.splits;
@@ -669,7 +714,9 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap kv_map, const AttnArgs a
   }
   const float k_sc = args.k_scale != nullptr ? args.k_scale[h] : 1.f;
   const float v_sc = args.v_scale != nullptr ? args.v_scale[h] : 1.f;
-  const float sm_scale = args.scale * k_sc * kLog2e;
+  const bool capped = args.softcap > 0.f;
+  const float sm_scale = capped ? 1.f : args.scale * k_sc * kLog2e;
+  const float cap_in = capped ? 2.f * kLog2e * args.scale * k_sc / args.softcap : 0.f, cap_out = args.softcap * kLog2e;
 
   float ot[NMB][4];
 #pragma unroll
@@ -710,6 +757,12 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap kv_map, const AttnArgs a
       }
     }
 
+    if (capped) {
+#pragma unroll
+      for (int tb = 0; tb < TK / 16; ++tb)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) st[tb][e] = cap_score(st[tb][e], cap_in, cap_out);
+    }
     // ---- scale, mask, online softmax over the token axis (per head column)
     float mx0 = -INFINITY, mx1 = -INFINITY;
 #pragma unroll
@@ -809,6 +862,18 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap kv_map, const AttnArgs a
   if (args.splits == 1) {
     T* o0 = reinterpret_cast<T*>(args.out) + ((size_t)q_row * args.Hq + head0) * D;
     T* o1 = reinterpret_cast<T*>(args.out) + ((size_t)q_row * args.Hq + head1) * D;
+    if (!KV8 && args.gate != nullptr) {
+      const T* g0 = reinterpret_cast<const T*>(args.gate) + q_row * args.ldg + (ok0 ? head0 : h * G) * D + g;
+      const T* g1 = reinterpret_cast<const T*>(args.gate) + q_row * args.ldg + (ok1 ? head1 : h * G) * D + g;
+#pragma unroll
+      for (int c = 0; c < NMB; ++c) {
+#pragma unroll
+        for (int hf = 0; hf < 2; ++hf) {
+          ot[c][2 * hf] *= __fdividef(1.f, 1.f + fast_exp2(-kLog2e * to_float(g0[c * 16 + 8 * hf])));
+          ot[c][2 * hf + 1] *= __fdividef(1.f, 1.f + fast_exp2(-kLog2e * to_float(g1[c * 16 + 8 * hf])));
+        }
+      }
+    }
 #pragma unroll
     for (int c = 0; c < NMB; ++c) {
       if (KV8) {
@@ -953,10 +1018,15 @@ MSGL_API int msgl_paged_attention(const void* kv_map, const void* q, void* out, 
                                   const void* v_scale, const void* mask, long long mask_stride, void* workspace,
                                   int B, int total_q, int max_q, int hq, int hk, int head_dim, int page_size,
                                   int num_pages, int layer, int num_layers, int kv_fp8, int causal, int window,
-                                  int splits, float scale, int dtype, cudaStream_t stream) {
+                                  int splits, float scale, int chunk, float softcap, const void* gate,
+                                  long long ldg, int dtype, cudaStream_t stream) {
   if (B == 0 || total_q == 0) return MSGL_OK;
-  if (hq % hk || 16 % (hq / hk)) {
-    msgl_set_error_text("attention: the GQA group size must divide 16");
+  if (hq % hk || hq / hk > 64) {
+    msgl_set_error_text("attention: up to 64 query heads per key / value head");
+    return MSGL_BAD_ARG;
+  }
+  if (gate != nullptr && kv_fp8) {
+    msgl_set_error_text("attention: no output gate with an fp8 pool");
     return MSGL_BAD_ARG;
   }
   if (splits < 1) splits = 1;
@@ -976,6 +1046,7 @@ MSGL_API int msgl_paged_attention(const void* kv_map, const void* q, void* out, 
   a.k_coord = layer; a.v_coord = num_layers + layer;
   a.causal = causal; a.window = window; a.splits = splits; a.total_q = total_q;
   a.scale = scale;
+  a.chunk = chunk; a.softcap = softcap; a.gate = gate; a.ldg = ldg;
   int* status = nullptr;
   cudaGetSymbolAddress((void**)&status, g_attn_status);
   a.status = status;
@@ -989,7 +1060,7 @@ MSGL_API int msgl_paged_attention(const void* kv_map, const void* q, void* out, 
     const int rows_heads = total_q * hq;
     const int warps = 4;
     const int blocks = (rows_heads + warps - 1) / warps;
-#define COMBINE(T, D) msgl_launch(attn_combine_kernel<T, D>, dim3(blocks), dim3(warps * 32), 0, stream, a.ws_o, a.ws_lse, (T*)out, rows_heads, splits, a.cu_q, a.B, a.Hq)
+#define COMBINE(T, D) msgl_launch(attn_combine_kernel<T, D>, dim3(blocks), dim3(warps * 32), 0, stream, a.ws_o, a.ws_lse, (T*)out, rows_heads, splits, a.cu_q, a.B, a.Hq, (const T*)a.gate, a.ldg)
     if (dtype == MSGL_BF16) {
       if (head_dim == 128) COMBINE(__nv_bfloat16, 128);
       else if (head_dim == 256) COMBINE(__nv_bfloat16, 256);
@@ -1073,5 +1144,5 @@ int msgl_paged_attention_noalloc(const void* kv_map, const void* q, void* out, c
   }
   return msgl_paged_attention(kv_map, q, out, block_table, bt_stride, cu_q, seq_lens, k_scale, v_scale, mask,
                               mask_stride, ws, B, total_q, max_q, hq, hk, head_dim, page_size, num_pages, layer,
-                              num_layers, kv_fp8, causal, window, splits, scale, dtype, stream);
+                              num_layers, kv_fp8, causal, window, splits, scale, 0, 0.f, nullptr, 0, dtype, stream);
 }

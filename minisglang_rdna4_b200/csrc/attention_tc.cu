@@ -63,8 +63,11 @@ struct TcArgs {
   const float* v_scale;
   float scale;
   int* status;
-  // position-pair form: one head, 256 consecutive query positions per CTA
   int window;          // > 0: a row sees the last ``window`` positions, its own included
+  int chunk;           // > 0: a row sees its own block of this many positions only
+  float softcap;       // c > 0: scores go through c tanh(s / c)
+  const void* cgate;   // [rows, Hq * ho] logits of a sigmoid gate per output channel (row stride ldcg), or null
+  long long ldcg;
   long long ldo, ho;   // element strides of a row and a head of out
   int v_chunks;        // 16-byte chunks of a value head
   const float* sink;   // [Hq] logits that only the softmax denominator counts, or null
@@ -131,21 +134,21 @@ template <typename T, bool KV8>
 __global__ void __launch_bounds__(256)
 kv_gather_kernel(const void* __restrict__ k_pool, const void* __restrict__ v_pool, T* __restrict__ kc,
                  T* __restrict__ vt, const int* __restrict__ blk_req, const int* __restrict__ req_info,
-                 const int* __restrict__ block_table, int bt_stride, int Hk, int page_size, long long t_cap) {
+                 const int* __restrict__ block_table, int bt_stride, int Hk, int page_size, long long t_cap, int d) {
   pdl_enter();
   __shared__ __align__(16) T vs[64][kD + 8];
   const int t0 = blockIdx.x * 64, h = blockIdx.y;
   const int req = blk_req[t0 >> 7];
-  const int kv_off = req_info[2 * req], kv_len = req_info[2 * req + 1];
+  const int kv_off = req_info[3 * req], kv_len = req_info[3 * req + 1], kv_lo = req_info[3 * req + 2];
 #pragma unroll
   for (int i = 0; i < 4; ++i) {
     const int id = threadIdx.x + i * 256;
     const int tt = id >> 4, c = id & 15;
-    const int tok = t0 + tt - kv_off;
+    const int tok = t0 + tt - kv_off + kv_lo;
     uint4 kq = make_uint4(0, 0, 0, 0), vq = make_uint4(0, 0, 0, 0);
-    if (tok >= 0 && tok < kv_len) {
+    if (tok >= kv_lo && tok < kv_len && c * 8 < d) {
       const int page = block_table[(long long)req * bt_stride + tok / page_size];
-      const long long src = (((long long)page * Hk + h) * page_size + tok % page_size) * kD + c * 8;
+      const long long src = (((long long)page * Hk + h) * page_size + tok % page_size) * d + c * 8;
       if constexpr (KV8) {
         kq = widen8<T>(*reinterpret_cast<const uint2*>(reinterpret_cast<const uint8_t*>(k_pool) + src));
         vq = widen8<T>(*reinterpret_cast<const uint2*>(reinterpret_cast<const uint8_t*>(v_pool) + src));
@@ -176,8 +179,8 @@ kv_gather_kernel(const void* __restrict__ k_pool, const void* __restrict__ v_poo
 // ------------------------------------------------------------------------------------------
 // 2. The attention kernel. grid = items x head pairs (heaviest items first), 320 threads.
 // ------------------------------------------------------------------------------------------
-// POS: the two tiles of a CTA are consecutive blocks of 128 positions of one head (every head has keys and
-// values of its own, so K / V tiles can only be shared along the positions) instead of two heads.
+// POS: the two tiles of a CTA are consecutive blocks of 128 positions of one head (where query heads that share keys
+// and values do not come in pairs, K / V tiles can only be shared along the positions) instead of two heads.
 template <typename T, bool POS>
 __global__ void __launch_bounds__(kTcThreads, 1)
 attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_constant__ CUtensorMap tma_k,
@@ -192,7 +195,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
   const int item_idx = blockIdx.x / args.pairs, pair = blockIdx.x - item_idx * args.pairs;
   const TcItem it = args.items[item_idx];
   const int head0 = POS ? pair : pair * 2;
-  const int hk = POS ? pair : head0 / (args.Hq / args.Hk);
+  const int hk = head0 / (args.Hq / args.Hk);
   const int nb = it.n_blocks;
 
   const uint32_t q_s = s_base + TcSmem::off_q, p_s = s_base + TcSmem::off_p, kv_s = s_base + TcSmem::off_kv;
@@ -330,7 +333,18 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
     const uint32_t s_addr = lane_base + t * 128, o_addr = lane_base + 256 + t * 128;
     const uint32_t p_row = p_s + t * 2 * kPanel + row * 128;
     const uint32_t swz = (uint32_t)(row & 7);
-    const float sl2 = args.scale * kLog2eTc * (args.k_scale != nullptr ? args.k_scale[hk] : 1.f);
+    const float raw_scale = args.scale * kLog2eTc * (args.k_scale != nullptr ? args.k_scale[hk] : 1.f);
+    // capped scores come out in units of log2: tanh(x) = 1 - 2 / (1 + e^(2x))
+    const bool capped = args.softcap > 0.f;
+    const float sl2 = capped ? 1.f : raw_scale;
+    const float cap_in = capped ? 2.f * raw_scale / args.softcap : 0.f, cap_out = args.softcap * kLog2eTc;
+    auto below = [&](int pos) {                        // last position ahead of what a row at pos sees
+      int lo = -1;
+      if (args.window > 0) lo = pos - args.window;
+      if (args.chunk > 0) lo = max(lo, pos - pos % args.chunk - 1);
+      return lo;
+    };
+    const int lo = below(q_pos), lo_last = below(tile_pos0 + kTile - 1);
 
     // The output row accumulates in tensor memory across KV blocks. The running maximum is only
     // raised when a block exceeds it by more than 2^8 (probabilities then stay below 256, exact
@@ -341,11 +355,9 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
     uint32_t s[4][32];
     bool ok = true;
     for (int j = 0; j < nb; ++j) {
-      const int kv0 = (POS ? it.kv_pos0 : 0) + j * kTile;
-      // the block reaches past some row's position, or starts below some row's window
-      const bool masked = kv0 + kTile - 1 > tile_pos0 ||
-                          (POS && args.window > 0 && kv0 <= tile_pos0 + kTile - 1 - args.window);
-      const int lo = POS && args.window > 0 ? q_pos - args.window : -1;
+      const int kv0 = it.kv_pos0 + j * kTile;
+      // the block reaches past some row's position, or starts below some row's window or chunk
+      const bool masked = kv0 + kTile - 1 > tile_pos0 || kv0 <= lo_last;
       if (!mbar_wait(s_full(t), (uint32_t)(j & 1), abort_flag, args.status, 209)) { ok = false; break; }
       tc_fence_after();
 #pragma unroll
@@ -354,11 +366,20 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
       tc_fence_before();
       mbar_arrive(s_free(t));                             // S is in registers: the next QK^T may start
       float mx = -INFINITY;
+      if (capped) {
+#pragma unroll
+        for (int c = 0; c < 4; ++c) {
+#pragma unroll
+          for (int i = 0; i < 32; ++i)
+            s[c][i] = __float_as_uint(
+                fmaf(-2.f * cap_out, __fdividef(1.f, 1.f + ex2f(__uint_as_float(s[c][i]) * cap_in)), cap_out));
+        }
+      }
 #pragma unroll
       for (int c = 0; c < 4; ++c) {
 #pragma unroll
         for (int i = 0; i < 32; ++i) {
-          if (masked && (kv0 + c * 32 + i > q_pos || (POS && kv0 + c * 32 + i <= lo))) s[c][i] = 0xFF800000u;   // -inf
+          if (masked && (kv0 + c * 32 + i > q_pos || kv0 + c * 32 + i <= lo)) s[c][i] = 0xFF800000u;   // -inf
           mx = fmaxf(mx, __uint_as_float(s[c][i]));
         }
       }
@@ -427,17 +448,25 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
       if (POS && args.gate != nullptr && out_row < it.q_rows)
         num *= 1.f / (1.f + __expf(-to_float(reinterpret_cast<const T*>(args.gate)[(it.q_row0 + out_row) * args.ldg + head])));
       const float inv = l > 0.f ? num / l : 0.f;
-      T* dst = reinterpret_cast<T*>(args.out) +
-               (POS ? (long long)(it.q_row0 + out_row) * args.ldo + head * args.ho
-                    : ((long long)(it.q_row0 + row) * args.Hq + head) * kD);
+      T* dst = reinterpret_cast<T*>(args.out) + (long long)(it.q_row0 + out_row) * args.ldo + head * args.ho;
+      const T* cg = args.cgate != nullptr
+                        ? reinterpret_cast<const T*>(args.cgate) + (it.q_row0 + out_row) * args.ldcg + head * args.ho
+                        : nullptr;
 #pragma unroll
       for (int c = 0; c < 4; ++c) tmem_ld_32x32b_x32(o_addr + c * 32, s[c]);
       tmem_ld_wait();
       if (out_row < it.q_rows) {
 #pragma unroll
         for (int c = 0; c < 16; ++c) {
-          if (POS && c >= args.v_chunks) break;
-          const uint32_t* o = &s[c >> 2][(c & 3) * 8];
+          if (c >= args.v_chunks) break;
+          uint32_t* o = &s[c >> 2][(c & 3) * 8];
+          if (cg != nullptr) {
+            float g[8];
+            load8(cg + 8 * c, g);
+#pragma unroll
+            for (int e = 0; e < 8; ++e)
+              o[e] = __float_as_uint(__uint_as_float(o[e]) * __fdividef(1.f, 1.f + ex2f(-kLog2eTc * g[e])));
+          }
           uint4 v;
           v.x = pack2_tc<T>(__uint_as_float(o[0]) * inv, __uint_as_float(o[1]) * inv);
           v.y = pack2_tc<T>(__uint_as_float(o[2]) * inv, __uint_as_float(o[3]) * inv);
@@ -563,39 +592,49 @@ MSGL_API int msgl_attn_prefill_pos(const void* q, long long ldq, long long hq_st
 
 // Causal prefill / extend attention for one layer. `kc` / `vt` are scratch buffers of
 // hk * t_cap * 128 16-bit elements each; `items` (n_items x 8 int32), `blk_req` (t_pad / 128
-// int32) and `req_info` (B x 2 int32: scratch offset, KV length) describe the step and are
-// built once per step by the caller. q and out are [total_q, hq, 128] with rows
-// `q_row_stride` / hq * 128 elements apart.
+// int32) and `req_info` (B x 3 int32: scratch offset, KV length, absolute position of the first
+// scratch row) describe the step (and the layer's window or chunk) and are built once per step by the caller. q and out
+// are [total_q, hq, d] with rows `q_row_stride` / hq * d elements apart, d 64 or 128; items of 128 positions pair
+// two query heads of a key / value head, items of 256 (`pos_form`) two blocks of one.
 MSGL_API int msgl_attn_prefill_tc(const void* q, long long q_row_stride, void* out, const void* k_pool,
                                   const void* v_pool, void* kc, void* vt, long long t_cap, int t_pad,
                                   const void* items, int n_items, const void* blk_req, const void* req_info,
                                   const void* block_table, int bt_stride, const void* k_scale, const void* v_scale,
-                                  int total_q, int hq, int hk, int page_size, int kv_fp8, float scale, int dtype,
-                                  cudaStream_t stream) {
+                                  int total_q, int hq, int hk, int d, int page_size, int kv_fp8, float scale,
+                                  int window, int chunk, float softcap, const void* gate, long long ldg, int pos_form,
+                                  int dtype, cudaStream_t stream) {
   if (n_items == 0 || total_q == 0) return MSGL_OK;
-  if (hq % hk || (hq / hk) % 2 || t_cap % 128 || t_pad % 128 || t_pad > t_cap || (q_row_stride % 8) ||
+  if (hq % hk || (!pos_form && (hq / hk) % 2) || (d != 64 && d != 128) || scale <= 0.f || (gate != nullptr && ldg % 8) ||
+      (uintptr_t)gate % 16 || t_cap % 128 || t_pad % 128 || t_pad > t_cap || (q_row_stride % 8) ||
       (dtype != MSGL_BF16 && dtype != MSGL_F16)) {
-    msgl_set_error_text("prefill attention: needs head_dim 128, an even GQA group, 16-bit q and a scratch of whole blocks");
+    msgl_set_error_text("prefill attention: needs rows of 64 or 128, pairs of heads or of blocks, 16-bit q, a positive scale "
+                        "and a scratch of whole blocks");
     return MSGL_BAD_ARG;
   }
   CUtensorMap mq, mk, mv;
   {
-    cuuint64_t dims[3] = {(cuuint64_t)kD, (cuuint64_t)hq, (cuuint64_t)total_q};
-    cuuint64_t strides[2] = {(cuuint64_t)kD * 2, (cuuint64_t)q_row_stride * 2};
+    cuuint64_t dims[3] = {(cuuint64_t)d, (cuuint64_t)hq, (cuuint64_t)total_q};
+    cuuint64_t strides[2] = {(cuuint64_t)d * 2, (cuuint64_t)q_row_stride * 2};
     cuuint32_t box[3] = {64, 1, 128};
     if (!encode_map(&mq, q, 3, dims, strides, box, "q")) return MSGL_CUDA_ERROR;
   }
-  {
+  if (pos_form) {
+    cuuint64_t kdims[3] = {(cuuint64_t)kD, (cuuint64_t)hk, (cuuint64_t)t_cap};
+    cuuint64_t kstr[2] = {(cuuint64_t)t_cap * kD * 2, (cuuint64_t)kD * 2};
+    cuuint32_t kbox[3] = {64, 1, 128};
+    if (!encode_map(&mk, kc, 3, kdims, kstr, kbox, "k")) return MSGL_CUDA_ERROR;
+    cuuint64_t vdims[3] = {(cuuint64_t)t_cap, (cuuint64_t)kD, (cuuint64_t)hk};
+    cuuint64_t vstr[2] = {(cuuint64_t)t_cap * 2, (cuuint64_t)t_cap * kD * 2};
+    cuuint32_t vbox[3] = {64, 128, 1};
+    if (!encode_map(&mv, vt, 3, vdims, vstr, vbox, "v")) return MSGL_CUDA_ERROR;
+  } else {
     cuuint64_t dims[2] = {(cuuint64_t)kD, (cuuint64_t)hk * (cuuint64_t)t_cap};
     cuuint64_t strides[1] = {(cuuint64_t)kD * 2};
     cuuint32_t box[2] = {64, 128};
     if (!encode_map(&mk, kc, 2, dims, strides, box, "k")) return MSGL_CUDA_ERROR;
-  }
-  {
-    cuuint64_t dims[2] = {(cuuint64_t)t_cap, (cuuint64_t)hk * kD};
-    cuuint64_t strides[1] = {(cuuint64_t)t_cap * 2};
-    cuuint32_t box[2] = {64, 128};
-    if (!encode_map(&mv, vt, 2, dims, strides, box, "v")) return MSGL_CUDA_ERROR;
+    cuuint64_t vdims[2] = {(cuuint64_t)t_cap, (cuuint64_t)hk * kD};
+    cuuint64_t vstr[1] = {(cuuint64_t)t_cap * 2};
+    if (!encode_map(&mv, vt, 2, vdims, vstr, box, "v")) return MSGL_CUDA_ERROR;
   }
   int* status = nullptr;
   cudaGetSymbolAddress((void**)&status, g_attn_tc_status);
@@ -603,15 +642,23 @@ MSGL_API int msgl_attn_prefill_tc(const void* q, long long q_row_stride, void* o
 #define GATHER(T, F8)                                                                                              \
   msgl_launch(kv_gather_kernel<T, F8>, dim3(ggrid), dim3(256), 0, stream, k_pool, v_pool, (T*)kc, (T*)vt, (const int*)blk_req,          \
                                                      (const int*)req_info, (const int*)block_table, bt_stride, hk, \
-                                                     page_size, t_cap)
+                                                     page_size, t_cap, d)
   if (dtype == MSGL_BF16) { if (kv_fp8) GATHER(__nv_bfloat16, true); else GATHER(__nv_bfloat16, false); }
   else { if (kv_fp8) GATHER(__half, true); else GATHER(__half, false); }
 #undef GATHER
   MSGL_CHECK_LAUNCH("kv_gather");
   TcArgs a = {};
-  a.items = (const TcItem*)items; a.n_items = n_items; a.pairs = hq / 2; a.Hq = hq; a.Hk = hk; a.t_cap = t_cap;
-  a.out = out; a.k_scale = (const float*)k_scale; a.v_scale = (const float*)v_scale; a.scale = scale;
-  a.status = status;
+  a.items = (const TcItem*)items; a.n_items = n_items; a.pairs = pos_form ? hq : hq / 2; a.Hq = hq; a.Hk = hk;
+  a.t_cap = t_cap; a.out = out; a.k_scale = (const float*)k_scale; a.v_scale = (const float*)v_scale; a.scale = scale;
+  a.status = status; a.window = window; a.chunk = chunk; a.softcap = softcap; a.cgate = gate; a.ldcg = ldg;
+  a.ldo = (long long)hq * d; a.ho = d; a.v_chunks = d / 8;
+  if (pos_form) {
+    if (dtype != MSGL_BF16) {
+      msgl_set_error_text("prefill attention: bf16 where query heads do not come in pairs");
+      return MSGL_BAD_ARG;
+    }
+    return launch_tc<__nv_bfloat16, true>(mq, mk, mv, a, stream);
+  }
   if (dtype == MSGL_BF16) return launch_tc<__nv_bfloat16, false>(mq, mk, mv, a, stream);
   return launch_tc<__half, false>(mq, mk, mv, a, stream);
 }

@@ -7,11 +7,11 @@
 //                    (token, k) pair a row in the expert-sorted order, record the expert of
 //                    every tile (sgl_kernel.moe_align_block_size in the reference's CUDA path,
 //                    python/minisgl/moe/fused.py:96-117)
-//   moe_permute    : gather token rows into expert-sorted order
+//   moe_permute    : gather token rows into expert-sorted order, times their weight where that acts on the input
 //   moe_combine    : out[t] = sum_k w[t,k] * y[row_of(t,k)] in a fixed k order
 //                    (mmq_fp8_moe_gather_reduce, python/minisgl/quant/kernels.py:877)
 //   moe_combine32  : the same sum in fp32 for an fp32 residual stream, with a shared expert's
-//                    output behind a sigmoid gate per token
+//                    output, behind a sigmoid gate per token where it has one
 //
 // Shapes are static for CUDA graphs: the sorted buffers are sized for the worst case
 // T*k + E*127 rows and tiles past the live count carry expert id -1, which the GEMM skips.
@@ -190,15 +190,26 @@ __global__ void moe_scatter_kernel(const int32_t* __restrict__ topk_ids, const i
 
 template <typename T>
 __global__ void moe_permute_kernel(const T* __restrict__ x, const int32_t* __restrict__ sorted_pair,
-                                   T* __restrict__ out, int hidden, int k, int rows) {
+                                   T* __restrict__ out, int hidden, int k, int rows, const float* __restrict__ topk_w) {
   pdl_enter();
   const int row = blockIdx.x;
   if (row >= rows) return;
   const int pair = sorted_pair[row];
   uint4* dst = reinterpret_cast<uint4*>(out + (size_t)row * hidden);
-  const int vecs = hidden / 8;
+  const int vecs = hidden / (16 / (int)sizeof(T));
   if (pair < 0) {
     for (int i = threadIdx.x; i < vecs; i += blockDim.x) dst[i] = make_uint4(0, 0, 0, 0);
+    return;
+  }
+  if (topk_w != nullptr) {
+    const float w = topk_w[pair];
+    for (int i = threadIdx.x * 8; i < hidden; i += blockDim.x * 8) {
+      float v[8];
+      load8(x + (size_t)(pair / k) * hidden + i, v);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) v[e] *= w;
+      store8(out + (size_t)row * hidden + i, v);
+    }
     return;
   }
   const uint4* src = reinterpret_cast<const uint4*>(x + (size_t)(pair / k) * hidden);
@@ -227,8 +238,8 @@ __global__ void moe_combine_kernel(const T* __restrict__ y, const float* __restr
   }
 }
 
-// out [tokens, cols] fp32; shared [tokens, shared_cols] (columns past that: no shared part), shared_gate: one logit
-// per token, ldg elements apart
+// out [tokens, cols] fp32; topk_w null: every weight is one (it acted on the input); shared [tokens, shared_cols]
+// (columns past that: no shared part), shared_gate: one logit per token, ldg elements apart, or null
 template <typename T>
 __global__ void __launch_bounds__(256) moe_combine32_kernel(const T* __restrict__ y, const float* __restrict__ topk_w,
                                                             const int32_t* __restrict__ pair_row,
@@ -237,7 +248,7 @@ __global__ void __launch_bounds__(256) moe_combine32_kernel(const T* __restrict_
                                                             float* __restrict__ out, int cols, int k) {
   pdl_enter();
   const int t = blockIdx.x;
-  const float sg = shared != nullptr ? 1.f / (1.f + expf(-shared_gate[t * ldg])) : 0.f;
+  const float sg = shared_gate != nullptr ? 1.f / (1.f + expf(-shared_gate[t * ldg])) : 1.f;
   for (int i = threadIdx.x * 8; i < cols; i += blockDim.x * 8) {
     float acc[8], v[8];
 #pragma unroll
@@ -250,7 +261,7 @@ __global__ void __launch_bounds__(256) moe_combine32_kernel(const T* __restrict_
     for (int kk = 0; kk < k; ++kk) {
       const int row = pair_row[(size_t)t * k + kk];
       if (row < 0) continue;
-      const float w = topk_w[(size_t)t * k + kk];
+      const float w = topk_w != nullptr ? topk_w[(size_t)t * k + kk] : 1.f;
       load8(y + (size_t)row * cols + i, v);
 #pragma unroll
       for (int e = 0; e < 8; ++e) acc[e] = fmaf(w, v[e], acc[e]);
@@ -265,7 +276,7 @@ MSGL_API int msgl_moe_combine32(const void* y, const void* topk_w, const void* p
                                 int shared_cols, const void* shared_gate, long long ldg, void* out, int tokens, int cols,
                                 int k, int dtype, cudaStream_t stream) {
   if (tokens == 0) return MSGL_OK;
-  if (tokens < 0 || cols % 8 || shared_cols % 8 || (shared != nullptr && shared_gate == nullptr)) return MSGL_BAD_ARG;
+  if (tokens < 0 || cols % 8 || shared_cols % 8) return MSGL_BAD_ARG;
   const int threads = cols / 8 < 256 ? ((cols / 8 + 31) / 32) * 32 : 256;
 #define COMBINE32(T)                                                                                                 \
   msgl_launch(moe_combine32_kernel<T>, dim3(tokens), dim3(threads), 0, stream, (const T*)y, (const float*)topk_w,    \
@@ -325,17 +336,21 @@ MSGL_API int msgl_moe_align(const void* topk_ids, const void* counts, void* offs
   return MSGL_OK;
 }
 
+// topk_w (optional): the weight of every (token, expert) pair, multiplied into its row
 MSGL_API int msgl_moe_permute(const void* x, const void* sorted_pair, void* out, int hidden, int k, int rows,
-                              int dtype, cudaStream_t stream) {
+                              const void* topk_w, int dtype, cudaStream_t stream) {
   if (rows == 0) return MSGL_OK;
   if (hidden % 8) return MSGL_BAD_ARG;
   int threads = hidden / 8 < 256 ? ((hidden / 8 + 31) / 32) * 32 : 256;
   if (dtype == MSGL_BF16)
     msgl_launch(moe_permute_kernel<__nv_bfloat16>, dim3(rows), dim3(threads), 0, stream, (const __nv_bfloat16*)x, (const int32_t*)sorted_pair,
-                                                                   (__nv_bfloat16*)out, hidden, k, rows);
+                                                                   (__nv_bfloat16*)out, hidden, k, rows, (const float*)topk_w);
   else if (dtype == MSGL_F16)
     msgl_launch(moe_permute_kernel<__half>, dim3(rows), dim3(threads), 0, stream, (const __half*)x, (const int32_t*)sorted_pair,
-                                                            (__half*)out, hidden, k, rows);
+                                                            (__half*)out, hidden, k, rows, (const float*)topk_w);
+  else if (dtype == MSGL_F32)
+    msgl_launch(moe_permute_kernel<float>, dim3(rows), dim3(threads), 0, stream, (const float*)x, (const int32_t*)sorted_pair,
+                                                           (float*)out, hidden, k, rows, (const float*)topk_w);
   else
     return MSGL_BAD_ARG;
   MSGL_CHECK_LAUNCH("moe_permute");

@@ -412,3 +412,197 @@ MSGL_API int msgl_store_kv(const void* k, const void* v, void* k_cache, void* v_
   MSGL_CHECK_LAUNCH("store_kv");
   return MSGL_OK;
 }
+
+// ------------------------------------------------------------------------------------------
+// Heads of a layer with a geometry of its own: RMS norm over all query (key) heads together or none, rotation of the
+// first `rot` channels in either pairing, division of every query and key head by its root mean square or none, store of
+// keys and values. fp32 throughout, rounded once at the end. One CTA per token, a warp per head; rows of 64 * NP columns
+// of which `dim` count (the others are zero).
+// ------------------------------------------------------------------------------------------
+namespace {
+
+struct HeadsRopeArgs {
+  const void* x;          // [tokens, ld]: hq query heads, then hk keys and hk values when there is a store
+  long long ld;
+  const float* q_w;       // [hq * D] / [hk * D] weights of the norm over all heads, or null
+  const float* k_w;
+  const float* totals;    // [tokens, 2] sums of squares over the heads of all ranks, or null
+  float q_count, k_count; // channels behind those sums
+  const int32_t* positions;
+  const float* cos_sin;   // [max_pos, rot], or null
+  void* q_out;            // [tokens, hq, D]
+  void* k_cache;          // [pages, hk, page_size, D], or null: queries alone
+  void* v_cache;
+  const int32_t* out_loc;
+  int hq, hk, dim, rot, page_size, interleaved, unit, max_pos, num_slots;
+  float eps;
+};
+
+template <typename T> __device__ __forceinline__ float2 load_pair(const T* p) {
+  if constexpr (sizeof(T) == 4) return *reinterpret_cast<const float2*>(p);
+  else return to_float2(*reinterpret_cast<const typename Pack2<T>::type*>(p));
+}
+template <typename T> __device__ __forceinline__ void store_pair(T* p, float a, float b) {
+  if constexpr (sizeof(T) == 4) *reinterpret_cast<float2*>(p) = make_float2(a, b);
+  else *reinterpret_cast<typename Pack2<T>::type*>(p) = Pack2<T>::make(a, b);
+}
+
+template <typename T, int NP>
+__global__ void __launch_bounds__(512) heads_rope_store_kernel(const HeadsRopeArgs a) {
+  pdl_enter();
+  constexpr int D = 64 * NP;
+  extern __shared__ __align__(16) float rows[];       // a rotated row per warp
+  __shared__ float part[2][16];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
+  const int token = blockIdx.x;
+  const int hk = a.k_cache != nullptr ? a.hk : 0;
+  const T* x = reinterpret_cast<const T*>(a.x) + token * a.ld;
+  float rq = 1.f, rk = 1.f;
+  if (a.q_w != nullptr) {
+    float sq = 0.f, sk = 0.f;
+    if (a.totals != nullptr) {
+      sq = a.totals[2 * token];
+      sk = a.totals[2 * token + 1];
+    } else {
+      for (int h = warp; h < a.hq + hk; h += nw) {
+        float s = 0.f;
+#pragma unroll
+        for (int i = 0; i < NP; ++i) {
+          const float2 v = load_pair(x + h * D + 64 * i + 2 * lane);
+          s = fmaf(v.x, v.x, fmaf(v.y, v.y, s));
+        }
+        if (h < a.hq) sq += s; else sk += s;
+      }
+      sq = warp_sum(sq);
+      sk = warp_sum(sk);
+      if (lane == 0) { part[0][warp] = sq; part[1][warp] = sk; }
+      __syncthreads();
+      sq = warp_sum(lane < nw ? part[0][lane] : 0.f);
+      sk = warp_sum(lane < nw ? part[1][lane] : 0.f);
+    }
+    rq = 1.f / sqrtf(sq / a.q_count + a.eps);
+    if (hk > 0) rk = 1.f / sqrtf(sk / a.k_count + a.eps);
+  }
+  int pos = a.positions[token];
+  if (a.rot > 0) {
+    (void)MSGL_OOB(pos, a.max_pos);
+    pos = pos < 0 ? 0 : (pos >= a.max_pos ? a.max_pos - 1 : pos);
+  }
+  const int half = a.rot >> 1;
+  const float* cs = a.cos_sin + (size_t)pos * a.rot;
+  int slot = -1;
+  if (hk > 0) {
+    slot = a.out_loc[token];
+    if (slot >= 0) (void)MSGL_OOB(slot, a.num_slots);
+    if (slot >= a.num_slots) slot = -1;
+  }
+  float* row = rows + warp * a.rot;
+  for (int h = warp; h < a.hq + 2 * hk; h += nw) {
+    const bool is_q = h < a.hq, is_v = h >= a.hq + hk;
+    if (!is_q && slot < 0) break;            // a padding row: nothing to store
+    float v[NP][2];
+#pragma unroll
+    for (int i = 0; i < NP; ++i) {
+      const float2 p = load_pair(x + h * D + 64 * i + 2 * lane);
+      v[i][0] = p.x;
+      v[i][1] = p.y;
+    }
+    if (!is_v) {
+      if (a.q_w != nullptr) {
+        const float r = is_q ? rq : rk;
+        const float* w = is_q ? a.q_w + h * D : a.k_w + (h - a.hq) * D;
+#pragma unroll
+        for (int i = 0; i < NP; ++i) {
+          const float2 p = load_pair(w + 64 * i + 2 * lane);
+          v[i][0] *= r * p.x;
+          v[i][1] *= r * p.y;
+        }
+      }
+      if (a.rot > 0 && a.interleaved) {
+#pragma unroll
+        for (int i = 0; i < NP; ++i) {
+          const int p = 32 * i + lane;
+          if (p < half) {
+            const float c = cs[p], s = cs[half + p], v0 = v[i][0], v1 = v[i][1];
+            v[i][0] = v0 * c - v1 * s;
+            v[i][1] = v1 * c + v0 * s;
+          }
+        }
+      } else if (a.rot > 0) {
+        __syncwarp();
+#pragma unroll
+        for (int i = 0; i < NP; ++i) {
+          const int e = 64 * i + 2 * lane;
+          if (e < a.rot) *reinterpret_cast<float2*>(row + e) = make_float2(v[i][0], v[i][1]);
+        }
+        __syncwarp();
+#pragma unroll
+        for (int i = 0; i < NP; ++i) {
+#pragma unroll
+          for (int j = 0; j < 2; ++j) {
+            const int e = 64 * i + 2 * lane + j;
+            if (e < a.rot) {
+              const bool first = e < half;
+              const int p = first ? e : e - half;
+              const float c = cs[p], s = cs[half + p];
+              v[i][j] = first ? v[i][j] * c - row[e + half] * s : v[i][j] * c + row[p] * s;
+            }
+          }
+        }
+      }
+      if (a.unit) {
+        float s = 0.f;
+#pragma unroll
+        for (int i = 0; i < NP; ++i) s = fmaf(v[i][0], v[i][0], fmaf(v[i][1], v[i][1], s));
+        const float r = 1.f / sqrtf(warp_sum(s) / (float)a.dim + a.eps);
+#pragma unroll
+        for (int i = 0; i < NP; ++i) { v[i][0] *= r; v[i][1] *= r; }
+      }
+    }
+    T* dst;
+    if (is_q) {
+      dst = reinterpret_cast<T*>(a.q_out) + ((size_t)token * a.hq + h) * D;
+    } else {
+      const int kvh = is_v ? h - a.hq - hk : h - a.hq;
+      dst = reinterpret_cast<T*>(is_v ? a.v_cache : a.k_cache) +
+            (((size_t)(slot / a.page_size) * hk + kvh) * a.page_size + slot % a.page_size) * D;
+    }
+#pragma unroll
+    for (int i = 0; i < NP; ++i) store_pair(dst + 64 * i + 2 * lane, v[i][0], v[i][1]);
+  }
+}
+
+}  // namespace
+
+MSGL_API int msgl_heads_rope_store(const void* x, long long ld, const void* q_w, const void* k_w, const void* totals,
+                                   float q_count, float k_count, const void* positions, const void* cos_sin, int rot,
+                                   void* q_out, void* k_cache, void* v_cache, const void* out_loc, int tokens, int hq,
+                                   int hk, int width, int dim, int page_size, float eps, int interleaved, int unit,
+                                   int max_pos, int num_slots, int dtype, cudaStream_t stream) {
+  if (tokens == 0) return MSGL_OK;
+  if (rot < 0 || rot % 2 || rot > dim || dim > width || hq <= 0 || ld % 2 || (rot > 0 && cos_sin == nullptr) ||
+      (k_cache != nullptr && (hk <= 0 || page_size <= 0 || (q_w != nullptr && k_w == nullptr))))
+    return MSGL_BAD_ARG;
+  HeadsRopeArgs a{x, ld, (const float*)q_w, (const float*)k_w, (const float*)totals, q_count, k_count,
+                  (const int32_t*)positions, (const float*)cos_sin, q_out, k_cache, v_cache, (const int32_t*)out_loc, hq, hk,
+                  dim, rot, page_size, interleaved, unit, max_pos, num_slots, eps};
+  const int heads = hq + (k_cache != nullptr ? 2 * hk : 0);
+  const int warps = heads < 16 ? heads : 16;
+  const size_t smem = interleaved ? 0 : (size_t)warps * rot * sizeof(float);
+#define HEADS_ROPE(T, NP) msgl_launch(heads_rope_store_kernel<T, NP>, dim3(tokens), dim3(32 * warps), smem, stream, a)
+#define HEADS_ROPE_WIDTHS(T)              \
+  do {                                    \
+    if (width == 64) HEADS_ROPE(T, 1);    \
+    else if (width == 128) HEADS_ROPE(T, 2); \
+    else if (width == 256) HEADS_ROPE(T, 4); \
+    else if (width == 512) HEADS_ROPE(T, 8); \
+    else return MSGL_BAD_ARG;             \
+  } while (0)
+  if (dtype == MSGL_BF16) HEADS_ROPE_WIDTHS(__nv_bfloat16);
+  else if (dtype == MSGL_F32) HEADS_ROPE_WIDTHS(float);
+  else return MSGL_BAD_ARG;
+#undef HEADS_ROPE_WIDTHS
+#undef HEADS_ROPE
+  MSGL_CHECK_LAUNCH("heads_rope_store");
+  return MSGL_OK;
+}

@@ -61,10 +61,13 @@ _SIGNATURES = {
     "msgl_attn_workspace_floats": (c_ll, [c_i, c_i, c_i, c_i]),
     "msgl_paged_attention": (c_i, [c_p, c_p, c_p, c_p, c_i, c_p, c_p, c_p, c_p, c_p, c_ll, c_p,
                                    c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_i,
-                                   c_f, c_i, c_p]),
+                                   c_f, c_i, c_f, c_p, c_ll, c_i, c_p]),
+    "msgl_paged_attention_f32": (c_i, [c_p] * 5 + [c_i, c_p, c_p] + [c_i] * 9 + [c_f, c_f, c_p, c_ll, c_p]),
+    "msgl_heads_rope_store": (c_i, [c_p, c_ll, c_p, c_p, c_p, c_f, c_f, c_p, c_p, c_i] + [c_p] * 4 + [c_i] * 6
+                              + [c_f] + [c_i] * 5 + [c_p]),
     "msgl_attn_status": (c_i, [c_i]),
     "msgl_attn_prefill_tc": (c_i, [c_p, c_ll, c_p, c_p, c_p, c_p, c_p, c_ll, c_i, c_p, c_i, c_p, c_p, c_p, c_i,
-                                   c_p, c_p, c_i, c_i, c_i, c_i, c_i, c_f, c_i, c_p]),
+                                   c_p, c_p, c_i, c_i, c_i, c_i, c_i, c_i, c_f, c_i, c_i, c_f, c_p, c_ll, c_i, c_i, c_p]),
     "msgl_attn_tc_status": (c_i, [c_i]),
     "msgl_attn_force_general_decode": (None, [c_i]),
     "msgl_attn_decode_stages": (None, [c_i]),
@@ -102,8 +105,9 @@ def bind(name: str, restype, argtypes) -> None:
     """Register the signature of an entry point added by another module (comm, moe …)."""
     _SIGNATURES[name] = (restype, argtypes)
     if _lib is not None:
-        fn = getattr(_lib, name)
-        fn.restype, fn.argtypes = restype, argtypes
+        fn = getattr(_lib, name, None)          # absent from a library of one family's kernels
+        if fn is not None:
+            fn.restype, fn.argtypes = restype, argtypes
 
 
 def check(rc: int, what: str) -> None:

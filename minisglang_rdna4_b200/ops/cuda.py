@@ -218,6 +218,33 @@ def qk_norm_rope_store(qkv, q_w, k_w, positions, cos_sin, hq, hk, head_dim, rota
     return q_out
 
 
+def heads_rope_store(x, heads, kv_heads, width, dim, positions, cos_sin, interleaved, eps, q_w=None, k_w=None,
+                     totals=None, unit=False, store=None):
+    assert x.dim() == 2 and x.stride(1) == 1 and positions.dtype == torch.int32
+    t = x.shape[0]
+    q_out = torch.empty((t, heads, width), dtype=x.dtype, device=x.device)
+    k_cache = v_cache = out_loc = sums = None
+    page_size = slots = 0
+    q_count, k_count = heads * dim, kv_heads * dim
+    if store is not None:
+        k_cache, v_cache, out_loc = store
+        page_size, slots = k_cache.shape[2], k_cache.shape[0] * k_cache.shape[2]
+        assert k_cache.dtype == v_cache.dtype == x.dtype and k_cache.is_contiguous() and v_cache.is_contiguous()
+        assert k_cache.shape[1] == kv_heads and k_cache.shape[3] == width
+    if totals is not None:
+        sums, q_count, k_count = totals
+        assert sums.is_contiguous() and sums.dtype == torch.float32 and sums.shape == (t, 2)
+    for w in (q_w, k_w):
+        assert w is None or (w.dtype == torch.float32 and w.is_contiguous())
+    rot, max_pos = (cos_sin.shape[1], cos_sin.shape[0]) if cos_sin is not None else (0, 0)
+    check(lib().msgl_heads_rope_store(
+        _p(x), x.stride(0), _p(q_w), _p(k_w), _p(sums), float(q_count), float(k_count), _p(positions), _p(cos_sin), rot,
+        _p(q_out), _p(k_cache), _p(v_cache), _p(out_loc), t, heads, kv_heads, width, dim, page_size, eps, int(interleaved),
+        int(unit), max_pos, slots, _dt(x), _stream()), "heads_rope_store")
+    _count("heads_rope_store", "heads_rope_store_kernel")
+    return q_out
+
+
 def store_kv(k, v, k_cache, v_cache, out_loc, k_scale=None, v_scale=None):
     hk, page_size, d = k_cache.shape[1], k_cache.shape[2], k_cache.shape[3]
     t = out_loc.numel()
@@ -252,7 +279,7 @@ def _kv_map(k_cache: torch.Tensor):
         buf = np.zeros(128, dtype=np.uint8)
         check(lib().msgl_attn_make_kv_map(buf.ctypes.data, root.data_ptr(), root.element_size(), d, ps, hk,
                                           pages_p1, 2 * layers), "attn_make_kv_map")
-        if len(_KV_MAPS) > 64:
+        if len(_KV_MAPS) > 512:            # layers with planes of their own have a map each
             _KV_MAPS.clear()
         hit = (buf, root)
         _KV_MAPS[key] = hit
@@ -278,11 +305,14 @@ def choose_splits(batch, hk, max_kv, decode):
 
 def paged_attention(q, k_cache, v_cache, block_table, cu_q, seq_lens, scale, *, causal=True, window=0, mask=None,
                     k_scale=None, v_scale=None, max_q=0, max_kv=0, decode=False, workspace=None, splits=None,
-                    plan=None, tc=None, mask_window=0):
+                    plan=None, tc=None, mask_window=0, chunk=0, softcap=0.0, gate=None):
     """``plan`` (a ``PrefillPlan``) or ``tc=True`` sends a causal prefill / extend step to the
     tcgen05 kernel when it covers the shape (``tc=True`` without a plan builds the step tables from
     the device lengths, which synchronises). Without either the general kernel runs: decode and
     verification steps must not change kernels with the number of rows per request."""
+    if q.dtype == torch.float32:
+        assert causal and mask is None
+        return _paged_attention_f32(q, k_cache, v_cache, block_table, cu_q, seq_lens, scale, window, chunk, softcap, gate)
     t, hq, d = q.shape
     pages_p1, hk, ps, _ = k_cache.shape
     if max_q <= 0:
@@ -320,8 +350,29 @@ def paged_attention(q, k_cache, v_cache, block_table, cu_q, seq_lens, scale, *, 
         desc.ctypes.data, _p(q), _p(out), _p(block_table), block_table.stride(0), _p(cu_q), _p(seq_lens),
         _p(k_scale), _p(v_scale), _p(mask), mask_stride, _p(workspace) if splits > 1 else None,
         b, t, max_q, hq, hk, d, ps, pages_p1 - 1, layer, layers, int(fp8), int(causal), int(window), splits,
-        float(scale), _dt(q), _stream()), "paged_attention")
+        float(scale), int(chunk), float(softcap), *_output_gate(gate, q), _dt(q), _stream()), "paged_attention")
     _count("paged_attention", "paged_attention_kernel", 2 if splits > 1 else 1)
+    return out
+
+
+def _output_gate(gate, q):
+    """Pointer and row stride of the logits of a gate per output channel."""
+    if gate is None:
+        return None, 0
+    assert gate.shape == (q.shape[0], q.shape[1] * q.shape[2]) and gate.stride(1) == 1 and gate.dtype == q.dtype
+    return gate.data_ptr(), gate.stride(0)
+
+
+def _paged_attention_f32(q, k_cache, v_cache, block_table, cu_q, seq_lens, scale, window, chunk, softcap, gate):
+    t, hq, d = q.shape
+    pages, hk, ps, _ = k_cache.shape
+    assert q.is_contiguous() and k_cache.is_contiguous() and v_cache.is_contiguous() and k_cache.dtype == torch.float32
+    out = torch.empty_like(q)
+    check(lib().msgl_paged_attention_f32(
+        _p(q), _p(k_cache), _p(v_cache), _p(out), _p(block_table), block_table.stride(0), _p(cu_q), _p(seq_lens),
+        seq_lens.numel(), t, hq, hk, d, ps, pages, int(window), int(chunk), float(scale), float(softcap),
+        *_output_gate(gate, q), _stream()), "paged_attention_f32")
+    _count("paged_attention_f32", "paged_attention_f32_kernel")
     return out
 
 
@@ -355,38 +406,61 @@ def _upload_tables(host: np.ndarray, device) -> torch.Tensor:
     return dev
 
 
+def _first_block(pos: np.ndarray, window: int, chunk: int = 0) -> np.ndarray:
+    """Start of the block of 128 positions that holds the first position a row at ``pos`` can see."""
+    lo = np.zeros_like(pos)
+    if window > 0:
+        lo = np.maximum(lo, pos - window + 1)
+    if chunk > 0:
+        lo = np.maximum(lo, pos // chunk * chunk)
+    return lo // 128 * 128
+
+
 class PrefillPlan:
-    """Per-step tables of the tensor-core prefill kernel: one item per (request, block of 128
+    """Per-step tables of the tensor-core prefill kernel: one item per (request, block of ``tile``
     query positions), heaviest first; the request of every 128-row scratch block; per request
-    the scratch offset and KV length. Built on the host from the step's lengths, one H2D copy."""
+    the scratch offset, KV length and first position in the scratch. Built on the host from the step's lengths, one H2D
+    copy. ``window`` / ``chunk``: the reach of the layers the plan is for. ``tile`` 256: the form for query heads that do
+    not come in pairs."""
 
-    __slots__ = ("tables", "n_items", "t_pad", "n_req", "off_blk", "off_req")
+    __slots__ = ("tables", "n_items", "t_pad", "n_req", "off_blk", "off_req", "tile")
 
-    def __init__(self, cu_q: np.ndarray, seq_lens: np.ndarray, device) -> None:
+    @staticmethod
+    def rows_in_reach(cu_q: np.ndarray, seq_lens: np.ndarray, window: int = 0, chunk: int = 0) -> int:
+        kv = np.asarray(seq_lens, dtype=np.int64)
+        lo = _first_block(kv - np.diff(np.asarray(cu_q, dtype=np.int64)[:kv.size + 1]), window, chunk)
+        return int(((kv - lo + 127) // 128 * 128).sum())
+
+    def __init__(self, cu_q: np.ndarray, seq_lens: np.ndarray, device, window: int = 0, chunk: int = 0,
+                 tile: int = 128) -> None:
         cu_q = np.asarray(cu_q, dtype=np.int64)
         kv = np.asarray(seq_lens, dtype=np.int64)
         b = int(kv.size)
         q_len = cu_q[1:b + 1] - cu_q[:b]
-        kv_pad = (kv + 127) // 128 * 128
+        kv_lo = _first_block(kv - q_len, window, chunk)
+        kv_pad = (kv - kv_lo + 127) // 128 * 128
         kv_off = np.concatenate([[0], np.cumsum(kv_pad)[:-1]]) if b else np.zeros(0, dtype=np.int64)
         self.t_pad = int(kv_pad.sum())
         self.n_req = b
-        n_tiles = (q_len + 127) // 128
+        self.tile = tile
+        n_tiles = (q_len + tile - 1) // tile
         req = np.repeat(np.arange(b), n_tiles)
         first = np.concatenate([[0], np.cumsum(n_tiles)[:-1]]) if b else np.zeros(0, dtype=np.int64)
         qb = np.arange(int(n_tiles.sum())) - np.repeat(first, n_tiles)
         items = np.zeros((req.size, 8), dtype=np.int32)
-        rows = np.minimum(128, q_len[req] - qb * 128)
-        pos0 = kv[req] - q_len[req] + qb * 128
-        items[:, 0] = cu_q[req] + qb * 128
+        rows = np.minimum(tile, q_len[req] - qb * tile)
+        pos0 = kv[req] - q_len[req] + qb * tile
+        kv0 = _first_block(pos0, window, chunk)
+        items[:, 0] = cu_q[req] + qb * tile
         items[:, 1] = rows
         items[:, 2] = pos0
-        items[:, 3] = kv_off[req]
-        items[:, 4] = (pos0 + rows + 127) // 128
+        items[:, 3] = kv_off[req] + kv0 - kv_lo[req]
+        items[:, 4] = (pos0 + rows - kv0 + 127) // 128
         items[:, 5] = req
+        items[:, 6] = kv0
         items = items[np.argsort(-items[:, 4], kind="stable")]
         blk_req = np.repeat(np.arange(b), kv_pad // 128).astype(np.int32)
-        req_info = np.stack([kv_off, kv], axis=1).astype(np.int32).reshape(-1)
+        req_info = np.stack([kv_off, kv, kv_lo], axis=1).astype(np.int32).reshape(-1)
         self.n_items = int(items.shape[0])
         self.off_blk = items.size
         self.off_req = self.off_blk + blk_req.size
@@ -428,7 +502,15 @@ def prefill_attention_tc_ok(q, k_cache, *, causal, window, mask, decode) -> bool
             and q.stride(1) == 128 and q.stride(0) % 8 == 0)
 
 
-def prefill_attention_tc(q, k_cache, v_cache, block_table, plan: PrefillPlan, scale, *, k_scale=None, v_scale=None):
+def prefill_heads_tc_ok(q, k_cache, scale) -> bool:
+    """Rows of 64 or 128 channels; any head counts (``PrefillPlan.tile``), windows, chunks, soft caps and gates."""
+    return (q.dtype == torch.bfloat16 and q.shape[2] in (64, 128) and q.is_contiguous() and scale > 0
+            and q.shape[1] % k_cache.shape[1] == 0)
+
+
+def prefill_attention_tc(q, k_cache, v_cache, block_table, plan: PrefillPlan, scale, *, k_scale=None, v_scale=None,
+                         window=0, chunk=0, softcap=0.0, gate=None):
+    """``plan`` was made for the same window and chunk."""
     t, hq, d = q.shape
     _, hk, ps, _ = k_cache.shape
     kc, vt, cap = _tc_scratch(q.device, q.dtype, hk, plan.t_pad)
@@ -439,7 +521,8 @@ def prefill_attention_tc(q, k_cache, v_cache, block_table, plan: PrefillPlan, sc
     check(lib().msgl_attn_prefill_tc(
         _p(q), q.stride(0), _p(out), _p(k_cache), _p(v_cache), _p(kc), _p(vt), cap, plan.t_pad,
         base, plan.n_items, base + 4 * plan.off_blk, base + 4 * plan.off_req, _p(block_table), block_table.stride(0),
-        _p(k_scale), _p(v_scale), t, hq, hk, ps, int(fp8), float(scale), _dt(q), _stream()), "attn_prefill_tc")
+        _p(k_scale), _p(v_scale), t, hq, hk, d, ps, int(fp8), float(scale), int(window), int(chunk), float(softcap),
+        *_output_gate(gate, q), int(plan.tile == 256), _dt(q), _stream()), "attn_prefill_tc")
     _count("prefill_attention", "attn_prefill_tc_kernel", 2)
     return out
 
@@ -992,13 +1075,13 @@ def _bind_linear():
 
     if hasattr(_bind_linear, "_done"):
         return
-    bind("msgl_add_norm", c_i, [c_p, c_p, c_p, c_i, c_ll, c_ll, c_p, c_p, c_i, c_i, c_i, c_f, c_i, c_i, c_p])
+    bind("msgl_add_norm", c_i, [c_p, c_p, c_p, c_i, c_ll, c_ll, c_p, c_p, c_i, c_i, c_i, c_f, c_i, c_p, c_f, c_i, c_p])
     bind("msgl_linear_attention", c_i, [c_p, c_p, c_p, c_ll, c_p, c_ll] + [c_p] * 8 + [c_i] * 7 + [c_f, c_f, c_i, c_i, c_p])
     bind("msgl_norm_gate", c_i, [c_p, c_p, c_ll, c_p, c_p, c_p, c_ll, c_i, c_i, c_f, c_f, c_i, c_i, c_p])
     _bind_linear._done = True
 
 
-def add_norm(x, delta, weight, eps, center, out_dtype, out_cols):
+def add_norm(x, delta, weight, eps, center, out_dtype, out_cols, post=None, mult=1.0):
     _bind_linear()
     assert x.is_contiguous() and x.dtype == torch.float32 and weight.dtype == torch.float32
     rows, width = x.shape
@@ -1013,7 +1096,7 @@ def add_norm(x, delta, weight, eps, center, out_dtype, out_cols):
     x_out = torch.empty_like(x) if delta is not None else x
     y = torch.empty((rows, out_cols), dtype=out_dtype, device=x.device)
     check(lib().msgl_add_norm(_p(x), _p(x_out), _p(delta), planes, plane_stride, ldd, _p(weight), _p(y), rows, width,
-                              out_cols, eps, int(center), _DT[out_dtype], _stream()), "add_norm")
+                              out_cols, eps, int(center), _p(post), mult, _DT[out_dtype], _stream()), "add_norm")
     _count("add_norm", "add_norm_kernel")
     return x_out, y
 

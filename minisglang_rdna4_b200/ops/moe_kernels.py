@@ -14,7 +14,7 @@ _lib.bind("msgl_moe_route", c_i, [c_p] * 5 + [c_i] * 5 + [c_f, c_i, c_i, c_ll, c
 _lib.bind("msgl_moe_combine32", c_i, [c_p, c_p, c_p, c_p, c_i, c_p, c_ll, c_p, c_i, c_i, c_i, c_i, c_p])
 _lib.bind("msgl_gemm_f32_grouped", c_i, [c_p, c_p, c_p, c_i, c_i, c_i, c_p, c_p])
 _lib.bind("msgl_moe_align", c_i, [c_p, c_p, c_p, c_p, c_p, c_p, c_p, c_p, c_i, c_i, c_i, c_i, c_i, c_i, c_p])
-_lib.bind("msgl_moe_permute", c_i, [c_p, c_p, c_p, c_i, c_i, c_i, c_i, c_p])
+_lib.bind("msgl_moe_permute", c_i, [c_p, c_p, c_p, c_i, c_i, c_i, c_p, c_i, c_p])
 _lib.bind("msgl_moe_combine", c_i, [c_p, c_p, c_p, c_p, c_i, c_i, c_i, c_i, c_p])
 _lib.bind("msgl_gemm_grouped", c_i, [c_i, c_p, c_ll, c_p, c_p, c_ll, c_i, c_i, c_i, c_p, c_i, c_p, c_p, c_i, c_i, c_p])
 
@@ -97,10 +97,7 @@ def moe_forward(x, w13, w2, topk_w, topk_ids, expert_offset=0, counts=None):
     k = topk_ids.shape[1]
     sorted_pair, pair_row, tile_expert, _meta = moe_align(topk_ids, expert_offset, e_local, counts)
     rows = sorted_pair.numel()
-    xs = torch.empty((rows, h), dtype=x.dtype, device=x.device)
-    check(lib().msgl_moe_permute(x.data_ptr(), sorted_pair.data_ptr(), xs.data_ptr(), h, k, rows, _DT[x.dtype],
-                                 K._stream()), "moe_permute")
-    K._count("moe_permute", "moe_permute_kernel")
+    xs = _permute(x, sorted_pair, k)
     hcur = gemm_grouped(xs, w13, tile_expert)
     act = K.act_and_mul(hcur)
     y = gemm_grouped(act, w2, tile_expert)
@@ -122,21 +119,22 @@ def gemm_f32_grouped(a, b, tile_expert):
     return out
 
 
-def experts_partial32(x, w13, w2, topk_w, topk_ids, limit, alpha, shared=None, shared_gate=None, counts=None):
-    """Clamped experts for an fp32 residual stream: ``w13 [E, 2I, K]``, ``w2 [E, N, I]`` -> fp32 ``[T, N]``; ``shared``
-    rows are added behind the sigmoid of ``shared_gate [T]`` (fp32 logits)."""
+def experts_partial32(x, w13, w2, topk_w, topk_ids, limit, alpha, shared=None, shared_gate=None, counts=None,
+                      act="clamped", on_input=False):
+    """Experts for an fp32 residual stream: ``w13 [E, 2I, K]``, ``w2 [E, N, I]`` -> fp32 ``[T, N]``; ``shared`` rows are
+    added, behind the sigmoid of ``shared_gate [T]`` (fp32 logits) where given. ``on_input``: the weights multiply the
+    experts' inputs."""
     t, k = topk_ids.shape
     sorted_pair, pair_row, tile_expert, _meta = moe_align(topk_ids, 0, w13.shape[0], counts)
     f32 = x.dtype == torch.float32
-    # rows of fp32 are permuted as twice as many 16-bit values
-    xs = _permute(x.view(torch.bfloat16), sorted_pair, k).view(torch.float32) if f32 else _permute(x, sorted_pair, k)
+    xs = _permute(x, sorted_pair, k, topk_w if on_input else None)
     mm = gemm_f32_grouped if f32 else gemm_grouped
-    y = mm(K.act_and_mul(mm(xs, w13, tile_expert), "clamped", alpha, limit), w2, tile_expert)
+    y = mm(K.act_and_mul(mm(xs, w13, tile_expert), act, alpha, limit), w2, tile_expert)
     n = w2.shape[1]
     out = torch.empty((t, n), dtype=torch.float32, device=x.device)
     if shared is not None:
         assert shared.is_contiguous() and shared.dtype == x.dtype and shared.shape[1] <= n
-    check(lib().msgl_moe_combine32(y.data_ptr(), topk_w.data_ptr(), pair_row.data_ptr(), K._p(shared),
+    check(lib().msgl_moe_combine32(y.data_ptr(), None if on_input else topk_w.data_ptr(), pair_row.data_ptr(), K._p(shared),
                                    0 if shared is None else shared.shape[1], K._p(shared_gate),
                                    0 if shared_gate is None else shared_gate.stride(0), out.data_ptr(), t, n, k, _DT[x.dtype],
                                    K._stream()), "moe_combine32")
@@ -177,10 +175,7 @@ def moe_forward_w4a8(x, w13_packed, w13_atoms, w2_packed, w2_atoms, topk_w, topk
     k = topk_ids.shape[1]
     sorted_pair, pair_row, tile_expert, _meta = moe_align(topk_ids, expert_offset, e_local)
     rows = sorted_pair.numel()
-    xs = torch.empty((rows, h), dtype=x.dtype, device=x.device)
-    check(lib().msgl_moe_permute(x.data_ptr(), sorted_pair.data_ptr(), xs.data_ptr(), h, k, rows, _DT[x.dtype],
-                                 K._stream()), "moe_permute")
-    K._count("moe_permute", "moe_permute_kernel")
+    xs = _permute(x, sorted_pair, k)
     xq, xsc = K.per_token_quant_fp8(xs)
     hcur = gemm_grouped_w4a8(xq, xsc, w13_packed, w13_atoms, tile_expert, x.dtype)
     aq, asc = K.silu_and_mul_quant(hcur)
@@ -195,11 +190,12 @@ def moe_forward_w4a8(x, w13_packed, w13_atoms, w2_packed, w2_atoms, topk_w, topk
 _lib.bind("msgl_gemm_grouped_w8a8", c_i, [c_p, c_ll, c_p, c_p, c_ll, c_i, c_i, c_i, c_p, c_i, c_p, c_p, c_i, c_i, c_p])
 
 
-def _permute(x, sorted_pair, k):
+def _permute(x, sorted_pair, k, topk_w=None):
+    """``topk_w [T, k]``: weight of every pair, multiplied into its row."""
     rows, h = sorted_pair.numel(), x.shape[1]
     xs = torch.empty((rows, h), dtype=x.dtype, device=x.device)
-    check(lib().msgl_moe_permute(x.data_ptr(), sorted_pair.data_ptr(), xs.data_ptr(), h, k, rows, _DT[x.dtype],
-                                 K._stream()), "moe_permute")
+    check(lib().msgl_moe_permute(x.data_ptr(), sorted_pair.data_ptr(), xs.data_ptr(), h, k, rows, K._p(topk_w),
+                                 _DT[x.dtype], K._stream()), "moe_permute")
     K._count("moe_permute", "moe_permute_kernel")
     return xs
 
