@@ -370,9 +370,18 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
 #pragma unroll
         for (int c = 0; c < 4; ++c) {
 #pragma unroll
-          for (int i = 0; i < 32; ++i)
-            s[c][i] = __float_as_uint(
-                fmaf(-2.f * cap_out, __fdividef(1.f, 1.f + ex2f(__uint_as_float(s[c][i]) * cap_in)), cap_out));
+          for (int i = 0; i < 32; i += 4) {
+            // one reciprocal for four: exponents held at 30 (tanh is 1 there in fp32), so that the product stays finite
+            float d[4];
+#pragma unroll
+            for (int e = 0; e < 4; ++e) d[e] = 1.f + ex2f(fminf(__uint_as_float(s[c][i + e]) * cap_in, 30.f));
+            const float p01 = d[0] * d[1], p23 = d[2] * d[3], r = __fdividef(-2.f * cap_out, p01 * p23);
+            const float r01 = r * p23, r23 = r * p01;
+            s[c][i] = __float_as_uint(fmaf(r01, d[1], cap_out));
+            s[c][i + 1] = __float_as_uint(fmaf(r01, d[0], cap_out));
+            s[c][i + 2] = __float_as_uint(fmaf(r23, d[3], cap_out));
+            s[c][i + 3] = __float_as_uint(fmaf(r23, d[2], cap_out));
+          }
         }
       }
 #pragma unroll

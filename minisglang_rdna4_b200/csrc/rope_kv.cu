@@ -416,8 +416,9 @@ MSGL_API int msgl_store_kv(const void* k, const void* v, void* k_cache, void* v_
 // ------------------------------------------------------------------------------------------
 // Heads of a layer with a geometry of its own: RMS norm over all query (key) heads together or none, rotation of the
 // first `rot` channels in either pairing, division of every query and key head by its root mean square or none, store of
-// keys and values. fp32 throughout, rounded once at the end. One CTA per token, a warp per head; rows of 64 * NP columns
-// of which `dim` count (the others are zero).
+// keys and values. fp32 throughout, rounded once at the end. One CTA per token; rows of a multiple of 64 columns of which
+// `dim` count (the others are zero). Two forms: sixteen columns per lane and every head in registers at once (rotated
+// channels a multiple of 16), and a warp per head with the rotation through shared memory (any sizes).
 // ------------------------------------------------------------------------------------------
 namespace {
 
@@ -572,6 +573,171 @@ __global__ void __launch_bounds__(512) heads_rope_store_kernel(const HeadsRopeAr
   }
 }
 
+// LPH lanes per head (D = 16 * LPH), NI heads per lane group. A lane has two runs of eight columns, both members of every
+// pair among them. A CTA takes tokens in turn; the next one's row is on its way while one is worked on.
+template <typename T, int LPH, int NI>
+__global__ void __launch_bounds__(384) heads_rope_store_vec_kernel(const HeadsRopeArgs a, int tokens) {
+  pdl_enter();
+  constexpr int D = 16 * LPH, HPW = 32 / LPH, Q = sizeof(T) / 2;
+  __shared__ float part[2][2][16];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
+  const int sub = lane % LPH;
+  const int hk = a.k_cache != nullptr ? a.hk : 0, total = a.hq + 2 * hk;
+  const int half = a.rot >> 1;
+  int col[2], angle;                       // first columns of the runs, first angle
+  bool turns;
+  if (a.interleaved) {
+    col[0] = 16 * sub;
+    col[1] = col[0] + 8;
+    turns = col[0] < a.rot;
+    angle = 8 * sub;
+  } else {
+    turns = 8 * sub < half;
+    col[0] = turns ? 8 * sub : a.rot + 16 * (sub - (half >> 3));
+    col[1] = turns ? half + 8 * sub : col[0] + 8;
+    angle = 8 * sub;
+  }
+  uint4 raw[NI][2][Q];
+  int pos = 0, slot = -1;
+  auto fetch = [&](int token) {
+    pos = a.positions[token];
+    if (hk > 0) slot = a.out_loc[token];
+#pragma unroll
+    for (int i = 0; i < NI; ++i) {
+      const int h = (i * nw + warp) * HPW + lane / LPH;
+      const T* src = reinterpret_cast<const T*>(a.x) + token * a.ld + h * D;
+#pragma unroll
+      for (int r = 0; r < 2; ++r)
+#pragma unroll
+        for (int j = 0; j < Q; ++j)
+          raw[i][r][j] = h < total ? reinterpret_cast<const uint4*>(src + col[r])[j] : make_uint4(0, 0, 0, 0);
+    }
+  };
+  if ((int)blockIdx.x < tokens) fetch(blockIdx.x);
+  int buf = 0;
+  for (int token = blockIdx.x; token < tokens; token += gridDim.x, buf ^= 1) {
+    float cs[8], sn[8];
+    if (turns) {
+      (void)MSGL_OOB(pos, a.max_pos);
+      pos = pos < 0 ? 0 : (pos >= a.max_pos ? a.max_pos - 1 : pos);
+      load8(a.cos_sin + (size_t)pos * a.rot + angle, cs);
+      load8(a.cos_sin + (size_t)pos * a.rot + half + angle, sn);
+    }
+    float v[NI][2][8];
+#pragma unroll
+    for (int i = 0; i < NI; ++i)
+#pragma unroll
+      for (int r = 0; r < 2; ++r) load8(reinterpret_cast<const T*>(raw[i][r]), v[i][r]);
+    int to = slot;
+    if (to >= 0) (void)MSGL_OOB(to, a.num_slots);
+    if (to >= a.num_slots) to = -1;
+    if (token + (int)gridDim.x < tokens) fetch(token + gridDim.x);
+    float rq = 1.f, rk = 1.f;
+    if (a.q_w != nullptr) {
+      float sq = 0.f, sk = 0.f;
+#pragma unroll
+      for (int i = 0; i < NI; ++i) {
+        const int h = (i * nw + warp) * HPW + lane / LPH;
+        float s = 0.f;
+#pragma unroll
+        for (int r = 0; r < 2; ++r)
+#pragma unroll
+          for (int e = 0; e < 8; ++e) s = fmaf(v[i][r][e], v[i][r][e], s);
+        if (h < a.hq) sq += s;
+        else if (h < a.hq + hk) sk += s;
+        if (h < a.hq + hk) {
+          const float* src = h < a.hq ? a.q_w + h * D : a.k_w + (h - a.hq) * D;
+#pragma unroll
+          for (int r = 0; r < 2; ++r) {
+            float w[8];
+            load8(src + col[r], w);
+#pragma unroll
+            for (int e = 0; e < 8; ++e) v[i][r][e] *= w[e];
+          }
+        }
+      }
+      if (a.totals != nullptr) {
+        sq = a.totals[2 * token];
+        sk = a.totals[2 * token + 1];
+      } else {
+        sq = warp_sum(sq);
+        sk = warp_sum(sk);
+        if (lane == 0) { part[buf][0][warp] = sq; part[buf][1][warp] = sk; }
+        __syncthreads();
+        sq = sk = 0.f;
+        for (int w = 0; w < nw; ++w) { sq += part[buf][0][w]; sk += part[buf][1][w]; }
+      }
+      rq = 1.f / sqrtf(sq / a.q_count + a.eps);
+      if (hk > 0) rk = 1.f / sqrtf(sk / a.k_count + a.eps);
+    }
+#pragma unroll
+    for (int i = 0; i < NI; ++i) {
+      const int h = (i * nw + warp) * HPW + lane / LPH;
+      const bool is_q = h < a.hq, is_v = h >= a.hq + hk;
+      if (turns && !is_v) {
+        if (a.interleaved) {
+#pragma unroll
+          for (int e = 0; e < 8; ++e) {
+            float& v0 = v[i][e >> 2][2 * (e & 3)];
+            float& v1 = v[i][e >> 2][2 * (e & 3) + 1];
+            const float t = v0;
+            v0 = t * cs[e] - v1 * sn[e];
+            v1 = v1 * cs[e] + t * sn[e];
+          }
+        } else {
+#pragma unroll
+          for (int e = 0; e < 8; ++e) {
+            const float t = v[i][0][e];
+            v[i][0][e] = t * cs[e] - v[i][1][e] * sn[e];
+            v[i][1][e] = v[i][1][e] * cs[e] + t * sn[e];
+          }
+        }
+      }
+      float scale = is_v ? 1.f : is_q ? rq : rk;
+      if (a.unit) {
+        float s = 0.f;
+#pragma unroll
+        for (int r = 0; r < 2; ++r)
+#pragma unroll
+          for (int e = 0; e < 8; ++e) s = fmaf(v[i][r][e], v[i][r][e], s);
+#pragma unroll
+        for (int o = 1; o < LPH; o <<= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
+        if (!is_v) scale /= sqrtf(scale * scale * s / (float)a.dim + a.eps);
+      }
+      if (h >= total || (!is_q && to < 0)) continue;
+      T* dst;
+      if (is_q) {
+        dst = reinterpret_cast<T*>(a.q_out) + ((size_t)token * a.hq + h) * D;
+      } else {
+        const int kvh = is_v ? h - a.hq - hk : h - a.hq;
+        dst = reinterpret_cast<T*>(is_v ? a.v_cache : a.k_cache) +
+              (((size_t)(to / a.page_size) * hk + kvh) * a.page_size + to % a.page_size) * D;
+      }
+#pragma unroll
+      for (int r = 0; r < 2; ++r) {
+        if (!is_v && (a.unit || a.q_w != nullptr)) {
+#pragma unroll
+          for (int e = 0; e < 8; ++e) v[i][r][e] *= scale;
+        }
+        store8(dst + col[r], v[i][r]);
+      }
+    }
+    __syncwarp();
+  }
+}
+
+template <typename T, int LPH>
+bool launch_heads_rope_vec(const HeadsRopeArgs& a, int tokens, int heads, cudaStream_t stream) {
+  const int groups = (heads + 32 / LPH - 1) / (32 / LPH);        // warps' worth of heads
+  const int ni = groups <= 12 ? 1 : 2;
+  const int warps = (groups + ni - 1) / ni;
+  if (warps > 12) return false;
+  const dim3 grid(tokens < 148 * 8 ? tokens : 148 * (24 / warps > 1 ? 24 / warps : 1));
+  if (ni == 1) msgl_launch(heads_rope_store_vec_kernel<T, LPH, 1>, grid, dim3(32 * warps), 0, stream, a, tokens);
+  else msgl_launch(heads_rope_store_vec_kernel<T, LPH, 2>, grid, dim3(32 * warps), 0, stream, a, tokens);
+  return true;
+}
+
 }  // namespace
 
 MSGL_API int msgl_heads_rope_store(const void* x, long long ld, const void* q_w, const void* k_w, const void* totals,
@@ -587,6 +753,20 @@ MSGL_API int msgl_heads_rope_store(const void* x, long long ld, const void* q_w,
                   (const int32_t*)positions, (const float*)cos_sin, q_out, k_cache, v_cache, (const int32_t*)out_loc, hq, hk,
                   dim, rot, page_size, interleaved, unit, max_pos, num_slots, eps};
   const int heads = hq + (k_cache != nullptr ? 2 * hk : 0);
+  if (rot % 16 == 0 && ld % 8 == 0 && (uintptr_t)x % 16 == 0 && width <= 256) {
+    bool done = false;
+#define HEADS_ROPE_VEC(T)                                                              \
+  done = width == 64    ? launch_heads_rope_vec<T, 4>(a, tokens, heads, stream)         \
+         : width == 128 ? launch_heads_rope_vec<T, 8>(a, tokens, heads, stream)        \
+         : width == 256 ? launch_heads_rope_vec<T, 16>(a, tokens, heads, stream) : false
+    if (dtype == MSGL_BF16) HEADS_ROPE_VEC(__nv_bfloat16);
+    else if (dtype == MSGL_F32) HEADS_ROPE_VEC(float);
+#undef HEADS_ROPE_VEC
+    if (done) {
+      MSGL_CHECK_LAUNCH("heads_rope_store");
+      return MSGL_OK;
+    }
+  }
   const int warps = heads < 16 ? heads : 16;
   const size_t smem = interleaved ? 0 : (size_t)warps * rot * sizeof(float);
 #define HEADS_ROPE(T, NP) msgl_launch(heads_rope_store_kernel<T, NP>, dim3(tokens), dim3(32 * warps), smem, stream, a)

@@ -69,13 +69,14 @@ class HeadAttentionLayer(BaseOP):
         copies = tp * self._hk // spec.kv_heads        # ranks that hold the same key head
         return get_comm().all_reduce(sums), spec.heads * spec.dim, spec.kv_heads * spec.dim * copies
 
+    def _post_load_self(self) -> None:
+        # what the kernels read past a head's channels is zero, whatever filled the weights
+        spec, d, weight = self._spec, self._d, self.in_proj.weight
+        own = self._hk if self._own else 0
+        for at, n, used in ((0, self._h, spec.dim), (self._h, own, spec.dim), (self._h + own, own, spec.vdim)):
+            weight[at * d:(at + n) * d].view(n, d, weight.shape[1])[:, used:] = 0
+
     def init_dummy(self, gen: torch.Generator, std: float = 0.02) -> None:
-        self.in_proj.init_dummy(gen, std)
-        spec, d = self._spec, self._d
-        rows = self.in_proj.weight
-        for at, n, used in ((0, self._h, spec.dim), (self._h, self._hk if self._own else 0, spec.dim),
-                            (self._h + self._hk, self._hk if self._own else 0, spec.vdim)):
-            rows[at * d:(at + n) * d].view(n, d, -1)[:, used:] = 0
         for name in ("q_norm", "k_norm"):
             if hasattr(self, name):
                 setattr(self, name, torch.ones_like(getattr(self, name)))
