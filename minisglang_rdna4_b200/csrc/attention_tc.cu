@@ -41,6 +41,8 @@ constexpr int kTile = 128;         // query rows per head tile, KV rows per bloc
 constexpr int kPanel = 16384;      // 128 rows x 128 bytes (64 16-bit columns), 128B-swizzled
 constexpr int kTcThreads = 384;   // warps 0-3: TMA / MMA / two idle; warps 4-7, 8-11: one head each
 constexpr float kLog2eTc = 1.4426950408889634f;
+constexpr float kFixedCap = 80.f;  // capped scores (in units of log2) up to this need no running maximum: 2^score, summed
+                                   // over any number of keys, stays far from both ends of the fp32 and bf16 ranges
 
 struct TcItem {        // one per (request, block of 128 query positions); eight int32
   int q_row0;          // first row of the tile in the packed q / out tensors
@@ -66,8 +68,7 @@ struct TcArgs {
   int window;          // > 0: a row sees the last ``window`` positions, its own included
   int chunk;           // > 0: a row sees its own block of this many positions only
   float softcap;       // c > 0: scores go through c tanh(s / c)
-  const void* cgate;   // [rows, Hq * ho] logits of a sigmoid gate per output channel (row stride ldcg), or null
-  long long ldcg;
+  int cgate;           // a sigmoid gate per output channel: its logits come through tma_g, in the layout of q
   long long ldo, ho;   // element strides of a row and a head of out
   int v_chunks;        // 16-byte chunks of a value head
   const float* sink;   // [Hq] logits that only the softmax denominator counts, or null
@@ -82,7 +83,7 @@ struct TcSmem {
   static constexpr int off_p = 4 * kPanel;              // [2 heads][2 panels]
   static constexpr int off_kv = 8 * kPanel;             // [3 slots][2 panels]
   static constexpr int off_bar = 14 * kPanel;
-  static constexpr int n_bars = 1 + 3 + 3 + 2 * 5;
+  static constexpr int n_bars = 1 + 3 + 3 + 2 * 5 + 2;
   static constexpr int bytes = off_bar + 256 + 1024;    // + slack to align the base to 1024
 };
 
@@ -91,6 +92,45 @@ __device__ __forceinline__ float ex2f(float x) {
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
 }
+// two fp32 operations per instruction
+__device__ __forceinline__ uint64_t f2(float a, float b) {
+  uint64_t r;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
+  return r;
+}
+__device__ __forceinline__ void unf2(uint64_t x, float& a, float& b) { asm("mov.b64 {%0, %1}, %2;" : "=f"(a), "=f"(b) : "l"(x)); }
+__device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b) {
+  uint64_t r;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+  return r;
+}
+__device__ __forceinline__ uint64_t add2(uint64_t a, uint64_t b) {
+  uint64_t r;
+  asm("add.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+  return r;
+}
+__device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
+  uint64_t r;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+  return r;
+}
+// 2^(cap_out tanh(x)) of four scores with cap_in s = 2 x log2(e): tanh(x) = 1 - 2 / (1 + e^(2x)), one reciprocal for the
+// four (exponents held at 30, where tanh is 1 in fp32, so that the product stays finite)
+__device__ __forceinline__ void capped_exp2(uint32_t* s, uint64_t cap_in, float m2cap, uint64_t cap_out, float (&p)[4]) {
+  const uint64_t one = f2(1.f, 1.f);
+  float a0, a1, b0, b1, t0, t1;
+  unf2(mul2(f2(__uint_as_float(s[0]), __uint_as_float(s[1])), cap_in), a0, a1);
+  unf2(mul2(f2(__uint_as_float(s[2]), __uint_as_float(s[3])), cap_in), b0, b1);
+  const uint64_t a = add2(f2(ex2f(fminf(a0, 30.f)), ex2f(fminf(a1, 30.f))), one);
+  const uint64_t b = add2(f2(ex2f(fminf(b0, 30.f)), ex2f(fminf(b1, 30.f))), one);
+  unf2(mul2(a, b), t0, t1);
+  const float r = __fdividef(m2cap, t0 * t1);
+  const uint64_t rr = f2(r * t1, r * t0);
+  unf2(fma2(rr, b, cap_out), a0, a1);
+  unf2(fma2(rr, a, cap_out), b0, b1);
+  p[0] = ex2f(a0); p[1] = ex2f(a1); p[2] = ex2f(b0); p[3] = ex2f(b1);
+}
+
 template <typename T> __device__ __forceinline__ uint32_t pack2_tc(float a, float b);
 template <> __device__ __forceinline__ uint32_t pack2_tc<__nv_bfloat16>(float a, float b) {
   __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
@@ -181,10 +221,12 @@ kv_gather_kernel(const void* __restrict__ k_pool, const void* __restrict__ v_poo
 // ------------------------------------------------------------------------------------------
 // POS: the two tiles of a CTA are consecutive blocks of 128 positions of one head (where query heads that share keys
 // and values do not come in pairs, K / V tiles can only be shared along the positions) instead of two heads.
-template <typename T, bool POS>
+// FIXCAP: scores are capped within kFixedCap.
+template <typename T, bool POS, bool FIXCAP>
 __global__ void __launch_bounds__(kTcThreads, 1)
 attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_constant__ CUtensorMap tma_k,
-                       const __grid_constant__ CUtensorMap tma_v, const TcArgs args) {
+                       const __grid_constant__ CUtensorMap tma_v, const __grid_constant__ CUtensorMap tma_g,
+                       const TcArgs args) {
   pdl_enter();
   extern __shared__ uint8_t smem_raw[];
   const uint32_t raw = smem_u32(smem_raw);
@@ -208,6 +250,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
   auto s_free = [&](int t) { return bar(8 + 5 * t); };
   auto p_full = [&](int t) { return bar(9 + 5 * t); };
   auto o_full = [&](int t) { return bar(10 + 5 * t); };
+  auto g_full = [&](int t) { return bar(17 + t); };
   volatile uint32_t* tmem_slot = reinterpret_cast<volatile uint32_t*>(smem + TcSmem::off_bar + 8 * TcSmem::n_bars);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(smem + TcSmem::off_bar + 8 * TcSmem::n_bars + 8);
 
@@ -219,6 +262,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
       mbar_init(s_free(t), 128);
       mbar_init(p_full(t), 128);
       mbar_init(o_full(t), 1);
+      mbar_init(g_full(t), 1);
     }
     *abort_flag = 0;
     fence_barrier_init();
@@ -335,9 +379,9 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
     const uint32_t swz = (uint32_t)(row & 7);
     const float raw_scale = args.scale * kLog2eTc * (args.k_scale != nullptr ? args.k_scale[hk] : 1.f);
     // capped scores come out in units of log2: tanh(x) = 1 - 2 / (1 + e^(2x))
-    const bool capped = args.softcap > 0.f;
+    const bool capped = !FIXCAP && args.softcap > 0.f;
     const float sl2 = capped ? 1.f : raw_scale;
-    const float cap_in = capped ? 2.f * raw_scale / args.softcap : 0.f, cap_out = args.softcap * kLog2eTc;
+    const float cap_in = FIXCAP || capped ? 2.f * raw_scale / args.softcap : 0.f, cap_out = args.softcap * kLog2eTc;
     auto below = [&](int pos) {                        // last position ahead of what a row at pos sees
       int lo = -1;
       if (args.window > 0) lo = pos - args.window;
@@ -360,11 +404,58 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
       const bool masked = kv0 + kTile - 1 > tile_pos0 || kv0 <= lo_last;
       if (!mbar_wait(s_full(t), (uint32_t)(j & 1), abort_flag, args.status, 209)) { ok = false; break; }
       tc_fence_after();
+      if (args.cgate && j == nb - 1 && row == 0) {
+        // the last product with the query tile is done: the gate's tile takes its place while this block is worked on
+        mbar_expect_tx(g_full(t), 2 * kPanel);
+        for (int p = 0; p < 2; ++p)
+          tma_load_3d(q_s + (t * 2 + p) * kPanel, &tma_g, g_full(t), 64 * p, head, it.q_row0 + (POS ? t * kTile : 0));
+      }
 #pragma unroll
       for (int c = 0; c < 4; ++c) tmem_ld_32x32b_x32(s_addr + c * 32, s[c]);
       tmem_ld_wait();
       tc_fence_before();
       mbar_arrive(s_free(t));                             // S is in registers: the next QK^T may start
+      if constexpr (FIXCAP) {
+        uint64_t sum = 0;
+#pragma unroll
+        for (int c = 0; c < 4; ++c) {
+#pragma unroll
+          for (int i = 0; i < 32; i += 4) {
+            float p[4];
+            capped_exp2(&s[c][i], f2(cap_in, cap_in), -2.f * cap_out, f2(cap_out, cap_out), p);
+            if (masked) {
+#pragma unroll
+              for (int e = 0; e < 4; ++e) {
+                const int tok = kv0 + c * 32 + i + e;
+                p[e] = tok > q_pos || tok <= lo ? 0.f : p[e];
+              }
+            }
+            sum = add2(sum, add2(f2(p[0], p[1]), f2(p[2], p[3])));
+            s[c][i >> 1] = pack2_tc<T>(p[0], p[1]);
+            s[c][(i >> 1) + 1] = pack2_tc<T>(p[2], p[3]);
+          }
+        }
+        float s0, s1;
+        unf2(sum, s0, s1);
+        l += s0 + s1;
+        // P V of the previous block is complete: the P buffer is free
+        if (j > 0 && !mbar_wait(o_full(t), (uint32_t)((j - 1) & 1), abort_flag, args.status, 210)) { ok = false; break; }
+#pragma unroll
+        for (int c = 0; c < 4; ++c) {
+          const uint32_t panel = p_row + (uint32_t)(c >> 1) * kPanel;
+#pragma unroll
+          for (int g = 0; g < 4; ++g) {
+            const uint32_t u = (uint32_t)((c & 1) * 4 + g);
+            asm volatile("st.shared.v4.b32 [%0], {%1, %2, %3, %4};" ::"r"(panel + ((u ^ swz) << 4)), "r"(s[c][g * 4]),
+                         "r"(s[c][g * 4 + 1]), "r"(s[c][g * 4 + 2]), "r"(s[c][g * 4 + 3])
+                         : "memory");
+          }
+        }
+        tc_fence_before();
+        fence_proxy_async();
+        mbar_arrive(p_full(t));
+        continue;
+      }
       float mx = -INFINITY;
       if (capped) {
 #pragma unroll
@@ -444,7 +535,8 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
       fence_proxy_async();
       mbar_arrive(p_full(t));
     }
-    if (ok && nb > 0 && mbar_wait(o_full(t), (uint32_t)((nb - 1) & 1), abort_flag, args.status, 211)) {
+    if (ok && nb > 0 && mbar_wait(o_full(t), (uint32_t)((nb - 1) & 1), abort_flag, args.status, 211) &&
+        (!args.cgate || mbar_wait(g_full(t), 0, abort_flag, args.status, 212))) {
       tc_fence_after();
       const int out_row = row + (POS ? t * kTile : 0);
       float num = args.v_scale != nullptr ? args.v_scale[hk] : 1.f;
@@ -458,9 +550,6 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
         num *= 1.f / (1.f + __expf(-to_float(reinterpret_cast<const T*>(args.gate)[(it.q_row0 + out_row) * args.ldg + head])));
       const float inv = l > 0.f ? num / l : 0.f;
       T* dst = reinterpret_cast<T*>(args.out) + (long long)(it.q_row0 + out_row) * args.ldo + head * args.ho;
-      const T* cg = args.cgate != nullptr
-                        ? reinterpret_cast<const T*>(args.cgate) + (it.q_row0 + out_row) * args.ldcg + head * args.ho
-                        : nullptr;
 #pragma unroll
       for (int c = 0; c < 4; ++c) tmem_ld_32x32b_x32(o_addr + c * 32, s[c]);
       tmem_ld_wait();
@@ -469,9 +558,11 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
         for (int c = 0; c < 16; ++c) {
           if (c >= args.v_chunks) break;
           uint32_t* o = &s[c >> 2][(c & 3) * 8];
-          if (cg != nullptr) {
+          if (args.cgate) {
             float g[8];
-            load8(cg + 8 * c, g);
+            load8(reinterpret_cast<const T*>(smem + TcSmem::off_q + (t * 2 + (c >> 3)) * kPanel + row * 128 +
+                                             (((c & 7) ^ (row & 7)) << 4)),
+                  g);
 #pragma unroll
             for (int e = 0; e < 8; ++e)
               o[e] = __float_as_uint(__uint_as_float(o[e]) * __fdividef(1.f, 1.f + ex2f(-kLog2eTc * g[e])));
@@ -484,6 +575,9 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
           *reinterpret_cast<uint4*>(dst + 8 * c) = v;
         }
       }
+    } else if (args.cgate && row == 0) {       // gave up: let the gate's copies land before the CTA exits
+      const uint64_t t0 = globaltimer_ns();
+      while (globaltimer_ns() - t0 < 200000ull) __nanosleep(1000);
     }
   }
   tc_fence_before();
@@ -507,17 +601,17 @@ bool encode_map(CUtensorMap* map, const void* base, int rank, const cuuint64_t* 
   return true;
 }
 
-template <typename T, bool POS>
-int launch_tc(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const TcArgs& a,
+template <typename T, bool POS, bool FIXCAP = false>
+int launch_tc(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const CUtensorMap& mg, const TcArgs& a,
               cudaStream_t stream) {
   static bool configured = false;
   if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(attn_prefill_tc_kernel<T, POS>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+    cudaError_t e = cudaFuncSetAttribute(attn_prefill_tc_kernel<T, POS, FIXCAP>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                          TcSmem::bytes);
     if (e != cudaSuccess) { msgl_set_error("prefill attention smem attribute", e); return MSGL_CUDA_ERROR; }
     configured = true;
   }
-  msgl_launch(attn_prefill_tc_kernel<T, POS>, dim3(a.n_items * a.pairs), dim3(kTcThreads), TcSmem::bytes, stream, mq, mk, mv, a);
+  msgl_launch(attn_prefill_tc_kernel<T, POS, FIXCAP>, dim3(a.n_items * a.pairs), dim3(kTcThreads), TcSmem::bytes, stream, mq, mk, mv, mg, a);
   MSGL_CHECK_LAUNCH("attn_prefill_tc");
   return MSGL_OK;
 }
@@ -596,7 +690,7 @@ MSGL_API int msgl_attn_prefill_pos(const void* q, long long ldq, long long hq_st
   a.items = (const TcItem*)items; a.n_items = n_items; a.pairs = h; a.Hq = h; a.Hk = h; a.t_cap = t_pad;
   a.out = out; a.scale = scale; a.status = status; a.window = window; a.ldo = ldo; a.ho = ho; a.v_chunks = dv / 8;
   a.sink = (const float*)sink; a.gate = gate; a.ldg = ldg;
-  return launch_tc<__nv_bfloat16, true>(mq, mk, mv, a, stream);
+  return launch_tc<__nv_bfloat16, true>(mq, mk, mv, mq, a, stream);
 }
 
 // Causal prefill / extend attention for one layer. `kc` / `vt` are scratch buffers of
@@ -620,12 +714,15 @@ MSGL_API int msgl_attn_prefill_tc(const void* q, long long q_row_stride, void* o
                         "and a scratch of whole blocks");
     return MSGL_BAD_ARG;
   }
-  CUtensorMap mq, mk, mv;
+  CUtensorMap mq, mk, mv, mg;
   {
     cuuint64_t dims[3] = {(cuuint64_t)d, (cuuint64_t)hq, (cuuint64_t)total_q};
     cuuint64_t strides[2] = {(cuuint64_t)d * 2, (cuuint64_t)q_row_stride * 2};
     cuuint32_t box[3] = {64, 1, 128};
     if (!encode_map(&mq, q, 3, dims, strides, box, "q")) return MSGL_CUDA_ERROR;
+    mg = mq;
+    strides[1] = (cuuint64_t)ldg * 2;
+    if (gate != nullptr && !encode_map(&mg, gate, 3, dims, strides, box, "gate")) return MSGL_CUDA_ERROR;
   }
   if (pos_form) {
     cuuint64_t kdims[3] = {(cuuint64_t)kD, (cuuint64_t)hk, (cuuint64_t)t_cap};
@@ -659,17 +756,20 @@ MSGL_API int msgl_attn_prefill_tc(const void* q, long long q_row_stride, void* o
   TcArgs a = {};
   a.items = (const TcItem*)items; a.n_items = n_items; a.pairs = pos_form ? hq : hq / 2; a.Hq = hq; a.Hk = hk;
   a.t_cap = t_cap; a.out = out; a.k_scale = (const float*)k_scale; a.v_scale = (const float*)v_scale; a.scale = scale;
-  a.status = status; a.window = window; a.chunk = chunk; a.softcap = softcap; a.cgate = gate; a.ldcg = ldg;
+  a.status = status; a.window = window; a.chunk = chunk; a.softcap = softcap; a.cgate = gate != nullptr;
   a.ldo = (long long)hq * d; a.ho = d; a.v_chunks = d / 8;
+  const bool fixcap = softcap > 0.f && softcap * kLog2eTc <= kFixedCap && dtype == MSGL_BF16;
   if (pos_form) {
     if (dtype != MSGL_BF16) {
       msgl_set_error_text("prefill attention: bf16 where query heads do not come in pairs");
       return MSGL_BAD_ARG;
     }
-    return launch_tc<__nv_bfloat16, true>(mq, mk, mv, a, stream);
+    return fixcap ? launch_tc<__nv_bfloat16, true, true>(mq, mk, mv, mg, a, stream)
+                  : launch_tc<__nv_bfloat16, true>(mq, mk, mv, mg, a, stream);
   }
-  if (dtype == MSGL_BF16) return launch_tc<__nv_bfloat16, false>(mq, mk, mv, a, stream);
-  return launch_tc<__half, false>(mq, mk, mv, a, stream);
+  if (fixcap) return launch_tc<__nv_bfloat16, false, true>(mq, mk, mv, mg, a, stream);
+  if (dtype == MSGL_BF16) return launch_tc<__nv_bfloat16, false>(mq, mk, mv, mg, a, stream);
+  return launch_tc<__half, false>(mq, mk, mv, mg, a, stream);
 }
 
 MSGL_API int msgl_attn_tc_status(int reset) {

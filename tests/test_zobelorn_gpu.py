@@ -225,13 +225,17 @@ def test_a_loud_key_is_seen_exactly_within_reach(form, kind, size, at):
     assert [bool(x) for x in got[:, 0, 0] > 4.5] == want
 
 
+@pytest.mark.parametrize("cap", [0.25, 4.0, 50.0, 60.0, 300.0])
 @pytest.mark.parametrize("form", ["general", "tc"])
-def test_capped_scores_far_out(form):
-    """Scores many times the cap, of both signs, in both kernels: the weights are those of the capped scores."""
-    n, d, ps, cap = 130, 64, 16, 4.0
+def test_capped_scores_far_out(form, cap):
+    """Scores many times the cap (and of its size), of both signs, in both kernels: the weights are those of the capped
+    scores, also where a row's keys all score close to the negative cap."""
+    n, d, ps = 130, 64, 16
     g = _gen(3)
     k, v = (torch.randn(9, 1, ps, d, generator=g).to(BF) for _ in range(2))
-    q = (torch.randn(n, 2, d, generator=g) * 200).to(BF)
+    q = (torch.randn(n, 2, d, generator=g) * torch.tensor([0.1, 1.0, 8.0, 60.0, 200.0]).repeat(26)[:, None, None]).to(BF)
+    k[..., 0] = 3.0
+    q[7::10, :, 0] = -cap
     bt = torch.randperm(9, generator=g).int()[None]
     cu, seq = torch.tensor([0, n], dtype=torch.int32), torch.tensor([n], dtype=torch.int32)
     want = ref.paged_attention(q.float(), k.float(), v.float(), bt, cu, seq, 1.0, softcap=cap)
