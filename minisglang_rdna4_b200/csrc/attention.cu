@@ -58,10 +58,10 @@ struct AttnArgs {
 __device__ int g_attn_status = 0;
 
 // first position that a row at pos can see
-__device__ __forceinline__ int first_visible(const AttnArgs& a, int pos) {
+template <bool EXT> __device__ __forceinline__ int first_visible(const AttnArgs& a, int pos) {
   int lo = 0;
   if (a.window > 0) lo = max(lo, pos - a.window + 1);
-  if (a.chunk > 0) lo = max(lo, pos - pos % a.chunk);
+  if (EXT && a.chunk > 0) lo = max(lo, pos - pos % a.chunk);
   return lo;
 }
 
@@ -118,7 +118,8 @@ __device__ __forceinline__ uint32_t pack_bf16x2(float a, float b) {
 // that take turns on the KV tiles (warp wk owns tiles wk, wk + NWK, ...) and merge their partial
 // softmax states at the end. Prefill uses 4 x 1, decode 1 x 4: a decode CTA has only one 16-row
 // tile of queries, so its parallelism has to come from the KV axis.
-template <typename T, bool KV8, int D, int NWQ, int NWK, int STAGES>
+// EXT: the form with chunks, a soft cap and an output gate.
+template <typename T, bool KV8, int D, int NWQ, int NWK, int STAGES, bool EXT>
 __global__ void __launch_bounds__(32 * (NWQ * NWK + 1))
 paged_attention_kernel(const __grid_constant__ CUtensorMap kv_map, const AttnArgs args) {
   pdl_enter();
@@ -159,7 +160,7 @@ paged_attention_kernel(const __grid_constant__ CUtensorMap kv_map, const AttnArg
   const bool use_mask = args.mask != nullptr;
   int kv_hi = (args.causal && !use_mask) ? min(kv_len, kv_len - q_len + q_end) : kv_len;
   int kv_lo = 0;
-  if (!use_mask) kv_lo = first_visible(args, kv_len - q_len + q_start);
+  if (!use_mask) kv_lo = first_visible<EXT>(args, kv_len - q_len + q_start);
   const int tile_lo = kv_lo / TK;
   const int n_tiles_all = kv_hi > kv_lo ? (kv_hi + TK - 1) / TK - tile_lo : 0;
   const int per_split = (n_tiles_all + args.splits - 1) / args.splits;
@@ -256,7 +257,7 @@ paged_attention_kernel(const __grid_constant__ CUtensorMap kv_map, const AttnArg
 
   const float k_sc = args.k_scale != nullptr ? args.k_scale[h] : 1.f;
   const float v_sc = args.v_scale != nullptr ? args.v_scale[h] : 1.f;
-  const bool capped = args.softcap > 0.f;
+  const bool capped = EXT && args.softcap > 0.f;
   const float sm_scale = capped ? 1.f : args.scale * k_sc * kLog2e;
   const float cap_in = capped ? 2.f * kLog2e * args.scale * k_sc / args.softcap : 0.f, cap_out = args.softcap * kLog2e;
   // per-row visible KV interval [lo, hi)
@@ -264,8 +265,10 @@ paged_attention_kernel(const __grid_constant__ CUtensorMap kv_map, const AttnArg
   int hi_a = kv_len, hi_b = kv_len, lo_a = 0, lo_b = 0;
   if (!use_mask) {
     if (args.causal) { hi_a = min(kv_len, pos_a + 1); hi_b = min(kv_len, pos_b + 1); }
-    lo_a = first_visible(args, pos_a);
-    lo_b = first_visible(args, pos_b);
+    if (EXT || args.window > 0) {
+      lo_a = first_visible<EXT>(args, pos_a);
+      lo_b = first_visible<EXT>(args, pos_b);
+    }
   }
   if (!ok_a) hi_a = 0;
   if (!ok_b) hi_b = 0;
@@ -480,7 +483,7 @@ paged_attention_kernel(const __grid_constant__ CUtensorMap kv_map, const AttnArg
   if (args.splits == 1) {
     T* oa = reinterpret_cast<T*>(args.out) + qoff_a;
     T* ob = reinterpret_cast<T*>(args.out) + qoff_b;
-    if (!KV8 && args.gate != nullptr) {
+    if (EXT && args.gate != nullptr) {
       const T* ga = reinterpret_cast<const T*>(args.gate) + (q_begin + (ok_a ? qi_a : q_start)) * args.ldg + head_a * D + 2 * j;
       const T* gb = reinterpret_cast<const T*>(args.gate) + (q_begin + (ok_b ? qi_b : q_start)) * args.ldg + head_b * D + 2 * j;
 #pragma unroll
@@ -595,7 +598,7 @@ __device__ __forceinline__ uint32_t movmatrix_trans(uint32_t x) {
   return y;
 }
 
-template <typename T, bool KV8, int D, int STAGES>
+template <typename T, bool KV8, int D, int STAGES, bool EXT>
 __global__ void __launch_bounds__(64)
 paged_decode_kernel(const __grid_constant__ CUtensorMap kv_map, const AttnArgs args) {
   // This kernel starts once the kernel ahead of it (the one that writes this step's q and the
@@ -628,7 +631,7 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap kv_map, const AttnArgs a
   const int q_row = args.cu_q[b];
   const int kv_len = args.seq_lens[b];
   const int kv_hi = kv_len;
-  const int kv_lo = first_visible(args, kv_len - 1);
+  const int kv_lo = first_visible<EXT>(args, kv_len - 1);
   const int tile_lo = kv_lo / TK;
   const int n_tiles_all = kv_hi > kv_lo ? (kv_hi + TK - 1) / TK - tile_lo : 0;
   const int per_split = (n_tiles_all + args.splits - 1) / args.splits;
@@ -714,7 +717,7 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap kv_map, const AttnArgs a
   }
   const float k_sc = args.k_scale != nullptr ? args.k_scale[h] : 1.f;
   const float v_sc = args.v_scale != nullptr ? args.v_scale[h] : 1.f;
-  const bool capped = args.softcap > 0.f;
+  const bool capped = EXT && args.softcap > 0.f;
   const float sm_scale = capped ? 1.f : args.scale * k_sc * kLog2e;
   const float cap_in = capped ? 2.f * kLog2e * args.scale * k_sc / args.softcap : 0.f, cap_out = args.softcap * kLog2e;
 
@@ -862,7 +865,7 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap kv_map, const AttnArgs a
   if (args.splits == 1) {
     T* o0 = reinterpret_cast<T*>(args.out) + ((size_t)q_row * args.Hq + head0) * D;
     T* o1 = reinterpret_cast<T*>(args.out) + ((size_t)q_row * args.Hq + head1) * D;
-    if (!KV8 && args.gate != nullptr) {
+    if (EXT && args.gate != nullptr) {
       const T* g0 = reinterpret_cast<const T*>(args.gate) + q_row * args.ldg + (ok0 ? head0 : h * G) * D + g;
       const T* g1 = reinterpret_cast<const T*>(args.gate) + q_row * args.ldg + (ok1 ? head1 : h * G) * D + g;
 #pragma unroll
@@ -903,24 +906,24 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap kv_map, const AttnArgs a
   }
 }
 
-template <typename T, bool KV8, int D, int STAGES>
+template <typename T, bool KV8, int D, int STAGES, bool EXT = false>
 int launch_decode(const CUtensorMap& map, const AttnArgs& a, cudaStream_t stream) {
   constexpr int ESZ = KV8 ? 1 : 2;
   constexpr int smem = STAGES * 2 * (D * ESZ / 128) * TK * 128 + 16 * STAGES + 64 + 1024;
   static bool configured = false;
   if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(paged_decode_kernel<T, KV8, D, STAGES>,
+    cudaError_t e = cudaFuncSetAttribute(paged_decode_kernel<T, KV8, D, STAGES, EXT>,
                                          cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
     if (e != cudaSuccess) { msgl_set_error("decode attention smem attribute", e); return MSGL_CUDA_ERROR; }
     configured = true;
   }
   dim3 grid(1, a.B * a.Hk, a.splits);
-  msgl_launch(paged_decode_kernel<T, KV8, D, STAGES>, dim3(grid), dim3(64), smem, stream, map, a);
+  msgl_launch(paged_decode_kernel<T, KV8, D, STAGES, EXT>, dim3(grid), dim3(64), smem, stream, map, a);
   MSGL_CHECK_LAUNCH("paged_decode");
   return MSGL_OK;
 }
 
-template <typename T, bool KV8, int D, int NWQ, int NWK, int STAGES>
+template <typename T, bool KV8, int D, int NWQ, int NWK, int STAGES, bool EXT = false>
 int launch_attn(const CUtensorMap& map, const AttnArgs& a, int q_tiles, cudaStream_t stream) {
   constexpr int ESZ = KV8 ? 1 : 2;
   constexpr int NW = NWQ * NWK;
@@ -929,19 +932,43 @@ int launch_attn(const CUtensorMap& map, const AttnArgs& a, int q_tiles, cudaStre
                 "merge buffer must fit in the stage memory");
   static bool configured = false;
   if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(paged_attention_kernel<T, KV8, D, NWQ, NWK, STAGES>,
+    cudaError_t e = cudaFuncSetAttribute(paged_attention_kernel<T, KV8, D, NWQ, NWK, STAGES, EXT>,
                                          cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
     if (e != cudaSuccess) { msgl_set_error("attention smem attribute", e); return MSGL_CUDA_ERROR; }
     configured = true;
   }
   dim3 grid(q_tiles, a.B * a.Hk, a.splits);
-  msgl_launch(paged_attention_kernel<T, KV8, D, NWQ, NWK, STAGES>, dim3(grid), dim3(32 * (NW + 1)), smem, stream, map, a);
+  msgl_launch(paged_attention_kernel<T, KV8, D, NWQ, NWK, STAGES, EXT>, dim3(grid), dim3(32 * (NW + 1)), smem, stream, map, a);
   MSGL_CHECK_LAUNCH("paged_attention");
   return MSGL_OK;
 }
 
 bool g_force_general_decode = false;
 int g_decode_stages = 2;   // shared-memory stages of the fp8 decode kernel (2, 3 or 4)
+
+// the form with chunks, a soft cap and an output gate: 16-bit pools
+template <typename T>
+int dispatch_attn_ext(const CUtensorMap& map, const AttnArgs& a, int d, int max_q, cudaStream_t stream) {
+  const int G = a.Hq / a.Hk;
+  if (max_q == 1 && G <= 8 && !g_force_general_decode) {
+    if (d == 128) return launch_decode<T, false, 128, 2, true>(map, a, stream);
+    if (d == 64) return launch_decode<T, false, 64, 3, true>(map, a, stream);
+  }
+  const bool small = max_q * G <= 16;
+  const int rows = small ? 16 : 64;
+  const int q_tiles = (max_q + rows / G - 1) / (rows / G);
+  if (d == 128)
+    return small ? launch_attn<T, false, 128, 1, 1, 3, true>(map, a, q_tiles, stream)
+                 : launch_attn<T, false, 128, 4, 1, 3, true>(map, a, q_tiles, stream);
+  if (d == 64)
+    return small ? launch_attn<T, false, 64, 1, 1, 3, true>(map, a, q_tiles, stream)
+                 : launch_attn<T, false, 64, 4, 1, 4, true>(map, a, q_tiles, stream);
+  if (d == 256)
+    return small ? launch_attn<T, false, 256, 1, 1, 2, true>(map, a, q_tiles, stream)
+                 : launch_attn<T, false, 256, 4, 1, 2, true>(map, a, q_tiles, stream);
+  msgl_set_error_text("attention: unsupported head_dim");
+  return MSGL_BAD_ARG;
+}
 
 template <typename T>
 int dispatch_attn(const CUtensorMap& map, const AttnArgs& a, bool kv8, int d, int max_q, cudaStream_t stream) {
@@ -1025,8 +1052,9 @@ MSGL_API int msgl_paged_attention(const void* kv_map, const void* q, void* out, 
     msgl_set_error_text("attention: up to 64 query heads per key / value head");
     return MSGL_BAD_ARG;
   }
-  if (gate != nullptr && kv_fp8) {
-    msgl_set_error_text("attention: no output gate with an fp8 pool");
+  const bool ext = chunk > 0 || softcap > 0.f || gate != nullptr;
+  if (ext && (kv_fp8 || mask != nullptr || dtype != MSGL_BF16)) {
+    msgl_set_error_text("attention: chunks, soft caps and output gates need a bf16 pool and take no mask");
     return MSGL_BAD_ARG;
   }
   if (splits < 1) splits = 1;
@@ -1052,7 +1080,8 @@ MSGL_API int msgl_paged_attention(const void* kv_map, const void* q, void* out, 
   a.status = status;
   const CUtensorMap& map = *reinterpret_cast<const CUtensorMap*>(kv_map);
   int rc;
-  if (dtype == MSGL_BF16) rc = dispatch_attn<__nv_bfloat16>(map, a, kv_fp8 != 0, head_dim, max_q, stream);
+  if (ext) rc = dispatch_attn_ext<__nv_bfloat16>(map, a, head_dim, max_q, stream);
+  else if (dtype == MSGL_BF16) rc = dispatch_attn<__nv_bfloat16>(map, a, kv_fp8 != 0, head_dim, max_q, stream);
   else if (dtype == MSGL_F16) rc = dispatch_attn<__half>(map, a, kv_fp8 != 0, head_dim, max_q, stream);
   else return MSGL_BAD_ARG;
   if (rc) return rc;

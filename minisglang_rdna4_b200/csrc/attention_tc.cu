@@ -170,11 +170,11 @@ template <typename T> __device__ __forceinline__ uint4 widen8(uint2 b) {
   return o;
 }
 
-template <typename T, bool KV8>
+template <typename T, bool KV8, int ROW>
 __global__ void __launch_bounds__(256)
 kv_gather_kernel(const void* __restrict__ k_pool, const void* __restrict__ v_pool, T* __restrict__ kc,
                  T* __restrict__ vt, const int* __restrict__ blk_req, const int* __restrict__ req_info,
-                 const int* __restrict__ block_table, int bt_stride, int Hk, int page_size, long long t_cap, int d) {
+                 const int* __restrict__ block_table, int bt_stride, int Hk, int page_size, long long t_cap) {
   pdl_enter();
   __shared__ __align__(16) T vs[64][kD + 8];
   const int t0 = blockIdx.x * 64, h = blockIdx.y;
@@ -186,9 +186,9 @@ kv_gather_kernel(const void* __restrict__ k_pool, const void* __restrict__ v_poo
     const int tt = id >> 4, c = id & 15;
     const int tok = t0 + tt - kv_off + kv_lo;
     uint4 kq = make_uint4(0, 0, 0, 0), vq = make_uint4(0, 0, 0, 0);
-    if (tok >= kv_lo && tok < kv_len && c * 8 < d) {
+    if (tok >= kv_lo && tok < kv_len && c * 8 < ROW) {
       const int page = block_table[(long long)req * bt_stride + tok / page_size];
-      const long long src = (((long long)page * Hk + h) * page_size + tok % page_size) * d + c * 8;
+      const long long src = (((long long)page * Hk + h) * page_size + tok % page_size) * ROW + c * 8;
       if constexpr (KV8) {
         kq = widen8<T>(*reinterpret_cast<const uint2*>(reinterpret_cast<const uint8_t*>(k_pool) + src));
         vq = widen8<T>(*reinterpret_cast<const uint2*>(reinterpret_cast<const uint8_t*>(v_pool) + src));
@@ -221,13 +221,16 @@ kv_gather_kernel(const void* __restrict__ k_pool, const void* __restrict__ v_poo
 // ------------------------------------------------------------------------------------------
 // POS: the two tiles of a CTA are consecutive blocks of 128 positions of one head (where query heads that share keys
 // and values do not come in pairs, K / V tiles can only be shared along the positions) instead of two heads.
-// FIXCAP: scores are capped within kFixedCap.
-template <typename T, bool POS, bool FIXCAP>
+// MODE: plain (for two heads: no reach, rows of 128), extended (reach, soft cap, gate, narrower rows), or extended with
+// scores that are capped within kFixedCap.
+enum { TC_PLAIN = 0, TC_EXTENDED = 1, TC_FIXED_CAP = 2 };
+template <typename T, bool POS, int MODE>
 __global__ void __launch_bounds__(kTcThreads, 1)
 attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_constant__ CUtensorMap tma_k,
                        const __grid_constant__ CUtensorMap tma_v, const __grid_constant__ CUtensorMap tma_g,
                        const TcArgs args) {
   pdl_enter();
+  constexpr bool EXT = MODE != TC_PLAIN, FIXCAP = MODE == TC_FIXED_CAP, REACH = POS || EXT;
   extern __shared__ uint8_t smem_raw[];
   const uint32_t raw = smem_u32(smem_raw);
   const uint32_t s_base = (raw + 1023u) & ~1023u;
@@ -379,13 +382,13 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
     const uint32_t swz = (uint32_t)(row & 7);
     const float raw_scale = args.scale * kLog2eTc * (args.k_scale != nullptr ? args.k_scale[hk] : 1.f);
     // capped scores come out in units of log2: tanh(x) = 1 - 2 / (1 + e^(2x))
-    const bool capped = !FIXCAP && args.softcap > 0.f;
+    const bool capped = EXT && !FIXCAP && args.softcap > 0.f, gated = EXT && args.cgate;
     const float sl2 = capped ? 1.f : raw_scale;
     const float cap_in = FIXCAP || capped ? 2.f * raw_scale / args.softcap : 0.f, cap_out = args.softcap * kLog2eTc;
     auto below = [&](int pos) {                        // last position ahead of what a row at pos sees
       int lo = -1;
-      if (args.window > 0) lo = pos - args.window;
-      if (args.chunk > 0) lo = max(lo, pos - pos % args.chunk - 1);
+      if (REACH && args.window > 0) lo = pos - args.window;
+      if (EXT && args.chunk > 0) lo = max(lo, pos - pos % args.chunk - 1);
       return lo;
     };
     const int lo = below(q_pos), lo_last = below(tile_pos0 + kTile - 1);
@@ -399,12 +402,12 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
     uint32_t s[4][32];
     bool ok = true;
     for (int j = 0; j < nb; ++j) {
-      const int kv0 = it.kv_pos0 + j * kTile;
+      const int kv0 = (REACH ? it.kv_pos0 : 0) + j * kTile;
       // the block reaches past some row's position, or starts below some row's window or chunk
-      const bool masked = kv0 + kTile - 1 > tile_pos0 || kv0 <= lo_last;
+      const bool masked = kv0 + kTile - 1 > tile_pos0 || (REACH && kv0 <= lo_last);
       if (!mbar_wait(s_full(t), (uint32_t)(j & 1), abort_flag, args.status, 209)) { ok = false; break; }
       tc_fence_after();
-      if (args.cgate && j == nb - 1 && row == 0) {
+      if (gated && j == nb - 1 && row == 0) {
         // the last product with the query tile is done: the gate's tile takes its place while this block is worked on
         mbar_expect_tx(g_full(t), 2 * kPanel);
         for (int p = 0; p < 2; ++p)
@@ -479,7 +482,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
       for (int c = 0; c < 4; ++c) {
 #pragma unroll
         for (int i = 0; i < 32; ++i) {
-          if (masked && (kv0 + c * 32 + i > q_pos || kv0 + c * 32 + i <= lo)) s[c][i] = 0xFF800000u;   // -inf
+          if (masked && (kv0 + c * 32 + i > q_pos || (REACH && kv0 + c * 32 + i <= lo))) s[c][i] = 0xFF800000u;   // -inf
           mx = fmaxf(mx, __uint_as_float(s[c][i]));
         }
       }
@@ -536,7 +539,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
       mbar_arrive(p_full(t));
     }
     if (ok && nb > 0 && mbar_wait(o_full(t), (uint32_t)((nb - 1) & 1), abort_flag, args.status, 211) &&
-        (!args.cgate || mbar_wait(g_full(t), 0, abort_flag, args.status, 212))) {
+        (!gated || mbar_wait(g_full(t), 0, abort_flag, args.status, 212))) {
       tc_fence_after();
       const int out_row = row + (POS ? t * kTile : 0);
       float num = args.v_scale != nullptr ? args.v_scale[hk] : 1.f;
@@ -549,16 +552,18 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
       if (POS && args.gate != nullptr && out_row < it.q_rows)
         num *= 1.f / (1.f + __expf(-to_float(reinterpret_cast<const T*>(args.gate)[(it.q_row0 + out_row) * args.ldg + head])));
       const float inv = l > 0.f ? num / l : 0.f;
-      T* dst = reinterpret_cast<T*>(args.out) + (long long)(it.q_row0 + out_row) * args.ldo + head * args.ho;
+      T* dst = reinterpret_cast<T*>(args.out) +
+               (REACH ? (long long)(it.q_row0 + out_row) * args.ldo + head * args.ho
+                      : ((long long)(it.q_row0 + row) * args.Hq + head) * kD);
 #pragma unroll
       for (int c = 0; c < 4; ++c) tmem_ld_32x32b_x32(o_addr + c * 32, s[c]);
       tmem_ld_wait();
       if (out_row < it.q_rows) {
 #pragma unroll
         for (int c = 0; c < 16; ++c) {
-          if (c >= args.v_chunks) break;
+          if (REACH && c >= args.v_chunks) break;
           uint32_t* o = &s[c >> 2][(c & 3) * 8];
-          if (args.cgate) {
+          if (gated) {
             float g[8];
             load8(reinterpret_cast<const T*>(smem + TcSmem::off_q + (t * 2 + (c >> 3)) * kPanel + row * 128 +
                                              (((c & 7) ^ (row & 7)) << 4)),
@@ -575,7 +580,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
           *reinterpret_cast<uint4*>(dst + 8 * c) = v;
         }
       }
-    } else if (args.cgate && row == 0) {       // gave up: let the gate's copies land before the CTA exits
+    } else if (gated && row == 0) {       // gave up: let the gate's copies land before the CTA exits
       const uint64_t t0 = globaltimer_ns();
       while (globaltimer_ns() - t0 < 200000ull) __nanosleep(1000);
     }
@@ -601,17 +606,17 @@ bool encode_map(CUtensorMap* map, const void* base, int rank, const cuuint64_t* 
   return true;
 }
 
-template <typename T, bool POS, bool FIXCAP = false>
+template <typename T, bool POS, int MODE>
 int launch_tc(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const CUtensorMap& mg, const TcArgs& a,
               cudaStream_t stream) {
   static bool configured = false;
   if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(attn_prefill_tc_kernel<T, POS, FIXCAP>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+    cudaError_t e = cudaFuncSetAttribute(attn_prefill_tc_kernel<T, POS, MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                          TcSmem::bytes);
     if (e != cudaSuccess) { msgl_set_error("prefill attention smem attribute", e); return MSGL_CUDA_ERROR; }
     configured = true;
   }
-  msgl_launch(attn_prefill_tc_kernel<T, POS, FIXCAP>, dim3(a.n_items * a.pairs), dim3(kTcThreads), TcSmem::bytes, stream, mq, mk, mv, mg, a);
+  msgl_launch(attn_prefill_tc_kernel<T, POS, MODE>, dim3(a.n_items * a.pairs), dim3(kTcThreads), TcSmem::bytes, stream, mq, mk, mv, mg, a);
   MSGL_CHECK_LAUNCH("attn_prefill_tc");
   return MSGL_OK;
 }
@@ -690,7 +695,7 @@ MSGL_API int msgl_attn_prefill_pos(const void* q, long long ldq, long long hq_st
   a.items = (const TcItem*)items; a.n_items = n_items; a.pairs = h; a.Hq = h; a.Hk = h; a.t_cap = t_pad;
   a.out = out; a.scale = scale; a.status = status; a.window = window; a.ldo = ldo; a.ho = ho; a.v_chunks = dv / 8;
   a.sink = (const float*)sink; a.gate = gate; a.ldg = ldg;
-  return launch_tc<__nv_bfloat16, true>(mq, mk, mv, mq, a, stream);
+  return launch_tc<__nv_bfloat16, true, TC_PLAIN>(mq, mk, mv, mq, a, stream);
 }
 
 // Causal prefill / extend attention for one layer. `kc` / `vt` are scratch buffers of
@@ -707,6 +712,11 @@ MSGL_API int msgl_attn_prefill_tc(const void* q, long long q_row_stride, void* o
                                   int window, int chunk, float softcap, const void* gate, long long ldg, int pos_form,
                                   int dtype, cudaStream_t stream) {
   if (n_items == 0 || total_q == 0) return MSGL_OK;
+  const bool ext = d != kD || window > 0 || chunk > 0 || softcap > 0.f || gate != nullptr;
+  if ((ext || pos_form) && (dtype != MSGL_BF16 || kv_fp8)) {
+    msgl_set_error_text("prefill attention: reaches, soft caps, gates, rows of 64 and unpaired query heads need bf16");
+    return MSGL_BAD_ARG;
+  }
   if (hq % hk || (!pos_form && (hq / hk) % 2) || (d != 64 && d != 128) || scale <= 0.f || (gate != nullptr && ldg % 8) ||
       (uintptr_t)gate % 16 || t_cap % 128 || t_pad % 128 || t_pad > t_cap || (q_row_stride % 8) ||
       (dtype != MSGL_BF16 && dtype != MSGL_F16)) {
@@ -745,12 +755,13 @@ MSGL_API int msgl_attn_prefill_tc(const void* q, long long q_row_stride, void* o
   int* status = nullptr;
   cudaGetSymbolAddress((void**)&status, g_attn_tc_status);
   const dim3 ggrid(t_pad / 64, hk);
-#define GATHER(T, F8)                                                                                              \
-  msgl_launch(kv_gather_kernel<T, F8>, dim3(ggrid), dim3(256), 0, stream, k_pool, v_pool, (T*)kc, (T*)vt, (const int*)blk_req,          \
+#define GATHER(T, F8, ROW)                                                                                              \
+  msgl_launch(kv_gather_kernel<T, F8, ROW>, dim3(ggrid), dim3(256), 0, stream, k_pool, v_pool, (T*)kc, (T*)vt, (const int*)blk_req,          \
                                                      (const int*)req_info, (const int*)block_table, bt_stride, hk, \
-                                                     page_size, t_cap, d)
-  if (dtype == MSGL_BF16) { if (kv_fp8) GATHER(__nv_bfloat16, true); else GATHER(__nv_bfloat16, false); }
-  else { if (kv_fp8) GATHER(__half, true); else GATHER(__half, false); }
+                                                     page_size, t_cap)
+  if (d == 64) GATHER(__nv_bfloat16, false, 64);
+  else if (dtype == MSGL_BF16) { if (kv_fp8) GATHER(__nv_bfloat16, true, 128); else GATHER(__nv_bfloat16, false, 128); }
+  else { if (kv_fp8) GATHER(__half, true, 128); else GATHER(__half, false, 128); }
 #undef GATHER
   MSGL_CHECK_LAUNCH("kv_gather");
   TcArgs a = {};
@@ -760,16 +771,13 @@ MSGL_API int msgl_attn_prefill_tc(const void* q, long long q_row_stride, void* o
   a.ldo = (long long)hq * d; a.ho = d; a.v_chunks = d / 8;
   const bool fixcap = softcap > 0.f && softcap * kLog2eTc <= kFixedCap && dtype == MSGL_BF16;
   if (pos_form) {
-    if (dtype != MSGL_BF16) {
-      msgl_set_error_text("prefill attention: bf16 where query heads do not come in pairs");
-      return MSGL_BAD_ARG;
-    }
-    return fixcap ? launch_tc<__nv_bfloat16, true, true>(mq, mk, mv, mg, a, stream)
-                  : launch_tc<__nv_bfloat16, true>(mq, mk, mv, mg, a, stream);
+    return fixcap ? launch_tc<__nv_bfloat16, true, TC_FIXED_CAP>(mq, mk, mv, mg, a, stream)
+                  : launch_tc<__nv_bfloat16, true, TC_EXTENDED>(mq, mk, mv, mg, a, stream);
   }
-  if (fixcap) return launch_tc<__nv_bfloat16, false, true>(mq, mk, mv, mg, a, stream);
-  if (dtype == MSGL_BF16) return launch_tc<__nv_bfloat16, false>(mq, mk, mv, mg, a, stream);
-  return launch_tc<__half, false>(mq, mk, mv, mg, a, stream);
+  if (fixcap) return launch_tc<__nv_bfloat16, false, TC_FIXED_CAP>(mq, mk, mv, mg, a, stream);
+  if (ext) return launch_tc<__nv_bfloat16, false, TC_EXTENDED>(mq, mk, mv, mg, a, stream);
+  if (dtype == MSGL_BF16) return launch_tc<__nv_bfloat16, false, TC_PLAIN>(mq, mk, mv, mg, a, stream);
+  return launch_tc<__half, false, TC_PLAIN>(mq, mk, mv, mg, a, stream);
 }
 
 MSGL_API int msgl_attn_tc_status(int reset) {
