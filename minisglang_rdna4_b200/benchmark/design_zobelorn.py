@@ -26,7 +26,7 @@ LLAMA = {"rope_type": "llama3", "factor": 8.0, "low_freq_factor": 1.0, "high_fre
 def _mixers(s: Dict):
     d = s["dim"]
     sizes = dict(heads=s["heads"], kv_heads=s["kv_heads"], dim=d, vdim=d, scale=d ** -0.5)
-    window = HeadLayer(**sizes, rotary=RotaryConfig(d, d, MAX_POS, 1e6, {"rope_type": "linear", "factor": 8.0}),
+    window = HeadLayer(**sizes, rotary=RotaryConfig(d, d, MAX_POS, 2e5, {"rope_type": "linear", "factor": 2.0}),
                        window=s["window"], softcap=30.0, joint_norm=True, gate=True)
     chunk = HeadLayer(**sizes, rotary=RotaryConfig(d, d, MAX_POS, 5e5, LLAMA, interleaved=True), chunk=MAX_POS,
                       unit_norm=True)
@@ -43,7 +43,7 @@ def zobelorn_config(s: Dict) -> ModelConfig:
     for i in range(s["layers"]):
         mixer = (chunk, window, chunk, replace(chunk, kv_from=i - 1))[i % 4]
         specs.append(LayerSpec(mixer, ff=s["ff"]) if i == 0 else LayerSpec(mixer, moe=moe))
-    return heads_config(specs, width=s["width"], vocab=s["vocab"], eps=1e-5, residual_multiplier=0.7, max_positions=MAX_POS)
+    return heads_config(specs, width=s["width"], vocab=s["vocab"], eps=1e-5, residual_multiplier=0.8, max_positions=MAX_POS)
 
 
 def laguna_config(s: Dict) -> ModelConfig:
@@ -106,7 +106,7 @@ def kernels(s: Dict) -> List[Dict]:
         # ---- Zobelorn: norms, heads, attention
         x, y, nw = rnd(t, w, dtype=f32), rnd(t, w, dtype=f32), torch.ones(w, device=dev)
         add("zobelorn", "norm of the output + add + norm (fp32 residual)", phase,
-            lambda: ops.add_norm(x, y, nw, 1e-5, False, bf, w, nw, 0.7), t * w * 14)
+            lambda: ops.add_norm(x, y, nw, 1e-5, False, bf, w, nw, 0.8), t * w * 14)
         pool = LayeredKVCache(b * per, ps, [(hk, d)], bf, dev)
         pool._planes[0].copy_(rnd(*pool._planes[0].shape))
         set_global_ctx(None)

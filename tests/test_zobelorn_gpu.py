@@ -195,7 +195,7 @@ def test_fp32_attention(hq, hk, d, kind, size):
 
 
 @pytest.mark.parametrize("form", ["general", "tc", "decode", "split", "fp32"])
-@pytest.mark.parametrize("kind,size", [("window", 64), ("window", 72), ("window", 128), ("window", 131), ("chunk", 64), ("chunk", 72),
+@pytest.mark.parametrize("kind,size", [("window", 64), ("window", 70), ("window", 128), ("window", 131), ("chunk", 64), ("chunk", 70),
                                        ("chunk", 128), ("chunk", 131)])
 @pytest.mark.parametrize("at", [0, 15, 16, 63, 64, 127, 128, 143, 144, 255])
 def test_a_loud_key_is_seen_exactly_within_reach(form, kind, size, at):
@@ -268,7 +268,7 @@ def test_rows_do_not_depend_on_how_a_prompt_was_cut():
 # ---------------------------------------------------------------------------------- the engine on the GPU
 # rows of 64, 128 and 256, groups of odd and even size, experts beyond one tile
 BIG = U.config([
-    U.chunk(6, 2, 64, 48, 100, mlp=U.dense(96)), U.window(5, 1, 80, 96, 72, rot=64, cap=9.0, scale=0.1, mlp=U.moe(16, 4, 48)),
+    U.chunk(6, 2, 64, 48, 100, mlp=U.dense(96)), U.window(5, 1, 80, 96, 76, rot=64, cap=9.0, scale=0.1, mlp=U.moe(16, 4, 48)),
     U.chunk(12, 2, 64, 48, 130, scale=0.9, kv_from=0, mlp=U.moe(5, 5, 33, shared=0)), U.window(2, 2, 128, 128, 128, cap=20.0, scale=0.09),
     U.chunk(3, 3, 136, 72, 60, rot=48, mlp=U.dense(130)),
 ], width=96, vocab=131)
