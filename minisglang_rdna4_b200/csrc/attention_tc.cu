@@ -1,4 +1,5 @@
-// Causal prefill / extend attention on the tcgen05 tensor cores (head_dim 128, even GQA group).
+// Causal prefill / extend attention on the tcgen05 tensor cores: head_dim 128 and an even GQA group, and extended forms
+// (rows of 64, any group, windows, chunks, capped scores, a gate on the output).
 //
 // The reference's prefill kernels (flash_prefill, flash_prefill_paged[_fp8];
 // python/minisgl/attention/hip.py:670-792, python/minisgl/attention/rdna4.py:419-503) walk the

@@ -283,6 +283,8 @@ class Engine:
         if mc.has_fp32_kernels and (self.kv_fp8 or self.kv_calibrating):
             raise ValueError(f"the K/V pool of {mc.model_type} has no fp8 form")
         self._head_geometry = mc.head_geometry(tp_) if mc.head_layers else None
+        if mc.head_layers and config.spec_algorithm != "none" and getattr(config, "spec_tree_width", 1) > 1:
+            raise ValueError(f"{mc.model_type} verifies draft chains (spec tree width 1): its attention takes no mask")
         if self.mla_latent:
             if self.kv_fp8 or self.kv_calibrating:
                 raise ValueError("the latent pool (MSGL_MLA_LATENT) is 16-bit only")

@@ -93,7 +93,7 @@ def weights(cfg, seed=0, sharp=2.0):
     return {k: t.to(torch.bfloat16) for k, t in out.items()}
 
 
-def clear_choices(cfg, path, seqs, margin=0.15):
+def clear_choices(cfg, path, seqs, margin=0.1):
     """The sequences with every token replaced whose choice of experts is a close call in some layer: in 16 bits it could fall
     the other way, and with it the rows that look back at the token."""
     from minisglang_rdna4_b200 import ops
@@ -113,7 +113,7 @@ def clear_choices(cfg, path, seqs, margin=0.15):
     try:
         for k, (name, seq) in enumerate(seqs.items()):
             g, seq = torch.Generator().manual_seed(77 + k), list(seq)
-            for _ in range(60):
+            for _ in range(300):
                 gaps.clear()
                 rep.step([(name, seq, [])], [name])
                 close = (torch.stack(gaps).amin(0) < margin).nonzero().flatten().tolist() if gaps else []
