@@ -91,13 +91,15 @@ class PagedAttentionBackend(BaseAttnBackend):
         )
 
     def forward_heads(self, q, layer: int, batch: Batch, *, scale: float, window: int = 0, chunk: int = 0,
-                      softcap: float = 0.0, gate=None):
+                      softcap: float = 0.0, gate=None, bias=None, sink=None, talk=None):
         """One layer of a model whose layers differ: ``q [T, H, width]`` against row ``layer`` of the pool, with the layer's
-        reach and soft cap; ``gate [T, H * width]``: logits of a sigmoid on the output channels."""
+        reach and soft cap; ``gate [T, H * width]``: logits of a sigmoid on the output channels. ``bias [H, reach]``: what a
+        score loses at each distance; ``sink [H]``: scores that only the softmax denominator counts; ``talk [H, H]``: head
+        h applies the sum over g of ``talk[h, g]`` times head g's weights to its own values."""
         md = batch.attn_metadata
         pool = get_global_ctx().kv_cache
         k_cache, v_cache = pool.k_cache(layer), pool.v_cache(layer)
-        extra = dict(window=window, chunk=chunk, softcap=softcap, gate=gate)
+        extra = dict(window=window, chunk=chunk, softcap=softcap, gate=gate, bias=bias, sink=sink, talk=talk)
         splits = 1
         if q.is_cuda:
             from ..ops import cuda as K
@@ -108,7 +110,8 @@ class PagedAttentionBackend(BaseAttnBackend):
                     return K.prefill_attention_tc(q, k_cache, v_cache, md.block_table, plan, scale, **extra)
             if md.decode and not self.single_split:
                 reach = min([r for r in (window, chunk, self.max_seq_len or md.max_kv) if r > 0])
-                splits = K.choose_splits(md.seq_lens.numel(), k_cache.shape[1], reach, True)
+                # mixed heads: a CTA has all of them
+                splits = K.choose_splits(md.seq_lens.numel(), 1 if talk is not None else k_cache.shape[1], reach, True)
         return ops.paged_attention(q, k_cache, v_cache, md.block_table, md.cu_q, md.seq_lens, scale, causal=True,
                                    max_q=md.max_q, max_kv=md.max_kv, decode=md.decode, workspace=md.workspace,
                                    splits=splits, **extra)

@@ -282,8 +282,8 @@ class Engine:
         self.mla_latent = bool(ENV.MLA_LATENT.value and mc.is_mla)
         if mc.has_fp32_kernels and (self.kv_fp8 or self.kv_calibrating):
             raise ValueError(f"the K/V pool of {mc.model_type} has no fp8 form")
-        self._head_geometry = mc.head_geometry(tp_) if mc.head_layers else None
-        if mc.head_layers and config.spec_algorithm != "none" and getattr(config, "spec_tree_width", 1) > 1:
+        self._head_geometry = (mc.head_geometry(tp_) or ((1, 64),)) if mc.layered else None
+        if mc.layered and config.spec_algorithm != "none" and getattr(config, "spec_tree_width", 1) > 1:
             raise ValueError(f"{mc.model_type} verifies draft chains (spec tree width 1): its attention takes no mask")
         if self.mla_latent:
             if self.kv_fp8 or self.kv_calibrating:
@@ -359,7 +359,8 @@ class Engine:
             conv_dim, st_heads, st_rows, st_cols = self._state_shape()
             self.gdn_state = GDNStateCache(mc.num_linear_layers, self.num_slots, conv_dim, mc.linear_conv_kernel_dim,
                                            st_heads, st_rows, st_cols, self._conv_state_dtype, self.device,
-                                           geometries=mc.state_geometries(config.tp_size))
+                                           geometries=mc.state_geometries(config.tp_size),
+                                           conv_geometries=mc.conv_geometries(config.tp_size))
             self.ledger.add("recurrent state", self.gdn_state.conv.numel() * self.gdn_state.conv.element_size()
                             + self.gdn_state.ssm.numel() * 4)
         self.ctx.gdn_state = self.gdn_state
@@ -369,7 +370,7 @@ class Engine:
             config.attention_backend, self.q_heads_local, self.kv_heads_local, mc.head_dim, self.device,
             max_batch=config.max_running_req, max_seq_len=self.max_seq_len,
             single_split=config.spec_algorithm != "none", latent=mc.latent_layers,
-            heads=[(div_even(m.heads, config.tp_size), m.row_pad) for m in mc.head_layers],
+            heads=[(m.heads if m.talk else div_even(m.heads, config.tp_size), m.row_pad) for m in mc.head_layers],
         )
         self.ctx.comm = comm_mod.get_comm()
         self._spec_exact = config.spec_algorithm != "none" and dev_kind == "cuda"
@@ -549,7 +550,7 @@ class Engine:
         if mc.input_conv_taps:                     # an input convolution runs on whole rows, on every rank
             return conv_dim, heads, rows, cols
         if mc.linear_layers:
-            return conv_dim, heads, rows, cols // tp
+            return sum(c * k for c, k in mc.conv_geometries(tp) or ()), heads, rows, cols // tp
         return conv_dim // tp, heads // tp, rows, cols
 
     def _free_memory(self) -> int:

@@ -1,4 +1,4 @@
-"""Per-request recurrent state of the linear-attention layers (gated delta net, Mamba-2, decaying states).
+"""Per-request recurrent state of the linear-attention layers (gated delta net, Mamba, Mamba-2, decaying states).
 
 Every linear-attention layer keeps, per request slot (the request's row of the page table), the
 last ``kernel - 1`` inputs of its causal convolution and one ``[Dk, Dv]`` fp32 state matrix per
@@ -17,7 +17,8 @@ import torch
 class GDNStateCache:
     def __init__(self, num_layers: int, num_slots: int, conv_dim: int, conv_kernel: int, num_v_heads: int,
                  head_k_dim: int, head_v_dim: int, dtype: torch.dtype, device,
-                 geometries: Optional[Sequence[Tuple[int, int, int]]] = None) -> None:
+                 geometries: Optional[Sequence[Tuple[int, int, int]]] = None,
+                 conv_geometries: Optional[Sequence[Tuple[int, int]]] = None) -> None:
         # no state matrix (num_v_heads 0): the state is the convolution tail alone. ``geometries``: (heads, rows, cols)
         # of every layer where they differ: a request's state matrices are then one run of floats, layer after layer
         self._geometries = tuple(geometries) if geometries is not None else None
@@ -30,7 +31,14 @@ class GDNStateCache:
             self.ssm = torch.zeros((num_layers, num_slots, num_v_heads, head_k_dim, head_v_dim), dtype=torch.float32,
                                    device=device)
         self.num_layers, self.num_slots = num_layers, num_slots
-        self.conv = torch.zeros((num_layers, num_slots, conv_dim, conv_kernel - 1), dtype=dtype, device=device)
+        # ``conv_geometries``: (channels, kept inputs) of every layer where they differ, one run of elements per request
+        self._conv_geometries = tuple(conv_geometries) if conv_geometries is not None else None
+        if self._conv_geometries is not None:
+            sizes = [c * k for c, k in self._conv_geometries]
+            self._conv_offsets = [sum(sizes[:i]) for i in range(len(sizes))]
+            self.conv = torch.zeros((1, num_slots, sum(sizes), 1), dtype=dtype, device=device)
+        else:
+            self.conv = torch.zeros((num_layers, num_slots, conv_dim, conv_kernel - 1), dtype=dtype, device=device)
         self._snapshots: Dict[object, Tuple[torch.Tensor, torch.Tensor]] = {}
         self._arena = None                      # pinned frames for snapshots kept on the host
         self.stream = None                      # the stream the snapshot / restore copies are issued on
@@ -55,6 +63,11 @@ class GDNStateCache:
         return num_layers * (conv_dim * (conv_kernel - 1) * itemsize + num_v_heads * dk * dv * 4)
 
     def conv_state(self, layer: int) -> torch.Tensor:
+        """``[slots, channels, kept inputs]`` of one layer (the slot stride may be longer than that)."""
+        if self._conv_geometries is not None:
+            c, k = self._conv_geometries[layer]
+            at = self._conv_offsets[layer]
+            return self.conv[0, :, at:at + c * k, 0].unflatten(1, (c, k))
         return self.conv[layer]
 
     def ssm_state(self, layer: int) -> torch.Tensor:

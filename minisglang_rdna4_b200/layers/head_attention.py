@@ -1,6 +1,7 @@
 """Grouped-query attention of a layer with a geometry of its own (``models.config.HeadLayer``): head counts, widths, rotation,
 reach (window or chunk), soft cap, norms of queries and keys, output gate; a layer may read the keys and values of an
-earlier one and then projects queries alone.
+earlier one and then projects queries alone. Further forms: scores with a logarithmic distance bias, a softmax that counts
+a zero score besides, and heads that apply a mixture of all heads' weights.
 
 One projection gives queries, keys, values and gates; every head takes ``row_pad`` columns of it, zeros past its
 channels, which change no dot product."""
@@ -21,11 +22,15 @@ from .rotary import get_rope_cache
 class HeadAttentionLayer(BaseOP):
     """``row``: index in the pool of the layer whose keys and values are read."""
 
-    def __init__(self, spec, row: int, width_pad: int, eps: float, dtype, device) -> None:
+    def __init__(self, spec, row: int, width_pad: int, eps: float, dtype, device, max_positions: int = 0) -> None:
+        """``max_positions``: the longest sequence, for distance biases without a window."""
+        self._max_distance = max_positions
         tp = get_tp_info().size
         self._spec, self._row, self._eps = spec, row, eps
-        self._h = div_even(spec.heads, tp)
-        self._hk = div_even(spec.kv_heads, tp, allow_replicate=True)
+        # heads whose weights are mixed are all on every rank; a rank hands on its share of them
+        self._h = spec.heads if spec.talk else div_even(spec.heads, tp)
+        self._hk = spec.kv_heads if spec.talk else div_even(spec.kv_heads, tp, allow_replicate=True)
+        self._mine = div_even(spec.heads, tp)
         self._own, self._d = spec.kv_from is None, spec.row_pad
         if torch.device(device).type == "cuda" and dtype != torch.float32 and self._d > 256:
             raise NotImplementedError(f"heads of {max(spec.dim, spec.vdim)} channels: the 16-bit attention kernels take 256")
@@ -37,10 +42,16 @@ class HeadAttentionLayer(BaseOP):
             if self._own:
                 self.k_norm = torch.empty((self._hk * self._d,), dtype=torch.float32, device=device)
         self._cos_sin = get_rope_cache(spec.rotary, device) if spec.rotary is not None else None
+        self._extra = {}
+        if spec.log_bias:
+            self.r1 = torch.empty((self._h,), dtype=torch.float32, device=device)
+            self.r2 = torch.empty((self._h,), dtype=torch.float32, device=device)
+        if spec.talk:
+            self.talk = torch.empty((self._h, self._h), dtype=torch.float32, device=device)
 
     @property
     def out_width(self) -> int:
-        return self._h * self._d
+        return self._mine * self._d
 
     def forward(self, x: torch.Tensor) -> torch.Tensor:
         """``x [T, width]`` -> the heads' values, gated, ``[T, heads * row_pad]``."""
@@ -55,7 +66,10 @@ class HeadAttentionLayer(BaseOP):
             self.q_norm if spec.joint_norm else None, self.k_norm if spec.joint_norm and self._own else None,
             self._totals(y), spec.unit_norm, store)
         out = ctx.attn_backend.forward_heads(q, self._row, batch, scale=spec.scale, window=spec.window, chunk=spec.chunk,
-                                             softcap=spec.softcap, gate=y[:, self._gate_at:] if spec.gate else None)
+                                             softcap=spec.softcap, gate=y[:, self._gate_at:] if spec.gate else None,
+                                             **self._extra)
+        if self._mine < self._h:
+            out = out[:, get_tp_info().rank * self._mine:][:, :self._mine]
         return out.reshape(out.shape[0], self.out_width)
 
     def _totals(self, y: torch.Tensor):
@@ -75,8 +89,21 @@ class HeadAttentionLayer(BaseOP):
         own = self._hk if self._own else 0
         for at, n, used in ((0, self._h, spec.dim), (self._h, own, spec.dim), (self._h + own, own, spec.vdim)):
             weight[at * d:(at + n) * d].view(n, d, weight.shape[1])[:, used:] = 0
+        if spec.log_bias:       # one number per head and distance in reach
+            far = torch.arange(spec.window or self._max_distance, dtype=torch.float64, device=weight.device)
+            bias = self.r1.double()[:, None] * torch.log1p(self.r2.double()[:, None] * far)
+            self._extra["bias"] = bias.float().contiguous()
+        if spec.zero_sink:
+            self._extra["sink"] = torch.zeros(self._h, dtype=torch.float32, device=weight.device)
+        if spec.talk:
+            self._extra["talk"] = self.talk
 
     def init_dummy(self, gen: torch.Generator, std: float = 0.02) -> None:
         for name in ("q_norm", "k_norm"):
             if hasattr(self, name):
                 setattr(self, name, torch.ones_like(getattr(self, name)))
+        if self._spec.log_bias:
+            self.r1, self.r2 = torch.ones_like(self.r1), torch.full_like(self.r2, 0.5)
+        if self._spec.talk:
+            mix = torch.randn(self.talk.shape, generator=gen, device=gen.device) * 0.1
+            self.talk = mix.to(self.talk.device) + torch.eye(self._h, device=self.talk.device)

@@ -1,7 +1,7 @@
 """Linear attention with a decaying state per head (no delta rule, no convolution): one projection to
 ``[q ‖ k ‖ v ‖ output gate (‖ low-rank decay input)]``, the recurrence on the request's state slot, a norm of the
 result (per head or over all heads) with the gate. ``models.config.LinearAttnLayer`` says which decay, activation,
-norm and gate a layer has."""
+rotation, norm and gate a layer has."""
 from __future__ import annotations
 
 import torch
@@ -13,6 +13,7 @@ from ..parallel.info import get_tp_info
 from ..utils import div_even
 from .base import BaseOP
 from .linear import ReplicatedLinear
+from .rotary import get_rope_cache
 
 
 def _pad16(n: int) -> int:
@@ -38,6 +39,8 @@ class LinearAttentionLayer(BaseOP):
             tp = get_tp_info()
             mine = spec.decay[tp.rank * self._h:(tp.rank + 1) * self._h]
             self._decay = torch.tensor(mine, dtype=torch.float32, device=device)
+        # neighbouring channels are pairs (checkpoints with half-split pairs are loaded in that order)
+        self._cos_sin = get_rope_cache(spec.rotary, device) if spec.rotary is not None else None
 
     @property
     def out_width(self) -> int:
@@ -48,12 +51,12 @@ class LinearAttentionLayer(BaseOP):
         batch = ctx.batch
         proj = self.in_proj.forward(x)
         if ctx.recurrent_journal is not None:
-            ctx.recurrent_journal.append((self, proj))
+            ctx.recurrent_journal.append((self, proj, batch.positions))
         md = batch.attn_metadata
         chunked = batch.is_prefill and not batch.spec_verify and md.max_q >= 8
-        return self._mix(proj, md.cu_q, batch.gdn_slots, batch.gdn_has_state, chunked)
+        return self._mix(proj, md.cu_q, batch.gdn_slots, batch.gdn_has_state, batch.positions, chunked)
 
-    def _mix(self, proj: torch.Tensor, cu_q, slots, has_state, chunked: bool) -> torch.Tensor:
+    def _mix(self, proj: torch.Tensor, cu_q, slots, has_state, positions, chunked: bool) -> torch.Tensor:
         """The recurrence over the projected rows (advances the state), norm and gate."""
         spec, kd, vd = self._spec, self._kd, self._vd
         q, k = (proj[:, i * kd:(i + 1) * kd].unflatten(1, (self._h, self._dk)) for i in range(2))
@@ -65,16 +68,21 @@ class LinearAttentionLayer(BaseOP):
             gate = (low, self.decay_up, self.decay_bias)
         state = get_global_ctx().gdn_state.ssm_state(self._state_row)
         o = ops.linear_attention(q, k, v, state, cu_q, slots, has_state, decay=self._decay, gate=gate, tau=spec.tau,
-                                 q_scale=spec.q_scale, act=spec.act, chunked=chunked)
+                                 q_scale=spec.q_scale, act=spec.act, chunked=chunked,
+                                 rope=None if self._cos_sin is None else (self._cos_sin, positions))
         total = None
         if spec.joint_norm and get_tp_info().size > 1:      # the other ranks hold the other heads
             total = get_comm().all_reduce(o.float().pow(2).sum((1, 2)))
         return ops.norm_gate(o, g, self.norm, self._eps, spec.vdim, spec.joint_norm, spec.gate_act, self.out_width,
                              total, spec.heads)
 
-    def replay(self, proj: torch.Tensor, cu_q, slots, has_state) -> None:
+    def replay(self, proj: torch.Tensor, cu_q, slots, has_state, positions) -> None:
         """Re-advance the (restored) states over the kept rows of a verify step."""
-        self._mix(proj, cu_q, slots, has_state, False)
+        self._mix(proj, cu_q, slots, has_state, positions, False)
+
+    def _post_load_self(self) -> None:
+        if not self._spec.weighted:
+            self.norm = torch.ones_like(self.norm)
 
     def init_dummy(self, gen: torch.Generator, std: float = 0.02) -> None:
         self.norm = torch.ones_like(self.norm)

@@ -260,6 +260,8 @@ class ResidualExperts(BaseOP):
         self.router = torch.empty((pad(spec.experts + int(self._gated), 8), width_pad), dtype=dtype, device=device)
         self.w13 = torch.empty((spec.experts, 2 * self._ff, width_pad), dtype=dtype, device=device)
         self.w2 = torch.empty((spec.experts, self._out, self._ff), dtype=dtype, device=device)
+        if spec.correction:        # of the scores that choose, not of the weights
+            self.correction = torch.empty((spec.experts,), dtype=torch.float32, device=device)
         if self._shared_ff:
             self.shared_up = ReplicatedLinear(width_pad, 2 * self._shared_ff, dtype, device)
             self.shared_down = ReplicatedLinear(self._shared_ff, width_pad, dtype, device)
@@ -274,24 +276,27 @@ class ResidualExperts(BaseOP):
                                               else ops.clamped_glu(up, s.shared_limit, s.alpha))
             gate = logits[:, s.experts] if self._gated else None
         counts = None
+        bias = self.correction if s.correction else None
         if x.is_cuda:
             from ..ops import moe_kernels
 
             counts = torch.empty(s.experts, dtype=torch.int32, device=x.device)
-            topk_w, topk_ids = moe_kernels.moe_route(logits[:, :s.experts], s.top, False, s.scoring, s.scale, counts,
-                                                     groups=s.groups, keep=s.keep)
+            topk_w, topk_ids = moe_kernels.moe_route(logits[:, :s.experts], s.top, s.renorm, s.scoring, s.scale, counts,
+                                                     bias=bias, groups=s.groups, keep=s.keep)
         elif s.groups > 1:
             from ..ops import ref
 
-            topk_w, topk_ids = ref.moe_route_grouped(logits[:, :s.experts], s.top, False, s.scoring, None, s.scale, s.groups,
-                                                     s.keep)
+            topk_w, topk_ids = ref.moe_route_grouped(logits[:, :s.experts], s.top, s.renorm, s.scoring, bias, s.scale,
+                                                     s.groups, s.keep)
         else:
-            topk_w, topk_ids = ops.moe_route(logits[:, :s.experts], s.top, False, s.scoring, None, s.scale)
+            topk_w, topk_ids = ops.moe_route(logits[:, :s.experts], s.top, s.renorm, s.scoring, bias, s.scale)
         y = ops.experts_partial32(x, self.w13, self.w2, topk_w, topk_ids, s.limit, s.alpha, shared, gate, counts, s.act,
                                   s.on_input)
         return get_comm().all_reduce(y) if get_tp_info().size > 1 else y
 
     def init_dummy(self, gen: torch.Generator, std: float = 0.02) -> None:
+        if self._spec.correction:
+            self.correction = torch.zeros_like(self.correction)
         for name in ("router", "w13", "w2"):
             t = getattr(self, name)
             w = torch.randn(t.shape, generator=gen, device=gen.device, dtype=torch.float32) * std

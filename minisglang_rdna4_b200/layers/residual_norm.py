@@ -1,4 +1,6 @@
-"""Norm of a layer with an fp32 residual stream: residual add and layer norm (no bias) or RMS norm in one pass."""
+"""Norms of a layer with an fp32 residual stream, in one pass with the residual add: layer norm (no bias) or RMS norm
+(``ResidualNorm``); layer norms with a bias on both sides of a sublayer, pairs of sublayers, depth averages
+(``BiasedNorm``, ``LayerHistory``; ``ops.residual_step`` does them together)."""
 from __future__ import annotations
 
 from typing import Optional
@@ -25,3 +27,21 @@ class ResidualNorm(BaseOP):
 
     def init_dummy(self, gen: torch.Generator, std: float = 0.02) -> None:
         self.weight = torch.ones_like(self.weight)
+
+class BiasedNorm(BaseOP):
+    """Weight and bias of a layer norm; ``residual_step`` applies it."""
+
+    def __init__(self, width: int, device) -> None:
+        self.weight = torch.empty((width,), dtype=torch.float32, device=device)
+        self.bias = torch.empty((width,), dtype=torch.float32, device=device)
+
+    def init_dummy(self, gen: torch.Generator, std: float = 0.02) -> None:
+        self.weight, self.bias = torch.ones_like(self.weight), torch.zeros_like(self.bias)
+
+
+class LayerHistory:
+    """The results of the layers so far in a step, ``[layers + 1, rows, width]`` fp32; row 0 is the embedding output."""
+
+    def __init__(self, layers: int, rows: int, width: int, device) -> None:
+        self.rows = torch.empty((layers + 1, rows, width), dtype=torch.float32, device=device)
+        self.count = 0

@@ -79,6 +79,11 @@ def _register_defaults() -> None:
     if "ZobelornForCausalLM" not in MODEL_REGISTRY:
         MODEL_REGISTRY.register("ZobelornForCausalLM")(ZobelornForCausalLM)
 
+    from .ligipel import LigipelForCausalLM
+
+    if "LigipelForCausalLM" not in MODEL_REGISTRY:
+        MODEL_REGISTRY.register("LigipelForCausalLM")(LigipelForCausalLM)
+
 
 def create_model(cfg: ModelConfig, dtype: torch.dtype, device):
     """Instantiate the model for ``cfg`` with uninitialised (or meta) parameters."""

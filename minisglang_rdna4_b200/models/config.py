@@ -81,8 +81,9 @@ class LinearAttnLayer:
     """One linear-attention layer without a delta rule: per head a ``[dim, vdim]`` state that decays and takes up
     ``k v^T`` of every token. The decay is one number per head (``decay``) or comes from the input, one per key channel:
     ``sigmoid(z) ** (1 / tau)`` with ``z`` a projection of rank ``gate_rank`` plus a bias (``decay`` None). ``act``: silu on
-    the projected q, k and v. The output is RMS-normed over all heads together (``joint_norm``) or per head with one
-    shared weight, and gated by ``gate_act`` of a projection."""
+    the projected q, k and v. ``rotary``: rotary positions on q and k. The output is RMS-normed over all heads together
+    (``joint_norm``) or per head with one shared weight (none with ``weighted`` False), and gated by ``gate_act`` of a
+    projection."""
 
     heads: int
     dim: int
@@ -94,6 +95,8 @@ class LinearAttnLayer:
     q_scale: float = 1.0
     joint_norm: bool = False
     gate_act: str = "silu"
+    rotary: Optional[RotaryConfig] = None
+    weighted: bool = True
 
     @property
     def dim_pad(self) -> int:
@@ -112,7 +115,9 @@ class HeadLayer:
     ``softcap`` c > 0: scores go through ``c tanh(s / c)``. ``joint_norm``: weighted RMS norms over all query heads and
     over all key heads together, ahead of the rotation. ``unit_norm``: every query and key head divided by its root mean
     square after the rotation. ``gate``: a sigmoid gate per output channel. ``kv_from``: the layer whose keys and
-    values are read instead of own ones."""
+    values are read instead of own ones. ``log_bias``: a score loses ``r1 ln(1 + r2 distance)``, with two numbers per
+    head. ``zero_sink``: the softmax denominator counts a score of 0 that belongs to no key. ``talk``: every head applies a
+    mixture of all heads' weights to its values."""
 
     heads: int
     kv_heads: int
@@ -127,6 +132,9 @@ class HeadLayer:
     unit_norm: bool = False
     gate: bool = False
     kv_from: Optional[int] = None
+    log_bias: bool = False
+    zero_sink: bool = False
+    talk: bool = False
 
     @property
     def row_pad(self) -> int:
@@ -136,11 +144,44 @@ class HeadLayer:
 
 
 @dataclass(frozen=True)
+class ScanLayer:
+    """A selective state-space mixer (Mamba): ``inner`` channels behind a causal convolution of ``taps``, each with a
+    ``state`` vector; step sizes come from a projection of rank ``dt_rank``."""
+
+    inner: int
+    state: int
+    dt_rank: int
+    taps: int
+
+    @property
+    def state_pad(self) -> int:
+        return _round_up(self.state, 4)
+
+    @property
+    def rank_pad(self) -> int:
+        return _round_up(self.dt_rank, 16)
+
+    def inner_pad(self, tp: int = 1) -> int:
+        """Channels of a rank, in the kernels."""
+        return _round_up(self.inner // tp, 16)
+
+
+@dataclass(frozen=True)
+class PairMixer:
+    """Two mixers that read the same rows; half the sum of their outputs, each RMS-normed over the width."""
+
+    left: HeadLayer
+    right: ScanLayer
+
+
+@dataclass(frozen=True)
 class ExpertSpec:
     """A mixture of ``experts`` feed-forwards of width ``ff`` of which each token uses ``top``, chosen by ``scoring`` among
     the best ``keep`` of ``groups`` groups; ``shared_ff`` > 0: a further one for every token, behind a sigmoid gate with
     ``shared_gated``. Activation: silu-gated, or with ``act`` "clamped" gate and up halves clamped at ``limit``,
-    ``g * sigmoid(alpha g) * (u + 1)``. ``on_input``: a chosen expert's weight multiplies what goes into it."""
+    ``g * sigmoid(alpha g) * (u + 1)``. ``on_input``: a chosen expert's weight multiplies what goes into it.
+    ``correction``: a number per expert that counts in the choice and not in the weights. ``renorm``: the chosen experts'
+    scores are divided by their sum."""
 
     experts: int
     top: int
@@ -156,6 +197,8 @@ class ExpertSpec:
     scoring: str = "softmax"
     on_input: bool = False
     shared_gated: bool = True
+    correction: bool = False
+    renorm: bool = False
 
 
 @dataclass(frozen=True)
@@ -163,7 +206,7 @@ class LayerSpec:
     """A sequential layer of a model whose layers are listed one by one: a mixer, and a feed-forward that is dense and
     gated (``ff`` > 0), a mixture of experts (``moe``) or absent."""
 
-    mixer: Any                              # LatentLayer | LinearAttnLayer | HeadLayer
+    mixer: Any                              # LatentLayer | LinearAttnLayer | HeadLayer | PairMixer
     ff: int = 0
     moe: Optional[ExpertSpec] = None
 
@@ -233,6 +276,7 @@ class ModelConfig:
     layer_specs: Optional[Tuple[LayerSpec, ...]] = None
     embedding_multiplier: float = 1.0
     residual_multiplier: float = 1.0        # of a sublayer's output where it joins the residual stream
+    depth_average: bool = False             # a layer's input is a weighted sum of the results of all layers before
     # misc
     sliding_window: Optional[int] = None
     layer_types: Optional[Tuple[str, ...]] = None
@@ -295,26 +339,39 @@ class ModelConfig:
         owner = layer if specs[layer].kv_from is None else specs[layer].kv_from
         return sum(1 for s in specs[:owner] if s is not None and s.kv_from is None)
 
+    def head_mixer(self, layer: int) -> Optional[HeadLayer]:
+        """The attention of a layer whose mixer is or contains one with keys and values per head."""
+        m = self.layer_specs[layer].mixer
+        m = m.left if isinstance(m, PairMixer) else m
+        return m if isinstance(m, HeadLayer) else None
+
     @property
     def head_layers(self) -> Tuple[HeadLayer, ...]:
-        """The layers of a model whose attention layers each have a geometry of their own."""
-        mixers = tuple(s.mixer for s in self.layer_specs or ())
-        return mixers if mixers and all(isinstance(m, HeadLayer) for m in mixers) else ()
+        """The attention layers, in layer order, of a model whose layers each have a geometry of their own."""
+        mixers = (self.head_mixer(i) for i in range(len(self.layer_specs or ())))
+        return tuple(m for m in mixers if m is not None)
 
     def head_geometry(self, tp: int = 1) -> Tuple[Tuple[int, int], ...]:
-        """``(kv heads of a rank, row width)`` of every layer with keys and values of its own, in layer order."""
-        return tuple((max(m.kv_heads // tp, 1), m.row_pad) for m in self.head_layers if m.kv_from is None)
+        """``(kv heads of a rank, row width)`` of every layer with keys and values of its own, in layer order. Heads whose
+        weights are mixed are on every rank."""
+        return tuple((m.kv_heads if m.talk else max(m.kv_heads // tp, 1), m.row_pad)
+                     for m in self.head_layers if m.kv_from is None)
 
     def head_row(self, layer: int) -> int:
         """Index in the pool of the layer whose keys and values ``layer`` reads."""
-        mixers = self.head_layers
-        owner = layer if mixers[layer].kv_from is None else mixers[layer].kv_from
-        return sum(1 for m in mixers[:owner] if m.kv_from is None)
+        donor = self.head_mixer(layer).kv_from
+        before = (self.head_mixer(i) for i in range(layer if donor is None else donor))
+        return sum(1 for m in before if m is not None and m.kv_from is None)
+
+    @property
+    def layered(self) -> bool:
+        """Described layer by layer, without attention latents: keys and values per head, a geometry per layer."""
+        return bool(self.layer_specs) and not self.latent_layers
 
     @property
     def has_fp32_kernels(self) -> bool:
         """Every kernel the model runs on a GPU has an fp32 form."""
-        return bool(self.latent_layers or self.head_layers)
+        return bool(self.latent_layers or self.layered)
 
     @property
     def is_recurrent(self) -> bool:
@@ -323,19 +380,28 @@ class ModelConfig:
                 or bool(self.layer_types) and any(t in ("linear_attention", "mamba") for t in self.layer_types))
 
     @property
-    def linear_layers(self) -> Tuple[Tuple[int, LinearAttnLayer], ...]:
-        """``(layer, spec)`` of the linear-attention layers of a model with ``layer_specs``."""
-        return tuple((i, s.mixer) for i, s in enumerate(self.layer_specs or ()) if isinstance(s.mixer, LinearAttnLayer))
+    def linear_layers(self) -> Tuple[Tuple[int, Any], ...]:
+        """``(layer, LinearAttnLayer | ScanLayer)`` of the layers with a recurrent state of a model with ``layer_specs``."""
+        mixers = ((i, s.mixer.right if isinstance(s.mixer, PairMixer) else s.mixer)
+                  for i, s in enumerate(self.layer_specs or ()))
+        return tuple((i, m) for i, m in mixers if isinstance(m, (LinearAttnLayer, ScanLayer)))
 
     def state_row(self, layer: int) -> int:
-        """Index of a linear-attention layer in the state cache."""
+        """Index of a layer with a recurrent state in the state cache."""
         return sum(1 for i, _ in self.linear_layers if i < layer)
 
     def state_geometries(self, tp: int = 1) -> Optional[Tuple[Tuple[int, int, int], ...]]:
         """``(heads, rows, cols)`` of every state layer where layers may differ; ``None``: ``recurrent_geometry``."""
         if not self.linear_layers:
             return None
-        return tuple((m.heads // tp, m.dim_pad, m.vdim_pad) for _, m in self.linear_layers)
+        return tuple((1, m.inner_pad(tp), m.state_pad) if isinstance(m, ScanLayer)
+                     else (m.heads // tp, m.dim_pad, m.vdim_pad) for _, m in self.linear_layers)
+
+    def conv_geometries(self, tp: int = 1) -> Optional[Tuple[Tuple[int, int], ...]]:
+        """``(channels, taps - 1)`` of the convolution tail of every state layer where layers may differ."""
+        if not any(isinstance(m, ScanLayer) for _, m in self.linear_layers):
+            return None
+        return tuple((m.inner_pad(tp), m.taps - 1) if isinstance(m, ScanLayer) else (0, 0) for _, m in self.linear_layers)
 
     @property
     def num_linear_layers(self) -> int:
@@ -351,7 +417,7 @@ class ModelConfig:
         """Layers that keep K/V pages."""
         if self.latent_layers:
             return len(self.latent_widths)
-        if self.head_layers:
+        if self.layered:
             return len(self.head_geometry())
         if self.model_type == "nemotron_h":
             return sum(1 for t in (self.layer_types or ()) if t == "attention")
@@ -395,8 +461,9 @@ class ModelConfig:
         over ``conv channels`` inputs and a ``[heads, rows, cols]`` fp32 state matrix per request (``heads`` 0: the window alone)."""
         if self.input_conv_taps:
             return self.hidden_size, 0, 0, 0
-        if self.linear_layers:                 # no convolution; the state matrices of all layers as one row
-            return 0, 1, 1, sum(m.heads * m.dim_pad * m.vdim_pad for _, m in self.linear_layers)
+        if self.linear_layers:                 # the convolution tails and state matrices of all layers as one row each
+            return (sum(c * k for c, k in self.conv_geometries() or ()), 1, 1,
+                    sum(h * r * c for h, r, c in self.state_geometries()))
         if self.mamba_num_heads:
             inter = self.mamba_num_heads * self.mamba_head_dim
             return (inter + 2 * self.mamba_n_groups * self.ssm_state_size, self.mamba_num_heads, self.mamba_head_dim,
@@ -456,6 +523,8 @@ class ModelConfig:
             return _rafodra_config(cfg, folder)
         if cfg.get("architecture") == "Zobelorn":
             return _zobelorn_config(cfg)
+        if cfg.get("architecture") == "Ligipel":
+            return _ligipel_config(cfg)
         vision = None
         if "text_config" in cfg and isinstance(cfg["text_config"], dict):
             if str(cfg.get("model_type", "")).startswith("gemma3") and cfg.get("vision_config"):
@@ -893,6 +962,86 @@ def heads_config(specs, width: int, vocab: int, eps: float, embedding_multiplier
         architectures=("ZobelornForCausalLM",), layer_specs=tuple(specs), embedding_multiplier=embedding_multiplier,
         residual_multiplier=residual_multiplier, max_position_embeddings=max_positions, eos_token_ids=eos_token_ids,
         bos_token_id=bos_token_id)
+
+
+def _pair_mixer(i: int, mix: Dict[str, Any]) -> PairMixer:
+    left, right = mix["left"], mix["right"]
+    attn = HeadLayer(heads=int(left["heads"]), kv_heads=int(left["kv_heads"]), dim=int(left["dim"]), vdim=int(left["vdim"]),
+                     scale=float(left["scale"]), window=int((left.get("mask") or {}).get("size") or 0), log_bias=True,
+                     zero_sink=True, talk=True)
+    if attn.heads % attn.kv_heads:
+        raise ValueError(f"layer {i}: {attn.heads} query heads over {attn.kv_heads} key / value heads")
+    return PairMixer(attn, ScanLayer(inner=int(right["inner"]), state=int(right["state"]), dt_rank=int(right["dt_rank"]),
+                                     taps=int(right["conv"])))
+
+
+def _retention_mixer(i: int, mix: Dict[str, Any], max_pos: int) -> LinearAttnLayer:
+    heads, dim, rot = int(mix["heads"]), int(mix["dim"]), mix.get("rot") or {}
+    decay, dims = tuple(float(d) for d in mix["decay"]), int(rot.get("dims", 0))
+    if len(decay) != heads:
+        raise ValueError(f"layer {i}: {len(decay)} decays for {heads} heads")
+    if dims % 2 or not 0 <= dims <= dim:
+        raise ValueError(f"layer {i}: {dims} rotated of {dim} channels")
+    # the checkpoint's half-split pairs become neighbours when the weights are loaded
+    rotary = RotaryConfig(dim, dims, max_pos, float(rot["base"]), interleaved=True) if dims else None
+    return LinearAttnLayer(heads=heads, dim=dim, vdim=int(mix["vdim"]), decay=decay, q_scale=dim ** -0.5, rotary=rotary,
+                           weighted=False)
+
+
+def _ligipel_config(cfg: Dict[str, Any]) -> ModelConfig:
+    """``layers`` lists every layer's mixer ("parallel": attention beside a selective scan; "retention") and feed-forward
+    with sizes of their own."""
+    max_pos = int(cfg.get("max_positions") or 131072)      # the design sets no limit: one for tables and buffers
+    specs: List[LayerSpec] = []
+    for i, layer in enumerate(cfg["layers"]):
+        kind, mix, mlp = layer["type"], layer["mixer"], layer.get("mlp")
+        if kind not in ("parallel", "retention"):
+            raise ValueError(f"layer {i}: unknown mixer type {kind!r}")
+        mixer = _pair_mixer(i, mix) if kind == "parallel" else _retention_mixer(i, mix, max_pos)
+        moe = None
+        if mlp is not None:
+            if mlp["kind"] != "moe":
+                raise ValueError(f"layer {i}: unknown feed-forward kind {mlp['kind']!r}")
+            router, shared = mlp["router"], mlp.get("shared")
+            moe = ExpertSpec(experts=int(router["experts"]), top=int(router["top"]), ff=int(mlp["expert"]["ff"]),
+                             shared_ff=int(shared["ff"]) if shared else 0, act="silu", shared_gated=False, correction=True,
+                             renorm=True)
+            if not 0 < moe.top <= moe.experts:
+                raise ValueError(f"layer {i}: {moe.top} of {moe.experts} experts")
+        specs.append(LayerSpec(mixer, 0, moe))
+    eos = cfg.get("eos_token_id")
+    eos_ids = tuple(eos) if isinstance(eos, (list, tuple)) else (() if eos is None else (int(eos),))
+    return pair_config(specs, width=int(cfg["width"]), vocab=int(cfg["vocab"]), eps=float(cfg["norm"]["eps"]),
+                       logit_scale=float(cfg["logit_scale"]), logit_softcap=float(cfg["logit_softcap"]), max_positions=max_pos,
+                       eos_token_ids=eos_ids, bos_token_id=cfg.get("bos_token_id"))
+
+
+def pair_config(specs, width: int, vocab: int, eps: float, logit_scale: float = 1.0, logit_softcap: float = 0.0,
+                max_positions: int = 131072, eos_token_ids: Tuple[int, ...] = (), bos_token_id=None) -> ModelConfig:
+    """A Ligipel configuration from its layers."""
+    attn = next((s.mixer.left for s in specs if isinstance(s.mixer, PairMixer)), None)
+    row = attn.row_pad if attn is not None else 64
+
+    def widest(s: LayerSpec) -> int:        # activations of one token
+        m = s.mixer
+        if isinstance(m, PairMixer):
+            left, right = m.left, m.right
+            mix = ((left.heads + 2 * left.kv_heads) * left.row_pad + left.heads * left.kv_heads * left.row_pad
+                   + 6 * right.inner_pad())
+        else:
+            mix = m.heads * (2 * m.dim + 3 * m.vdim)
+        return max(mix, s.moe.top * s.moe.ff + s.moe.shared_ff if s.moe else 0)
+
+    # the results of all layers are kept through a step, in fp32
+    kept = 2 * (len(specs) + 1) * width
+    return ModelConfig(
+        num_layers=len(specs), num_qo_heads=attn.heads if attn is not None else 1,
+        num_kv_heads=attn.kv_heads if attn is not None else 1, head_dim=row, hidden_size=width, vocab_size=vocab,
+        intermediate_size=max(widest(s) for s in specs) + kept // 2, rms_norm_eps=eps,
+        rotary_config=RotaryConfig(row, 0, max_positions, base=10000.0), model_type="ligipel",
+        architectures=("LigipelForCausalLM",), layer_specs=tuple(specs), linear_conv_kernel_dim=2, depth_average=True,
+        output_multiplier=logit_scale, final_logit_softcapping=logit_softcap or None, max_position_embeddings=max_positions,
+        eos_token_ids=eos_token_ids, bos_token_id=bos_token_id)
 
 
 def _default_arch(model_type: str) -> List[str]:

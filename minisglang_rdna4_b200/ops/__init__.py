@@ -135,15 +135,15 @@ def store_kv(k, v, k_cache, v_cache, out_loc, k_scale=None, v_scale=None):
 def paged_attention(q, k_cache, v_cache, block_table, cu_q, seq_lens, scale: float, *, causal: bool = True,
                     window: int = 0, mask=None, k_scale=None, v_scale=None, max_q: int = 0,
                     max_kv: int = 0, decode: bool = False, workspace=None, splits=None, mask_window: int = 0,
-                    chunk: int = 0, softcap: float = 0.0, gate=None):
+                    chunk: int = 0, softcap: float = 0.0, gate=None, bias=None, sink=None, talk=None):
     if q.is_cuda:
         return _cuda().paged_attention(q, k_cache, v_cache, block_table, cu_q, seq_lens, scale,
                                        causal=causal, window=window, mask=mask, k_scale=k_scale,
                                        v_scale=v_scale, max_q=max_q, max_kv=max_kv, decode=decode,
                                        workspace=workspace, splits=splits, mask_window=mask_window, chunk=chunk,
-                                       softcap=softcap, gate=gate)
+                                       softcap=softcap, gate=gate, bias=bias, sink=sink, talk=talk)
     return ref.paged_attention(q, k_cache, v_cache, block_table, cu_q, seq_lens, scale, causal, window,
-                               mask, k_scale, v_scale, mask_window, chunk, softcap, gate)
+                               mask, k_scale, v_scale, mask_window, chunk, softcap, gate, bias, sink, talk)
 
 
 # ---------------------------------------------------------------------------- GEMMs
@@ -287,11 +287,13 @@ def add_norm(x, delta, weight, eps: float, center: bool, out_dtype, out_cols: in
 
 
 def linear_attention(q, k, v, state, cu_q, slots, has_state, decay=None, gate=None, tau: float = 1.0,
-                     q_scale: float = 1.0, act: bool = False, chunked: bool = False):
-    """``chunked``: the step may take the tensor-core form (prompts); otherwise every row takes the recurrent one."""
+                     q_scale: float = 1.0, act: bool = False, chunked: bool = False, rope=None):
+    """``chunked``: the step may take the tensor-core form (prompts); otherwise every row takes the recurrent one.
+    ``rope = (cos_sin, positions)``: q and k are rotated first, neighbouring channels as pairs, in fp32."""
     if q.is_cuda:
-        return _cuda().linear_attention(q, k, v, state, cu_q, slots, has_state, decay, gate, tau, q_scale, act, chunked)
-    return ref.linear_attention(q, k, v, state, cu_q, slots, has_state, decay, gate, tau, q_scale, act)
+        return _cuda().linear_attention(q, k, v, state, cu_q, slots, has_state, decay, gate, tau, q_scale, act, chunked,
+                                        rope)
+    return ref.linear_attention(q, k, v, state, cu_q, slots, has_state, decay, gate, tau, q_scale, act, rope)
 
 
 def norm_gate(o, g, weight, eps: float, vdim: int, joint: bool, act: str, out_cols: int, total=None,
@@ -299,6 +301,32 @@ def norm_gate(o, g, weight, eps: float, vdim: int, joint: bool, act: str, out_co
     if o.is_cuda:
         return _cuda().norm_gate(o, g, weight, eps, vdim, joint, act, out_cols, total, total_heads)
     return ref.norm_gate(o, g, weight, eps, vdim, joint, act, out_cols, total, total_heads)
+
+
+# ---------------------------------------------------------------------------- selective scan, norms around a sublayer
+def causal_conv_silu(x, weight, bias, conv_state, cu_q, slots, has_state):
+    """A filter per channel over the current and earlier rows of a sequence (last tap: the current one), bias, silu.
+    ``x [T, C]``, ``weight [C, taps]`` and ``bias [C]`` fp32, ``conv_state [slots, C, taps - 1]``, updated in place."""
+    fn = _cuda().causal_conv_silu if x.is_cuda else ref.causal_conv_silu
+    return fn(x, weight, bias, conv_state, cu_q, slots, has_state)
+
+
+def selective_scan(x, dt, dt_bias, a, b, c, skip, z, state, cu_q, slots, has_state, chunked: bool = False):
+    """``S <- exp(dt a) S + dt x B``, ``y = S C + skip x`` per channel with ``dt`` the softplus of ``dt + dt_bias``; returns
+    ``y silu(z)``. ``chunked``: the step may take the form for prompts."""
+    fn = _cuda().selective_scan if x.is_cuda else ref.selective_scan
+    return fn(x, dt, dt_bias, a, b, c, skip, z, state, cu_q, slots, has_state, chunked)
+
+
+def residual_step(x, delta, norm, eps: float, out_dtype, out_cols: int, pair=None, post=None, history=None, coef=None):
+    """The end of a sublayer and the norm of the next, in one pass: ``(new residual, y [T, out_cols])``.
+
+    ``delta`` (fp32 rows, possibly unreduced K ranges; with ``pair = (w, w')`` two of them): the sublayer's output, or half
+    the sum of two RMS-normed and weighted ones. It takes the layer norm ``post`` (weight, bias) and is added to ``x`` (None:
+    zero). ``history`` (``layers.residual_norm.LayerHistory``): the sum is a layer's result and joins it; with ``coef``
+    the residual that goes on is the sum of ``coef[j]`` times result j. ``y``: the layer norm ``norm`` of it."""
+    fn = _cuda().residual_step if norm[0].is_cuda else ref.residual_step
+    return fn(x, delta, norm, eps, out_dtype, out_cols, pair, post, history, coef)
 
 
 def clamped_glu(x, limit: float, alpha: float):

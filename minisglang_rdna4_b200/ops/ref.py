@@ -208,7 +208,8 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
                     scale: float, causal: bool = True, window: int = 0,
                     mask: Optional[torch.Tensor] = None, k_scale: Optional[torch.Tensor] = None,
                     v_scale: Optional[torch.Tensor] = None, mask_window: int = 0, chunk: int = 0, softcap: float = 0.0,
-                    gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+                    gate: Optional[torch.Tensor] = None, bias: Optional[torch.Tensor] = None,
+                    sink: Optional[torch.Tensor] = None, talk: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Attention of packed queries over paged KV.
 
     ``q`` ``[T, Hq, D]``; request ``b`` owns rows ``cu_q[b]:cu_q[b+1]`` which are the LAST
@@ -220,7 +221,9 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
     ``mask_window`` KV positions of each request; earlier positions are visible to every row
     (of a sliding-window layer: to the rows that have them inside their window).
     ``chunk`` > 0: a row sees its own block of ``chunk`` positions only. ``softcap`` c > 0: ``c tanh(score / c)``.
-    ``gate [T, Hq * D]``: the output is multiplied by its sigmoid.
+    ``gate [T, Hq * D]``: the output is multiplied by its sigmoid. ``bias [Hq, reach]``: what a score loses at each
+    distance. ``sink [Hq]``: a score that only the softmax denominator counts. ``talk [Hq, Hq]``: head h applies
+    ``sum_g talk[h, g]`` times head g's weights.
     """
     t, hq, d = q.shape
     hk, ps = k_cache.shape[1], k_cache.shape[2]
@@ -247,6 +250,9 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
             s = softcap * torch.tanh(s / softcap)
         q_pos = torch.arange(kv_len - q_len, kv_len, device=q.device)[:, None]
         k_pos = torch.arange(kv_len, device=q.device)[None, :]
+        if bias is not None:
+            far = (q_pos - k_pos).clamp(0, bias.shape[1] - 1)
+            s = s - bias.float()[:, far].view(hk, group, q_len, kv_len)
         if mask is not None and mask_window:
             w = min(mask_window, kv_len)
             full = torch.zeros(q_len, kv_len, dtype=torch.float32, device=q.device)
@@ -264,8 +270,12 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
                 s = s.masked_fill((k_pos <= q_pos - window)[None, None], float("-inf"))
             if chunk > 0:
                 s = s.masked_fill((k_pos < q_pos - q_pos % chunk)[None, None], float("-inf"))
-        p = torch.softmax(s, dim=-1)
+        if sink is not None:
+            s = torch.cat([s, sink.float().view(hk, group, 1, 1).expand(hk, group, q_len, 1)], -1)
+        p = torch.softmax(s, dim=-1)[..., :kv_len]
         p = torch.nan_to_num(p, nan=0.0)
+        if talk is not None:
+            p = torch.einsum("hg,gqk->hqk", talk.float(), p.reshape(hq, q_len, kv_len)).view(hk, group, q_len, kv_len)
         o = torch.einsum("hgqk,hkd->hgqd", p, vv)  # [hk, g, q, d]
         out[qs:qe] = o.permute(2, 0, 1, 3).reshape(q_len, hq, d)
     if gate is not None:
@@ -790,12 +800,17 @@ def add_norm(x: torch.Tensor, delta: Optional[torch.Tensor], weight: torch.Tenso
 
 def linear_attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, state: torch.Tensor, cu_q: torch.Tensor,
                      slots: torch.Tensor, has_state: torch.Tensor, decay: Optional[torch.Tensor] = None, gate=None,
-                     tau: float = 1.0, q_scale: float = 1.0, act: bool = False) -> torch.Tensor:
+                     tau: float = 1.0, q_scale: float = 1.0, act: bool = False, rope=None) -> torch.Tensor:
     """Per head ``S <- diag(alpha_t) S + k_t v_t^T``, ``o_t = S^T q_t`` over packed sequences; ``q``, ``k [T, H, dk]``,
     ``v [T, H, dv]``, ``state [slots, H, dk, dv]`` fp32, updated in place. ``alpha``: ``decay [H]``, or per key channel
-    ``sigmoid(low W^T + bias) ** (1 / tau)`` from ``gate = (low [T, r], W [H * dk, r], bias [H * dk])``."""
+    ``sigmoid(low W^T + bias) ** (1 / tau)`` from ``gate = (low [T, r], W [H * dk, r], bias [H * dk])``. ``rope = (cos_sin
+    [positions, dims], positions [T])``: neighbouring channels of q and k are rotated first."""
     t, h, dk = q.shape
     qf, kf, vf = (F.silu(x.float()) if act else x.float() for x in (q, k, v))
+    if rope is not None:
+        dims, cs = rope[0].shape[1], rope[0][rope[1].long()].float()
+        qf, kf = (torch.cat([_rotate(x[..., :dims], cs[:, :dims // 2], cs[:, dims // 2:], True), x[..., dims:]], -1)
+                  for x in (qf, kf))
     qf = qf * q_scale
     if gate is not None:
         low, w, bias = gate
@@ -830,6 +845,56 @@ def norm_gate(o: torch.Tensor, g: torch.Tensor, weight: torch.Tensor, eps: float
     gf = g.float().reshape(t, h, dv)
     y = x * (torch.sigmoid(gf) if act == "sigmoid" else F.silu(gf))
     return F.pad(y.reshape(t, h * dv), (0, out_cols - h * dv)).to(o.dtype)
+
+
+def causal_conv_silu(x: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor, conv_state: torch.Tensor,
+                     cu_q: torch.Tensor, slots: torch.Tensor, has_state: torch.Tensor) -> torch.Tensor:
+    if weight.shape[1] == 1:
+        return F.silu(x.float() * weight[:, 0].float() + bias.float()).to(x.dtype)
+    return causal_conv1d(x, weight, conv_state, cu_q, slots, has_state, bias)
+
+
+def selective_scan(x: torch.Tensor, dt: torch.Tensor, dt_bias: torch.Tensor, a: torch.Tensor, b: torch.Tensor,
+                   c: torch.Tensor, skip: torch.Tensor, z: torch.Tensor, state: torch.Tensor, cu_q: torch.Tensor,
+                   slots: torch.Tensor, has_state: torch.Tensor, chunked: bool = False) -> torch.Tensor:
+    """Selective scan, token by token: ``x, dt, z [T, C]``, ``a [C, N]``, ``b, c [T, N]``, ``state [slots, 1, C, N]`` fp32,
+    updated in place."""
+    step = F.softplus(dt.float() + dt_bias.float(), threshold=40.0)
+    xf, bf, cf = x.float(), b.float(), c.float()
+    y = torch.empty(x.shape, dtype=torch.float32, device=x.device)
+    for i in range(cu_q.numel() - 1):
+        slot = int(slots[i])
+        s = state[slot, 0].clone() if int(has_state[i]) else torch.zeros_like(state[slot, 0])
+        for t in range(int(cu_q[i]), int(cu_q[i + 1])):
+            s = s * torch.exp(step[t][:, None] * a) + (step[t] * xf[t])[:, None] * bf[t]
+            y[t] = s @ cf[t]
+        state[slot, 0] = s
+    return ((y + skip * xf) * F.silu(z.float())).to(x.dtype)
+
+
+def residual_step(x: Optional[torch.Tensor], delta, norm, eps: float, out_dtype: torch.dtype, out_cols: int, pair=None,
+                  post=None, history=None, coef=None) -> Tuple[torch.Tensor, torch.Tensor]:
+    """See ``ops.residual_step``."""
+    width = norm[0].shape[0]
+
+    def layer_norm(y, weight, bias):
+        d = y - y.mean(-1, keepdim=True)
+        return d * torch.rsqrt(d.pow(2).mean(-1, keepdim=True) + eps) * weight + bias
+
+    if pair is not None:
+        u = sum(d[:, :width].float() * torch.rsqrt(d[:, :width].float().pow(2).mean(-1, keepdim=True) + eps) * w
+                for d, w in zip(delta, pair)) * 0.5
+    else:
+        u = delta[:, :width].float()
+    if post is not None:
+        u = layer_norm(u, *post)
+    xn = u if x is None else x + u
+    if history is not None:
+        history.rows[history.count] = xn
+        history.count += 1
+        if coef is not None:
+            xn = torch.einsum("j,jtw->tw", coef, history.rows[:history.count])
+    return xn, F.pad(layer_norm(xn, *norm), (0, out_cols - width)).to(out_dtype)
 
 
 def clamped_glu(x: torch.Tensor, limit: float, alpha: float) -> torch.Tensor:

@@ -86,7 +86,7 @@ class Replayer(Scheduler):
             out.wait()
             if wanted.size:
                 logits = out.logits[torch.from_numpy(wanted).long().to(out.logits.device)] if decode else out.logits
-                result = logits.float().cpu()
+                result = eng.sampler.condition_logits(logits, BatchSamplingArgs()).float().cpu()
         for name in end:
             req = self._live.pop(name)
             req.cached_len = req.device_len
@@ -133,7 +133,8 @@ def main(argv: Optional[Sequence[str]] = None) -> int:
 
         if not os.path.exists(_lib.LIB_PATH):
             if mc.has_fp32_kernels:
-                part = "heads" if mc.head_layers else "layered" if mc.layer_specs else "latent"
+                part = ("pair" if mc.depth_average else "heads" if mc.layered else "layered" if mc.layer_specs
+                        else "latent")
                 _lib.use_part(build.build_cuda(part=part))
             else:
                 build.build_cuda()

@@ -313,8 +313,8 @@ def _rollback_recurrent(eng, journal, slots, saved, cu, kept, finished) -> None:
     cu_new = torch.tensor(np.concatenate([[0], np.cumsum([kept[i] for i in part])]), dtype=torch.int32).to(dev)
     sub_slots = slots.index_select(0, which).to(torch.int32)
     has_state = torch.ones(len(part), dtype=torch.int32, device=dev)
-    for layer, proj in journal:
-        layer.replay(proj.index_select(0, rows), cu_new, sub_slots, has_state)
+    for layer, proj, *more in journal:          # more: further per-row inputs
+        layer.replay(proj.index_select(0, rows), cu_new, sub_slots, has_state, *(m.index_select(0, rows) for m in more))
 
 
 def _verify_plan(sched, batch: Batch, drafts):
