@@ -1,7 +1,11 @@
 // Paged attention in true fp32 (the 32-bit serving mode): grouped-query heads over an fp32 pool, causal, with a sliding
-// window or chunks, a soft cap on the scores and a sigmoid gate on the output. One CTA per (query row, head), blocks of 128
-// keys: a thread scores a key, then sums channels. Plain FMA arithmetic, blocks counted from the first visible key, so
-// that a row's result depends on nothing but its own keys.
+// window or chunks, a soft cap or a distance bias on the scores, a sink in the softmax denominator and a sigmoid gate on the
+// output. One CTA per (query row, head), blocks of 128 keys: a thread scores a key, then sums channels. Plain FMA arithmetic,
+// blocks counted from the first visible key, so that a row's result depends on nothing but its own keys.
+//
+// Heads that mix their weights: every head's weights meet the values of every key / value head (a CTA per value head), and
+// head_mix_kernel adds them up, out[h] = sum_g talk[h, g] o[g, value head of h]. The attention kernel also has a 16-bit form
+// for such layers with sizes that the tensor-core kernels do not take.
 #include "common.cuh"
 
 using namespace msgl;
@@ -11,10 +15,10 @@ namespace {
 constexpr int kKeys = 128, kMaxD = 512;
 
 struct F32AttnArgs {
-  const float* q;        // [rows, Hq, D]
-  const float* k;        // [pages, Hk, page_size, D]
-  const float* v;
-  float* out;            // [rows, Hq, D]
+  const void* q;         // [rows, Hq, D]
+  const void* k;         // [pages, Hk, page_size, D]
+  const void* v;
+  void* out;             // [rows, Hq, D], or [rows, Hq, Hk, D] with every head on all values
   const int32_t* block_table;
   const int32_t* cu_q;
   const int32_t* seq_lens;
@@ -22,29 +26,42 @@ struct F32AttnArgs {
   long long ldg;
   int bt_stride, B, Hq, Hk, D, page_size, pages, window, chunk;
   float scale, softcap;
+  const float* bias;     // [Hq, reach]: what a score loses at each distance, or null
+  int reach;
+  const float* sink;     // [Hq] scores that only the denominator counts, or null
 };
 
+__device__ __forceinline__ float4 load4f(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 load4f(const __nv_bfloat16* p) {
+  const uint2 q = *reinterpret_cast<const uint2*>(p);
+  const float2 u = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&q.x));
+  const float2 v = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&q.y));
+  return make_float4(u.x, u.y, v.x, v.y);
+}
+
+// ALL: grid.z value heads
+template <typename T, bool ALL>
 __global__ void __launch_bounds__(kKeys) paged_attention_f32_kernel(const F32AttnArgs a) {
   pdl_enter();
   __shared__ float q[kMaxD], p[kKeys], scratch[32];
   __shared__ long long at[kKeys];
   const int row = blockIdx.x, head = blockIdx.y, t = threadIdx.x;
-  const int hk = head / (a.Hq / a.Hk);
-  float* out = a.out + ((size_t)row * a.Hq + head) * a.D;
+  const int hk = head / (a.Hq / a.Hk), hv = ALL ? (int)blockIdx.z : hk;
+  T* out = reinterpret_cast<T*>(a.out) + (((size_t)row * a.Hq + head) * (ALL ? a.Hk : 1) + (ALL ? hv : 0)) * a.D;
   int b = 0, hi = a.B;                   // the request of this row
   while (hi - b > 1) {
     const int mid = (b + hi) >> 1;
     if (a.cu_q[mid] <= row) b = mid; else hi = mid;
   }
   if (row < a.cu_q[b] || row >= a.cu_q[b + 1]) {          // padding of a captured batch
-    for (int c = t; c < a.D; c += kKeys) out[c] = 0.f;
+    for (int c = t; c < a.D; c += kKeys) out[c] = from_float<T>(0.f);
     return;
   }
   const int pos = a.seq_lens[b] - (a.cu_q[b + 1] - row);
   int lo = 0;
   if (a.window > 0) lo = max(lo, pos - a.window + 1);
   if (a.chunk > 0) lo = max(lo, pos - pos % a.chunk);
-  for (int c = t; c < a.D; c += kKeys) q[c] = a.q[((size_t)row * a.Hq + head) * a.D + c];
+  for (int c = t; c < a.D; c += kKeys) q[c] = to_float(reinterpret_cast<const T*>(a.q)[((size_t)row * a.Hq + head) * a.D + c]);
   float acc[kMaxD / kKeys] = {}, m = -INFINITY, l = 0.f;
   for (int k0 = lo; k0 <= pos; k0 += kKeys) {
     const int tok = k0 + t;
@@ -54,15 +71,17 @@ __global__ void __launch_bounds__(kKeys) paged_attention_f32_kernel(const F32Att
       int page = a.block_table[(size_t)b * a.bt_stride + min(tok / a.page_size, a.bt_stride - 1)];
       (void)MSGL_OOB(page, a.pages);
       page = page < 0 ? 0 : (page >= a.pages ? a.pages - 1 : page);
-      at[t] = (((long long)page * a.Hk + hk) * a.page_size + tok % a.page_size) * a.D;
-      const float* k = a.k + at[t];
+      const long long first = (long long)page * a.Hk * a.page_size + tok % a.page_size;
+      at[t] = (first + (long long)hv * a.page_size) * a.D;
+      const T* k = reinterpret_cast<const T*>(a.k) + (first + (long long)hk * a.page_size) * a.D;
       float dot = 0.f;
       for (int c = 0; c < a.D; c += 4) {
-        const float4 x = *reinterpret_cast<const float4*>(k + c);
+        const float4 x = load4f(k + c);
         dot = fmaf(q[c], x.x, fmaf(q[c + 1], x.y, fmaf(q[c + 2], x.z, fmaf(q[c + 3], x.w, dot))));
       }
       s = dot * a.scale;
       if (a.softcap > 0.f) s = a.softcap * tanhf(s / a.softcap);
+      if (a.bias != nullptr) s -= a.bias[(size_t)head * a.reach + min(pos - tok, a.reach - 1)];
     }
     const float mn = fmaxf(m, block_max(s, scratch)), alpha = expf(m - mn), e = tok <= pos ? expf(s - mn) : 0.f;
     p[t] = e;
@@ -73,16 +92,57 @@ __global__ void __launch_bounds__(kKeys) paged_attention_f32_kernel(const F32Att
       const int c = t + i * kKeys;
       if (c >= a.D) break;
       float o = acc[i] * alpha;
-      for (int j = 0; j < n; ++j) o = fmaf(p[j], a.v[at[j] + c], o);
+      for (int j = 0; j < n; ++j) o = fmaf(p[j], to_float(reinterpret_cast<const T*>(a.v)[at[j] + c]), o);
       acc[i] = o;
     }
+  }
+  float num = 1.f;
+  if (a.sink != nullptr) {
+    const float mn = fmaxf(m, a.sink[head]);
+    num = expf(m - mn);
+    l = l * num + expf(a.sink[head] - mn);
   }
   for (int i = 0; i < kMaxD / kKeys; ++i) {
     const int c = t + i * kKeys;
     if (c >= a.D) break;
-    float o = acc[i] / l;
+    float o = acc[i] * num / l;
     if (a.gate != nullptr) o *= 1.f / (1.f + expf(-a.gate[row * a.ldg + head * a.D + c]));
-    out[c] = o;
+    out[c] = from_float<T>(o);
+  }
+}
+
+// o [rows, H, width] with value head c at columns c * D on; out [rows, H, D]. A thread sums a pair of channels for every
+// head of one value head, so that the rows are read once: grid (rows, Hk), D / 2 threads per part of the heads.
+template <typename T>
+__global__ void __launch_bounds__(256) head_mix_kernel(const T* __restrict__ o, const float* __restrict__ talk,
+                                                       T* __restrict__ out, int H, int Hk, int D, int width) {
+  pdl_enter();
+  extern __shared__ float mix[];               // [group][H]
+  const int row = blockIdx.x, hk = blockIdx.y, group = H / Hk;
+  for (int i = threadIdx.x; i < group * H; i += blockDim.x) mix[i] = talk[(size_t)hk * group * H + i];
+  __syncthreads();
+  const int pairs = D / 2, parts = blockDim.x / pairs, part = threadIdx.x / pairs;
+  if (part >= parts) return;
+  const T* src = o + (size_t)row * H * width + hk * D + (threadIdx.x - part * pairs) * 2;
+  T* dst = out + ((size_t)row * H + hk * group) * D + (threadIdx.x - part * pairs) * 2;
+  for (int h0 = part * 4; h0 < group; h0 += parts * 4) {
+    float acc[4][2] = {};
+#pragma unroll 4
+    for (int g = 0; g < H; ++g) {
+      const float u = to_float(src[(size_t)g * width]), v = to_float(src[(size_t)g * width + 1]);
+#pragma unroll
+      for (int k = 0; k < 4; ++k) {
+        const float f = h0 + k < group ? mix[(h0 + k) * H + g] : 0.f;
+        acc[k][0] = fmaf(f, u, acc[k][0]);
+        acc[k][1] = fmaf(f, v, acc[k][1]);
+      }
+    }
+#pragma unroll
+    for (int k = 0; k < 4; ++k)
+      if (h0 + k < group) {
+        dst[(size_t)(h0 + k) * D] = from_float<T>(acc[k][0]);
+        dst[(size_t)(h0 + k) * D + 1] = from_float<T>(acc[k][1]);
+      }
   }
 }
 
@@ -91,16 +151,45 @@ __global__ void __launch_bounds__(kKeys) paged_attention_f32_kernel(const F32Att
 MSGL_API int msgl_paged_attention_f32(const void* q, const void* k, const void* v, void* out, const void* block_table,
                                       int bt_stride, const void* cu_q, const void* seq_lens, int B, int rows, int hq, int hk,
                                       int d, int page_size, int pages, int window, int chunk, float scale, float softcap,
-                                      const void* gate, long long ldg, cudaStream_t stream) {
+                                      const void* gate, long long ldg, const void* bias, int reach, const void* sink,
+                                      int all_values, int dtype, cudaStream_t stream) {
   if (B == 0 || rows == 0) return MSGL_OK;
   if (hk <= 0 || hq % hk || d <= 0 || d % 4 || d > kMaxD || page_size <= 0 || bt_stride < 1) {
     msgl_set_error_text("fp32 attention: heads of up to 512 channels");
     return MSGL_BAD_ARG;
   }
-  F32AttnArgs a{(const float*)q, (const float*)k, (const float*)v, (float*)out, (const int32_t*)block_table,
-                (const int32_t*)cu_q, (const int32_t*)seq_lens, (const float*)gate, ldg, bt_stride, B, hq, hk, d, page_size,
-                pages, window, chunk, scale, softcap};
-  msgl_launch(paged_attention_f32_kernel, dim3(rows, hq), dim3(kKeys), 0, stream, a);
+  if ((bias != nullptr && reach <= 0) || (all_values && (gate != nullptr || hk > 65535)) ||
+      (dtype != MSGL_F32 && !(dtype == MSGL_BF16 && all_values)))
+    return MSGL_BAD_ARG;
+  F32AttnArgs a{q, k, v, out, (const int32_t*)block_table, (const int32_t*)cu_q, (const int32_t*)seq_lens, (const float*)gate,
+                ldg, bt_stride, B, hq, hk, d, page_size, pages, window, chunk, scale, softcap, (const float*)bias, reach,
+                (const float*)sink};
+  const dim3 grid(rows, hq, all_values ? hk : 1);
+  if (dtype == MSGL_BF16) msgl_launch(paged_attention_f32_kernel<__nv_bfloat16, true>, dim3(grid), dim3(kKeys), 0, stream, a);
+  else if (all_values) msgl_launch(paged_attention_f32_kernel<float, true>, dim3(grid), dim3(kKeys), 0, stream, a);
+  else msgl_launch(paged_attention_f32_kernel<float, false>, dim3(grid), dim3(kKeys), 0, stream, a);
   MSGL_CHECK_LAUNCH("paged_attention_f32");
+  return MSGL_OK;
+}
+
+// o [rows, H, width] (value head c at columns c * D on), talk [H, H] fp32 -> out [rows, H, D]
+MSGL_API int msgl_head_mix(const void* o, const void* talk, void* out, int rows, int h, int hk, int d, int width, int dtype,
+                           cudaStream_t stream) {
+  if (rows <= 0) return rows == 0 ? MSGL_OK : MSGL_BAD_ARG;
+  if (hk <= 0 || h % hk || d <= 0 || d % 2 || d > 512 || width < hk * d || (size_t)h * (h / hk) * 4 > 48 * 1024) {
+    msgl_set_error_text("head_mix: heads of up to 512 channels, 48 KiB of weights per value head");
+    return MSGL_BAD_ARG;
+  }
+  const dim3 grid(rows, hk);
+  const size_t smem = (size_t)h * (h / hk) * 4;
+  if (dtype == MSGL_BF16)
+    msgl_launch(head_mix_kernel<__nv_bfloat16>, dim3(grid), dim3(256), smem, stream, (const __nv_bfloat16*)o,
+                (const float*)talk, (__nv_bfloat16*)out, h, hk, d, width);
+  else if (dtype == MSGL_F32)
+    msgl_launch(head_mix_kernel<float>, dim3(grid), dim3(256), smem, stream, (const float*)o, (const float*)talk, (float*)out,
+                h, hk, d, width);
+  else
+    return MSGL_BAD_ARG;
+  MSGL_CHECK_LAUNCH("head_mix");
   return MSGL_OK;
 }

@@ -1,5 +1,6 @@
 // Causal prefill / extend attention on the tcgen05 tensor cores: head_dim 128 and an even GQA group, and extended forms
-// (rows of 64, any group, windows, chunks, capped scores, a gate on the output).
+// (rows of 64, any group, windows, chunks, capped scores, a gate on the output, a distance bias, every head on the values of
+// all key / value heads).
 //
 // The reference's prefill kernels (flash_prefill, flash_prefill_paged[_fp8];
 // python/minisgl/attention/hip.py:670-792, python/minisgl/attention/rdna4.py:419-503) walk the
@@ -75,6 +76,9 @@ struct TcArgs {
   const float* sink;   // [Hq] logits that only the softmax denominator counts, or null
   const void* gate;    // [rows, ...] logits of a sigmoid gate per row and head (row stride ldg), or null
   long long ldg;
+  const float* bias;   // TC_BIASED: [Hq][reach], what a score loses at each distance
+  int reach;
+  int v_blocks;        // TC_BIASED: blocks of 128 value columns that every query head meets (a CTA each); 0: its own head's
 };
 
 __device__ int g_attn_tc_status = 0;
@@ -175,7 +179,7 @@ template <typename T, bool KV8, int ROW>
 __global__ void __launch_bounds__(256)
 kv_gather_kernel(const void* __restrict__ k_pool, const void* __restrict__ v_pool, T* __restrict__ kc,
                  T* __restrict__ vt, const int* __restrict__ blk_req, const int* __restrict__ req_info,
-                 const int* __restrict__ block_table, int bt_stride, int Hk, int page_size, long long t_cap) {
+                 const int* __restrict__ block_table, int bt_stride, int Hk, int page_size, long long t_cap, int v_rows) {
   pdl_enter();
   __shared__ __align__(16) T vs[64][kD + 8];
   const int t0 = blockIdx.x * 64, h = blockIdx.y;
@@ -213,7 +217,7 @@ kv_gather_kernel(const void* __restrict__ k_pool, const void* __restrict__ v_poo
     o.y = (uint32_t)col[2 * rs] | ((uint32_t)col[3 * rs] << 16);
     o.z = (uint32_t)col[4 * rs] | ((uint32_t)col[5 * rs] << 16);
     o.w = (uint32_t)col[6 * rs] | ((uint32_t)col[7 * rs] << 16);
-    *reinterpret_cast<uint4*>(vt + ((long long)h * kD + d) * t_cap + t0 + ch * 8) = o;
+    if (d < v_rows) *reinterpret_cast<uint4*>(vt + ((long long)h * v_rows + d) * t_cap + t0 + ch * 8) = o;
   }
 }
 
@@ -222,26 +226,29 @@ kv_gather_kernel(const void* __restrict__ k_pool, const void* __restrict__ v_poo
 // ------------------------------------------------------------------------------------------
 // POS: the two tiles of a CTA are consecutive blocks of 128 positions of one head (where query heads that share keys
 // and values do not come in pairs, K / V tiles can only be shared along the positions) instead of two heads.
-// MODE: plain (for two heads: no reach, rows of 128), extended (reach, soft cap, gate, narrower rows), or extended with
-// scores that are capped within kFixedCap.
-enum { TC_PLAIN = 0, TC_EXTENDED = 1, TC_FIXED_CAP = 2 };
+// MODE: plain (for two heads: no reach, rows of 128), extended (reach, soft cap, gate, narrower rows), extended with
+// scores that are capped within kFixedCap, or with a distance bias, a sink and values of all heads.
+enum { TC_PLAIN = 0, TC_EXTENDED = 1, TC_FIXED_CAP = 2, TC_BIASED = 3 };
 template <typename T, bool POS, int MODE>
 __global__ void __launch_bounds__(kTcThreads, 1)
 attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_constant__ CUtensorMap tma_k,
                        const __grid_constant__ CUtensorMap tma_v, const __grid_constant__ CUtensorMap tma_g,
                        const TcArgs args) {
   pdl_enter();
-  constexpr bool EXT = MODE != TC_PLAIN, FIXCAP = MODE == TC_FIXED_CAP, REACH = POS || EXT;
+  constexpr bool EXT = MODE != TC_PLAIN, FIXCAP = MODE == TC_FIXED_CAP, BIAS = MODE == TC_BIASED, REACH = POS || EXT;
   extern __shared__ uint8_t smem_raw[];
   const uint32_t raw = smem_u32(smem_raw);
   const uint32_t s_base = (raw + 1023u) & ~1023u;
   uint8_t* smem = smem_raw + (s_base - raw);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
 
-  const int item_idx = blockIdx.x / args.pairs, pair = blockIdx.x - item_idx * args.pairs;
+  const int v_blocks = BIAS ? max(args.v_blocks, 1) : 1;
+  const int item_idx = blockIdx.x / (args.pairs * v_blocks), in_item = blockIdx.x - item_idx * args.pairs * v_blocks;
+  const int pair = in_item / v_blocks;
   const TcItem it = args.items[item_idx];
   const int head0 = POS ? pair : pair * 2;
   const int hk = head0 / (args.Hq / args.Hk);
+  const int hv = BIAS && args.v_blocks > 0 ? in_item - pair * v_blocks : hk;      // block of value columns
   const int nb = it.n_blocks;
 
   const uint32_t q_s = s_base + TcSmem::off_q, p_s = s_base + TcSmem::off_p, kv_s = s_base + TcSmem::off_kv;
@@ -304,14 +311,14 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
         if constexpr (POS) {
           for (int p = 0; p < 2; ++p) {
             if ((i & 1) == 0) tma_load_3d(dst + p * kPanel, &tma_k, kv_full(slot), 64 * p, hk, it.kv_off + j * kTile);
-            else tma_load_3d(dst + p * kPanel, &tma_v, kv_full(slot), it.kv_off + j * kTile + 64 * p, 0, hk);
+            else tma_load_3d(dst + p * kPanel, &tma_v, kv_full(slot), it.kv_off + j * kTile + 64 * p, 0, hv);
           }
         } else if ((i & 1) == 0) {
           tma_load_2d(dst, &tma_k, kv_full(slot), 0, k_row0 + j * kTile);
           tma_load_2d(dst + kPanel, &tma_k, kv_full(slot), 64, k_row0 + j * kTile);
         } else {
-          tma_load_2d(dst, &tma_v, kv_full(slot), it.kv_off + j * kTile, hk * kD);
-          tma_load_2d(dst + kPanel, &tma_v, kv_full(slot), it.kv_off + j * kTile + 64, hk * kD);
+          tma_load_2d(dst, &tma_v, kv_full(slot), it.kv_off + j * kTile, hv * kD);
+          tma_load_2d(dst + kPanel, &tma_v, kv_full(slot), it.kv_off + j * kTile + 64, hv * kD);
         }
       }
       if (*abort_flag) {  // let copies that are still in flight land before the CTA exits
@@ -383,8 +390,9 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
     const uint32_t swz = (uint32_t)(row & 7);
     const float raw_scale = args.scale * kLog2eTc * (args.k_scale != nullptr ? args.k_scale[hk] : 1.f);
     // capped scores come out in units of log2: tanh(x) = 1 - 2 / (1 + e^(2x))
-    const bool capped = EXT && !FIXCAP && args.softcap > 0.f, gated = EXT && args.cgate;
-    const float sl2 = capped ? 1.f : raw_scale;
+    const bool capped = EXT && !FIXCAP && !BIAS && args.softcap > 0.f, gated = EXT && !BIAS && args.cgate;
+    const float sl2 = capped ? 1.f : BIAS ? kLog2eTc : raw_scale;
+    const float* bias = BIAS ? args.bias + (size_t)head * args.reach : nullptr;
     const float cap_in = FIXCAP || capped ? 2.f * raw_scale / args.softcap : 0.f, cap_out = args.softcap * kLog2eTc;
     auto below = [&](int pos) {                        // last position ahead of what a row at pos sees
       int lo = -1;
@@ -461,6 +469,24 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
         continue;
       }
       float mx = -INFINITY;
+      if constexpr (BIAS) {
+        if (masked) {
+#pragma unroll
+          for (int c = 0; c < 4; ++c)
+#pragma unroll
+            for (int i = 0; i < 32; ++i) {
+              const int far = min(max(q_pos - kv0 - c * 32 - i, 0), args.reach - 1);
+              s[c][i] = __float_as_uint(fmaf(__uint_as_float(s[c][i]), args.scale, -__ldg(bias + far)));
+            }
+        } else {                       // every distance of the block is in the table
+          const float* at = bias + (q_pos - kv0 - (kTile - 1));
+#pragma unroll
+          for (int c = 0; c < 4; ++c)
+#pragma unroll
+            for (int i = 0; i < 32; ++i)
+              s[c][i] = __float_as_uint(fmaf(__uint_as_float(s[c][i]), args.scale, -__ldg(at + (kTile - 1 - c * 32 - i))));
+        }
+      }
       if (capped) {
 #pragma unroll
         for (int c = 0; c < 4; ++c) {
@@ -544,7 +570,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
       tc_fence_after();
       const int out_row = row + (POS ? t * kTile : 0);
       float num = args.v_scale != nullptr ? args.v_scale[hk] : 1.f;
-      if (POS && args.sink != nullptr) {
+      if ((POS || BIAS) && args.sink != nullptr) {
         // m is in units of raw scores; the sink is not scaled
         const float sk = args.sink[head] * kLog2eTc, ms = (m == -INFINITY ? 0.f : m) * sl2, mn = fmaxf(ms, sk);
         num *= ex2f(ms - mn);
@@ -554,7 +580,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
         num *= 1.f / (1.f + __expf(-to_float(reinterpret_cast<const T*>(args.gate)[(it.q_row0 + out_row) * args.ldg + head])));
       const float inv = l > 0.f ? num / l : 0.f;
       T* dst = reinterpret_cast<T*>(args.out) +
-               (REACH ? (long long)(it.q_row0 + out_row) * args.ldo + head * args.ho
+               (REACH ? (long long)(it.q_row0 + out_row) * args.ldo + head * args.ho + (BIAS && args.v_blocks > 0 ? hv * kD : 0)
                       : ((long long)(it.q_row0 + row) * args.Hq + head) * kD);
 #pragma unroll
       for (int c = 0; c < 4; ++c) tmem_ld_32x32b_x32(o_addr + c * 32, s[c]);
@@ -617,7 +643,7 @@ int launch_tc(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& m
     if (e != cudaSuccess) { msgl_set_error("prefill attention smem attribute", e); return MSGL_CUDA_ERROR; }
     configured = true;
   }
-  msgl_launch(attn_prefill_tc_kernel<T, POS, MODE>, dim3(a.n_items * a.pairs), dim3(kTcThreads), TcSmem::bytes, stream, mq, mk, mv, mg, a);
+  msgl_launch(attn_prefill_tc_kernel<T, POS, MODE>, dim3(a.n_items * a.pairs * (MODE == TC_BIASED && a.v_blocks > 0 ? a.v_blocks : 1)), dim3(kTcThreads), TcSmem::bytes, stream, mq, mk, mv, mg, a);
   MSGL_CHECK_LAUNCH("attn_prefill_tc");
   return MSGL_OK;
 }
@@ -710,9 +736,15 @@ MSGL_API int msgl_attn_prefill_tc(const void* q, long long q_row_stride, void* o
                                   const void* items, int n_items, const void* blk_req, const void* req_info,
                                   const void* block_table, int bt_stride, const void* k_scale, const void* v_scale,
                                   int total_q, int hq, int hk, int d, int page_size, int kv_fp8, float scale,
-                                  int window, int chunk, float softcap, const void* gate, long long ldg, int pos_form,
-                                  int dtype, cudaStream_t stream) {
+                                  int window, int chunk, float softcap, const void* gate, long long ldg, const void* bias,
+                                  int reach, const void* sink, int all_values, int pos_form, int dtype,
+                                  cudaStream_t stream) {
   if (n_items == 0 || total_q == 0) return MSGL_OK;
+  if (bias == nullptr ? (all_values || sink != nullptr)
+                      : (reach <= 0 || softcap > 0.f || gate != nullptr || dtype != MSGL_BF16 || kv_fp8)) {
+    msgl_set_error_text("prefill attention: a distance bias stands without soft cap, gate and fp8, sinks and mixed heads with one");
+    return MSGL_BAD_ARG;
+  }
   const bool ext = d != kD || window > 0 || chunk > 0 || softcap > 0.f || gate != nullptr;
   if ((ext || pos_form) && (dtype != MSGL_BF16 || kv_fp8)) {
     msgl_set_error_text("prefill attention: reaches, soft caps, gates, rows of 64 and unpaired query heads need bf16");
@@ -725,6 +757,8 @@ MSGL_API int msgl_attn_prefill_tc(const void* q, long long q_row_stride, void* o
                         "and a scratch of whole blocks");
     return MSGL_BAD_ARG;
   }
+  const int v_rows = all_values && d == 64 ? 64 : kD;      // value channels of a head in the scratch
+  const int v_blocks = all_values ? (hk * d + kD - 1) / kD : hk;
   CUtensorMap mq, mk, mv, mg;
   {
     cuuint64_t dims[3] = {(cuuint64_t)d, (cuuint64_t)hq, (cuuint64_t)total_q};
@@ -740,7 +774,7 @@ MSGL_API int msgl_attn_prefill_tc(const void* q, long long q_row_stride, void* o
     cuuint64_t kstr[2] = {(cuuint64_t)t_cap * kD * 2, (cuuint64_t)kD * 2};
     cuuint32_t kbox[3] = {64, 1, 128};
     if (!encode_map(&mk, kc, 3, kdims, kstr, kbox, "k")) return MSGL_CUDA_ERROR;
-    cuuint64_t vdims[3] = {(cuuint64_t)t_cap, (cuuint64_t)kD, (cuuint64_t)hk};
+    cuuint64_t vdims[3] = {(cuuint64_t)t_cap, (cuuint64_t)kD, (cuuint64_t)v_blocks};
     cuuint64_t vstr[2] = {(cuuint64_t)t_cap * 2, (cuuint64_t)t_cap * kD * 2};
     cuuint32_t vbox[3] = {64, 128, 1};
     if (!encode_map(&mv, vt, 3, vdims, vstr, vbox, "v")) return MSGL_CUDA_ERROR;
@@ -749,7 +783,7 @@ MSGL_API int msgl_attn_prefill_tc(const void* q, long long q_row_stride, void* o
     cuuint64_t strides[1] = {(cuuint64_t)kD * 2};
     cuuint32_t box[2] = {64, 128};
     if (!encode_map(&mk, kc, 2, dims, strides, box, "k")) return MSGL_CUDA_ERROR;
-    cuuint64_t vdims[2] = {(cuuint64_t)t_cap, (cuuint64_t)hk * kD};
+    cuuint64_t vdims[2] = {(cuuint64_t)t_cap, (cuuint64_t)v_blocks * kD};
     cuuint64_t vstr[1] = {(cuuint64_t)t_cap * 2};
     if (!encode_map(&mv, vt, 2, vdims, vstr, box, "v")) return MSGL_CUDA_ERROR;
   }
@@ -759,7 +793,7 @@ MSGL_API int msgl_attn_prefill_tc(const void* q, long long q_row_stride, void* o
 #define GATHER(T, F8, ROW)                                                                                              \
   msgl_launch(kv_gather_kernel<T, F8, ROW>, dim3(ggrid), dim3(256), 0, stream, k_pool, v_pool, (T*)kc, (T*)vt, (const int*)blk_req,          \
                                                      (const int*)req_info, (const int*)block_table, bt_stride, hk, \
-                                                     page_size, t_cap)
+                                                     page_size, t_cap, v_rows)
   if (d == 64) GATHER(__nv_bfloat16, false, 64);
   else if (dtype == MSGL_BF16) { if (kv_fp8) GATHER(__nv_bfloat16, true, 128); else GATHER(__nv_bfloat16, false, 128); }
   else { if (kv_fp8) GATHER(__half, true, 128); else GATHER(__half, false, 128); }
@@ -769,7 +803,12 @@ MSGL_API int msgl_attn_prefill_tc(const void* q, long long q_row_stride, void* o
   a.items = (const TcItem*)items; a.n_items = n_items; a.pairs = pos_form ? hq : hq / 2; a.Hq = hq; a.Hk = hk;
   a.t_cap = t_cap; a.out = out; a.k_scale = (const float*)k_scale; a.v_scale = (const float*)v_scale; a.scale = scale;
   a.status = status; a.window = window; a.chunk = chunk; a.softcap = softcap; a.cgate = gate != nullptr;
-  a.ldo = (long long)hq * d; a.ho = d; a.v_chunks = d / 8;
+  a.ho = all_values ? v_blocks * kD : d; a.ldo = a.ho * hq; a.v_chunks = all_values ? 16 : d / 8;
+  if (bias != nullptr) {
+    a.bias = (const float*)bias; a.reach = reach; a.sink = (const float*)sink; a.v_blocks = all_values ? v_blocks : 0;
+    return pos_form ? launch_tc<__nv_bfloat16, true, TC_BIASED>(mq, mk, mv, mg, a, stream)
+                    : launch_tc<__nv_bfloat16, false, TC_BIASED>(mq, mk, mv, mg, a, stream);
+  }
   const bool fixcap = softcap > 0.f && softcap * kLog2eTc <= kFixedCap && dtype == MSGL_BF16;
   if (pos_form) {
     return fixcap ? launch_tc<__nv_bfloat16, true, TC_FIXED_CAP>(mq, mk, mv, mg, a, stream)

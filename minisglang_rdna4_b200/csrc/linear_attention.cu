@@ -8,7 +8,8 @@
 //                                 not a plain 16-bit input is split into two bf16 terms.
 //   norm_gate_kernel              RMS norm of the result (per head or over all heads) times a gate
 //
-// Sequences are packed rows described by cu_q; a sequence without a state (has_state == 0) starts from zeros.
+// Sequences are packed rows described by cu_q; a sequence without a state (has_state == 0) starts from zeros. Queries and
+// keys may be rotated by position first (neighbouring channels are pairs), in fp32.
 #include "common.cuh"
 #include "ptx.cuh"
 
@@ -52,7 +53,18 @@ struct LinArgs {
   const float* bias;      // [H * dk]
   int H, dk, dv, rank, act, num_slots;
   float inv_tau, q_scale;
+  const float* cos_sin;   // [max_pos, rot]: cosines then sines of the pairs (2 i, 2 i + 1) of q and k, or null
+  const int32_t* positions;
+  int rot, max_pos;
 };
+
+// channel c of a row at a position: its share of the rotation and its partner's
+__device__ __forceinline__ float2 turn_of(const LinArgs& a, int pos, int c) {
+  pos = pos < 0 ? 0 : (pos < a.max_pos ? pos : a.max_pos - 1);
+  const float* cs = a.cos_sin + (size_t)pos * a.rot + (c >> 1);
+  const float sn = cs[a.rot >> 1];
+  return make_float2(cs[0], (c & 1) ? sn : -sn);
+}
 
 // ------------------------------------------------------------------------------------------ recurrent form
 // grid (dv / 32, H, B), 128 threads: thread (row group rg of 16, column group cg of 8) owns the rows rg, rg + 16, ... and
@@ -93,6 +105,16 @@ __global__ void __launch_bounds__(128) linear_attn_recurrent_kernel(const LinArg
         if (a.act) {
           qv = silu_as<T>(qv);
           kv = silu_as<T>(kv);
+        }
+        if (a.cos_sin != nullptr && c < a.rot) {
+          float qp = to_float(q[t * a.ld + (c ^ 1)]), kp = to_float(k[t * a.ld + (c ^ 1)]);
+          if (a.act) {
+            qp = silu_as<T>(qp);
+            kp = silu_as<T>(kp);
+          }
+          const float2 f = turn_of(a, a.positions[t], c);
+          qv = qv * f.x + qp * f.y;
+          kv = kv * f.x + kp * f.y;
         }
         al = scalar;
         if (a.decay == nullptr) {
@@ -237,7 +259,8 @@ template <int DK> struct ChunkSmem {
 // multiplied by 2^b_end once, and the scores q k^T between the chunk's tokens over their channels. None of that depends
 // on the chunks before, so groups of such warps work on different chunks at once. A chunk whose decay leaves the range
 // of the factors is handed over token by token. Stages go through named barriers.
-template <int DK>
+// ROT: q and k are rotated in fp32 by the producers; a lane holds the cosine (even channel) or sine (odd) of its pair.
+template <int DK, bool ROT>
 __global__ void __launch_bounds__(128 + ChunkSmem<DK>::G * DK, DK <= 64 ? 2 : 1) linear_attn_chunk_kernel(const LinArgs a) {
   pdl_enter();
   using L = ChunkSmem<DK>;
@@ -419,6 +442,19 @@ __global__ void __launch_bounds__(128 + ChunkSmem<DK>::G * DK, DK <= 64 ? 2 : 1)
   } else {
     fixed = fmaxf(log2f(a.decay[h]), -1e4f);
   }
+  float part_of_turn[ROT ? kC : 1];
+  const int pos0 = ROT ? a.positions[lo] : 0;
+  auto fetch_turns = [&](int start) {
+    if constexpr (ROT) {
+#pragma unroll
+      for (int t = 0; t < kC; ++t) {
+        const int pos = min(max(pos0 + min(start + t, len - 1), 0), a.max_pos - 1);
+        part_of_turn[t] = ch < a.rot ? a.cos_sin[(size_t)pos * a.rot + (ch >> 1) + (ch & 1) * (a.rot >> 1)]
+                                     : (ch & 1) ? 0.f : 1.f;
+      }
+    }
+  };
+  fetch_turns(grp * kC);
   int stage = 0, round = 0;
   for (int start = grp * kC; start < len; start += G * kC, ++round) {
     const int n = min(kC, len - start);
@@ -441,6 +477,17 @@ __global__ void __launch_bounds__(128 + ChunkSmem<DK>::G * DK, DK <= 64 ? 2 : 1)
           qf[t] = silu(qf[t]);
           kf[t] = silu(kf[t]);
         }
+      }
+      if constexpr (ROT) {
+#pragma unroll
+        for (int t = 0; t < kC; ++t) {
+          const float other = __shfl_xor_sync(0xffffffffu, part_of_turn[t], 1);
+          const float cs = (lane & 1) ? other : part_of_turn[t], sn = (lane & 1) ? part_of_turn[t] : -other;
+          const float qp = __shfl_xor_sync(0xffffffffu, qf[t], 1), kp = __shfl_xor_sync(0xffffffffu, kf[t], 1);
+          qf[t] = qf[t] * cs + qp * sn;
+          kf[t] = kf[t] * cs + kp * sn;
+        }
+        fetch_turns(start + G * kC);
       }
 #pragma unroll
       for (int t = 0; t < kC; ++t) qf[t] *= a.q_scale;
@@ -554,22 +601,25 @@ __global__ void __launch_bounds__(128 + ChunkSmem<DK>::G * DK, DK <= 64 ? 2 : 1)
   for (int i = max(stage - NS, 0); i < stage; ++i) bar_sync(EMPTY + grp * NS + i % NS, NT);
 }
 
-template <int DK> int launch_chunk(const LinArgs& a, int B, cudaStream_t s) {
+template <int DK, bool ROT> int launch_chunk_form(const LinArgs& a, int B, cudaStream_t s) {
   const int bytes = ChunkSmem<DK>::bytes(a.rank);
   static int set = 0;
   if (bytes > set) {
     const cudaError_t e =
-        cudaFuncSetAttribute(linear_attn_chunk_kernel<DK>, cudaFuncAttributeMaxDynamicSharedMemorySize, bytes);
+        cudaFuncSetAttribute(linear_attn_chunk_kernel<DK, ROT>, cudaFuncAttributeMaxDynamicSharedMemorySize, bytes);
     if (e != cudaSuccess) {
       msgl_set_error("linear_attention smem", e);
       return MSGL_CUDA_ERROR;
     }
     set = bytes;
   }
-  msgl_launch(linear_attn_chunk_kernel<DK>, dim3((a.dv + kCols - 1) / kCols, a.H, B), dim3(128 + ChunkSmem<DK>::G * DK), bytes,
-              s, a);
+  msgl_launch(linear_attn_chunk_kernel<DK, ROT>, dim3((a.dv + kCols - 1) / kCols, a.H, B),
+              dim3(128 + ChunkSmem<DK>::G * DK), bytes, s, a);
   MSGL_CHECK_LAUNCH("linear_attn_chunk");
   return MSGL_OK;
+}
+template <int DK> int launch_chunk(const LinArgs& a, int B, cudaStream_t s) {
+  return a.cos_sin != nullptr ? launch_chunk_form<DK, true>(a, B, s) : launch_chunk_form<DK, false>(a, B, s);
 }
 
 template <typename T> int launch_recurrent(const LinArgs& a, int B, cudaStream_t s) {
@@ -639,16 +689,19 @@ MSGL_API int msgl_linear_attention(const void* q, const void* k, const void* v, 
                                    long long slot_stride, const void* cu_q, const void* slots, const void* has_state,
                                    void* out, const void* decay, const void* low, const void* up, const void* bias, int B,
                                    int H, int dk, int dv, int rank, int act, int num_slots, float inv_tau, float q_scale,
-                                   int chunked, int dtype, cudaStream_t stream) {
+                                   const void* cos_sin, const void* positions, int rot, int max_pos, int chunked, int dtype,
+                                   cudaStream_t stream) {
   if (B <= 0) return B == 0 ? MSGL_OK : MSGL_BAD_ARG;
   if (H <= 0 || dk <= 0 || dv <= 0 || dk % 16 || dv % 16 || B > 65535 || H > 65535 || ld % 8 || slot_stride % 4 ||
       (uintptr_t)state % 16 || (uintptr_t)q % 16 || (uintptr_t)k % 16 || (uintptr_t)v % 16 || (uintptr_t)out % 16 ||
       (decay == nullptr && (low == nullptr || up == nullptr || bias == nullptr || rank <= 0 || (uintptr_t)low % 16 ||
-                            (uintptr_t)up % 16)))
+                            (uintptr_t)up % 16)) ||
+      (cos_sin != nullptr && (positions == nullptr || rot <= 0 || rot % 2 || rot > dk || max_pos <= 0)))
     return MSGL_BAD_ARG;
   LinArgs a{q, k, v, ld, (float*)state, slot_stride, (const int32_t*)cu_q, (const int32_t*)slots,
             (const int32_t*)has_state, out, (const float*)decay, low, up, (const float*)bias, H, dk, dv,
-            decay != nullptr ? 0 : rank, act, num_slots, inv_tau, q_scale};
+            decay != nullptr ? 0 : rank, act, num_slots, inv_tau, q_scale, (const float*)cos_sin, (const int32_t*)positions, rot,
+            max_pos};
   if (dtype == MSGL_F32) return launch_recurrent<float>(a, B, stream);
   if (dtype != MSGL_BF16) return MSGL_BAD_ARG;
   constexpr int kMaxSmem = 225 * 1024;

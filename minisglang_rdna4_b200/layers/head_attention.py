@@ -90,7 +90,7 @@ class HeadAttentionLayer(BaseOP):
         for at, n, used in ((0, self._h, spec.dim), (self._h, own, spec.dim), (self._h + own, own, spec.vdim)):
             weight[at * d:(at + n) * d].view(n, d, weight.shape[1])[:, used:] = 0
         if spec.log_bias:       # one number per head and distance in reach
-            far = torch.arange(spec.window or self._max_distance, dtype=torch.float64, device=weight.device)
+            far = torch.arange(spec.window or self._max_distance + 256, dtype=torch.float64, device=weight.device)
             bias = self.r1.double()[:, None] * torch.log1p(self.r2.double()[:, None] * far)
             self._extra["bias"] = bias.float().contiguous()
         if spec.zero_sink:

@@ -50,13 +50,13 @@ class SelectiveScanLayer(BaseOP):
             ctx.recurrent_journal.append((self, proj))
         md = batch.attn_metadata
         chunked = batch.is_prefill and not batch.spec_verify and md.max_q >= 8
-        return self._mix(proj, md.cu_q, batch.gdn_slots, batch.gdn_has_state, chunked)
+        return self._mix(proj, md.cu_q, batch.gdn_slots, batch.gdn_has_state, chunked, md.max_q)
 
-    def _mix(self, proj: torch.Tensor, cu_q, slots, has_state, chunked: bool) -> torch.Tensor:
+    def _mix(self, proj: torch.Tensor, cu_q, slots, has_state, chunked: bool, max_q: int = 0) -> torch.Tensor:
         """Convolution and recurrence over the projected rows; advances both states."""
         st, c, r, n = get_global_ctx().gdn_state, self._c, self._r, self._n
         x = ops.causal_conv_silu(proj[:, :c], self.conv, self.conv_bias, st.conv_state(self._state_row), cu_q, slots,
-                                 has_state)
+                                 has_state, max_q)
         y = self.x_proj.forward(x)
         if get_tp_info().size > 1:             # the other ranks hold the other channels
             y = get_comm().all_reduce(y)

@@ -304,11 +304,12 @@ def norm_gate(o, g, weight, eps: float, vdim: int, joint: bool, act: str, out_co
 
 
 # ---------------------------------------------------------------------------- selective scan, norms around a sublayer
-def causal_conv_silu(x, weight, bias, conv_state, cu_q, slots, has_state):
+def causal_conv_silu(x, weight, bias, conv_state, cu_q, slots, has_state, max_q: int = 0):
     """A filter per channel over the current and earlier rows of a sequence (last tap: the current one), bias, silu.
     ``x [T, C]``, ``weight [C, taps]`` and ``bias [C]`` fp32, ``conv_state [slots, C, taps - 1]``, updated in place."""
-    fn = _cuda().causal_conv_silu if x.is_cuda else ref.causal_conv_silu
-    return fn(x, weight, bias, conv_state, cu_q, slots, has_state)
+    if x.is_cuda:
+        return _cuda().causal_conv_silu(x, weight, bias, conv_state, cu_q, slots, has_state, max_q)
+    return ref.causal_conv_silu(x, weight, bias, conv_state, cu_q, slots, has_state)
 
 
 def selective_scan(x, dt, dt_bias, a, b, c, skip, z, state, cu_q, slots, has_state, chunked: bool = False):

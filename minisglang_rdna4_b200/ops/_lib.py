@@ -62,12 +62,15 @@ _SIGNATURES = {
     "msgl_paged_attention": (c_i, [c_p, c_p, c_p, c_p, c_i, c_p, c_p, c_p, c_p, c_p, c_ll, c_p,
                                    c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_i,
                                    c_f, c_i, c_f, c_p, c_ll, c_i, c_p]),
-    "msgl_paged_attention_f32": (c_i, [c_p] * 5 + [c_i, c_p, c_p] + [c_i] * 9 + [c_f, c_f, c_p, c_ll, c_p]),
+    "msgl_paged_attention_f32": (c_i, [c_p] * 5 + [c_i, c_p, c_p] + [c_i] * 9 + [c_f, c_f, c_p, c_ll, c_p, c_i, c_p, c_i, c_i,
+                                                                              c_p]),
+    "msgl_head_mix": (c_i, [c_p] * 3 + [c_i] * 6 + [c_p]),
     "msgl_heads_rope_store": (c_i, [c_p, c_ll, c_p, c_p, c_p, c_f, c_f, c_p, c_p, c_i] + [c_p] * 4 + [c_i] * 6
                               + [c_f] + [c_i] * 5 + [c_p]),
     "msgl_attn_status": (c_i, [c_i]),
     "msgl_attn_prefill_tc": (c_i, [c_p, c_ll, c_p, c_p, c_p, c_p, c_p, c_ll, c_i, c_p, c_i, c_p, c_p, c_p, c_i,
-                                   c_p, c_p, c_i, c_i, c_i, c_i, c_i, c_i, c_f, c_i, c_i, c_f, c_p, c_ll, c_i, c_i, c_p]),
+                                   c_p, c_p, c_i, c_i, c_i, c_i, c_i, c_i, c_f, c_i, c_i, c_f, c_p, c_ll, c_p, c_i, c_p, c_i,
+                                   c_i, c_i, c_p]),
     "msgl_attn_tc_status": (c_i, [c_i]),
     "msgl_attn_force_general_decode": (None, [c_i]),
     "msgl_attn_decode_stages": (None, [c_i]),

@@ -305,14 +305,17 @@ def choose_splits(batch, hk, max_kv, decode):
 
 def paged_attention(q, k_cache, v_cache, block_table, cu_q, seq_lens, scale, *, causal=True, window=0, mask=None,
                     k_scale=None, v_scale=None, max_q=0, max_kv=0, decode=False, workspace=None, splits=None,
-                    plan=None, tc=None, mask_window=0, chunk=0, softcap=0.0, gate=None):
+                    plan=None, tc=None, mask_window=0, chunk=0, softcap=0.0, gate=None, bias=None, sink=None, talk=None):
     """``plan`` (a ``PrefillPlan``) or ``tc=True`` sends a causal prefill / extend step to the
     tcgen05 kernel when it covers the shape (``tc=True`` without a plan builds the step tables from
     the device lengths, which synchronises). Without either the general kernel runs: decode and
     verification steps must not change kernels with the number of rows per request."""
-    if q.dtype == torch.float32:
+    if q.dtype == torch.float32 or talk is not None:
         assert causal and mask is None
-        return _paged_attention_f32(q, k_cache, v_cache, block_table, cu_q, seq_lens, scale, window, chunk, softcap, gate)
+        return _paged_attention_f32(q, k_cache, v_cache, block_table, cu_q, seq_lens, scale, window, chunk, softcap, gate, bias,
+                                    sink, talk)
+    if bias is not None or sink is not None:
+        raise NotImplementedError("16-bit attention takes a distance bias and a sink with mixed heads")
     t, hq, d = q.shape
     pages_p1, hk, ps, _ = k_cache.shape
     if max_q <= 0:
@@ -363,16 +366,37 @@ def _output_gate(gate, q):
     return gate.data_ptr(), gate.stride(0)
 
 
-def _paged_attention_f32(q, k_cache, v_cache, block_table, cu_q, seq_lens, scale, window, chunk, softcap, gate):
+def _distance_bias(bias, hq):
+    """Pointer and length of a table of what a score loses at each distance."""
+    if bias is None:
+        return None, 0
+    assert bias.dtype == torch.float32 and bias.is_contiguous() and bias.shape[0] == hq
+    return bias.data_ptr(), bias.shape[1]
+
+
+def _paged_attention_f32(q, k_cache, v_cache, block_table, cu_q, seq_lens, scale, window, chunk, softcap, gate, bias, sink,
+                         talk):
     t, hq, d = q.shape
     pages, hk, ps, _ = k_cache.shape
-    assert q.is_contiguous() and k_cache.is_contiguous() and v_cache.is_contiguous() and k_cache.dtype == torch.float32
-    out = torch.empty_like(q)
+    assert q.is_contiguous() and k_cache.is_contiguous() and v_cache.is_contiguous() and k_cache.dtype == q.dtype
+    out = torch.empty((t, hq, d if talk is None else hk * d), dtype=q.dtype, device=q.device)
     check(lib().msgl_paged_attention_f32(
         _p(q), _p(k_cache), _p(v_cache), _p(out), _p(block_table), block_table.stride(0), _p(cu_q), _p(seq_lens),
         seq_lens.numel(), t, hq, hk, d, ps, pages, int(window), int(chunk), float(scale), float(softcap),
-        *_output_gate(gate, q), _stream()), "paged_attention_f32")
+        *_output_gate(gate, q), *_distance_bias(bias, hq), _p(sink), int(talk is not None), _dt(q), _stream()),
+        "paged_attention_f32")
     _count("paged_attention_f32", "paged_attention_f32_kernel")
+    return out if talk is None else head_mix(out, talk, hk, d)
+
+
+def head_mix(o, talk, hk, d):
+    """``o [T, H, width]`` (value head c at columns ``c * d`` on) -> ``[T, H, d]``: head h gets the sum over g of
+    ``talk[h, g]`` times head g's rows of h's own value head."""
+    t, hq, width = o.shape
+    assert o.is_contiguous() and talk.dtype == torch.float32 and talk.is_contiguous() and talk.shape == (hq, hq)
+    out = torch.empty((t, hq, d), dtype=o.dtype, device=o.device)
+    check(lib().msgl_head_mix(_p(o), _p(talk), _p(out), t, hq, hk, d, width, _dt(o), _stream()), "head_mix")
+    _count("head_mix", "head_mix_kernel")
     return out
 
 
@@ -509,12 +533,12 @@ def prefill_heads_tc_ok(q, k_cache, scale) -> bool:
 
 
 def prefill_attention_tc(q, k_cache, v_cache, block_table, plan: PrefillPlan, scale, *, k_scale=None, v_scale=None,
-                         window=0, chunk=0, softcap=0.0, gate=None):
+                         window=0, chunk=0, softcap=0.0, gate=None, bias=None, sink=None, talk=None):
     """``plan`` was made for the same window and chunk."""
     t, hq, d = q.shape
     _, hk, ps, _ = k_cache.shape
     kc, vt, cap = _tc_scratch(q.device, q.dtype, hk, plan.t_pad)
-    out = torch.empty((t, hq, d), dtype=q.dtype, device=q.device)
+    out = torch.empty((t, hq, d if talk is None else -(-hk * d // 128) * 128), dtype=q.dtype, device=q.device)
     tb = plan.tables
     base = tb.data_ptr()
     fp8 = k_cache.dtype == torch.float8_e4m3fn
@@ -522,9 +546,10 @@ def prefill_attention_tc(q, k_cache, v_cache, block_table, plan: PrefillPlan, sc
         _p(q), q.stride(0), _p(out), _p(k_cache), _p(v_cache), _p(kc), _p(vt), cap, plan.t_pad,
         base, plan.n_items, base + 4 * plan.off_blk, base + 4 * plan.off_req, _p(block_table), block_table.stride(0),
         _p(k_scale), _p(v_scale), t, hq, hk, d, ps, int(fp8), float(scale), int(window), int(chunk), float(softcap),
-        *_output_gate(gate, q), int(plan.tile == 256), _dt(q), _stream()), "attn_prefill_tc")
+        *_output_gate(gate, q), *_distance_bias(bias, hq), _p(sink), int(talk is not None), int(plan.tile == 256), _dt(q),
+        _stream()), "attn_prefill_tc")
     _count("prefill_attention", "attn_prefill_tc_kernel", 2)
-    return out
+    return out if talk is None else head_mix(out, talk, hk, d)
 
 
 # ------------------------------------------------------------------------------------------ GEMM
@@ -1076,7 +1101,8 @@ def _bind_linear():
     if hasattr(_bind_linear, "_done"):
         return
     bind("msgl_add_norm", c_i, [c_p, c_p, c_p, c_i, c_ll, c_ll, c_p, c_p, c_i, c_i, c_i, c_f, c_i, c_p, c_f, c_i, c_p])
-    bind("msgl_linear_attention", c_i, [c_p, c_p, c_p, c_ll, c_p, c_ll] + [c_p] * 8 + [c_i] * 7 + [c_f, c_f, c_i, c_i, c_p])
+    bind("msgl_linear_attention", c_i, [c_p, c_p, c_p, c_ll, c_p, c_ll] + [c_p] * 8 + [c_i] * 7
+         + [c_f, c_f, c_p, c_p, c_i, c_i, c_i, c_i, c_p])
     bind("msgl_norm_gate", c_i, [c_p, c_p, c_ll, c_p, c_p, c_p, c_ll, c_i, c_i, c_f, c_f, c_i, c_i, c_p])
     _bind_linear._done = True
 
@@ -1102,7 +1128,7 @@ def add_norm(x, delta, weight, eps, center, out_dtype, out_cols, post=None, mult
 
 
 def linear_attention(q, k, v, state, cu_q, slots, has_state, decay=None, gate=None, tau=1.0, q_scale=1.0, act=False,
-                     chunked=False):
+                     chunked=False, rope=None):
     """See ``ref.linear_attention``; ``q``, ``k``, ``v`` and the low-rank input are views of the same projected rows, head
     widths multiples of 16. ``chunked``: the tensor-core form where it covers the sizes (16-bit prompts)."""
     _bind_linear()
@@ -1116,11 +1142,16 @@ def linear_attention(q, k, v, state, cu_q, slots, has_state, decay=None, gate=No
     if gate is not None:
         assert (t == 1 or low.stride(0) == ld) and low.stride(-1) == 1 and up.is_contiguous() and up.dtype == low.dtype == q.dtype
         assert bias.dtype == torch.float32 and up.shape == (h * dk, low.shape[1])
+    cos_sin, positions = rope if rope is not None else (None, None)
+    if rope is not None:
+        assert cos_sin.dtype == torch.float32 and cos_sin.is_contiguous() and positions.dtype == torch.int32
+        assert positions.numel() >= t
     out = torch.empty((t, h, dv), dtype=q.dtype, device=q.device)
     check(lib().msgl_linear_attention(
         _p(q), _p(k), _p(v), ld, _p(state), state.stride(0), _p(cu_q), _p(slots), _p(has_state), _p(out), _p(decay), _p(low),
         _p(up), _p(bias), cu_q.numel() - 1, h, dk, dv, 0 if low is None else low.shape[1], int(act), state.shape[0], 1.0 / tau,
-        q_scale, int(chunked), _dt(q), _stream()), "linear_attention")
+        q_scale, _p(cos_sin), _p(positions), 0 if rope is None else cos_sin.shape[1], 0 if rope is None else cos_sin.shape[0],
+        int(chunked), _dt(q), _stream()), "linear_attention")
     _count("linear_attention" + ("_chunked" if chunked else ""),
            "linear_attn_chunk_kernel" if chunked and q.dtype == torch.bfloat16 else "linear_attn_recurrent_kernel")
     return out
@@ -1138,6 +1169,88 @@ def norm_gate(o, g, weight, eps, vdim, joint, act, out_cols, total=None, total_h
                                int(act == "silu"), _dt(o), _stream()), "norm_gate")
     _count("norm_gate", "norm_gate_kernel")
     return out
+
+
+# ------------------------------------------------------------------------------------------ selective scan, norms around a sublayer
+def _bind_scan():
+    from ._lib import bind, c_f, c_i, c_ll, c_p
+
+    if hasattr(_bind_scan, "_done"):
+        return
+    bind("msgl_causal_conv_silu", c_i, [c_p, c_ll, c_p, c_p, c_p, c_ll] + [c_p] * 4 + [c_i] * 6 + [c_p])
+    bind("msgl_selective_scan", c_i, [c_p] * 6 + [c_ll, c_p, c_p, c_ll, c_p, c_ll] + [c_p] * 4 + [c_i] * 6 + [c_p])
+    _bind_scan._done = True
+
+
+def causal_conv_silu(x, weight, bias, conv_state, cu_q, slots, has_state, max_q=0):
+    _bind_scan()
+    t, c = x.shape
+    assert x.stride(1) == 1 and weight.is_contiguous() and weight.dtype == bias.dtype == torch.float32
+    assert conv_state.dtype == x.dtype and conv_state.shape[1:] == (c, weight.shape[1] - 1)
+    assert conv_state.shape[2] == 0 or conv_state[0].is_contiguous()
+    out = torch.empty((t, c), dtype=x.dtype, device=x.device)
+    check(lib().msgl_causal_conv_silu(_p(x), x.stride(0), _p(weight), _p(bias), _p(conv_state), conv_state.stride(0), _p(cu_q),
+                                      _p(slots), _p(has_state), _p(out), cu_q.numel() - 1, c, weight.shape[1], max_q or t,
+                                      conv_state.shape[0], _dt(x), _stream()), "causal_conv_silu")
+    _count("causal_conv_silu", "causal_conv_silu_kernel")
+    return out
+
+
+def selective_scan(x, dt, dt_bias, a, b, c, skip, z, state, cu_q, slots, has_state, chunked=False):
+    """See ``ops.selective_scan``; ``b`` and ``c`` are views of the same rows, channels a multiple of 16, states of 4."""
+    _bind_scan()
+    t, ch = x.shape
+    n = a.shape[1]
+    assert x.is_contiguous() and dt.is_contiguous() and dt.dtype == torch.float32 and a.is_contiguous() and z.stride(1) == 1
+    assert b.stride(1) == c.stride(1) == 1 and b.stride(0) == c.stride(0) and b.dtype == c.dtype == z.dtype == x.dtype
+    assert state.dtype == torch.float32 and state.shape[1:] == (1, ch, n) and state[0].is_contiguous()
+    for w in (dt_bias, a, skip):
+        assert w.dtype == torch.float32
+    out = torch.empty((t, ch), dtype=x.dtype, device=x.device)
+    check(lib().msgl_selective_scan(
+        _p(x), _p(dt), _p(dt_bias), _p(a), _p(b), _p(c), b.stride(0), _p(skip), _p(z), z.stride(0), _p(state), state.stride(0),
+        _p(cu_q), _p(slots), _p(has_state), _p(out), cu_q.numel() - 1, ch, n, state.shape[0], int(chunked), _dt(x), _stream()),
+        "selective_scan")
+    _count("selective_scan" + ("_tiles" if chunked else ""),
+           "scan_tiles_kernel" if chunked and x.dtype != torch.float32 else "scan_rows_kernel")
+    return out
+
+
+def residual_step(x, delta, norm, eps, out_dtype, out_cols, pair=None, post=None, history=None, coef=None):
+    """See ``ops.residual_step``."""
+    from ._lib import bind, c_f, c_i, c_ll, c_p
+
+    if not hasattr(residual_step, "_done"):
+        bind("msgl_residual_step", c_i, [c_p, c_p, c_i, c_ll, c_ll, c_p, c_i, c_ll, c_ll] + [c_p] * 5 + [c_i] + [c_p] * 5
+             + [c_i] * 3 + [c_f, c_i, c_p])
+        residual_step._done = True
+    width, rows = norm[0].shape[0], 0
+    args = []
+    for d in (delta if pair is not None else (delta,)):
+        d = d.planes if isinstance(d, SplitPartial) else d.unsqueeze(0)
+        rows = d.shape[1]
+        assert d.dtype == torch.float32 and d.stride(2) == 1 and d.shape[2] >= width
+        args += [_p(d), d.shape[0], d.stride(0), d.stride(1)]
+    args += [None, 0, 0, 0] if pair is None else []
+    for w in (*norm, *(pair or ()), *(post or ())):
+        assert w.dtype == torch.float32 and w.numel() == width
+    assert x is None or (x.is_contiguous() and x.dtype == torch.float32 and x.shape == (rows, width))
+    n = 0
+    if history is not None:
+        n, history.count = history.count, history.count + 1
+        assert history.rows.is_contiguous() and history.rows.shape[1:] == (rows, width) and n < history.rows.shape[0]
+        assert coef is None or (coef.dtype == torch.float32 and coef.numel() == n + 1)
+    own = history is None or coef is not None
+    x_out = torch.empty((rows, width), dtype=torch.float32, device=norm[0].device) if own else history.rows[n]
+    y = torch.empty((rows, out_cols), dtype=out_dtype, device=norm[0].device)
+    w0, w1 = pair or (None, None)
+    pw, pb = post or (None, None)
+    check(lib().msgl_residual_step(
+        _p(x), *args, _p(w0), _p(w1), _p(pw), _p(pb), None if history is None else _p(history.rows), n, _p(coef),
+        _p(x_out) if own else None, _p(norm[0]), _p(norm[1]), _p(y), rows, width, out_cols, eps, _DT[out_dtype], _stream()),
+        "residual_step")
+    _count("residual_step", "residual_step_kernel")
+    return x_out, y
 
 
 # ------------------------------------------------------------------------------------------ latent attention
