@@ -39,8 +39,9 @@ class LayerPlans:
 
 class PagedAttentionBackend(BaseAttnBackend):
     def __init__(self, num_q_heads: int, num_kv_heads: int, head_dim: int, device,
-                 max_batch: int = 0, max_seq_len: int = 0, single_split: bool = False, heads=None) -> None:
-        """``heads``: ``(query heads, row width)`` per layer where layers differ."""
+                 max_batch: int = 0, max_seq_len: int = 0, single_split: bool = False, heads=None, talk=None) -> None:
+        """``heads``: ``(query heads, row width)`` per layer where layers differ; ``talk``: ``(query heads, key / value heads,
+        row width)`` of those whose heads mix their weights."""
         self.hq, self.hk, self.d = num_q_heads, num_kv_heads, head_dim
         self.layered = bool(heads)
         self.device = device
@@ -51,11 +52,13 @@ class PagedAttentionBackend(BaseAttnBackend):
         self.max_seq_len = max_seq_len
         self.single_split = single_split
         self._workspace: Optional[torch.Tensor] = None
+        self._talk_workspace: Optional[torch.Tensor] = None
         if torch.device(device).type == "cuda":
             from ..ops import cuda as K
 
             hq, d = max(heads, key=lambda s: s[0] * (s[1] + 1)) if heads else (num_q_heads, head_dim)
             self._workspace = K.attention_workspace(max(max_batch, 1), hq, d, device)
+            self._talk_workspace = K.talk_workspace(talk, device) if talk else None
             K.force_general_decode_attention(single_split)
 
     def prepare_metadata(self, batch: Batch, block_table, cu_q, seq_lens, max_q: int, max_kv: int,
@@ -110,11 +113,13 @@ class PagedAttentionBackend(BaseAttnBackend):
                     return K.prefill_attention_tc(q, k_cache, v_cache, md.block_table, plan, scale, **extra)
             if md.decode and not self.single_split:
                 reach = min([r for r in (window, chunk, self.max_seq_len or md.max_kv) if r > 0])
-                # mixed heads: a CTA has all of them
-                splits = K.choose_splits(md.seq_lens.numel(), 1 if talk is not None else k_cache.shape[1], reach, True)
+                if talk is not None:               # a CTA has all heads
+                    splits = K.talk_splits(md.seq_lens.numel(), q.shape[1], k_cache.shape[1], q.shape[2], reach)
+                else:
+                    splits = K.choose_splits(md.seq_lens.numel(), k_cache.shape[1], reach, True)
         return ops.paged_attention(q, k_cache, v_cache, md.block_table, md.cu_q, md.seq_lens, scale, causal=True,
-                                   max_q=md.max_q, max_kv=md.max_kv, decode=md.decode, workspace=md.workspace,
-                                   splits=splits, **extra)
+                                   max_q=md.max_q, max_kv=md.max_kv, decode=md.decode,
+                                   workspace=md.workspace if talk is None else self._talk_workspace, splits=splits, **extra)
 
     def forward(self, q, layer: int, batch: Batch, *, scale: float, window: int = 0, swa: bool = False):
         md = batch.attn_metadata

@@ -77,7 +77,7 @@ PARTS = {
     "heads": ["elementwise", "gemm_tcgen05", "gemm_f32", "norm_conv", "residual_norm", "rope_kv", "attention",
               "attention_f32", "attention_tc", "moe", "sampling"],
     "pair": ["elementwise", "gemm_tcgen05", "gemm_f32", "norm_conv", "residual_norm", "rope_kv", "attention",
-             "attention_f32", "attention_tc", "linear_attention", "selective_scan", "moe", "sampling"],
+             "attention_f32", "attention_tc", "attention_talk", "linear_attention", "selective_scan", "moe", "sampling"],
 }
 
 

@@ -261,6 +261,182 @@ template <typename T> int launch_rows(const ScanArgs& a, int B, cudaStream_t s) 
   return MSGL_OK;
 }
 
+// ------------------------------------------------------------------------------------------ prompts
+__device__ __forceinline__ void cp16(uint32_t dst, const void* src, bool valid) {
+  const int n = valid ? 16 : 0;
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(n) : "memory");
+}
+__device__ __forceinline__ void cp8(uint32_t dst, const void* src, bool valid) {
+  const int n = valid ? 8 : 0;
+  asm volatile("cp.async.ca.shared.global [%0], [%1], 8, %2;" ::"r"(dst), "l"(src), "r"(n) : "memory");
+}
+
+constexpr int kTile = 32;      // tokens
+template <int LN, int G> struct TileSmem {
+  static constexpr int CH = 128 / LN, NP = LN * G * 4;      // channels of a CTA, states
+  // raw rows, two deep: x, z, B ‖ C in 16 bits, dt
+  static constexpr int off_z = kTile * CH * 2, off_dt = 2 * off_z, off_bc = off_dt + kTile * CH * 4;
+  static constexpr int raw = off_bc + kTile * 2 * NP * 2;
+  static constexpr int off_step = 2 * raw;                    // (dt, dt x) [tile][CH]
+  static constexpr int off_b = off_step + kTile * CH * 8;     // B and C in fp32 [tile][2][NP]
+  static constexpr int off_y = off_b + kTile * 2 * NP * 4;    // [tile][CH]
+  static constexpr int bytes = off_y + kTile * CH * 4;
+};
+
+// grid (channels / CH, B), 128 threads. Per tile: softplus and products of all (token, channel) pairs; the recurrence, LN
+// lanes per channel; skip, gate and store of all pairs. The next tile's rows arrive meanwhile.
+template <int LN, int G>
+__global__ void __launch_bounds__(128) scan_tiles_kernel(const ScanArgs a) {
+  pdl_enter();
+  using bf = __nv_bfloat16;
+  using L = TileSmem<LN, G>;
+  constexpr int CH = L::CH, NP = L::NP;
+  extern __shared__ __align__(16) uint8_t smem[];
+  const uint32_t base = (uint32_t)__cvta_generic_to_shared(smem);
+  const int tid = threadIdx.x, b = blockIdx.y, cl = tid / LN, ln = tid % LN, c_first = blockIdx.x * CH, c = c_first + cl;
+  const int lo = a.cu_q[b], len = a.cu_q[b + 1] - lo;
+  if (len <= 0) return;
+  const int slot = a.slots[b];
+  if (MSGL_OOB(slot, a.num_slots) || slot < 0 || slot >= a.num_slots) return;
+  const bf* x = reinterpret_cast<const bf*>(a.x) + (size_t)lo * a.channels + c_first;
+  const bf* z = reinterpret_cast<const bf*>(a.z) + (size_t)lo * a.ldz + c_first;
+  const float* dt = a.dt + (size_t)lo * a.channels + c_first;
+  const bf* B = reinterpret_cast<const bf*>(a.B) + (size_t)lo * a.ldb;
+  const bf* C = reinterpret_cast<const bf*>(a.Cm) + (size_t)lo * a.ldb;
+  const int left = min(CH, a.channels - c_first);
+  auto fetch = [&](int t0, int buf) {
+    if (t0 < len) {
+      const uint32_t dst = base + buf * L::raw;
+      for (int i = tid; i < kTile * CH / 8; i += 128) {
+        const int t = i / (CH / 8), k = i % (CH / 8) * 8;
+        const bool ok = t0 + t < len && k < left;
+        cp16(dst + i * 16, x + (ok ? (size_t)(t0 + t) * a.channels + k : 0), ok);
+        cp16(dst + L::off_z + i * 16, z + (ok ? (size_t)(t0 + t) * a.ldz + k : 0), ok);
+      }
+      for (int i = tid; i < kTile * CH / 4; i += 128) {
+        const int t = i / (CH / 4), k = i % (CH / 4) * 4;
+        const bool ok = t0 + t < len && k < left;
+        cp16(dst + L::off_dt + i * 16, dt + (ok ? (size_t)(t0 + t) * a.channels + k : 0), ok);
+      }
+      for (int i = tid; i < kTile * 2 * NP / 4; i += 128) {
+        const int t = i / (2 * NP / 4), k = i % (2 * NP / 4) * 4, n = k < NP ? k : k - NP;
+        const bool ok = t0 + t < len && n < a.N;
+        cp8(dst + L::off_bc + i * 8, (k < NP ? B : C) + (ok ? (size_t)(t0 + t) * a.ldb + n : 0), ok);
+      }
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  fetch(0, 0);
+
+  const bool live = c < a.channels, keep = a.has_state[b] != 0;
+  float* S = a.state + slot * a.slot_stride + (size_t)(live ? c : 0) * a.N;
+  const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+  float4 s[G], A[G];
+#pragma unroll
+  for (int g = 0; g < G; ++g) {
+    const int n = (g * LN + ln) * 4;
+    s[g] = keep && live && n < a.N ? *reinterpret_cast<const float4*>(S + n) : zero;
+    A[g] = live && n < a.N ? *reinterpret_cast<const float4*>(a.A + (size_t)c * a.N + n) : zero;
+    A[g].x *= kLog2e; A[g].y *= kLog2e; A[g].z *= kLog2e; A[g].w *= kLog2e;
+  }
+  // the channel that this thread takes ahead of and behind the recurrence
+  constexpr int ROWS = 128 / CH;             // tokens side by side
+  const int pc = tid % CH, pt = tid / CH;
+  const bool plive = pc < left;
+  const float bias = plive ? a.dt_bias[c_first + pc] : 0.f, skip = plive ? a.skip[c_first + pc] : 0.f;
+  float2* step = reinterpret_cast<float2*>(smem + L::off_step);
+  float* bc = reinterpret_cast<float*>(smem + L::off_b);
+  float* ys = reinterpret_cast<float*>(smem + L::off_y);
+  for (int t0 = 0, buf = 0; t0 < len; t0 += kTile, buf ^= 1) {
+    const int n = min(kTile, len - t0);
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();                         // the tile is there, and the one before is done with its buffers
+    fetch(t0 + kTile, buf ^ 1);
+    const uint8_t* raw = smem + buf * L::raw;
+    const bf* xs = reinterpret_cast<const bf*>(raw);
+    const bf* zs = reinterpret_cast<const bf*>(raw + L::off_z);
+    const float* ds = reinterpret_cast<const float*>(raw + L::off_dt);
+#pragma unroll
+    for (int t = pt; t < kTile; t += ROWS) {
+      const float d = t < n ? softplus<bf>(ds[t * CH + pc] + bias) : 0.f;       // past the end: the state stays
+      step[t * CH + pc] = make_float2(d, d * to_float(xs[t * CH + pc]));
+    }
+    for (int i = tid; i < kTile * 2 * NP / 4; i += 128)
+      *reinterpret_cast<float4*>(bc + i * 4) = load4f(reinterpret_cast<const bf*>(raw + L::off_bc) + i * 4);
+    __syncthreads();
+    for (int t = 0; t < n; t += 4) {
+      float y[4];
+#pragma unroll
+      for (int k = 0; k < 4; ++k) {
+        const float2 d = step[(t + k) * CH + cl];
+        const float* row = bc + (t + k) * 2 * NP + ln * 4;
+        float4 Bv[G], Cv[G];
+#pragma unroll
+        for (int g = 0; g < G; ++g) {
+          Bv[g] = *reinterpret_cast<const float4*>(row + g * LN * 4);
+          Cv[g] = *reinterpret_cast<const float4*>(row + NP + g * LN * 4);
+        }
+        y[k] = advance<bf, G>(s, A, Bv, Cv, d.x, d.y);
+      }
+      // sums over the lanes of a channel; every exchange halves the tokens a lane is left with
+      if constexpr (LN == 1) {
+#pragma unroll
+        for (int k = 0; k < 4; ++k) ys[(t + k) * CH + cl] = y[k];
+      } else {
+        const bool up = ln & 1;
+        const float v0 = (up ? y[2] : y[0]) + __shfl_xor_sync(0xffffffffu, up ? y[0] : y[2], 1);
+        const float v1 = (up ? y[3] : y[1]) + __shfl_xor_sync(0xffffffffu, up ? y[1] : y[3], 1);
+        if constexpr (LN == 2) {
+          ys[(t + 2 * up) * CH + cl] = v0;
+          ys[(t + 2 * up + 1) * CH + cl] = v1;
+        } else {
+          const bool up2 = ln & 2;
+          float w = (up2 ? v1 : v0) + __shfl_xor_sync(0xffffffffu, up2 ? v0 : v1, 2);
+#pragma unroll
+          for (int m = 4; m < LN; m <<= 1) w += __shfl_xor_sync(0xffffffffu, w, m);
+          if (ln < 4) ys[(t + 2 * up + up2) * CH + cl] = w;
+        }
+      }
+    }
+    __syncthreads();
+    if (plive) {
+      bf* out = reinterpret_cast<bf*>(a.out) + (size_t)(lo + t0) * a.channels + c_first + pc;
+#pragma unroll 4
+      for (int t = pt; t < n; t += ROWS)
+        out[(size_t)t * a.channels] = __float2bfloat16(fmaf(skip, to_float(xs[t * CH + pc]), ys[t * CH + pc]) *
+                                                       silu<bf>(to_float(zs[t * CH + pc])));
+    }
+  }
+#pragma unroll
+  for (int g = 0; g < G; ++g) {
+    const int n = (g * LN + ln) * 4;
+    if (live && n < a.N) *reinterpret_cast<float4*>(S + n) = s[g];
+  }
+}
+
+template <int LN, int G> int launch_tiles_form(const ScanArgs& a, int B, cudaStream_t s) {
+  using L = TileSmem<LN, G>;
+  static bool set = false;
+  if (!set) {
+    const cudaError_t e = cudaFuncSetAttribute(scan_tiles_kernel<LN, G>, cudaFuncAttributeMaxDynamicSharedMemorySize, L::bytes);
+    if (e != cudaSuccess) { msgl_set_error("selective_scan smem", e); return MSGL_CUDA_ERROR; }
+    set = true;
+  }
+  msgl_launch(scan_tiles_kernel<LN, G>, dim3((a.channels + L::CH - 1) / L::CH, B), dim3(128), L::bytes, s, a);
+  MSGL_CHECK_LAUNCH("selective_scan");
+  return MSGL_OK;
+}
+int launch_tiles(const ScanArgs& a, int B, cudaStream_t s) {
+  if (a.N <= 4) return launch_tiles_form<1, 1>(a, B, s);
+  if (a.N <= 8) return launch_tiles_form<2, 1>(a, B, s);
+  if (a.N <= 16) return launch_tiles_form<4, 1>(a, B, s);
+  if (a.N <= 32) return launch_tiles_form<4, 2>(a, B, s);
+  if (a.N <= 64) return launch_tiles_form<8, 2>(a, B, s);
+  if (a.N <= 128) return launch_tiles_form<8, 4>(a, B, s);
+  if (a.N <= 256) return launch_tiles_form<16, 4>(a, B, s);
+  return launch_rows<__nv_bfloat16>(a, B, s);
+}
+
 }  // namespace
 
 // x [T, channels] with row stride ldx (channels even); out [T, channels]
@@ -307,6 +483,5 @@ MSGL_API int msgl_selective_scan(const void* x, const void* dt, const void* dt_b
                    channels, N, num_slots};
   if (dtype == MSGL_F32) return launch_rows<float>(a, batch, stream);
   if (dtype != MSGL_BF16) return MSGL_BAD_ARG;
-  (void)tiles;
-  return launch_rows<__nv_bfloat16>(a, batch, stream);
+  return tiles ? launch_tiles(a, batch, stream) : launch_rows<__nv_bfloat16>(a, batch, stream);
 }

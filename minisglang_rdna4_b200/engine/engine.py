@@ -370,7 +370,8 @@ class Engine:
             config.attention_backend, self.q_heads_local, self.kv_heads_local, mc.head_dim, self.device,
             max_batch=config.max_running_req, max_seq_len=self.max_seq_len,
             single_split=config.spec_algorithm != "none", latent=mc.latent_layers,
-            heads=[(m.heads if m.talk else div_even(m.heads, config.tp_size), m.row_pad) for m in mc.head_layers],
+            heads=[(1 if m.talk else div_even(m.heads, config.tp_size), m.row_pad) for m in mc.head_layers],
+            talk=[(m.heads, m.kv_heads, m.row_pad) for m in mc.head_layers if m.talk],
         )
         self.ctx.comm = comm_mod.get_comm()
         self._spec_exact = config.spec_algorithm != "none" and dev_kind == "cuda"

@@ -310,6 +310,10 @@ def paged_attention(q, k_cache, v_cache, block_table, cu_q, seq_lens, scale, *, 
     tcgen05 kernel when it covers the shape (``tc=True`` without a plan builds the step tables from
     the device lengths, which synchronises). Without either the general kernel runs: decode and
     verification steps must not change kernels with the number of rows per request."""
+    if talk is not None and talk_attention_ok(q, k_cache, chunk, softcap, gate):
+        assert causal and mask is None
+        return talk_attention(q, k_cache, v_cache, block_table, cu_q, seq_lens, scale, talk, bias, sink, window, decode,
+                              splits or 1, workspace)
     if q.dtype == torch.float32 or talk is not None:
         assert causal and mask is None
         return _paged_attention_f32(q, k_cache, v_cache, block_table, cu_q, seq_lens, scale, window, chunk, softcap, gate, bias,
@@ -387,6 +391,44 @@ def _paged_attention_f32(q, k_cache, v_cache, block_table, cu_q, seq_lens, scale
         "paged_attention_f32")
     _count("paged_attention_f32", "paged_attention_f32_kernel")
     return out if talk is None else head_mix(out, talk, hk, d)
+
+
+def talk_attention_ok(q, k_cache, chunk=0, softcap=0.0, gate=None) -> bool:
+    """Sizes of the decode kernel for mixed heads; others take the plain one."""
+    return (q.dtype == torch.bfloat16 and q.shape[2] in (64, 128) and q.shape[1] <= 64 and k_cache.shape[2] in (8, 16, 32, 64)
+            and not chunk and not softcap and gate is None)
+
+
+def talk_splits(batch: int, heads: int, hk: int, d: int, reach: int) -> int:
+    """Key ranges of a decode step with mixed heads: a CTA per SM, two blocks of 64 keys or more in a range."""
+    groups = -(-hk // (2 if hk <= 2 or (heads > 32 and d == 128) else 4))
+    return int(max(1, min(148 // max(batch * groups, 1), reach // 128, 16)))
+
+
+def talk_workspace(heads, device):
+    """For the largest split step of layers of ``(heads, kv heads, width)``: rows times ranges stay within 148."""
+    need = max(int(lib().msgl_talk_workspace_floats(148, h, hk, d, 1)) for h, hk, d in heads)
+    return workspace("mixed-head attention partials", need, torch.float32, device)
+
+
+def talk_attention(q, k_cache, v_cache, block_table, cu_q, seq_lens, scale, talk, bias=None, sink=None, window=0, decode=False,
+                   splits=1, workspace=None):
+    """Attention with mixed heads for single query rows: one pass over keys and values for all heads."""
+    t, hq, d = q.shape
+    pages_p1, hk, ps, _ = k_cache.shape
+    desc, layer, layers = _kv_map(k_cache)
+    assert q.is_contiguous() and talk.dtype == torch.float32 and talk.is_contiguous() and talk.shape == (hq, hq)
+    if splits > 1:
+        need = int(lib().msgl_talk_workspace_floats(t, hq, hk, d, splits))
+        if workspace is None or workspace.numel() < need:
+            workspace = torch.empty(need, dtype=torch.float32, device=q.device)
+    out = torch.empty_like(q)
+    check(lib().msgl_talk_attention(
+        desc.ctypes.data, _p(q), _p(out), _p(block_table), block_table.stride(0), _p(cu_q), _p(seq_lens),
+        *_distance_bias(bias, hq), _p(sink), _p(talk), _p(workspace) if splits > 1 else None, seq_lens.numel(), t, hq, hk, d, ps,
+        pages_p1 - 1, layer, layers, int(window), splits, int(decode), float(scale), _stream()), "talk_attention")
+    _count("talk_attention", "talk_decode_kernel", 2 if splits > 1 else 1)
+    return out
 
 
 def head_mix(o, talk, hk, d):
@@ -875,7 +917,7 @@ def gemm_fp8_block_status(reset=True) -> int:
 def attn_status(reset=True) -> int:
     a = int(lib().msgl_attn_status(int(reset)))
     b = int(lib().msgl_attn_tc_status(int(reset)))
-    return a or b
+    return a or b or int(lib().msgl_talk_status(int(reset)))
 
 
 # ------------------------------------------------------------------------------------------ sampling
