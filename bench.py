@@ -84,7 +84,7 @@ def parse_args():
     ap.add_argument("--no-matched", action="store_true",
                     help="skip the extra bf16-weights / bf16-KV run of this repository that is reported beside "
                          "the quantised number for a like-for-like ratio against the bf16 reference arm")
-    ap.add_argument("--design", default=None, choices=["mitilix", "rafodra", "zobelorn"],
+    ap.add_argument("--design", default=None, choices=["mitilix", "rafodra", "zobelorn", "ligipel"],
                     help="instead of the workload: prefill / decode throughput and kernel rooflines of this design "
                          "beside the closest family at equal size (minisglang_rdna4_b200/benchmark/design.py)")
     ap.add_argument("--size", default="all", choices=["small", "large", "all"], help="with --design")

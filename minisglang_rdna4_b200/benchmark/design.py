@@ -1,8 +1,9 @@
 """Prefill and decode throughput of a design beside the closest family at equal size, and the time of every kernel of
 both against its roofline: Mitilix beside a Mistral-shaped decoder (grouped-query sliding-window attention, gated MLP);
-Rafodra beside the Qwen3-Next hybrid (``design_rafodra.py``); Zobelorn beside Laguna (``design_zobelorn.py``).
+Rafodra beside the Qwen3-Next hybrid (``design_rafodra.py``); Zobelorn beside Laguna (``design_zobelorn.py``); Ligipel beside
+Nemotron-H (``design_ligipel.py``).
 
-``python bench.py --design mitilix|rafodra|zobelorn [--size small|large]`` prints one JSON line per (size, model) and one per kernel.
+``python bench.py --design mitilix|rafodra|zobelorn|ligipel [--size small|large]`` prints one JSON line per (size, model) and one per kernel.
 Random weights, synthetic token ids, one GPU. Throughput comes from CUDA events around every engine step of
 ``LLM.generate``; a kernel is timed with CUDA events over many launches of which each flushes L2 first."""
 from __future__ import annotations
@@ -269,6 +270,10 @@ def run(design: str, size: str, what: str, clocks) -> None:
         from . import design_zobelorn as d
 
         sizes, pair, kernel_rows = d.SIZES, (("zobelorn", d.zobelorn_config), ("laguna", d.laguna_config)), d.kernels
+    elif design == "ligipel":
+        from . import design_ligipel as d
+
+        sizes, pair, kernel_rows = d.SIZES, (("ligipel", d.ligipel_config), ("nemotron_h", d.nemotron_config)), d.kernels
     else:
         sizes, pair, kernel_rows = SIZES, (("mitilix", mitilix_config), ("mistral", mistral_config)), kernels
     names = list(sizes) if size == "all" else [size]
