@@ -108,7 +108,8 @@ class PagedAttentionBackend(BaseAttnBackend):
             from ..ops import cuda as K
 
             if md.layer_plans is not None and K.prefill_heads_tc_ok(q, k_cache, scale):
-                plan = md.layer_plans.of(window, chunk, q.shape[1] // k_cache.shape[1])
+                # (a CTA of the form with a distance bias has one head)
+                plan = md.layer_plans.of(window, chunk, 2 if bias is not None else q.shape[1] // k_cache.shape[1])
                 if plan is not None:
                     return K.prefill_attention_tc(q, k_cache, v_cache, md.block_table, plan, scale, **extra)
             if md.decode and not self.single_split:

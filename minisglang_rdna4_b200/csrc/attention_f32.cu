@@ -111,39 +111,41 @@ __global__ void __launch_bounds__(kKeys) paged_attention_f32_kernel(const F32Att
   }
 }
 
-// o [rows, H, width] with value head c at columns c * D on; out [rows, H, D]. A thread sums a pair of channels for every
-// head of one value head, so that the rows are read once: grid (rows, Hk), D / 2 threads per part of the heads.
+// o [rows, H, width] with value head c at columns c * D on; out [rows, H, D]. A thread sums eight channels for up to eight
+// heads of one value head, so that the rows are read once per eight heads: grid (rows * Hk * D / 8 / 128, parts of a group).
 template <typename T>
-__global__ void __launch_bounds__(256) head_mix_kernel(const T* __restrict__ o, const float* __restrict__ talk,
-                                                       T* __restrict__ out, int H, int Hk, int D, int width) {
+__global__ void __launch_bounds__(128) head_mix_kernel(const T* __restrict__ o, const float* __restrict__ talk,
+                                                       T* __restrict__ out, int rows, int H, int Hk, int D, int width) {
   pdl_enter();
-  extern __shared__ float mix[];               // [group][H]
-  const int row = blockIdx.x, hk = blockIdx.y, group = H / Hk;
-  for (int i = threadIdx.x; i < group * H; i += blockDim.x) mix[i] = talk[(size_t)hk * group * H + i];
-  __syncthreads();
-  const int pairs = D / 2, parts = blockDim.x / pairs, part = threadIdx.x / pairs;
-  if (part >= parts) return;
-  const T* src = o + (size_t)row * H * width + hk * D + (threadIdx.x - part * pairs) * 2;
-  T* dst = out + ((size_t)row * H + hk * group) * D + (threadIdx.x - part * pairs) * 2;
-  for (int h0 = part * 4; h0 < group; h0 += parts * 4) {
-    float acc[4][2] = {};
-#pragma unroll 4
-    for (int g = 0; g < H; ++g) {
-      const float u = to_float(src[(size_t)g * width]), v = to_float(src[(size_t)g * width + 1]);
-#pragma unroll
-      for (int k = 0; k < 4; ++k) {
-        const float f = h0 + k < group ? mix[(h0 + k) * H + g] : 0.f;
-        acc[k][0] = fmaf(f, u, acc[k][0]);
-        acc[k][1] = fmaf(f, v, acc[k][1]);
-      }
-    }
-#pragma unroll
-    for (int k = 0; k < 4; ++k)
-      if (h0 + k < group) {
-        dst[(size_t)(h0 + k) * D] = from_float<T>(acc[k][0]);
-        dst[(size_t)(h0 + k) * D + 1] = from_float<T>(acc[k][1]);
-      }
+  extern __shared__ float mix[];               // [Hk][H][8]: weights of this part's heads, zero past the group
+  const int group = H / Hk, h0 = blockIdx.y * 8, n = min(8, group - h0);
+  for (int i = threadIdx.x; i < Hk * H * 8; i += 128) {
+    const int k = i & 7, g = (i >> 3) % H, c = (i >> 3) / H;
+    mix[i] = k < n ? talk[(size_t)(c * group + h0 + k) * H + g] : 0.f;
   }
+  __syncthreads();
+  const int per_row = Hk * D / 8;
+  const long long id = (long long)blockIdx.x * 128 + threadIdx.x;
+  const int row = (int)(id / per_row), col = (int)(id - (long long)row * per_row) * 8, c = col / D;
+  if (row >= rows) return;
+  const T* src = o + (size_t)row * H * width + col;
+  const float* w = mix + (size_t)c * H * 8;
+  float acc[8][8] = {};
+#pragma unroll 8
+  for (int g = 0; g < H; ++g) {
+    float x[8];
+    load8(src + (size_t)g * width, x);
+    const float4 f0 = *reinterpret_cast<const float4*>(w + g * 8), f1 = *reinterpret_cast<const float4*>(w + g * 8 + 4);
+    const float f[8] = {f0.x, f0.y, f0.z, f0.w, f1.x, f1.y, f1.z, f1.w};
+#pragma unroll
+    for (int k = 0; k < 8; ++k)
+#pragma unroll
+      for (int e = 0; e < 8; ++e) acc[k][e] = fmaf(f[k], x[e], acc[k][e]);
+  }
+  T* dst = out + ((size_t)row * H + c * group + h0) * D + col % D;
+#pragma unroll
+  for (int k = 0; k < 8; ++k)
+    if (k < n) store8(dst + (size_t)k * D, acc[k]);
 }
 
 }  // namespace
@@ -172,24 +174,30 @@ MSGL_API int msgl_paged_attention_f32(const void* q, const void* k, const void* 
   return MSGL_OK;
 }
 
-// o [rows, H, width] (value head c at columns c * D on), talk [H, H] fp32 -> out [rows, H, D]
+// o [rows, H, width] (value head c at columns c * d on), talk [H, H] fp32 -> out [rows, H, d]
 MSGL_API int msgl_head_mix(const void* o, const void* talk, void* out, int rows, int h, int hk, int d, int width, int dtype,
                            cudaStream_t stream) {
   if (rows <= 0) return rows == 0 ? MSGL_OK : MSGL_BAD_ARG;
-  if (hk <= 0 || h % hk || d <= 0 || d % 2 || d > 512 || width < hk * d || (size_t)h * (h / hk) * 4 > 48 * 1024) {
-    msgl_set_error_text("head_mix: heads of up to 512 channels, 48 KiB of weights per value head");
+  const size_t smem = (size_t)h * hk * 32;
+  if (hk <= 0 || h % hk || d <= 0 || d % 8 || width % 8 || width < hk * d || smem > 200 * 1024 || (uintptr_t)o % 16 ||
+      (uintptr_t)out % 16) {
+    msgl_set_error_text("head_mix: widths in eights, up to 6400 pairs of a query and a key / value head");
     return MSGL_BAD_ARG;
   }
-  const dim3 grid(rows, hk);
-  const size_t smem = (size_t)h * (h / hk) * 4;
-  if (dtype == MSGL_BF16)
-    msgl_launch(head_mix_kernel<__nv_bfloat16>, dim3(grid), dim3(256), smem, stream, (const __nv_bfloat16*)o,
-                (const float*)talk, (__nv_bfloat16*)out, h, hk, d, width);
-  else if (dtype == MSGL_F32)
-    msgl_launch(head_mix_kernel<float>, dim3(grid), dim3(256), smem, stream, (const float*)o, (const float*)talk, (float*)out,
-                h, hk, d, width);
-  else
-    return MSGL_BAD_ARG;
+  const long long threads = (long long)rows * hk * d / 8;
+  const dim3 grid((unsigned)((threads + 127) / 128), (h / hk + 7) / 8);
+#define HEAD_MIX(T)                                                                                                     \
+  do {                                                                                                                  \
+    if (smem > 48 * 1024 &&                                                                                             \
+        cudaFuncSetAttribute(head_mix_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) \
+      return MSGL_CUDA_ERROR;                                                                                           \
+    msgl_launch(head_mix_kernel<T>, dim3(grid), dim3(128), smem, stream, (const T*)o, (const float*)talk, (T*)out, rows, \
+                h, hk, d, width);                                                                                       \
+  } while (0)
+  if (dtype == MSGL_BF16) HEAD_MIX(__nv_bfloat16);
+  else if (dtype == MSGL_F32) HEAD_MIX(float);
+  else return MSGL_BAD_ARG;
+#undef HEAD_MIX
   MSGL_CHECK_LAUNCH("head_mix");
   return MSGL_OK;
 }

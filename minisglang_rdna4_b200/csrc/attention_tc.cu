@@ -76,9 +76,6 @@ struct TcArgs {
   const float* sink;   // [Hq] logits that only the softmax denominator counts, or null
   const void* gate;    // [rows, ...] logits of a sigmoid gate per row and head (row stride ldg), or null
   long long ldg;
-  const float* bias;   // TC_BIASED: [Hq][reach], what a score loses at each distance
-  int reach;
-  int v_blocks;        // TC_BIASED: blocks of 128 value columns that every query head meets (a CTA each); 0: its own head's
 };
 
 __device__ int g_attn_tc_status = 0;
@@ -226,29 +223,26 @@ kv_gather_kernel(const void* __restrict__ k_pool, const void* __restrict__ v_poo
 // ------------------------------------------------------------------------------------------
 // POS: the two tiles of a CTA are consecutive blocks of 128 positions of one head (where query heads that share keys
 // and values do not come in pairs, K / V tiles can only be shared along the positions) instead of two heads.
-// MODE: plain (for two heads: no reach, rows of 128), extended (reach, soft cap, gate, narrower rows), extended with
-// scores that are capped within kFixedCap, or with a distance bias, a sink and values of all heads.
-enum { TC_PLAIN = 0, TC_EXTENDED = 1, TC_FIXED_CAP = 2, TC_BIASED = 3 };
+// MODE: plain (for two heads: no reach, rows of 128), extended (reach, soft cap, gate, narrower rows), or extended with
+// scores that are capped within kFixedCap.
+enum { TC_PLAIN = 0, TC_EXTENDED = 1, TC_FIXED_CAP = 2 };
 template <typename T, bool POS, int MODE>
 __global__ void __launch_bounds__(kTcThreads, 1)
 attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_constant__ CUtensorMap tma_k,
                        const __grid_constant__ CUtensorMap tma_v, const __grid_constant__ CUtensorMap tma_g,
                        const TcArgs args) {
   pdl_enter();
-  constexpr bool EXT = MODE != TC_PLAIN, FIXCAP = MODE == TC_FIXED_CAP, BIAS = MODE == TC_BIASED, REACH = POS || EXT;
+  constexpr bool EXT = MODE != TC_PLAIN, FIXCAP = MODE == TC_FIXED_CAP, REACH = POS || EXT;
   extern __shared__ uint8_t smem_raw[];
   const uint32_t raw = smem_u32(smem_raw);
   const uint32_t s_base = (raw + 1023u) & ~1023u;
   uint8_t* smem = smem_raw + (s_base - raw);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
 
-  const int v_blocks = BIAS ? max(args.v_blocks, 1) : 1;
-  const int item_idx = blockIdx.x / (args.pairs * v_blocks), in_item = blockIdx.x - item_idx * args.pairs * v_blocks;
-  const int pair = in_item / v_blocks;
+  const int item_idx = blockIdx.x / args.pairs, pair = blockIdx.x - item_idx * args.pairs;
   const TcItem it = args.items[item_idx];
   const int head0 = POS ? pair : pair * 2;
   const int hk = head0 / (args.Hq / args.Hk);
-  const int hv = BIAS && args.v_blocks > 0 ? in_item - pair * v_blocks : hk;      // block of value columns
   const int nb = it.n_blocks;
 
   const uint32_t q_s = s_base + TcSmem::off_q, p_s = s_base + TcSmem::off_p, kv_s = s_base + TcSmem::off_kv;
@@ -311,14 +305,14 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
         if constexpr (POS) {
           for (int p = 0; p < 2; ++p) {
             if ((i & 1) == 0) tma_load_3d(dst + p * kPanel, &tma_k, kv_full(slot), 64 * p, hk, it.kv_off + j * kTile);
-            else tma_load_3d(dst + p * kPanel, &tma_v, kv_full(slot), it.kv_off + j * kTile + 64 * p, 0, hv);
+            else tma_load_3d(dst + p * kPanel, &tma_v, kv_full(slot), it.kv_off + j * kTile + 64 * p, 0, hk);
           }
         } else if ((i & 1) == 0) {
           tma_load_2d(dst, &tma_k, kv_full(slot), 0, k_row0 + j * kTile);
           tma_load_2d(dst + kPanel, &tma_k, kv_full(slot), 64, k_row0 + j * kTile);
         } else {
-          tma_load_2d(dst, &tma_v, kv_full(slot), it.kv_off + j * kTile, hv * kD);
-          tma_load_2d(dst + kPanel, &tma_v, kv_full(slot), it.kv_off + j * kTile + 64, hv * kD);
+          tma_load_2d(dst, &tma_v, kv_full(slot), it.kv_off + j * kTile, hk * kD);
+          tma_load_2d(dst + kPanel, &tma_v, kv_full(slot), it.kv_off + j * kTile + 64, hk * kD);
         }
       }
       if (*abort_flag) {  // let copies that are still in flight land before the CTA exits
@@ -390,9 +384,8 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
     const uint32_t swz = (uint32_t)(row & 7);
     const float raw_scale = args.scale * kLog2eTc * (args.k_scale != nullptr ? args.k_scale[hk] : 1.f);
     // capped scores come out in units of log2: tanh(x) = 1 - 2 / (1 + e^(2x))
-    const bool capped = EXT && !FIXCAP && !BIAS && args.softcap > 0.f, gated = EXT && !BIAS && args.cgate;
-    const float sl2 = capped ? 1.f : BIAS ? kLog2eTc : raw_scale;
-    const float* bias = BIAS ? args.bias + (size_t)head * args.reach : nullptr;
+    const bool capped = EXT && !FIXCAP && args.softcap > 0.f, gated = EXT && args.cgate;
+    const float sl2 = capped ? 1.f : raw_scale;
     const float cap_in = FIXCAP || capped ? 2.f * raw_scale / args.softcap : 0.f, cap_out = args.softcap * kLog2eTc;
     auto below = [&](int pos) {                        // last position ahead of what a row at pos sees
       int lo = -1;
@@ -469,24 +462,6 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
         continue;
       }
       float mx = -INFINITY;
-      if constexpr (BIAS) {
-        if (masked) {
-#pragma unroll
-          for (int c = 0; c < 4; ++c)
-#pragma unroll
-            for (int i = 0; i < 32; ++i) {
-              const int far = min(max(q_pos - kv0 - c * 32 - i, 0), args.reach - 1);
-              s[c][i] = __float_as_uint(fmaf(__uint_as_float(s[c][i]), args.scale, -__ldg(bias + far)));
-            }
-        } else {                       // every distance of the block is in the table
-          const float* at = bias + (q_pos - kv0 - (kTile - 1));
-#pragma unroll
-          for (int c = 0; c < 4; ++c)
-#pragma unroll
-            for (int i = 0; i < 32; ++i)
-              s[c][i] = __float_as_uint(fmaf(__uint_as_float(s[c][i]), args.scale, -__ldg(at + (kTile - 1 - c * 32 - i))));
-        }
-      }
       if (capped) {
 #pragma unroll
         for (int c = 0; c < 4; ++c) {
@@ -570,7 +545,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
       tc_fence_after();
       const int out_row = row + (POS ? t * kTile : 0);
       float num = args.v_scale != nullptr ? args.v_scale[hk] : 1.f;
-      if ((POS || BIAS) && args.sink != nullptr) {
+      if (POS && args.sink != nullptr) {
         // m is in units of raw scores; the sink is not scaled
         const float sk = args.sink[head] * kLog2eTc, ms = (m == -INFINITY ? 0.f : m) * sl2, mn = fmaxf(ms, sk);
         num *= ex2f(ms - mn);
@@ -580,7 +555,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
         num *= 1.f / (1.f + __expf(-to_float(reinterpret_cast<const T*>(args.gate)[(it.q_row0 + out_row) * args.ldg + head])));
       const float inv = l > 0.f ? num / l : 0.f;
       T* dst = reinterpret_cast<T*>(args.out) +
-               (REACH ? (long long)(it.q_row0 + out_row) * args.ldo + head * args.ho + (BIAS && args.v_blocks > 0 ? hv * kD : 0)
+               (REACH ? (long long)(it.q_row0 + out_row) * args.ldo + head * args.ho
                       : ((long long)(it.q_row0 + row) * args.Hq + head) * kD);
 #pragma unroll
       for (int c = 0; c < 4; ++c) tmem_ld_32x32b_x32(o_addr + c * 32, s[c]);
@@ -617,6 +592,426 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_c
   if (warp == 1) tmem_dealloc(tmem_base, 512);
 }
 
+// ------------------------------------------------------------------------------------------
+// 3. The form with a distance bias and a sink, whose heads may meet the values of all key / value heads. A unit of work is
+// (128 query positions, query head, up to two blocks of 128 value columns); one CTA per SM takes units in turn, heaviest
+// first, and loads and multiplies for the next one while the last blocks and the output of this one are worked on. S is
+// double-buffered in tensor memory (2 x 128 columns) ahead of the output (256 columns). Two teams of eight warps take the
+// KV blocks in turn, a thread per query row and half of the block's keys; the running maximum passes from one team to the
+// other through shared memory, so that the output has one scale: as above it moves by more than 2^8 only, and then the
+// warps that moved it rescale their rows once the block before is in. Two more warps lay out the bias of a block ahead of
+// its team: its 255 distances in the order of the keys, in four copies shifted by one float each, so that a row reads its
+// own 128 of them as aligned 16-byte words without conflicts.
+// ------------------------------------------------------------------------------------------
+struct BiasedArgs {
+  const TcItem* items;
+  int n_units, heads, group, v_blocks, v_groups, all_values;   // v_groups: pairs of value blocks, a unit each
+  long long t_cap;
+  __nv_bfloat16* out;        // row stride ldo, head stride ho
+  long long ldo, ho;
+  int v_chunks;              // 16-byte chunks of a value block
+  float scale;               // in units of log2
+  const float* table;        // [heads][entries]: entry i is minus the bias (in units of log2) at distance zero - i
+  int entries, zero;
+  const float* sink;         // [heads], or null
+  int window;
+  int* status;
+};
+
+__device__ __forceinline__ void tmem_ld_32x32b_x16(uint32_t taddr, uint32_t (&r)[16]) {
+  asm volatile(
+      "tcgen05.ld.sync.aligned.32x32b.x16.b32 {%0, %1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15}, [%16];"
+      : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]), "=r"(r[8]),
+        "=r"(r[9]), "=r"(r[10]), "=r"(r[11]), "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15])
+      : "r"(taddr)
+      : "memory");
+}
+__device__ __forceinline__ void tmem_st_32x32b_x16(uint32_t taddr, const uint32_t (&r)[16]) {
+  asm volatile(
+      "tcgen05.st.sync.aligned.32x32b.x16.b32 [%0], {%1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15, %16};"
+      ::"r"(taddr), "r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3]), "r"(r[4]), "r"(r[5]), "r"(r[6]), "r"(r[7]), "r"(r[8]),
+        "r"(r[9]), "r"(r[10]), "r"(r[11]), "r"(r[12]), "r"(r[13]), "r"(r[14]), "r"(r[15])
+      : "memory");
+}
+
+struct BiasedSmem {
+  static constexpr int slots = 3;
+  static constexpr int off_q = 0;                       // 2 panels
+  static constexpr int off_p = 2 * kPanel;              // [2 blocks][2 panels]; at a unit's end its output rows
+  static constexpr int off_ring = 6 * kPanel;           // [slots][2 panels]
+  static constexpr int off_bar = off_ring + slots * 2 * kPanel;
+  static constexpr int n_bars = 3 + 2 * slots + 2 * 6;
+  // running maxima after a block of either parity [2][128]; maxima of a block's halves [2 teams][2][128]; row sums of the
+  // four parts at a unit's end
+  static constexpr int off_row = off_bar + 256, off_top = off_row + 1024, off_sum = off_top + 2048;
+  static constexpr int copy = 264;                      // floats from one copy of a block's bias to the next: 8 banks on
+  static constexpr int off_bias = off_sum + 2048;       // [2 blocks][4 copies]
+  static constexpr int bytes = off_bias + 2 * 4 * copy * 4 + 1024;    // + slack to align the base to 1024
+};
+constexpr int kBiasedThreads = 640;     // warps 0-3: TMA / MMA / bias; warps 4-11, 12-19: the teams
+
+struct BiasedUnit {
+  TcItem it;
+  int head, hk, vb0, nv;
+  __device__ __forceinline__ BiasedUnit(const BiasedArgs& a, int u) {
+    const int per_item = a.heads * a.v_groups, i = u / per_item, in_item = u - i * per_item;
+    it = a.items[i];
+    head = in_item / a.v_groups;
+    hk = head / a.group;
+    vb0 = a.all_values ? (in_item - head * a.v_groups) * 2 : hk;
+    nv = a.all_values ? min(2, a.v_blocks - vb0) : 1;
+  }
+};
+
+__global__ void __launch_bounds__(kBiasedThreads, 1)
+attn_prefill_biased_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_constant__ CUtensorMap tma_k,
+                           const __grid_constant__ CUtensorMap tma_v, const BiasedArgs args) {
+  pdl_enter();
+  using T = __nv_bfloat16;
+  using L = BiasedSmem;
+  extern __shared__ uint8_t smem_raw[];
+  const uint32_t raw = smem_u32(smem_raw);
+  const uint32_t s_base = (raw + 1023u) & ~1023u;
+  uint8_t* smem = smem_raw + (s_base - raw);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+
+  const uint32_t q_s = s_base + L::off_q, p_s = s_base + L::off_p, ring = s_base + L::off_ring;
+  auto bar = [&](int i) { return s_base + L::off_bar + 8u * (uint32_t)i; };
+  const uint32_t q_full = bar(0), q_free = bar(1), o_free = bar(2);
+  auto kv_full = [&](int s) { return bar(3 + s); };
+  auto kv_empty = [&](int s) { return bar(3 + L::slots + s); };
+  auto of_block = [&](int kind, int b) { return bar(3 + 2 * L::slots + 2 * kind + b); };
+  auto s_full = [&](int b) { return of_block(0, b); };
+  auto s_free = [&](int b) { return of_block(1, b); };
+  auto p_full = [&](int b) { return of_block(2, b); };
+  auto o_done = [&](int b) { return of_block(3, b); };
+  auto bias_full = [&](int b) { return of_block(4, b); };
+  auto bias_free = [&](int b) { return of_block(5, b); };
+  volatile uint32_t* tmem_slot = reinterpret_cast<volatile uint32_t*>(smem + L::off_bar + 8 * L::n_bars);
+  volatile int* abort_flag = reinterpret_cast<volatile int*>(smem + L::off_bar + 8 * L::n_bars + 8);
+  float* row_m = reinterpret_cast<float*>(smem + L::off_row);
+
+  if (threadIdx.x == 0) {
+    mbar_init(q_full, 1);
+    mbar_init(q_free, 1);
+    mbar_init(o_free, 512);
+    for (int s = 0; s < L::slots; ++s) { mbar_init(kv_full(s), 1); mbar_init(kv_empty(s), 1); }
+    for (int b = 0; b < 2; ++b) {
+      mbar_init(s_full(b), 1);
+      mbar_init(s_free(b), 256);
+      mbar_init(p_full(b), 256);
+      mbar_init(o_done(b), 1);
+      mbar_init(bias_full(b), 64);
+      mbar_init(bias_free(b), 256);
+    }
+    *abort_flag = 0;
+    fence_barrier_init();
+    prefetch_tensormap(&tma_q);
+    prefetch_tensormap(&tma_k);
+    prefetch_tensormap(&tma_v);
+  }
+  if (warp == 1) {
+    tmem_alloc(smem_u32(const_cast<uint32_t*>(tmem_slot)), 512);
+    tmem_relinquish();
+  }
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem_base = *tmem_slot;
+  // Blocks are counted through all units of the CTA: block g has the parity g & 1 in every double buffer and is the
+  // (g >> 1)-th user of it.
+  auto turn = [](int g) { return (uint32_t)((g >> 1) & 1); };
+
+  if (warp < 4) {
+    if (warp == 0 && lane == 0) {
+      // -------------------------------------------------------------- TMA producer, per unit: Q K0 K1 | K2 V0 | K3 V1 | ...
+      int n = 0, k = 0;
+      bool ok = true;
+      auto take_slot = [&]() {
+        const int slot = n % L::slots;
+        ok = ok && mbar_wait(kv_empty(slot), (uint32_t)((n / L::slots & 1) ^ 1), abort_flag, args.status, 231);
+        if (ok) mbar_expect_tx(kv_full(slot), 2 * kPanel);
+        ++n;
+        return slot;
+      };
+      for (int u = blockIdx.x; u < args.n_units && ok; u += gridDim.x, ++k) {
+        const BiasedUnit w(args, u);
+        const int nb = w.it.n_blocks, k_row0 = (int)((long long)w.hk * args.t_cap) + w.it.kv_off;
+        if (k > 0) ok = mbar_wait(q_free, (uint32_t)((k - 1) & 1), abort_flag, args.status, 230);
+        if (!ok) break;
+        mbar_expect_tx(q_full, 2 * kPanel);
+        for (int p = 0; p < 2; ++p) tma_load_3d(q_s + p * kPanel, &tma_q, q_full, 64 * p, w.head, w.it.q_row0);
+        auto load_k = [&](int j) {
+          const int slot = take_slot();
+          for (int p = 0; p < 2 && ok; ++p)
+            tma_load_2d(ring + (slot * 2 + p) * kPanel, &tma_k, kv_full(slot), 64 * p, k_row0 + j * kTile);
+        };
+        for (int j = 0; j < 2 && j < nb && ok; ++j) load_k(j);
+        for (int j = 0; j < nb && ok; ++j) {
+          if (j + 2 < nb) load_k(j + 2);
+          for (int v = 0; v < w.nv && ok; ++v) {
+            const int slot = take_slot();
+            for (int p = 0; p < 2 && ok; ++p)
+              tma_load_2d(ring + (slot * 2 + p) * kPanel, &tma_v, kv_full(slot), w.it.kv_off + j * kTile + 64 * p,
+                          (w.vb0 + v) * kD);
+          }
+        }
+      }
+      if (*abort_flag) {  // let copies that are still in flight land before the CTA exits
+        const uint64_t t0 = globaltimer_ns();
+        while (globaltimer_ns() - t0 < 200000ull) __nanosleep(1000);
+      }
+    } else if (warp == 1 && lane == 0) {
+      // -------------------------------------------------------------- MMA issuer
+      constexpr uint32_t idesc = idesc_dense(TcFmt<T>::fmt, TcFmt<T>::fmt, 128, 128);
+      int n = 0, k = 0, g0 = 0;
+      bool ok = true;
+      auto next_full = [&](int code) {
+        ok = ok && mbar_wait(kv_full(n % L::slots), (uint32_t)(n / L::slots & 1), abort_flag, args.status, code);
+        return ring + (n % L::slots) * 2 * kPanel;
+      };
+      for (int u = blockIdx.x; u < args.n_units && ok; u += gridDim.x, ++k) {
+        const BiasedUnit w(args, u);
+        const int nb = w.it.n_blocks;
+        ok = mbar_wait(q_full, (uint32_t)(k & 1), abort_flag, args.status, 232);
+        auto issue_s = [&](int j) {
+          const int g = g0 + j;
+          if (g > 1) ok = ok && mbar_wait(s_free(g & 1), turn(g - 2), abort_flag, args.status, 234);
+          const uint32_t k_tile = next_full(233);
+          if (!ok) return;
+          tc_fence_after();
+#pragma unroll
+          for (int kk = 0; kk < 8; ++kk)
+            mma_f16(tmem_base + (g & 1) * 128, smem_desc_sw128(q_s + (kk >> 2) * kPanel + (kk & 3) * 32),
+                    smem_desc_sw128(k_tile + (kk >> 2) * kPanel + (kk & 3) * 32), idesc, kk > 0 ? 1u : 0u);
+          tc_commit(s_full(g & 1));
+          tc_commit(kv_empty(n % L::slots));
+          if (j == nb - 1) tc_commit(q_free);
+          ++n;
+        };
+        for (int j = 0; j < 2 && j < nb && ok; ++j) issue_s(j);
+        for (int j = 0; ok && j < nb; ++j) {
+          const int g = g0 + j;
+          if (j + 2 < nb) issue_s(j + 2);
+          // the unit before has read its output
+          if (j == 0 && k > 0) ok = ok && mbar_wait(o_free, (uint32_t)((k - 1) & 1), abort_flag, args.status, 229);
+          ok = ok && mbar_wait(p_full(g & 1), turn(g), abort_flag, args.status, 235);
+          for (int v = 0; v < w.nv && ok; ++v) {
+            const uint32_t v_tile = next_full(236);
+            if (!ok) break;
+            tc_fence_after();
+#pragma unroll
+            for (int kk = 0; kk < 8; ++kk)
+              mma_f16(tmem_base + 256 + v * 128, smem_desc_sw128(p_s + ((g & 1) * 2 + (kk >> 2)) * kPanel + (kk & 3) * 32),
+                      smem_desc_sw128(v_tile + (kk >> 2) * kPanel + (kk & 3) * 32), idesc, (kk > 0 || j > 0) ? 1u : 0u);
+            if (v == w.nv - 1) tc_commit(o_done(g & 1));
+            tc_commit(kv_empty(n % L::slots));
+            ++n;
+          }
+        }
+        g0 += nb;
+      }
+    } else if (warp >= 2) {
+      // -------------------------------------------------------------- bias: entry i of a block is the distance of row r and
+      // key k with i = k - r + 127
+      const int i0 = (threadIdx.x - 64) * 4;
+      int g = 0;
+      bool ok = true;
+      for (int u = blockIdx.x; u < args.n_units; u += gridDim.x) {
+        const BiasedUnit w(args, u);
+        const float* line = args.table + (size_t)w.head * args.entries + args.zero - w.it.q_pos0 - 127 + w.it.kv_pos0 + i0;
+        for (int j = 0; j < w.it.n_blocks; ++j, ++g) {
+          float x[7];
+#pragma unroll
+          for (int i = 0; i < 7; ++i) x[i] = __ldg(line + j * kTile + i);
+          if (g > 1) ok = ok && mbar_wait(bias_free(g & 1), turn(g - 2), abort_flag, args.status, 241);
+          float* dst = reinterpret_cast<float*>(smem + L::off_bias) + (g & 1) * 4 * L::copy + i0;
+#pragma unroll
+          for (int c = 0; c < 4; ++c)
+            *reinterpret_cast<float4*>(dst + c * L::copy) = make_float4(x[c], x[c + 1], x[c + 2], x[c + 3]);
+          mbar_arrive(bias_full(g & 1));
+        }
+      }
+    }
+  } else {
+    // ---------------------------------------------------------------- softmax / output teams
+    const int part = (warp - 4) >> 2, t = part >> 1, half = part & 1, quarter = warp & 3, row = quarter * 32 + lane;
+    const uint32_t lane_base = tmem_base + ((uint32_t)(quarter * 32) << 16);
+    const uint32_t s_addr = lane_base + t * 128 + half * 64, o_addr = lane_base + 256;
+    const uint32_t p_row = p_s + (t * 2 + half) * kPanel + row * 128;
+    const uint32_t swz = (uint32_t)(row & 7);
+    const int first = 127 - row + half * 64;             // the bias entry of this row and half's first key
+    const float4* bias = reinterpret_cast<const float4*>(reinterpret_cast<const float*>(smem + L::off_bias) +
+                                                         (t * 4 + (first & 3)) * L::copy + (first & ~3));
+    const uint64_t scale2 = f2(args.scale, args.scale);
+    float* sums = reinterpret_cast<float*>(smem + L::off_sum);
+    float* top_of = reinterpret_cast<float*>(smem + L::off_top) + t * 256;      // [half][128]
+    uint32_t s[2][32];
+    bool ok = true;
+    int g0 = 0;
+    for (int u = blockIdx.x; u < args.n_units; u += gridDim.x) {
+      const BiasedUnit w(args, u);
+      const int nb = w.it.n_blocks, q_pos = w.it.q_pos0 + row;
+      const int lo = args.window > 0 ? q_pos - args.window : -1;                // last position ahead of the window
+      const int lo_last = args.window > 0 ? w.it.q_pos0 + kTile - 1 - args.window : -1;
+      float m = -INFINITY, l = 0.f;
+      for (int j = (t ^ g0) & 1; j < nb; j += 2) {
+        const int g = g0 + j, kv0 = w.it.kv_pos0 + j * kTile + half * 64;
+        ok = ok && mbar_wait(s_full(t), turn(g), abort_flag, args.status, 237);
+        tc_fence_after();
+        tmem_ld_32x32b_x32(s_addr, s[0]);
+        tmem_ld_32x32b_x32(s_addr + 32, s[1]);
+        tmem_ld_wait();
+        tc_fence_before();
+        mbar_arrive(s_free(t));
+        ok = ok && mbar_wait(bias_full(t), turn(g), abort_flag, args.status, 242);
+        float mx[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
+        const bool cut = kv0 + 63 > w.it.q_pos0 || kv0 <= lo_last;   // the half crosses some row's diagonal or window
+#pragma unroll
+        for (int c = 0; c < 2; ++c) {
+#pragma unroll
+          for (int i = 0; i < 32; i += 4) {
+            const float4 x = bias[c * 8 + (i >> 2)];
+            float x0, x1, x2, x3;
+            unf2(fma2(f2(__uint_as_float(s[c][i]), __uint_as_float(s[c][i + 1])), scale2, f2(x.x, x.y)), x0, x1);
+            unf2(fma2(f2(__uint_as_float(s[c][i + 2]), __uint_as_float(s[c][i + 3])), scale2, f2(x.z, x.w)), x2, x3);
+            s[c][i] = __float_as_uint(x0);
+            s[c][i + 1] = __float_as_uint(x1);
+            s[c][i + 2] = __float_as_uint(x2);
+            s[c][i + 3] = __float_as_uint(x3);
+          }
+          if (cut) {
+#pragma unroll
+            for (int i = 0; i < 32; ++i) {
+              const int tok = kv0 + c * 32 + i;
+              if (tok > q_pos || tok <= lo) s[c][i] = 0xFF800000u;   // -inf
+            }
+          }
+#pragma unroll
+          for (int i = 0; i < 32; ++i) mx[i & 3] = fmaxf(mx[i & 3], __uint_as_float(s[c][i]));
+        }
+        mbar_arrive(bias_free(t));
+        top_of[half * 128 + row] = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3]));
+        // both halves of the block; then the other team's decision on the block before, and this one
+        asm volatile("bar.sync %0, 256;" ::"r"(4 + t) : "memory");
+        const float top = fmaxf(top_of[row], top_of[128 + row]);
+        if (j > 0) asm volatile("bar.sync %0, 512;" ::"r"(3 - t) : "memory");
+        else asm volatile("bar.sync %0, 256;" ::"r"(4 + t) : "memory");        // the maxima have been read, here too
+        const float before = j > 0 ? row_m[(t ^ 1) * 128 + row] : -INFINITY;
+        const bool grow = top - before > 8.f;              // false when both are -inf (NaN compares false)
+        const float now = grow ? top : before;
+        if (half == 0) row_m[t * 128 + row] = now;
+        if (j + 1 < nb) asm volatile("bar.arrive %0, 512;" ::"r"(2 + t) : "memory");
+        if (now != m) {
+          l *= ex2f(m - now);                                // m = -inf: 0
+          m = now;
+        }
+        if (j > 0 && half < w.nv && __any_sync(0xFFFFFFFFu, grow)) {
+          // O may be rescaled when the product of the block before is in; a half takes one value block
+          ok = ok && mbar_wait(o_done(t ^ 1), turn(g - 1), abort_flag, args.status, 238);
+          tc_fence_after();
+          const float alpha = grow ? ex2f(before - now) : 1.f;
+          uint32_t r[16];
+#pragma unroll 1
+          for (int c = 0; c < 8; ++c) {
+            tmem_ld_32x32b_x16(o_addr + half * 128 + c * 16, r);
+            tmem_ld_wait();
+#pragma unroll
+            for (int i = 0; i < 16; ++i) r[i] = __float_as_uint(__uint_as_float(r[i]) * alpha);
+            tmem_st_32x32b_x16(o_addr + half * 128 + c * 16, r);
+          }
+          tmem_st_wait();
+        }
+        // the product two blocks ago is in: this team's P buffer is free
+        if (g > 1) ok = ok && mbar_wait(o_done(t), turn(g - 2), abort_flag, args.status, 239);
+        const float mb = m == -INFINITY ? 0.f : m;
+        const uint64_t mb2 = f2(-mb, -mb);
+        uint64_t sum[2] = {0, 0};
+#pragma unroll
+        for (int c = 0; c < 2; ++c) {
+#pragma unroll
+          for (int gg = 0; gg < 4; ++gg) {
+            uint32_t pk[4];
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+              const int i = gg * 8 + e * 2;
+              float x0, x1;
+              unf2(add2(f2(__uint_as_float(s[c][i]), __uint_as_float(s[c][i + 1])), mb2), x0, x1);
+              x0 = ex2f(x0);
+              x1 = ex2f(x1);
+              sum[e & 1] = add2(sum[e & 1], f2(x0, x1));
+              pk[e] = pack2_tc<T>(x0, x1);
+            }
+            const uint32_t c16 = (uint32_t)(c * 4 + gg);
+            asm volatile("st.shared.v4.b32 [%0], {%1, %2, %3, %4};" ::"r"(p_row + ((c16 ^ swz) << 4)), "r"(pk[0]),
+                         "r"(pk[1]), "r"(pk[2]), "r"(pk[3])
+                         : "memory");
+          }
+        }
+        float l0, l1;
+        unf2(add2(sum[0], sum[1]), l0, l1);
+        l += l0 + l1;
+        tc_fence_before();
+        fence_proxy_async();
+        mbar_arrive(p_full(t));
+      }
+      // ---- sums of all parts on the last scale, the sink, the output: a quarter of the value columns each
+      const int g_last = g0 + nb - 1;
+      asm volatile("bar.sync 1, 512;" ::: "memory");
+      const float last = row_m[(g_last & 1) * 128 + row];
+      sums[part * 128 + row] = l > 0.f ? l * ex2f(m - last) : 0.f;
+      asm volatile("bar.sync 1, 512;" ::: "memory");
+      float sum = sums[row] + sums[128 + row] + sums[256 + row] + sums[384 + row];
+      ok = ok && mbar_wait(o_done(g_last & 1), turn(g_last), abort_flag, args.status, 240);
+      tc_fence_after();
+      if (t < w.nv) {
+#pragma unroll
+        for (int c = 0; c < 2; ++c) tmem_ld_32x32b_x32(o_addr + part * 64 + c * 32, s[c]);
+        tmem_ld_wait();
+      }
+      tc_fence_before();
+      mbar_arrive(o_free);
+      if (ok && t < w.nv) {
+        float num = 1.f;
+        if (args.sink != nullptr) {
+          const float sk = args.sink[w.head] * kLog2eTc, ms = last == -INFINITY ? sk : last, mn = fmaxf(ms, sk);
+          num = ex2f(ms - mn);
+          sum = fmaf(sum, num, ex2f(sk - mn));
+        }
+        const float inv = sum > 0.f ? num / sum : 0.f;
+        // through this warp's own rows of P (all products have read them), so that whole lines leave
+#pragma unroll
+        for (int c = 0; c < 8; ++c) {
+          const uint32_t* o = &s[c >> 2][(c & 3) * 8];
+          asm volatile("st.shared.v4.b32 [%0], {%1, %2, %3, %4};" ::"r"(p_row + (((uint32_t)c ^ swz) << 4)),
+                       "r"(pack2_tc<T>(__uint_as_float(o[0]) * inv, __uint_as_float(o[1]) * inv)),
+                       "r"(pack2_tc<T>(__uint_as_float(o[2]) * inv, __uint_as_float(o[3]) * inv)),
+                       "r"(pack2_tc<T>(__uint_as_float(o[4]) * inv, __uint_as_float(o[5]) * inv)),
+                       "r"(pack2_tc<T>(__uint_as_float(o[6]) * inv, __uint_as_float(o[7]) * inv))
+                       : "memory");
+        }
+        __syncwarp();
+        const int c = lane & 7;
+        T* dst = args.out + w.head * args.ho + (args.all_values ? (w.vb0 + t) * kD : 0) + half * 64 + c * 8;
+        if (half * 8 + c < args.v_chunks) {
+#pragma unroll
+          for (int i = 0; i < 8; ++i) {
+            const int r = quarter * 32 + i * 4 + (lane >> 3);
+            if (r < w.it.q_rows)
+              *reinterpret_cast<uint4*>(dst + (long long)(w.it.q_row0 + r) * args.ldo) = *reinterpret_cast<const uint4*>(
+                  smem + L::off_p + (t * 2 + half) * kPanel + r * 128 + ((c ^ (r & 7)) << 4));
+          }
+        }
+        __syncwarp();
+      }
+      g0 += nb;
+    }
+  }
+  tc_fence_before();
+  __syncthreads();
+  if (warp == 1) tmem_dealloc(tmem_base, 512);
+}
+
 bool encode_map(CUtensorMap* map, const void* base, int rank, const cuuint64_t* dims, const cuuint64_t* strides,
                 const cuuint32_t* box, const char* what) {
   msgl_encode_tiled_fn enc = msgl_get_encode_tiled();
@@ -643,7 +1038,7 @@ int launch_tc(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& m
     if (e != cudaSuccess) { msgl_set_error("prefill attention smem attribute", e); return MSGL_CUDA_ERROR; }
     configured = true;
   }
-  msgl_launch(attn_prefill_tc_kernel<T, POS, MODE>, dim3(a.n_items * a.pairs * (MODE == TC_BIASED && a.v_blocks > 0 ? a.v_blocks : 1)), dim3(kTcThreads), TcSmem::bytes, stream, mq, mk, mv, mg, a);
+  msgl_launch(attn_prefill_tc_kernel<T, POS, MODE>, dim3(a.n_items * a.pairs), dim3(kTcThreads), TcSmem::bytes, stream, mq, mk, mv, mg, a);
   MSGL_CHECK_LAUNCH("attn_prefill_tc");
   return MSGL_OK;
 }
@@ -737,12 +1132,13 @@ MSGL_API int msgl_attn_prefill_tc(const void* q, long long q_row_stride, void* o
                                   const void* block_table, int bt_stride, const void* k_scale, const void* v_scale,
                                   int total_q, int hq, int hk, int d, int page_size, int kv_fp8, float scale,
                                   int window, int chunk, float softcap, const void* gate, long long ldg, const void* bias,
-                                  int reach, const void* sink, int all_values, int pos_form, int dtype,
+                                  int entries, int zero, const void* sink, int all_values, int pos_form, int dtype,
                                   cudaStream_t stream) {
   if (n_items == 0 || total_q == 0) return MSGL_OK;
   if (bias == nullptr ? (all_values || sink != nullptr)
-                      : (reach <= 0 || softcap > 0.f || gate != nullptr || dtype != MSGL_BF16 || kv_fp8)) {
-    msgl_set_error_text("prefill attention: a distance bias stands without soft cap, gate and fp8, sinks and mixed heads with one");
+                      : (entries <= 0 || zero < 0 || softcap > 0.f || chunk > 0 || pos_form ||
+                         gate != nullptr || dtype != MSGL_BF16 || kv_fp8)) {
+    msgl_set_error_text("prefill attention: a distance bias stands without soft cap, chunks, gate and fp8; sinks and mixed heads with one");
     return MSGL_BAD_ARG;
   }
   const bool ext = d != kD || window > 0 || chunk > 0 || softcap > 0.f || gate != nullptr;
@@ -750,7 +1146,7 @@ MSGL_API int msgl_attn_prefill_tc(const void* q, long long q_row_stride, void* o
     msgl_set_error_text("prefill attention: reaches, soft caps, gates, rows of 64 and unpaired query heads need bf16");
     return MSGL_BAD_ARG;
   }
-  if (hq % hk || (!pos_form && (hq / hk) % 2) || (d != 64 && d != 128) || scale <= 0.f || (gate != nullptr && ldg % 8) ||
+  if (hq % hk || (!pos_form && bias == nullptr && (hq / hk) % 2) || (d != 64 && d != 128) || scale <= 0.f || (gate != nullptr && ldg % 8) ||
       (uintptr_t)gate % 16 || t_cap % 128 || t_pad % 128 || t_pad > t_cap || (q_row_stride % 8) ||
       (dtype != MSGL_BF16 && dtype != MSGL_F16)) {
     msgl_set_error_text("prefill attention: needs rows of 64 or 128, pairs of heads or of blocks, 16-bit q, a positive scale "
@@ -805,9 +1201,26 @@ MSGL_API int msgl_attn_prefill_tc(const void* q, long long q_row_stride, void* o
   a.status = status; a.window = window; a.chunk = chunk; a.softcap = softcap; a.cgate = gate != nullptr;
   a.ho = all_values ? v_blocks * kD : d; a.ldo = a.ho * hq; a.v_chunks = all_values ? 16 : d / 8;
   if (bias != nullptr) {
-    a.bias = (const float*)bias; a.reach = reach; a.sink = (const float*)sink; a.v_blocks = all_values ? v_blocks : 0;
-    return pos_form ? launch_tc<__nv_bfloat16, true, TC_BIASED>(mq, mk, mv, mg, a, stream)
-                    : launch_tc<__nv_bfloat16, false, TC_BIASED>(mq, mk, mv, mg, a, stream);
+    static bool configured = false;
+    if (!configured) {
+      cudaError_t e = cudaFuncSetAttribute(attn_prefill_biased_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                           BiasedSmem::bytes);
+      if (e != cudaSuccess) { msgl_set_error("prefill attention smem attribute", e); return MSGL_CUDA_ERROR; }
+      configured = true;
+    }
+    const int v_groups = all_values ? (v_blocks + 1) / 2 : 1, units = n_items * hq * v_groups;
+    static int sms = 0;
+    if (sms == 0) {
+      int dev = 0;
+      cudaGetDevice(&dev);
+      cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
+    }
+    BiasedArgs ba{a.items, units, hq, hq / hk, v_blocks, v_groups, all_values, t_cap, (__nv_bfloat16*)out, a.ldo, a.ho,
+                  a.v_chunks, scale * kLog2eTc, (const float*)bias, entries, zero, (const float*)sink, window, status};
+    msgl_launch(attn_prefill_biased_kernel, dim3(units < sms ? units : sms), dim3(kBiasedThreads), BiasedSmem::bytes, stream, mq,
+                mk, mv, ba);
+    MSGL_CHECK_LAUNCH("attn_prefill_biased");
+    return MSGL_OK;
   }
   const bool fixcap = softcap > 0.f && softcap * kLog2eTc <= kFixedCap && dtype == MSGL_BF16;
   if (pos_form) {

@@ -72,7 +72,7 @@ _SIGNATURES = {
                               + [c_f] + [c_i] * 5 + [c_p]),
     "msgl_attn_status": (c_i, [c_i]),
     "msgl_attn_prefill_tc": (c_i, [c_p, c_ll, c_p, c_p, c_p, c_p, c_p, c_ll, c_i, c_p, c_i, c_p, c_p, c_p, c_i,
-                                   c_p, c_p, c_i, c_i, c_i, c_i, c_i, c_i, c_f, c_i, c_i, c_f, c_p, c_ll, c_p, c_i, c_p, c_i,
+                                   c_p, c_p, c_i, c_i, c_i, c_i, c_i, c_i, c_f, c_i, c_i, c_f, c_p, c_ll, c_p, c_i, c_i, c_p, c_i,
                                    c_i, c_i, c_p]),
     "msgl_attn_tc_status": (c_i, [c_i]),
     "msgl_attn_force_general_decode": (None, [c_i]),

@@ -378,6 +378,24 @@ def _distance_bias(bias, hq):
     return bias.data_ptr(), bias.shape[1]
 
 
+_BIAS_ROWS: Dict[Tuple, Tuple] = {}
+
+
+def _bias_rows(bias):
+    """The table of the prefill kernel: what a score gains at each distance, in units of log2 and in the order of the keys
+    (ever nearer ones), zeros for distances that a block has and no row sees. Returns ``(table [H, entries], entry of
+    distance 0)``."""
+    key = (bias.data_ptr(), tuple(bias.shape), bias.device)
+    hit = _BIAS_ROWS.get(key)
+    if hit is None or hit[0] is not bias:
+        pad = 384                                   # a tile's rows and a block's keys beyond the reach, on either side
+        table = torch.nn.functional.pad((bias * -1.4426950408889634).flip(1), (pad, pad)).contiguous()
+        if len(_BIAS_ROWS) > 512:
+            _BIAS_ROWS.clear()
+        _BIAS_ROWS[key] = hit = (bias, table, pad + bias.shape[1] - 1)
+    return hit[1], hit[2]
+
+
 def _paged_attention_f32(q, k_cache, v_cache, block_table, cu_q, seq_lens, scale, window, chunk, softcap, gate, bias, sink,
                          talk):
     t, hq, d = q.shape
@@ -584,12 +602,13 @@ def prefill_attention_tc(q, k_cache, v_cache, block_table, plan: PrefillPlan, sc
     tb = plan.tables
     base = tb.data_ptr()
     fp8 = k_cache.dtype == torch.float8_e4m3fn
+    rows, zero = (None, 0) if bias is None else _bias_rows(bias)
     check(lib().msgl_attn_prefill_tc(
         _p(q), q.stride(0), _p(out), _p(k_cache), _p(v_cache), _p(kc), _p(vt), cap, plan.t_pad,
         base, plan.n_items, base + 4 * plan.off_blk, base + 4 * plan.off_req, _p(block_table), block_table.stride(0),
         _p(k_scale), _p(v_scale), t, hq, hk, d, ps, int(fp8), float(scale), int(window), int(chunk), float(softcap),
-        *_output_gate(gate, q), *_distance_bias(bias, hq), _p(sink), int(talk is not None), int(plan.tile == 256), _dt(q),
-        _stream()), "attn_prefill_tc")
+        *_output_gate(gate, q), _p(rows), 0 if rows is None else rows.shape[1], zero, _p(sink), int(talk is not None),
+        int(plan.tile == 256), _dt(q), _stream()), "attn_prefill_tc")
     _count("prefill_attention", "attn_prefill_tc_kernel", 2)
     return out if talk is None else head_mix(out, talk, hk, d)
 

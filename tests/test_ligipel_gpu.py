@@ -202,7 +202,7 @@ def test_prompts_of_mixed_heads(hq, hk, width, window):
     q, k, v, scale = q.to(BF), k.to(BF), v.to(BF), 1.5 * width ** -0.5
     want = ref.paged_attention(q.float(), k.float(), v.float(), bt, cu, seq, scale, window=window, bias=bias, sink=sink, talk=talk)
     kg, vg = U.split_planes(k.to(DEV), v.to(DEV))
-    plan = K.PrefillPlan(cu.numpy(), seq.numpy(), DEV, window, tile=256 if hq // hk % 2 else 128)
+    plan = K.PrefillPlan(cu.numpy(), seq.numpy(), DEV, window)
     got = K.prefill_attention_tc(q.to(DEV), kg, vg, bt.to(DEV), plan, scale, window=window,
                                  **dict(zip(("bias", "sink", "talk"), _dev(bias, sink, talk))))
     torch.testing.assert_close(got.float().cpu(), want, rtol=3e-2, atol=3e-2 * float(want.pow(2).mean().sqrt() + 1))
@@ -286,7 +286,7 @@ def test_engine_portions_batches_and_reuse(model, dtype):
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 @pytest.mark.parametrize("cfg", [
-    U.config([U.pair(1, 1, 4, 5, 3, inner=6, state=2, rank=1, taps=2), U.retention(1, 6, 5), U.retention(2, 4, 3, rot=2)], width=20,
+    U.config([U.pair(1, 1, 4, 5, 3, inner=6, state=2, rank=1, taps=2), U.retention(1, 6, 5), U.retention(2, 4, 3, rot=2)], width=40,
              vocab=7, scale=1.0, cap=30.0),
     U.config([U.pair(7, 7, 130, 150, 300, inner=200, state=70, rank=40, taps=2), U.retention(2, 70, 130, rot=64)], width=40,
              vocab=64),
