@@ -111,8 +111,18 @@ __global__ void __launch_bounds__(kKeys) paged_attention_f32_kernel(const F32Att
   }
 }
 
-// o [rows, H, width] with value head c at columns c * D on; out [rows, H, D]. A thread sums eight channels for up to eight
-// heads of one value head, so that the rows are read once per eight heads: grid (rows * Hk * D / 8 / 128, parts of a group).
+__device__ __forceinline__ void store4(float* p, const float (&x)[4]) {
+  *reinterpret_cast<float4*>(p) = make_float4(x[0], x[1], x[2], x[3]);
+}
+__device__ __forceinline__ void store4(__nv_bfloat16* p, const float (&x)[4]) {
+  uint2 q;
+  *reinterpret_cast<__nv_bfloat162*>(&q.x) = __floats2bfloat162_rn(x[0], x[1]);
+  *reinterpret_cast<__nv_bfloat162*>(&q.y) = __floats2bfloat162_rn(x[2], x[3]);
+  *reinterpret_cast<uint2*>(p) = q;
+}
+
+// o [rows, H, width] with value head c at columns c * D on; out [rows, H, D]. A thread sums four channels for up to eight
+// heads of one value head, so that the rows are read once per eight heads: grid (rows * Hk * D / 4 / 128, parts of a group).
 template <typename T>
 __global__ void __launch_bounds__(128) head_mix_kernel(const T* __restrict__ o, const float* __restrict__ talk,
                                                        T* __restrict__ out, int rows, int H, int Hk, int D, int width) {
@@ -124,28 +134,30 @@ __global__ void __launch_bounds__(128) head_mix_kernel(const T* __restrict__ o, 
     mix[i] = k < n ? talk[(size_t)(c * group + h0 + k) * H + g] : 0.f;
   }
   __syncthreads();
-  const int per_row = Hk * D / 8;
+  const int per_row = Hk * D / 4;
   const long long id = (long long)blockIdx.x * 128 + threadIdx.x;
-  const int row = (int)(id / per_row), col = (int)(id - (long long)row * per_row) * 8, c = col / D;
+  const int row = (int)(id / per_row), col = (int)(id - (long long)row * per_row) * 4, c = col / D;
   if (row >= rows) return;
   const T* src = o + (size_t)row * H * width + col;
   const float* w = mix + (size_t)c * H * 8;
-  float acc[8][8] = {};
+  float acc[8][4] = {};
 #pragma unroll 8
   for (int g = 0; g < H; ++g) {
-    float x[8];
-    load8(src + (size_t)g * width, x);
+    const float4 x = load4f(src + (size_t)g * width);
     const float4 f0 = *reinterpret_cast<const float4*>(w + g * 8), f1 = *reinterpret_cast<const float4*>(w + g * 8 + 4);
     const float f[8] = {f0.x, f0.y, f0.z, f0.w, f1.x, f1.y, f1.z, f1.w};
 #pragma unroll
-    for (int k = 0; k < 8; ++k)
-#pragma unroll
-      for (int e = 0; e < 8; ++e) acc[k][e] = fmaf(f[k], x[e], acc[k][e]);
+    for (int k = 0; k < 8; ++k) {
+      acc[k][0] = fmaf(f[k], x.x, acc[k][0]);
+      acc[k][1] = fmaf(f[k], x.y, acc[k][1]);
+      acc[k][2] = fmaf(f[k], x.z, acc[k][2]);
+      acc[k][3] = fmaf(f[k], x.w, acc[k][3]);
+    }
   }
   T* dst = out + ((size_t)row * H + c * group + h0) * D + col % D;
 #pragma unroll
   for (int k = 0; k < 8; ++k)
-    if (k < n) store8(dst + (size_t)k * D, acc[k]);
+    if (k < n) store4(dst + (size_t)k * D, acc[k]);
 }
 
 }  // namespace
@@ -184,7 +196,7 @@ MSGL_API int msgl_head_mix(const void* o, const void* talk, void* out, int rows,
     msgl_set_error_text("head_mix: widths in eights, up to 6400 pairs of a query and a key / value head");
     return MSGL_BAD_ARG;
   }
-  const long long threads = (long long)rows * hk * d / 8;
+  const long long threads = (long long)rows * hk * d / 4;
   const dim3 grid((unsigned)((threads + 127) / 128), (h / hk + 7) / 8);
 #define HEAD_MIX(T)                                                                                                     \
   do {                                                                                                                  \

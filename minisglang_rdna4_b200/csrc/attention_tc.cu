@@ -749,11 +749,12 @@ attn_prefill_biased_kernel(const __grid_constant__ CUtensorMap tma_q, const __gr
         for (int j = 0; j < 2 && j < nb && ok; ++j) load_k(j);
         for (int j = 0; j < nb && ok; ++j) {
           if (j + 2 < nb) load_k(j + 2);
+          // two value blocks: a slot has 64 keys of both, one operand of 256 rows; one block: its 128 keys
           for (int v = 0; v < w.nv && ok; ++v) {
             const int slot = take_slot();
             for (int p = 0; p < 2 && ok; ++p)
-              tma_load_2d(ring + (slot * 2 + p) * kPanel, &tma_v, kv_full(slot), w.it.kv_off + j * kTile + 64 * p,
-                          (w.vb0 + v) * kD);
+              tma_load_2d(ring + (slot * 2 + p) * kPanel, &tma_v, kv_full(slot),
+                          w.it.kv_off + j * kTile + 64 * (w.nv == 2 ? v : p), (w.vb0 + (w.nv == 2 ? p : 0)) * kD);
           }
         }
       }
@@ -764,6 +765,7 @@ attn_prefill_biased_kernel(const __grid_constant__ CUtensorMap tma_q, const __gr
     } else if (warp == 1 && lane == 0) {
       // -------------------------------------------------------------- MMA issuer
       constexpr uint32_t idesc = idesc_dense(TcFmt<T>::fmt, TcFmt<T>::fmt, 128, 128);
+      constexpr uint32_t idesc2 = idesc_dense(TcFmt<T>::fmt, TcFmt<T>::fmt, 128, 256);
       int n = 0, k = 0, g0 = 0;
       bool ok = true;
       auto next_full = [&](int code) {
@@ -800,10 +802,18 @@ attn_prefill_biased_kernel(const __grid_constant__ CUtensorMap tma_q, const __gr
             const uint32_t v_tile = next_full(236);
             if (!ok) break;
             tc_fence_after();
+            const uint32_t p_tile = p_s + (g & 1) * 2 * kPanel;
+            if (w.nv == 2) {
 #pragma unroll
-            for (int kk = 0; kk < 8; ++kk)
-              mma_f16(tmem_base + 256 + v * 128, smem_desc_sw128(p_s + ((g & 1) * 2 + (kk >> 2)) * kPanel + (kk & 3) * 32),
-                      smem_desc_sw128(v_tile + (kk >> 2) * kPanel + (kk & 3) * 32), idesc, (kk > 0 || j > 0) ? 1u : 0u);
+              for (int kk = 0; kk < 4; ++kk)
+                mma_f16(tmem_base + 256, smem_desc_sw128(p_tile + v * kPanel + kk * 32), smem_desc_sw128(v_tile + kk * 32),
+                        idesc2, (v > 0 || kk > 0 || j > 0) ? 1u : 0u);
+            } else {
+#pragma unroll
+              for (int kk = 0; kk < 8; ++kk)
+                mma_f16(tmem_base + 256, smem_desc_sw128(p_tile + (kk >> 2) * kPanel + (kk & 3) * 32),
+                        smem_desc_sw128(v_tile + (kk >> 2) * kPanel + (kk & 3) * 32), idesc, (kk > 0 || j > 0) ? 1u : 0u);
+            }
             if (v == w.nv - 1) tc_commit(o_done(g & 1));
             tc_commit(kv_empty(n % L::slots));
             ++n;
@@ -906,11 +916,12 @@ attn_prefill_biased_kernel(const __grid_constant__ CUtensorMap tma_q, const __gr
           l *= ex2f(m - now);                                // m = -inf: 0
           m = now;
         }
-        if (j > 0 && half < w.nv && __any_sync(0xFFFFFFFFu, grow)) {
+        // (rows that have seen nothing yet have nothing to rescale)
+        if (j > 0 && half < w.nv && __any_sync(0xFFFFFFFFu, grow && before != -INFINITY)) {
           // O may be rescaled when the product of the block before is in; a half takes one value block
           ok = ok && mbar_wait(o_done(t ^ 1), turn(g - 1), abort_flag, args.status, 238);
           tc_fence_after();
-          const float alpha = grow ? ex2f(before - now) : 1.f;
+          const float alpha = grow && before != -INFINITY ? ex2f(before - now) : 1.f;
           uint32_t r[16];
 #pragma unroll 1
           for (int c = 0; c < 8; ++c) {
