@@ -16,7 +16,7 @@ from ..models.config import (
 SIZES = {
     "small": dict(width=2048, heads=16, kv_heads=2, dim=128, window=1024, inner=4096, state=16, rank=128, rheads=8, rdim=128,
                   rvdim=256, experts=32, top=4, eff=768, layers=8, vocab=32768),
-    "large": dict(width=4096, heads=32, kv_heads=4, dim=128, window=1024, inner=8192, state=16, rank=256, rheads=16, rdim=128,
+    "large": dict(width=4096, heads=32, kv_heads=2, dim=128, window=1024, inner=8192, state=16, rank=256, rheads=16, rdim=128,
                   rvdim=256, experts=32, top=4, eff=1536, layers=8, vocab=32768),
 }
 MAX_POS = 4096

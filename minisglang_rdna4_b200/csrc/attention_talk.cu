@@ -6,8 +6,9 @@
 // weights of every head meet the values of every key / value head, and the mixture is taken at the end, when the softmax
 // denominators are known. Per block of 64 keys eight consumer warps take three steps: S^T = K Q^T with the keys on the
 // 16-row side of the warp MMA and the heads of a group on the 8-column side; softmax, a warp per row; O += P V with the
-// heads on the 16-row side, a warp per slice of value columns. A producer warp streams the block's K tiles, then its V
-// tiles, through a ring of shared-memory slots with TMA. Ranges are merged, and heads mixed, by talk_merge_kernel.
+// heads on the 16-row side, a warp per slice of value columns. Two producer warps stream the block's K tiles, then its V
+// tiles, through a ring of shared-memory slots with 16-byte asynchronous copies (a TMA box ends at a page and at 128 bytes,
+// and issuing so many small ones takes longer than the copies). Ranges are merged, and heads mixed, by talk_merge_kernel.
 #include "common.cuh"
 #include "ptx.cuh"
 
@@ -18,6 +19,7 @@ namespace {
 
 constexpr int TK = 64;            // keys per block
 constexpr int kWarps = 8;         // consumer warps
+constexpr int kCopyThreads = 64;
 constexpr float kLog2e = 1.4426950408889634f;
 using bf = __nv_bfloat16;
 
@@ -25,6 +27,8 @@ __device__ int g_talk_status = 0;
 
 struct TalkArgs {
   const bf* q;              // [rows, H, D]
+  const bf* k;              // [pages, Hk, page_size, D]
+  const bf* v;
   bf* out;                  // [rows, H, D]
   const int32_t* block_table;
   const int32_t* cu_q;
@@ -33,7 +37,7 @@ struct TalkArgs {
   const float* sink;        // [H], or null
   const float* talk;        // [H, H]
   float* ws;                // splits > 1: O [splits][rows][H][Hk * D], then m and l [splits][rows][H]
-  int bt_stride, B, rows, H, Hk, page_size, num_pages, reach, window, splits, k_coord, v_coord, decode;
+  int bt_stride, B, rows, H, Hk, page_size, num_pages, reach, window, splits, decode;
   float scale;
   int* status;
 };
@@ -69,7 +73,8 @@ template <int D, int MT, int GN> struct TalkSmem {
   static constexpr int off_row = off_p + rows * ldp * 2;                 // alpha, m, l: [rows] each
   static constexpr int off_bar = off_row + rows * 12;
   static constexpr int off_ring = (off_bar + 512 + 1023) / 1024 * 1024;
-  static constexpr int fit = (225 * 1024 - off_ring) / slot;
+  static constexpr int per_sm = MT * GN * (D / 64) <= 8 ? 2 : 1;         // CTAs that fit an SM (registers, too)
+  static constexpr int fit = (226 * 1024 / per_sm - 1024 - off_ring - 1024) / slot;
   static constexpr int slots = fit < 24 ? fit : 24;
   static constexpr int bytes = off_ring + slots * slot + 1024;
   // the end of a row that is not split: O of all heads in place of the ring
@@ -77,8 +82,7 @@ template <int D, int MT, int GN> struct TalkSmem {
 };
 
 template <int D, int MT, int GN>
-__global__ void __launch_bounds__(kWarps * 32 + 32, 1) talk_decode_kernel(const __grid_constant__ CUtensorMap kv_map,
-                                                                       const TalkArgs a) {
+__global__ void __launch_bounds__(kWarps * 32 + kCopyThreads, TalkSmem<D, MT, GN>::per_sm) talk_decode_kernel(const TalkArgs a) {
   using L = TalkSmem<D, MT, GN>;
   constexpr int CW = D / 16, VG = kWarps / CW;       // column slices of 16; groups of warps on different value heads
   constexpr int GW = GN / VG > 0 ? GN / VG : 1;      // value heads per warp
@@ -111,51 +115,56 @@ __global__ void __launch_bounds__(kWarps * 32 + 32, 1) talk_decode_kernel(const 
 
   if (threadIdx.x == 0) {
     for (int s = 0; s < L::slots; ++s) {
-      mbar_init(full(s), 1);
+      mbar_init(full(s), kCopyThreads);
       mbar_init(empty(s), kWarps);
     }
     *abort_flag = 0;
     fence_barrier_init();
-    prefetch_tensormap(&kv_map);
   }
   __syncthreads();
 
-  if (warp == kWarps) {
-    // ------------------------------------------------------------------ producer
+  if (warp >= kWarps) {
+    // ------------------------------------------------------------------ producers
     // Tables and keys of earlier steps may be read before the kernel ahead has finished; only the blocks with this step's
-    // own rows wait for it.
-    if (lane == 0) {
-      const int32_t* bt = a.block_table + (size_t)b * a.bt_stride;
-      const int pages = TK / a.page_size, newest = max(kv_len - (q_hi - q_lo), 0) / TK;
-      bool waited = false;
-      int slot = 0;
-      uint32_t phase = 1;
-      for (int t = 0; t < n_tiles && !*abort_flag; ++t) {
-        if (!waited && t0 + t >= newest) {
-          pdl_wait();
-          waited = true;
-        }
-        for (int i = 0; i < Hk + nv; ++i) {
-          const int h = i < Hk ? i : c0 + i - Hk;
-          if (!mbar_wait(empty(slot), phase, abort_flag, a.status, 221)) break;
-          mbar_expect_tx(full(slot), L::slot);
-          for (int p = 0; p < pages; ++p) {
-            int page = bt[min((t0 + t) * pages + p, a.bt_stride - 1)];
-            (void)MSGL_OOB(page, a.num_pages + 1);
-            page = page < 0 ? 0 : (page > a.num_pages ? a.num_pages : page);
+    // own rows wait for it. A thread copies one 16-byte column of every ROWS-th token.
+    constexpr int CH = D / 8, ROWS = kCopyThreads / CH, N = TK / ROWS;
+    const int32_t* bt = a.block_table + (size_t)b * a.bt_stride;
+    const int ps = a.page_size, pages = TK / ps, newest = max(kv_len - (q_hi - q_lo), 0) / TK;
+    const int id = threadIdx.x - kWarps * 32, c = id % CH, r0 = id / CH;
+    bool waited = false, ok = true;
+    int slot = 0;
+    uint32_t phase = 1;
+    for (int t = 0; t < n_tiles && ok; ++t) {
+      int page = bt[min((t0 + t) * pages + lane % pages, a.bt_stride - 1)];
+      (void)MSGL_OOB(page, a.num_pages + 1);
+      page = page < 0 ? 0 : (page > a.num_pages ? a.num_pages : page);
+      int from[N];                 // row of head 0 in the pool
 #pragma unroll
-            for (int pl = 0; pl < D / 64; ++pl)
-              tma_load_5d(ring + slot * L::slot + pl * TK * 128 + p * a.page_size * 128, &kv_map, full(slot), pl * 64, 0, h,
-                          page, i < Hk ? a.k_coord : a.v_coord);
-          }
-          if (++slot == L::slots) { slot = 0; phase ^= 1u; }
-        }
+      for (int i = 0; i < N; ++i) {
+        const int tok = r0 + i * ROWS, p = tok / ps;
+        from[i] = __shfl_sync(0xffffffffu, page, p) * Hk * ps + tok - p * ps;
       }
-      if (*abort_flag) {          // let copies that are still in flight land before the CTA exits
-        const uint64_t t_end = globaltimer_ns();
-        while (globaltimer_ns() - t_end < 200000ull) __nanosleep(1000);
+      if (!waited && t0 + t >= newest) {
+        pdl_wait();
+        waited = true;
+      }
+      for (int i = 0; i < Hk + nv && ok; ++i) {
+        const int h = i < Hk ? i : c0 + i - Hk;
+        const bf* src = (i < Hk ? a.k : a.v) + c * 8;
+        ok = mbar_wait(empty(slot), phase, abort_flag, a.status, 221);
+        if (!ok) break;
+        const uint32_t dst = ring + slot * L::slot + (c >> 3) * TK * 128;
+#pragma unroll
+        for (int k = 0; k < N; ++k) {
+          const int tok = r0 + k * ROWS;
+          asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst + tok * 128 + (((c & 7) ^ (tok & 7)) << 4)),
+                       "l"(src + (size_t)(from[k] + h * ps) * D) : "memory");
+        }
+        asm volatile("cp.async.mbarrier.arrive.noinc.shared::cta.b64 [%0];" ::"r"(full(slot)) : "memory");
+        if (++slot == L::slots) { slot = 0; phase ^= 1u; }
       }
     }
+    asm volatile("cp.async.wait_all;" ::: "memory");
     return;
   }
 
@@ -197,9 +206,22 @@ __global__ void __launch_bounds__(kWarps * 32 + 32, 1) talk_decode_kernel(const 
     const int tok0 = (t0 + t) * TK;
     // ---- S^T = K Q^T, scaled, less the bias, in units of log2
     for (int c = 0; c < Hk; ++c) {
+      const int nb0 = (half + c) & 1;
+      // the bias of the first column block, ahead of its keys
+      float bias[4] = {};
+      auto load_bias = [&](int nb) {
+        if (a.bias == nullptr) return;
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int h = min(c * gs + nb * 8 + 2 * j + (e & 1), H - 1), far = pos - tok0 - mt * 16 - r8 - (e >> 1) * 8;
+          bias[e] = __ldg(a.bias + (size_t)h * a.reach + min(max(far, 0), a.reach - 1));
+        }
+      };
+      if (nb0 < nblk) load_bias(nb0);
       ok = ok && mbar_wait(full(slot), phase, abort_flag, a.status, 222);
       const uint32_t k_s = ring + slot * L::slot;
-      for (int nb = (half + c) & 1; nb < nblk; nb += 2) {
+      for (int nb = nb0; nb < nblk; nb += 2) {
+        if (nb > nb0) load_bias(nb);
         float s[4] = {};
         const int trow = mt * 16 + (lane & 15);
         const uint32_t k_row = k_s + trow * 128, q_row = base + L::off_q + min(c * gs + nb * 8 + (lane & 7), L::rows - 1) * L::ldq;
@@ -219,9 +241,7 @@ __global__ void __launch_bounds__(kWarps * 32 + 32, 1) talk_decode_kernel(const 
         for (int e = 0; e < 4; ++e) {
           const int k = nb * 8 + 2 * j + (e & 1), h = c * gs + k, key = mt * 16 + r8 + (e >> 1) * 8, tok = tok0 + key;
           if (k < gs) {
-            float v = s[e] * a.scale;
-            if (a.bias != nullptr) v -= __ldg(a.bias + (size_t)h * a.reach + min(max(pos - tok, 0), a.reach - 1));
-            S[h * L::lds + key] = tok > pos || tok < lo ? -INFINITY : v * kLog2e;
+            S[h * L::lds + key] = tok > pos || tok < lo ? -INFINITY : fmaf(s[e], a.scale, -bias[e]) * kLog2e;
           }
         }
       }
@@ -372,51 +392,82 @@ __global__ void __launch_bounds__(kWarps * 32 + 32, 1) talk_decode_kernel(const 
   }
 }
 
-// Merge of the ranges and mixture of the heads: grid (rows, Hk, parts of the group), 128 threads; a thread sums D / 128
-// channels (a half of them idle at D = 64) for eight heads at a time.
+// Merge of the ranges and mixture of the heads: grid (rows, Hk, parts of the group), a warp per query head in turn (four
+// channels per lane; two heads at a time at D = 64), eight mixed heads in its registers, summed over the warps at the end.
 template <int D>
-__global__ void __launch_bounds__(D) talk_merge_kernel(const TalkArgs a) {
+__global__ void __launch_bounds__(256) talk_merge_kernel(const TalkArgs a) {
   pdl_enter();
-  extern __shared__ float sm[];              // weight of (split, head): [splits][H]; then talk rows [8][H]
+  extern __shared__ float sm[];              // weight of (split, head): [splits][H]; talk rows [H][8]; sums [8 warps][8][D]
+  constexpr int PER = 128 / D;               // heads side by side in a warp
   const int row = blockIdx.x, c = blockIdx.y, H = a.H, gs = H / a.Hk, h0 = blockIdx.z * 8, n = min(8, gs - h0);
-  const size_t rh = (size_t)a.rows * H;
-  const float* tm = a.ws + a.splits * rh * a.Hk * D + (size_t)row * H;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const size_t rh = (size_t)a.rows * H, plane = rh * a.Hk * D;
+  const float* tm = a.ws + a.splits * plane + (size_t)row * H;
   const float* tl = tm + a.splits * rh;
-  float* talk = sm + a.splits * H;
-  for (int h = threadIdx.x; h < H; h += D) {
-    float mx = a.sink != nullptr ? a.sink[h] * kLog2e : -INFINITY;
-    const float floor_ = mx;
+  float* talk = sm + (a.splits * H + 3) / 4 * 4;
+  float* part = talk + H * 8;
+  for (int h = tid; h < H; h += 256) {
+    const float floor_ = a.sink != nullptr ? a.sink[h] * kLog2e : -INFINITY;
+    float mx = floor_;
     for (int s = 0; s < a.splits; ++s) mx = fmaxf(mx, tm[s * rh + h]);
     float den = a.sink != nullptr ? ex2f(floor_ - mx) : 0.f;
     for (int s = 0; s < a.splits; ++s) {
       const float ms = tm[s * rh + h], w = ms == -INFINITY ? 0.f : ex2f(ms - mx);
       sm[s * H + h] = w;
-      if (w > 0.f) den = fmaf(w, tl[s * rh + h], den);
+      if (ms != -INFINITY) den = fmaf(w, tl[s * rh + h], den);
     }
     const float inv = den > 0.f ? 1.f / den : 0.f;
     for (int s = 0; s < a.splits; ++s) sm[s * H + h] *= inv;
   }
-  for (int i = threadIdx.x; i < n * H; i += D) talk[i] = a.talk[(size_t)(c * gs + h0) * H + i];
+  for (int i = tid; i < H * 8; i += 256) {
+    const int g = i >> 3, k = i & 7;
+    talk[i] = k < n ? a.talk[(size_t)(c * gs + h0 + k) * H + g] : 0.f;
+  }
+  // ranges with keys come first; the others have written nothing but their maximum
+  int used = 0;
+  for (int s = 0; s < a.splits; ++s) used += tm[s * rh] != -INFINITY;
   __syncthreads();
-  const int d = threadIdx.x;
-  float acc[8] = {};
-  for (int g = 0; g < H; ++g) {
-    float x = 0.f;
+  const int d = lane * 4 % D;
+  float acc[8][4] = {};
+  for (int g = warp * PER + lane * 4 / D; g < H; g += 8 * PER) {
+    float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
     const float* src = a.ws + (((size_t)row * H + g) * a.Hk + c) * D + d;
 #pragma unroll 4
-    for (int s = 0; s < a.splits; ++s) {
+    for (int s = 0; s < used; ++s) {
       const float w = sm[s * H + g];
-      if (w != 0.f) x = fmaf(w, src[s * rh * a.Hk * D], x);
+      const float4 y = *reinterpret_cast<const float4*>(src + s * plane);
+      x.x = fmaf(w, y.x, x.x);
+      x.y = fmaf(w, y.y, x.y);
+      x.z = fmaf(w, y.z, x.z);
+      x.w = fmaf(w, y.w, x.w);
     }
 #pragma unroll
-    for (int k = 0; k < 8; ++k) acc[k] = k < n ? fmaf(talk[k * H + g], x, acc[k]) : 0.f;
+    for (int k = 0; k < 8; ++k) {
+      const float f = talk[g * 8 + k];
+      acc[k][0] = fmaf(f, x.x, acc[k][0]);
+      acc[k][1] = fmaf(f, x.y, acc[k][1]);
+      acc[k][2] = fmaf(f, x.z, acc[k][2]);
+      acc[k][3] = fmaf(f, x.w, acc[k][3]);
+    }
   }
 #pragma unroll
-  for (int k = 0; k < 8; ++k)
-    if (k < n) a.out[((size_t)row * H + c * gs + h0 + k) * D + d] = __float2bfloat16(acc[k]);
+  for (int k = 0; k < 8; ++k) {
+    if (PER == 2)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) acc[k][e] += __shfl_xor_sync(0xffffffffu, acc[k][e], 16);
+    if (PER == 1 || lane < 16)
+      *reinterpret_cast<float4*>(part + (warp * 8 + k) * D + d) = make_float4(acc[k][0], acc[k][1], acc[k][2], acc[k][3]);
+  }
+  __syncthreads();
+  for (int i = tid; i < n * D; i += 256) {
+    float x = 0.f;
+#pragma unroll
+    for (int w = 0; w < 8; ++w) x += part[w * 8 * D + i];
+    a.out[((size_t)row * H + c * gs + h0) * D + i] = __float2bfloat16(x);
+  }
 }
 
-template <int D, int MT, int GN> int launch_talk(const CUtensorMap& map, const TalkArgs& a, cudaStream_t s) {
+template <int D, int MT, int GN> int launch_talk(const TalkArgs& a, cudaStream_t s) {
   using L = TalkSmem<D, MT, GN>;
   static bool set = false;
   if (!set) {
@@ -425,27 +476,27 @@ template <int D, int MT, int GN> int launch_talk(const CUtensorMap& map, const T
     if (e != cudaSuccess) { msgl_set_error("talk attention smem", e); return MSGL_CUDA_ERROR; }
     set = true;
   }
-  msgl_launch(talk_decode_kernel<D, MT, GN>, dim3(a.splits, (a.Hk + GN - 1) / GN, a.rows), dim3(kWarps * 32 + 32), L::bytes, s,
-              map, a);
+  msgl_launch(talk_decode_kernel<D, MT, GN>, dim3(a.splits, (a.Hk + GN - 1) / GN, a.rows),
+              dim3(kWarps * 32 + kCopyThreads), L::bytes, s, a);
   MSGL_CHECK_LAUNCH("talk_decode");
   if (a.splits > 1) {
-    const size_t smem = (size_t)(a.splits + 8) * a.H * 4;
-    msgl_launch(talk_merge_kernel<D>, dim3(a.rows, a.Hk, (a.H / a.Hk + 7) / 8), dim3(D), smem, s, a);
+    const size_t smem = ((size_t)(a.splits * a.H + 3) / 4 * 4 + 8 * a.H + 64 * D) * 4;      // 48 KiB at the most
+    msgl_launch(talk_merge_kernel<D>, dim3(a.rows, a.Hk, (a.H / a.Hk + 7) / 8), dim3(256), smem, s, a);
     MSGL_CHECK_LAUNCH("talk_merge");
   }
   return MSGL_OK;
 }
 
-template <int D> int dispatch_talk(const CUtensorMap& map, const TalkArgs& a, cudaStream_t s) {
+template <int D> int dispatch_talk(const TalkArgs& a, cudaStream_t s) {
   const int mt = a.H <= 16 ? 1 : a.H <= 32 ? 2 : 4;
   if (a.Hk <= 2) {
-    if (mt == 1) return launch_talk<D, 1, 2>(map, a, s);
-    if (mt == 2) return launch_talk<D, 2, 2>(map, a, s);
-    return launch_talk<D, 4, 2>(map, a, s);
+    if (mt == 1) return launch_talk<D, 1, 2>(a, s);
+    if (mt == 2) return launch_talk<D, 2, 2>(a, s);
+    return launch_talk<D, 4, 2>(a, s);
   }
-  if (mt == 1) return launch_talk<D, 1, 4>(map, a, s);
-  if (mt == 2) return launch_talk<D, 2, 4>(map, a, s);
-  return launch_talk<D, 4, D == 64 ? 4 : 2>(map, a, s);
+  if (mt == 1) return launch_talk<D, 1, 4>(a, s);
+  if (mt == 2) return launch_talk<D, 2, 4>(a, s);
+  return launch_talk<D, 4, D == 64 ? 4 : 2>(a, s);
 }
 
 }  // namespace
@@ -455,27 +506,24 @@ MSGL_API long long msgl_talk_workspace_floats(int rows, int h, int hk, int d, in
   return (long long)splits * rows * h * ((long long)hk * d + 2);
 }
 
-// q, out [rows, h, d] bf16 (d 64 or 128, up to 64 heads); kv_map: msgl_attn_make_kv_map's of the pool buffer. decode: row i is
-// request i. bias [h, reach] fp32 or null; sink [h] or null; talk [h, h].
-MSGL_API int msgl_talk_attention(const void* kv_map, const void* q, void* out, const void* block_table, int bt_stride,
-                                 const void* cu_q, const void* seq_lens, const void* bias, int reach, const void* sink,
+// q, out [rows, h, d] bf16 (d 64 or 128, up to 64 heads); k, v [pages, hk, page_size, d]. decode: row i is request i. bias [h, reach] fp32 or null; sink [h] or null; talk [h, h].
+MSGL_API int msgl_talk_attention(const void* k, const void* v, const void* q, void* out, const void* block_table,
+                                 int bt_stride, const void* cu_q, const void* seq_lens, const void* bias, int reach, const void* sink,
                                  const void* talk, void* workspace, int B, int rows, int h, int hk, int d, int page_size,
-                                 int num_pages, int layer, int layers, int window, int splits, int decode, float scale,
-                                 cudaStream_t stream) {
+                                 int num_pages, int window, int splits, int decode, float scale, cudaStream_t stream) {
   if (B == 0 || rows == 0) return MSGL_OK;
   if (hk <= 0 || h % hk || h > 64 || (d != 64 && d != 128) || page_size < 8 || TK % page_size || bt_stride < 1 ||
-      (bias != nullptr && reach <= 0) || talk == nullptr || splits < 1 || splits > 32 || rows > 65535 ||
+      (bias != nullptr && reach <= 0) || talk == nullptr || splits < 1 || splits > 16 || rows > 65535 || (uintptr_t)k % 16 || (uintptr_t)v % 16 || (uintptr_t)q % 16 ||
       (splits > 1 && workspace == nullptr) || (decode && rows > B)) {
     msgl_set_error_text("talk attention: rows of 64 or 128, up to 64 heads, pages of 8 to 64");
     return MSGL_BAD_ARG;
   }
   int* status = nullptr;
   cudaGetSymbolAddress((void**)&status, g_talk_status);
-  TalkArgs a{(const bf*)q, (bf*)out, (const int32_t*)block_table, (const int32_t*)cu_q, (const int32_t*)seq_lens,
+  TalkArgs a{(const bf*)q, (const bf*)k, (const bf*)v, (bf*)out, (const int32_t*)block_table, (const int32_t*)cu_q, (const int32_t*)seq_lens,
              (const float*)bias, (const float*)sink, (const float*)talk, (float*)workspace, bt_stride, B, rows, h, hk,
-             page_size, num_pages, reach, window, splits, layer, layers + layer, decode, scale, status};
-  const CUtensorMap& map = *reinterpret_cast<const CUtensorMap*>(kv_map);
-  return d == 64 ? dispatch_talk<64>(map, a, stream) : dispatch_talk<128>(map, a, stream);
+             page_size, num_pages, reach, window, splits, decode, scale, status};
+  return d == 64 ? dispatch_talk<64>(a, stream) : dispatch_talk<128>(a, stream);
 }
 
 MSGL_API int msgl_talk_status(int reset) {

@@ -64,7 +64,7 @@ _SIGNATURES = {
                                    c_f, c_i, c_f, c_p, c_ll, c_i, c_p]),
     "msgl_paged_attention_f32": (c_i, [c_p] * 5 + [c_i, c_p, c_p] + [c_i] * 9 + [c_f, c_f, c_p, c_ll, c_p, c_i, c_p, c_i, c_i,
                                                                               c_p]),
-    "msgl_talk_attention": (c_i, [c_p] * 4 + [c_i] + [c_p] * 3 + [c_i] + [c_p] * 3 + [c_i] * 12 + [c_f, c_p]),
+    "msgl_talk_attention": (c_i, [c_p] * 5 + [c_i] + [c_p] * 3 + [c_i] + [c_p] * 3 + [c_i] * 10 + [c_f, c_p]),
     "msgl_talk_workspace_floats": (c_ll, [c_i] * 5),
     "msgl_talk_status": (c_i, [c_i]),
     "msgl_head_mix": (c_i, [c_p] * 3 + [c_i] * 6 + [c_p]),

@@ -418,14 +418,16 @@ def talk_attention_ok(q, k_cache, chunk=0, softcap=0.0, gate=None) -> bool:
 
 
 def talk_splits(batch: int, heads: int, hk: int, d: int, reach: int) -> int:
-    """Key ranges of a decode step with mixed heads: a CTA per SM, two blocks of 64 keys or more in a range."""
-    groups = -(-hk // (2 if hk <= 2 or (heads > 32 and d == 128) else 4))
-    return int(max(1, min(148 // max(batch * groups, 1), reach // 128, 16)))
+    """Key ranges of a decode step with mixed heads: as many CTAs as fit the SMs, two blocks of 64 keys or more in a range."""
+    mt = 1 if heads <= 16 else 2 if heads <= 32 else 4
+    gn = 2 if hk <= 2 or (mt == 4 and d == 128) else 4
+    room = 148 * (2 if mt * gn * (d // 64) <= 8 else 1)
+    return int(max(1, min(room // max(batch * -(-hk // gn), 1), reach // 128, 16)))
 
 
 def talk_workspace(heads, device):
-    """For the largest split step of layers of ``(heads, kv heads, width)``: rows times ranges stay within 148."""
-    need = max(int(lib().msgl_talk_workspace_floats(148, h, hk, d, 1)) for h, hk, d in heads)
+    """For the largest split step of layers of ``(heads, kv heads, width)``: rows times ranges stay within two per SM."""
+    need = max(int(lib().msgl_talk_workspace_floats(296, h, hk, d, 1)) for h, hk, d in heads)
     return workspace("mixed-head attention partials", need, torch.float32, device)
 
 
@@ -434,17 +436,17 @@ def talk_attention(q, k_cache, v_cache, block_table, cu_q, seq_lens, scale, talk
     """Attention with mixed heads for single query rows: one pass over keys and values for all heads."""
     t, hq, d = q.shape
     pages_p1, hk, ps, _ = k_cache.shape
-    desc, layer, layers = _kv_map(k_cache)
     assert q.is_contiguous() and talk.dtype == torch.float32 and talk.is_contiguous() and talk.shape == (hq, hq)
+    assert k_cache.is_contiguous() and v_cache.is_contiguous() and k_cache.dtype == v_cache.dtype == q.dtype
     if splits > 1:
         need = int(lib().msgl_talk_workspace_floats(t, hq, hk, d, splits))
         if workspace is None or workspace.numel() < need:
             workspace = torch.empty(need, dtype=torch.float32, device=q.device)
     out = torch.empty_like(q)
     check(lib().msgl_talk_attention(
-        desc.ctypes.data, _p(q), _p(out), _p(block_table), block_table.stride(0), _p(cu_q), _p(seq_lens),
+        _p(k_cache), _p(v_cache), _p(q), _p(out), _p(block_table), block_table.stride(0), _p(cu_q), _p(seq_lens),
         *_distance_bias(bias, hq), _p(sink), _p(talk), _p(workspace) if splits > 1 else None, seq_lens.numel(), t, hq, hk, d, ps,
-        pages_p1 - 1, layer, layers, int(window), splits, int(decode), float(scale), _stream()), "talk_attention")
+        pages_p1 - 1, int(window), splits, int(decode), float(scale), _stream()), "talk_attention")
     _count("talk_attention", "talk_decode_kernel", 2 if splits > 1 else 1)
     return out
 

@@ -97,7 +97,7 @@ def weights(cfg, seed=0, sharp=2.0):
     return {k: t.to(torch.bfloat16) for k, t in out.items()}
 
 
-def clear_choices(cfg, path, seqs, margin=0.02):
+def clear_choices(cfg, path, seqs, margin=0.05):
     """The sequences with every token replaced whose choice of experts is a close call in some layer: in 16 bits it could fall
     the other way, and with it the rows after the token."""
     from minisglang_rdna4_b200 import ops
