@@ -232,13 +232,35 @@ __device__ __forceinline__ float2 centre(const float (&u)[NC][V], int width, flo
   return make_float2(mean, 1.f / sqrtf(block_sum(s, scratch) / (float)width + eps));
 }
 
+// two block sums at once; scratch holds 64 floats
+__device__ __forceinline__ float2 block_sum2(float a, float b, float* scratch) {
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = (blockDim.x + 31) >> 5;
+  a = warp_sum(a);
+  b = warp_sum(b);
+  __syncthreads();
+  if (lane == 0) {
+    scratch[warp] = a;
+    scratch[32 + warp] = b;
+  }
+  __syncthreads();
+  return make_float2(warp_sum(lane < nw ? scratch[lane] : 0.f), warp_sum(lane < nw ? scratch[32 + lane] : 0.f));
+}
+
 template <typename T, int V, int NC, bool PAIR>
 __global__ void __launch_bounds__(1024) residual_step_kernel(const StepArgs a) {
   pdl_enter();
-  __shared__ float scratch[32];
+  __shared__ float scratch[64];
   const size_t row = blockIdx.x;
   const int first = threadIdx.x, step = blockDim.x;
-  float u[NC][V];
+  const size_t plane = (size_t)a.rows * a.width, at = row * a.width;
+  float u[NC][V], x[NC][V];
+#pragma unroll
+  for (int g = 0; g < NC; ++g) {
+    const int c = (g * step + first) * V;
+#pragma unroll
+    for (int v = 0; v < V; ++v) x[g][v] = 0.f;
+    if (a.x != nullptr && c < a.width) load_v<V>(a.x + at + c, x[g]);
+  }
   load_planes<V, NC>(a.d[0], a.planes[0], a.plane_stride[0], row * a.ldd[0], a.width, first, step, u);
   if constexpr (PAIR) {
     float e[NC][V];
@@ -251,8 +273,8 @@ __global__ void __launch_bounds__(1024) residual_step_kernel(const StepArgs a) {
         s0 = fmaf(u[g][v], u[g][v], s0);
         s1 = fmaf(e[g][v], e[g][v], s1);
       }
-    const float r0 = 0.5f / sqrtf(block_sum(s0, scratch) / (float)a.width + a.eps);
-    const float r1 = 0.5f / sqrtf(block_sum(s1, scratch) / (float)a.width + a.eps);
+    const float2 ss = block_sum2(s0, s1, scratch);
+    const float r0 = 0.5f / sqrtf(ss.x / (float)a.width + a.eps), r1 = 0.5f / sqrtf(ss.y / (float)a.width + a.eps);
 #pragma unroll
     for (int g = 0; g < NC; ++g) {
       const int c = (g * step + first) * V;
@@ -271,18 +293,13 @@ __global__ void __launch_bounds__(1024) residual_step_kernel(const StepArgs a) {
       for (int v = 0; v < V; ++v) u[g][v] = (u[g][v] - m.x) * m.y * a.post_w[c + v] + a.post_b[c + v];
     }
   }
-  const size_t plane = (size_t)a.rows * a.width, at = row * a.width;
   const float own = a.coef != nullptr ? a.coef[a.n] : 1.f;
 #pragma unroll
   for (int g = 0; g < NC; ++g) {
     const int c = (g * step + first) * V;
     if (c >= a.width) continue;
-    if (a.x != nullptr) {
-      float q[V];
-      load_v<V>(a.x + at + c, q);
 #pragma unroll
-      for (int v = 0; v < V; ++v) u[g][v] += q[v];
-    }
+    for (int v = 0; v < V; ++v) u[g][v] += x[g][v];
     if (a.hist != nullptr) store_v<V>(a.hist + a.n * plane + at + c, u[g]);
 #pragma unroll
     for (int v = 0; v < V; ++v) u[g][v] *= own;
@@ -341,7 +358,7 @@ template <typename T, bool PAIR> int residual_step_typed(const StepArgs& a, cuda
   for (int i = 0; i < (PAIR ? 2 : 1); ++i)
     vec = vec && a.ldd[i] % 4 == 0 && a.plane_stride[i] % 4 == 0 && (uintptr_t)a.d[i] % 16 == 0;
   const int groups = (a.cols + (vec ? 3 : 0)) / (vec ? 4 : 1);
-  const int want = a.rows <= 512 ? 512 : 256;
+  const int want = a.rows <= 512 ? 512 : 128;
   int nc = (groups + want - 1) / want;
   nc = nc <= 1 ? 1 : nc <= 2 ? 2 : nc <= 4 ? 4 : 8;
   const int threads = ((groups + nc - 1) / nc + 31) / 32 * 32;

@@ -56,14 +56,28 @@ struct ConvArgs {
   int channels, taps, num_slots;
 };
 
-// grid (channels / 256, stretches of tokens, B), a channel pair per thread. A stretch reads the taps - 1 rows ahead of it
+// grid (channels / 512, stretches of tokens, B), four channels per thread. A stretch reads the taps - 1 rows ahead of it
 // again. Only the first one touches the tail: it reads the old one and, when its rows are done, writes the new one.
-constexpr int kStretch = 64;
+constexpr int kStretch = 32;
+__device__ __forceinline__ float4 load4f(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 load4f(const __nv_bfloat16* p) {
+  const uint2 q = *reinterpret_cast<const uint2*>(p);
+  const float2 u = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&q.x));
+  const float2 v = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&q.y));
+  return make_float4(u.x, u.y, v.x, v.y);
+}
+__device__ __forceinline__ void store4f(float* p, float4 x) { *reinterpret_cast<float4*>(p) = x; }
+__device__ __forceinline__ void store4f(__nv_bfloat16* p, float4 x) {
+  uint2 q;
+  *reinterpret_cast<__nv_bfloat162*>(&q.x) = __floats2bfloat162_rn(x.x, x.y);
+  *reinterpret_cast<__nv_bfloat162*>(&q.y) = __floats2bfloat162_rn(x.z, x.w);
+  *reinterpret_cast<uint2*>(p) = q;
+}
+
 template <typename T, int TAPS>
 __global__ void __launch_bounds__(128) causal_conv_silu_kernel(const ConvArgs a) {
   pdl_enter();
-  using P2 = typename std::conditional<sizeof(T) == 2, uint32_t, float2>::type;
-  const int c = (blockIdx.x * 128 + threadIdx.x) * 2, b = blockIdx.z;
+  const int c = (blockIdx.x * 128 + threadIdx.x) * 4, b = blockIdx.z;
   if (c >= a.channels) return;
   const int lo = a.cu_q[b], len = a.cu_q[b + 1] - lo;
   const int t0 = blockIdx.y * kStretch, t1 = min(t0 + kStretch, len);
@@ -74,54 +88,49 @@ __global__ void __launch_bounds__(128) causal_conv_silu_kernel(const ConvArgs a)
   const T* x = reinterpret_cast<const T*>(a.x) + lo * a.ldx + c;
   T* out = reinterpret_cast<T*>(a.out) + (size_t)lo * a.channels + c;
   const bool keep = a.has_state[b] != 0;
-  auto load2 = [&](const T* p, float& u, float& v) {
-    union { P2 w; T e[2]; } q;
-    q.w = *reinterpret_cast<const P2*>(p);
-    u = to_float(q.e[0]);
-    v = to_float(q.e[1]);
-  };
-  float w[2][TAPS], h[2][TAPS];           // h[.][TAPS - 1]: the current input
+  float w[TAPS][4];
 #pragma unroll
-  for (int j = 0; j < TAPS; ++j) {
-    w[0][j] = a.w[(size_t)c * TAPS + j];
-    w[1][j] = a.w[(size_t)(c + 1) * TAPS + j];
-  }
-  const float b0 = a.bias[c], b1 = a.bias[c + 1];
+  for (int j = 0; j < TAPS; ++j)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) w[j][e] = a.w[(size_t)(c + e) * TAPS + j];
+  const float4 bias = load4f(a.bias + c);
+  float4 h[TAPS];                         // h[TAPS - 1]: the current input
 #pragma unroll
   for (int j = 0; j < TAPS - 1; ++j) {
-    const int t = t0 - (TAPS - 1) + j;    // the input that h[.][j + 1] is ahead of the first step's shift
-    h[0][j + 1] = h[1][j + 1] = 0.f;
-    if (t >= 0) load2(x + t * a.ldx, h[0][j + 1], h[1][j + 1]);
+    const int t = t0 - (TAPS - 1) + j;    // the input that h[j + 1] is ahead of the first step's shift
+    h[j + 1] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (t >= 0) h[j + 1] = load4f(x + t * a.ldx);
     else if (keep) {
-      h[0][j + 1] = to_float(st[t + TAPS - 1]);
-      h[1][j + 1] = to_float(st[TAPS - 1 + t + TAPS - 1]);
+      const T* s = st + t + TAPS - 1;
+      h[j + 1] = make_float4(to_float(s[0]), to_float(s[TAPS - 1]), to_float(s[2 * (TAPS - 1)]), to_float(s[3 * (TAPS - 1)]));
     }
   }
 #pragma unroll 8
   for (int t = t0; t < t1; ++t) {
-    float acc0 = b0, acc1 = b1;
 #pragma unroll
-    for (int j = 0; j < TAPS - 1; ++j) { h[0][j] = h[0][j + 1]; h[1][j] = h[1][j + 1]; }
-    load2(x + t * a.ldx, h[0][TAPS - 1], h[1][TAPS - 1]);
+    for (int j = 0; j < TAPS - 1; ++j) h[j] = h[j + 1];
+    h[TAPS - 1] = load4f(x + t * a.ldx);
+    float4 acc = bias;
 #pragma unroll
     for (int j = 0; j < TAPS; ++j) {
-      acc0 = fmaf(w[0][j], h[0][j], acc0);
-      acc1 = fmaf(w[1][j], h[1][j], acc1);
+      acc.x = fmaf(w[j][0], h[j].x, acc.x);
+      acc.y = fmaf(w[j][1], h[j].y, acc.y);
+      acc.z = fmaf(w[j][2], h[j].z, acc.z);
+      acc.w = fmaf(w[j][3], h[j].w, acc.w);
     }
-    union { P2 w; T e[2]; } q;
-    q.e[0] = from_float<T>(silu<T>(acc0));
-    q.e[1] = from_float<T>(silu<T>(acc1));
-    *reinterpret_cast<P2*>(out + (size_t)t * a.channels) = q.w;
+    store4f(out + (size_t)t * a.channels, make_float4(silu<T>(acc.x), silu<T>(acc.y), silu<T>(acc.z), silu<T>(acc.w)));
   }
   if (t0 == 0) {
     if (t1 < len) {
 #pragma unroll
-      for (int j = 0; j < TAPS - 1; ++j) load2(x + (len - (TAPS - 1) + j) * a.ldx, h[0][j + 1], h[1][j + 1]);
+      for (int j = 0; j < TAPS - 1; ++j) h[j + 1] = load4f(x + (len - (TAPS - 1) + j) * a.ldx);
     }
 #pragma unroll
     for (int j = 0; j < TAPS - 1; ++j) {
-      st[j] = from_float<T>(h[0][j + 1]);
-      st[TAPS - 1 + j] = from_float<T>(h[1][j + 1]);
+      st[j] = from_float<T>(h[j + 1].x);
+      st[TAPS - 1 + j] = from_float<T>(h[j + 1].y);
+      st[2 * (TAPS - 1) + j] = from_float<T>(h[j + 1].z);
+      st[3 * (TAPS - 1) + j] = from_float<T>(h[j + 1].w);
     }
   }
 }
@@ -168,29 +177,54 @@ struct ScanArgs {
   int channels, N, num_slots;
 };
 
-template <typename T> __device__ __forceinline__ float4 load4f(const T* p);
-template <> __device__ __forceinline__ float4 load4f<float>(const float* p) { return *reinterpret_cast<const float4*>(p); }
-template <> __device__ __forceinline__ float4 load4f<__nv_bfloat16>(const __nv_bfloat16* p) {
-  const uint2 q = *reinterpret_cast<const uint2*>(p);
-  const float2 u = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&q.x));
-  const float2 v = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&q.y));
-  return make_float4(u.x, u.y, v.x, v.y);
+// two fp32 operations per instruction
+__device__ __forceinline__ uint64_t f2(float a, float b) {
+  uint64_t r;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
+  return r;
+}
+__device__ __forceinline__ float2 unf2(uint64_t x) {
+  float2 r;
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(r.x), "=f"(r.y) : "l"(x));
+  return r;
+}
+__device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b) {
+  uint64_t r;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+  return r;
+}
+__device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
+  uint64_t r;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+  return r;
+}
+struct Four { uint64_t lo, hi; };
+__device__ __forceinline__ Four four(float4 x) { return {f2(x.x, x.y), f2(x.z, x.w)}; }
+__device__ __forceinline__ float4 unfour(Four x) {
+  const float2 a = unf2(x.lo), b = unf2(x.hi);
+  return make_float4(a.x, a.y, b.x, b.y);
+}
+template <typename T> __device__ __forceinline__ uint64_t decay2(uint64_t dta) {
+  const float2 x = unf2(dta);
+  return f2(decay<T>(x.x), decay<T>(x.y));
 }
 
 // One step of the states a lane owns (4 G of them): returns its part of y.
 template <typename T, int G>
-__device__ __forceinline__ float advance(float4 (&s)[G], const float4 (&A)[G], const float4 (&B)[G], const float4 (&C)[G],
+__device__ __forceinline__ float advance(Four (&s)[G], const Four (&A)[G], const float4 (&B)[G], const float4 (&C)[G],
                                          float dt, float dtx) {
-  float y = 0.f;
+  const uint64_t dt2 = f2(dt, dt), dtx2 = f2(dtx, dtx);
+  uint64_t y = 0;
 #pragma unroll
   for (int g = 0; g < G; ++g) {
-    s[g].x = fmaf(s[g].x, decay<T>(dt * A[g].x), dtx * B[g].x);
-    s[g].y = fmaf(s[g].y, decay<T>(dt * A[g].y), dtx * B[g].y);
-    s[g].z = fmaf(s[g].z, decay<T>(dt * A[g].z), dtx * B[g].z);
-    s[g].w = fmaf(s[g].w, decay<T>(dt * A[g].w), dtx * B[g].w);
-    y = fmaf(s[g].x, C[g].x, fmaf(s[g].y, C[g].y, fmaf(s[g].z, C[g].z, fmaf(s[g].w, C[g].w, y))));
+    const Four b = four(B[g]), c = four(C[g]);
+    s[g].lo = fma2(s[g].lo, decay2<T>(mul2(dt2, A[g].lo)), mul2(dtx2, b.lo));
+    s[g].hi = fma2(s[g].hi, decay2<T>(mul2(dt2, A[g].hi)), mul2(dtx2, b.hi));
+    y = g == 0 ? mul2(s[g].lo, c.lo) : fma2(s[g].lo, c.lo, y);
+    y = fma2(s[g].hi, c.hi, y);
   }
-  return y;
+  const float2 r = unf2(y);
+  return r.x + r.y;
 }
 
 // grid (channels * LN / 128, B)
@@ -207,13 +241,14 @@ __global__ void __launch_bounds__(128) scan_rows_kernel(const ScanArgs a) {
   float* S = a.state + slot * a.slot_stride + (size_t)ch * a.N;
   const bool keep = a.has_state[b] != 0;
   const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
-  float4 s[G], A[G];
+  Four s[G], A[G];
 #pragma unroll
   for (int g = 0; g < G; ++g) {
     const int n = (g * LN + ln) * 4;
-    s[g] = keep && n < a.N ? *reinterpret_cast<const float4*>(S + n) : zero;
-    A[g] = n < a.N ? *reinterpret_cast<const float4*>(a.A + (size_t)ch * a.N + n) : zero;
-    A[g].x *= kAUnit<T>; A[g].y *= kAUnit<T>; A[g].z *= kAUnit<T>; A[g].w *= kAUnit<T>;
+    s[g] = four(keep && n < a.N ? *reinterpret_cast<const float4*>(S + n) : zero);
+    float4 x = n < a.N ? *reinterpret_cast<const float4*>(a.A + (size_t)ch * a.N + n) : zero;
+    x.x *= kAUnit<T>; x.y *= kAUnit<T>; x.z *= kAUnit<T>; x.w *= kAUnit<T>;
+    A[g] = four(x);
   }
   const float bias = a.dt_bias[ch], skip = a.skip[ch];
   for (int t = lo; t < hi; ++t) {
@@ -237,7 +272,7 @@ __global__ void __launch_bounds__(128) scan_rows_kernel(const ScanArgs a) {
 #pragma unroll
   for (int g = 0; g < G; ++g) {
     const int n = (g * LN + ln) * 4;
-    if (live && n < a.N) *reinterpret_cast<float4*>(S + n) = s[g];
+    if (live && n < a.N) *reinterpret_cast<float4*>(S + n) = unfour(s[g]);
   }
 }
 
@@ -279,8 +314,10 @@ template <int LN, int G> struct TileSmem {
   static constexpr int raw = off_bc + kTile * 2 * NP * 2;
   static constexpr int off_step = 2 * raw;                    // (dt, dt x) [tile][CH]
   static constexpr int off_b = off_step + kTile * CH * 8;     // B and C in fp32 [tile][2][NP]
-  static constexpr int off_y = off_b + kTile * 2 * NP * 4;    // [tile][CH]
-  static constexpr int bytes = off_y + kTile * CH * 4;
+  // [tile][CH], rows apart so that the tokens that a warp stores at once lie on different banks
+  static constexpr int LDY = CH + 32 / LN;
+  static constexpr int off_y = off_b + kTile * 2 * NP * 4;
+  static constexpr int bytes = off_y + kTile * LDY * 4;
 };
 
 // grid (channels / CH, B), 128 threads. Per tile: softplus and products of all (token, channel) pairs; the recurrence, LN
@@ -331,13 +368,14 @@ __global__ void __launch_bounds__(128) scan_tiles_kernel(const ScanArgs a) {
   const bool live = c < a.channels, keep = a.has_state[b] != 0;
   float* S = a.state + slot * a.slot_stride + (size_t)(live ? c : 0) * a.N;
   const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
-  float4 s[G], A[G];
+  Four s[G], A[G];
 #pragma unroll
   for (int g = 0; g < G; ++g) {
     const int n = (g * LN + ln) * 4;
-    s[g] = keep && live && n < a.N ? *reinterpret_cast<const float4*>(S + n) : zero;
-    A[g] = live && n < a.N ? *reinterpret_cast<const float4*>(a.A + (size_t)c * a.N + n) : zero;
-    A[g].x *= kLog2e; A[g].y *= kLog2e; A[g].z *= kLog2e; A[g].w *= kLog2e;
+    s[g] = four(keep && live && n < a.N ? *reinterpret_cast<const float4*>(S + n) : zero);
+    float4 x = live && n < a.N ? *reinterpret_cast<const float4*>(a.A + (size_t)c * a.N + n) : zero;
+    x.x *= kLog2e; x.y *= kLog2e; x.z *= kLog2e; x.w *= kLog2e;
+    A[g] = four(x);
   }
   // the channel that this thread takes ahead of and behind the recurrence
   constexpr int ROWS = 128 / CH;             // tokens side by side
@@ -381,20 +419,20 @@ __global__ void __launch_bounds__(128) scan_tiles_kernel(const ScanArgs a) {
       // sums over the lanes of a channel; every exchange halves the tokens a lane is left with
       if constexpr (LN == 1) {
 #pragma unroll
-        for (int k = 0; k < 4; ++k) ys[(t + k) * CH + cl] = y[k];
+        for (int k = 0; k < 4; ++k) ys[(t + k) * L::LDY + cl] = y[k];
       } else {
         const bool up = ln & 1;
         const float v0 = (up ? y[2] : y[0]) + __shfl_xor_sync(0xffffffffu, up ? y[0] : y[2], 1);
         const float v1 = (up ? y[3] : y[1]) + __shfl_xor_sync(0xffffffffu, up ? y[1] : y[3], 1);
         if constexpr (LN == 2) {
-          ys[(t + 2 * up) * CH + cl] = v0;
-          ys[(t + 2 * up + 1) * CH + cl] = v1;
+          ys[(t + 2 * up) * L::LDY + cl] = v0;
+          ys[(t + 2 * up + 1) * L::LDY + cl] = v1;
         } else {
           const bool up2 = ln & 2;
           float w = (up2 ? v1 : v0) + __shfl_xor_sync(0xffffffffu, up2 ? v0 : v1, 2);
 #pragma unroll
           for (int m = 4; m < LN; m <<= 1) w += __shfl_xor_sync(0xffffffffu, w, m);
-          if (ln < 4) ys[(t + 2 * up + up2) * CH + cl] = w;
+          if (ln < 4) ys[(t + 2 * up + up2) * L::LDY + cl] = w;
         }
       }
     }
@@ -403,14 +441,14 @@ __global__ void __launch_bounds__(128) scan_tiles_kernel(const ScanArgs a) {
       bf* out = reinterpret_cast<bf*>(a.out) + (size_t)(lo + t0) * a.channels + c_first + pc;
 #pragma unroll 4
       for (int t = pt; t < n; t += ROWS)
-        out[(size_t)t * a.channels] = __float2bfloat16(fmaf(skip, to_float(xs[t * CH + pc]), ys[t * CH + pc]) *
+        out[(size_t)t * a.channels] = __float2bfloat16(fmaf(skip, to_float(xs[t * CH + pc]), ys[t * L::LDY + pc]) *
                                                        silu<bf>(to_float(zs[t * CH + pc])));
     }
   }
 #pragma unroll
   for (int g = 0; g < G; ++g) {
     const int n = (g * LN + ln) * 4;
-    if (live && n < a.N) *reinterpret_cast<float4*>(S + n) = s[g];
+    if (live && n < a.N) *reinterpret_cast<float4*>(S + n) = unfour(s[g]);
   }
 }
 
@@ -439,18 +477,18 @@ int launch_tiles(const ScanArgs& a, int B, cudaStream_t s) {
 
 }  // namespace
 
-// x [T, channels] with row stride ldx (channels even); out [T, channels]
+// x [T, channels] with row stride ldx (channels a multiple of 4); out [T, channels]
 MSGL_API int msgl_causal_conv_silu(const void* x, long long ldx, const void* w, const void* bias, void* state,
                                    long long slot_stride, const void* cu_q, const void* slots, const void* has_state,
                                    void* out, int B, int channels, int taps, int max_q, int num_slots, int dtype,
                                    cudaStream_t stream) {
   if (B <= 0) return B == 0 ? MSGL_OK : MSGL_BAD_ARG;
-  if (channels <= 0 || channels % 2 || taps <= 0 || max_q <= 0 || B > 65535 || ldx % 2 || (uintptr_t)x % 8 ||
-      (uintptr_t)out % 8)
+  if (channels <= 0 || channels % 4 || taps <= 0 || max_q <= 0 || B > 65535 || ldx % 4 || (uintptr_t)x % 16 ||
+      (uintptr_t)out % 16 || (uintptr_t)bias % 16)
     return MSGL_BAD_ARG;
   const ConvArgs a{x, ldx, (const float*)w, (const float*)bias, state, slot_stride, (const int32_t*)cu_q,
                    (const int32_t*)slots, (const int32_t*)has_state, out, channels, taps, num_slots};
-  const dim3 grid((channels + 255) / 256, (max_q + kStretch - 1) / kStretch, B);
+  const dim3 grid((channels + 511) / 512, (max_q + kStretch - 1) / kStretch, B);
 #define CONV(T)                                                                                          \
   do {                                                                                                   \
     if (taps == 1) msgl_launch(causal_conv_silu_kernel<T, 1>, grid, dim3(128), 0, stream, a);            \

@@ -235,7 +235,8 @@ def test_a_loud_key_is_seen_exactly_within_the_window(at, window):
 
 
 # ---------------------------------------------------------------------------------- engine
-LIMITS = {"float32": 2e-4, "bfloat16": 0.1}
+# (limit, cap): in 16 bits the norm of a mixer's output enlarges the rounding of a row whose mixed heads nearly cancel
+LIMITS = {"float32": (2e-4, None), "bfloat16": (0.05, 0.2)}
 LONG = U.config([
     U.pair(4, 2, 40, 64, 90, inner=96, state=16, rank=16, taps=4, mlp=U.moe(8, 2, 48, shared=64)),
     U.retention(2, 64, 64, base=1e4, decay=[0.9, 0.999], mlp=U.moe(4, 2, 32)),
@@ -256,16 +257,16 @@ def model(request, tmp_path_factory):
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 def test_engine_portions_batches_and_reuse(model, dtype):
     cfg, w, path, seqs, want = model
-    limit = LIMITS[dtype]
+    limit, cap = LIMITS[dtype]
     rep = make_replayer(path, dtype, 896, "cuda")
     for sizes in ([1000], [100, 1, 2, 63], [2, 65]):
         for name in seqs:
-            U.play(rep, seqs, [[(name, n)] for n in U.cuts(len(seqs[name]), sizes)], want, limit)
+            U.play(rep, seqs, [[(name, n)] for n in U.cuts(len(seqs[name]), sizes)], want, limit, cap)
     # decoding alone (captured graphs) after most of the prompt
     n = len(seqs["c"]) - 24
-    U.play(rep, seqs, [[("c", n)]] + [[("c", 1)]] * 24, want, limit)
+    U.play(rep, seqs, [[("c", n)]] + [[("c", 1)]] * 24, want, limit, cap)
     # everyone together, then mixed portions and single tokens with slots and pages taken again
-    U.play(rep, seqs, [[(n, len(s)) for n, s in seqs.items()]], want, limit)
+    U.play(rep, seqs, [[(n, len(s)) for n, s in seqs.items()]], want, limit, cap)
     at = {n: 0 for n in seqs}
     plan, k = [], 0
     while any(at[n] < len(seqs[n]) for n in seqs):
@@ -279,7 +280,7 @@ def test_engine_portions_batches_and_reuse(model, dtype):
         k += 1
         if step:
             plan.append(step)
-    U.play(rep, seqs, plan, want, limit)
+    U.play(rep, seqs, plan, want, limit, cap)
     assert rep.engine.graph_runner is None or rep.engine.graph_runner.replays > 0
     rep.engine.shutdown()
 
@@ -299,7 +300,7 @@ def test_engine_other_sizes(cfg, dtype, tmp_path):
     seqs = {"a": U.tokens(cfg, 90, 1), "b": U.tokens(cfg, 3, 2)}
     rep = make_replayer(path, dtype, 256, "cuda")
     steps = [[("a", 70)], [("a", 1), ("b", 2)], [("a", 1), ("b", 1)], [("a", 2)], [("a", 1)], [("a", 1)], [("a", 14)]]
-    U.play(rep, seqs, steps, U.reference(cfg, w, seqs), LIMITS[dtype])
+    U.play(rep, seqs, steps, U.reference(cfg, w, seqs), *LIMITS[dtype])
     rep.engine.shutdown()
 
 
@@ -331,7 +332,7 @@ def test_long_decoding_follows_the_graphs(tmp_path):
     w = U.weights(cfg, 4)
     rep = make_replayer(U.save(tmp_path, cfg, w), "float32", 320, "cuda")
     seqs = {"a": U.tokens(cfg, 300, 9)}
-    U.play(rep, seqs, [[("a", 5)]] + [[("a", 1)]] * 295, U.reference(cfg, w, seqs), LIMITS["float32"])
+    U.play(rep, seqs, [[("a", 5)]] + [[("a", 1)]] * 295, U.reference(cfg, w, seqs), *LIMITS["float32"])
     rep.engine.shutdown()
 
 
