@@ -176,7 +176,7 @@ def kernels(s: Dict) -> List[Dict]:
             lambda: ops.norm_gate(o, lin[:, 2 * rh * rd + rh * rv:], gw, 1e-5, rv, False, "silu", rh * rv), t * rh * rv * 6)
         # ---- feed-forward
         hx, logits = rnd(t, w), rnd(t, e, dtype=f32)
-        counts, corr = torch.empty(e, dtype=torch.int32, device=dev), rnd(e, dtype=f32)
+        counts, corr = torch.empty(e, dtype=torch.int32, device=dev), rnd(e, dtype=f32) * 0.01
         add("ligipel", "routing", phase, lambda: M.moe_route(logits, top, True, "softmax", 1.0, counts, bias=corr),
             t * (e * 4 + top * 8))
         lb = rnd(t, e)

@@ -1012,8 +1012,8 @@ def _ligipel_config(cfg: Dict[str, Any]) -> ModelConfig:
     eos = cfg.get("eos_token_id")
     eos_ids = tuple(eos) if isinstance(eos, (list, tuple)) else (() if eos is None else (int(eos),))
     return pair_config(specs, width=int(cfg["width"]), vocab=int(cfg["vocab"]), eps=float(cfg["norm"]["eps"]),
-                       logit_scale=float(cfg["logit_scale"]), logit_softcap=float(cfg["logit_softcap"]), max_positions=max_pos,
-                       eos_token_ids=eos_ids, bos_token_id=cfg.get("bos_token_id"))
+                       logit_scale=float(cfg.get("logit_scale") or 1.0), logit_softcap=float(cfg.get("logit_softcap") or 0.0),
+                       max_positions=max_pos, eos_token_ids=eos_ids, bos_token_id=cfg.get("bos_token_id"))
 
 
 def pair_config(specs, width: int, vocab: int, eps: float, logit_scale: float = 1.0, logit_softcap: float = 0.0,
